@@ -329,6 +329,8 @@ class ExecutionPlan:
 def decoder_step_operators(cfg, rows: int, tp_size: int = 1, topology_id: str = "single") -> tuple[OpSignature, ...]:
     """Operator signatures of one decode step of a decoder (the shapes the graphs of capacity ``rows`` were captured
     with): what ``cubic qualify`` and the readiness seal identify a captured step by."""
+    if getattr(cfg, "family", "") == "layered":
+        return layered_step_operators(cfg, rows, topology_id)
     H, D = cfg.hidden_size, cfg.head_dim
     from ..models.config import kv_heads_of_rank
     hq, hkv = cfg.num_q_heads // tp_size, kv_heads_of_rank(cfg.num_kv_heads, 0, tp_size)[1]
@@ -356,3 +358,31 @@ def decoder_step_operators(cfg, rows: int, tp_size: int = 1, topology_id: str = 
         ops += [linear("gate_up", 2 * inter, H), linear("down", H, inter)]
     ops.append(linear("lm_head", cfg.vocab_size // tp_size, H))
     return tuple(ops)
+
+
+def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple[OpSignature, ...]:
+    """Operator signatures of one decode step of a layered decoder: the distinct operators of its layer runs."""
+    from ..models.layered import LatentSpec
+    W, act = cfg.hidden_size, "fp32" if cfg.dtype == "float32" else "bf16"
+    ops: dict[tuple, OpSignature] = {}
+
+    def add(op, layout, n, k, **shape):
+        shape = {"k": k, "m": rows, "n": n, **shape}
+        key = (op, layout, tuple(sorted(shape.items())))
+        if key not in ops:
+            ops[key] = OpSignature(op, BatchPhase.DECODE, (TensorSpec("x", act, ("m", k)),), (TensorSpec("y", act, ("m", n)),),
+                                   "fp32", layout, tuple(sorted(shape.items())), topology_id)
+
+    add("norm.rms", "residual32", W, W)
+    if cfg.loop is not None:
+        add("linear.bf16", "loop_entry", W, 2 * W)
+    for i, _ in cfg.runs:
+        l, m = cfg.layers[i], cfg.layers[i].mixer
+        if isinstance(m, LatentSpec):
+            add("attention.latent", "paged", m.out_width, m.q_rank + m.kv_rank, heads=m.heads, window=m.window or cfg.max_position)
+        else:
+            add("delta_rule." + ("channel" if m.per_channel else "head"), "state32", m.out_width, m.channels, heads=m.heads,
+                taps=m.conv)
+        add("linear.bf16", "parallel_out", W, m.out_width + l.ff)
+    add("linear.bf16", "lm_head", cfg.vocab_size, W)
+    return tuple(ops.values())

@@ -57,6 +57,7 @@ __device__ __forceinline__ float philox_uniform(unsigned long long seed, unsigne
 
 struct SampleParams {
   const __nv_bfloat16* logits;  // [rows, ld]
+  const float* logits32;        // [rows, ld] instead of `logits` when set (models that run in 32-bit)
   const uint32_t* mask;         // [rows, mask_words] allowed-token bits or null
   const float* temperature;     // [rows] 0 = greedy
   const float* top_p;           // [rows]
@@ -110,6 +111,7 @@ sample_kernel(const SampleParams p) {
   pdl_wait();
   pdl_launch_dependents();
   const __nv_bfloat16* lg = p.logits + static_cast<size_t>(row) * p.ld;
+  const float* lg32 = p.logits32 ? p.logits32 + static_cast<size_t>(row) * p.ld : nullptr;
   const uint32_t* mk = p.mask ? p.mask + static_cast<size_t>(row) * p.mask_words : nullptr;
   const float temp = p.temperature ? p.temperature[row] : 0.f;
   int K = 1;
@@ -123,7 +125,7 @@ sample_kernel(const SampleParams p) {
     Cand best{-INFINITY, 0x7fffffff};
     for (int i = threadIdx.x; i < p.vocab; i += kSampleThreads) {
       if (mk && !((mk[i >> 5] >> (i & 31)) & 1u)) continue;
-      float v = __bfloat162float(lg[i]);
+      float v = lg32 ? lg32[i] : __bfloat162float(lg[i]);
       if (!(v == v)) v = -INFINITY;  // NaN never wins
       // strictly after the previous pick in (value desc, id asc) order
       if (v < pv || (v == pv && i > pi)) {
@@ -390,13 +392,15 @@ reasoning_budget_kernel(int* __restrict__ ids, const int* __restrict__ row_slot,
 
 extern "C" {
 
-int cb_sample(const void* logits, int ld, const void* mask, int mask_words, const void* temperature,
+// `f32`: the logits are fp32 instead of bf16.
+int cb_sample(const void* logits, int f32, int ld, const void* mask, int mask_words, const void* temperature,
               const void* top_p, const void* top_k, const void* seeds, const void* counters, void* out_ids,
               void* out_logprob, void* out_value, int id_offset, int rows, int vocab, void* stream) {
   using namespace cb;
   if (rows <= 0) return 0;
   SampleParams p;
-  p.logits = static_cast<const __nv_bfloat16*>(logits);
+  p.logits = f32 ? nullptr : static_cast<const __nv_bfloat16*>(logits);
+  p.logits32 = f32 ? static_cast<const float*>(logits) : nullptr;
   p.mask = static_cast<const uint32_t*>(mask);
   p.temperature = static_cast<const float*>(temperature);
   p.top_p = static_cast<const float*>(top_p);

@@ -144,9 +144,10 @@ wq_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
           bulk_g2s(smem_u32(st + x_bytes + kATileBytes + kCodeBytes), msrc, kMeta, bar);
         }
       };
+      const int x_col0 = p.diag_n ? (n_tile * kTileN / p.diag_n) * p.K : 0;
       auto load_x = [&](int i, int s) {
         uint8_t* st = smem + static_cast<size_t>(s) * stage_bytes;
-        tma_load_2d(smem_u32(st), &tmap_x, (kb_lo + i) * kBK, m0, smem_u32(&ctl->full[s]));
+        tma_load_2d(smem_u32(st), &tmap_x, x_col0 + (kb_lo + i) * kBK, m0, smem_u32(&ctl->full[s]));
       };
       // weights of the first S stages go out before anything else, so that an
       // all-gather still in flight overlaps with weight streaming
@@ -441,6 +442,12 @@ wq_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
           const float4 f0 = *reinterpret_cast<const float4*>(stg + mm * kTileN + (idx & 15) * 8);
           const float4 f1 = *reinterpret_cast<const float4*>(stg + mm * kTileN + (idx & 15) * 8 + 4);
           float v[8] = {f0.x, f0.y, f0.z, f0.w, f1.x, f1.y, f1.z, f1.w};
+          if (FMT == kFmtBf16 && p.wide) {
+            float lo[4] = {v[0], v[1], v[2], v[3]}, hi[4] = {v[4], v[5], v[6], v[7]};
+            store_wide4(p, m, n0, lo);
+            store_wide4(p, m, n0 + 4, hi);
+            continue;
+          }
           if (vec_ok && n0 + 7 < p.N) {
             __nv_bfloat16* dst;
             if (p.tp.mode & kTpScatterPush) {
@@ -549,7 +556,10 @@ wq_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
           }
           const int m = m0 + mm;
           const float o4[4] = {acc.x, acc.y, acc.z, acc.w};
-          if ((p.tp.mode & kTpScatterPush) && n_base + c4 + 3 < p.N && ((p.N & 3) == 0)) {
+          if (FMT == kFmtBf16 && p.wide) {
+            float v[4] = {acc.x * p.alpha, acc.y * p.alpha, acc.z * p.alpha, acc.w * p.alpha};
+            store_wide4(p, m, n_base + c4, v);
+          } else if ((p.tp.mode & kTpScatterPush) && n_base + c4 + 3 < p.N && ((p.N & 3) == 0)) {
             const int o = m / p.tp.rows_per_rank;
             const int lr = m - o * p.tp.rows_per_rank;
             uint2 ov;
@@ -619,7 +629,11 @@ wq_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
             const float4 v = ld_cluster_f4(cluster_map(stg0, static_cast<uint32_t>(sp)) + off);
             acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
           }
-          const float o4[4] = {acc.x * p.alpha, acc.y * p.alpha, acc.z * p.alpha, acc.w * p.alpha};
+          float o4[4] = {acc.x * p.alpha, acc.y * p.alpha, acc.z * p.alpha, acc.w * p.alpha};
+          if (FMT == kFmtBf16 && p.wide) {
+            store_wide4(p, m0 + mm, n_base + c4, o4);
+            continue;
+          }
           if (p.tp.mode & kTpScatterPush) {
             // partial rows go straight to the receive buffer of the rank that owns them (slot = this rank)
             const int m = m0 + mm;
@@ -757,6 +771,21 @@ static int launch_fmt(const CUtensorMap& tx, const CUtensorMap& tw, WqGemmParams
 
 }  // namespace cb
 
+// Operands of a bf16 GEMM with the wide epilogue (cb_bf16_gemm_wide).
+struct CbWideGemm {
+  const void* x;              // bf16 [M, ldx], x_cols columns are readable
+  int ldx, x_cols;
+  const void* w;              // bf16 [N, K], K a multiple of 64
+  void* y;                    // bf16 [M, ldy] or null
+  void* y32;                  // fp32 [M, ldy] or null
+  int ldy;
+  const void* residual32;     // fp32 [M, ldy] or null
+  void* y2;                   // bf16 [M, ldy2] or null
+  int ldy2, n_split, diag_n;
+  int M, N, K;
+  int stream_k, splits, min_units;
+};
+
 // Per-launch options of the common launcher.  Everything that steers ONE launch travels in this struct (not in
 // process-wide variables), so launches made concurrently from several host threads cannot see each other's choices.
 struct WqLaunchOpts {
@@ -770,6 +799,7 @@ struct WqLaunchOpts {
   bool stream_k = false;
   int min_units = 0;
   long long workspace_bytes = 0;
+  const struct CbWideGemm* wide = nullptr;   // bf16 weights: wide epilogue and block-diagonal weights
 };
 
 #ifdef CB_KERNEL_TRACE
@@ -901,6 +931,19 @@ static int wq_gemm_dispatch(int fmt, const void* x, int ldx, const void* codes, 
   p.status = static_cast<uint32_t*>(status);
   p.M = M; p.N = N; p.K = K; p.ldy = ldy; p.alpha = alpha;
   p.swiglu = o.swiglu;
+  uint64_t x_cols = static_cast<uint64_t>(K);
+  if (o.wide) {
+    const CbWideGemm& g = *o.wide;
+    if (fmt != kFmtBf16 || residual || link || o.swiglu || o.tiles || g.x_cols <= 0 || g.x_cols > ldx) return -61;
+    if ((!g.y && !g.y32) || (g.y && g.y32) || (g.y2 && (g.y32 || (g.n_split & 3) || g.n_split < 0))) return -62;
+    if (g.diag_n && (stream_k || g.diag_n < 0 || (g.diag_n % kTileN) != 0)) return -63;
+    p.wide = 1;
+    p.y32 = static_cast<float*>(g.y32);
+    p.residual32 = static_cast<const float*>(g.residual32);
+    p.y2 = static_cast<__nv_bfloat16*>(g.y2);
+    p.ldy2 = g.ldy2; p.n_split = g.n_split; p.diag_n = g.diag_n;
+    x_cols = static_cast<uint64_t>(g.x_cols);
+  }
   if (p.swiglu && (residual || (link && (link->mode & kTpScatterPush)))) return -51;
   p.tp.mode = kTpNone;
   if (link && link->mode != kTpNone) {
@@ -953,7 +996,7 @@ static int wq_gemm_dispatch(int fmt, const void* x, int ldx, const void* codes, 
     const uint64_t w_rows = static_cast<uint64_t>(N) * (o.tiles ? o.num_experts : 1);
     if (make_tmap_u8(&tx, x, M, K, ldx, p.pair ? p.mb / 2 : p.mb) != 0) return -20;
     if (make_tmap_u8(&tw, codes, w_rows, K, K, kTileN) != 0) return -21;
-  } else if (make_tmap_bf16(&tx, x, M, K, ldx, p.pair ? p.mb / 2 : p.mb) != 0) {
+  } else if (make_tmap_bf16(&tx, x, M, x_cols, ldx, p.pair ? p.mb / 2 : p.mb) != 0) {
     return -20;
   } else if (fmt == kFmtBf16) {
     const uint64_t w_rows = static_cast<uint64_t>(N) * (o.tiles ? o.num_experts : 1);
@@ -990,6 +1033,20 @@ static int wq_gemm_dispatch(int fmt, const void* x, int ldx, const void* codes, 
     case kFmtFp8Block: return launch_fmt<kFmtFp8Block>(tx, tw, p, grid, smem, st);
     default: return launch_fmt<kFmtBf16>(tx, tw, p, grid, smem, st);
   }
+}
+
+// y = x W^T in bf16 with fp32 accumulation, written through the wide epilogue (see WqGemmParams::wide): fp32 output added
+// to an fp32 residual, or a second output behind the squared relu.  `diag_n`: block-diagonal weights.
+int cb_bf16_gemm_wide(const CbWideGemm* g, void* workspace, long long workspace_bytes, void* counters, void* status,
+                      void* stream) {
+  if (!g) return -60;
+  WqLaunchOpts o;
+  o.wide = g;
+  o.stream_k = g->stream_k != 0;
+  o.min_units = g->min_units;
+  o.workspace_bytes = workspace_bytes;
+  return wq_gemm_dispatch(cb::kFmtBf16, g->x, g->ldx, g->w, nullptr, g->y, g->ldy, nullptr, 1.f, g->M, g->N, g->K, g->K,
+                          o.stream_k ? 1 : g->splits, workspace, counters, status, stream, nullptr, o);
 }
 
 static std::atomic<int> g_grouped_persistent{1};

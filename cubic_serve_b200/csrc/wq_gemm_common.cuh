@@ -96,6 +96,16 @@ struct WqGemmParams {
   // per-tile kernel with K splits: the `splits` CTAs of a tile form a thread-block cluster and sum their fp32 partial
   // tiles through distributed shared memory (no workspace, no fences, no arrival counter)
   int cluster_splitk;
+  // wide epilogue (store_wide4): results leave as fp32, added to an fp32 residual stream, or the features from n_split on
+  // leave through the squared relu into a second buffer (a projection whose rows are [mixer inputs | feed-forward up])
+  int wide;
+  float* y32;               // fp32 [M, ldy] instead of y
+  const float* residual32;  // added to y32 (may be y32 itself)
+  __nv_bfloat16* y2;        // [M, ldy2]: feature n >= n_split goes to y2[m, n - n_split]
+  int ldy2, n_split;        // n_split is a multiple of 4
+  // block-diagonal weights (per-tile kernel): weight rows [g diag_n, (g + 1) diag_n) multiply x columns [g K, (g + 1) K);
+  // diag_n is a multiple of the 128-row tile, 0 = an ordinary matrix
+  int diag_n;
   // persistent stream-K kernel only (wq_gemm_sk.cu)
   int n_tiles, tiles;       // tile = m_tile * n_tiles + n_tile
   int sk_tiles, sk_ctas;    // tiles [0, sk_tiles) are dealt by k-block to CTAs [0, sk_ctas); the rest are whole
@@ -175,6 +185,52 @@ __device__ __forceinline__ void store_act4(const WqGemmParams& p, int m, int n_t
 #pragma unroll
     for (int j = 0; j < 4; ++j)
       if (n0 + j < n_out) dst[j] = __float2bfloat16(a[j]);
+  }
+}
+// Four consecutive output features n0..n0+3 (n0 % 4 == 0) of row m, already scaled, through the wide epilogue.
+__device__ __forceinline__ void store_wide4(const WqGemmParams& p, int m, int n0, float (&v)[4]) {
+  if (n0 >= p.N) return;
+  const bool whole = n0 + 3 < p.N;
+  if (p.y32) {
+    const size_t off = static_cast<size_t>(m) * p.ldy + n0;
+    if (whole && (p.ldy & 3) == 0) {
+      float4 o = make_float4(v[0], v[1], v[2], v[3]);
+      if (p.residual32) {
+        const float4 r = *reinterpret_cast<const float4*>(p.residual32 + off);
+        o.x += r.x; o.y += r.y; o.z += r.z; o.w += r.w;
+      }
+      *reinterpret_cast<float4*>(p.y32 + off) = o;
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (n0 + j < p.N) p.y32[off + j] = v[j] + (p.residual32 ? p.residual32[off + j] : 0.f);
+    }
+    return;
+  }
+  __nv_bfloat16* dst;
+  bool vec;
+  if (p.y2 && n0 >= p.n_split) {
+    // the projection is rounded to bf16 before the activation, as a separate activation kernel would read it
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float u = fmaxf(__bfloat162float(__float2bfloat16(v[j])), 0.f);
+      v[j] = u * u;
+    }
+    dst = p.y2 + static_cast<size_t>(m) * p.ldy2 + (n0 - p.n_split);
+    vec = (p.ldy2 & 3) == 0;
+  } else {
+    dst = p.y + static_cast<size_t>(m) * p.ldy + n0;
+    vec = (p.ldy & 3) == 0;
+  }
+  if (whole && vec) {
+    uint2 ov;
+    ov.x = pack_bf16x2(v[0], v[1]);
+    ov.y = pack_bf16x2(v[2], v[3]);
+    *reinterpret_cast<uint2*>(dst) = ov;
+  } else {
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (n0 + j < p.N) dst[j] = __float2bfloat16(v[j]);
   }
 }
 // offset of activation feature j (0..63) of a tile inside a 128-float tile row: gate value there, up value 16 on

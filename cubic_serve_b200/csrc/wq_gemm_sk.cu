@@ -181,9 +181,16 @@ __device__ __forceinline__ void tail_bar() {
 
 // Four consecutive output features n0..n0+3 of row m from unscaled fp32 accumulators: scale, add the residual,
 // round once to bf16, store locally or (scatter-push) into the receive buffer of the rank that owns row m.
+template <int FMT>
 __device__ __forceinline__ void sk_store4(const WqGemmParams& p, int m, int n0, const float4 v) {
   if (n0 >= p.N) return;
   float o4[4] = {v.x * p.alpha, v.y * p.alpha, v.z * p.alpha, v.w * p.alpha};
+  if constexpr (FMT == kFmtBf16) {
+    if (p.wide) {
+      store_wide4(p, m, n0, o4);
+      return;
+    }
+  }
   __nv_bfloat16* dst;
   const __nv_bfloat16* res = nullptr;
   bool vec;
@@ -282,7 +289,7 @@ __device__ __noinline__ void sk_reduce_write_act(const WqGemmParams& p, const fl
 // whoever does it) and write those rows.  `own` (optional) is this CTA's own part
 // still in shared memory, read instead of its copy in L2.  kBatch items per thread are in flight at once: the
 // partials come from L2 at ~1 k cycles per round trip, so the loop is latency bound without batching.
-template <int kBatch, int kPartUnroll>
+template <int FMT, int kBatch, int kPartUnroll>
 __device__ __forceinline__ void sk_reduce_write(const WqGemmParams& p, const SkSegment& seg, int unit, int tid,
                                                 int nthreads, int m0, int row_lo, int row_hi, int n_base, const float* own) {
   const size_t part_elems = static_cast<size_t>(p.mb) * kTileN;
@@ -326,7 +333,7 @@ __device__ __forceinline__ void sk_reduce_write(const WqGemmParams& p, const SkS
 #pragma unroll
     for (int b = 0; b < kBatch; ++b) {
       const int idx = base + b * nthreads;
-      if (idx < items) sk_store4(p, m0 + row_lo + (idx >> 5), n_base + (idx & 31) * 4, acc[b]);
+      if (idx < items) sk_store4<FMT>(p, m0 + row_lo + (idx >> 5), n_base + (idx & 31) * 4, acc[b]);
     }
   }
 }
@@ -622,7 +629,7 @@ wq_gemm_sk_kernel(const __grid_constant__ CUtensorMap tmap_x,
           }
         } else if (ok)
           for (int idx = tt; idx < rows_here * (kTileN / 4); idx += nthr)
-            sk_store4(p, m0 + (idx >> 5), n_base + (idx & 31) * 4, *reinterpret_cast<const float4*>(stg + static_cast<size_t>(idx) * 4));
+            sk_store4<FMT>(p, m0 + (idx >> 5), n_base + (idx & 31) * 4, *reinterpret_cast<const float4*>(stg + static_cast<size_t>(idx) * 4));
       } else {
         if (ok) {
           float* slot = sk_slot(p, unit, seg.part);
@@ -650,7 +657,7 @@ wq_gemm_sk_kernel(const __grid_constant__ CUtensorMap tmap_x,
         if (ctl->is_last && !*abort_flag) {
           __threadfence();
           finalized = true;
-          sk_reduce_write<4, 2>(p, seg, unit, tt, nthr, m0, 0, rows_here, n_base, stg);
+          sk_reduce_write<FMT, 4, 2>(p, seg, unit, tt, nthr, m0, 0, rows_here, n_base, stg);
         }
       }
       if (p.tp.mode & kTpScatterPush) {
@@ -684,8 +691,8 @@ wq_gemm_sk_kernel(const __grid_constant__ CUtensorMap tmap_x,
           // sliced: thread 0 has acquired the counter and the barrier orders the CTA behind it; the partials are
           // read from L2 (ld.cg), where the writers' fences put them
           if (!sliced) __threadfence();
-          if (sliced) sk_reduce_write<2, 4>(p, ds, unit, tt, nthr, c.m0, row_lo, row_hi, c.n_tile * kTileN, nullptr);
-          else sk_reduce_write<4, 2>(p, ds, unit, tt, nthr, c.m0, row_lo, row_hi, c.n_tile * kTileN, nullptr);
+          if (sliced) sk_reduce_write<FMT, 2, 4>(p, ds, unit, tt, nthr, c.m0, row_lo, row_hi, c.n_tile * kTileN, nullptr);
+          else sk_reduce_write<FMT, 4, 2>(p, ds, unit, tt, nthr, c.m0, row_lo, row_hi, c.n_tile * kTileN, nullptr);
         }
         if (sliced) {
           tail_bar();
@@ -866,7 +873,7 @@ wq_gemm_sk_kernel(const __grid_constant__ CUtensorMap tmap_x,
                 if (!whole) {
                   *reinterpret_cast<float4*>(slot + static_cast<size_t>(c0 + row) * kTileN) = v;
                 } else if (c0 + row < rows_here) {
-                  sk_store4(p, m0 + c0 + row, n_base + quad * 32 + f4, v);
+                  sk_store4<FMT>(p, m0 + c0 + row, n_base + quad * 32 + f4, v);
                 }
               }
             }

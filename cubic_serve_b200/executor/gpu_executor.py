@@ -13,7 +13,7 @@ chunks (variable token counts) launch the same kernels eagerly.
 from __future__ import annotations
 
 import logging
-from dataclasses import dataclass
+from dataclasses import dataclass, field, replace
 
 import numpy as np
 import torch
@@ -51,6 +51,8 @@ class Segment:
     # [(offset, rows [n, layers, hidden])]: additions to the hidden state at media positions after the first decoder
     # layers (towers with intermediate outputs; executors that state ``accepts_deepstack``)
     deep_embeds: object = None
+    # offsets of this segment's tokens whose logits are wanted (``GpuExecutor.execute_logits``)
+    logit_offsets: list = field(default_factory=list)
 
 
 class _Staging:
@@ -278,7 +280,7 @@ class GpuExecutor:
         self._fill = self.builder._fill
         self.invalidate_page_rows = self.builder.invalidate_page_rows
         v_local = runner.w.lm_head.n
-        self.logits = torch.empty(max_rows, v_local, dtype=torch.bfloat16, device=self.device)
+        self.logits = torch.empty(max_rows, v_local, dtype=getattr(runner, "logits_dtype", torch.bfloat16), device=self.device)
         self.out_ids = torch.zeros(max_rows * rows_per_request, dtype=torch.int32, device=self.device)
         # two result buffers: a step may be launched before the previous step's ids have been read (``launch`` / ``collect``)
         self.out_host = torch.zeros(2, max_rows * rows_per_request, dtype=torch.int32, pin_memory=torch.cuda.is_available())
@@ -466,6 +468,44 @@ class GpuExecutor:
     def execute(self, segs: list[Segment]) -> np.ndarray:
         """Run one step and return the sampled token id of every sampling segment (host array)."""
         return self.collect(self.launch(segs))
+
+    @torch.no_grad()
+    def execute_logits(self, segs: list[Segment]) -> list[np.ndarray]:
+        """Run one step that samples nothing and return, per segment, the fp32 logits ``[wanted, vocab]`` at its
+        ``logit_offsets``.  The step is the one ``execute`` runs: a decode step replays its graph, a step with portions of
+        prompts launches the same kernels eagerly; only the rows that reach the output head differ."""
+        if self.runner.tp is not None or self.runner.pp is not None:
+            raise NotImplementedError("logits of chosen positions are read on one GPU")
+        if self.use_graphs and all(len(s.token_ids) == 1 for s in segs) and self.graph_rt.dispatch(len(segs)) is not None:
+            self.collect(self.launch([replace(s, sample=True, temperature=0.0, mask=None) for s in segs]))
+            got = self.logits[:len(segs)].float().cpu().numpy()
+            return [got[i:i + 1] if s.logit_offsets else got[:0] for i, s in enumerate(segs)]
+        if self._upload_pending:
+            self._uploaded.synchronize()
+            self._upload_pending = False
+        b, _ = self._fill([replace(s, sample=False) for s in segs])
+        rows, base = [], 0
+        for s in segs:
+            rows += [base + int(o) for o in s.logit_offsets]
+            base += len(s.token_ids)
+        out = np.empty((len(rows), self.logits.shape[1]), dtype=np.float32)
+        with torch.cuda.stream(self.stream):
+            self.h2d_bytes_last = self.stage.upload()
+            hidden = self.runner.forward_hidden(b)
+            if rows:
+                index = torch.tensor(rows, dtype=torch.int64, device=self.device)
+                for i in range(0, len(rows), self.max_rows):
+                    b.logit_rows = index[i:i + self.max_rows]
+                    b.num_logit_rows = b.logit_rows.numel()
+                    part = self.runner.forward_logits(b, hidden, self.logits)
+                    out[i:i + b.num_logit_rows] = part.float().cpu().numpy()
+            self.stream.synchronize()
+        self.kernel_launches_last = self.runner.launches_per_step
+        split, i = [], 0
+        for s in segs:
+            split.append(out[i:i + len(s.logit_offsets)])
+            i += len(s.logit_offsets)
+        return split
 
     def launch(self, segs: list[Segment], feedback_rows: int = 0) -> dict:
         """Enqueue one step without waiting for it: stage + upload the inputs, replay the graph (or run eagerly),

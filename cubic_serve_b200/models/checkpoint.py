@@ -214,8 +214,34 @@ class AdmittedCheckpoint:
         return _dense_of(self.cfg.quant.method, self.payload(module), (rows, self.cfg.hidden_size), self.cfg.quant)
 
 
+def layered_config_of(path: Path):
+    """Configuration of a layered checkpoint directory (``models/layered.py``), or None when it is not one."""
+    from .layered import architecture_of, parse_layered_config
+    raw = json.loads((path / "config.json").read_text())
+    if architecture_of(raw) is None:
+        return None
+    shapes = {n: r.shape for n, r in SafetensorsDirectory(path).tensors.items()}
+    return parse_layered_config(raw, shapes, name=path.resolve().name)
+
+
+def _admit_layered(path: Path, raw: dict) -> AdmittedCheckpoint:
+    from .layered import LayeredConfigError, check_inventory, parse_layered_config
+    store = SafetensorsDirectory(path)
+    shapes = {n: r.shape for n, r in store.tensors.items()}
+    try:
+        cfg = parse_layered_config(raw, shapes, name=path.resolve().name)
+        check_inventory(cfg, shapes)
+    except (LayeredConfigError, KeyError, TypeError) as exc:
+        raise CheckpointError(f"{path.name}: {exc}") from exc
+    return AdmittedCheckpoint(cfg, store, {}, {n: n for n in shapes}, raw_config=raw)
+
+
 def admit_checkpoint(path: str | Path) -> AdmittedCheckpoint:
     path = Path(path)
+    from .layered import architecture_of
+    raw = json.loads((path / "config.json").read_text())
+    if architecture_of(raw) is not None:
+        return _admit_layered(path, raw)
     cfg = ModelConfig.from_hf_config(path / "config.json")
     store = SafetensorsDirectory(path)
     linears, plain = logical_inventory(cfg)
@@ -306,6 +332,17 @@ def inspect_checkpoint(path: str | Path) -> dict:
                 "tensors": len(store.tensors), "elements": sum(math.prod(t.shape) for t in store.tensors.values()),
                 "manifest_digest": WeightManifest.from_store(store).digest, "execution_mode": "eager"}
     ck = admit_checkpoint(path)
+    if ck.cfg.family == "layered":
+        from .layered import LatentSpec
+        c = ck.cfg
+        mixers = [("latent" if isinstance(l.mixer, LatentSpec) else "channel_delta" if l.mixer.per_channel else "delta")
+                  for l in c.layers]
+        return {"model": c.name, "family": c.family, "architecture": c.architecture, "layers": c.num_layers,
+                "layer_runs": len(c.runs), "hidden": c.hidden_size, "vocab": c.vocab_size,
+                "mixers": {k: mixers.count(k) for k in sorted(set(mixers))}, "loop": c.loop,
+                "cache_bytes_per_token": c.page_bytes // 16, "state_bytes_per_request": c.state_bytes_per_request,
+                "tensors": len(ck.store.tensors), "elements": sum(math.prod(t.shape) for t in ck.store.tensors.values()),
+                "manifest_digest": WeightManifest.from_store(ck.store).digest}
     total = sum(math.prod(t.shape) for t in ck.store.tensors.values())
     by_dtype: dict[str, int] = {}
     for t in ck.store.tensors.values():

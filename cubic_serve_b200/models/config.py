@@ -288,4 +288,11 @@ def _qwen4_exp_tiny():
     return tiny_config()
 
 
+def _layered(name: str):
+    from . import layered
+    return layered.NAMED[name]()
+
+
+NAMED_CONFIGS["layered-tiny"] = lambda: _layered("layered-tiny")
+NAMED_CONFIGS["layered-8b"] = lambda: _layered("layered-8b")
 NAMED_CONFIGS["qwen4-exp-tiny"] = _qwen4_exp_tiny          # served by the eager executor of ``models/qwen4_exp.py``

@@ -1,0 +1,190 @@
+"""Plain model of the layered decoders (``Bumodra`` checkpoints): the oracle of the native runner and the model of the
+eager execution mode.
+
+Everything is written from the equations, token by token where the mechanism is a recurrence, one function per
+mechanism, on the raw ``config.json`` dictionary and the checkpoint's tensors by name.  It shares no code with
+``models/layered.py`` (configuration, packing) or the kernels, so that the two can be compared.  Arithmetic is done in
+the dtype of ``Oracle.dtype`` (fp32 by default, fp64 for comparisons that should not see the oracle's own rounding).
+
+``Oracle.forward`` runs one request's new tokens against its explicit state; prefill in portions, token-by-token decoding
+and one pass over the whole sequence give the same logits.
+"""
+from __future__ import annotations
+
+import copy
+import math
+
+import numpy as np
+import torch
+
+
+# ------------------------------------------------------------------ mechanisms
+def rms(x: torch.Tensor, eps: float) -> torch.Tensor:
+    """``x / sqrt(mean(x^2) + eps)`` over the last axis."""
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
+
+
+def rms_around_zero(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+    """RMS norm whose stored weight is the deviation from one."""
+    return rms(x, eps) * (1.0 + w)
+
+
+def unit(x: torch.Tensor) -> torch.Tensor:
+    return x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)
+
+
+def silu(x: torch.Tensor) -> torch.Tensor:
+    return x / (1.0 + torch.exp(-x))
+
+
+def softplus(x: torch.Tensor) -> torch.Tensor:
+    return torch.clamp(x, min=0) + torch.log1p(torch.exp(-x.abs()))
+
+
+def short_conv(x: torch.Tensor, w: torch.Tensor, past: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    """Causal depthwise convolution over time and silu.  ``x`` [n, C] new inputs, ``w`` [C, taps] with the current input's
+    tap last, ``past`` [taps - 1, C] inputs before ``x``.  Returns the outputs and the new ``past``."""
+    taps = w.shape[1]
+    ext = torch.cat([past, x])
+    out = torch.zeros_like(x)
+    for j in range(taps):
+        out = out + w[:, j] * ext[j:j + x.shape[0]]
+    return silu(out), ext[ext.shape[0] - (taps - 1):].clone()
+
+
+def delta_step(S: torch.Tensor, q, k, v, beta, decay) -> tuple[torch.Tensor, torch.Tensor]:
+    """One token of the gated delta rule for all heads.  ``S`` [H, dim, vdim]; ``q``, ``k`` [H, dim]; ``v`` [H, vdim];
+    ``beta`` [H]; ``decay`` [H, dim] (a head's scalar decay repeated, or one factor per key channel)."""
+    S = decay.unsqueeze(-1) * S
+    held = torch.einsum("hkv,hk->hv", S, k)
+    u = beta.unsqueeze(-1) * (v - held)
+    S = S + k.unsqueeze(-1) * u.unsqueeze(1)
+    return torch.einsum("hkv,hk->hv", S, q), S
+
+
+def windowed_attention(q, k, v, first: int, window: int | None, scale: float) -> torch.Tensor:
+    """Softmax attention of queries at positions ``first ..`` over keys at positions ``0 ..``: position i sees j with
+    ``0 <= i - j < window``.  ``q`` [n, H, d], ``k`` [m, H, d], ``v`` [m, H, e]."""
+    n, m = q.shape[0], k.shape[0]
+    i = torch.arange(first, first + n).unsqueeze(1)
+    j = torch.arange(m).unsqueeze(0)
+    seen = (i - j) >= 0
+    if window is not None:
+        seen &= (i - j) < window
+    s = torch.einsum("nhd,mhd->hnm", q, k) * scale
+    s = s.masked_fill(~seen, float("-inf"))
+    return torch.einsum("hnm,mhe->nhe", torch.softmax(s, -1), v)
+
+
+def squared_relu(x: torch.Tensor) -> torch.Tensor:
+    return torch.clamp(x, min=0) ** 2
+
+
+# ------------------------------------------------------------------ layers
+def delta_mixer(w, p: str, m: dict, h, st: dict, eps: float, per_channel: bool) -> torch.Tensor:
+    H, G, d, e = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    n = h.shape[0]
+    if not st:
+        for t, c in (("q", G * d), ("k", G * d), ("v", H * e)):
+            st[t] = torch.zeros(m["conv"] - 1, c, dtype=h.dtype)
+        st["S"] = torch.zeros(H, d, e, dtype=h.dtype)
+    mixed = {}
+    for t in ("q", "k", "v"):
+        mixed[t], st[t] = short_conv(h @ w[f"{p}.{t}"].T, w[f"{p}.{t}.conv"], st[t])
+    rep = torch.arange(H) // (H // G)
+    q = unit(mixed["q"].view(n, G, d))[:, rep] * d ** -0.5
+    k = unit(mixed["k"].view(n, G, d))[:, rep]
+    v = mixed["v"].view(n, H, e)
+    beta = 1.0 / (1.0 + torch.exp(-(h @ w[f"{p}.b"].T)))
+    rate = -torch.exp(w[f"{p}.A_log"])
+    if per_channel:
+        a = softplus((h @ w[f"{p}.a1"].T) @ w[f"{p}.a2"].T + w[f"{p}.dt_bias"]).view(n, H, d)
+        decay = torch.exp(rate.view(1, H, 1) * a)
+        z = (h @ w[f"{p}.g1"].T) @ w[f"{p}.g2"].T
+        gate = 1.0 / (1.0 + torch.exp(-z))
+    else:
+        a = softplus(h @ w[f"{p}.a"].T + w[f"{p}.dt_bias"])
+        decay = torch.exp(rate * a).unsqueeze(-1).expand(n, H, d)
+        gate = silu(h @ w[f"{p}.g"].T)
+    o = torch.empty(n, H, e, dtype=h.dtype)
+    for t in range(n):
+        o[t], st["S"] = delta_step(st["S"], q[t], k[t], v[t], beta[t], decay[t])
+    o = rms(o, eps) * w[f"{p}.norm"] * gate.view(n, H, e)
+    return o.reshape(n, H * e) @ w[f"{p}.o"].T
+
+
+def latent_mixer(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    H, d, e = m["heads"], m["dim"], m["vdim"]
+    n = h.shape[0]
+    cq = rms(h @ w[f"{p}.dq"].T, eps) * w[f"{p}.dq.norm"]
+    q = (cq @ w[f"{p}.uq"].T).view(n, H, d)
+    c = rms(h @ w[f"{p}.dkv"].T, eps) * w[f"{p}.dkv.norm"]
+    first = st["c"].shape[0] if st else 0
+    st["c"] = torch.cat([st["c"], c]) if st else c
+    k = (st["c"] @ w[f"{p}.uk"].T).view(-1, H, d)
+    v = (st["c"] @ w[f"{p}.uv"].T).view(-1, H, e)
+    mask = m.get("mask")
+    o = windowed_attention(q, k, v, first, mask["size"] if mask else None, m["scale"])
+    gate = 1.0 / (1.0 + torch.exp(-(h @ w[f"{p}.g"].T)))
+    o = o * gate.unsqueeze(-1)
+    return o.reshape(n, H * e) @ w[f"{p}.o"].T
+
+
+def layer_schedule(cfg: dict) -> list[tuple[int, bool]]:
+    """The layer runs in order: (layer index, whether the pass's entry projection comes right before it)."""
+    loop = cfg.get("loop")
+    n = len(cfg["layers"])
+    if not loop:
+        return [(i, False) for i in range(n)]
+    a, b, r = loop["start"], loop["stop"], loop["times"]
+    return ([(i, False) for i in range(a)] + [(i, i == a) for _ in range(r) for i in range(a, b)]
+            + [(i, False) for i in range(b, n)])
+
+
+class Oracle:
+    def __init__(self, cfg: dict, weights: dict[str, torch.Tensor], dtype=torch.float32) -> None:
+        self.cfg, self.dtype = cfg, dtype
+        self.w = {n: t.to(dtype) if t.is_floating_point() else t for n, t in weights.items()}
+        self.schedule = layer_schedule(cfg)
+
+    def new_state(self) -> "OracleState":
+        return OracleState([{} for _ in self.schedule])
+
+    @torch.no_grad()
+    def forward(self, tokens, state=None, positions3=None, embeds=None, last_only: bool = False, trace: list | None = None):
+        """Append ``tokens`` to ``state``; returns (logits, state).  ``trace`` receives the residual after every run."""
+        w, cfg = self.w, self.cfg
+        eps = float(cfg["norm"]["eps"])
+        state = state if state is not None else self.new_state()
+        ids = torch.as_tensor(list(tokens), dtype=torch.long)
+        x0 = rms_around_zero(w["embed"][ids], w["embed.norm"], eps)
+        x = x0
+        for (i, enters), st in zip(self.schedule, state.runs):
+            if enters:
+                x = torch.cat([x, x0], -1) @ w["loop.in"].T
+            layer, p = cfg["layers"][i], f"l{i}"
+            h = rms_around_zero(x, w[f"{p}.norm1"], eps)
+            kind, m = layer["type"], layer["mixer"]
+            if kind == "latent_attention":
+                y = latent_mixer(w, f"{p}.mix", m, h, st, eps)
+            elif kind in ("delta", "channel_delta"):
+                y = delta_mixer(w, f"{p}.mix", m, h, st, eps, kind == "channel_delta")
+            else:
+                raise ValueError(f"unknown mixer {kind!r}")
+            if layer.get("mlp"):
+                y = y + squared_relu(h @ w[f"{p}.mlp.up"].T) @ w[f"{p}.mlp.down"].T
+            x = x + y
+            if trace is not None:
+                trace.append(x.clone())
+        state.length += len(ids)
+        if last_only:
+            x = x[-1:]
+        return rms_around_zero(x, w["final.norm"], eps) @ w["head"].T, state
+
+
+class OracleState:
+    def __init__(self, runs: list[dict]) -> None:
+        self.runs, self.length = runs, 0
+
+    def copy(self) -> "OracleState":
+        return copy.deepcopy(self)

@@ -70,6 +70,24 @@ def _builtin() -> None:
     register(ModelDefinition("qwen3_5_moe", ("Qwen3_5MoeForCausalLM",),
                              description="hybrid decoder with routed experts", **common))
 
+    from .layered import ARCHITECTURES as LAYERED, load_layered_weights, random_layered_weights
+
+    def parse_layered(path: Path):
+        from .checkpoint import layered_config_of
+        return layered_config_of(Path(path))
+
+    def runner_layered(cfg, weights, **kw):
+        from .layered_runner import LayeredRunner
+        kw.pop("k_bits", None), kw.pop("v_bits", None)          # latents are cached in the activation type
+        if kw.pop("kv_rotation", False):
+            raise ModelRegistryError("cache rotation applies to quantized key / value caches, not to cached latents")
+        return LayeredRunner(cfg, weights, **kw)
+
+    register(ModelDefinition("layered", LAYERED, parse_config=parse_layered, random_weights=random_layered_weights,
+                             load_weights=load_layered_weights, build_runner=runner_layered,
+                             description="parallel layers with a mixer each (delta rule per head or per channel, windowed "
+                                         "latent attention), optional loop over a run of layers, fp32 residual"))
+
     def parse_q4(path: Path):
         from .qwen4_exp import parse_qwen4_exp_config_json
         p = Path(path)

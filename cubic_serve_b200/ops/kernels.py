@@ -501,7 +501,7 @@ def sample(logits: torch.Tensor, out_ids: torch.Tensor, temperature: torch.Tenso
            mask: torch.Tensor | None = None, out_logprob: torch.Tensor | None = None,
            vocab: int | None = None, out_value: torch.Tensor | None = None, id_offset: int = 0) -> torch.Tensor:
     rows = logits.shape[0]
-    code = native.lib().cb_sample(logits.data_ptr(), logits.stride(0), _ptr(mask),
+    code = native.lib().cb_sample(logits.data_ptr(), int(logits.dtype == torch.float32), logits.stride(0), _ptr(mask),
                                   0 if mask is None else mask.stride(0), _ptr(temperature), _ptr(top_p), _ptr(top_k),
                                   _ptr(seeds), _ptr(counters), out_ids.data_ptr(), _ptr(out_logprob),
                                   _ptr(out_value), int(id_offset), rows, vocab or logits.shape[1], _stream())
@@ -716,3 +716,135 @@ class ReasoningBudget:
                                                 self.fpos.data_ptr(), rows, self.end_token_id, self._seq,
                                                 len(self.forced), _stream())
         native.check(code, "cb_reasoning_budget")
+
+
+# ------------------------------------------------------------------ layered decoders (models/layered.py)
+def _seg(seg: GdnSegments) -> "native.GdnSegmentsStruct":
+    return seg.struct()
+
+
+def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: torch.Tensor | None = None,
+              relu2: torch.Tensor | None = None, split: int = 0, diag_rows: int = 0, ws: Workspace | None = None,
+              stream_k: bool | None = None, splits: int | None = None) -> None:
+    """``x @ W^T`` with bf16-stored weights through the wide epilogue.
+
+    ``x`` fp32: everything is fp32 (``csrc/layered.cu``); ``x`` bf16: tcgen05 with fp32 accumulation.  ``out`` gets the
+    product; an fp32 ``out`` may be added to ``residual`` (the same tensor: in-place accumulation).  With ``relu2`` the
+    features from ``split`` on leave there as ``max(v, 0)^2`` and ``out`` holds the first ``split``.  ``diag_rows``:
+    block-diagonal weights, see ``models/layered.py::BlockDiagonal``.  ``x`` may have fewer columns than ``w.k``: the rest
+    read as zero."""
+    m, k = x.shape[0], w.k
+    assert w.fmt == FMT_BF16 and x.stride(1) == 1 and out.stride(1) == 1 and out.shape[0] == m
+    assert out.shape[1] == (split if relu2 is not None else w.n), (out.shape, split, w.n)
+    assert residual is None or (residual.dtype == torch.float32 and residual.stride(0) == out.stride(0))
+    if relu2 is not None:
+        assert relu2.dtype == x.dtype and relu2.stride(1) == 1 and relu2.shape == (m, w.n - split) and split % 4 == 0
+    x_cols = min(x.shape[1], x.stride(0))
+    l = native.lib()
+    if x.dtype == torch.float32:
+        assert out.dtype == torch.float32
+        a = native.F32GemmStruct(x.data_ptr(), x.stride(0), x_cols, w.codes.data_ptr(), out.data_ptr(), out.stride(0),
+                                 _ptr(residual), _ptr(relu2), 0 if relu2 is None else relu2.stride(0), split, diag_rows, m,
+                                 w.n, k)
+        native.check(l.cb_f32_gemm(ctypes.byref(a), _stream()), "cb_f32_gemm")
+        return
+    wide32 = out.dtype == torch.float32
+    assert residual is None or wide32
+    ws = ws or workspace(x.device)
+    if stream_k is None:
+        stream_k = splits is None and not diag_rows and use_stream_k(m, w.n, FMT_BF16, sm_count(x.device), k)
+    if splits is None:
+        splits = 1 if stream_k else choose_splits(m, w.n, k, fmt=FMT_BF16)
+    if splits > 1 and l.cb_wq_gemm_workspace_bytes(m, w.n, splits) > ws.gemm.numel():
+        splits = 1
+    from .strategies import active
+    a = native.WideGemmStruct(x.data_ptr(), x.stride(0), x_cols, w.codes.data_ptr(), None if wide32 else out.data_ptr(),
+                              out.data_ptr() if wide32 else None, out.stride(0), _ptr(residual), _ptr(relu2),
+                              0 if relu2 is None else relu2.stride(0), split, diag_rows, m, w.n, k, int(stream_k), splits,
+                              active().gemm.stream_k_min_units)
+    code = l.cb_bf16_gemm_wide(ctypes.byref(a), ws.gemm.data_ptr(), ws.gemm.numel(), ws.gemm_counters.data_ptr(),
+                               ws.status.data_ptr(), _stream())
+    native.check(code, "cb_bf16_gemm_wide")
+
+
+def row_norm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float, rows: torch.Tensor | None = None) -> None:
+    """``out[i] = x[i] / rms(x[i]) * weight`` from the fp32 residual stream (``rows``: int64 indices of the rows taken)."""
+    assert x.dtype == weight.dtype == torch.float32 and x.is_contiguous() and out.stride(1) == 1
+    n = x.shape[0] if rows is None else rows.numel()
+    assert out.shape[0] >= n
+    native.check(native.lib().cb_row_norm(x.data_ptr(), _ptr(rows), weight.data_ptr(), out.data_ptr(), out.stride(0), n,
+                                          x.shape[1], float(eps), int(out.dtype == torch.float32), _stream()), "cb_row_norm")
+
+
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, eps: float,
+               x0: torch.Tensor | None = None) -> None:
+    """``x`` (and ``x0``) = RMS norm of the embedding rows, fp32."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and table.dtype == torch.bfloat16
+    native.check(native.lib().cb_embed_norm(ids.data_ptr(), table.data_ptr(), weight.data_ptr(), x.data_ptr(), _ptr(x0),
+                                            x.shape[0], x.shape[1], table.shape[0], float(eps), _stream()), "cb_embed_norm")
+
+
+def concat_rows(x: torch.Tensor, x0: torch.Tensor, out: torch.Tensor) -> None:
+    """``out = [x ; x0]`` along the columns, in ``out``'s type."""
+    native.check(native.lib().cb_concat_rows(x.data_ptr(), x0.data_ptr(), out.data_ptr(), out.stride(0), x.shape[0],
+                                             x.shape[1], int(out.dtype == torch.float32), _stream()), "cb_concat_rows")
+
+
+def conv_silu(x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, seg: GdnSegments, out: torch.Tensor) -> None:
+    """Causal depthwise convolution of any number of taps + SiLU over ``x[T, C]`` per request segment; ``state``
+    ``[slots, taps - 1, C]`` (activation type) is read and replaced.  ``w``: fp32 ``[C, taps]``, last tap = current input."""
+    c, taps = w.shape
+    assert w.dtype == torch.float32 and w.is_contiguous() and state.dtype == x.dtype == out.dtype
+    assert x.shape[1] == out.shape[1] == c and x.stride(1) == out.stride(1) == 1
+    assert state.is_contiguous() and (taps == 1 or tuple(state.shape[1:]) == (taps - 1, c))
+    st = _seg(seg)
+    native.check(native.lib().cb_conv_silu(x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), w.data_ptr(),
+                                           state.data_ptr(), ctypes.byref(st), c, taps, x.shape[0],
+                                           int(x.dtype == torch.float32), _stream()), "cb_conv_silu")
+
+
+def delta_rule(qkv: torch.Tensor, b: torch.Tensor, a: torch.Tensor, z: torch.Tensor, a_log: torch.Tensor,
+               dt_bias: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, seg: GdnSegments, out: torch.Tensor,
+               kv_heads: int, dim: int, eps: float, sigmoid_gate: bool, decode: bool, raw: torch.Tensor) -> int:
+    """Gated delta rule and gated norm of every head, see ``csrc/delta_rule.cu``.  ``state`` fp32 ``[slots, H, vdim, stride]``;
+    ``a`` has one decay logit per head, or one per (head, key channel) when it has ``H dim`` columns.  ``raw``: fp32 scratch
+    of at least ``T H vdim`` elements.  Returns the launches made at most."""
+    H, e, ds = state.shape[1:]
+    T = qkv.shape[0]
+    channel = dt_bias.numel() != H
+    assert state.dtype == torch.float32 and state.is_contiguous() and dt_bias.numel() in (H, H * dim)
+    assert all(t.stride(1) == 1 and t.dtype == qkv.dtype for t in (qkv, b, a, z, out))
+    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (a_log, dt_bias, norm_w))
+    assert raw.dtype == torch.float32 and raw.numel() >= T * H * e and out.shape[1] == H * e
+    d = native.DeltaRuleStruct(qkv.data_ptr(), qkv.stride(0), b.data_ptr(), b.stride(0), a.data_ptr(), a.stride(0),
+                               z.data_ptr(), z.stride(0), a_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr(),
+                               state.data_ptr(), out.data_ptr(), out.stride(0), raw.data_ptr(), H, kv_heads, dim, e, ds,
+                               float(eps), int(sigmoid_gate), int(channel), int(decode), T, int(qkv.dtype == torch.float32))
+    st = _seg(seg)
+    native.check(native.lib().cb_delta_rule(ctypes.byref(d), ctypes.byref(st), _stream()), "cb_delta_rule")
+    return 2
+
+
+def latent_prepare(proj: torch.Tensor, q_rank: int, c_off: int, rank: int, q_norm: torch.Tensor, c_norm: torch.Tensor,
+                   cq: torch.Tensor, cache: torch.Tensor, slots: torch.Tensor, eps: float) -> None:
+    """RMS norms of the query latent (columns ``[0, q_rank)`` of ``proj``) into ``cq`` and of the cache latent (columns
+    ``[c_off, c_off + rank)``) into its page of ``cache`` ``[pages, 16, rank padded]``."""
+    assert cache.is_contiguous() and cache.dtype == proj.dtype == cq.dtype and slots.dtype == torch.int32
+    native.check(native.lib().cb_latent_prepare(proj.data_ptr(), proj.stride(0), 0, q_rank, c_off, rank, q_norm.data_ptr(),
+                                                c_norm.data_ptr(), cq.data_ptr(), cq.stride(0), cache.data_ptr(),
+                                                cache.shape[2], slots.data_ptr(), proj.shape[0], float(eps),
+                                                int(proj.dtype == torch.float32), _stream()), "cb_latent_prepare")
+
+
+def latent_attention(q: torch.Tensor, gate: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor, seg: GdnSegments,
+                     out: torch.Tensor, heads: int, window: int, scale: float) -> None:
+    """Windowed softmax attention of latent-space queries ``q [T, H Rp]`` over the paged latents, times the heads' sigmoid
+    gates (``gate [T, H]`` logits).  ``window`` 0: every earlier token."""
+    T, rp = q.shape[0], cache.shape[2]
+    assert q.shape[1] == out.shape[1] == heads * rp and q.is_contiguous() and out.is_contiguous()
+    assert q.dtype == out.dtype == gate.dtype == cache.dtype and page_table.dtype == torch.int32
+    a = native.LatentAttnStruct(q.data_ptr(), out.data_ptr(), cache.data_ptr(), gate.data_ptr(), gate.stride(0),
+                                page_table.data_ptr(), page_table.shape[1], heads, rp, window, float(scale), T,
+                                int(q.dtype == torch.float32))
+    st = _seg(seg)
+    native.check(native.lib().cb_latent_attn(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_latent_attn")

@@ -197,7 +197,7 @@ def _declare(l: ctypes.CDLL) -> None:
     l.cb_paged_attn_partial_floats.restype = ll
     l.cb_paged_attn.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i, i, i, i, i, i, i, f, i, vp, vp, vp, vp]
     l.cb_paged_attn.restype = i
-    l.cb_sample.argtypes = [vp, i, vp, i, vp, vp, vp, vp, vp, vp, vp, vp, i, i, i, vp]
+    l.cb_sample.argtypes = [vp, i, i, vp, i, vp, vp, vp, vp, vp, vp, vp, vp, i, i, i, vp]
     l.cb_sample.restype = i
     l.cb_verify_greedy.argtypes = [vp, vp, vp, i, vp, vp, vp, i, vp]
     l.cb_verify_greedy.restype = i
@@ -261,6 +261,19 @@ def _declare(l: ctypes.CDLL) -> None:
     l.cb_canary_fill.restype = i
     l.cb_canary_check.argtypes = [vp, ll, ctypes.c_uint, i, vp, vp]
     l.cb_canary_check.restype = i
+    # layered decoders: fp32 residual stream, delta rule of any head size, latent attention
+    l.cb_bf16_gemm_wide.argtypes = [vp, vp, ll, vp, vp, vp]
+    l.cb_f32_gemm.argtypes = [vp, vp]
+    l.cb_row_norm.argtypes = [vp, vp, vp, vp, i, i, i, f, i, vp]
+    l.cb_embed_norm.argtypes = [vp, vp, vp, vp, vp, i, i, i, f, vp]
+    l.cb_concat_rows.argtypes = [vp, vp, vp, i, i, i, i, vp]
+    l.cb_conv_silu.argtypes = [vp, i, vp, i, vp, vp, vp, i, i, i, i, vp]
+    l.cb_delta_rule.argtypes = [vp, vp, vp]
+    l.cb_latent_prepare.argtypes = [vp, i, i, i, i, i, vp, vp, vp, i, vp, i, vp, i, f, i, vp]
+    l.cb_latent_attn.argtypes = [vp, vp, vp]
+    for name in ("bf16_gemm_wide", "f32_gemm", "row_norm", "embed_norm", "concat_rows", "conv_silu", "delta_rule",
+                 "latent_prepare", "latent_attn"):
+        getattr(l, f"cb_{name}").restype = i
     # fp8 (e4m3 x e4m3) tensor path: activation quantizers and the GEMM entries
     l.cb_fp8_quantize_rows.argtypes = [vp, i, vp, i, vp, i, i, vp]
     l.cb_fp8_quantize_rows.restype = i
@@ -296,6 +309,42 @@ class GdnDeltaStruct(ctypes.Structure):
                 ("dt_bias", ctypes.c_void_p), ("norm_w", ctypes.c_void_p), ("state", ctypes.c_void_p),
                 ("out", ctypes.c_void_p), ("ldo", ctypes.c_int), ("Hk", ctypes.c_int), ("Hv", ctypes.c_int),
                 ("eps_norm", ctypes.c_float), ("eps_l2", ctypes.c_float), ("commit", ctypes.c_int)]
+
+
+class WideGemmStruct(ctypes.Structure):
+    """Mirror of ``CbWideGemm`` in ``csrc/wq_gemm.cu``."""
+    _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("x_cols", ctypes.c_int), ("w", ctypes.c_void_p),
+                ("y", ctypes.c_void_p), ("y32", ctypes.c_void_p), ("ldy", ctypes.c_int), ("residual32", ctypes.c_void_p),
+                ("y2", ctypes.c_void_p), ("ldy2", ctypes.c_int), ("n_split", ctypes.c_int), ("diag_n", ctypes.c_int),
+                ("M", ctypes.c_int), ("N", ctypes.c_int), ("K", ctypes.c_int), ("stream_k", ctypes.c_int),
+                ("splits", ctypes.c_int), ("min_units", ctypes.c_int)]
+
+
+class F32GemmStruct(ctypes.Structure):
+    """Mirror of ``CbF32Gemm`` in ``csrc/layered.cu``."""
+    _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("x_cols", ctypes.c_int), ("w", ctypes.c_void_p),
+                ("y", ctypes.c_void_p), ("ldy", ctypes.c_int), ("residual", ctypes.c_void_p), ("y2", ctypes.c_void_p),
+                ("ldy2", ctypes.c_int), ("n_split", ctypes.c_int), ("diag_n", ctypes.c_int), ("M", ctypes.c_int),
+                ("N", ctypes.c_int), ("K", ctypes.c_int)]
+
+
+class DeltaRuleStruct(ctypes.Structure):
+    """Mirror of ``CbDeltaRule`` in ``csrc/delta_rule.cu``."""
+    _fields_ = [("qkv", ctypes.c_void_p), ("ldq", ctypes.c_int), ("b", ctypes.c_void_p), ("ldb", ctypes.c_int),
+                ("a", ctypes.c_void_p), ("lda", ctypes.c_int), ("z", ctypes.c_void_p), ("ldz", ctypes.c_int),
+                ("a_log", ctypes.c_void_p), ("dt_bias", ctypes.c_void_p), ("norm_w", ctypes.c_void_p),
+                ("state", ctypes.c_void_p), ("out", ctypes.c_void_p), ("ldo", ctypes.c_int), ("raw", ctypes.c_void_p),
+                ("H", ctypes.c_int), ("G", ctypes.c_int), ("d", ctypes.c_int), ("e", ctypes.c_int), ("ds", ctypes.c_int),
+                ("eps", ctypes.c_float), ("sigmoid_gate", ctypes.c_int), ("channel", ctypes.c_int),
+                ("decode", ctypes.c_int), ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
+
+
+class LatentAttnStruct(ctypes.Structure):
+    """Mirror of ``CbLatentAttn`` in ``csrc/latent_attn.cu``."""
+    _fields_ = [("q", ctypes.c_void_p), ("out", ctypes.c_void_p), ("cache", ctypes.c_void_p), ("gate", ctypes.c_void_p),
+                ("ldg", ctypes.c_int), ("page_table", ctypes.c_void_p), ("max_pages", ctypes.c_int), ("H", ctypes.c_int),
+                ("Rp", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float), ("tokens", ctypes.c_int),
+                ("f32", ctypes.c_int)]
 
 
 class ReduceNormStruct(ctypes.Structure):

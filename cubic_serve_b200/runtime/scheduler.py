@@ -351,6 +351,36 @@ class ContinuousScheduler:
         scheduled.add(r.request_id)
         return True
 
+    # ------------------------------------------------------------- imposed steps
+    def imposed_plan(self, entries: list[tuple[Request, int]]) -> BatchPlan:
+        """The plan of a step whose batch is given from outside: the next ``n`` tokens of every listed request, which are
+        known already (replays of token traces).  A waiting request is admitted at its first entry; pages are reserved as
+        for any other step, but nobody is preempted for them: a batch that does not fit is the caller's error."""
+        plan = BatchPlan([])
+        for r, n in entries:
+            if n < 1 or r.num_computed + n > r.num_tokens:
+                raise ValueError(f"request {r.request_id}: {n} tokens asked for, {r.remaining} are known")
+            if r.status is RequestStatus.WAITING:
+                if not self._free_slots:
+                    raise AdmissionError("no request slot is free", status=429)
+                r.arrival = next(self._clock)
+                r.slot = self._free_slots.pop()
+                r.status = RequestStatus.RUNNING
+                self.running.append(r)
+            if r.status is not RequestStatus.RUNNING:
+                raise ValueError(f"request {r.request_id} is {r.status.value}")
+            if r.num_computed + n > self.cfg.max_model_len:
+                raise AdmissionError(f"request {r.request_id} exceeds max_model_len {self.cfg.max_model_len}")
+            self._ensure_pages(r, r.num_computed + n, plan.copies)
+            plan.segments.append(PlannedSegment(r, r.num_computed, n, False))
+        return plan
+
+    def release(self, r: Request, reason: FinishReason = FinishReason.STOP) -> None:
+        """End a request from outside: its pages and its slot are free for others."""
+        if r in self.waiting:
+            self.waiting.remove(r)
+        self._retire(r, reason)
+
     def lookahead_plan(self, prev: BatchPlan) -> BatchPlan | None:
         """The decode step that follows ``prev`` if ``prev`` finishes nobody, planned BEFORE ``prev`` is committed.
 
