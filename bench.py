@@ -57,6 +57,9 @@ def parse_args():
     ap.add_argument("--no-check", action="store_true", help="skip the untimed multi-GPU logit check")
     ap.add_argument("--accept", type=float, default=0.7,
                     help="forced per-depth acceptance probability of speculative rounds (random weights never agree)")
+    ap.add_argument("--layered", action="store_true",
+                    help="instead of the headline workload: the layered decoders beside the closest existing model at equal "
+                         "size, one JSON line per kernel and per model (one GPU)")
     return ap.parse_args()
 
 
@@ -119,6 +122,13 @@ def main() -> None:
     args = parse_args()
     if args.impl == "reference":
         run_reference(args)
+        return
+    if args.layered:
+        from cubic_serve_b200.benchmarks import layered
+        sampler = ClockSampler(0)
+        sampler.start()
+        layered.run(args.steps)
+        print(json.dumps({"clocks": sampler.stop()}), flush=True)
         return
     import numpy as np
     import torch

@@ -1,0 +1,277 @@
+"""Layered decoders beside the closest existing model at equal size: kernels against their rooflines, prefill and decode
+throughput of whole models (``bench.py --layered``).
+
+The closest model is the hybrid family (Gated DeltaNet layers with periodic full attention) with bf16 weights; its SwiGLU
+feed-forward has three matrices where the layered one has two, so its width is two thirds: equal parameters.  Weights are
+random, prompts are random ids, one GPU.  Kernel times are CUDA-event times inside CUDA graphs with L2 flushed; the roofline
+of a kernel is the slower of its bytes over the copy bandwidth and its operations over the pipe that runs them.
+"""
+from __future__ import annotations
+
+import json
+from pathlib import Path
+
+import torch
+
+from ..models.config import ModelConfig, QuantSpec
+from ..models.layered import DeltaSpec, LatentSpec, LayeredConfig, LayerSpec
+from ..ops import kernels as K, wq_pack
+from ..utils.kernel_bench import DEV, timeit_graph
+
+FP32_FLOPS = 148 * 128 * 2 * 1.965e9      # one fp32 multiply-add per lane and cycle
+
+
+def peaks() -> dict:
+    p = Path(__file__).resolve().parents[2] / "MEASURED_PEAKS.json"
+    if p.is_file():
+        d = json.loads(p.read_text())
+        return {"hbm": d["hbm_gbs"] * 1e9, "bf16": d["bf16_tflops"] * 1e12, "source": "measured"}
+    return {"hbm": 6.65e12, "bf16": 1.59e15, "source": "fallback"}
+
+
+def layered_config(width: int, layers: int) -> LayeredConfig:
+    """Real-model layer sizes at ``width``: heads of 128, feed-forward 3 x width, low ranks of 128, latents of 512."""
+    h = width // 128
+    ff = 3 * width
+    delta = LayerSpec(DeltaSpec(h, h // 2, 128, 128, 4), ff)
+    channel = LayerSpec(DeltaSpec(h, h, 128, 128, 4, True, 128, 128), ff)
+    latent = LayerSpec(LatentSpec(h, 128, 128, 1536, 512, 128 ** -0.5, 1024), ff)
+    return LayeredConfig(f"layered-{width}", 32768, width, (delta, channel, delta, latent) * (layers // 4), 1e-6)
+
+
+def hybrid_config(width: int, layers: int) -> ModelConfig:
+    h = width // 128
+    return ModelConfig(name=f"hybrid-{width}", family="qwen3_5", num_layers=layers, hidden_size=width, num_q_heads=h,
+                       num_kv_heads=max(1, h // 4), head_dim=128, intermediate_size=2 * width, vocab_size=32768, rope_theta=1e7,
+                       rotary_dim=64, qk_norm=True, zero_centered_norm=True, gdn_interval=4, gdn_k_heads=h // 2, gdn_v_heads=h,
+                       attn_output_gate=True, quant=QuantSpec("none", 16, 0))
+
+
+# ------------------------------------------------------------------ kernels
+def _segments(requests: int, tokens: int, pos0: int) -> K.GdnSegments:
+    i32 = dict(dtype=torch.int32, device=DEV)
+    return K.GdnSegments(torch.arange(requests, **i32) * tokens, torch.full((requests,), tokens, **i32),
+                         torch.arange(requests, **i32), torch.full((requests,), pos0, **i32), requests)
+
+
+def _line(name: str, ms: float, nbytes: float, flops: float, flop_peak: float, pk: dict) -> dict:
+    roof = max(nbytes / pk["hbm"], flops / flop_peak)
+    return {"kernel": name, "us": round(ms * 1e3, 1), "roofline_us": round(roof * 1e6, 1),
+            "bound": "memory" if nbytes / pk["hbm"] >= flops / flop_peak else "arithmetic",
+            f"fraction_of_{pk['source']}": round(roof * 1e3 / ms, 3)}
+
+
+def bench_delta(requests: int, tokens: int, heads: int, key_heads: int, channel: bool, flush, pk) -> list[dict]:
+    d, T, H, G = 128, requests * tokens, heads, key_heads
+    C = 2 * G * d + H * d
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    seg = _segments(requests, tokens, 5)
+    proj = torch.randn(T, C, device=DEV).to(torch.bfloat16)
+    conv_w = torch.randn(4, C, device=DEV) * 0.3
+    conv_state = torch.zeros(requests, 3, C, **bf)
+    state = torch.randn(requests, H, d, d, device=DEV) * 0.01
+    out = torch.empty(T, H * d, **bf)
+    b, z = torch.randn(T, H, **bf), torch.randn(T, H * d, **bf)
+    a = torch.randn(T, H * d if channel else H, **bf)
+    dt = torch.zeros(H * d if channel else H, device=DEV)
+    a_log, norm_w = torch.full((H,), -2.0, device=DEV), torch.ones(d, device=DEV)
+    sc = K.DeltaScratch(T, [(H, G, d, d, channel)], torch.bfloat16, DEV)
+    decode = tokens == 1
+    prep = timeit_graph(lambda: K.delta_prepare(proj, b, a, conv_w, conv_state, a_log, dt, seg, sc, H, G, d, d), flush, launches=5)
+    walk = timeit_graph(lambda: K.delta_walk(z, norm_w, state, seg, out, sc, G, d, 1e-6, channel, channel, decode), flush,
+                        launches=5)
+    kind = "channel" if channel else "head"
+    shape = f"{requests} x {tokens} tokens, {H} heads"
+    conv_io = T * C * 4 + 2 * requests * 3 * C * 2
+    return [_line(f"delta_prepare per {kind} [{shape}]", prep, conv_io + T * (H + a.shape[1]) * 2, 0, 1, pk),
+            _line(f"delta_walk + norm per {kind} [{shape}]", walk, 2 * state.numel() * 4 + T * (C + 2 * H * d) * 2,
+                  4 * 2.0 * T * H * d * d, FP32_FLOPS, pk),
+            _line(f"both per {kind} [{shape}]", prep + walk, 2 * state.numel() * 4 + conv_io + T * (2 * H * d + H + a.shape[1]) * 2,
+                  4 * 2.0 * T * H * d * d, FP32_FLOPS, pk)]
+
+
+def bench_gdn(requests: int, tokens: int, hv: int, hk: int, flush, pk) -> list[dict]:
+    d, T = 128, requests * tokens
+    C = (2 * hk + hv) * d
+    seg = _segments(requests, tokens, 5)
+    proj = torch.randn(T, C + hv * d + 2 * hv, device=DEV).to(torch.bfloat16)
+    w = torch.randn(C, 4, device=DEV) * 0.3
+    conv_state = torch.zeros(requests, 3, C, dtype=torch.bfloat16, device=DEV)
+    state = torch.randn(requests, hv, d, d, device=DEV) * 0.01
+    mix = torch.empty(T, C, dtype=torch.bfloat16, device=DEV)
+    out = torch.empty(T, hv * d, dtype=torch.bfloat16, device=DEV)
+    a_log, dt_bias, norm_w = torch.full((hv,), -2.0, device=DEV), torch.zeros(hv, device=DEV), torch.ones(d, device=DEV)
+    conv = timeit_graph(lambda: K.gdn_conv(proj, w, conv_state, seg, mix), flush, launches=5)
+    delta = timeit_graph(lambda: K.gdn_delta(mix, proj[:, C:C + hv * d], proj[:, C + hv * d:], a_log, dt_bias, norm_w, state,
+                                             seg, out, hk, hv), flush, launches=5)
+    shape = f"{requests} x {tokens} tokens, {hv} heads"
+    conv_io = T * C * 4 + 2 * requests * 3 * C * 2
+    return [_line(f"gdn_conv [{shape}]", conv, conv_io, 0, 1, pk),
+            _line(f"gdn_conv + gdn_delta [{shape}]", conv + delta, 2 * state.numel() * 4 + conv_io + T * (2 * hv * d + 2 * hv) * 2,
+                  4 * 2.0 * T * hv * d * d, FP32_FLOPS, pk),
+            _line(f"gdn_delta [{shape}]", delta, 2 * state.numel() * 4 + T * (C + 2 * hv * d + 2 * hv) * 2,
+                  4 * 2.0 * T * hv * d * d, FP32_FLOPS, pk)]
+
+
+def _visible(tokens: int, ctx: int, window: int) -> int:
+    """Keys seen by the ``tokens`` last positions of a context of ``ctx`` tokens."""
+    return sum(min(p + 1, window) if window else p + 1 for p in range(ctx - tokens, ctx))
+
+
+def bench_latent(requests: int, tokens: int, ctx: int, heads: int, rank: int, window: int, flush, pk) -> list[dict]:
+    T, per = requests * tokens, -(-ctx // 16)
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    cache = torch.randn(requests * per + 1, 16, rank, **bf)
+    table = (torch.randperm(requests * per, device=DEV).to(torch.int32) + 1).view(requests, per)
+    q, out, gate = torch.randn(T, heads * rank, **bf) * 0.05, torch.empty(T, heads * rank, **bf), torch.randn(T, heads, **bf)
+    seg = _segments(requests, tokens, ctx - tokens)
+    ms = timeit_graph(lambda: K.latent_attention(q, gate, cache, table, seg, out, heads, window, 0.1, decode=tokens == 1), flush,
+                      launches=5)
+    K.workspace(torch.device(DEV)).check_status()
+    pairs = requests * _visible(tokens, ctx, window)
+    keys = requests * (min(ctx, window + tokens) if window else ctx)
+    return [_line(f"latent_attn [{requests} x {tokens} at {ctx}, window {window}, {heads} heads, rank {rank}]", ms,
+                  keys * rank * 2 + 2 * T * heads * rank * 2, 4.0 * pairs * heads * rank, pk["bf16"], pk)]
+
+
+def bench_paged(requests: int, tokens: int, ctx: int, hq: int, hkv: int, flush, pk) -> list[dict]:
+    from ..ops import eager
+    d, T, per = 128, requests * tokens, -(-ctx // 16)
+    blob = K.kv_blob_bytes(d, 8, 8)
+    cache = torch.randint(0, 255, (requests * per + 1, hkv, blob), dtype=torch.uint8, device=DEV)
+    lay = eager.blob_layout(d, 8, 8)
+    one = torch.full((64,), 0.01, device=DEV).view(torch.uint8)
+    cache[:, :, lay["k_scale"]:lay["v_code"]] = one
+    cache[:, :, lay["v_scale"]:] = one
+    table = (torch.randperm(requests * per, device=DEV).to(torch.int32) + 1).view(requests, per)
+    q = torch.randn(T, hq, d, device=DEV, dtype=torch.bfloat16)
+    out = torch.empty_like(q)
+    qb = 16 // (hq // hkv)
+    blocks = [(r, r * tokens + i, min(qb, tokens - i), ctx - tokens + i + 1) for r in range(requests) for i in range(0, tokens, qb)]
+    rb = torch.tensor(blocks, dtype=torch.int32, device=DEV).t().contiguous()
+    splits = max(1, min(32, 296 // (len(blocks) * hkv)))
+    ms = timeit_graph(lambda: K.paged_attention(q, out, cache, table, rb[0], rb[1], rb[2], rb[3], hq, hkv, d, 8, 8, splits=splits),
+                      flush, launches=5)
+    K.workspace(torch.device(DEV)).check_status()
+    pairs = requests * _visible(tokens, ctx, 0)
+    return [_line(f"paged_attn int8 [{requests} x {tokens} at {ctx}, {hq}/{hkv} heads]", ms,
+                  requests * per * hkv * blob + 2 * T * hq * d * 2, 4.0 * pairs * hq * d, pk["bf16"], pk)]
+
+
+def bench_products(m: int, width: int, flush, pk) -> list[dict]:
+    """The two large products of a layer with their fused epilogues, beside the same shapes through the plain GEMM."""
+    h, ff = width // 128, 3 * width
+    split = 4 * width + 2 * h
+    x = torch.randn(m, width, device=DEV).to(torch.bfloat16)
+    w_in = wq_pack.pack_bf16(torch.randn(split + ff, width, device=DEV) * 0.02)
+    w_out = wq_pack.pack_bf16(torch.randn(width, width + ff, device=DEV) * 0.02)
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    proj, operand = torch.empty(m, split, **bf), torch.randn(m, width + ff, **bf)
+    res, y_in, y_out = torch.zeros(m, width, device=DEV), torch.empty(m, split + ff, **bf), torch.empty(m, width, **bf)
+    out = []
+    for name, fn, n, k, extra in (
+            ("wide_gemm in (relu^2, two outputs)", lambda: K.wide_gemm(x, w_in, proj, relu2=operand[:, width:], split=split), w_in.n, w_in.k, 0),
+            ("wq_gemm bf16, same shape", lambda: K.wq_gemm(x, w_in, out=y_in), w_in.n, w_in.k, 0),
+            ("wide_gemm out (fp32 residual)", lambda: K.wide_gemm(operand, w_out, res, residual=res), w_out.n, w_out.k, m * width * 6),
+            ("wq_gemm bf16, same shape", lambda: K.wq_gemm(operand, w_out, out=y_out), w_out.n, w_out.k, 0)):
+        ms = timeit_graph(fn, flush, launches=5)
+        out.append(_line(f"{name} [{m} x {n} x {k}]", ms, (n * k + m * (n + k)) * 2 + extra, 2.0 * m * n * k, pk["bf16"], pk))
+    K.workspace(torch.device(DEV)).check_status()
+    return out
+
+
+def bench_rows(m: int, width: int, flush, pk) -> list[dict]:
+    x, w = torch.randn(m, width, device=DEV), torch.ones(width, device=DEV)
+    h = torch.empty(m, width, dtype=torch.bfloat16, device=DEV)
+    xb, wb = x.to(torch.bfloat16), w.to(torch.bfloat16)
+    a = timeit_graph(lambda: K.row_norm(x, w, h, 1e-6), flush, launches=5)
+    b = timeit_graph(lambda: K.rmsnorm(xb, wb, 1e-6, out=h), flush, launches=5)
+    return [_line(f"row_norm fp32 in [{m} x {width}]", a, m * width * 6, 0, 1, pk),
+            _line(f"rmsnorm bf16 in [{m} x {width}]", b, m * width * 4, 0, 1, pk)]
+
+
+def kernels(width: int = 4096) -> list[dict]:
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=DEV)
+    pk = peaks()
+    h = width // 128
+    out = []
+    for requests, tokens in ((256, 1), (8, 1024), (1, 4096)):
+        out += bench_delta(requests, tokens, h, h // 2, False, flush, pk)
+        out += bench_delta(requests, tokens, h, h, True, flush, pk)
+        out += bench_gdn(requests, tokens, h, h // 2, flush, pk)
+    for requests, tokens, ctx in ((256, 1, 1280), (1, 1, 4096), (8, 1024, 1024), (1, 4096, 4096)):
+        out += bench_latent(requests, tokens, ctx, h, 512, 1024, flush, pk)
+        out += bench_paged(requests, tokens, ctx, h, max(1, h // 4), flush, pk)
+    for m in (16, 256, 4096):
+        out += bench_products(m, width, flush, pk)
+        out += bench_rows(m, width, flush, pk)
+    return out
+
+
+# ------------------------------------------------------------------ whole models
+def model_throughput(cfg, concurrency: int, prompt: int, steps: int, warmup: int = 4, budget: int = 8192) -> dict:
+    """Prefill and decode rates of a random model through the serving engine."""
+    import gc
+    import time
+
+    import numpy as np
+
+    from ..executor.gpu_executor import GpuExecutor
+    from ..models import registry
+    from ..runtime.engine import LLMEngine
+    from ..runtime.scheduler import SamplingParams, SchedulerConfig
+    dev = torch.device("cuda", torch.cuda.current_device())
+    defn = registry.get(cfg.family)
+    weights = defn.random_weights(cfg, dev, 0)
+    max_len = prompt + steps + warmup + 24
+    pages = concurrency * (-(-max_len // 16)) + 8
+    runner = defn.build_runner(cfg, weights, num_pages=pages, max_tokens=budget, max_requests=concurrency)
+    ex = GpuExecutor(runner, max_rows=concurrency, max_prefill_tokens=budget, max_model_len=max_len)
+    ex.capture_decode_graphs([concurrency])
+    ex.timing = True
+    eng = LLMEngine(ex, num_pages=pages, scheduler_config=SchedulerConfig(
+        max_running_requests=concurrency, max_batched_tokens=budget, prefill_chunk_tokens=budget, max_model_len=max_len,
+        enable_prefix_cache=False))
+    rng = np.random.default_rng(1)
+    rates = []
+    for turn in range(2):                              # the first turn warms the prefill path up
+        for p in rng.integers(0, cfg.vocab_size, size=(concurrency, prompt)).tolist():
+            eng.add_request(p, SamplingParams(max_tokens=steps + warmup + 8, ignore_eos=True))
+        ex.device_ms = []
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        while any(r.remaining > 1 for r in eng.scheduler.running + eng.scheduler.waiting) or eng.scheduler.waiting:
+            eng.step()
+        torch.cuda.synchronize()
+        rates.append((concurrency * prompt / (sum(ex.device_ms) / 1e3), concurrency * prompt / (time.perf_counter() - t0)))
+        for _ in range(warmup):
+            eng.step()
+        ex.device_ms = []
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        emitted = sum(len(eng.step()) for _ in range(steps))
+        torch.cuda.synchronize()
+        wall = time.perf_counter() - t0
+        ms = sorted(ex.device_ms)
+        launches = ex.kernel_launches_last
+        while eng.has_unfinished:                      # a few more tokens end every request
+            eng.step()
+    runner.ws.check_status()
+    out = {"model": cfg.name, "layers": cfg.num_layers, "weights_gb": round(weights.nbytes() / 1e9, 2), "concurrency": concurrency,
+           "prompt": prompt, "prefill_tok_s_device": round(rates[-1][0]), "prefill_tok_s_wall": round(rates[-1][1]),
+           "decode_ms_per_step": round(ms[len(ms) // 2], 3), "decode_tok_s_device": round(concurrency / ms[len(ms) // 2] * 1e3),
+           "decode_tok_s_wall": round(emitted / wall), "launches_per_decode_step": launches}
+    del eng, ex, runner, weights
+    gc.collect()
+    torch.cuda.empty_cache()
+    return out
+
+
+def run(steps: int = 32) -> None:
+    """Prints one JSON line per measurement."""
+    for line in kernels():
+        print(json.dumps(line), flush=True)
+    for width, layers in ((2048, 8), (4096, 8)):
+        for concurrency, prompt in ((1, 4096), (16, 1024), (256, 1024)):
+            for cfg in (layered_config(width, layers), hybrid_config(width, layers)):
+                print(json.dumps(model_throughput(cfg, concurrency, prompt, steps)), flush=True)

@@ -1,364 +1,467 @@
 // Gated delta rule layers of any head size, with one decay per head or one per key channel, and the short causal
 // convolution in front of them (the fixed 128 x 128, four-tap form of the hybrid family is gdn.cu).
 //
-//   conv_silu_kernel     depthwise causal convolution of any number of taps + SiLU; token tiles run in parallel, the
-//                        last taps - 1 inputs of every channel are the request's convolution state
-//   delta_rule_kernel    per (head, segment, slice of value rows): unit q / k, beta = sigmoid(b),
-//                        g = exp(-exp(A_log) softplus(a + dt_bias)) per head or per (head, key channel), then per token
-//                            S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
-//                        and the gated RMS norm of a head's output
-//   gated_norm_kernel    that norm as a kernel of its own, when a head's value rows are split over several blocks
+//   delta_prepare_kernel  everything of a token that does not depend on the state, all tokens in parallel: depthwise
+//                         causal convolution of any number of taps + SiLU, unit q / k and k . q,
+//                         beta = sigmoid(b), g = exp(-exp(A_log) softplus(a + dt_bias)) per head or per key channel;
+//                         the last taps - 1 inputs of every channel are the request's convolution state
+//   delta_walk_kernel     the recurrence, per (head, segment, slice of value rows), token by token:
+//                             S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   delta_step_kernel     the same for segments of one token (decode), with the gated RMS norm of the head's output
+//   gated_norm_kernel     that norm as a kernel of its own
 //
 // S^T q is taken from the decayed state before the write: o = S^T q + (k . q) u, so that both reductions over the key
 // channels of a token happen at once.  The state [slot][head][value row][key channel] is fp32 and stays in registers for
-// a whole segment; all arithmetic is fp32.  Only the projections and the convolution's outputs have the activation type.
+// a whole segment; everything is computed in fp32 and what passes between the kernels is fp32, except the value rows,
+// which keep the activation type.
 #include "segments.cuh"
 #include "launch.cuh"
 
 namespace cb {
-
-// ------------------------------------------------------------------ short convolution
-static constexpr int kConvRows = 16;       // tokens per block
-static constexpr int kConvThreads = 128;   // two channels per thread
 
 template <typename T> struct Pair2;
 template <> struct Pair2<__nv_bfloat16> { using type = __nv_bfloat162; };
 template <> struct Pair2<float> { using type = float2; };
 __device__ __forceinline__ float2 to_f2(__nv_bfloat162 v) { return __bfloat1622float2(v); }
 __device__ __forceinline__ float2 to_f2(float2 v) { return v; }
-__device__ __forceinline__ void store2(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __float22bfloat162_rn(v); }
-__device__ __forceinline__ void store2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float softplus_of(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float gate_of(float z, int sigmoid) { return (sigmoid ? 1.f : z) / (1.f + expf(-z)); }
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return __ffma2_rn(a, b, c); }
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) { return __fmul2_rn(a, b); }
 
-// The block that holds a segment's first tokens also replaces the convolution state: it is the only one that reads it.
-template <typename T, int TAPS>
-__global__ void __launch_bounds__(kConvThreads)
-conv_silu_kernel(const T* __restrict__ x, int ldx, T* __restrict__ y, int ldy, const float* __restrict__ w,   // [C, TAPS]
-                 T* __restrict__ state,                                                                       // [slots, TAPS - 1, C]
-                 Segments sg, int C) {
-  using P = typename Pair2<T>::type;
-  pdl_wait();
-  pdl_launch_dependents();
-  int s, off;
-  if (!find_tile(sg, kConvRows, blockIdx.y, s, off)) return;
-  const int c = (blockIdx.x * kConvThreads + threadIdx.x) * 2;
-  if (c >= C) return;
-  const int n = sg.count[s];
-  const T* xp = x + static_cast<size_t>(sg.row0[s]) * ldx + c;
-  T* yp = y + static_cast<size_t>(sg.row0[s]) * ldy + c;
-  float2 wv[TAPS];
-#pragma unroll
-  for (int j = 0; j < TAPS; ++j) wv[j] = make_float2(w[static_cast<size_t>(c) * TAPS + j], w[static_cast<size_t>(c + 1) * TAPS + j]);
-  constexpr int H = TAPS - 1;
-  float2 hist[H > 0 ? H : 1];               // inputs at t - H .. t - 1
-  T* st = state + static_cast<size_t>(sg.slot[s]) * H * C + c;
-  if (off == 0) {
-    const bool fresh = sg.pos0[s] == 0;
-#pragma unroll
-    for (int j = 0; j < H; ++j)
-      hist[j] = fresh ? make_float2(0.f, 0.f) : to_f2(*reinterpret_cast<const P*>(st + static_cast<size_t>(j) * C));
-    // new state: inputs n - H .. n - 1, where negative indices are entries of the old state
-#pragma unroll
-    for (int j = 0; j < H; ++j) {
-      const int t = n - H + j;
-      float2 v = make_float2(0.f, 0.f);
-      if (t >= 0) {
-        v = to_f2(*reinterpret_cast<const P*>(xp + static_cast<size_t>(t) * ldx));
-      } else {
-#pragma unroll
-        for (int i = 0; i < H; ++i) if (i == t + H) v = hist[i];
-      }
-      store2(st + static_cast<size_t>(j) * C, v);
-    }
-  } else {
-#pragma unroll
-    for (int j = 0; j < H; ++j) {            // a tile that is not the first starts at least kConvRows >= H tokens in
-      hist[j] = to_f2(*reinterpret_cast<const P*>(xp + static_cast<size_t>(off - H + j) * ldx));
-    }
-  }
-  const int end = min(n, off + kConvRows);
-#pragma unroll 4
-  for (int t = off; t < end; ++t) {
-    const float2 v = to_f2(*reinterpret_cast<const P*>(xp + static_cast<size_t>(t) * ldx));
-    float2 a = make_float2(wv[H].x * v.x, wv[H].y * v.y);
-#pragma unroll
-    for (int j = 0; j < H; ++j) { a.x = fmaf(wv[j].x, hist[j].x, a.x); a.y = fmaf(wv[j].y, hist[j].y, a.y); }
-    store2(yp + static_cast<size_t>(t) * ldy, make_float2(silu_exact(a.x), silu_exact(a.y)));
-#pragma unroll
-    for (int j = 0; j + 1 < H; ++j) hist[j] = hist[j + 1];
-    if (H > 0) hist[H - 1] = v;
-  }
-}
+// ------------------------------------------------------------------ preparation
+static constexpr int kPrepRows = 16;       // tokens per warp
+static constexpr int kPrepWarps = 4;
 
-// ------------------------------------------------------------------ delta rule
 template <typename T>
-struct DeltaRule {
-  const T* qkv; int ldq;      // after the convolution: q [G d] | k [G d] | v [H e]
+struct DeltaPrep {
+  const T* x; int ldx;        // projections before the convolution: q [G d] | k [G d] | v [H e]
   const T* b; int ldb;        // [H] step size logits
   const T* a; int lda;        // decay logits: [H] or [H d]
-  const T* z; int ldz;        // output gate [H e]
+  const float* w;             // [taps][ldw] convolution weights, the last row multiplies the current input
+  int ldw, taps;
+  T* state;                   // [slots, taps - 1, ldw]
   const float* a_log;         // [H]
   const float* dt_bias;       // [H] or [H d]
-  const float* norm_w;        // [e]
-  float* state;               // [slots, H, e, ds]
-  T* out; int ldo;            // [H e]
-  float* raw;                 // fp32 [T, H e]: outputs before the norm (value rows split over blocks), or null
-  int H, G, d, e, ds;         // ds: row stride of the state, d rounded up to 4
-  float eps;
-  int sigmoid_gate;           // output gate sigmoid(z) instead of silu(z)
+  float* q;                   // [T, G, ds] unit queries times d^-1/2
+  float* k;                   // [T, G, ds] unit keys
+  float* kq;                  // [T, G]
+  T* v;                       // [T, H, es]
+  float2* coef;               // [T, H] {beta, decay per head (1 with channel decays)}
+  float* g;                   // [T, H, ds] channel decays or null
+  int H, G, d, e, ds, es;
   Segments sg;
 };
 
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return __ffma2_rn(a, b, c); }
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) { return __fmul2_rn(a, b); }
-__device__ __forceinline__ float gate_of(float z, int sigmoid) { return (sigmoid ? 1.f : z) / (1.f + expf(-z)); }
-__device__ __forceinline__ float softplus_of(float x) { return x > 20.f ? x + log1pf(expf(-x)) : log1pf(expf(x)); }
+// The convolution of `NP` channel pairs (c0 + 64 i, + 1) of token t, one lane; pairs at or behind `lim` read as zero.
+// `odd`: heads of odd width, whose channels are read one at a time.
+template <typename T, int NP>
+__device__ __forceinline__ void conv_pairs(const DeltaPrep<T>& p, const T* xr, const T* st, bool fresh, int t, int c0, int base,
+                                           int lim, bool odd, float2 (&out)[NP]) {
+  using P = typename Pair2<T>::type;
+#pragma unroll
+  for (int i = 0; i < NP; ++i) out[i] = make_float2(0.f, 0.f);
+  const int H = p.taps - 1;
+#pragma unroll 1
+  for (int j = 0; j < p.taps; ++j) {
+    const int tt = t - H + j;
+    if (tt < 0 && fresh) continue;
+    const T* src = (tt >= 0 ? xr + static_cast<ptrdiff_t>(tt) * p.ldx : st + static_cast<ptrdiff_t>(tt + H) * p.ldw) + base;
+    const float* wr = p.w + static_cast<size_t>(j) * p.ldw + base;
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      const int c = c0 + 64 * i;
+      if (c >= lim) continue;
+      float2 v, w;
+      if (!odd) {
+        v = to_f2(*reinterpret_cast<const P*>(src + c));
+        w = *reinterpret_cast<const float2*>(wr + c);
+      } else {
+        v = make_float2(to_f(src[c]), c + 1 < lim ? to_f(src[c + 1]) : 0.f);
+        w = make_float2(wr[c], c + 1 < lim ? wr[c + 1] : 0.f);
+      }
+      out[i] = fma2(w, v, out[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NP; ++i) out[i] = make_float2(silu_exact(out[i].x), silu_exact(out[i].y));
+}
 
-// KD: key channels covered by a row's lanes (d <= KD).  LPR = KD / 16 lanes share a state row, lane l holds the float4
-// chunks l + LPR c (c < 4); a thread holds RPT rows.  NB tokens are prepared at a time.
-//
-// PIPE: the block has kPrepWarps more warps that prepare the operands of the next NB tokens and normalise the outputs
-// of the previous NB while the other warps walk the recurrence (two shared-memory buffers, one barrier per NB tokens).
-// Without it (decode: one token per segment) all warps do both in turn, and two blocks share an SM so that one's
-// state traffic overlaps the other's arithmetic.
-static constexpr int kPrepWarps = 8;
+// The convolution state of channels [base, base + n) becomes the segment's last taps - 1 inputs.  Called after the
+// outputs that need the old state, by the warp that produced them; a lane touches the same channels in both.
+template <typename T>
+__device__ __forceinline__ void conv_state(const DeltaPrep<T>& p, const T* xr, T* st, bool fresh, int count, int base, int n) {
+  const int H = p.taps - 1;
+  for (int c = threadIdx.x & 31; c < n; c += 32)
+    for (int j = 0; j < H; ++j) {            // entry j moves down from entry j + count, which is read before it is written
+      const int t = count - H + j;
+      T v = from_f<T>(0.f);
+      if (t >= 0) v = xr[static_cast<ptrdiff_t>(t) * p.ldx + base + c];
+      else if (!fresh) v = st[static_cast<ptrdiff_t>(t + H) * p.ldw + base + c];
+      st[static_cast<ptrdiff_t>(j) * p.ldw + base + c] = v;
+    }
+}
 
-template <int KD> struct DeltaShape {
-  static constexpr int LPR = KD / 16;
-  static constexpr int NB = KD <= 128 ? 16 : 8;
-  static constexpr int kMaxRowThreads = 256;
+// A warp per (head slot, tile of kPrepRows tokens): slots [0, G) are key heads (q and k), slots [G, G + H) value heads
+// (v, step size, decays).  NP: channel pairs per lane of a key head (d <= 64 NP).
+template <typename T, int NP>
+__global__ void __launch_bounds__(32 * kPrepWarps)
+delta_prepare_kernel(const DeltaPrep<T> p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  int s, off;
+  if (!find_tile(p.sg, kPrepRows, blockIdx.y, s, off)) return;
+  const int slot = blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (slot >= p.G + p.H) return;
+  const int count = p.sg.count[s], end = min(count, off + kPrepRows);
+  const bool fresh = p.sg.pos0[s] == 0;
+  const size_t row0 = p.sg.row0[s];
+  const T* xr = p.x + row0 * p.ldx;
+  T* st = p.state + static_cast<size_t>(p.sg.slot[s]) * (p.taps - 1) * p.ldw;
+  if (slot < p.G) {
+    const int qb = slot * p.d, kb = (p.G + slot) * p.d;
+    const bool odd = p.d & 1;
+    const float scale = 1.f / sqrtf(static_cast<float>(p.d));
+    for (int t = off; t < end; ++t) {
+      float2 q[NP], k[NP];
+      conv_pairs<T, NP>(p, xr, st, fresh, t, 2 * lane, qb, p.d, odd, q);
+      conv_pairs<T, NP>(p, xr, st, fresh, t, 2 * lane, kb, p.d, odd, k);
+      float qq = 0.f, kk = 0.f, qk = 0.f;
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        qq = fmaf(q[i].x, q[i].x, qq); qq = fmaf(q[i].y, q[i].y, qq);
+        kk = fmaf(k[i].x, k[i].x, kk); kk = fmaf(k[i].y, k[i].y, kk);
+        qk = fmaf(q[i].x, k[i].x, qk); qk = fmaf(q[i].y, k[i].y, qk);
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        qq += __shfl_xor_sync(0xffffffffu, qq, o);
+        kk += __shfl_xor_sync(0xffffffffu, kk, o);
+        qk += __shfl_xor_sync(0xffffffffu, qk, o);
+      }
+      const float qi = 1.f / sqrtf(qq + 1e-6f) * scale, ki = 1.f / sqrtf(kk + 1e-6f);
+      const size_t o = ((row0 + t) * p.G + slot) * p.ds;
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        const int c = 2 * lane + 64 * i;             // columns [d, ds) get zeros
+        if (c < p.ds) {
+          *reinterpret_cast<float2*>(p.q + o + c) = make_float2(q[i].x * qi, q[i].y * qi);
+          *reinterpret_cast<float2*>(p.k + o + c) = make_float2(k[i].x * ki, k[i].y * ki);
+        }
+      }
+      if (lane == 0) p.kq[(row0 + t) * p.G + slot] = qk * qi * ki;
+    }
+    if (off == 0) {
+      __syncwarp();                                  // read in pairs, replaced channel by channel
+      conv_state(p, xr, st, fresh, count, qb, p.d);
+      conv_state(p, xr, st, fresh, count, kb, p.d);
+    }
+    return;
+  }
+  const int h = slot - p.G, vb = 2 * p.G * p.d + h * p.e;
+  const bool odd = (p.e & 1) || (vb & 1);
+  for (int t = off; t < end; ++t)
+    for (int c = 2 * lane; c < p.e; c += 64) {
+      float2 v[1];
+      conv_pairs<T, 1>(p, xr, st, fresh, t, c, vb, p.e, odd, v);
+      T* dst = p.v + ((row0 + t) * p.H + h) * p.es + c;        // es is even: the pair's second column exists
+      dst[0] = from_f<T>(v[0].x);
+      dst[1] = from_f<T>(v[0].y);
+    }
+  const float rate = -expf(p.a_log[h]);
+  if (off + lane < end && lane < kPrepRows) {
+    const size_t r = row0 + off + lane;
+    const float beta = 1.f / (1.f + expf(-to_f(p.b[r * p.ldb + h])));
+    const float decay = p.g ? 1.f : expf(rate * softplus_of(to_f(p.a[r * p.lda + h]) + p.dt_bias[h]));
+    p.coef[r * p.H + h] = make_float2(beta, decay);
+  }
+  if (p.g)
+    for (int t = off; t < end; ++t)
+      for (int c = lane; c < p.ds; c += 32)
+        p.g[((row0 + t) * p.H + h) * p.ds + c] =
+            c < p.d ? expf(rate * softplus_of(to_f(p.a[(row0 + t) * p.lda + h * p.d + c]) + p.dt_bias[h * p.d + c])) : 0.f;
+  if (off == 0) {
+    __syncwarp();
+    conv_state(p, xr, st, fresh, count, vb, p.e);
+  }
+}
+
+// ------------------------------------------------------------------ recurrence
+template <typename T>
+struct DeltaWalk {
+  const float* q; const float* k; const float* kq;
+  const T* v; const float2* coef; const float* g;     // as written by the preparation
+  const T* z; int ldz;                                // output gate [H e] (delta_step_kernel)
+  const float* norm_w;                                // [e]
+  float* state;                                       // [slots, H, e, ds]
+  T* out; int ldo;                                    // [H e]
+  float* raw;                                         // fp32 [T, H e]: outputs before the norm, or null
+  int H, G, d, e, ds, es;
+  float eps;
+  int sigmoid_gate;                                   // output gate sigmoid(z) instead of silu(z)
+  Segments sg;
 };
 
-template <typename T, int KD, int RPT, bool CHANNEL, bool PIPE>
-__global__ void __launch_bounds__(PIPE ? 256 + 32 * kPrepWarps : 256, PIPE ? 1 : 2)
-delta_rule_kernel(const DeltaRule<T> p) {
-  constexpr int LPR = DeltaShape<KD>::LPR, NB = PIPE ? DeltaShape<KD>::NB : 1;
-  constexpr int KV = KD / 32;
-  constexpr int OPS = CHANNEL ? 3 : 2;                    // q, k (, g) rows per token
+// KD: key channels covered by a row's lanes (d <= KD).  LPR = KD / 16 lanes share a state row, lane l holds the float4
+// chunks l + LPR c (c < 4); a thread holds RPT rows.
+template <int KD> struct DeltaShape {
+  static constexpr int LPR = KD / 16;
+  static constexpr int NB = KD <= 128 ? 16 : 8;       // tokens staged at a time
+};
+
+template <int LPR, int RPT>
+__device__ __forceinline__ void load_state(const float* sp, int ds, int e, int v_first, int v_step, int l, bool use, float2 (&S)[RPT][8]) {
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) {
+    const int v = v_first + i * v_step;
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const int col = 4 * (l + LPR * c);
+      float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (use && v < e && col < ds) t = *reinterpret_cast<const float4*>(sp + static_cast<size_t>(v) * ds + col);
+      S[i][2 * c] = make_float2(t.x, t.y);
+      S[i][2 * c + 1] = make_float2(t.z, t.w);
+    }
+  }
+}
+template <int LPR, int RPT>
+__device__ __forceinline__ void store_state(float* sp, int ds, int e, int v_first, int v_step, int l, const float2 (&S)[RPT][8]) {
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) {
+    const int v = v_first + i * v_step;
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const int col = 4 * (l + LPR * c);
+      if (v < e && col < ds)
+        *reinterpret_cast<float4*>(sp + static_cast<size_t>(v) * ds + col) =
+            make_float4(S[i][2 * c].x, S[i][2 * c].y, S[i][2 * c + 1].x, S[i][2 * c + 1].y);
+    }
+  }
+}
+
+// One token: decays the state, updates it with (k, v) and returns the outputs of the thread's rows (the same value in
+// all lanes of a row).  `get(which, c)` yields the float4 chunk c of q (0), k (1), g (2).
+template <int LPR, int RPT, bool CHANNEL, typename Get>
+__device__ __forceinline__ void delta_token(float2 (&S)[RPT][8], Get get, float beta, float decay, float kq,
+                                            const float (&va)[RPT], float (&o)[RPT]) {
+  float2 k2[8], aa[RPT], bb[RPT];
+  const float2 g1 = make_float2(decay, decay);
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) { aa[i] = make_float2(0.f, 0.f); bb[i] = make_float2(0.f, 0.f); }
+#pragma unroll
+  for (int c = 0; c < 4; ++c) {
+    const float4 q4 = get(0, c), k4 = get(1, c);
+    float2 ga = g1, gb = g1;
+    if constexpr (CHANNEL) {
+      const float4 g4 = get(2, c);
+      ga = make_float2(g4.x, g4.y);
+      gb = make_float2(g4.z, g4.w);
+    }
+    k2[2 * c] = make_float2(k4.x, k4.y);
+    k2[2 * c + 1] = make_float2(k4.z, k4.w);
+    const float2 q0 = make_float2(q4.x, q4.y), q1 = make_float2(q4.z, q4.w);
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      S[i][2 * c] = mul2(S[i][2 * c], ga);
+      S[i][2 * c + 1] = mul2(S[i][2 * c + 1], gb);
+      aa[i] = fma2(S[i][2 * c], k2[2 * c], aa[i]);
+      bb[i] = fma2(S[i][2 * c], q0, bb[i]);
+      aa[i] = fma2(S[i][2 * c + 1], k2[2 * c + 1], aa[i]);
+      bb[i] = fma2(S[i][2 * c + 1], q1, bb[i]);
+    }
+  }
+  float sa[RPT];
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) { sa[i] = aa[i].x + aa[i].y; o[i] = bb[i].x + bb[i].y; }
+#pragma unroll
+  for (int sh = 1; sh < LPR; sh <<= 1)
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      sa[i] += __shfl_xor_sync(0xffffffffu, sa[i], sh);
+      o[i] += __shfl_xor_sync(0xffffffffu, o[i], sh);
+    }
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) {
+    const float u = beta * (va[i] - sa[i]);
+    o[i] = fmaf(kq, u, o[i]);
+    const float2 u2 = make_float2(u, u);
+#pragma unroll
+    for (int c = 0; c < 8; ++c) S[i][c] = fma2(k2[c], u2, S[i][c]);
+  }
+}
+
+template <int B>
+__device__ __forceinline__ void cp_async(void* dst, const void* src) {
+  if constexpr (B == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"(B) : "memory");
+}
+
+// Segments of many tokens: NB tokens' operands arrive by cp.async while the previous NB are walked; one barrier per NB
+// tokens.  Outputs leave through shared memory, before the norm.
+template <typename T, int KD, int RPT, bool CHANNEL>
+__global__ void __launch_bounds__(256, 2)
+delta_walk_kernel(const DeltaWalk<T> p) {
+  constexpr int LPR = DeltaShape<KD>::LPR, NB = DeltaShape<KD>::NB, OPS = CHANNEL ? 3 : 2;
   extern __shared__ __align__(16) float sm[];
   pdl_wait();
   pdl_launch_dependents();
   const int head = blockIdx.x, s = blockIdx.y;
   const int n = p.sg.count[s];
   if (n <= 0) return;
-  const int row_threads = PIPE ? blockDim.x - 32 * kPrepWarps : blockDim.x;
-  const int VT = row_threads / LPR * RPT;                 // value rows of this block
-  const int v0 = blockIdx.z * VT;
-  const int e_here = min(VT, p.e - v0);
-  const int buf_floats = NB * (OPS * KD + VT + 4);
-  float* const obuf = sm + (PIPE ? 2 : 1) * buf_floats;   // [PIPE ? 2 : 1][NB][VT]
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const bool rower = tid < row_threads;
-  const int l = tid % LPR, grp = tid / LPR, ngrp = row_threads / LPR;
+  const int VT = blockDim.x / LPR * RPT;              // value rows of this block
+  const int v0 = blockIdx.z * VT, e_here = min(VT, p.e - v0);
+  const int es = p.es;
+  // per buffer: operands [OPS][NB][KD], coefficients [NB] float4, value rows [NB][es] (the whole head's, T)
+  const int buf_floats = NB * (OPS * KD + 4) + NB * es * static_cast<int>(sizeof(T)) / 4;
+  float* const obuf = sm + 2 * buf_floats;            // [2][NB][VT]
+  const int tid = threadIdx.x;
+  const int l = tid % LPR, grp = tid / LPR, ngrp = blockDim.x / LPR;
   const size_t row0 = p.sg.row0[s];
   const int hq = head / (p.H / p.G);
-  const float rate = -expf(p.a_log[head]);
-
-  // the state's loads are issued first: their latency covers the preparation of the first tokens
   float* sp = p.state + (static_cast<size_t>(p.sg.slot[s]) * p.H + head) * p.e * p.ds;
   float2 S[RPT][8];
-  const bool fresh = p.sg.pos0[s] == 0;
-#pragma unroll
-  for (int i = 0; i < RPT; ++i) {
-    const int v = v0 + grp + i * ngrp;
-#pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      const int col = 4 * (l + LPR * c);
-      float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (rower && !fresh && v < p.e && col < p.ds) t = *reinterpret_cast<const float4*>(sp + static_cast<size_t>(v) * p.ds + col);
-      S[i][2 * c] = make_float2(t.x, t.y);
-      S[i][2 * c + 1] = make_float2(t.z, t.w);
+  load_state<LPR, RPT>(sp, p.ds, p.e, v0 + grp, ngrp, l, p.sg.pos0[s] != 0, S);
+
+  auto coefs = [&](int b) { return sm + b * buf_floats + NB * OPS * KD; };
+  auto values = [&](int b) { return reinterpret_cast<T*>(sm + b * buf_floats + NB * (OPS * KD + 4)); };
+  const int chunks = p.ds / 4, vchunks = es * static_cast<int>(sizeof(T)) / 16;
+  auto fetch = [&](int blk) {
+    const int t0 = blk * NB, nb = min(NB, n - t0), b = blk & 1;
+    float* buf = sm + b * buf_floats;
+    for (int i = tid; i < nb * chunks; i += blockDim.x) {
+      const int j = i / chunks, c = (i - j * chunks) * 4;
+      const size_t r = row0 + t0 + j;
+      cp_async<16>(buf + j * KD + c, p.q + (r * p.G + hq) * p.ds + c);
+      cp_async<16>(buf + (NB + j) * KD + c, p.k + (r * p.G + hq) * p.ds + c);
+      if constexpr (CHANNEL) cp_async<16>(buf + (2 * NB + j) * KD + c, p.g + (r * p.H + head) * p.ds + c);
     }
-  }
-
-  auto bufq = [&](int b) { return sm + b * buf_floats; };
-  auto bufc = [&](int b) { return sm + b * buf_floats + NB * OPS * KD; };          // float4 per token: 16-byte aligned
-  auto bufv = [&](int b) { return sm + b * buf_floats + NB * (OPS * KD + 4); };
-
-  // operands of token t (of the segment) into slot j of buffer b: `part` 0 unit q and k, beta, k . q, scalar decay;
-  // 1 the value rows; 2 the channel decays
-  auto prep = [&](int t, int j, int b, int part) {
-    const size_t r = row0 + t;
-    const T* row = p.qkv + r * p.ldq;
-    if (part == 0) {
-      float q[KV], k[KV];
-#pragma unroll
-      for (int i = 0; i < KV; ++i) {
-        const int c = lane + 32 * i;
-        q[i] = c < p.d ? to_f(row[hq * p.d + c]) : 0.f;
-        k[i] = c < p.d ? to_f(row[(p.G + hq) * p.d + c]) : 0.f;
-      }
-      const float bl = to_f(p.b[r * p.ldb + head]);
-      const float al = CHANNEL ? 0.f : to_f(p.a[r * p.lda + head]) + p.dt_bias[head];
-      float qq = 0.f, kk = 0.f, qk = 0.f;
-#pragma unroll
-      for (int i = 0; i < KV; ++i) { qq = fmaf(q[i], q[i], qq); kk = fmaf(k[i], k[i], kk); }
-      qq = warp_sum(qq);
-      kk = warp_sum(kk);
-      const float qi = 1.f / sqrtf(qq + 1e-6f) * (1.f / sqrtf(static_cast<float>(p.d))), ki = 1.f / sqrtf(kk + 1e-6f);
-      float* qs = bufq(b) + j * KD;
-      float* ks = qs + NB * KD;
-#pragma unroll
-      for (int i = 0; i < KV; ++i) {
-        q[i] *= qi;
-        k[i] *= ki;
-        qs[lane + 32 * i] = q[i];
-        ks[lane + 32 * i] = k[i];
-        qk = fmaf(q[i], k[i], qk);
-      }
-      qk = warp_sum(qk);
-      if (lane == 0)
-        *reinterpret_cast<float4*>(bufc(b) + j * 4) =
-            make_float4(1.f / (1.f + expf(-bl)), CHANNEL ? 1.f : expf(rate * softplus_of(al)), qk, 0.f);
-    } else if (part == 1) {
-      float* vs = bufv(b) + j * VT;
-      const T* vr = row + 2 * p.G * p.d + head * p.e + v0;
-      for (int c = lane; c < e_here; c += 32) vs[c] = to_f(vr[c]);
-    } else {
-      float* gs = bufq(b) + (2 * NB + j) * KD;
-      const T* ar = p.a + r * p.lda + head * p.d;
-#pragma unroll
-      for (int i = 0; i < KV; ++i) {
-        const int c = lane + 32 * i;
-        gs[c] = c < p.d ? expf(rate * softplus_of(to_f(ar[c]) + p.dt_bias[head * p.d + c])) : 0.f;
-      }
+    T* vs = values(b);
+    for (int i = tid; i < nb * vchunks; i += blockDim.x) {
+      const int j = i / vchunks, c = (i - j * vchunks) * (16 / static_cast<int>(sizeof(T)));
+      cp_async<16>(vs + j * es + c, p.v + ((row0 + t0 + j) * p.H + head) * es + c);
+    }
+    if (tid < nb) {
+      const size_t r = row0 + t0 + tid;
+      cp_async<8>(coefs(b) + tid * 4, p.coef + r * p.H + head);
+      cp_async<4>(coefs(b) + tid * 4 + 2, p.kq + r * p.G + hq);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // columns [ds, KD) of the operand rows are never fetched: zero once
+  if (p.ds < KD)
+    for (int i = tid; i < 2 * OPS * NB * (KD - p.ds); i += blockDim.x) {
+      const int rowi = i / (KD - p.ds), c = p.ds + i % (KD - p.ds);
+      (sm + (rowi / (OPS * NB)) * buf_floats)[(rowi % (OPS * NB)) * KD + c] = 0.f;
+    }
+  auto put = [&](int blk) {                           // outputs of block blk to memory
+    const int t0 = blk * NB, nb = min(NB, n - t0);
+    const float* ob = obuf + (blk & 1) * NB * VT;
+    for (int i = tid; i < nb * VT; i += blockDim.x) {
+      const int j = i / VT, v = i - j * VT;
+      if (v < e_here) p.raw[(row0 + t0 + j) * (static_cast<size_t>(p.H) * p.e) + head * p.e + v0 + v] = ob[i];
     }
   };
-
-  // gated norm of token t's outputs (slot j of buffer b), or their raw store when the head is split
-  auto finish = [&](int t, int j, int b) {
-    const float* o = obuf + (b * NB + j) * VT;
-    const size_t r = row0 + t;
-    if (p.raw) {
-      float* dst = p.raw + r * (static_cast<size_t>(p.H) * p.e) + head * p.e + v0;
-      for (int c = lane; c < e_here; c += 32) dst[c] = o[c];
-      return;
-    }
-    float ss = 0.f;
-    for (int c = lane; c < p.e; c += 32) ss = fmaf(o[c], o[c], ss);
-    const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.e) + p.eps);
-    const T* zr = p.z + r * p.ldz + head * p.e;
-    T* dst = p.out + r * p.ldo + head * p.e;
-    for (int c = lane; c < p.e; c += 32)
-      dst[c] = from_f<T>(o[c] * inv * p.norm_w[c] * gate_of(to_f(zr[c]), p.sigmoid_gate));
-  };
-
-  // the recurrence over nb tokens of buffer b
-  auto walk = [&](int nb, int b) {
-    const float* qb = bufq(b);
-    const float* vb = bufv(b);
-    const float* cb_ = bufc(b);
-    float* ob = obuf + b * NB * VT;
+  const int blocks = (n + NB - 1) / NB;
+  fetch(0);
+  for (int blk = 0; blk < blocks; ++blk) {
+    const int b = blk & 1, nb = min(NB, n - blk * NB);
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    __syncthreads();                                  // operands of blk are here; everybody has left blk - 1
+    if (blk + 1 < blocks) fetch(blk + 1);
+    if (blk > 0) put(blk - 1);
+    const float* buf = sm + b * buf_floats;
+    const float* cf = coefs(b);
+    const T* vs = values(b) + v0 + grp;
+    float* ob = obuf + b * NB * VT + grp;
 #pragma unroll 1
     for (int j = 0; j < nb; ++j) {
-      const float4 co = *reinterpret_cast<const float4*>(cb_ + j * 4);
-      const float2 g1 = make_float2(co.y, co.y);
-      float2 k2[8], aa[RPT], bb[RPT];
-      float va[RPT];
+      const float4 co = *reinterpret_cast<const float4*>(cf + j * 4);
+      float va[RPT], o[RPT];
 #pragma unroll
-      for (int i = 0; i < RPT; ++i) {
-        aa[i] = make_float2(0.f, 0.f);
-        bb[i] = make_float2(0.f, 0.f);
-        va[i] = vb[j * VT + grp + i * ngrp];
+      for (int i = 0; i < RPT; ++i) va[i] = v0 + grp + i * ngrp < p.e ? to_f(vs[j * es + i * ngrp]) : 0.f;
+      delta_token<LPR, RPT, CHANNEL>(
+          S, [&](int w, int c) { return *reinterpret_cast<const float4*>(buf + (w * NB + j) * KD + 4 * (l + LPR * c)); },
+          co.x, co.y, co.z, va, o);
+      if (l == 0) {
+#pragma unroll
+        for (int i = 0; i < RPT; ++i) ob[j * VT + i * ngrp] = o[i];
       }
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const int col = 4 * (l + LPR * c);
-        const float4 q4 = *reinterpret_cast<const float4*>(qb + j * KD + col);
-        const float4 k4 = *reinterpret_cast<const float4*>(qb + (NB + j) * KD + col);
-        float2 ga = g1, gb = g1;
-        if constexpr (CHANNEL) {
-          const float4 g4 = *reinterpret_cast<const float4*>(qb + (2 * NB + j) * KD + col);
-          ga = make_float2(g4.x, g4.y);
-          gb = make_float2(g4.z, g4.w);
-        }
-        k2[2 * c] = make_float2(k4.x, k4.y);
-        k2[2 * c + 1] = make_float2(k4.z, k4.w);
-        const float2 q0 = make_float2(q4.x, q4.y), q1 = make_float2(q4.z, q4.w);
-#pragma unroll
-        for (int i = 0; i < RPT; ++i) {
-          S[i][2 * c] = mul2(S[i][2 * c], ga);
-          S[i][2 * c + 1] = mul2(S[i][2 * c + 1], gb);
-          aa[i] = fma2(S[i][2 * c], k2[2 * c], aa[i]);
-          bb[i] = fma2(S[i][2 * c], q0, bb[i]);
-          aa[i] = fma2(S[i][2 * c + 1], k2[2 * c + 1], aa[i]);
-          bb[i] = fma2(S[i][2 * c + 1], q1, bb[i]);
-        }
-      }
-      float sa[RPT], sb[RPT];
-#pragma unroll
-      for (int i = 0; i < RPT; ++i) { sa[i] = aa[i].x + aa[i].y; sb[i] = bb[i].x + bb[i].y; }
-#pragma unroll
-      for (int sh = 1; sh < LPR; sh <<= 1)
-#pragma unroll
-        for (int i = 0; i < RPT; ++i) {
-          sa[i] += __shfl_xor_sync(0xffffffffu, sa[i], sh);
-          sb[i] += __shfl_xor_sync(0xffffffffu, sb[i], sh);
-        }
-#pragma unroll
-      for (int i = 0; i < RPT; ++i) {
-        const float u = co.x * (va[i] - sa[i]);
-        if (l == 0) ob[j * VT + grp + i * ngrp] = fmaf(co.z, u, sb[i]);
-        const float2 u2 = make_float2(u, u);
-#pragma unroll
-        for (int c = 0; c < 8; ++c) S[i][c] = fma2(k2[c], u2, S[i][c]);
-      }
-    }
-  };
-
-  if constexpr (PIPE) {
-    const int pw = warp - (row_threads >> 5);
-    const int blocks = (n + NB - 1) / NB;
-    auto prep_block = [&](int blk) {
-      const int t0 = blk * NB, nb = min(NB, n - t0), b = blk & 1;
-      // a token per warp and turn, its parts back to back so that their loads are in flight together
-#pragma unroll 2
-      for (int j = pw; j < nb; j += kPrepWarps) {
-        prep(t0 + j, j, b, 0);
-        prep(t0 + j, j, b, 1);
-        if constexpr (CHANNEL) prep(t0 + j, j, b, 2);
-      }
-    };
-    auto finish_block = [&](int blk) {
-      const int t0 = blk * NB, nb = min(NB, n - t0);
-      for (int j = pw; j < nb; j += kPrepWarps) finish(t0 + j, j, blk & 1);
-    };
-    if (!rower) prep_block(0);
-    __syncthreads();
-    for (int blk = 0; blk < blocks; ++blk) {
-      if (rower) {
-        walk(min(NB, n - blk * NB), blk & 1);
-      } else {
-        if (blk > 0) finish_block(blk - 1);
-        if (blk + 1 < blocks) prep_block(blk + 1);
-      }
-      __syncthreads();
-    }
-    if (!rower) finish_block(blocks - 1);
-  } else {
-    const int nwarps = blockDim.x >> 5;
-    for (int t = 0; t < n; ++t) {
-      for (int part = warp; part < OPS; part += nwarps) prep(t, 0, 0, part);
-      __syncthreads();
-      walk(1, 0);
-      __syncthreads();
-      if (warp == 0) finish(t, 0, 0);
-      // the outputs of this token are read by warp 0 while the others prepare the next one; they are overwritten only
-      // after the next barrier
     }
   }
-  if (!rower) return;
+  __syncthreads();
+  put(blocks - 1);
+  store_state<LPR, RPT>(sp, p.ds, p.e, v0 + grp, ngrp, l, S);
+}
+
+// Segments of one token.  The state's loads go out first; the operands are a few cached rows.
+template <typename T, int KD, int RPT, bool CHANNEL>
+__global__ void __launch_bounds__(256, 2)
+delta_step_kernel(const DeltaWalk<T> p) {
+  constexpr int LPR = DeltaShape<KD>::LPR;
+  extern __shared__ __align__(16) float sm[];         // [VT]
+  __shared__ float red[8];
+  const int head = blockIdx.x, s = blockIdx.y, tid = threadIdx.x;
+  const int VT = blockDim.x / LPR * RPT, v0 = blockIdx.z * VT;
+  const int l = tid % LPR, grp = tid / LPR, ngrp = blockDim.x / LPR;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (p.sg.count[s] <= 0) return;
+  const size_t r = p.sg.row0[s];
+  const int hq = head / (p.H / p.G);
+  float* sp = p.state + (static_cast<size_t>(p.sg.slot[s]) * p.H + head) * p.e * p.ds;
+  float2 S[RPT][8];
+  load_state<LPR, RPT>(sp, p.ds, p.e, v0 + grp, ngrp, l, p.sg.pos0[s] != 0, S);
+  const float* qr = p.q + (r * p.G + hq) * p.ds;
+  const float* kr = p.k + (r * p.G + hq) * p.ds;
+  const float* gr = CHANNEL ? p.g + (r * p.H + head) * p.ds : nullptr;
+  const float2 co = p.coef[r * p.H + head];
+  const float kq = p.kq[r * p.G + hq];
+  float va[RPT], o[RPT];
 #pragma unroll
   for (int i = 0; i < RPT; ++i) {
     const int v = v0 + grp + i * ngrp;
+    va[i] = v < p.e ? to_f(p.v[(r * p.H + head) * p.es + v]) : 0.f;
+  }
+  delta_token<LPR, RPT, CHANNEL>(
+      S,
+      [&](int w, int c) {
+        const int col = 4 * (l + LPR * c);
+        const float* src = w == 0 ? qr : w == 1 ? kr : gr;
+        return col < p.ds ? *reinterpret_cast<const float4*>(src + col) : make_float4(0.f, 0.f, 0.f, 0.f);
+      },
+      co.x, co.y, kq, va, o);
+  store_state<LPR, RPT>(sp, p.ds, p.e, v0 + grp, ngrp, l, S);
+  if (p.raw) {
+    if (l == 0) {
 #pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      const int col = 4 * (l + LPR * c);
-      if (v < p.e && col < p.ds)
-        *reinterpret_cast<float4*>(sp + static_cast<size_t>(v) * p.ds + col) =
-            make_float4(S[i][2 * c].x, S[i][2 * c].y, S[i][2 * c + 1].x, S[i][2 * c + 1].y);
+      for (int i = 0; i < RPT; ++i)
+        if (v0 + grp + i * ngrp < p.e) p.raw[(r * p.H + head) * p.e + v0 + grp + i * ngrp] = o[i];
+    }
+    return;
+  }
+  // gated norm: the whole head is in this block
+  float ss = 0.f;
+  if (l == 0) {
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      const int v = grp + i * ngrp;
+      if (v < p.e) {
+        sm[v] = o[i];
+        ss = fmaf(o[i], o[i], ss);
+      }
     }
   }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+  for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) ss += red[w];
+  const float inv = 1.f / sqrtf(ss / static_cast<float>(p.e) + p.eps);
+  for (int v = tid; v < p.e; v += blockDim.x)
+    p.out[r * p.ldo + head * p.e + v] =
+        from_f<T>(sm[v] * inv * p.norm_w[v] * gate_of(to_f(p.z[r * p.ldz + head * p.e + v]), p.sigmoid_gate));
 }
 
 // out = raw / rms(raw) * norm_w * gate(z) per (token, head); a warp each.
@@ -374,81 +477,77 @@ gated_norm_kernel(const float* __restrict__ raw, const T* __restrict__ z, int ld
   const size_t t = static_cast<size_t>(item / H);
   const int h = static_cast<int>(item % H);
   const float* o = raw + static_cast<size_t>(item) * e;
-  float ss = 0.f;
-  for (int c = lane; c < e; c += 32) ss = fmaf(o[c], o[c], ss);
+  const T* zr = z + t * ldz + h * e;
+  T* dst = out + t * ldo + h * e;
+  float v[8], g[8], ss = 0.f;                        // up to 256 columns in registers
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int c = lane + 32 * i;
+    v[i] = c < e ? o[c] : 0.f;
+    g[i] = c < e ? to_f(zr[c]) : 0.f;
+    ss = fmaf(v[i], v[i], ss);
+  }
+  for (int c = lane + 256; c < e; c += 32) ss = fmaf(o[c], o[c], ss);
   const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(e) + eps);
-  for (int c = lane; c < e; c += 32)
-    out[t * ldo + h * e + c] = from_f<T>(o[c] * inv * w[c] * gate_of(to_f(z[t * ldz + h * e + c]), sigmoid_gate));
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int c = lane + 32 * i;
+    if (c < e) dst[c] = from_f<T>(v[i] * inv * w[c] * gate_of(g[i], sigmoid_gate));
+  }
+  for (int c = lane + 256; c < e; c += 32) dst[c] = from_f<T>(o[c] * inv * w[c] * gate_of(to_f(zr[c]), sigmoid_gate));
 }
 
 // ------------------------------------------------------------------ host
-template <typename T>
-static int conv_launch(const void* x, int ldx, void* y, int ldy, const void* w, void* state, const Segments& sg, int C,
-                       int taps, int tokens, cudaStream_t st) {
-  const dim3 grid((C / 2 + kConvThreads - 1) / kConvThreads, max_tiles(tokens, sg.num, kConvRows));
-  auto go = [&](auto kernel) {
-    return static_cast<int>(launch(kernel, grid, dim3(kConvThreads), 0, st, static_cast<const T*>(x), ldx,
-                                   static_cast<T*>(y), ldy, static_cast<const float*>(w), static_cast<T*>(state), sg, C));
-  };
-  switch (taps) {
-    case 1: return go(conv_silu_kernel<T, 1>);
-    case 2: return go(conv_silu_kernel<T, 2>);
-    case 3: return go(conv_silu_kernel<T, 3>);
-    case 4: return go(conv_silu_kernel<T, 4>);
-    case 5: return go(conv_silu_kernel<T, 5>);
-    case 6: return go(conv_silu_kernel<T, 6>);
-    case 7: return go(conv_silu_kernel<T, 7>);
-    case 8: return go(conv_silu_kernel<T, 8>);
+template <typename T, int KD, int RPT, bool CHANNEL, bool STEP>
+static int delta_go(const DeltaWalk<T>& p, int threads, int vtiles, cudaStream_t st) {
+  const int VT = threads / DeltaShape<KD>::LPR * RPT;
+  const dim3 grid(p.H, p.sg.num, vtiles);
+  if constexpr (STEP) {
+    return static_cast<int>(launch(delta_step_kernel<T, KD, RPT, CHANNEL>, grid, dim3(threads), sizeof(float) * VT, st, p));
+  } else {
+    constexpr int NB = DeltaShape<KD>::NB;
+    const size_t smem = 2 * (sizeof(float) * NB * ((CHANNEL ? 3 : 2) * KD + 4 + VT) + sizeof(T) * NB * p.es);
+    auto kernel = delta_walk_kernel<T, KD, RPT, CHANNEL>;
+    static bool configured[64] = {};     // per device
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -18;
+    if (!configured[dev]) {
+      const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      if (e != cudaSuccess) return static_cast<int>(e);
+      configured[dev] = true;
+    }
+    if (smem > 200 * 1024) return -14;
+    return static_cast<int>(launch(kernel, grid, dim3(threads), smem, st, p));
   }
-  return -12;
-}
-
-template <typename T, int KD, int RPT, bool CHANNEL, bool PIPE>
-static int delta_go(const DeltaRule<T>& p, int row_threads, int vtiles, cudaStream_t st) {
-  constexpr int NB = PIPE ? DeltaShape<KD>::NB : 1;
-  const int VT = row_threads / DeltaShape<KD>::LPR * RPT;
-  const size_t smem = sizeof(float) * (PIPE ? 2 : 1) * NB * ((CHANNEL ? 3 : 2) * KD + 2 * VT + 4);
-  auto kernel = delta_rule_kernel<T, KD, RPT, CHANNEL, PIPE>;
-  static bool configured[64] = {};     // per device
-  int dev = 0;
-  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -18;
-  if (!configured[dev]) {
-    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    configured[dev] = true;
-  }
-  return static_cast<int>(launch(kernel, dim3(p.H, p.sg.num, vtiles), dim3(row_threads + (PIPE ? 32 * kPrepWarps : 0)), smem,
-                                 st, p));
 }
 
 template <typename T, int KD>
-static int delta_kd(DeltaRule<T> p, bool channel, bool decode, int tokens, float* raw, cudaStream_t st) {
+static int delta_kd(DeltaWalk<T> p, bool channel, bool step, int tokens, float* raw, cudaStream_t st) {
   constexpr int LPR = DeltaShape<KD>::LPR;
-  // rows per thread: four amortise the operand loads from shared memory; one spreads a head over more blocks when the
-  // step has too few (head, request) pairs to fill the device
-  const int max_rows4 = 256 / LPR * 4, max_rows1 = 256 / LPR;
-  const bool spread = !decode && static_cast<long long>(p.H) * p.sg.num < 148;
-  const int rpt = (spread || p.e <= max_rows1 / 2) ? 1 : 4;
-  const int max_rows = rpt == 4 ? max_rows4 : max_rows1;
-  const int vtiles = (p.e + max_rows - 1) / max_rows;
-  const int rows = (p.e + vtiles - 1) / vtiles;
-  int row_threads = (rows + rpt - 1) / rpt * LPR;
-  row_threads = (row_threads + 31) / 32 * 32;
-  // blocks cover row_threads / LPR * rpt rows each
-  const int vt = row_threads / LPR * rpt;
-  const int tiles = (p.e + vt - 1) / vt;
-  p.raw = tiles > 1 ? raw : nullptr;
-  if (tiles > 1 && !raw) return -13;
+  // four rows per thread amortise the operand loads; one row per thread spreads a head over more blocks when the step
+  // has too few (head, request) pairs to fill the device
+  const int max1 = 256 / LPR, max4 = max1 * 4;
+  const bool spread = !step && static_cast<long long>(p.H) * p.sg.num < 148;
+  const int rpt = (spread || p.e <= max1 / 2) ? 1 : 4;
+  const int max_rows = rpt == 4 ? max4 : max1;
+  const int parts = (p.e + max_rows - 1) / max_rows;
+  const int rows = (p.e + parts - 1) / parts;
+  const int threads = ((rows + rpt - 1) / rpt * LPR + 31) / 32 * 32;
+  const int vt = threads / LPR * rpt;
+  const int vtiles = (p.e + vt - 1) / vt;
+  const bool norm = !step || vtiles > 1;             // the norm runs as a kernel of its own
+  p.raw = norm ? raw : nullptr;
+  if (norm && !raw) return -13;
   int rc;
-  if (decode) {
-    if (rpt == 4) rc = channel ? delta_go<T, KD, 4, true, false>(p, row_threads, tiles, st) : delta_go<T, KD, 4, false, false>(p, row_threads, tiles, st);
-    else rc = channel ? delta_go<T, KD, 1, true, false>(p, row_threads, tiles, st) : delta_go<T, KD, 1, false, false>(p, row_threads, tiles, st);
+  if (step) {
+    if (rpt == 4) rc = channel ? delta_go<T, KD, 4, true, true>(p, threads, vtiles, st) : delta_go<T, KD, 4, false, true>(p, threads, vtiles, st);
+    else rc = channel ? delta_go<T, KD, 1, true, true>(p, threads, vtiles, st) : delta_go<T, KD, 1, false, true>(p, threads, vtiles, st);
   } else if (rpt == 4) {
-    rc = channel ? delta_go<T, KD, 4, true, true>(p, row_threads, tiles, st) : delta_go<T, KD, 4, false, true>(p, row_threads, tiles, st);
+    rc = channel ? delta_go<T, KD, 4, true, false>(p, threads, vtiles, st) : delta_go<T, KD, 4, false, false>(p, threads, vtiles, st);
   } else {
-    rc = channel ? delta_go<T, KD, 1, true, true>(p, row_threads, tiles, st) : delta_go<T, KD, 1, false, true>(p, row_threads, tiles, st);
+    rc = channel ? delta_go<T, KD, 1, true, false>(p, threads, vtiles, st) : delta_go<T, KD, 1, false, false>(p, threads, vtiles, st);
   }
-  if (rc || tiles == 1) return rc;
+  if (rc || !norm) return rc;
   const long long items = static_cast<long long>(tokens) * p.H;
   return static_cast<int>(launch(gated_norm_kernel<T>, dim3(static_cast<unsigned>((items + 7) / 8)), dim3(256), 0, st,
                                  static_cast<const float*>(raw), p.z, p.ldz, p.norm_w, p.out, p.ldo, tokens, p.H, p.e, p.eps,
@@ -459,72 +558,115 @@ static int delta_kd(DeltaRule<T> p, bool channel, bool decode, int tokens, float
 
 extern "C" {
 
-struct CbDeltaRule {
-  const void* qkv; int ldq;
+struct CbDeltaPrep {
+  const void* x; int ldx;
   const void* b; int ldb;
   const void* a; int lda;
-  const void* z; int ldz;
+  const void* w; int ldw, taps;
+  void* state;
   const void* a_log;
   const void* dt_bias;
+  void* q;
+  void* k;
+  void* kq;
+  void* v;
+  void* coef;
+  void* g;
+  int H, G, d, e, ds, es, tokens, f32;
+};
+
+struct CbDeltaWalk {
+  const void* q;
+  const void* k;
+  const void* kq;
+  const void* v;
+  const void* coef;
+  const void* g;
+  const void* z; int ldz;
   const void* norm_w;
   void* state;
   void* out; int ldo;
   void* raw;
-  int H, G, d, e, ds;
+  int H, G, d, e, ds, es;
   float eps;
-  int sigmoid_gate, channel, decode, tokens, f32;
+  int sigmoid_gate, decode, tokens, f32;
 };
-
-// `C` and the row strides are even; `taps` 1..8.  `f32`: activations and state are fp32.
-int cb_conv_silu(const void* x, int ldx, void* y, int ldy, const void* w, void* state, const CbSegments* seg, int C, int taps,
-                 int tokens, int f32, void* stream) {
-  using namespace cb;
-  if (!seg || seg->num <= 0 || tokens <= 0) return 0;
-  if (C <= 0 || (C & 1) || (ldx & 1) || (ldy & 1) || taps < 1 || taps > 8) return -10;
-  const int tiles = max_tiles(tokens, seg->num, kConvRows);
-  if (tiles > 65535) return -11;
-  const Segments sg = make_segments(seg);
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return f32 ? conv_launch<float>(x, ldx, y, ldy, w, state, sg, C, taps, tokens, st)
-             : conv_launch<__nv_bfloat16>(x, ldx, y, ldy, w, state, sg, C, taps, tokens, st);
-}
 
 }  // extern "C"
 
 namespace cb {
+
 template <typename T>
-static int delta_typed(const CbDeltaRule* a, const CbSegments* seg, cudaStream_t st) {
-  DeltaRule<T> p;
-  p.qkv = static_cast<const T*>(a->qkv); p.ldq = a->ldq;
+static int prep_typed(const CbDeltaPrep* a, const CbSegments* seg, cudaStream_t st) {
+  DeltaPrep<T> p;
+  p.x = static_cast<const T*>(a->x); p.ldx = a->ldx;
   p.b = static_cast<const T*>(a->b); p.ldb = a->ldb;
   p.a = static_cast<const T*>(a->a); p.lda = a->lda;
-  p.z = static_cast<const T*>(a->z); p.ldz = a->ldz;
+  p.w = static_cast<const float*>(a->w); p.ldw = a->ldw; p.taps = a->taps;
+  p.state = static_cast<T*>(a->state);
   p.a_log = static_cast<const float*>(a->a_log);
   p.dt_bias = static_cast<const float*>(a->dt_bias);
+  p.q = static_cast<float*>(a->q); p.k = static_cast<float*>(a->k); p.kq = static_cast<float*>(a->kq);
+  p.v = static_cast<T*>(a->v);
+  p.coef = static_cast<float2*>(a->coef);
+  p.g = static_cast<float*>(a->g);
+  p.H = a->H; p.G = a->G; p.d = a->d; p.e = a->e; p.ds = a->ds; p.es = a->es;
+  p.sg = make_segments(seg);
+  const int tiles = max_tiles(a->tokens, seg->num, kPrepRows);
+  if (tiles > 65535) return -11;
+  const dim3 grid((a->G + a->H + kPrepWarps - 1) / kPrepWarps, tiles);
+  if (a->d <= 64) return static_cast<int>(launch(delta_prepare_kernel<T, 1>, grid, dim3(32 * kPrepWarps), 0, st, p));
+  if (a->d <= 128) return static_cast<int>(launch(delta_prepare_kernel<T, 2>, grid, dim3(32 * kPrepWarps), 0, st, p));
+  return static_cast<int>(launch(delta_prepare_kernel<T, 4>, grid, dim3(32 * kPrepWarps), 0, st, p));
+}
+
+template <typename T>
+static int walk_typed(const CbDeltaWalk* a, const CbSegments* seg, cudaStream_t st) {
+  DeltaWalk<T> p;
+  p.q = static_cast<const float*>(a->q); p.k = static_cast<const float*>(a->k); p.kq = static_cast<const float*>(a->kq);
+  p.v = static_cast<const T*>(a->v);
+  p.coef = static_cast<const float2*>(a->coef);
+  p.g = static_cast<const float*>(a->g);
+  p.z = static_cast<const T*>(a->z); p.ldz = a->ldz;
   p.norm_w = static_cast<const float*>(a->norm_w);
   p.state = static_cast<float*>(a->state);
   p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
   p.raw = nullptr;
-  p.H = a->H; p.G = a->G; p.d = a->d; p.e = a->e; p.ds = a->ds;
+  p.H = a->H; p.G = a->G; p.d = a->d; p.e = a->e; p.ds = a->ds; p.es = a->es;
   p.eps = a->eps; p.sigmoid_gate = a->sigmoid_gate;
   p.sg = make_segments(seg);
+  const bool channel = a->g != nullptr, step = a->decode != 0;
   float* raw = static_cast<float*>(a->raw);
-  if (a->d <= 64) return delta_kd<T, 64>(p, a->channel != 0, a->decode != 0, a->tokens, raw, st);
-  if (a->d <= 128) return delta_kd<T, 128>(p, a->channel != 0, a->decode != 0, a->tokens, raw, st);
-  return delta_kd<T, 256>(p, a->channel != 0, a->decode != 0, a->tokens, raw, st);
+  if (a->d <= 64) return delta_kd<T, 64>(p, channel, step, a->tokens, raw, st);
+  if (a->d <= 128) return delta_kd<T, 128>(p, channel, step, a->tokens, raw, st);
+  return delta_kd<T, 256>(p, channel, step, a->tokens, raw, st);
 }
+
+static bool delta_sizes_ok(int H, int G, int d, int e, int ds, int es, const CbSegments* seg) {
+  return H > 0 && G > 0 && (H % G) == 0 && d > 0 && d <= 256 && e > 0 && ds >= d && (ds & 3) == 0 && es >= e && (es & 7) == 0 &&
+         seg->num <= 65535;
+}
+
 }  // namespace cb
 
 extern "C" {
 
-// `decode`: every segment has at most one row.  `raw`: fp32 scratch [tokens, H e].
-int cb_delta_rule(const CbDeltaRule* a, const CbSegments* seg, void* stream) {
+// `ldw` (channels of a weight row and of a state row) and `ldx` are even; `f32`: activations and convolution state are fp32.
+int cb_delta_prepare(const CbDeltaPrep* a, const CbSegments* seg, void* stream) {
   if (!a || !seg || seg->num <= 0 || a->tokens <= 0) return 0;
-  if (a->H <= 0 || a->G <= 0 || (a->H % a->G) != 0 || a->d <= 0 || a->d > 256 || a->e <= 0 || a->ds < a->d || (a->ds & 3) ||
-      seg->num > 65535)
+  if (!cb::delta_sizes_ok(a->H, a->G, a->d, a->e, a->ds, a->es, seg) || a->taps < 1 || a->taps > cb::kPrepRows || (a->ldx & 1) || (a->ldw & 1) ||
+      a->ldw < 2 * a->G * a->d + a->H * a->e)
     return -10;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return a->f32 ? cb::delta_typed<float>(a, seg, st) : cb::delta_typed<__nv_bfloat16>(a, seg, st);
+  return a->f32 ? cb::prep_typed<float>(a, seg, st) : cb::prep_typed<__nv_bfloat16>(a, seg, st);
+}
+
+// `decode`: every segment has at most one row.  `raw`: fp32 scratch [tokens, H e].
+int cb_delta_walk(const CbDeltaWalk* a, const CbSegments* seg, void* stream) {
+  if (!a || !seg || seg->num <= 0 || a->tokens <= 0) return 0;
+  if (!cb::delta_sizes_ok(a->H, a->G, a->d, a->e, a->ds, a->es, seg)) return -10;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return a->f32 ? cb::walk_typed<float>(a, seg, st) : cb::walk_typed<__nv_bfloat16>(a, seg, st);
 }
 
 }  // extern "C"

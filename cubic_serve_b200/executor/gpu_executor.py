@@ -299,6 +299,12 @@ class GpuExecutor:
         self._uploaded = torch.cuda.Event()
         self._upload_pending = False
         self._launches = 0
+        self._after_current_stream()
+
+    def _after_current_stream(self) -> None:
+        """Steps run on a stream of their own: everything queued so far on the caller's stream (weights, zero-filled caches
+        and buffers) comes before them."""
+        self.stream.wait_stream(torch.cuda.current_stream(self.device))
 
     @property
     def reasoning_end_id(self) -> int | None:
@@ -318,6 +324,7 @@ class GpuExecutor:
             self._mask_host = torch.empty(rows, words, dtype=torch.int32, pin_memory=torch.cuda.is_available())
             self._mask_dev = torch.full((rows, words), -1, dtype=torch.int32, device=self.device)     # everything allowed
             self._mask_rows_dirty = 0
+            self._after_current_stream()
 
     def _stage_masks(self, segs: list[Segment]) -> bool:
         """Upload the allowed-token bitmasks of this step's sampled rows; rows without one allow everything.
@@ -374,8 +381,8 @@ class GpuExecutor:
             # the warm-up run below must not touch real cache pages: the single real row is turned into padding too
             self.stage.h["slots"][:cap] = -1
             self.stage.h["rb_qcount"][:cap] = 0
-            self.stage.upload()
             with torch.cuda.stream(self.stream):
+                self.stage.upload()                # on the steps' stream: the step below reads it
                 for _ in range(2):
                     self._body(b)
                 self.stream.synchronize()

@@ -27,7 +27,7 @@ from ..ops import wq_pack
 from .config import QuantSpec
 
 ARCHITECTURES = ("Bumodra",)
-MAX_CONV_TAPS, MAX_DELTA_DIM, MAX_LATENT = 8, 256, 1024      # limits of the kernels
+MAX_CONV_TAPS, MAX_DELTA_DIM, MAX_LATENT = 16, 256, 1024      # limits of the kernels
 
 
 class LayeredConfigError(ValueError):
@@ -89,7 +89,8 @@ class LatentSpec:
 
     @property
     def rank_padded(self) -> int:
-        return round_up(self.kv_rank, 64)
+        """Columns of a cached latent: the widths the attention kernels are built for."""
+        return next((p for p in (64, 128, 256, 512) if self.kv_rank <= p), MAX_LATENT)
 
     @property
     def out_width(self) -> int:
@@ -98,7 +99,7 @@ class LatentSpec:
     def validate(self) -> None:
         if min(self.heads, self.dim, self.vdim, self.q_rank, self.kv_rank) <= 0 or self.window < 0:
             raise LayeredConfigError("latent attention sizes are positive")
-        if self.rank_padded > MAX_LATENT:
+        if self.kv_rank > MAX_LATENT:
             raise LayeredConfigError(f"latents of up to {MAX_LATENT} channels are served")
 
 
@@ -360,7 +361,7 @@ class BlockDiagonal:
 @dataclass
 class DeltaWeights:
     spec: DeltaSpec
-    conv_w: torch.Tensor             # fp32 [conv_width, taps]
+    conv_w: torch.Tensor             # fp32 [taps, conv_width]
     a_log: torch.Tensor
     dt_bias: torch.Tensor
     norm_w: torch.Tensor
@@ -454,8 +455,8 @@ def pack_layer(cfg: LayeredConfig, i: int, get) -> LayerWeights:
         rows.add(get(f"{p}.q"), get(f"{p}.k"), get(f"{p}.v"))
         b_off = rows.add(get(f"{p}.b"))
         conv = torch.cat([get(f"{p}.{t}.conv") for t in "qkv"]).float()
-        conv_w = torch.zeros(m.conv_width, m.conv, device=conv.device)
-        conv_w[:m.channels] = conv
+        conv_w = torch.zeros(m.conv, m.conv_width, device=conv.device)
+        conv_w[:, :m.channels] = conv.t()
         common = dict(spec=m, conv_w=conv_w.contiguous(), a_log=f32(f"{p}.A_log"), dt_bias=f32(f"{p}.dt_bias"),
                       norm_w=f32(f"{p}.norm"), b_off=b_off)
         if m.per_channel:

@@ -70,14 +70,14 @@ class LayeredRunner(StepRunner):
         # operands of the output products ([mixer output | feed-forward]) by layout, scratch by width: layers share them
         self._operands: dict = {}
         self._scratch: dict = {}
-        raw = 1
+        delta = []
         for l in weights.layers:
             key = (l.mixer.spec.out_width, l.out_off, l.ff, l.out.k)
             self._operands.setdefault(key, buf(l.out.k))
             self._need("proj", l.split)
             if isinstance(l.mixer, DeltaWeights):
-                self._need("conv", l.mixer.spec.conv_width)
-                raw = max(raw, T * l.mixer.spec.out_width)
+                m = l.mixer.spec
+                delta.append((m.heads, m.kv_heads, m.dim, m.vdim, m.per_channel))
                 if l.mixer.low is not None:
                     self._need("low", l.mixer.low.n)
             else:
@@ -87,7 +87,7 @@ class LayeredRunner(StepRunner):
                 self._need("ql", m.heads * m.rank_padded)
                 self._need("ol", m.heads * m.rank_padded)
         self._scratch = {n: torch.zeros(T * c, dtype=act, device=dev) for n, c in self._scratch.items()}
-        self.raw = torch.empty(raw, dtype=torch.float32, device=dev)
+        self.delta = K.DeltaScratch(T, delta, act, dev) if delta else None
         self.trace: list | None = None         # a list here receives a copy of the residual after every layer run
 
     def _need(self, name: str, cols: int) -> None:
@@ -126,7 +126,7 @@ class LayeredRunner(StepRunner):
             K.wide_gemm(h, l.proj, proj, relu2=up, split=l.split, ws=self.ws)
             mixed = operand[:, :m.spec.out_width]
             n += 3 + (self._delta(m, proj, run, b, mixed, decode) if isinstance(m, DeltaWeights)
-                      else self._latent(m, proj, run, b, mixed))
+                      else self._latent(m, proj, run, b, mixed, decode))
             K.wide_gemm(operand, l.out, x, residual=x, ws=self.ws)
             if self.trace is not None:
                 self.trace.append(x.clone())
@@ -135,8 +135,6 @@ class LayeredRunner(StepRunner):
 
     def _delta(self, m: DeltaWeights, proj, run: _DeltaRun, b, out, decode: bool) -> int:
         s, T = m.spec, proj.shape[0]
-        conv = self._rows("conv", T, s.conv_width)
-        K.conv_silu(proj[:, :s.conv_width], m.conv_w, run.conv, b.segments, conv)
         n = 1
         if m.low is not None:
             low = self._rows("low", T, m.low.n)
@@ -145,10 +143,12 @@ class LayeredRunner(StepRunner):
             n += 1
         else:
             a, z = proj[:, m.a_off:m.a_off + s.heads], proj[:, m.z_off:m.z_off + s.out_width]
-        return n + K.delta_rule(conv, proj[:, m.b_off:m.b_off + s.heads], a, z, m.a_log, m.dt_bias, m.norm_w, run.state,
-                                b.segments, out, s.kv_heads, s.dim, self.cfg.rms_eps, s.per_channel, decode, self.raw)
+        K.delta_prepare(proj[:, :s.conv_width], proj[:, m.b_off:m.b_off + s.heads], a, m.conv_w, run.conv, m.a_log, m.dt_bias,
+                        b.segments, self.delta, s.heads, s.kv_heads, s.dim, s.vdim)
+        return n + K.delta_walk(z, m.norm_w, run.state, b.segments, out, self.delta, s.kv_heads, s.dim, self.cfg.rms_eps,
+                                s.per_channel, s.per_channel, decode)
 
-    def _latent(self, m: LatentWeights, proj, cache: torch.Tensor, b, out) -> int:
+    def _latent(self, m: LatentWeights, proj, cache: torch.Tensor, b, out, decode: bool) -> int:
         s, T = m.spec, proj.shape[0]
         wide = s.heads * s.rank_padded
         cq = self._rows("cq%d" % s.q_rank, T, round_up(s.q_rank, 64))
@@ -157,7 +157,7 @@ class LayeredRunner(StepRunner):
         K.wide_gemm(cq, m.uq, q, ws=self.ws)
         K.wide_gemm(q, m.absorb.w, ql, diag_rows=m.absorb.rows, ws=self.ws)
         K.latent_attention(ql, proj[:, m.g_off:m.g_off + s.heads], cache, b.page_table, b.segments, ol, s.heads, s.window,
-                           s.scale)
+                           s.scale, decode=decode, ws=self.ws)
         K.wide_gemm(ol, m.value.w, out, diag_rows=m.value.rows, ws=self.ws)
         return 5
 

@@ -790,39 +790,67 @@ def concat_rows(x: torch.Tensor, x0: torch.Tensor, out: torch.Tensor) -> None:
                                              x.shape[1], int(out.dtype == torch.float32), _stream()), "cb_concat_rows")
 
 
-def conv_silu(x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, seg: GdnSegments, out: torch.Tensor) -> None:
-    """Causal depthwise convolution of any number of taps + SiLU over ``x[T, C]`` per request segment; ``state``
-    ``[slots, taps - 1, C]`` (activation type) is read and replaced.  ``w``: fp32 ``[C, taps]``, last tap = current input."""
-    c, taps = w.shape
-    assert w.dtype == torch.float32 and w.is_contiguous() and state.dtype == x.dtype == out.dtype
-    assert x.shape[1] == out.shape[1] == c and x.stride(1) == out.stride(1) == 1
-    assert state.is_contiguous() and (taps == 1 or tuple(state.shape[1:]) == (taps - 1, c))
+class DeltaScratch:
+    """Fixed-address buffers between the preparation and the recurrence of delta layers, for up to ``max_tokens`` rows of the
+    largest layer they are made for (layers share them)."""
+
+    def __init__(self, max_tokens: int, sizes, act: torch.dtype, device) -> None:
+        """``sizes``: (heads, key heads, key width, value width, per channel) of every layer."""
+        f32 = dict(dtype=torch.float32, device=device)
+        most = lambda f: max(f(*s) for s in sizes)                                     # noqa: E731
+        T = max_tokens
+        self.q = torch.zeros(T * most(lambda H, G, d, e, c: G * (-(-d // 4) * 4)), **f32)
+        self.k = torch.zeros_like(self.q)
+        self.kq = torch.zeros(T * most(lambda H, G, d, e, c: G), **f32)
+        self.v = torch.zeros(T * most(lambda H, G, d, e, c: H * (-(-e // 8) * 8)), dtype=act, device=device)
+        self.coef = torch.zeros(T * most(lambda H, G, d, e, c: 2 * H), **f32)
+        self.g = torch.zeros(max(1, T * most(lambda H, G, d, e, c: H * (-(-d // 4) * 4) if c else 0)), **f32)
+        self.raw = torch.zeros(T * most(lambda H, G, d, e, c: H * e), **f32)
+
+
+def delta_prepare(x: torch.Tensor, b: torch.Tensor, a: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor,
+                  a_log: torch.Tensor, dt_bias: torch.Tensor, seg: GdnSegments, sc: DeltaScratch, heads: int, kv_heads: int,
+                  dim: int, vdim: int) -> None:
+    """Everything of a delta layer's tokens that does not depend on its state (``csrc/delta_rule.cu``): causal depthwise
+    convolution + SiLU of ``x [T, q | k | v]`` with ``conv_w`` fp32 ``[taps, channels]`` (the last row multiplies the current
+    input) and the requests' last inputs ``conv_state [slots, taps - 1, channels]``, which are read and replaced; unit q / k;
+    step sizes and decays from the logits ``b`` and ``a``."""
+    taps, ldw = conv_w.shape
+    channel = dt_bias.numel() != heads
+    assert conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_state.dtype == x.dtype == a.dtype == b.dtype
+    assert conv_state.is_contiguous() and (taps == 1 or tuple(conv_state.shape[1:]) == (taps - 1, ldw))
+    assert x.shape[1] == ldw and x.stride(1) == b.stride(1) == a.stride(1) == 1 and dt_bias.numel() in (heads, heads * dim)
+    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (a_log, dt_bias))
+    ds, es = -(-dim // 4) * 4, -(-vdim // 8) * 8
+    T = x.shape[0]
+    assert sc.q.numel() >= T * kv_heads * ds and sc.v.numel() >= T * heads * es and sc.v.dtype == x.dtype
+    assert not channel or sc.g.numel() >= T * heads * ds
+    p = native.DeltaPrepStruct(x.data_ptr(), x.stride(0), b.data_ptr(), b.stride(0), a.data_ptr(), a.stride(0),
+                               conv_w.data_ptr(), ldw, taps, conv_state.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(),
+                               sc.q.data_ptr(), sc.k.data_ptr(), sc.kq.data_ptr(), sc.v.data_ptr(), sc.coef.data_ptr(),
+                               sc.g.data_ptr() if channel else None, heads, kv_heads, dim, vdim, ds, es, T,
+                               int(x.dtype == torch.float32))
     st = _seg(seg)
-    native.check(native.lib().cb_conv_silu(x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), w.data_ptr(),
-                                           state.data_ptr(), ctypes.byref(st), c, taps, x.shape[0],
-                                           int(x.dtype == torch.float32), _stream()), "cb_conv_silu")
+    native.check(native.lib().cb_delta_prepare(ctypes.byref(p), ctypes.byref(st), _stream()), "cb_delta_prepare")
 
 
-def delta_rule(qkv: torch.Tensor, b: torch.Tensor, a: torch.Tensor, z: torch.Tensor, a_log: torch.Tensor,
-               dt_bias: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, seg: GdnSegments, out: torch.Tensor,
-               kv_heads: int, dim: int, eps: float, sigmoid_gate: bool, decode: bool, raw: torch.Tensor) -> int:
-    """Gated delta rule and gated norm of every head, see ``csrc/delta_rule.cu``.  ``state`` fp32 ``[slots, H, vdim, stride]``;
-    ``a`` has one decay logit per head, or one per (head, key channel) when it has ``H dim`` columns.  ``raw``: fp32 scratch
-    of at least ``T H vdim`` elements.  Returns the launches made at most."""
+def delta_walk(z: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, seg: GdnSegments, out: torch.Tensor,
+               sc: DeltaScratch, kv_heads: int, dim: int, eps: float, sigmoid_gate: bool, channel: bool, decode: bool) -> int:
+    """The recurrence over the rows prepared by ``delta_prepare`` and the gated norm of every head.  ``state`` fp32
+    ``[slots, H, vdim, stride]`` is read and replaced; ``channel``: one decay per key channel; ``decode``: every segment has
+    at most one row.  Returns the launches made (at most)."""
     H, e, ds = state.shape[1:]
-    T = qkv.shape[0]
-    channel = dt_bias.numel() != H
-    assert state.dtype == torch.float32 and state.is_contiguous() and dt_bias.numel() in (H, H * dim)
-    assert all(t.stride(1) == 1 and t.dtype == qkv.dtype for t in (qkv, b, a, z, out))
-    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (a_log, dt_bias, norm_w))
-    assert raw.dtype == torch.float32 and raw.numel() >= T * H * e and out.shape[1] == H * e
-    d = native.DeltaRuleStruct(qkv.data_ptr(), qkv.stride(0), b.data_ptr(), b.stride(0), a.data_ptr(), a.stride(0),
-                               z.data_ptr(), z.stride(0), a_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr(),
-                               state.data_ptr(), out.data_ptr(), out.stride(0), raw.data_ptr(), H, kv_heads, dim, e, ds,
-                               float(eps), int(sigmoid_gate), int(channel), int(decode), T, int(qkv.dtype == torch.float32))
+    T = z.shape[0]
+    assert state.dtype == torch.float32 and state.is_contiguous() and ds == -(-dim // 4) * 4
+    assert z.dtype == out.dtype == sc.v.dtype and z.stride(1) == out.stride(1) == 1 and out.shape[1] == H * e
+    assert norm_w.dtype == torch.float32 and sc.raw.numel() >= T * H * e
+    p = native.DeltaWalkStruct(sc.q.data_ptr(), sc.k.data_ptr(), sc.kq.data_ptr(), sc.v.data_ptr(), sc.coef.data_ptr(),
+                               sc.g.data_ptr() if channel else None, z.data_ptr(), z.stride(0), norm_w.data_ptr(),
+                               state.data_ptr(), out.data_ptr(), out.stride(0), sc.raw.data_ptr(), H, kv_heads, dim, e, ds,
+                               -(-e // 8) * 8, float(eps), int(sigmoid_gate), int(decode), T, int(z.dtype == torch.float32))
     st = _seg(seg)
-    native.check(native.lib().cb_delta_rule(ctypes.byref(d), ctypes.byref(st), _stream()), "cb_delta_rule")
-    return 2
+    native.check(native.lib().cb_delta_walk(ctypes.byref(p), ctypes.byref(st), _stream()), "cb_delta_walk")
+    return 1 if decode else 2
 
 
 def latent_prepare(proj: torch.Tensor, q_rank: int, c_off: int, rank: int, q_norm: torch.Tensor, c_norm: torch.Tensor,
@@ -837,14 +865,34 @@ def latent_prepare(proj: torch.Tensor, q_rank: int, c_off: int, rank: int, q_nor
 
 
 def latent_attention(q: torch.Tensor, gate: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor, seg: GdnSegments,
-                     out: torch.Tensor, heads: int, window: int, scale: float) -> None:
+                     out: torch.Tensor, heads: int, window: int, scale: float, decode: bool = False, splits: int | None = None,
+                     ws: Workspace | None = None) -> None:
     """Windowed softmax attention of latent-space queries ``q [T, H Rp]`` over the paged latents, times the heads' sigmoid
-    gates (``gate [T, H]`` logits).  ``window`` 0: every earlier token."""
+    gates (``gate [T, H]`` logits).  ``window`` 0: every earlier token.  ``decode``: every segment has at most one row.
+    ``splits``: key splits of the bf16 form (None: as many as fill the device)."""
     T, rp = q.shape[0], cache.shape[2]
     assert q.shape[1] == out.shape[1] == heads * rp and q.is_contiguous() and out.is_contiguous()
     assert q.dtype == out.dtype == gate.dtype == cache.dtype and page_table.dtype == torch.int32
+    f32 = q.dtype == torch.float32
+    l = native.lib()
+    partial = None
+    if f32 or rp > 512:
+        splits = 1
+    else:
+        units = ctypes.c_int(0)
+        l.cb_latent_attn_partial_floats(T, seg.num, heads, rp, int(decode), 1, ctypes.byref(units))
+        if splits is None:
+            from .strategies import active
+            a = active().attention
+            # a block walks tiles of 64 keys: no more splits than the longest row has tiles
+            keys = page_table.shape[1] * PAGE_TOKENS if window <= 0 else min(window, page_table.shape[1] * PAGE_TOKENS)
+            splits = min(a.max_splits, -(-keys // 64), max(1, a.target_ctas // (1 if decode else 2) // units.value))
+        if splits > 1:
+            ws = ws or workspace(q.device)
+            ws.ensure_attn(l.cb_latent_attn_partial_floats(T, seg.num, heads, rp, int(decode), splits, None))
+            partial = ws.attn.data_ptr()
     a = native.LatentAttnStruct(q.data_ptr(), out.data_ptr(), cache.data_ptr(), gate.data_ptr(), gate.stride(0),
-                                page_table.data_ptr(), page_table.shape[1], heads, rp, window, float(scale), T,
-                                int(q.dtype == torch.float32))
+                                page_table.data_ptr(), page_table.shape[1], heads, rp, window, float(scale), T, int(f32),
+                                int(decode), splits, partial)
     st = _seg(seg)
-    native.check(native.lib().cb_latent_attn(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_latent_attn")
+    native.check(l.cb_latent_attn(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_latent_attn")

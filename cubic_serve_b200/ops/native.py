@@ -267,11 +267,13 @@ def _declare(l: ctypes.CDLL) -> None:
     l.cb_row_norm.argtypes = [vp, vp, vp, vp, i, i, i, f, i, vp]
     l.cb_embed_norm.argtypes = [vp, vp, vp, vp, vp, i, i, i, f, vp]
     l.cb_concat_rows.argtypes = [vp, vp, vp, i, i, i, i, vp]
-    l.cb_conv_silu.argtypes = [vp, i, vp, i, vp, vp, vp, i, i, i, i, vp]
-    l.cb_delta_rule.argtypes = [vp, vp, vp]
+    l.cb_delta_prepare.argtypes = [vp, vp, vp]
+    l.cb_delta_walk.argtypes = [vp, vp, vp]
     l.cb_latent_prepare.argtypes = [vp, i, i, i, i, i, vp, vp, vp, i, vp, i, vp, i, f, i, vp]
     l.cb_latent_attn.argtypes = [vp, vp, vp]
-    for name in ("bf16_gemm_wide", "f32_gemm", "row_norm", "embed_norm", "concat_rows", "conv_silu", "delta_rule",
+    l.cb_latent_attn_partial_floats.argtypes = [i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
+    l.cb_latent_attn_partial_floats.restype = ll
+    for name in ("bf16_gemm_wide", "f32_gemm", "row_norm", "embed_norm", "concat_rows", "delta_prepare", "delta_walk",
                  "latent_prepare", "latent_attn"):
         getattr(l, f"cb_{name}").restype = i
     # fp8 (e4m3 x e4m3) tensor path: activation quantizers and the GEMM entries
@@ -328,15 +330,25 @@ class F32GemmStruct(ctypes.Structure):
                 ("N", ctypes.c_int), ("K", ctypes.c_int)]
 
 
-class DeltaRuleStruct(ctypes.Structure):
-    """Mirror of ``CbDeltaRule`` in ``csrc/delta_rule.cu``."""
-    _fields_ = [("qkv", ctypes.c_void_p), ("ldq", ctypes.c_int), ("b", ctypes.c_void_p), ("ldb", ctypes.c_int),
-                ("a", ctypes.c_void_p), ("lda", ctypes.c_int), ("z", ctypes.c_void_p), ("ldz", ctypes.c_int),
-                ("a_log", ctypes.c_void_p), ("dt_bias", ctypes.c_void_p), ("norm_w", ctypes.c_void_p),
-                ("state", ctypes.c_void_p), ("out", ctypes.c_void_p), ("ldo", ctypes.c_int), ("raw", ctypes.c_void_p),
-                ("H", ctypes.c_int), ("G", ctypes.c_int), ("d", ctypes.c_int), ("e", ctypes.c_int), ("ds", ctypes.c_int),
-                ("eps", ctypes.c_float), ("sigmoid_gate", ctypes.c_int), ("channel", ctypes.c_int),
-                ("decode", ctypes.c_int), ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
+class DeltaPrepStruct(ctypes.Structure):
+    """Mirror of ``CbDeltaPrep`` in ``csrc/delta_rule.cu``."""
+    _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("b", ctypes.c_void_p), ("ldb", ctypes.c_int),
+                ("a", ctypes.c_void_p), ("lda", ctypes.c_int), ("w", ctypes.c_void_p), ("ldw", ctypes.c_int),
+                ("taps", ctypes.c_int), ("state", ctypes.c_void_p), ("a_log", ctypes.c_void_p), ("dt_bias", ctypes.c_void_p),
+                ("q", ctypes.c_void_p), ("k", ctypes.c_void_p), ("kq", ctypes.c_void_p), ("v", ctypes.c_void_p),
+                ("coef", ctypes.c_void_p), ("g", ctypes.c_void_p), ("H", ctypes.c_int), ("G", ctypes.c_int),
+                ("d", ctypes.c_int), ("e", ctypes.c_int), ("ds", ctypes.c_int), ("es", ctypes.c_int),
+                ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
+
+
+class DeltaWalkStruct(ctypes.Structure):
+    """Mirror of ``CbDeltaWalk`` in ``csrc/delta_rule.cu``."""
+    _fields_ = [("q", ctypes.c_void_p), ("k", ctypes.c_void_p), ("kq", ctypes.c_void_p), ("v", ctypes.c_void_p),
+                ("coef", ctypes.c_void_p), ("g", ctypes.c_void_p), ("z", ctypes.c_void_p), ("ldz", ctypes.c_int),
+                ("norm_w", ctypes.c_void_p), ("state", ctypes.c_void_p), ("out", ctypes.c_void_p), ("ldo", ctypes.c_int),
+                ("raw", ctypes.c_void_p), ("H", ctypes.c_int), ("G", ctypes.c_int), ("d", ctypes.c_int),
+                ("e", ctypes.c_int), ("ds", ctypes.c_int), ("es", ctypes.c_int), ("eps", ctypes.c_float),
+                ("sigmoid_gate", ctypes.c_int), ("decode", ctypes.c_int), ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
 
 
 class LatentAttnStruct(ctypes.Structure):
@@ -344,7 +356,7 @@ class LatentAttnStruct(ctypes.Structure):
     _fields_ = [("q", ctypes.c_void_p), ("out", ctypes.c_void_p), ("cache", ctypes.c_void_p), ("gate", ctypes.c_void_p),
                 ("ldg", ctypes.c_int), ("page_table", ctypes.c_void_p), ("max_pages", ctypes.c_int), ("H", ctypes.c_int),
                 ("Rp", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float), ("tokens", ctypes.c_int),
-                ("f32", ctypes.c_int)]
+                ("f32", ctypes.c_int), ("decode", ctypes.c_int), ("splits", ctypes.c_int), ("partial", ctypes.c_void_p)]
 
 
 class ReduceNormStruct(ctypes.Structure):
