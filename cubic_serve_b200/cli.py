@@ -151,7 +151,8 @@ def build_parser() -> argparse.ArgumentParser:
     g = s.add_argument_group("Model and generation")
     g.add_argument("--compute-mode", choices=("wna16", "wna8"), default="wna16",
                    help="wna16: packed weights, 16-bit activations (the only mode of this build; wna8 is refused)")
-    g.add_argument("--dtype", choices=("bfloat16",), default="bfloat16")
+    g.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16",
+                   help="activations and products; float32 is available for the layered decoders")
     g.add_argument("--max-model-len", type=int)
     g.add_argument("--chat-template")
     g.add_argument("--reasoning-parser", default="auto")
@@ -248,7 +249,12 @@ def _reference(args) -> int:
         ck = admit_checkpoint(args.model)
         cfg = ck.cfg
     stateful = None
-    if cfg is None or getattr(cfg, "family", "") == "qwen4_exp":
+    if cfg is not None and getattr(cfg, "family", "") == "layered":
+        from .models.layered import random_tensors
+        from .models.layered_reference import Oracle
+        stateful = Oracle(ck.raw_config if ck is not None else cfg.to_config(),
+                          {n: ck.store.get(n) for n in ck.plain} if ck is not None else random_tensors(cfg, args.seed))
+    elif cfg is None or getattr(cfg, "family", "") == "qwen4_exp":
         from .models.qwen4_exp import Qwen4ExpModel, admit_qwen4_exp_checkpoint, random_qwen4_exp_weights
         if cfg is None:
             cfg, weights, _ = admit_qwen4_exp_checkpoint(args.model)
@@ -364,7 +370,9 @@ def _inspect(args) -> int:
     else:
         info = inspect_checkpoint(args.model)
         cfg = None
-    if args.tp * args.pp * args.ep > 1:
+    if args.tp * args.pp * args.ep > 1 and info.get("family") == "layered":
+        info["partition_error"] = "layered decoders are served on one GPU"
+    elif args.tp * args.pp * args.ep > 1:
         from pathlib import Path
 
         from .models.config import ModelConfig

@@ -78,6 +78,24 @@ class StateSpec:
 
 
 @dataclass(frozen=True)
+class LatentCacheSpec:
+    """Paged latent cache of a layered decoder: one row per token and attention run, in the activation type."""
+    page_bytes: int           # one page across all attention runs
+    runs: int
+    page_tokens: int = PAGE_TOKENS
+
+    def bytes_per_token(self) -> float:
+        return self.page_bytes / self.page_tokens
+
+
+@dataclass(frozen=True)
+class DeltaStateSpec:
+    """Recurrent state of a layered decoder's delta runs (fp32 delta-rule state and convolution inputs)."""
+    runs: int
+    bytes_per_request: int
+
+
+@dataclass(frozen=True)
 class TensorEntry:
     name: str
     dtype: str
@@ -112,8 +130,8 @@ class ModelSpec:
     name: str
     family: str
     config_digest: str
-    cache: CacheSpec
-    state: StateSpec | None
+    cache: CacheSpec | LatentCacheSpec
+    state: StateSpec | DeltaStateSpec | None
     manifest: WeightManifest | None = None
 
     @staticmethod
@@ -126,6 +144,16 @@ class ModelSpec:
         cache = CacheSpec(hi - lo - n_gdn, kv_local, cfg.head_dim, k_bits, v_bits)
         state = StateSpec(n_gdn, cfg.gdn_k_heads // tp, cfg.gdn_v_heads // tp) if n_gdn else None
         return ModelSpec(cfg.name, cfg.family, digest_of(dataclasses.asdict(cfg)), cache, state, manifest)
+
+    @staticmethod
+    def from_layered(cfg, manifest: WeightManifest | None = None) -> "ModelSpec":
+        """Of a layered decoder (``models/layered.py``): every layer RUN has its own cache or state."""
+        from ..models.layered import LatentSpec
+        attn = sum(isinstance(cfg.layers[i].mixer, LatentSpec) for i, _ in cfg.runs)
+        delta = len(cfg.runs) - attn
+        state = DeltaStateSpec(delta, cfg.state_bytes_per_request) if delta else None
+        return ModelSpec(cfg.name, cfg.family, digest_of(dataclasses.asdict(cfg)), LatentCacheSpec(cfg.page_bytes, attn), state,
+                         manifest)
 
     @property
     def digest(self) -> str:

@@ -24,8 +24,6 @@ template <> struct Pair2<__nv_bfloat16> { using type = __nv_bfloat162; };
 template <> struct Pair2<float> { using type = float2; };
 __device__ __forceinline__ float2 to_f2(__nv_bfloat162 v) { return __bfloat1622float2(v); }
 __device__ __forceinline__ float2 to_f2(float2 v) { return v; }
-__device__ __forceinline__ float silu_exact(float x) { return x / (1.f + expf(-x)); }
-__device__ __forceinline__ float softplus_of(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float gate_of(float z, int sigmoid) { return (sigmoid ? 1.f : z) / (1.f + expf(-z)); }
 __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return __ffma2_rn(a, b, c); }
 __device__ __forceinline__ float2 mul2(float2 a, float2 b) { return __fmul2_rn(a, b); }
@@ -54,45 +52,100 @@ struct DeltaPrep {
   Segments sg;
 };
 
-// The convolution of `NP` channel pairs (c0 + 64 i, + 1) of token t, one lane; pairs at or behind `lim` read as zero.
-// `odd`: heads of odd width, whose channels are read one at a time.
-template <typename T, int NP>
-__device__ __forceinline__ void conv_pairs(const DeltaPrep<T>& p, const T* xr, const T* st, bool fresh, int t, int c0, int base,
-                                           int lim, bool odd, float2 (&out)[NP]) {
+// Exponential and softplus of the decays.  In a bf16 model the logits are bf16: the fast forms' absolute error (1e-7 and a
+// few ulp of the exponential) is far below what the logits carry; fp32 models use the exact ones.
+template <typename T> __device__ __forceinline__ float exp_of(float x) { return sizeof(T) == 2 ? __expf(x) : expf(x); }
+template <typename T> __device__ __forceinline__ float softplus_of(float x) {
+  const float e = exp_of<T>(-fabsf(x));
+  return fmaxf(x, 0.f) + (sizeof(T) == 2 ? __logf(1.f + e) : log1pf(e));
+}
+template <typename T> __device__ __forceinline__ float silu_of(float x) { return sizeof(T) == 2 ? silu_fast(x) : x / (1.f + expf(-x)); }
+
+// Two neighbouring channels p[0], p[1] where `ok`, zeros elsewhere: one predicated load, so that the loads of a whole tile can
+// be in flight at once.  ODD: the pair may start at an odd channel and its second channel exists only where `ok1`.
+template <typename T, bool ODD>
+__device__ __forceinline__ float2 load_pair(const T* p, bool ok, bool ok1) {
   using P = typename Pair2<T>::type;
-#pragma unroll
-  for (int i = 0; i < NP; ++i) out[i] = make_float2(0.f, 0.f);
-  const int H = p.taps - 1;
-#pragma unroll 1
-  for (int j = 0; j < p.taps; ++j) {
-    const int tt = t - H + j;
-    if (tt < 0 && fresh) continue;
-    const T* src = (tt >= 0 ? xr + static_cast<ptrdiff_t>(tt) * p.ldx : st + static_cast<ptrdiff_t>(tt + H) * p.ldw) + base;
-    const float* wr = p.w + static_cast<size_t>(j) * p.ldw + base;
-#pragma unroll
-    for (int i = 0; i < NP; ++i) {
-      const int c = c0 + 64 * i;
-      if (c >= lim) continue;
-      float2 v, w;
-      if (!odd) {
-        v = to_f2(*reinterpret_cast<const P*>(src + c));
-        w = *reinterpret_cast<const float2*>(wr + c);
-      } else {
-        v = make_float2(to_f(src[c]), c + 1 < lim ? to_f(src[c + 1]) : 0.f);
-        w = make_float2(wr[c], c + 1 < lim ? wr[c + 1] : 0.f);
-      }
-      out[i] = fma2(w, v, out[i]);
-    }
-  }
-#pragma unroll
-  for (int i = 0; i < NP; ++i) out[i] = make_float2(silu_exact(out[i].x), silu_exact(out[i].y));
+  if constexpr (ODD) return make_float2(ok ? to_f(p[0]) : 0.f, ok1 ? to_f(p[1]) : 0.f);
+  float2 v = make_float2(0.f, 0.f);
+  if (ok) v = to_f2(*reinterpret_cast<const P*>(p));
+  return v;
 }
 
+// Convolution + SiLU of one channel pair along a segment's tokens.  TAPS > 0: weights and the last inputs in registers; the
+// caller reads the inputs of several tokens ahead and feeds them in order (heads of even width).  TAPS 0: any number of taps
+// and any width, everything is read again for every token.
+template <typename T, int TAPS>
+struct ConvPair {
+  static constexpr int R = TAPS > 0 ? TAPS : 1;
+  float2 w[R], hist[R];
+  const DeltaPrep<T>* p;
+  const T* xr;
+  const T* st;
+  bool fresh, ok, ok1;
+  int col;                                                        // first channel of the pair
+
+  __device__ __forceinline__ float2 input(int t) const {          // input at token t of the segment, t >= -(taps - 1)
+    const T* src = t >= 0 ? xr + static_cast<ptrdiff_t>(t) * p->ldx : st + static_cast<ptrdiff_t>(t + p->taps - 1) * p->ldw;
+    const bool there = t >= 0 || !fresh;
+    return load_pair<T, TAPS == 0>(src + col, ok && there, ok1 && there);
+  }
+  __device__ __forceinline__ float2 weight(int j) const {
+    return load_pair<float, TAPS == 0>(p->w + static_cast<size_t>(j) * p->ldw + col, ok, ok1);
+  }
+  __device__ __forceinline__ void begin(const DeltaPrep<T>& prm, const T* x, const T* state, bool fr, int base, int c, int lim,
+                                        int t0) {
+    p = &prm; xr = x; st = state; fresh = fr; col = base + c; ok = c < lim; ok1 = c + 1 < lim;
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) w[j] = weight(j);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) hist[j] = input(t0 - (TAPS - 1) + j);
+    }
+  }
+  __device__ __forceinline__ float2 ahead(int t, int end) const { // the input `token` wants, t >= 0; nothing behind the tile
+    if constexpr (TAPS == 0) return make_float2(0.f, 0.f);
+    return load_pair<T, false>(xr + static_cast<ptrdiff_t>(t) * p->ldx + col, ok && t < end, false);
+  }
+  __device__ __forceinline__ float2 token(int t, float2 v) {      // tokens in order from t0 on
+    float2 a;
+    if constexpr (TAPS > 0) {
+      a = mul2(w[TAPS - 1], v);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) a = fma2(w[j], hist[j], a);
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j] = hist[j + 1];
+      if constexpr (TAPS > 1) hist[TAPS - 2] = v;
+    } else {
+      a = make_float2(0.f, 0.f);
+#pragma unroll 1
+      for (int j = 0; j < p->taps; ++j) a = fma2(weight(j), input(t - (p->taps - 1) + j), a);
+    }
+    return make_float2(silu_of<T>(a.x), silu_of<T>(a.y));
+  }
+  // The pair's new convolution state, written by the tile that holds the segment's first tokens (the only reader of the old
+  // one): from the registers when it holds the last tokens too, else from the inputs.
+  __device__ __forceinline__ void save(T* state, int count, bool whole) const {
+    if constexpr (TAPS > 1) {
+      float2 v[TAPS - 1];
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) v[j] = whole ? hist[j] : input(count - (TAPS - 1) + j);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        T* dst = state + static_cast<ptrdiff_t>(j) * p->ldw + col;
+        if (ok) dst[0] = from_f<T>(v[j].x);
+        if (ok1) dst[1] = from_f<T>(v[j].y);
+      }
+    }
+  }
+};
+
 // The convolution state of channels [base, base + n) becomes the segment's last taps - 1 inputs.  Called after the
-// outputs that need the old state, by the warp that produced them; a lane touches the same channels in both.
+// outputs that need the old state, by the warp that produced them.
 template <typename T>
 __device__ __forceinline__ void conv_state(const DeltaPrep<T>& p, const T* xr, T* st, bool fresh, int count, int base, int n) {
   const int H = p.taps - 1;
+  __syncwarp();                              // read in pairs, replaced channel by channel
   for (int c = threadIdx.x & 31; c < n; c += 32)
     for (int j = 0; j < H; ++j) {            // entry j moves down from entry j + count, which is read before it is written
       const int t = count - H + j;
@@ -103,9 +156,9 @@ __device__ __forceinline__ void conv_state(const DeltaPrep<T>& p, const T* xr, T
     }
 }
 
-// A warp per (head slot, tile of kPrepRows tokens): slots [0, G) are key heads (q and k), slots [G, G + H) value heads
-// (v, step size, decays).  NP: channel pairs per lane of a key head (d <= 64 NP).
-template <typename T, int NP>
+// A warp per (slot, tile of kPrepRows tokens): slots [0, G) are key heads (q and k), [G, G + H) value heads (v, step size,
+// decay per head), [G + H, G + 2 H) channel decays.  NP: channel pairs per lane of a key head (d <= 64 NP).
+template <typename T, int NP, int TAPS>
 __global__ void __launch_bounds__(32 * kPrepWarps)
 delta_prepare_kernel(const DeltaPrep<T> p) {
   pdl_wait();
@@ -114,7 +167,7 @@ delta_prepare_kernel(const DeltaPrep<T> p) {
   if (!find_tile(p.sg, kPrepRows, blockIdx.y, s, off)) return;
   const int slot = blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
-  if (slot >= p.G + p.H) return;
+  if (slot >= p.G + (p.g ? 2 : 1) * p.H) return;
   const int count = p.sg.count[s], end = min(count, off + kPrepRows);
   const bool fresh = p.sg.pos0[s] == 0;
   const size_t row0 = p.sg.row0[s];
@@ -122,15 +175,33 @@ delta_prepare_kernel(const DeltaPrep<T> p) {
   T* st = p.state + static_cast<size_t>(p.sg.slot[s]) * (p.taps - 1) * p.ldw;
   if (slot < p.G) {
     const int qb = slot * p.d, kb = (p.G + slot) * p.d;
-    const bool odd = p.d & 1;
     const float scale = 1.f / sqrtf(static_cast<float>(p.d));
-    for (int t = off; t < end; ++t) {
+    ConvPair<T, TAPS> cq[NP], ck[NP];
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      cq[i].begin(p, xr, st, fresh, qb, 2 * lane + 64 * i, p.d, off);
+      ck[i].begin(p, xr, st, fresh, kb, 2 * lane + 64 * i, p.d, off);
+    }
+    constexpr int AH = NP == 1 ? 8 : NP == 2 ? 4 : 2;  // tokens whose inputs are read at once
+    for (int t0 = off; t0 < end; t0 += AH) {
+      float2 xq[AH][NP], xk[AH][NP];
+#pragma unroll
+      for (int u = 0; u < AH; ++u)
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          xq[u][i] = cq[i].ahead(t0 + u, end);
+          xk[u][i] = ck[i].ahead(t0 + u, end);
+        }
+#pragma unroll
+      for (int u = 0; u < AH; ++u) {
+      const int t = t0 + u;
+      if (t >= end) break;
       float2 q[NP], k[NP];
-      conv_pairs<T, NP>(p, xr, st, fresh, t, 2 * lane, qb, p.d, odd, q);
-      conv_pairs<T, NP>(p, xr, st, fresh, t, 2 * lane, kb, p.d, odd, k);
       float qq = 0.f, kk = 0.f, qk = 0.f;
 #pragma unroll
       for (int i = 0; i < NP; ++i) {
+        q[i] = cq[i].token(t, xq[u][i]);
+        k[i] = ck[i].token(t, xk[u][i]);
         qq = fmaf(q[i].x, q[i].x, qq); qq = fmaf(q[i].y, q[i].y, qq);
         kk = fmaf(k[i].x, k[i].x, kk); kk = fmaf(k[i].y, k[i].y, kk);
         qk = fmaf(q[i].x, k[i].x, qk); qk = fmaf(q[i].y, k[i].y, qk);
@@ -152,39 +223,66 @@ delta_prepare_kernel(const DeltaPrep<T> p) {
         }
       }
       if (lane == 0) p.kq[(row0 + t) * p.G + slot] = qk * qi * ki;
+      }
     }
     if (off == 0) {
-      __syncwarp();                                  // read in pairs, replaced channel by channel
-      conv_state(p, xr, st, fresh, count, qb, p.d);
-      conv_state(p, xr, st, fresh, count, kb, p.d);
+      if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          cq[i].save(st, count, end == count);
+          ck[i].save(st, count, end == count);
+        }
+      } else {
+        conv_state(p, xr, st, fresh, count, qb, p.d);
+        conv_state(p, xr, st, fresh, count, kb, p.d);
+      }
     }
-    return;
-  }
-  const int h = slot - p.G, vb = 2 * p.G * p.d + h * p.e;
-  const bool odd = (p.e & 1) || (vb & 1);
-  for (int t = off; t < end; ++t)
+  } else if (slot < p.G + p.H) {
+    const int h = slot - p.G, vb = 2 * p.G * p.d + h * p.e;
     for (int c = 2 * lane; c < p.e; c += 64) {
-      float2 v[1];
-      conv_pairs<T, 1>(p, xr, st, fresh, t, c, vb, p.e, odd, v);
-      T* dst = p.v + ((row0 + t) * p.H + h) * p.es + c;        // es is even: the pair's second column exists
-      dst[0] = from_f<T>(v[0].x);
-      dst[1] = from_f<T>(v[0].y);
+      ConvPair<T, TAPS> cv;
+      cv.begin(p, xr, st, fresh, vb, c, p.e, off);
+      for (int t0 = off; t0 < end; t0 += 8) {
+        float2 xv[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) xv[u] = cv.ahead(t0 + u, end);
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+        const int t = t0 + u;
+        if (t >= end) break;
+        const float2 v = cv.token(t, xv[u]);
+        T* dst = p.v + ((row0 + t) * p.H + h) * p.es + c;      // es is even: the pair's second column exists
+        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(v.x, v.y);
+        else *reinterpret_cast<float2*>(dst) = v;
+        }
+      }
+      if (TAPS > 0 && off == 0) cv.save(st, count, end == count);
     }
-  const float rate = -expf(p.a_log[h]);
-  if (off + lane < end && lane < kPrepRows) {
-    const size_t r = row0 + off + lane;
-    const float beta = 1.f / (1.f + expf(-to_f(p.b[r * p.ldb + h])));
-    const float decay = p.g ? 1.f : expf(rate * softplus_of(to_f(p.a[r * p.lda + h]) + p.dt_bias[h]));
-    p.coef[r * p.H + h] = make_float2(beta, decay);
-  }
-  if (p.g)
-    for (int t = off; t < end; ++t)
-      for (int c = lane; c < p.ds; c += 32)
-        p.g[((row0 + t) * p.H + h) * p.ds + c] =
-            c < p.d ? expf(rate * softplus_of(to_f(p.a[(row0 + t) * p.lda + h * p.d + c]) + p.dt_bias[h * p.d + c])) : 0.f;
-  if (off == 0) {
-    __syncwarp();
-    conv_state(p, xr, st, fresh, count, vb, p.e);
+    if (off + lane < end && lane < kPrepRows) {
+      const size_t r = row0 + off + lane;
+      const float beta = 1.f / (1.f + expf(-to_f(p.b[r * p.ldb + h])));
+      const float decay =
+          p.g ? 1.f : expf(-expf(p.a_log[h]) * softplus_of<float>(to_f(p.a[r * p.lda + h]) + p.dt_bias[h]));
+      p.coef[r * p.H + h] = make_float2(beta, decay);
+    }
+    if (TAPS == 0 && off == 0) conv_state(p, xr, st, fresh, count, vb, p.e);
+  } else {
+    const int h = slot - p.G - p.H;
+    const float rate = -expf(p.a_log[h]);
+    for (int c = lane; c < p.ds; c += 32) {
+      const float dt = c < p.d ? p.dt_bias[h * p.d + c] : 0.f;
+      float* dst = p.g + (row0 * p.H + h) * p.ds + c;
+      const T* src = p.a + row0 * p.lda + h * p.d + c;
+      for (int t0 = off; t0 < end; t0 += 8) {
+        float v[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) v[u] = c < p.d && t0 + u < end ? to_f(src[static_cast<size_t>(t0 + u) * p.lda]) : 0.f;
+#pragma unroll
+        for (int u = 0; u < 8; ++u)
+          if (t0 + u < end)
+            dst[static_cast<size_t>(t0 + u) * p.H * p.ds] = c < p.d ? exp_of<T>(rate * softplus_of<T>(v[u] + dt)) : 0.f;
+      }
+    }
   }
 }
 
@@ -241,11 +339,12 @@ __device__ __forceinline__ void store_state(float* sp, int ds, int e, int v_firs
   }
 }
 
-// One token: decays the state, updates it with (k, v) and returns the outputs of the thread's rows (the same value in
-// all lanes of a row).  `get(which, c)` yields the float4 chunk c of q (0), k (1), g (2).
+// One token: decays the state, updates it with (k, v) and returns the output of ONE of the thread's rows: row l of the
+// thread for its row's lanes l < RPT (a lane l >= RPT repeats row l % RPT).  `get(which, c)` yields the float4 chunk c of q (0), k (1), g (2).
 template <int LPR, int RPT, bool CHANNEL, typename Get>
-__device__ __forceinline__ void delta_token(float2 (&S)[RPT][8], Get get, float beta, float decay, float kq,
-                                            const float (&va)[RPT], float (&o)[RPT]) {
+__device__ __forceinline__ float delta_token(float2 (&S)[RPT][8], Get get, float beta, float decay, float kq,
+                                             const float (&va)[RPT]) {
+  float o[RPT];
   float2 k2[8], aa[RPT], bb[RPT];
   const float2 g1 = make_float2(decay, decay);
 #pragma unroll
@@ -275,21 +374,44 @@ __device__ __forceinline__ void delta_token(float2 (&S)[RPT][8], Get get, float 
   float sa[RPT];
 #pragma unroll
   for (int i = 0; i < RPT; ++i) { sa[i] = aa[i].x + aa[i].y; o[i] = bb[i].x + bb[i].y; }
+  if constexpr (RPT == 4 && LPR >= 4) {
+    // the four rows' sums are dealt over the lanes while they are added (2 + 1 exchanges instead of 4 per step), then
+    // spread back: lane l ends with the totals of row l & 3
+    const int l = threadIdx.x % LPR;
+    const bool b0 = l & 1, b1 = l & 2;
+    const float a01 = (b0 ? sa[1] : sa[0]) + __shfl_xor_sync(0xffffffffu, b0 ? sa[0] : sa[1], 1);
+    const float a23 = (b0 ? sa[3] : sa[2]) + __shfl_xor_sync(0xffffffffu, b0 ? sa[2] : sa[3], 1);
+    const float o01 = (b0 ? o[1] : o[0]) + __shfl_xor_sync(0xffffffffu, b0 ? o[0] : o[1], 1);
+    const float o23 = (b0 ? o[3] : o[2]) + __shfl_xor_sync(0xffffffffu, b0 ? o[2] : o[3], 1);
+    float a = (b1 ? a23 : a01) + __shfl_xor_sync(0xffffffffu, b1 ? a01 : a23, 2);
+    float r = (b1 ? o23 : o01) + __shfl_xor_sync(0xffffffffu, b1 ? o01 : o23, 2);
 #pragma unroll
-  for (int sh = 1; sh < LPR; sh <<= 1)
-#pragma unroll
-    for (int i = 0; i < RPT; ++i) {
-      sa[i] += __shfl_xor_sync(0xffffffffu, sa[i], sh);
-      o[i] += __shfl_xor_sync(0xffffffffu, o[i], sh);
+    for (int sh = 4; sh < LPR; sh <<= 1) {
+      a += __shfl_xor_sync(0xffffffffu, a, sh);
+      r += __shfl_xor_sync(0xffffffffu, r, sh);
     }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) sa[i] = __shfl_sync(0xffffffffu, a, i, 4);
+    o[0] = r;                                        // the total of row l & 3: the caller's lane l stores that row
+  } else {
+#pragma unroll
+    for (int sh = 1; sh < LPR; sh <<= 1)
+#pragma unroll
+      for (int i = 0; i < RPT; ++i) {
+        sa[i] += __shfl_xor_sync(0xffffffffu, sa[i], sh);
+        o[i] += __shfl_xor_sync(0xffffffffu, o[i], sh);
+      }
+  }
+  float mine = 0.f;
 #pragma unroll
   for (int i = 0; i < RPT; ++i) {
     const float u = beta * (va[i] - sa[i]);
-    o[i] = fmaf(kq, u, o[i]);
+    if (RPT == 1 || (static_cast<int>(threadIdx.x) & 3) == i) mine = u;
     const float2 u2 = make_float2(u, u);
 #pragma unroll
     for (int c = 0; c < 8; ++c) S[i][c] = fma2(k2[c], u2, S[i][c]);
   }
+  return fmaf(kq, mine, o[0]);
 }
 
 template <int B>
@@ -378,16 +500,13 @@ delta_walk_kernel(const DeltaWalk<T> p) {
 #pragma unroll 1
     for (int j = 0; j < nb; ++j) {
       const float4 co = *reinterpret_cast<const float4*>(cf + j * 4);
-      float va[RPT], o[RPT];
+      float va[RPT];
 #pragma unroll
       for (int i = 0; i < RPT; ++i) va[i] = v0 + grp + i * ngrp < p.e ? to_f(vs[j * es + i * ngrp]) : 0.f;
-      delta_token<LPR, RPT, CHANNEL>(
+      const float o = delta_token<LPR, RPT, CHANNEL>(
           S, [&](int w, int c) { return *reinterpret_cast<const float4*>(buf + (w * NB + j) * KD + 4 * (l + LPR * c)); },
-          co.x, co.y, co.z, va, o);
-      if (l == 0) {
-#pragma unroll
-        for (int i = 0; i < RPT; ++i) ob[j * VT + i * ngrp] = o[i];
-      }
+          co.x, co.y, co.z, va);
+      if (l < RPT) ob[j * VT + l * ngrp] = o;
     }
   }
   __syncthreads();
@@ -418,41 +537,30 @@ delta_step_kernel(const DeltaWalk<T> p) {
   const float* gr = CHANNEL ? p.g + (r * p.H + head) * p.ds : nullptr;
   const float2 co = p.coef[r * p.H + head];
   const float kq = p.kq[r * p.G + hq];
-  float va[RPT], o[RPT];
+  float va[RPT];
 #pragma unroll
   for (int i = 0; i < RPT; ++i) {
     const int v = v0 + grp + i * ngrp;
     va[i] = v < p.e ? to_f(p.v[(r * p.H + head) * p.es + v]) : 0.f;
   }
-  delta_token<LPR, RPT, CHANNEL>(
+  const float o = delta_token<LPR, RPT, CHANNEL>(
       S,
       [&](int w, int c) {
         const int col = 4 * (l + LPR * c);
         const float* src = w == 0 ? qr : w == 1 ? kr : gr;
         return col < p.ds ? *reinterpret_cast<const float4*>(src + col) : make_float4(0.f, 0.f, 0.f, 0.f);
       },
-      co.x, co.y, kq, va, o);
+      co.x, co.y, kq, va);
   store_state<LPR, RPT>(sp, p.ds, p.e, v0 + grp, ngrp, l, S);
+  const int v_mine = v0 + grp + l * ngrp;              // the row this lane has the output of
+  const bool has = l < RPT && v_mine < p.e;
   if (p.raw) {
-    if (l == 0) {
-#pragma unroll
-      for (int i = 0; i < RPT; ++i)
-        if (v0 + grp + i * ngrp < p.e) p.raw[(r * p.H + head) * p.e + v0 + grp + i * ngrp] = o[i];
-    }
+    if (has) p.raw[(r * p.H + head) * p.e + v_mine] = o;
     return;
   }
   // gated norm: the whole head is in this block
-  float ss = 0.f;
-  if (l == 0) {
-#pragma unroll
-    for (int i = 0; i < RPT; ++i) {
-      const int v = grp + i * ngrp;
-      if (v < p.e) {
-        sm[v] = o[i];
-        ss = fmaf(o[i], o[i], ss);
-      }
-    }
-  }
+  if (has) sm[v_mine] = o;
+  float ss = has ? o * o : 0.f;
   ss = warp_sum(ss);
   if ((tid & 31) == 0) red[tid >> 5] = ss;
   __syncthreads();
@@ -527,7 +635,7 @@ static int delta_kd(DeltaWalk<T> p, bool channel, bool step, int tokens, float* 
   // four rows per thread amortise the operand loads; one row per thread spreads a head over more blocks when the step
   // has too few (head, request) pairs to fill the device
   const int max1 = 256 / LPR, max4 = max1 * 4;
-  const bool spread = !step && static_cast<long long>(p.H) * p.sg.num < 148;
+  const bool spread = !step && static_cast<long long>(p.H) * p.sg.num < 74;
   const int rpt = (spread || p.e <= max1 / 2) ? 1 : 4;
   const int max_rows = rpt == 4 ? max4 : max1;
   const int parts = (p.e + max_rows - 1) / max_rows;
@@ -611,13 +719,19 @@ static int prep_typed(const CbDeltaPrep* a, const CbSegments* seg, cudaStream_t 
   p.coef = static_cast<float2*>(a->coef);
   p.g = static_cast<float*>(a->g);
   p.H = a->H; p.G = a->G; p.d = a->d; p.e = a->e; p.ds = a->ds; p.es = a->es;
-  p.sg = make_segments(seg);
+  p.sg = make_segments(seg, a->tokens);
   const int tiles = max_tiles(a->tokens, seg->num, kPrepRows);
   if (tiles > 65535) return -11;
-  const dim3 grid((a->G + a->H + kPrepWarps - 1) / kPrepWarps, tiles);
-  if (a->d <= 64) return static_cast<int>(launch(delta_prepare_kernel<T, 1>, grid, dim3(32 * kPrepWarps), 0, st, p));
-  if (a->d <= 128) return static_cast<int>(launch(delta_prepare_kernel<T, 2>, grid, dim3(32 * kPrepWarps), 0, st, p));
-  return static_cast<int>(launch(delta_prepare_kernel<T, 4>, grid, dim3(32 * kPrepWarps), 0, st, p));
+  const dim3 grid((a->G + (a->g ? 2 : 1) * a->H + kPrepWarps - 1) / kPrepWarps, tiles);
+  auto go = [&](auto kernel) { return static_cast<int>(launch(kernel, grid, dim3(32 * kPrepWarps), 0, st, p)); };
+  const int taps = a->taps >= 2 && a->taps <= 4 && ((a->d | a->e) & 1) == 0 ? a->taps : 0;
+  if (a->d <= 64)
+    return taps == 2 ? go(delta_prepare_kernel<T, 1, 2>) : taps == 3 ? go(delta_prepare_kernel<T, 1, 3>)
+         : taps == 4 ? go(delta_prepare_kernel<T, 1, 4>) : go(delta_prepare_kernel<T, 1, 0>);
+  if (a->d <= 128)
+    return taps == 2 ? go(delta_prepare_kernel<T, 2, 2>) : taps == 3 ? go(delta_prepare_kernel<T, 2, 3>)
+         : taps == 4 ? go(delta_prepare_kernel<T, 2, 4>) : go(delta_prepare_kernel<T, 2, 0>);
+  return taps == 4 ? go(delta_prepare_kernel<T, 4, 4>) : go(delta_prepare_kernel<T, 4, 0>);
 }
 
 template <typename T>
@@ -634,7 +748,7 @@ static int walk_typed(const CbDeltaWalk* a, const CbSegments* seg, cudaStream_t 
   p.raw = nullptr;
   p.H = a->H; p.G = a->G; p.d = a->d; p.e = a->e; p.ds = a->ds; p.es = a->es;
   p.eps = a->eps; p.sigmoid_gate = a->sigmoid_gate;
-  p.sg = make_segments(seg);
+  p.sg = make_segments(seg, a->tokens);
   const bool channel = a->g != nullptr, step = a->decode != 0;
   float* raw = static_cast<float*>(a->raw);
   if (a->d <= 64) return delta_kd<T, 64>(p, channel, step, a->tokens, raw, st);

@@ -235,9 +235,24 @@ latent_attn_mma_kernel(const LatentMma p) {
 #pragma unroll
       for (int c = 0; c < 4; ++c) o[i][j][c] = 0.f;
 
+  // fragment addresses: the row of every fragment load is congruent to lane & 7 modulo 8, so the swizzled chunk depends on
+  // the position inside a 128-byte group only and everything else is an immediate offset
   const uint32_t q_base = smem_u32(qs) + (wm * 16 + (lane & 15)) * ROWB;
-  const uint32_t q_sw = (lane & 7);
-  const uint32_t p_base = smem_u32(ps);
+  const int n_row = wn * (NS * 8) + (lane & 7) + (NS > 1 ? (lane >> 4) << 3 : 0);
+  const uint32_t v_row = ((lane & 7) + ((lane >> 3) & 1) * 8) * ROWB;
+  uint32_t q_at[4], c_at[4], v_at[NT > 1 ? NT / 2 : 1];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    q_at[i] = q_base + (((i * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
+    c_at[i] = n_row * ROWB + (((i * 2 + ((lane >> 3) & 1)) ^ (lane & 7)) << 4);
+  }
+#pragma unroll
+  for (int j = 0; j < (NT > 1 ? NT / 2 : 1); ++j)
+    v_at[j] = v_row + (((warp * NT + 2 * j + (NT > 1 ? lane >> 4 : 0)) ^ (lane & 7)) << 4);
+  const uint32_t p_at0 = smem_u32(ps) + (lane & 15) * 128;
+  uint32_t p_at[kKeyTile / 16];
+#pragma unroll
+  for (int ks = 0; ks < kKeyTile / 16; ++ks) p_at[ks] = p_at0 + (((ks * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
   for (int t = t_lo; t < t_hi; ++t) {
     const int b = (t - t_lo) & 1;
     if (t + 1 < t_hi) load_tile(t + 1, b ^ 1);       // its buffer was released by the barrier that ended the last turn
@@ -251,16 +266,14 @@ latent_attn_mma_kernel(const LatentMma p) {
     for (int j = 0; j < NS; ++j)
 #pragma unroll
       for (int c = 0; c < 4; ++c) sfr[j][c] = sodd[j][c] = 0.f;
-    const int n_row = wn * (NS * 8) + (lane & 7) + (NS > 1 ? (lane >> 4) << 3 : 0);
 #pragma unroll
     for (int kk = 0; kk < RP / 16; ++kk) {
       uint32_t qa[4];
-      ldsm4(qa, q_base + (((kk * 2 + (lane >> 4)) ^ q_sw) << 4));
+      ldsm4(qa, q_at[kk & 3] + (kk >> 2) * 128);
 #pragma unroll
       for (int j = 0; j < NS; j += 2) {
         uint32_t cb[4];
-        const int r = n_row + j * 8;
-        const uint32_t addr = c_base + r * ROWB + (((kk * 2 + ((lane >> 3) & 1)) ^ (r & 7)) << 4);
+        const uint32_t addr = c_base + c_at[kk & 3] + (kk >> 2) * 128 + j * 8 * ROWB;
         if constexpr (NS == 1) {
           ldsm2(cb, addr);
           mma_bf16(kk & 1 ? sodd[j] : sfr[j], qa, cb[0], cb[1]);
@@ -327,18 +340,13 @@ latent_attn_mma_kernel(const LatentMma p) {
     for (int ks = 0; ks < kKeyTile / 16; ++ks) {
       uint32_t pa[MT][4];
 #pragma unroll
-      for (int i = 0; i < MT; ++i) {
-        const int r = i * 16 + (lane & 15);
-        ldsm4(pa[i], p_base + r * 128 + (((ks * 2 + (lane >> 4)) ^ (r & 7)) << 4));
-      }
-      const int r = ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
-      const uint32_t vrow = c_base + r * ROWB;
+      for (int i = 0; i < MT; ++i) ldsm4(pa[i], p_at[ks] + i * 16 * 128);
 #pragma unroll
       for (int j = 0; j < NT; j += 2) {
         uint32_t vb[4];
-        const int chunk = warp * NT + j;
-        if constexpr (NT == 1) ldsm2_t(vb, vrow + ((chunk ^ (r & 7)) << 4));
-        else ldsm4_t(vb, vrow + (((chunk + (lane >> 4)) ^ (r & 7)) << 4));
+        const uint32_t addr = c_base + v_at[j / 2] + ks * 16 * ROWB;
+        if constexpr (NT == 1) ldsm2_t(vb, addr);
+        else ldsm4_t(vb, addr);
 #pragma unroll
         for (int i = 0; i < MT; ++i) {
           mma_bf16(o[i][j], pa[i], vb[0], vb[1]);
@@ -453,16 +461,16 @@ template <int MR, int NCH>
 static int mma_go(const LatentMma& p, dim3 grid, cudaStream_t st) {
   constexpr int ROWB = NCH * 128, WN = 128 / MR;
   const size_t smem = static_cast<size_t>(MR) * ROWB + 2 * key_tile<MR>() * ROWB + MR * 128 + sizeof(float) * MR * (2 + 2 * WN);
+  auto kernel = latent_attn_mma_kernel<MR, NCH>;
   static bool configured[64] = {};     // per device
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -18;
   if (!configured[dev]) {
-    const cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<MR, NCH>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                               static_cast<int>(smem));
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev] = true;
   }
-  const cudaError_t rc = launch(latent_attn_mma_kernel<MR, NCH>, grid, dim3(256), smem, st, p);
+  const cudaError_t rc = launch(kernel, grid, dim3(256), smem, st, p);
   if (rc != cudaSuccess || p.splits == 1) return static_cast<int>(rc);
   return static_cast<int>(launch(latent_merge_kernel<NCH>, dim3(grid.x, grid.y, MR / 8), dim3(256), 0, st, p, MR));
 }
@@ -523,7 +531,7 @@ static int latent_attn_typed(const CbLatentAttn* a, const CbSegments* seg, cudaS
   p.gate = static_cast<const T*>(a->gate); p.ldg = a->ldg;
   p.page_table = static_cast<const int*>(a->page_table);
   p.max_pages = a->max_pages; p.H = a->H; p.Rp = a->Rp; p.window = a->window; p.scale = a->scale;
-  p.sg = make_segments(seg);
+  p.sg = make_segments(seg, a->tokens);
   const dim3 grid(a->tokens, (a->H + 3) / 4);
   if (a->Rp <= 64) return static_cast<int>(launch(latent_attn_kernel<T, 2>, grid, dim3(128), 0, st, p));
   if (a->Rp <= 128) return static_cast<int>(launch(latent_attn_kernel<T, 4>, grid, dim3(128), 0, st, p));
@@ -565,7 +573,7 @@ int cb_latent_attn(const CbLatentAttn* a, const CbSegments* seg, void* stream) {
     p.a.gate = static_cast<const __nv_bfloat16*>(a->gate); p.a.ldg = a->ldg;
     p.a.page_table = static_cast<const int*>(a->page_table);
     p.a.max_pages = a->max_pages; p.a.H = a->H; p.a.Rp = a->Rp; p.a.window = a->window; p.a.scale = a->scale;
-    p.a.sg = make_segments(seg);
+    p.a.sg = make_segments(seg, a->tokens);
     int mr;
     mma_shape(a->H, a->decode != 0, mr, p.hb, p.qb);
     p.splits = a->splits > 1 ? a->splits : 1;

@@ -12,6 +12,7 @@ struct Segments {
   const int* slot;      // [num] request slot: state row and page-table row
   const int* pos0;      // [num] absolute position of the first row (0 = fresh state)
   int num;
+  int single;           // every segment has at most one row, row s belongs to segment s (decode)
 };
 
 __device__ __forceinline__ float to_f(float v) { return v; }
@@ -24,6 +25,11 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float
 // segment.  Called by whole warps; false when the step has fewer tiles.  The grid of a kernel that uses it holds at
 // most (T + num (rows - 1)) / rows tiles.
 __device__ __forceinline__ bool find_tile(const Segments& sg, int rows, int tile, int& seg, int& off) {
+  if (sg.single) {
+    seg = tile;
+    off = 0;
+    return tile < sg.num && sg.count[tile] > 0;
+  }
   const int lane = threadIdx.x & 31;
   int base = 0;
   for (int s0 = 0; s0 < sg.num; s0 += 32) {
@@ -65,8 +71,9 @@ struct CbSegments {
 }
 
 namespace cb {
-static inline Segments make_segments(const CbSegments* s) {
+// `tokens`: rows of the step; as many rows as segments means one row each
+static inline Segments make_segments(const CbSegments* s, int tokens) {
   return Segments{static_cast<const int*>(s->row0), static_cast<const int*>(s->count), static_cast<const int*>(s->slot),
-                  static_cast<const int*>(s->pos0), s->num};
+                  static_cast<const int*>(s->pos0), s->num, tokens == s->num ? 1 : 0};
 }
 }  // namespace cb

@@ -12,10 +12,10 @@ and one pass over the whole sequence give the same logits.
 from __future__ import annotations
 
 import copy
-import math
 
-import numpy as np
 import torch
+
+from ..executor.stateful_executor import StatefulEagerExecutor
 
 
 # ------------------------------------------------------------------ mechanisms
@@ -188,3 +188,19 @@ class OracleState:
 
     def copy(self) -> "OracleState":
         return copy.deepcopy(self)
+
+
+class LayeredEagerExecutor(StatefulEagerExecutor):
+    """``execute(segments)`` of the eager execution mode: one explicit state per request slot (no pages, no prefix sharing)."""
+
+    accepts_features = False
+
+    def __init__(self, cfg, weights: dict[str, torch.Tensor], raw_config: dict | None = None) -> None:
+        self.cfg = cfg
+        super().__init__(Oracle(raw_config if raw_config is not None else cfg.to_config(), weights))
+
+    def _new_state(self) -> OracleState:
+        return self.model.new_state()
+
+    def _copy(self, state: OracleState) -> OracleState:
+        return state.copy()

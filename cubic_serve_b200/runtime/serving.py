@@ -57,6 +57,8 @@ def plan_kv_pages(free_bytes: int, reserve_bytes: int, cfg, tp: int, k_bits: int
     """Pages that fit in the remaining device memory (one page = 16 tokens of every local layer's rank-local KV
     heads; ``layers`` = decoder layers held by this pipeline stage, default all)."""
     from ..contracts.model import CacheSpec, ModelSpec, StateSpec
+    if getattr(cfg, "family", "") == "layered":
+        return ModelSpec.from_layered(cfg).kv_pages(free_bytes, reserve_bytes, max_model_len, max_running, state_snapshots)
     n_layers = layers or cfg.num_layers
     n_gdn = sum(cfg.layer_is_gdn(i) for i in range(cfg.num_layers)) if layers is None else 0
     from ..models.config import kv_heads_of_rank
@@ -75,6 +77,8 @@ def build_backend(args, devices: list[int], tp: int, spec, k_bits: int, v_bits: 
     from ..runtime.engine import LLMEngine
     from ..runtime.scheduler import SchedulerConfig
     if tp != 1 or args.pp_size != 1:
+        if _is_layered(args.model):
+            raise SystemExit("layered decoders are served on one GPU")
         from ..executor.multiproc import build_multiproc_backend
         for flag in ("startup_numerical_audit", "tune_launch_plans"):
             if getattr(args, flag, False):
@@ -82,6 +86,13 @@ def build_backend(args, devices: list[int], tp: int, spec, k_bits: int, v_bits: 
                             "(run `cubic qualify` on one GPU of the node instead)", flag.replace("_", "-"))
         return build_multiproc_backend(args, devices, tp, spec, k_bits, v_bits)
     model = args.model
+    layered = _is_layered(model)
+    if layered and spec is not None and getattr(spec, "method", "none") != "none":
+        raise SystemExit("layered decoders have no draft head and no review pass over their recurrent state: serve without "
+                         "--speculative-config")
+    if getattr(args, "dtype", "bfloat16") != "bfloat16" and not layered:
+        raise SystemExit("--dtype float32 is available for the layered decoders; use --execution-mode eager for fp32 arithmetic "
+                         "of the other families")
     eager = args.execution_mode != "cuda" or not torch.cuda.is_available()
     gguf_weights = None
     if model.startswith("random:"):
@@ -104,6 +115,11 @@ def build_backend(args, devices: list[int], tp: int, spec, k_bits: int, v_bits: 
         from ..models.checkpoint import admit_checkpoint
         ck = admit_checkpoint(model)
         cfg = ck.cfg
+    if layered:
+        from ..models.layered import with_dtype
+        cfg = with_dtype(cfg, getattr(args, "dtype", "bfloat16"))
+        if ck is not None:
+            ck.cfg = cfg
     max_len = args.max_model_len or min(cfg.max_position, 8192)
     sched = SchedulerConfig(max_running_requests=args.max_running_requests, max_batched_tokens=args.token_budget,
                             prefill_chunk_tokens=min(args.prefill_chunk_tokens, args.token_budget), max_model_len=max_len,
@@ -114,7 +130,12 @@ def build_backend(args, devices: list[int], tp: int, spec, k_bits: int, v_bits: 
         if gguf_weights is not None:
             raise SystemExit("eager execution mode serves checkpoint directories and random:<config> models")
         pages = 4096
-        if cfg.is_moe or cfg.is_hybrid or cfg.qkv_bias:
+        if layered:
+            from ..models.layered import random_tensors
+            from ..models.layered_reference import LayeredEagerExecutor
+            tensors = {n: ck.store.get(n) for n in ck.plain} if ck is not None else random_tensors(cfg, args.seed)
+            executor = LayeredEagerExecutor(cfg, tensors, None if ck is None else ck.raw_config)
+        elif cfg.is_moe or cfg.is_hybrid or cfg.qkv_bias:
             # the families beyond the dense full-attention decoder (experts, shared experts, Gated DeltaNet layers,
             # projection biases, any head width) run on the eager family model with per-request state
             from ..models.eager_family import EagerFamilyExecutor, family_weights_from_checkpoint, random_family_weights
@@ -187,7 +208,9 @@ def build_backend(args, devices: list[int], tp: int, spec, k_bits: int, v_bits: 
                 runner.enable_reasoning_budget(*think)       # thinking-token budgets are enforced on the device
             executor = GpuExecutor(runner, max_rows=args.max_running_requests, max_prefill_tokens=args.token_budget,
                                    max_model_len=max_len)
-            if getattr(args, "tune_launch_plans", False):
+            if getattr(args, "tune_launch_plans", False) and layered:
+                log.warning("--tune-launch-plans measures the quantized projections; layered decoders use the built-in rules")
+            elif getattr(args, "tune_launch_plans", False):
                 # measured launch form per (projection, decode capacity); kept as start-up evidence, so measured once
                 from ..contracts.implementation import identity
                 from ..ops import autotune
@@ -224,6 +247,20 @@ def _gguf_architecture(path: str) -> str | None:
     import gguf
     f = gguf.GGUFReader(str(path)).fields.get("general.architecture")
     return None if f is None else bytes(f.parts[f.data[0]]).decode()
+
+
+def _is_layered(model: str) -> bool:
+    """Whether ``model`` (checkpoint directory or random:<config>) is a layered decoder (``models/layered.py``)."""
+    import json
+
+    from ..models.layered import NAMED, architecture_of
+    if model.startswith("random:"):
+        return model.split(":", 1)[1] in NAMED
+    p = Path(model) / "config.json"
+    try:
+        return p.is_file() and architecture_of(json.loads(p.read_text())) is not None
+    except (OSError, ValueError):
+        return False
 
 
 def _model_type_of(model: str) -> str | None:
