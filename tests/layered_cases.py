@@ -1,0 +1,114 @@
+"""Configurations and weights of the layered-decoder tests: raw ``config.json`` dictionaries and seeded tensors, made here
+without the product's own helpers."""
+from __future__ import annotations
+
+import math
+
+import torch
+
+
+def delta(heads, kv_heads, dim, vdim, conv, ff):
+    return {"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def channel(heads, kv_heads, dim, vdim, conv, ff):
+    return {**delta(heads, kv_heads, dim, vdim, conv, ff), "type": "channel_delta"}
+
+
+def latent(heads, dim, vdim, q_rank, kv_rank, size, scale, ff):
+    return {"type": "latent_attention",
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "scale": scale,
+                      "mask": {"size": size} if size else None},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def config(vocab, width, layers, loop=None, eps=1e-5):
+    return {"architecture": "Bumodra", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": eps},
+            "loop": dict(zip(("start", "stop", "times"), loop)) if loop else None}
+
+
+CASES = {
+    # every mixer, a loop in the middle, a layer without a feed-forward
+    "all": config(200, 96, [delta(4, 2, 24, 40, 4, 96), latent(5, 16, 24, 40, 48, 19, 0.3, 72), channel(3, 3, 32, 16, 2, 0),
+                            latent(2, 32, 16, 32, 64, 33, 0.2, 64)], (1, 3, 2), 1e-6),
+    # no loop; one head; equal and unit sizes; a single tap; a window of one token
+    "small": config(70, 64, [latent(1, 16, 16, 16, 16, 1, 0.25, 64), delta(1, 1, 16, 16, 1, 64), channel(2, 1, 8, 12, 3, 48)],
+                    None, 1e-5),
+    # odd widths, many taps, the whole model looped three times, full attention
+    "odd": config(123, 68, [channel(2, 2, 7, 9, 5, 44), delta(6, 3, 20, 13, 3, 36), latent(3, 12, 20, 24, 20, 0, 0.35, 40)],
+                  (0, 3, 3), 1e-4),
+    # wide heads, a loop that runs once, many heads of attention, window over several pages
+    "wide": config(256, 128, [delta(2, 1, 128, 144, 4, 128), latent(40, 8, 8, 64, 136, 50, 0.35, 0),
+                              channel(2, 1, 160, 64, 4, 96)], (2, 3, 1), 1e-6),
+}
+LOW_RANKS = (12, 20)          # inner sizes of the low-rank decay and gate projections
+
+
+def tensors(cfg: dict, seed: int = 0) -> dict[str, torch.Tensor]:
+    g = torch.Generator().manual_seed(seed)
+    W, out = cfg["width"], {}
+
+    def mat(name, n, k, gain=1.0):
+        out[name] = (torch.randn(n, k, generator=g) * gain / math.sqrt(k)).to(torch.bfloat16)
+
+    def vec(name, n, mean=0.0, std=0.2):
+        out[name] = (mean + std * torch.randn(n, generator=g)).to(torch.bfloat16)
+
+    mat("embed", cfg["vocab"], W, math.sqrt(W))
+    vec("embed.norm", W)
+    vec("final.norm", W)
+    mat("head", cfg["vocab"], W)
+    if cfg["loop"]:
+        mat("loop.in", W, 2 * W)
+    for i, l in enumerate(cfg["layers"]):
+        m, p = l["mixer"], f"l{i}.mix"
+        vec(f"l{i}.norm1", W)
+        H, e = m["heads"], m["vdim"]
+        if l["type"] == "latent_attention":
+            mat(f"{p}.dq", m["q_rank"], W)
+            vec(f"{p}.dq.norm", m["q_rank"], 1.0)
+            mat(f"{p}.uq", H * m["dim"], m["q_rank"], 2.0)
+            mat(f"{p}.dkv", m["kv_rank"], W)
+            vec(f"{p}.dkv.norm", m["kv_rank"], 1.0)
+            mat(f"{p}.uk", H * m["dim"], m["kv_rank"], 2.0)
+            mat(f"{p}.uv", H * e, m["kv_rank"])
+            mat(f"{p}.g", H, W)
+        else:
+            for t, c in (("q", m["kv_heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", H * e)):
+                mat(f"{p}.{t}", c, W)
+                mat(f"{p}.{t}.conv", c, m["conv"])
+            mat(f"{p}.b", H, W)
+            vec(f"{p}.A_log", H, -1.5, 0.5)
+            vec(f"{p}.norm", e, 1.0)
+            if l["type"] == "channel_delta":
+                ra, rg = LOW_RANKS
+                mat(f"{p}.a1", ra, W)
+                mat(f"{p}.a2", H * m["dim"], ra)
+                vec(f"{p}.dt_bias", H * m["dim"], 0.0, 0.5)
+                mat(f"{p}.g1", rg, W)
+                mat(f"{p}.g2", H * e, rg)
+            else:
+                mat(f"{p}.a", H, W)
+                vec(f"{p}.dt_bias", H, 0.0, 0.5)
+                mat(f"{p}.g", H * e, W)
+        mat(f"{p}.o", W, H * e)
+        if l["mlp"]:
+            mat(f"l{i}.mlp.up", l["mlp"]["ff"], W)
+            mat(f"l{i}.mlp.down", W, l["mlp"]["ff"])
+    return out
+
+
+def write(path, cfg: dict, weights: dict[str, torch.Tensor]):
+    import json
+
+    from safetensors.torch import save_file
+    path.mkdir(parents=True, exist_ok=True)
+    save_file(weights, str(path / "model.safetensors"))
+    (path / "config.json").write_text(json.dumps(cfg))
+    return path
+
+
+def prompt(cfg: dict, n: int, seed: int) -> list[int]:
+    g = torch.Generator().manual_seed(1000 + seed)
+    return torch.randint(0, cfg["vocab"], (n,), generator=g).tolist()
