@@ -157,8 +157,9 @@ __device__ __forceinline__ void conv_state(const DeltaPrep<T>& p, const T* xr, T
 }
 
 // A warp per (slot, tile of kPrepRows tokens): slots [0, G) are key heads (q and k), [G, G + H) value heads (v, step size,
-// decay per head), [G + H, G + 2 H) channel decays.  NP: channel pairs per lane of a key head (d <= 64 NP).
-template <typename T, int NP, int TAPS>
+// decay per head), [G + H, G + 2 H) channel decays.  NP: channel pairs per lane of a key head (d <= 64 NP).  STEP: segments of
+// one token (decode): nothing is read ahead, which leaves registers for more warps.
+template <typename T, int NP, int TAPS, bool STEP>
 __global__ void __launch_bounds__(32 * kPrepWarps)
 delta_prepare_kernel(const DeltaPrep<T> p) {
   pdl_wait();
@@ -182,7 +183,7 @@ delta_prepare_kernel(const DeltaPrep<T> p) {
       cq[i].begin(p, xr, st, fresh, qb, 2 * lane + 64 * i, p.d, off);
       ck[i].begin(p, xr, st, fresh, kb, 2 * lane + 64 * i, p.d, off);
     }
-    constexpr int AH = NP == 1 ? 8 : NP == 2 ? 4 : 2;  // tokens whose inputs are read at once
+    constexpr int AH = STEP ? 1 : NP == 1 ? 8 : NP == 2 ? 4 : 2;  // tokens whose inputs are read at once
     for (int t0 = off; t0 < end; t0 += AH) {
       float2 xq[AH][NP], xk[AH][NP];
 #pragma unroll
@@ -239,24 +240,35 @@ delta_prepare_kernel(const DeltaPrep<T> p) {
     }
   } else if (slot < p.G + p.H) {
     const int h = slot - p.G, vb = 2 * p.G * p.d + h * p.e;
-    for (int c = 2 * lane; c < p.e; c += 64) {
-      ConvPair<T, TAPS> cv;
-      cv.begin(p, xr, st, fresh, vb, c, p.e, off);
-      for (int t0 = off; t0 < end; t0 += 8) {
-        float2 xv[8];
+    constexpr int AH = STEP ? 1 : 4;
+    for (int c0 = 2 * lane; c0 < p.e; c0 += 128) {             // two pairs at a time
+      ConvPair<T, TAPS> cv[2];
 #pragma unroll
-        for (int u = 0; u < 8; ++u) xv[u] = cv.ahead(t0 + u, end);
+      for (int i = 0; i < 2; ++i) cv[i].begin(p, xr, st, fresh, vb, c0 + 64 * i, p.e, off);
+      for (int t0 = off; t0 < end; t0 += AH) {
+        float2 xv[AH][2];
 #pragma unroll
-        for (int u = 0; u < 8; ++u) {
-        const int t = t0 + u;
-        if (t >= end) break;
-        const float2 v = cv.token(t, xv[u]);
-        T* dst = p.v + ((row0 + t) * p.H + h) * p.es + c;      // es is even: the pair's second column exists
-        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(v.x, v.y);
-        else *reinterpret_cast<float2*>(dst) = v;
+        for (int u = 0; u < AH; ++u)
+#pragma unroll
+          for (int i = 0; i < 2; ++i) xv[u][i] = cv[i].ahead(t0 + u, end);
+#pragma unroll
+        for (int u = 0; u < AH; ++u) {
+          const int t = t0 + u;
+          if (t >= end) break;
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const float2 v = cv[i].token(t, xv[u][i]);
+            T* dst = p.v + ((row0 + t) * p.H + h) * p.es + c0 + 64 * i;      // es is even: the pair's second column exists
+            if (!cv[i].ok) continue;
+            if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(v.x, v.y);
+            else *reinterpret_cast<float2*>(dst) = v;
+          }
         }
       }
-      if (TAPS > 0 && off == 0) cv.save(st, count, end == count);
+      if (TAPS > 0 && off == 0) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) cv[i].save(st, count, end == count);
+      }
     }
     if (off + lane < end && lane < kPrepRows) {
       const size_t r = row0 + off + lane;
@@ -269,18 +281,27 @@ delta_prepare_kernel(const DeltaPrep<T> p) {
   } else {
     const int h = slot - p.G - p.H;
     const float rate = -expf(p.a_log[h]);
-    for (int c = lane; c < p.ds; c += 32) {
-      const float dt = c < p.d ? p.dt_bias[h * p.d + c] : 0.f;
-      float* dst = p.g + (row0 * p.H + h) * p.ds + c;
-      const T* src = p.a + row0 * p.lda + h * p.d + c;
-      for (int t0 = off; t0 < end; t0 += 8) {
-        float v[8];
+    constexpr int AH = STEP ? 1 : 4;
+    for (int c0 = lane; c0 < p.ds; c0 += 128) {                // four channels x AH tokens read at once
+      float dt[4];
 #pragma unroll
-        for (int u = 0; u < 8; ++u) v[u] = c < p.d && t0 + u < end ? to_f(src[static_cast<size_t>(t0 + u) * p.lda]) : 0.f;
+      for (int i = 0; i < 4; ++i) dt[i] = c0 + 32 * i < p.d ? p.dt_bias[h * p.d + c0 + 32 * i] : 0.f;
+      float* dst = p.g + (row0 * p.H + h) * p.ds + c0;
+      const T* src = p.a + row0 * p.lda + h * p.d + c0;
+      for (int t0 = off; t0 < end; t0 += AH) {
+        float v[AH][4];
 #pragma unroll
-        for (int u = 0; u < 8; ++u)
-          if (t0 + u < end)
-            dst[static_cast<size_t>(t0 + u) * p.H * p.ds] = c < p.d ? exp_of<T>(rate * softplus_of<T>(v[u] + dt)) : 0.f;
+        for (int u = 0; u < AH; ++u)
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            v[u][i] = c0 + 32 * i < p.d && t0 + u < end ? to_f(src[static_cast<size_t>(t0 + u) * p.lda + 32 * i]) : 0.f;
+#pragma unroll
+        for (int u = 0; u < AH; ++u)
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            if (t0 + u < end && c0 + 32 * i < p.ds)
+              dst[static_cast<size_t>(t0 + u) * p.H * p.ds + 32 * i] =
+                  c0 + 32 * i < p.d ? exp_of<T>(rate * softplus_of<T>(v[u][i] + dt[i])) : 0.f;
       }
     }
   }
@@ -725,13 +746,12 @@ static int prep_typed(const CbDeltaPrep* a, const CbSegments* seg, cudaStream_t 
   const dim3 grid((a->G + (a->g ? 2 : 1) * a->H + kPrepWarps - 1) / kPrepWarps, tiles);
   auto go = [&](auto kernel) { return static_cast<int>(launch(kernel, grid, dim3(32 * kPrepWarps), 0, st, p)); };
   const int taps = a->taps >= 2 && a->taps <= 4 && ((a->d | a->e) & 1) == 0 ? a->taps : 0;
-  if (a->d <= 64)
-    return taps == 2 ? go(delta_prepare_kernel<T, 1, 2>) : taps == 3 ? go(delta_prepare_kernel<T, 1, 3>)
-         : taps == 4 ? go(delta_prepare_kernel<T, 1, 4>) : go(delta_prepare_kernel<T, 1, 0>);
-  if (a->d <= 128)
-    return taps == 2 ? go(delta_prepare_kernel<T, 2, 2>) : taps == 3 ? go(delta_prepare_kernel<T, 2, 3>)
-         : taps == 4 ? go(delta_prepare_kernel<T, 2, 4>) : go(delta_prepare_kernel<T, 2, 0>);
-  return taps == 4 ? go(delta_prepare_kernel<T, 4, 4>) : go(delta_prepare_kernel<T, 4, 0>);
+  const bool step = p.sg.single != 0;
+#define CB_PREP(NP, TAPS) (step ? go(delta_prepare_kernel<T, NP, TAPS, true>) : go(delta_prepare_kernel<T, NP, TAPS, false>))
+  if (a->d <= 64) return taps == 2 ? CB_PREP(1, 2) : taps == 3 ? CB_PREP(1, 3) : taps == 4 ? CB_PREP(1, 4) : CB_PREP(1, 0);
+  if (a->d <= 128) return taps == 2 ? CB_PREP(2, 2) : taps == 3 ? CB_PREP(2, 3) : taps == 4 ? CB_PREP(2, 4) : CB_PREP(2, 0);
+  return taps == 4 ? CB_PREP(4, 4) : CB_PREP(4, 0);
+#undef CB_PREP
 }
 
 template <typename T>
