@@ -366,10 +366,10 @@ template <int LPR, int RPT, bool CHANNEL, typename Get>
 __device__ __forceinline__ float delta_token(float2 (&S)[RPT][8], Get get, float beta, float decay, float kq,
                                              const float (&va)[RPT]) {
   float o[RPT];
-  float2 k2[8], aa[RPT], bb[RPT];
+  float2 k2[8], aa[RPT], bb[RPT], a2[RPT], b2[RPT];   // two chains per sum
   const float2 g1 = make_float2(decay, decay);
 #pragma unroll
-  for (int i = 0; i < RPT; ++i) { aa[i] = make_float2(0.f, 0.f); bb[i] = make_float2(0.f, 0.f); }
+  for (int i = 0; i < RPT; ++i) aa[i] = bb[i] = a2[i] = b2[i] = make_float2(0.f, 0.f);
 #pragma unroll
   for (int c = 0; c < 4; ++c) {
     const float4 q4 = get(0, c), k4 = get(1, c);
@@ -388,13 +388,25 @@ __device__ __forceinline__ float delta_token(float2 (&S)[RPT][8], Get get, float
       S[i][2 * c + 1] = mul2(S[i][2 * c + 1], gb);
       aa[i] = fma2(S[i][2 * c], k2[2 * c], aa[i]);
       bb[i] = fma2(S[i][2 * c], q0, bb[i]);
-      aa[i] = fma2(S[i][2 * c + 1], k2[2 * c + 1], aa[i]);
-      bb[i] = fma2(S[i][2 * c + 1], q1, bb[i]);
+      if constexpr (RPT == 1) {
+        a2[i] = fma2(S[i][2 * c + 1], k2[2 * c + 1], a2[i]);
+        b2[i] = fma2(S[i][2 * c + 1], q1, b2[i]);
+      } else {
+        aa[i] = fma2(S[i][2 * c + 1], k2[2 * c + 1], aa[i]);
+        bb[i] = fma2(S[i][2 * c + 1], q1, bb[i]);
+      }
     }
   }
   float sa[RPT];
 #pragma unroll
-  for (int i = 0; i < RPT; ++i) { sa[i] = aa[i].x + aa[i].y; o[i] = bb[i].x + bb[i].y; }
+  for (int i = 0; i < RPT; ++i) {
+    if constexpr (RPT == 1) {
+      aa[i].x += a2[i].x; aa[i].y += a2[i].y;
+      bb[i].x += b2[i].x; bb[i].y += b2[i].y;
+    }
+    sa[i] = aa[i].x + aa[i].y;
+    o[i] = bb[i].x + bb[i].y;
+  }
   if constexpr (RPT == 4 && LPR >= 4) {
     // the four rows' sums are dealt over the lanes while they are added (2 + 1 exchanges instead of 4 per step), then
     // spread back: lane l ends with the totals of row l & 3
@@ -442,9 +454,13 @@ __device__ __forceinline__ void cp_async(void* dst, const void* src) {
 }
 
 // Segments of many tokens: NB tokens' operands arrive by cp.async while the previous NB are walked; one barrier per NB
-// tokens.  Outputs leave through shared memory, before the norm.
+// tokens.  Outputs leave through shared memory, before the norm.  With one row per thread (few blocks: the chain of tokens
+// is what takes the time) kHelpers more threads do the copies in and out.
+static constexpr int kHelpers = 128;
+template <int RPT> constexpr int helper_threads() { return RPT == 1 ? kHelpers : 0; }
+
 template <typename T, int KD, int RPT, bool CHANNEL>
-__global__ void __launch_bounds__(256, 2)
+__global__ void __launch_bounds__(256 + helper_threads<RPT>(), RPT == 1 ? 1 : 2)
 delta_walk_kernel(const DeltaWalk<T> p) {
   constexpr int LPR = DeltaShape<KD>::LPR, NB = DeltaShape<KD>::NB, OPS = CHANNEL ? 3 : 2;
   extern __shared__ __align__(16) float sm[];
@@ -453,42 +469,51 @@ delta_walk_kernel(const DeltaWalk<T> p) {
   const int head = blockIdx.x, s = blockIdx.y;
   const int n = p.sg.count[s];
   if (n <= 0) return;
-  const int VT = blockDim.x / LPR * RPT;              // value rows of this block
+  constexpr int HELP = helper_threads<RPT>();
+  const int row_threads = blockDim.x - HELP;
+  const int VT = row_threads / LPR * RPT;             // value rows of this block
   const int v0 = blockIdx.z * VT, e_here = min(VT, p.e - v0);
   const int es = p.es;
   // per buffer: operands [OPS][NB][KD], coefficients [NB] float4, value rows [NB][es] (the whole head's, T)
   const int buf_floats = NB * (OPS * KD + 4) + NB * es * static_cast<int>(sizeof(T)) / 4;
   float* const obuf = sm + 2 * buf_floats;            // [2][NB][VT]
   const int tid = threadIdx.x;
-  const int l = tid % LPR, grp = tid / LPR, ngrp = blockDim.x / LPR;
+  const int l = tid % LPR, grp = tid / LPR, ngrp = row_threads / LPR;
+  const bool rower = tid < row_threads, copier = HELP == 0 || !rower;
   const size_t row0 = p.sg.row0[s];
   const int hq = head / (p.H / p.G);
   float* sp = p.state + (static_cast<size_t>(p.sg.slot[s]) * p.H + head) * p.e * p.ds;
   float2 S[RPT][8];
-  load_state<LPR, RPT>(sp, p.ds, p.e, v0 + grp, ngrp, l, p.sg.pos0[s] != 0, S);
+  load_state<LPR, RPT>(sp, p.ds, p.e, v0 + grp, ngrp, l, rower && p.sg.pos0[s] != 0, S);
 
   auto coefs = [&](int b) { return sm + b * buf_floats + NB * OPS * KD; };
   auto values = [&](int b) { return reinterpret_cast<T*>(sm + b * buf_floats + NB * (OPS * KD + 4)); };
   const int chunks = p.ds / 4, vchunks = es * static_cast<int>(sizeof(T)) / 16;
-  auto fetch = [&](int blk) {
+  const int warp = (tid - (HELP ? row_threads : 0)) >> 5, lane = tid & 31, warps = (HELP ? HELP : row_threads) >> 5;
+  auto fetch = [&](int blk) {                         // a warp per token row
     const int t0 = blk * NB, nb = min(NB, n - t0), b = blk & 1;
     float* buf = sm + b * buf_floats;
-    for (int i = tid; i < nb * chunks; i += blockDim.x) {
-      const int j = i / chunks, c = (i - j * chunks) * 4;
-      const size_t r = row0 + t0 + j;
-      cp_async<16>(buf + j * KD + c, p.q + (r * p.G + hq) * p.ds + c);
-      cp_async<16>(buf + (NB + j) * KD + c, p.k + (r * p.G + hq) * p.ds + c);
-      if constexpr (CHANNEL) cp_async<16>(buf + (2 * NB + j) * KD + c, p.g + (r * p.H + head) * p.ds + c);
-    }
     T* vs = values(b);
-    for (int i = tid; i < nb * vchunks; i += blockDim.x) {
-      const int j = i / vchunks, c = (i - j * vchunks) * (16 / static_cast<int>(sizeof(T)));
-      cp_async<16>(vs + j * es + c, p.v + ((row0 + t0 + j) * p.H + head) * es + c);
-    }
-    if (tid < nb) {
-      const size_t r = row0 + t0 + tid;
-      cp_async<8>(coefs(b) + tid * 4, p.coef + r * p.H + head);
-      cp_async<4>(coefs(b) + tid * 4 + 2, p.kq + r * p.G + hq);
+    for (int j = warp; j < nb; j += warps) {
+      const size_t r = row0 + t0 + j;
+      const float* qr = p.q + (r * p.G + hq) * p.ds;
+      const float* kr = p.k + (r * p.G + hq) * p.ds;
+#pragma unroll
+      for (int i = 0; i < (KD + 127) / 128; ++i) {
+        const int c = lane + 32 * i;
+        if (c < chunks) {
+          cp_async<16>(buf + j * KD + c * 4, qr + c * 4);
+          cp_async<16>(buf + (NB + j) * KD + c * 4, kr + c * 4);
+          if constexpr (CHANNEL) cp_async<16>(buf + (2 * NB + j) * KD + c * 4, p.g + (r * p.H + head) * p.ds + c * 4);
+        }
+      }
+      const T* vr = p.v + (r * p.H + head) * es;
+      for (int c = lane; c < vchunks; c += 32) {
+        constexpr int E = 16 / static_cast<int>(sizeof(T));
+        cp_async<16>(vs + j * es + c * E, vr + c * E);
+      }
+      if (lane == 0) cp_async<8>(coefs(b) + j * 4, p.coef + r * p.H + head);
+      if (lane == 1) cp_async<4>(coefs(b) + j * 4 + 2, p.kq + r * p.G + hq);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -501,24 +526,27 @@ delta_walk_kernel(const DeltaWalk<T> p) {
   auto put = [&](int blk) {                           // outputs of block blk to memory
     const int t0 = blk * NB, nb = min(NB, n - t0);
     const float* ob = obuf + (blk & 1) * NB * VT;
-    for (int i = tid; i < nb * VT; i += blockDim.x) {
-      const int j = i / VT, v = i - j * VT;
-      if (v < e_here) p.raw[(row0 + t0 + j) * (static_cast<size_t>(p.H) * p.e) + head * p.e + v0 + v] = ob[i];
+    for (int j = warp; j < nb; j += warps) {
+      float* dst = p.raw + (row0 + t0 + j) * (static_cast<size_t>(p.H) * p.e) + head * p.e + v0;
+      for (int v = lane; v < e_here; v += 32) dst[v] = ob[j * VT + v];
     }
   };
   const int blocks = (n + NB - 1) / NB;
-  fetch(0);
+  if (copier) fetch(0);
   for (int blk = 0; blk < blocks; ++blk) {
     const int b = blk & 1, nb = min(NB, n - blk * NB);
-    asm volatile("cp.async.wait_all;" ::: "memory");
+    if (copier) asm volatile("cp.async.wait_all;" ::: "memory");
     __syncthreads();                                  // operands of blk are here; everybody has left blk - 1
-    if (blk + 1 < blocks) fetch(blk + 1);
-    if (blk > 0) put(blk - 1);
+    if (copier) {
+      if (blk + 1 < blocks) fetch(blk + 1);
+      if (blk > 0) put(blk - 1);
+    }
+    if (HELP && !rower) continue;
     const float* buf = sm + b * buf_floats;
     const float* cf = coefs(b);
     const T* vs = values(b) + v0 + grp;
     float* ob = obuf + b * NB * VT + grp;
-#pragma unroll 1
+#pragma unroll (RPT == 1 ? 4 : 1)
     for (int j = 0; j < nb; ++j) {
       const float4 co = *reinterpret_cast<const float4*>(cf + j * 4);
       float va[RPT];
@@ -531,8 +559,8 @@ delta_walk_kernel(const DeltaWalk<T> p) {
     }
   }
   __syncthreads();
-  put(blocks - 1);
-  store_state<LPR, RPT>(sp, p.ds, p.e, v0 + grp, ngrp, l, S);
+  if (copier) put(blocks - 1);
+  if (rower) store_state<LPR, RPT>(sp, p.ds, p.e, v0 + grp, ngrp, l, S);
 }
 
 // Segments of one token.  The state's loads go out first; the operands are a few cached rows.
@@ -646,7 +674,7 @@ static int delta_go(const DeltaWalk<T>& p, int threads, int vtiles, cudaStream_t
       configured[dev] = true;
     }
     if (smem > 200 * 1024) return -14;
-    return static_cast<int>(launch(kernel, grid, dim3(threads), smem, st, p));
+    return static_cast<int>(launch(kernel, grid, dim3(threads + helper_threads<RPT>()), smem, st, p));
   }
 }
 
@@ -658,7 +686,13 @@ static int delta_kd(DeltaWalk<T> p, bool channel, bool step, int tokens, float* 
   const int max1 = 256 / LPR, max4 = max1 * 4;
   const bool spread = !step && static_cast<long long>(p.H) * p.sg.num < 74;
   const int rpt = (spread || p.e <= max1 / 2) ? 1 : 4;
-  const int max_rows = rpt == 4 ? max4 : max1;
+  int max_rows = rpt == 4 ? max4 : max1;
+  if (spread) {
+    // a head over as many blocks as still give every block an SM of its own
+    const int warp_rows = 32 / LPR, blocks = 148 / (p.H * p.sg.num);
+    const int rows = ((p.e + blocks - 1) / blocks + warp_rows - 1) / warp_rows * warp_rows;
+    max_rows = rows < 2 * warp_rows ? 2 * warp_rows : rows > max1 ? max1 : rows;
+  }
   const int parts = (p.e + max_rows - 1) / max_rows;
   const int rows = (p.e + parts - 1) / parts;
   const int threads = ((rows + rpt - 1) / rpt * LPR + 31) / 32 * 32;
