@@ -604,3 +604,26 @@ def test_trace_run_program(tmp_path):
         la, lb = oracle.forward(a)[0], oracle.forward(b)[0]
         off(np.fromfile(out / "0.f32", "<f4").reshape(2, -1), la[[0, 28]], dtype)
         off(np.fromfile(out / "1.f32", "<f4").reshape(2, -1), torch.stack([lb[20], la[29]]), dtype)
+
+
+def test_imposed_steps_of_a_quantized_decoder(tmp_path):
+    """The same session drives the other native decoders: portions and decode graphs give the logits of one pass."""
+    from cubic_serve_b200.models.checkpoint import write_random_checkpoint
+    from cubic_serve_b200.models.config import ModelConfig, QuantSpec
+    from cubic_serve_b200.runtime.imposed import ImposedSession
+    from cubic_serve_b200.utils.trace_run import build_engine
+    cfg = ModelConfig(name="dense", num_layers=2, hidden_size=256, num_q_heads=4, num_kv_heads=2, head_dim=128, intermediate_size=512,
+                      vocab_size=512, quant=QuantSpec("cubic", 4, 128))
+    s = ImposedSession(build_engine(str(write_random_checkpoint(tmp_path, cfg, seed=1, std=0.05)), "bfloat16", 256))
+    ids = np.random.default_rng(0).integers(0, 512, 90).tolist()
+    whole = s.step([("a", ids, list(range(90)))])[0]
+    s.end(["a"])
+    got, i = [], 0
+    for c in (40, 1, 2, 46, 1):
+        got.append(s.step([("b", ids[i:i + c], list(range(c)))])[0])
+        i += c
+    d = torch.as_tensor(np.concatenate(got) - whole).double()
+    assert (d.pow(2).mean(-1).sqrt() < 3e-2 * torch.as_tensor(whole).double().pow(2).mean(-1).sqrt()).all()
+    with pytest.raises(SystemExit) as e:
+        build_engine(str(tmp_path), "float32", 256)
+    assert e.value.code == 3
