@@ -1,5 +1,5 @@
-"""Plain model of the layered decoders (``Bumodra`` checkpoints): the oracle of the native runner and the model of the
-eager execution mode.
+"""Plain model of the layered decoders (``Bumodra`` and ``Loduzen`` checkpoints): the oracle of the native runner and the
+model of the eager execution mode.
 
 Everything is written from the equations, token by token where the mechanism is a recurrence, one function per
 mechanism, on the raw ``config.json`` dictionary and the checkpoint's tensors by name.  It shares no code with
@@ -12,6 +12,7 @@ and one pass over the whole sequence give the same logits.
 from __future__ import annotations
 
 import copy
+import math
 
 import torch
 
@@ -41,12 +42,13 @@ def softplus(x: torch.Tensor) -> torch.Tensor:
     return torch.clamp(x, min=0) + torch.log1p(torch.exp(-x.abs()))
 
 
-def short_conv(x: torch.Tensor, w: torch.Tensor, past: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
-    """Causal depthwise convolution over time and silu.  ``x`` [n, C] new inputs, ``w`` [C, taps] with the current input's
-    tap last, ``past`` [taps - 1, C] inputs before ``x``.  Returns the outputs and the new ``past``."""
+def short_conv(x: torch.Tensor, w: torch.Tensor, past: torch.Tensor,
+               bias: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+    """Causal depthwise convolution over time (with a bias per channel) and silu.  ``x`` [n, C] new inputs, ``w`` [C, taps]
+    with the current input's tap last, ``past`` [taps - 1, C] inputs before ``x``.  Returns the outputs and the new ``past``."""
     taps = w.shape[1]
     ext = torch.cat([past, x])
-    out = torch.zeros_like(x)
+    out = torch.zeros_like(x) if bias is None else bias.expand_as(x).clone()
     for j in range(taps):
         out = out + w[:, j] * ext[j:j + x.shape[0]]
     return silu(out), ext[ext.shape[0] - (taps - 1):].clone()
@@ -78,6 +80,71 @@ def windowed_attention(q, k, v, first: int, window: int | None, scale: float) ->
 
 def squared_relu(x: torch.Tensor) -> torch.Tensor:
     return torch.clamp(x, min=0) ** 2
+
+
+def gelu_tanh(x: torch.Tensor) -> torch.Tensor:
+    """The tanh form of gelu."""
+    return 0.5 * x * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (x + 0.044715 * x ** 3)))
+
+
+def rotary_frequencies(rot: dict) -> tuple[torch.Tensor, float]:
+    """(radians per position of every rotated pair, factor on cosine and sine), fp64.  With ``scaling`` (YaRN) the slow pairs
+    are stretched by ``factor``, the fast ones stay, a ramp over the pair index lies between."""
+    n, base = rot["dims"], float(rot["base"])
+    f = [base ** (-2.0 * i / n) for i in range(n // 2)]
+    sc = rot.get("scaling")
+    if not sc:
+        return torch.tensor(f, dtype=torch.float64), 1.0
+
+    def pair_of(turns: float) -> float:                    # the (doubled) index that turns this often over ``original`` tokens
+        return n * math.log(sc["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    lo, hi = max(math.floor(pair_of(sc["fast"])), 0), min(math.ceil(pair_of(sc["slow"])), n - 1)
+    out = []
+    for i, fi in enumerate(f):
+        ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        out.append(fi / sc["factor"] * ramp + fi * (1.0 - ramp))
+    return torch.tensor(out, dtype=torch.float64), 0.1 * math.log(sc["factor"]) + 1.0
+
+
+def rotate_pairs(x: torch.Tensor, first: int, freq: torch.Tensor, mult: float) -> torch.Tensor:
+    """Rotary positions ``first ..`` on ``x`` [n, H, d]: neighbouring channels (2 i, 2 i + 1) of the first ``2 len(freq)``."""
+    n, r = x.shape[0], 2 * freq.numel()
+    a = torch.arange(first, first + n, dtype=torch.float64).unsqueeze(1) * freq
+    c, s = (torch.cos(a) * mult).to(x.dtype).unsqueeze(1), (torch.sin(a) * mult).to(x.dtype).unsqueeze(1)
+    out = x.clone()
+    u, v = x[..., 0:r:2], x[..., 1:r:2]
+    out[..., 0:r:2] = u * c - v * s
+    out[..., 1:r:2] = v * c + u * s
+    return out
+
+
+def sink_attention(q, k, v, first: int, window: int | None, scale: float) -> torch.Tensor:
+    """Like ``windowed_attention`` with one more score of zero in the softmax that has no value, and fewer key heads: query
+    head h uses key head ``h // (H / G)``.  ``q`` [n, H, d], ``k`` [m, G, d], ``v`` [m, G, e]."""
+    n, H, m = q.shape[0], q.shape[1], k.shape[0]
+    rep = torch.arange(H) // (H // k.shape[1])
+    i, j = torch.arange(first, first + n).unsqueeze(1), torch.arange(m).unsqueeze(0)
+    seen = (i - j) >= 0
+    if window is not None:
+        seen &= (i - j) < window
+    s = torch.einsum("nhd,mhd->hnm", q, k[:, rep]) * scale
+    s = s.masked_fill(~seen, float("-inf"))
+    s = torch.cat([s, torch.zeros(H, n, 1, dtype=s.dtype)], -1)
+    return torch.einsum("hnm,mhe->nhe", torch.softmax(s, -1)[..., :m], v[:, rep])
+
+
+def linear_step(S: torch.Tensor, q, k, v, decay) -> tuple[torch.Tensor, torch.Tensor]:
+    """One token of a linear recurrence for all heads: the state decays, takes ``k v^T`` and is read by ``q``.  ``S``
+    [H, dim, vdim]; ``q``, ``k``, ``decay`` [H, dim]; ``v`` [H, vdim]."""
+    S = decay.unsqueeze(-1) * S + k.unsqueeze(-1) * v.unsqueeze(1)
+    return torch.einsum("hkv,hk->hv", S, q), S
+
+
+def gated_parts_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, parts: int, eps: float) -> torch.Tensor:
+    """``y silu(z)``, every one of ``parts`` equal parts over its own root mean square, times ``w``."""
+    y = y * silu(z)
+    return rms(y.view(*y.shape[:-1], parts, -1), eps).reshape(y.shape) * w
 
 
 # ------------------------------------------------------------------ layers
@@ -130,6 +197,78 @@ def latent_mixer(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
     return o.reshape(n, H * e) @ w[f"{p}.o"].T
 
 
+def attention_branch(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    """Grouped-query attention whose values are the keys as projected (before norm and rotation), with a sink."""
+    H, G, d = m["heads"], m["kv_heads"], m["dim"]
+    n = h.shape[0]
+    q, k = (h @ w[f"{p}.q"].T).view(n, H, d), (h @ w[f"{p}.k"].T).view(n, G, d)
+    first = st["k"].shape[0] if st else 0
+    freq, mult = rotary_frequencies(m["rot"])
+    turned = rotate_pairs(rms(k, eps) * w[f"{p}.k.norm"], first, freq, mult)
+    q = rotate_pairs(rms(q, eps) * w[f"{p}.q.norm"], first, freq, mult)
+    st["k"] = torch.cat([st["k"], turned]) if st else turned
+    st["v"] = torch.cat([st["v"], k]) if "v" in st else k
+    mask = m.get("mask")
+    o = sink_attention(q, st["k"], st["v"], first, mask["size"] if mask else None, m["scale"])
+    return o.reshape(n, H * d) @ w[f"{p}.o"].T
+
+
+def gated_linear_branch(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    H, d, e = m["heads"], m["dim"], m["vdim"]
+    n = h.shape[0]
+    if not st:
+        st["S"] = torch.zeros(H, d, e, dtype=h.dtype)
+    q, k = (h @ w[f"{p}.q"].T).view(n, H, d) * d ** -0.5, (h @ w[f"{p}.k"].T).view(n, H, d)
+    v = (h @ w[f"{p}.v"].T).view(n, H, e)
+    z = (h @ w[f"{p}.a1"].T) @ w[f"{p}.a2"].T + w[f"{p}.a2.b"]
+    alpha = ((1.0 / (1.0 + torch.exp(-z))) ** (1.0 / m["tau"])).view(n, H, d)
+    o = torch.empty(n, H, e, dtype=h.dtype)
+    for t in range(n):
+        o[t], st["S"] = linear_step(st["S"], q[t], k[t], v[t], alpha[t])
+    o = (rms(o, eps) * w[f"{p}.norm"]).reshape(n, H * e) * silu(h @ w[f"{p}.g"].T)
+    return o @ w[f"{p}.o"].T
+
+
+def parallel_mixer(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    left = attention_branch(w, f"{p}.left", m["left"], h, st.setdefault("left", {}), eps)
+    right = gated_linear_branch(w, f"{p}.right", m["right"], h, st.setdefault("right", {}), eps)
+    return m["left_scale"] * left + m["right_scale"] * right
+
+
+def ssd_mixer(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    """State-space duality layer (Mamba-2): [z | x | B | C | dt] from one projection, x, B and C through the convolution."""
+    H, P, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+    n, inner = h.shape[0], H * P
+    z, xbc, dt = (h @ w[f"{p}.in"].T).split([inner, inner + 2 * G * N, H], -1)
+    if not st:
+        st["past"] = torch.zeros(m["conv"] - 1, xbc.shape[1], dtype=h.dtype)
+        st["S"] = torch.zeros(H, N, P, dtype=h.dtype)
+    xbc, st["past"] = short_conv(xbc, w[f"{p}.conv"], st["past"], w[f"{p}.conv.b"])
+    x, B, C = xbc.split([inner, G * N, G * N], -1)
+    rep = torch.arange(H) // (H // G)
+    x, B, C = x.view(n, H, P), B.view(n, G, N)[:, rep], C.view(n, G, N)[:, rep]
+    dt = softplus(dt + w[f"{p}.dt_bias"])
+    decay = torch.exp(-torch.exp(w[f"{p}.A_log"]) * dt).unsqueeze(-1).expand(n, H, N)
+    y = torch.empty(n, H, P, dtype=h.dtype)
+    for t in range(n):
+        y[t], st["S"] = linear_step(st["S"], C[t], B[t], dt[t].unsqueeze(-1) * x[t], decay[t])
+    y = (y + w[f"{p}.D"].unsqueeze(-1) * x).reshape(n, inner)
+    return gated_parts_norm(y, z, w[f"{p}.norm"], m["norm_groups"], eps) @ w[f"{p}.o"].T
+
+
+def gated_feed_forward(w, p: str, h) -> torch.Tensor:
+    return (gelu_tanh(h @ w[f"{p}.gate"].T) * (h @ w[f"{p}.up"].T)) @ w[f"{p}.down"].T
+
+
+def token_side(w, p: str, x, e, eps: float) -> torch.Tensor:
+    """What a layer takes from its part ``e`` of the token's side embedding, gated by the residual."""
+    y = (gelu_tanh(x @ w[f"{p}.gate"].T) * e) @ w[f"{p}.proj"].T
+    return rms(y, eps) * w[f"{p}.norm"]
+
+
+SEQUENTIAL_MIXERS = {"parallel": parallel_mixer, "mamba2": ssd_mixer}
+
+
 def layer_schedule(cfg: dict) -> list[tuple[int, bool]]:
     """The layer runs in order: (layer index, whether the pass's entry projection comes right before it)."""
     loop = cfg.get("loop")
@@ -157,6 +296,8 @@ class Oracle:
         eps = float(cfg["norm"]["eps"])
         state = state if state is not None else self.new_state()
         ids = torch.as_tensor(list(tokens), dtype=torch.long)
+        if cfg["architecture"] == "Loduzen":
+            return self._sequential(ids, state, eps, last_only, trace)
         x0 = rms_around_zero(w["embed"][ids], w["embed.norm"], eps)
         x = x0
         for (i, enters), st in zip(self.schedule, state.runs):
@@ -180,6 +321,28 @@ class Oracle:
         if last_only:
             x = x[-1:]
         return rms_around_zero(x, w["final.norm"], eps) @ w["head"].T, state
+
+
+    def _sequential(self, ids, state, eps: float, last_only: bool, trace):
+        """Pre-norm layers, mixer then feed-forward then the token's side input; plain norm weights, tied output head."""
+        w, cfg = self.w, self.cfg
+        side = cfg.get("token_side")
+        x = w["embed"][ids]
+        for i, (layer, st) in enumerate(zip(cfg["layers"], state.runs)):
+            p = f"l{i}"
+            h = rms(x, eps) * w[f"{p}.norm1"]
+            x = x + SEQUENTIAL_MIXERS[layer["type"]](w, f"{p}.mix", layer["mixer"], h, st, eps)
+            if layer.get("mlp"):
+                x = x + gated_feed_forward(w, f"{p}.mlp", rms(x, eps) * w[f"{p}.norm2"])
+            if side:
+                e = w["side.embed"][ids, i * side["dim"]:(i + 1) * side["dim"]]
+                x = x + token_side(w, f"{p}.side", x, e, eps)
+            if trace is not None:
+                trace.append(x.clone())
+        state.length += len(ids)
+        if last_only:
+            x = x[-1:]
+        return (rms(x, eps) * w["final.norm"]) @ w["embed"].T, state
 
 
 class OracleState:
