@@ -75,7 +75,7 @@ def bench_delta(requests: int, tokens: int, heads: int, key_heads: int, channel:
     a = torch.randn(T, H * d if channel else H, **bf)
     dt = torch.zeros(H * d if channel else H, device=DEV)
     a_log, norm_w = torch.full((H,), -2.0, device=DEV), torch.ones(d, device=DEV)
-    sc = K.DeltaScratch(T, [(H, G, d, d, channel)], torch.bfloat16, DEV)
+    sc = K.RecurrenceScratch(T, [(H, G, d, d, channel)], torch.bfloat16, DEV)
     decode = tokens == 1
     prep = timeit_graph(lambda: K.delta_prepare(proj, b, a, conv_w, conv_state, a_log, dt, seg, sc, H, G, d, d), flush, launches=5)
     walk = timeit_graph(lambda: K.delta_walk(z, norm_w, state, seg, out, sc, G, d, 1e-6, channel, channel, decode), flush,

@@ -79,7 +79,8 @@ class StateSpec:
 
 @dataclass(frozen=True)
 class LatentCacheSpec:
-    """Paged latent cache of a layered decoder: one row per token and attention run, in the activation type."""
+    """Paged cache of a layered decoder (latents, or keys and values): rows per token and attention run, in the activation
+    type."""
     page_bytes: int           # one page across all attention runs
     runs: int
     page_tokens: int = PAGE_TOKENS
@@ -90,7 +91,7 @@ class LatentCacheSpec:
 
 @dataclass(frozen=True)
 class DeltaStateSpec:
-    """Recurrent state of a layered decoder's delta runs (fp32 delta-rule state and convolution inputs)."""
+    """Recurrent state of a layered decoder's recurrent runs (fp32 state and convolution inputs)."""
     runs: int
     bytes_per_request: int
 
@@ -148,10 +149,9 @@ class ModelSpec:
     @staticmethod
     def from_layered(cfg, manifest: WeightManifest | None = None) -> "ModelSpec":
         """Of a layered decoder (``models/layered.py``): every layer RUN has its own cache or state."""
-        from ..models.layered import LatentSpec
-        attn = sum(isinstance(cfg.layers[i].mixer, LatentSpec) for i, _ in cfg.runs)
-        delta = len(cfg.runs) - attn
-        state = DeltaStateSpec(delta, cfg.state_bytes_per_request) if delta else None
+        from ..models.layered import ATTENTION_SPECS, RECURRENT_SPECS
+        attn, recurrent = cfg.run_parts(ATTENTION_SPECS), cfg.run_parts(RECURRENT_SPECS)
+        state = DeltaStateSpec(recurrent, cfg.state_bytes_per_request) if recurrent else None
         return ModelSpec(cfg.name, cfg.family, digest_of(dataclasses.asdict(cfg)), LatentCacheSpec(cfg.page_bytes, attn), state,
                          manifest)
 

@@ -362,7 +362,7 @@ def decoder_step_operators(cfg, rows: int, tp_size: int = 1, topology_id: str = 
 
 def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple[OpSignature, ...]:
     """Operator signatures of one decode step of a layered decoder: the distinct operators of its layer runs."""
-    from ..models.layered import LatentSpec
+    from ..models.layered import AttentionSpec, DeltaSpec, LatentSpec, SsdSpec
     W, act = cfg.hidden_size, "fp32" if cfg.dtype == "float32" else "bf16"
     ops: dict[tuple, OpSignature] = {}
 
@@ -377,12 +377,28 @@ def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple
     if cfg.loop is not None:
         add("linear.bf16", "loop_entry", W, 2 * W)
     for i, _ in cfg.runs:
-        l, m = cfg.layers[i], cfg.layers[i].mixer
-        if isinstance(m, LatentSpec):
-            add("attention.latent", "paged", m.out_width, m.q_rank + m.kv_rank, heads=m.heads, window=m.window or cfg.max_position)
+        l = cfg.layers[i]
+        for m in l.mixer.parts:
+            if isinstance(m, LatentSpec):
+                add("attention.latent", "paged", m.out_width, m.q_rank + m.kv_rank, heads=m.heads, window=m.window or cfg.max_position)
+            elif isinstance(m, AttentionSpec):
+                add("attention.gqa", "paged", m.out_width, (m.heads + m.kv_heads) * m.dim, heads=m.heads,
+                    window=m.window or cfg.max_position)
+            elif isinstance(m, DeltaSpec):
+                add("delta_rule." + ("channel" if m.per_channel else "head"), "state32", m.out_width, m.channels, heads=m.heads,
+                    taps=m.conv)
+            elif isinstance(m, SsdSpec):
+                add("linear_recurrence.head", "state32", m.out_width, m.channels, heads=m.heads, taps=m.conv)
+            else:
+                add("linear_recurrence.channel", "state32", m.out_width, 2 * m.heads * m.dim, heads=m.heads)
+        if cfg.design.sequential:
+            add("linear.bf16", "out", W, l.mixer.out_width)
+            if l.ff:
+                add("linear.bf16", "gate_up", 2 * l.ff, W)
+                add("linear.bf16", "down", W, l.ff)
         else:
-            add("delta_rule." + ("channel" if m.per_channel else "head"), "state32", m.out_width, m.channels, heads=m.heads,
-                taps=m.conv)
-        add("linear.bf16", "parallel_out", W, m.out_width + l.ff)
+            add("linear.bf16", "parallel_out", W, l.mixer.out_width + l.ff)
+        if cfg.side_dim:
+            add("token_side", "residual32", W, cfg.side_dim)
     add("linear.bf16", "lm_head", cfg.vocab_size, W)
     return tuple(ops.values())

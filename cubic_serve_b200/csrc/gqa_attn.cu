@@ -1,0 +1,722 @@
+// Grouped-query attention of the layered decoders over a paged cache in the activation type: head norms, rotary pairs, a sliding
+// window and a softmax entry without a value (sink).  A value is the raw key of its token, as projected.
+//
+//   gqa_prepare_kernel    RMS norm of every query and key head, rotary positions on neighbouring channel pairs; keys and values
+//                         to their page
+//   gqa_prefill_kernel    bf16: blocks of (token, head) rows of one key head on the tensor cores
+//   gqa_decode_kernel,    bf16, one token per segment: the query heads of a key head are the rows, a warp walks whole pages;
+//   gqa_merge_kernel      key splits are merged in split order
+//   gqa_row_kernel        fp32 models: a warp per (token, head)
+//
+// The cache is [pages][key head][key, value][16][P], P the head width rounded up to 64, zero columns behind the head.  Scores,
+// softmax weights and sums are fp32; the weights are rounded to bf16 as the operand of the second product of the bf16 kernels.
+#include <type_traits>
+
+#include "segments.cuh"
+#include "launch.cuh"
+#include "mma.cuh"
+
+namespace cb {
+
+static constexpr int kGqaPage = 16;
+static constexpr float kLog2e = 1.4426950408889634f;
+
+template <typename T>
+struct GqaPrep {
+  const T* x; int ldx;        // projections
+  int q_off, k_off;           // columns of q [H d] and k [G d]
+  const float* qw;            // [d]
+  const float* kw;
+  const float* freq;          // [pairs] radians per position
+  float mult;                 // factor on cosine and sine
+  const int* positions;       // [T]
+  const int* slots;           // [T] cache row, < 0: none
+  T* q;                       // [T, H, P]
+  T* cache;
+  int H, G, d, P, pairs;
+  float eps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+gqa_prepare_kernel(const GqaPrep<T> p) {
+  __shared__ float2 turn[128];
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (static_cast<int>(threadIdx.x) < p.pairs) {
+    // the rounding error of the product is put back to first order: angles of far positions keep their fraction of a turn
+    const float pos = static_cast<float>(p.positions[t]), f = p.freq[threadIdx.x];
+    const float a = pos * f, e = fmaf(pos, f, -a);
+    float s, c;
+    sincosf(a, &s, &c);
+    turn[threadIdx.x] = make_float2(fmaf(-e, s, c) * p.mult, fmaf(e, c, s) * p.mult);
+  }
+  __syncthreads();
+  const int slot = p.slots[t];
+  const bool even = ((p.d | p.q_off | p.k_off | p.ldx) & 1) == 0;
+  for (int hh = blockIdx.y * 4 + warp; hh < p.H + p.G; hh += 4 * gridDim.y) {
+    const bool key = hh >= p.H;
+    if (key && slot < 0) continue;
+    const T* src = p.x + t * p.ldx + (key ? p.k_off + (hh - p.H) * p.d : p.q_off + hh * p.d);
+    const float* w = key ? p.kw : p.qw;
+    float2 v[4];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = 2 * (lane + 32 * i);
+      v[i] = make_float2(0.f, 0.f);
+      if (even) {
+        if (c < p.d) {
+          if constexpr (sizeof(T) == 2) v[i] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src + c));
+          else v[i] = *reinterpret_cast<const float2*>(src + c);
+        }
+      } else {
+        if (c < p.d) v[i].x = to_f(src[c]);
+        if (c + 1 < p.d) v[i].y = to_f(src[c + 1]);
+      }
+      ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, ss));
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.d) + p.eps);
+    T* dst;
+    if (key) {
+      const size_t page = static_cast<size_t>(slot / kGqaPage), row = slot % kGqaPage;
+      dst = p.cache + ((page * p.G + (hh - p.H)) * 2 * kGqaPage + row) * p.P;
+    } else {
+      dst = p.q + (t * p.H + hh) * p.P;
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int j = lane + 32 * i, c = 2 * j;
+      if (c >= p.P) continue;
+      float2 n = make_float2(c < p.d ? v[i].x * inv * w[c] : 0.f, c + 1 < p.d ? v[i].y * inv * w[c + 1] : 0.f);
+      if (j < p.pairs) {
+        const float2 r = turn[j];
+        n = make_float2(n.x * r.x - n.y * r.y, fmaf(n.y, r.x, n.x * r.y));
+      }
+      T* val = dst + kGqaPage * p.P;
+      if constexpr (sizeof(T) == 2) {
+        *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(n.x, n.y);
+        if (key) *reinterpret_cast<uint32_t*>(val + c) = pack_bf16x2(v[i].x, v[i].y);
+      } else {
+        *reinterpret_cast<float2*>(dst + c) = n;
+        if (key) *reinterpret_cast<float2*>(val + c) = v[i];
+      }
+    }
+  }
+}
+
+template <typename T>
+struct GqaAttn {
+  const T* q;                 // [T, H, P]
+  T* out; int ldo;            // [T, H d]
+  const T* cache;
+  const int* page_table;      // [slots, max_pages]
+  int max_pages;
+  int H, G, d, P, window;     // window <= 0: every earlier token
+  float scale, out_scale;
+  float sink;                 // score of the entry without a value, -inf: none
+  Segments sg;
+};
+
+// ------------------------------------------------------------------ fp32
+template <int NR>
+__global__ void __launch_bounds__(128)
+gqa_row_kernel(const GqaAttn<float> p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  int s, off;
+  if (!find_tile(p.sg, 1, blockIdx.x, s, off)) return;
+  const int lane = threadIdx.x & 31;
+  const int h = blockIdx.y * 4 + (threadIdx.x >> 5);
+  if (h >= p.H) return;
+  const int kh = h / (p.H / p.G);
+  const size_t row = static_cast<size_t>(p.sg.row0[s]) + off;
+  const int pos = p.sg.pos0[s] + off;
+  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int* pages = p.page_table + static_cast<size_t>(p.sg.slot[s]) * p.max_pages;
+  const float* qr = p.q + (row * p.H + h) * p.P;
+  float q[NR], acc[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    q[i] = qr[lane + 32 * i] * p.scale;
+    acc[i] = 0.f;
+  }
+  float m = p.sink, l = p.sink == -INFINITY ? 0.f : 1.f;
+  for (int j = lo; j <= pos; ++j) {
+    const float* kr = p.cache + ((static_cast<size_t>(pages[j / kGqaPage]) * p.G + kh) * 2 * kGqaPage + j % kGqaPage) * p.P;
+    const float* vr = kr + kGqaPage * p.P;
+    float v[NR], sdot = 0.f;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      v[i] = vr[lane + 32 * i];
+      sdot = fmaf(q[i], kr[lane + 32 * i], sdot);
+    }
+    sdot = warp_sum(sdot);
+    const float mn = fmaxf(m, sdot);
+    const float f = expf(m - mn), w = expf(sdot - mn);
+    m = mn;
+    l = l * f + w;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) acc[i] = fmaf(w, v[i], acc[i] * f);
+  }
+  const float g = p.out_scale / l;
+  float* orow = p.out + row * p.ldo + h * p.d;
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int c = lane + 32 * i;
+    if (c < p.d) orow[c] = acc[i] * g;
+  }
+}
+
+// ------------------------------------------------------------------ bf16, prompts and mixed steps
+using bf16 = __nv_bfloat16;
+
+struct GqaMma {
+  GqaAttn<bf16> a;
+  int hb, qb;                 // heads and tokens of a block (hb * qb rows at most)
+  int head_tiles;             // blocks of hb heads that share a key head
+  int splits;
+  float* partial;             // decode: [segment][key head tile][split][16][P + 2]
+};
+
+__device__ __forceinline__ void store_pair(bf16* row, int c, int d, float x, float y) {
+  if (c + 1 < d && (d & 1) == 0) {
+    *reinterpret_cast<uint32_t*>(row + c) = pack_bf16x2(x, y);
+  } else {
+    if (c < d) row[c] = __float2bfloat16(x);
+    if (c + 1 < d) row[c + 1] = __float2bfloat16(y);
+  }
+}
+
+// NW warps of 16 rows each, row = token * hb + head; key tiles of 64 keys in two buffers, 16-byte chunks XOR-swizzled by the row.
+// A warp keeps its rows' scores, weights and outputs in registers: no exchange between warps.
+template <int NW, int NCH>
+__global__ void __launch_bounds__(32 * NW)
+gqa_prefill_kernel(const GqaMma p) {
+  constexpr int P = NCH * 64, ROWB = P * 2, MR = 16 * NW, KT = 64, CH = P / 8, NT = P / 8;
+  extern __shared__ __align__(128) uint8_t lsm[];
+  uint8_t* qs = lsm;                                  // [MR][ROWB]
+  uint8_t* kvs = qs + MR * ROWB;                      // [2 buffers][key, value][KT][ROWB]
+  pdl_wait();
+  pdl_launch_dependents();
+  const GqaAttn<bf16>& a = p.a;
+  int s, off;
+  if (!find_tile(a.sg, p.qb, blockIdx.x, s, off)) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int R = a.H / a.G, kh = blockIdx.y / p.head_tiles, hq0 = (blockIdx.y % p.head_tiles) * p.hb;
+  const int heads = min(p.hb, R - hq0), h0 = kh * R + hq0;
+  const int toks = min(p.qb, a.sg.count[s] - off);
+  const size_t row0 = static_cast<size_t>(a.sg.row0[s]) + off;
+  const int pos0 = a.sg.pos0[s] + off;
+  const int* pages = a.page_table + static_cast<size_t>(a.sg.slot[s]) * a.max_pages;
+  const int kmin = a.window > 0 ? max(0, pos0 - a.window + 1) & ~(kGqaPage - 1) : 0;
+  const int kend = pos0 + toks;
+  const int tiles = (kend - kmin + KT - 1) / KT;
+
+  auto load_tile = [&](int t, int b) {
+    const uint32_t dst0 = smem_u32(kvs + b * 2 * KT * ROWB);
+#pragma unroll
+    for (int i = 0; i < KT * CH / (32 * NW); ++i) {
+      const int idx = tid + i * 32 * NW;
+      const int r = idx / CH, c = idx % CH;
+      const int key = kmin + t * KT + r;
+      const bool ok = key < kend;
+      const int page = ok ? pages[key / kGqaPage] : 0;
+      const bf16* src = a.cache + ((static_cast<size_t>(page) * a.G + kh) * 2 * kGqaPage + key % kGqaPage) * P + c * 8;
+      const uint32_t at = dst0 + r * ROWB + ((c ^ (r & 7)) << 4);
+      cp_async16(at, src, ok);
+      cp_async16(at + KT * ROWB, src + kGqaPage * P, ok);
+    }
+  };
+  for (int idx = tid; idx < MR * CH; idx += 32 * NW) {
+    const int r = idx / CH, c = idx % CH;
+    const int tok = r / p.hb, h = r - tok * p.hb;
+    const bool ok = tok < toks && h < heads;
+    cp_async16(smem_u32(qs) + r * ROWB + ((c ^ (r & 7)) << 4),
+               a.q + ((row0 + (ok ? tok : 0)) * a.H + h0 + (ok ? h : 0)) * P + c * 8, ok);
+  }
+  load_tile(0, 0);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+
+  // visible keys of the thread's two rows; rows without a query see none
+  int lim_lo[2], lim_hi[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = warp * 16 + g + 8 * i;
+    const int tok = r / p.hb, h = r - tok * p.hb;
+    lim_hi[i] = tok < toks && h < heads ? pos0 + tok : -1;
+    lim_lo[i] = a.window > 0 ? pos0 + tok - a.window + 1 : 0;
+  }
+  // of the whole warp
+  const int tok_a = min(warp * 16 / p.hb, toks - 1), tok_b = min((warp * 16 + 15) / p.hb, toks - 1);
+  const bool idle = warp * 16 / p.hb >= toks;
+  const int see_lo = a.window > 0 ? pos0 + tok_a - a.window + 1 : 0, see_hi = pos0 + tok_b;     // some row sees these
+  const int all_lo = a.window > 0 ? pos0 + tok_b - a.window + 1 : 0, all_hi = pos0 + tok_a;     // every row sees these
+  const float sc = a.scale * kLog2e;
+  float m2[2] = {-INFINITY, -INFINITY}, l2[2] = {0.f, 0.f};
+  float o[NT][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) o[j][c] = 0.f;
+
+  const uint32_t q_base = smem_u32(qs) + (warp * 16 + (lane & 15)) * ROWB;
+  uint32_t q_at[4], k_at[4], v_at[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {                       // the swizzled chunk depends on the place inside a 128-byte group only
+    q_at[i] = q_base + (((i * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
+    k_at[i] = ((lane & 7) + ((lane >> 4) << 3)) * ROWB + (((i * 2 + ((lane >> 3) & 1)) ^ (lane & 7)) << 4);
+    v_at[i] = (lane & 15) * ROWB + (((i * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
+  }
+  for (int t = 0; t < tiles; ++t) {
+    const int b = t & 1;
+    if (t + 1 < tiles) load_tile(t + 1, b ^ 1);       // its buffer was released by the barrier that ended the last turn
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();
+    const int key_t = kmin + t * KT;
+    if (!idle && key_t <= see_hi && key_t + KT > see_lo) {
+      const uint32_t k_base = smem_u32(kvs + b * 2 * KT * ROWB), v_base = k_base + KT * ROWB;
+      float sf[8][4];
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) sf[j][c] = 0.f;
+#pragma unroll
+      for (int kk = 0; kk < P / 16; ++kk) {
+        uint32_t qa[4];
+        ldsm4(qa, q_at[kk & 3] + (kk >> 2) * 128);
+#pragma unroll
+        for (int j = 0; j < 8; j += 2) {
+          uint32_t cb[4];
+          ldsm4(cb, k_base + k_at[kk & 3] + (kk >> 2) * 128 + j * 8 * ROWB);
+          mma_bf16(sf[j], qa, cb[0], cb[1]);
+          mma_bf16(sf[j + 1], qa, cb[2], cb[3]);
+        }
+      }
+      const bool whole = key_t >= all_lo && key_t + KT - 1 <= all_hi;
+      float mx[2] = {m2[0], m2[1]};
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const int key = key_t + j * 8 + 2 * t4 + (c & 1), i = c >> 1;
+          sf[j][c] = whole || (key >= lim_lo[i] && key <= lim_hi[i]) ? sf[j][c] * sc : -INFINITY;
+          mx[i] = fmaxf(mx[i], sf[j][c]);
+        }
+      float al[2], use[2];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+        mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+        use[i] = mx[i] == -INFINITY ? 0.f : mx[i];
+        al[i] = exp2f(m2[i] - use[i]);
+        m2[i] = mx[i];
+        l2[i] *= al[i];
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          sf[j][c] = exp2f(sf[j][c] - use[c >> 1]);
+          l2[c >> 1] += sf[j][c];
+        }
+#pragma unroll
+      for (int j = 0; j < NT; ++j) { o[j][0] *= al[0]; o[j][1] *= al[0]; o[j][2] *= al[1]; o[j][3] *= al[1]; }
+#pragma unroll
+      for (int ks = 0; ks < KT / 16; ++ks) {
+        const uint32_t pa[4] = {pack_bf16x2(sf[2 * ks][0], sf[2 * ks][1]), pack_bf16x2(sf[2 * ks][2], sf[2 * ks][3]),
+                                pack_bf16x2(sf[2 * ks + 1][0], sf[2 * ks + 1][1]), pack_bf16x2(sf[2 * ks + 1][2], sf[2 * ks + 1][3])};
+#pragma unroll
+        for (int j = 0; j < NT / 2; ++j) {
+          uint32_t vb[4];
+          ldsm4_t(vb, v_base + v_at[j & 3] + (j >> 2) * 128 + ks * 16 * ROWB);
+          mma_bf16(o[2 * j], pa, vb[0], vb[1]);
+          mma_bf16(o[2 * j + 1], pa, vb[2], vb[3]);
+        }
+      }
+    }
+    __syncthreads();                                  // the tile's buffer is free again
+  }
+  asm volatile("cp.async.wait_all;" ::: "memory");
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    l2[i] += __shfl_xor_sync(0xffffffffu, l2[i], 1);
+    l2[i] += __shfl_xor_sync(0xffffffffu, l2[i], 2);
+    const int r = warp * 16 + g + 8 * i;
+    const int tok = r / p.hb, h = r - tok * p.hb;
+    if (tok >= toks || h >= heads) continue;
+    const float f = a.out_scale / (l2[i] + exp2f(a.sink * kLog2e - m2[i]));
+    bf16* row = a.out + (row0 + tok) * a.ldo + (h0 + h) * a.d;
+#pragma unroll
+    for (int j = 0; j < NT; ++j) store_pair(row, j * 8 + 2 * t4, a.d, o[j][2 * i] * f, o[j][2 * i + 1] * f);
+  }
+}
+
+// ------------------------------------------------------------------ bf16, one token per segment
+// Four warps deal the pages of a (segment, key head, split) among themselves; each has its own ring of kRing pages.  The rows of
+// a product are the query heads of the key head (up to 16 of them).
+static constexpr int kRing = 3;
+
+template <int NCH>
+__global__ void __launch_bounds__(128)
+gqa_decode_kernel(const GqaMma p) {
+  constexpr int P = NCH * 64, ROWB = P * 2, CH = P / 8, NT = P / 8, PAGEB = 2 * kGqaPage * ROWB;
+  extern __shared__ __align__(128) uint8_t lsm[];     // [4 warps][kRing][key, value][16][ROWB], then the warps' results
+  pdl_wait();
+  pdl_launch_dependents();
+  const GqaAttn<bf16>& a = p.a;
+  const int s = blockIdx.x;
+  if (a.sg.count[s] <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int R = a.H / a.G, kh = blockIdx.y / p.head_tiles, hq0 = (blockIdx.y % p.head_tiles) * 16;
+  const int heads = min(16, R - hq0), h0 = kh * R + hq0;
+  const size_t row = a.sg.row0[s];
+  const int pos = a.sg.pos0[s];
+  const int* pages = a.page_table + static_cast<size_t>(a.sg.slot[s]) * a.max_pages;
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int pg_all = pos / kGqaPage + 1, pg_first = lo / kGqaPage, per = (pg_all - pg_first + p.splits - 1) / p.splits;
+  const int pg_lo = min(pg_all, pg_first + static_cast<int>(blockIdx.z) * per), pg_hi = min(pg_all, pg_lo + per);
+  uint8_t* ring = lsm + warp * kRing * PAGEB;
+
+  auto load_page = [&](int pg, int b) {               // nothing behind the last page
+    if (pg < pg_hi) {
+      const bf16* src = a.cache + (static_cast<size_t>(pages[pg]) * a.G + kh) * 2 * kGqaPage * P;
+      const uint32_t dst0 = smem_u32(ring + b * PAGEB);
+#pragma unroll
+      for (int i = 0; i < 2 * kGqaPage * CH / 32; ++i) {
+        const int idx = lane + i * 32;
+        const int r = idx / CH, c = idx % CH;         // rows 0-15 keys, 16-31 values
+        cp_async16(dst0 + r * ROWB + ((c ^ (r & 7)) << 4), src + r * P + c * 8, true);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+#pragma unroll
+  for (int i = 0; i < kRing - 1; ++i) load_page(pg_lo + warp + 4 * i, i);
+  uint32_t qa[P / 16][4];
+#pragma unroll
+  for (int kk = 0; kk < P / 16; ++kk)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int h = g + 8 * (i & 1), c = kk * 16 + 2 * t4 + 8 * (i >> 1);
+      qa[kk][i] = h < heads ? *reinterpret_cast<const uint32_t*>(a.q + (row * a.H + h0 + h) * P + c) : 0u;
+    }
+  const float sc = a.scale * kLog2e;
+  float m2[2] = {-INFINITY, -INFINITY}, l2[2] = {0.f, 0.f};
+  float o[NT][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) o[j][c] = 0.f;
+  uint32_t k_at[4], v_at[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    k_at[i] = ((lane & 7) + ((lane >> 4) << 3)) * ROWB + (((i * 2 + ((lane >> 3) & 1)) ^ (lane & 7)) << 4);
+    v_at[i] = (lane & 15) * ROWB + (((i * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
+  }
+  int b = 0;
+  for (int pg = pg_lo + warp; pg < pg_hi; pg += 4) {
+    load_page(pg + 4 * (kRing - 1), (b + kRing - 1) % kRing);
+    asm volatile("cp.async.wait_group %0;" ::"n"(kRing - 1) : "memory");
+    __syncwarp();
+    const uint32_t k_base = smem_u32(ring + b * PAGEB), v_base = k_base + kGqaPage * ROWB;
+    float sf[2][4] = {};
+    float s2[2][4] = {};                              // two chains
+#pragma unroll
+    for (int kk = 0; kk < P / 16; ++kk) {
+      uint32_t cb[4];
+      ldsm4(cb, k_base + k_at[kk & 3] + (kk >> 2) * 128);
+      mma_bf16(kk & 1 ? s2[0] : sf[0], qa[kk], cb[0], cb[1]);
+      mma_bf16(kk & 1 ? s2[1] : sf[1], qa[kk], cb[2], cb[3]);
+    }
+    float mx[2] = {m2[0], m2[1]};
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int key = pg * kGqaPage + j * 8 + 2 * t4 + (c & 1);
+        sf[j][c] = key >= lo && key <= pos ? (sf[j][c] + s2[j][c]) * sc : -INFINITY;
+        mx[c >> 1] = fmaxf(mx[c >> 1], sf[j][c]);
+      }
+    float use[2], al[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+      use[i] = mx[i] == -INFINITY ? 0.f : mx[i];
+      al[i] = exp2f(m2[i] - use[i]);
+    }
+    if (__any_sync(0xffffffffu, mx[0] > m2[0] || mx[1] > m2[1])) {
+#pragma unroll
+      for (int j = 0; j < NT; ++j) { o[j][0] *= al[0]; o[j][1] *= al[0]; o[j][2] *= al[1]; o[j][3] *= al[1]; }
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      m2[i] = mx[i];
+      l2[i] *= al[i];
+    }
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        sf[j][c] = exp2f(sf[j][c] - use[c >> 1]);
+        l2[c >> 1] += sf[j][c];
+      }
+    const uint32_t pa[4] = {pack_bf16x2(sf[0][0], sf[0][1]), pack_bf16x2(sf[0][2], sf[0][3]), pack_bf16x2(sf[1][0], sf[1][1]),
+                            pack_bf16x2(sf[1][2], sf[1][3])};
+#pragma unroll
+    for (int j = 0; j < NT / 2; ++j) {
+      uint32_t vb[4];
+      ldsm4_t(vb, v_base + v_at[j & 3] + (j >> 2) * 128);
+      mma_bf16(o[2 * j], pa, vb[0], vb[1]);
+      mma_bf16(o[2 * j + 1], pa, vb[2], vb[3]);
+    }
+    __syncwarp();                                     // the page's buffer is free again
+    b = b + 1 == kRing ? 0 : b + 1;
+  }
+  asm volatile("cp.async.wait_all;" ::: "memory");
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    l2[i] += __shfl_xor_sync(0xffffffffu, l2[i], 1);
+    l2[i] += __shfl_xor_sync(0xffffffffu, l2[i], 2);
+  }
+  __syncthreads();                                    // all rings are done: their memory takes the warps' results
+  constexpr int LD = P + 2;
+  float* res = reinterpret_cast<float*>(lsm);         // [4][16][LD]: output columns, maximum, sum
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    float* dst = res + (warp * 16 + g + 8 * i) * LD;
+#pragma unroll
+    for (int j = 0; j < NT; ++j) *reinterpret_cast<float2*>(dst + j * 8 + 2 * t4) = make_float2(o[j][2 * i], o[j][2 * i + 1]);
+    if (t4 == 0) *reinterpret_cast<float2*>(dst + P) = make_float2(m2[i], l2[i]);
+  }
+  __syncthreads();
+  const size_t unit = static_cast<size_t>(s) * gridDim.y + blockIdx.y;
+  for (int r = warp; r < heads; r += 4) {
+    float mx = -INFINITY, f[4], l = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) mx = fmaxf(mx, res[(w * 16 + r) * LD + P]);
+    const float use = mx == -INFINITY ? 0.f : mx;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      f[w] = exp2f(res[(w * 16 + r) * LD + P] - use);
+      l += f[w] * res[(w * 16 + r) * LD + P + 1];
+    }
+    float* part = p.partial + ((unit * p.splits + blockIdx.z) * 16 + r) * LD;
+    const float scale = p.splits > 1 ? 1.f : a.out_scale / (l + exp2f(a.sink * kLog2e - use));
+#pragma unroll
+    for (int i = 0; i < P / 64; ++i) {
+      const int c = 2 * (lane + 32 * i);
+      float2 v = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        const float2 u = *reinterpret_cast<const float2*>(res + (w * 16 + r) * LD + c);
+        v.x = fmaf(f[w], u.x, v.x);
+        v.y = fmaf(f[w], u.y, v.y);
+      }
+      if (p.splits > 1) *reinterpret_cast<float2*>(part + c) = v;
+      else store_pair(a.out + row * a.ldo + (h0 + r) * a.d, c, a.d, v.x * scale, v.y * scale);
+    }
+    if (p.splits > 1 && lane == 0) *reinterpret_cast<float2*>(part + P) = make_float2(mx, l);
+  }
+}
+
+// A warp per row of a unit.
+template <int NCH>
+__global__ void __launch_bounds__(128)
+gqa_merge_kernel(const GqaMma p) {
+  constexpr int P = NCH * 64, LD = P + 2;
+  pdl_wait();
+  pdl_launch_dependents();
+  const GqaAttn<bf16>& a = p.a;
+  const int s = blockIdx.x, lane = threadIdx.x & 31, r = blockIdx.z * 4 + (threadIdx.x >> 5);
+  if (a.sg.count[s] <= 0) return;
+  const int R = a.H / a.G, kh = blockIdx.y / p.head_tiles, hq0 = (blockIdx.y % p.head_tiles) * 16;
+  if (r >= min(16, R - hq0)) return;
+  const size_t unit = static_cast<size_t>(s) * gridDim.y + blockIdx.y;
+  const float* part = p.partial + (unit * p.splits * 16 + r) * LD;
+  constexpr int step = 16 * LD;
+  float mx = a.sink * kLog2e;
+  for (int z = 0; z < p.splits; ++z) mx = fmaxf(mx, part[z * step + P]);
+  float l = exp2f(a.sink * kLog2e - mx);
+  float2 v[NCH];
+#pragma unroll
+  for (int i = 0; i < NCH; ++i) v[i] = make_float2(0.f, 0.f);
+  for (int z = 0; z < p.splits; ++z) {
+    const float f = exp2f(part[z * step + P] - mx);   // 0 for a split that saw no key
+    l += f * part[z * step + P + 1];
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+      const float2 u = *reinterpret_cast<const float2*>(part + z * step + 2 * (lane + 32 * i));
+      v[i].x = fmaf(f, u.x, v[i].x);
+      v[i].y = fmaf(f, u.y, v[i].y);
+    }
+  }
+  const float f = a.out_scale / l;
+  bf16* row = a.out + static_cast<size_t>(a.sg.row0[s]) * a.ldo + (kh * R + hq0 + r) * a.d;
+#pragma unroll
+  for (int i = 0; i < NCH; ++i) store_pair(row, 2 * (lane + 32 * i), a.d, v[i].x * f, v[i].y * f);
+}
+
+// ------------------------------------------------------------------ host
+template <typename K>
+static int gqa_go(K kernel, dim3 grid, int threads, size_t smem, const GqaMma& p, bool (&configured)[64], cudaStream_t st) {
+  int dev = 0;                                        // dynamic shared memory is configured once per device
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -18;
+  if (!configured[dev]) {
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured[dev] = true;
+  }
+  return static_cast<int>(launch(kernel, grid, dim3(threads), smem, st, p));
+}
+
+template <int NW, int NCH>
+static int gqa_prefill(const GqaMma& p, dim3 grid, cudaStream_t st) {
+  static bool configured[64] = {};
+  return gqa_go(gqa_prefill_kernel<NW, NCH>, grid, 32 * NW, static_cast<size_t>(16 * NW + 256) * NCH * 128, p, configured, st);
+}
+
+template <int NCH>
+static int gqa_decode(const GqaMma& p, dim3 grid, cudaStream_t st) {
+  static bool configured[64] = {};
+  const int rc = gqa_go(gqa_decode_kernel<NCH>, grid, 128, static_cast<size_t>(4) * kRing * 2 * kGqaPage * NCH * 128, p, configured, st);
+  if (rc || p.splits == 1) return rc;
+  return static_cast<int>(launch(gqa_merge_kernel<NCH>, dim3(grid.x, grid.y, 4), dim3(128), 0, st, p));
+}
+
+// Rows of a block of the prompt form: 128 when the step then still has enough blocks, else 64.
+static void gqa_shape(int tokens, int segs, int H, int G, int& nw, int& hb, int& qb, int& head_tiles) {
+  const int R = H / G;
+  for (nw = 8; nw >= 4; nw -= 4) {
+    hb = R < 16 * nw ? R : 16 * nw;
+    qb = 16 * nw / hb;
+    head_tiles = (R + hb - 1) / hb;
+    if (static_cast<long long>(max_tiles(tokens, segs, qb)) * G * head_tiles >= 296) return;
+  }
+  nw = 4;
+}
+
+}  // namespace cb
+
+extern "C" {
+
+struct CbGqaPrep {
+  const void* x; int ldx, q_off, k_off;
+  const void* qw;
+  const void* kw;
+  const void* freq;
+  float mult;
+  const void* positions;
+  const void* slots;
+  void* q;
+  void* cache;
+  int H, G, d, P, pairs;
+  float eps;
+  int tokens, f32;
+};
+
+struct CbGqaAttn {
+  const void* q;
+  void* out; int ldo;
+  const void* cache;
+  const void* page_table;
+  int max_pages, H, G, d, P, window;
+  float scale, out_scale, sink;
+  int tokens, f32;
+  int decode;                 // every segment has at most one row, row s belongs to segment s
+  int splits;                 // key splits of the decode form (1 = none)
+  void* partial;              // fp32 scratch of cb_gqa_attn_partial_floats elements (splits > 1)
+};
+
+// Scratch of a split decode launch; `units` receives the blocks of one split.
+long long cb_gqa_attn_partial_floats(int tokens, int segs, int H, int G, int P, int decode, int splits, int* units) {
+  if (!decode) return 0;
+  const long long n = static_cast<long long>(segs) * G * ((H / G + 15) / 16);
+  if (units) *units = static_cast<int>(n);
+  return splits > 1 ? n * splits * 16 * (P + 2) : 0;
+}
+
+int cb_gqa_prepare(const CbGqaPrep* a, void* stream) {
+  using namespace cb;
+  if (!a || a->tokens <= 0) return 0;
+  if (a->H <= 0 || a->G <= 0 || a->d <= 0 || a->P < a->d || a->P > 256 || (a->P & 63) || a->pairs < 0 || 2 * a->pairs > a->d) return -10;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  // few tokens: more blocks per token
+  const int ny = a->tokens >= 1024 ? 1 : min((a->H + a->G + 3) / 4, 8);
+  auto go = [&](auto kernel, auto p) {
+    using T = std::remove_pointer_t<decltype(p.q)>;
+    p.x = static_cast<const T*>(a->x); p.ldx = a->ldx; p.q_off = a->q_off; p.k_off = a->k_off;
+    p.qw = static_cast<const float*>(a->qw); p.kw = static_cast<const float*>(a->kw);
+    p.freq = static_cast<const float*>(a->freq); p.mult = a->mult;
+    p.positions = static_cast<const int*>(a->positions); p.slots = static_cast<const int*>(a->slots);
+    p.q = static_cast<T*>(a->q); p.cache = static_cast<T*>(a->cache);
+    p.H = a->H; p.G = a->G; p.d = a->d; p.P = a->P; p.pairs = a->pairs; p.eps = a->eps;
+    return static_cast<int>(launch(kernel, dim3(a->tokens, ny), dim3(128), 0, st, p));
+  };
+  return a->f32 ? go(gqa_prepare_kernel<float>, GqaPrep<float>{}) : go(gqa_prepare_kernel<bf16>, GqaPrep<bf16>{});
+}
+
+int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
+  using namespace cb;
+  if (!a || !seg || seg->num <= 0 || a->tokens <= 0) return 0;
+  if (a->H <= 0 || a->G <= 0 || (a->H % a->G) || a->d <= 0 || a->P < a->d || a->P > 256 || (a->P & 63) || a->ldo < a->H * a->d) return -10;
+  if (a->splits > 1 && (!a->decode || !a->partial || a->splits > 65535)) return -12;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  auto fill = [&](auto& p) {
+    using T = std::remove_pointer_t<decltype(p.out)>;
+    p.q = static_cast<const T*>(a->q);
+    p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
+    p.cache = static_cast<const T*>(a->cache);
+    p.page_table = static_cast<const int*>(a->page_table); p.max_pages = a->max_pages;
+    p.H = a->H; p.G = a->G; p.d = a->d; p.P = a->P; p.window = a->window;
+    p.scale = a->scale; p.out_scale = a->out_scale; p.sink = a->sink;
+    p.sg = make_segments(seg, a->tokens);
+  };
+  if (a->f32) {
+    GqaAttn<float> p;
+    fill(p);
+    const dim3 grid(a->tokens, (a->H + 3) / 4);
+    switch (a->P / 64) {
+      case 1: return static_cast<int>(launch(gqa_row_kernel<2>, grid, dim3(128), 0, st, p));
+      case 2: return static_cast<int>(launch(gqa_row_kernel<4>, grid, dim3(128), 0, st, p));
+      case 3: return static_cast<int>(launch(gqa_row_kernel<6>, grid, dim3(128), 0, st, p));
+    }
+    return static_cast<int>(launch(gqa_row_kernel<8>, grid, dim3(128), 0, st, p));
+  }
+  GqaMma p;
+  fill(p.a);
+  p.splits = a->splits > 1 ? a->splits : 1;
+  p.partial = static_cast<float*>(a->partial);
+  if (a->decode) {
+    p.hb = 16; p.qb = 1;
+    p.head_tiles = (a->H / a->G + 15) / 16;
+    const dim3 grid(seg->num, a->G * p.head_tiles, p.splits);
+    if (grid.y > 65535) return -11;
+    switch (a->P / 64) {
+      case 1: return gqa_decode<1>(p, grid, st);
+      case 2: return gqa_decode<2>(p, grid, st);
+      case 3: return gqa_decode<3>(p, grid, st);
+    }
+    return gqa_decode<4>(p, grid, st);
+  }
+  int nw;
+  gqa_shape(a->tokens, seg->num, a->H, a->G, nw, p.hb, p.qb, p.head_tiles);
+  const dim3 grid(max_tiles(a->tokens, seg->num, p.qb), a->G * p.head_tiles);
+  if (grid.y > 65535) return -11;
+  switch (a->P / 64 * 10 + nw) {
+    case 14: return gqa_prefill<4, 1>(p, grid, st);
+    case 18: return gqa_prefill<8, 1>(p, grid, st);
+    case 24: return gqa_prefill<4, 2>(p, grid, st);
+    case 28: return gqa_prefill<8, 2>(p, grid, st);
+    case 34: return gqa_prefill<4, 3>(p, grid, st);
+    case 38: return gqa_prefill<8, 3>(p, grid, st);
+    case 44: return gqa_prefill<4, 4>(p, grid, st);
+  }
+  return gqa_prefill<8, 4>(p, grid, st);
+}
+
+}  // extern "C"

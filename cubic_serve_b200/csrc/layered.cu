@@ -2,6 +2,7 @@
 // layer's norm writes the activation type T (bf16, or fp32 when the model runs in 32-bit).
 #include "segments.cuh"
 #include "launch.cuh"
+#include "mma.cuh"
 
 namespace cb {
 
@@ -103,6 +104,235 @@ concat_rows_kernel(const float* __restrict__ x, const float* __restrict__ x0, T*
   }
 }
 
+// A row of up to 8192 columns (a multiple of 4) over the block's threads in registers, four columns at a time.
+struct Row8 {
+  float4 v[8];
+  template <typename F> __device__ __forceinline__ void each(int W, F f) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int c = threadIdx.x + i * kRowThreads;
+      if (c < (W >> 2)) f(c, v[i]);
+    }
+  }
+};
+__device__ __forceinline__ float dot4(float4 a, float4 b) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w))); }
+__device__ __forceinline__ float4 load4(const float* p, int c) { return reinterpret_cast<const float4*>(p)[c]; }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p, int c) {
+  const uint2 u = reinterpret_cast<const uint2*>(p)[c];
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float* p, int c, float4 v) { reinterpret_cast<float4*>(p)[c] = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, int c, float4 v) {
+  reinterpret_cast<uint2*>(p)[c] = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+// x[t] = table[ids[t]] (fp32) and h[t] = x[t] * w / rms(x[t])
+template <typename T>
+__global__ void __launch_bounds__(kRowThreads)
+embed_rows_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__ table, const float* __restrict__ w,
+                  float* __restrict__ x, T* __restrict__ h, int ldh, int W, int vocab, float eps) {
+  __shared__ float red[8];
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t t = blockIdx.x;
+  const int id = min(max(ids[t], 0), vocab - 1);
+  const __nv_bfloat16* e = table + static_cast<size_t>(id) * W;
+  float* xr = x + t * W;
+  T* hr = h + t * ldh;
+  float ss = 0.f;
+  if ((W & 3) == 0 && W <= 32 * kRowThreads) {
+    Row8 r;
+    r.each(W, [&](int c, float4& v) { v = load4(e, c); ss += dot4(v, v); store4(xr, c, v); });
+    const float inv = 1.f / sqrtf(row_sum(ss, red) / static_cast<float>(W) + eps);
+    r.each(W, [&](int c, float4& v) {
+      const float4 g = load4(w, c);
+      store4(hr, c, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+    });
+    return;
+  }
+  for (int c = threadIdx.x; c < W; c += kRowThreads) {
+    const float v = __bfloat162float(e[c]);
+    ss = fmaf(v, v, ss);
+    xr[c] = v;
+  }
+  const float inv = 1.f / sqrtf(row_sum(ss, red) / static_cast<float>(W) + eps);
+  for (int c = threadIdx.x; c < W; c += kRowThreads) hr[c] = from_f<T>(__bfloat162float(e[c]) * inv * w[c]);
+}
+
+// x[t] += y[t] * w / rms(y[t]); then, with h, h[t] = x[t] * w2 / rms(x[t]): a normed addition to the residual and the norm that
+// reads it next
+template <typename T>
+__global__ void __launch_bounds__(kRowThreads)
+add_norm_rows_kernel(const T* __restrict__ y, int ldy, const float* __restrict__ w, float* __restrict__ x,
+                     const float* __restrict__ w2, T* __restrict__ h, int ldh, int W, float eps) {
+  __shared__ float red[8], red2[8];
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t t = blockIdx.x;
+  const T* yr = y + t * ldy;
+  float* xr = x + t * W;
+  float ss = 0.f, s2 = 0.f;
+  if ((W & 3) == 0 && (ldy & 3) == 0 && W <= 32 * kRowThreads) {
+    Row8 r, o;
+    r.each(W, [&](int c, float4& v) { v = load4(yr, c); ss += dot4(v, v); });
+    o.each(W, [&](int c, float4& v) { v = load4(xr, c); });
+    const float inv = 1.f / sqrtf(row_sum(ss, red) / static_cast<float>(W) + eps);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int c = threadIdx.x + i * kRowThreads;
+      if (c >= (W >> 2)) continue;
+      const float4 g = load4(w, c), v = r.v[i];
+      float4& u = o.v[i];
+      u.x = fmaf(v.x * inv, g.x, u.x); u.y = fmaf(v.y * inv, g.y, u.y);
+      u.z = fmaf(v.z * inv, g.z, u.z); u.w = fmaf(v.w * inv, g.w, u.w);
+      store4(xr, c, u);
+      s2 += dot4(u, u);
+    }
+    if (!h) return;
+    const float in2 = 1.f / sqrtf(row_sum(s2, red2) / static_cast<float>(W) + eps);
+    T* hr = h + t * ldh;
+    o.each(W, [&](int c, float4& u) {
+      const float4 g = load4(w2, c);
+      store4(hr, c, make_float4(u.x * in2 * g.x, u.y * in2 * g.y, u.z * in2 * g.z, u.w * in2 * g.w));
+    });
+    return;
+  }
+  for (int c = threadIdx.x; c < W; c += kRowThreads) { const float v = to_f(yr[c]); ss = fmaf(v, v, ss); }
+  const float inv = 1.f / sqrtf(row_sum(ss, red) / static_cast<float>(W) + eps);
+  for (int c = threadIdx.x; c < W; c += kRowThreads) {
+    const float u = fmaf(to_f(yr[c]) * inv, w[c], xr[c]);
+    xr[c] = u;
+    s2 = fmaf(u, u, s2);
+  }
+  if (!h) return;
+  const float in2 = 1.f / sqrtf(row_sum(s2, red2) / static_cast<float>(W) + eps);
+  for (int c = threadIdx.x; c < W; c += kRowThreads) h[t * ldh + c] = from_f<T>(xr[c] * in2 * w2[c]);
+}
+
+// ------------------------------------------------------------------ gate of a token's side input
+// out[t, n] = gelu_tanh(x[t] . w[n]) * table[ids[t], col + n] with few outputs n: the fp32 residual is read once and rounded on
+// its way into the product (bf16 models).
+struct SideGate {
+  const float* x; int W;
+  const __nv_bfloat16* w; int ldw;        // [dim, ldw], zero columns behind W
+  const int* ids;
+  const __nv_bfloat16* table; int ldt, col, vocab;
+  void* out; int ldo;
+  int T, dim;
+};
+
+static constexpr int kSideWarps = 8;
+
+// A block takes 16 tokens and 8 NB outputs; its warps and the blocks of its cluster (grid.z) deal the columns of x in chunks of
+// 32.  Lane (g, t4) feeds the columns 8 t4 .. + 7 of a chunk to two tensor-core steps: which column goes to which place of a step
+// is the same for both operands, so 16-byte loads make the fragments.
+template <int NB>
+__global__ void __launch_bounds__(32 * kSideWarps)
+side_gate_mma_kernel(const SideGate p) {
+  __shared__ float part[kSideWarps][16][NB * 8 + 1];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+  const int t0 = blockIdx.x * 16, n0 = blockIdx.y * NB * 8;
+  pdl_wait();
+  pdl_launch_dependents();
+  float acc[NB][4] = {};
+  const int chunks = (p.W + 31) / 32, step = kSideWarps * gridDim.z;
+  const bool vec = (p.W & 3) == 0;
+  for (int ch = blockIdx.z * kSideWarps + warp; ch < chunks; ch += step) {
+    const int k = ch * 32 + 8 * t4;
+    float a[2][8];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int t = t0 + g + 8 * i;
+      const float* xr = p.x + static_cast<size_t>(t) * p.W + k;
+#pragma unroll
+      for (int j = 0; j < 8; j += 4) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (t < p.T) {
+          if (vec) {
+            if (k + j < p.W) v = *reinterpret_cast<const float4*>(xr + j);
+          } else {
+            if (k + j < p.W) v.x = xr[j];
+            if (k + j + 1 < p.W) v.y = xr[j + 1];
+            if (k + j + 2 < p.W) v.z = xr[j + 2];
+            if (k + j + 3 < p.W) v.w = xr[j + 3];
+          }
+        }
+        a[i][j] = v.x; a[i][j + 1] = v.y; a[i][j + 2] = v.z; a[i][j + 3] = v.w;
+      }
+    }
+    uint4 b[NB];
+#pragma unroll
+    for (int n = 0; n < NB; ++n) {
+      const int row = n0 + n * 8 + g;
+      b[n] = row < p.dim ? *reinterpret_cast<const uint4*>(p.w + static_cast<size_t>(row) * p.ldw + k) : make_uint4(0, 0, 0, 0);
+    }
+    const uint32_t a0[4] = {pack_bf16x2(a[0][0], a[0][1]), pack_bf16x2(a[1][0], a[1][1]), pack_bf16x2(a[0][2], a[0][3]), pack_bf16x2(a[1][2], a[1][3])};
+    const uint32_t a1[4] = {pack_bf16x2(a[0][4], a[0][5]), pack_bf16x2(a[1][4], a[1][5]), pack_bf16x2(a[0][6], a[0][7]), pack_bf16x2(a[1][6], a[1][7])};
+#pragma unroll
+    for (int n = 0; n < NB; ++n) {
+      mma_bf16(acc[n], a0, b[n].x, b[n].y);
+      mma_bf16(acc[n], a1, b[n].z, b[n].w);
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < NB; ++n)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) part[warp][g + 8 * (c >> 1)][n * 8 + 2 * t4 + (c & 1)] = acc[n][c];
+  __syncthreads();
+  const int cluster = gridDim.z;
+  if (cluster > 1) {
+    for (int i = threadIdx.x; i < 16 * NB * 8; i += blockDim.x) {
+      const int r = i / (NB * 8), n = i % (NB * 8);
+      float z = 0.f;
+#pragma unroll
+      for (int w = 0; w < kSideWarps; ++w) z += part[w][r][n];
+      part[0][r][n] = z;
+    }
+    __syncwarp();
+    cluster_sync_all();
+  }
+  // the blocks of a cluster share the rows
+  for (int i = threadIdx.x + blockIdx.z * blockDim.x; i < 16 * NB * 8; i += blockDim.x * cluster) {
+    const int r = i / (NB * 8), n = i % (NB * 8), t = t0 + r;
+    if (t >= p.T || n0 + n >= p.dim) continue;
+    float z = 0.f;
+    if (cluster > 1) {
+      const uint32_t at = smem_u32(&part[0][r][n]);
+      for (int c = 0; c < cluster; ++c) z += ld_cluster_f32(cluster_map(at, c));
+    } else {
+#pragma unroll
+      for (int w = 0; w < kSideWarps; ++w) z += part[w][r][n];
+    }
+    const int id = min(max(p.ids[t], 0), p.vocab - 1);
+    const float e = __bfloat162float(p.table[static_cast<size_t>(id) * p.ldt + p.col + n0 + n]);
+    static_cast<__nv_bfloat16*>(p.out)[static_cast<size_t>(t) * p.ldo + n0 + n] = __float2bfloat16(gelu_tanh_fast(z) * e);
+  }
+  __syncwarp();
+  if (cluster > 1) cluster_sync_all();                   // nobody leaves while others read its sums
+}
+
+// The same in 32-bit, a block per token and a warp per output.
+__global__ void __launch_bounds__(32 * kSideWarps)
+side_gate_f32_kernel(const SideGate p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t t = blockIdx.x;
+  const int lane = threadIdx.x & 31;
+  const float* xr = p.x + t * p.W;
+  const int id = min(max(p.ids[t], 0), p.vocab - 1);
+  for (int n = threadIdx.x >> 5; n < p.dim; n += kSideWarps) {
+    const __nv_bfloat16* wr = p.w + static_cast<size_t>(n) * p.ldw;
+    float z = 0.f;
+    for (int c = lane; c < p.W; c += 32) z = fmaf(xr[c], __bfloat162float(wr[c]), z);
+    z = warp_sum(z);
+    if (lane == 0)
+      static_cast<float*>(p.out)[t * p.ldo + n] =
+          gelu_tanh(z) * __bfloat162float(p.table[static_cast<size_t>(id) * p.ldt + p.col + n]);
+  }
+}
+
 // ------------------------------------------------------------------ fp32 matrix product
 // y[m, n] = sum_k x[m, k] w[n, k] with fp32 x and bf16-stored weights (exact in fp32), fused multiply-adds in k order:
 // the product of a model that runs in 32-bit.  64 x 64 tile, 4 x 4 results per thread.  Epilogue and block-diagonal
@@ -114,6 +344,7 @@ struct F32Gemm {
   const float* residual;
   float* y2; int ldy2, n_split, diag_n;
   int M, N, K;
+  int glu;                    // gated gelu: 16 gate rows and 16 up rows of w in turn, y gets N / 2 features
 };
 
 __global__ void __launch_bounds__(256)
@@ -147,6 +378,21 @@ f32_gemm_kernel(const F32Gemm p) {
         for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
     }
     __syncthreads();
+  }
+  if (p.glu) {
+    // a thread's four columns are gate columns of features f .. f + 3 (tx & 4 clear) or their up columns, which the thread
+    // four places on holds
+    const int f = (n0 >> 1) + (tx >> 3) * 16 + (tx & 3) * 4;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int m = m0 + ty * 4 + i;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float u = __shfl_down_sync(0xffffffffu, acc[i][j], 4);
+        if (!(tx & 4) && m < p.M && f + j < (p.N >> 1)) p.y[static_cast<size_t>(m) * p.ldy + f + j] = gelu_tanh(acc[i][j]) * u;
+      }
+    }
+    return;
   }
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -211,6 +457,63 @@ int cb_concat_rows(const void* x, const void* x0, void* out, int ldo, int n, int
                                  static_cast<__nv_bfloat16*>(out), ldo, W));
 }
 
+int cb_embed_rows(const void* ids, const void* table, const void* w, void* x, void* h, int ldh, int n, int W, int vocab, float eps,
+                  int f32, void* stream) {
+  using namespace cb;
+  if (n <= 0) return 0;
+  if (W <= 0 || vocab <= 0 || ldh < W || (ldh & 3)) return -10;
+  auto go = [&](auto kernel, auto* out) {
+    return static_cast<int>(launch(kernel, dim3(n), dim3(kRowThreads), 0, static_cast<cudaStream_t>(stream),
+                                   static_cast<const int*>(ids), static_cast<const __nv_bfloat16*>(table),
+                                   static_cast<const float*>(w), static_cast<float*>(x), out, ldh, W, vocab, eps));
+  };
+  return f32 ? go(embed_rows_kernel<float>, static_cast<float*>(h)) : go(embed_rows_kernel<__nv_bfloat16>, static_cast<__nv_bfloat16*>(h));
+}
+
+// `h` may be null
+int cb_add_norm_rows(const void* y, int ldy, const void* w, void* x, const void* w2, void* h, int ldh, int n, int W, float eps,
+                     int f32, void* stream) {
+  using namespace cb;
+  if (n <= 0) return 0;
+  if (W <= 0 || ldy < W || (h && (ldh < W || (ldh & 3) || !w2))) return -10;
+  auto go = [&](auto kernel, auto* src) {
+    using P = decltype(src);
+    return static_cast<int>(launch(kernel, dim3(n), dim3(kRowThreads), 0, static_cast<cudaStream_t>(stream), src, ldy,
+                                   static_cast<const float*>(w), static_cast<float*>(x), static_cast<const float*>(w2),
+                                   static_cast<P>(h), ldh, W, eps));
+  };
+  return f32 ? go(add_norm_rows_kernel<float>, static_cast<float*>(const_cast<void*>(y)))
+             : go(add_norm_rows_kernel<__nv_bfloat16>, static_cast<__nv_bfloat16*>(const_cast<void*>(y)));
+}
+
+int cb_side_gate(const void* x, int W, const void* w, int ldw, const void* ids, const void* table, int ldt, int col, void* out,
+                 int ldo, int n, int dim, int vocab, int f32, void* stream) {
+  using namespace cb;
+  if (n <= 0) return 0;
+  if (W <= 0 || dim <= 0 || vocab <= 0 || ldw < (W + 31) / 32 * 32 || (ldw & 7) || ldo < dim || col < 0 || col + dim > ldt) return -10;
+  SideGate p;
+  p.x = static_cast<const float*>(x); p.W = W;
+  p.w = static_cast<const __nv_bfloat16*>(w); p.ldw = ldw;
+  p.ids = static_cast<const int*>(ids);
+  p.table = static_cast<const __nv_bfloat16*>(table); p.ldt = ldt; p.col = col; p.vocab = vocab;
+  p.out = out; p.ldo = ldo; p.T = n; p.dim = dim;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32) return static_cast<int>(launch(side_gate_f32_kernel, dim3(n), dim3(32 * kSideWarps), 0, st, p));
+  const int nb = dim <= 8 ? 1 : dim <= 16 ? 2 : dim <= 32 ? 4 : 8;
+  const int tiles = (n + 15) / 16, ny = (dim + nb * 8 - 1) / (nb * 8);
+  if (ny > 65535) return -11;
+  // few tokens: a cluster shares the columns, as long as every warp of it has at least two chunks
+  int cluster = 1;
+  while (cluster < 8 && tiles * ny * cluster * 2 <= 148 && (W + 31) / 32 >= 4 * cluster * kSideWarps) cluster *= 2;
+  const dim3 grid(tiles, ny, cluster), shape(1, 1, cluster);
+  switch (nb) {
+    case 1: return static_cast<int>(launch(side_gate_mma_kernel<1>, grid, dim3(32 * kSideWarps), 0, st, shape, p));
+    case 2: return static_cast<int>(launch(side_gate_mma_kernel<2>, grid, dim3(32 * kSideWarps), 0, st, shape, p));
+    case 4: return static_cast<int>(launch(side_gate_mma_kernel<4>, grid, dim3(32 * kSideWarps), 0, st, shape, p));
+  }
+  return static_cast<int>(launch(side_gate_mma_kernel<8>, grid, dim3(32 * kSideWarps), 0, st, shape, p));
+}
+
 struct CbF32Gemm {
   const void* x; int ldx, x_cols;
   const void* w;
@@ -218,6 +521,7 @@ struct CbF32Gemm {
   const void* residual;
   void* y2; int ldy2, n_split, diag_n;
   int M, N, K;
+  int glu;
 };
 
 int cb_f32_gemm(const CbF32Gemm* a, void* stream) {
@@ -231,6 +535,8 @@ int cb_f32_gemm(const CbF32Gemm* a, void* stream) {
   p.residual = static_cast<const float*>(a->residual);
   p.y2 = static_cast<float*>(a->y2); p.ldy2 = a->ldy2; p.n_split = a->n_split; p.diag_n = a->diag_n;
   p.M = a->M; p.N = a->N; p.K = a->K;
+  p.glu = a->glu;
+  if (p.glu && (p.glu != 2 || p.y2 || p.residual || p.diag_n || (p.N % 32) != 0 || p.ldy < p.N / 2)) return -13;
   const dim3 grid((a->N + 63) / 64, (a->M + 63) / 64);
   if (grid.y > 65535) return -12;
   return static_cast<int>(launch(f32_gemm_kernel, grid, dim3(256), 0, static_cast<cudaStream_t>(stream), p));

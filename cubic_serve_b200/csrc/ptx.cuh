@@ -275,6 +275,11 @@ __device__ __forceinline__ bool mbar_wait_park_cluster(uint32_t bar, uint32_t pa
     }
   }
 }
+__device__ __forceinline__ float ld_cluster_f32(uint32_t cluster_addr) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(cluster_addr) : "memory");
+  return v;
+}
 // 16 bytes from the shared memory of a CTA of the cluster (address from cluster_map)
 __device__ __forceinline__ float4 ld_cluster_f4(uint32_t cluster_addr) {
   float4 v;
@@ -413,6 +418,12 @@ __device__ __forceinline__ uint32_t atom_add_acq_rel_gpu(uint32_t* p, uint32_t v
 // that applies SwiGLU uses this one function, so the fused and the stand-alone activation agree bit for bit.
 __device__ __forceinline__ float silu_fast(float x) {
   return __fdividef(x, 1.f + __expf(-x));
+}
+
+// The tanh form of gelu as x times a sigmoid, 0.5 (1 + tanh u) = 1 / (1 + e^-2u), with the same limits as silu_fast.
+__device__ __forceinline__ float gelu_tanh_fast(float x) {
+  const float u2 = 1.5957691216057308f * x * fmaf(0.044715f * x, x, 1.f);   // 2 sqrt(2 / pi) (x + 0.044715 x^3)
+  return __fdividef(x, 1.f + __expf(-u2));
 }
 
 __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {

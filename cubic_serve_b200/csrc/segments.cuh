@@ -21,6 +21,10 @@ template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 
+__device__ __forceinline__ float gelu_tanh(float x) {
+  return 0.5f * x * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * x * x, x, x)));
+}
+
 // Tile `tile` of the step when every segment is cut into tiles of `rows` rows: its segment and first row inside the
 // segment.  Called by whole warps; false when the step has fewer tiles.  The grid of a kernel that uses it holds at
 // most (T + num (rows - 1)) / rows tiles.

@@ -784,6 +784,7 @@ struct CbWideGemm {
   int ldy2, n_split, diag_n;
   int M, N, K;
   int stream_k, splits, min_units;
+  int glu;                    // gated activation (Glu): w's rows are interleaved, y [M, ldy] gets N / 2 features
 };
 
 // Per-launch options of the common launcher.  Everything that steers ONE launch travels in this struct (not in
@@ -936,6 +937,8 @@ static int wq_gemm_dispatch(int fmt, const void* x, int ldx, const void* codes, 
     const CbWideGemm& g = *o.wide;
     if (fmt != kFmtBf16 || residual || link || o.swiglu || o.tiles || g.x_cols <= 0 || g.x_cols > ldx) return -61;
     if ((!g.y && !g.y32) || (g.y && g.y32) || (g.y2 && (g.y32 || (g.n_split & 3) || g.n_split < 0))) return -62;
+    if (g.glu && (!g.y || g.y2 || g.diag_n || g.glu < 0 || g.glu > kGluGelu || (N % 32) != 0 || ldy < N / 2)) return -64;
+    p.swiglu = g.glu;
     if (g.diag_n && (stream_k || g.diag_n < 0 || (g.diag_n % kTileN) != 0)) return -63;
     p.wide = 1;
     p.y32 = static_cast<float*>(g.y32);
@@ -1036,7 +1039,8 @@ static int wq_gemm_dispatch(int fmt, const void* x, int ldx, const void* codes, 
 }
 
 // y = x W^T in bf16 with fp32 accumulation, written through the wide epilogue (see WqGemmParams::wide): fp32 output added
-// to an fp32 residual, or a second output behind the squared relu.  `diag_n`: block-diagonal weights.
+// to an fp32 residual, a second output behind the squared relu, or the gated activation of interleaved [gate ; up] rows.
+// `diag_n`: block-diagonal weights.
 int cb_bf16_gemm_wide(const CbWideGemm* g, void* workspace, long long workspace_bytes, void* counters, void* status,
                       void* stream) {
   if (!g) return -60;

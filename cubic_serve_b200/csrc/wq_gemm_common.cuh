@@ -88,7 +88,8 @@ struct WqGemmParams {
   unsigned long long* trace;  // optional pipeline timeline of CTA (0,0,0): [iteration][8] clock64 stamps
   // fused SwiGLU epilogue (gate/up projection): the weight rows were interleaved at load time so that a
   // 128-row tile holds 64 output features as four blocks of {16 gate rows, 16 up rows}; the epilogue writes
-  // act[m, 64 * n_tile + 16 * q + i] = silu(tile row 32 q + i) * (tile row 32 q + 16 + i), ldy = row stride of act
+  // act[m, 64 * n_tile + 16 * q + i] = silu(tile row 32 q + i) * (tile row 32 q + 16 + i), ldy = row stride of act;
+  // kGluGelu: the tanh form of gelu instead of silu
   int swiglu;
   // persistent kernel on CTA pairs (cta_group::2): the schedule's tile is a PAIR of adjacent weight tiles, CTA rank r of
   // the pair owns weight tile 2 * pair_tile + r and loads batch rows [m0 + r * mb / 2, + mb / 2) of the activation tile
@@ -161,12 +162,14 @@ __device__ __forceinline__ bool wait_counter_gpu(const uint32_t* p, uint32_t tar
   }
 }
 
-// SwiGLU on a pair of accumulators, with the rounding points of the unfused path (the projection's output is
+enum Glu : int { kGluNone = 0, kGluSilu = 1, kGluGelu = 2 };
+
+// Gated activation on a pair of accumulators, with the rounding points of the unfused path (the projection's output is
 // rounded to bf16, the activation is computed in fp32 from those and rounded once)
-__device__ __forceinline__ float silu_mul(float g, float u) {
+__device__ __forceinline__ float glu_mul(int kind, float g, float u) {
   g = __bfloat162float(__float2bfloat16(g));
   u = __bfloat162float(__float2bfloat16(u));
-  return silu_fast(g) * u;
+  return (kind == kGluGelu ? gelu_tanh_fast(g) : silu_fast(g)) * u;
 }
 // Four consecutive activation features j0..j0+3 (j0 % 4 == 0) of tile `n_tile` for row m from the fp32 gate / up
 // values of the tile row (already scaled by alpha)
@@ -174,7 +177,7 @@ __device__ __forceinline__ void store_act4(const WqGemmParams& p, int m, int n_t
   const int n_out = p.N >> 1;
   const int n0 = n_tile * 64 + j0;
   if (n0 >= n_out) return;
-  const float a[4] = {silu_mul(g.x, u.x), silu_mul(g.y, u.y), silu_mul(g.z, u.z), silu_mul(g.w, u.w)};
+  const float a[4] = {glu_mul(p.swiglu, g.x, u.x), glu_mul(p.swiglu, g.y, u.y), glu_mul(p.swiglu, g.z, u.z), glu_mul(p.swiglu, g.w, u.w)};
   __nv_bfloat16* dst = p.y + static_cast<size_t>(m) * p.ldy + n0;
   if ((p.ldy & 3) == 0 && n0 + 3 < n_out) {
     uint2 ov;

@@ -333,13 +333,11 @@ def inspect_checkpoint(path: str | Path) -> dict:
                 "manifest_digest": WeightManifest.from_store(store).digest, "execution_mode": "eager"}
     ck = admit_checkpoint(path)
     if ck.cfg.family == "layered":
-        from .layered import LatentSpec
         c = ck.cfg
-        mixers = [("latent" if isinstance(l.mixer, LatentSpec) else "channel_delta" if l.mixer.per_channel else "delta")
-                  for l in c.layers]
+        mixers = [l.mixer.label for l in c.layers]
         return {"model": c.name, "family": c.family, "architecture": c.architecture, "layers": c.num_layers,
                 "layer_runs": len(c.runs), "hidden": c.hidden_size, "vocab": c.vocab_size,
-                "mixers": {k: mixers.count(k) for k in sorted(set(mixers))}, "loop": c.loop,
+                "mixers": {k: mixers.count(k) for k in sorted(set(mixers))}, "loop": c.loop, "side_dim": c.side_dim,
                 "cache_bytes_per_token": c.page_bytes // 16, "state_bytes_per_request": c.state_bytes_per_request,
                 "tensors": len(ck.store.tensors), "elements": sum(math.prod(t.shape) for t in ck.store.tensors.values()),
                 "manifest_digest": WeightManifest.from_store(ck.store).digest}

@@ -1,18 +1,26 @@
-"""Layered decoders: every layer names its own token mixer, a run of layers may be repeated, the residual stream is fp32.
+"""Layered decoders: every layer names its own token mixer, the residual stream is fp32.
 
-``config.json`` of such a checkpoint has ``architecture`` (``Bumodra``), ``vocab``, ``width``, ``norm.eps``, the list
-``layers`` and optionally ``loop``.  A layer is parallel: mixer and feed-forward read the same norm and their outputs are
-added to the residual together.  ``loop`` = {start, stop, times} runs the layers ``start .. stop - 1`` ``times`` times with
-the same weights, each pass with its own cache and state; a pass starts with a projection of [residual ; embedding output].
+``config.json`` of such a checkpoint has ``architecture``, ``vocab``, ``width``, ``norm.eps`` and the list ``layers``.  What
+the layers of an architecture have in common is its entry in ``DESIGNS``:
 
-Mixers (``MIXERS``; another one is added there, in ``pack_layer`` and in ``models/layered_runner.py``):
+* ``Bumodra``: parallel layers (mixer and feed-forward read the same norm and are added to the residual together); ``loop`` =
+  {start, stop, times} runs the layers ``start .. stop - 1`` ``times`` times with the same weights, each pass with its own
+  cache and state; a pass starts with a projection of [residual ; embedding output];
+* ``Loduzen``: sequential layers (mixer, then feed-forward, each behind a norm of its own), tied output head; ``token_side`` =
+  {dim} adds, after the feed-forward, what the layer takes from its part of a second embedding of the token.
+
+Mixers (another one is a spec, a reader in ``_MIXER_READERS``, an inventory entry, a ``_pack_*`` function and a method of
+``models/layered_runner.py``):
 
 * ``delta`` / ``channel_delta``: short convolution, gated delta rule with one decay per head / per (head, key channel);
-* ``latent_attention``: attention over cached latents with a sliding window and a gate per head.
+* ``latent_attention``: attention over cached latents with a sliding window and a gate per head;
+* ``mamba2``: short convolution, scalar-decay linear recurrence (state-space duality), gated norm in equal parts;
+* ``parallel``: two mixers that read the same norm, each scaled: sliding-window grouped-query attention with head norms,
+  rotary pairs, a softmax sink and values that are the raw keys; and gated linear attention with a decay per key channel.
 
-Weights are packed for the parallel layout: ONE matrix holds all projections that read the norm (mixer inputs, then the
-feed-forward's up rows), ONE matrix holds both output projections side by side ([o | down]), so a layer has two large
-products whatever its mixer is.  Rows and columns are padded with zeros to what the GEMM asks for.
+ONE matrix holds all projections that read a layer's norm and ONE the output projections side by side, whatever the mixer is:
+with parallel layers the first also has the feed-forward's up rows and the second its down columns ([o | down]).  Rows and
+columns are padded with zeros to what the GEMM asks for.
 """
 from __future__ import annotations
 
@@ -24,10 +32,28 @@ from pathlib import Path
 import torch
 
 from ..ops import wq_pack
+from ..ops.eager import rope_inv_freq
 from .config import QuantSpec
 
-ARCHITECTURES = ("Bumodra",)
-MAX_CONV_TAPS, MAX_DELTA_DIM, MAX_LATENT = 16, 256, 1024      # limits of the kernels
+MAX_CONV_TAPS, MAX_DELTA_DIM, MAX_LATENT, MAX_HEAD = 16, 256, 1024, 256      # limits of the kernels
+
+
+@dataclass(frozen=True)
+class Design:
+    """What the layers of an architecture have in common."""
+    mixers: tuple[str, ...]
+    sequential: bool             # mixer and feed-forward one after the other, each with a norm; else in parallel behind one
+    norm_offset: float           # a norm's factor is this plus its stored weight
+    embed_norm: bool             # the embedding is normed before the first layer
+    tied_head: bool              # the output head is the embedding table
+    ff: str                      # "squared_relu" (up, down) or "gelu_glu" (gate, up, down)
+
+
+DESIGNS = {
+    "Bumodra": Design(("delta", "channel_delta", "latent_attention"), False, 1.0, True, False, "squared_relu"),
+    "Loduzen": Design(("parallel", "mamba2"), True, 0.0, False, True, "gelu_glu"),
+}
+ARCHITECTURES = tuple(DESIGNS)
 
 
 class LayeredConfigError(ValueError):
@@ -39,8 +65,24 @@ def round_up(n: int, m: int) -> int:
 
 
 # ------------------------------------------------------------------ configuration
+class MixerSpec:
+    """A layer's token mixer: sizes and constants.  ``parts``: the mixers it consists of (itself, unless it is a pair)."""
+
+    @property
+    def parts(self) -> tuple["MixerSpec", ...]:
+        return (self,)
+
+    def page_bytes(self, act_bytes: int) -> int:
+        """One 16-token page of its cache."""
+        return 0
+
+    def state_bytes(self, act_bytes: int) -> int:
+        """Recurrent state of a request."""
+        return 0
+
+
 @dataclass(frozen=True)
-class DeltaSpec:
+class DeltaSpec(MixerSpec):
     heads: int
     kv_heads: int
     dim: int
@@ -64,6 +106,10 @@ class DeltaSpec:
         return round_up(self.dim, 4)
 
     @property
+    def label(self) -> str:
+        return "channel_delta" if self.per_channel else "delta"
+
+    @property
     def out_width(self) -> int:
         return self.heads * self.vdim
 
@@ -78,7 +124,7 @@ class DeltaSpec:
 
 
 @dataclass(frozen=True)
-class LatentSpec:
+class LatentSpec(MixerSpec):
     heads: int
     dim: int
     vdim: int
@@ -86,6 +132,10 @@ class LatentSpec:
     kv_rank: int
     scale: float
     window: int = 0              # 0: every earlier token
+    label = "latent"
+
+    def page_bytes(self, act_bytes: int) -> int:
+        return 16 * self.rank_padded * act_bytes
 
     @property
     def rank_padded(self) -> int:
@@ -104,9 +154,163 @@ class LatentSpec:
 
 
 @dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions on neighbouring channel pairs of the first ``dims`` channels.  ``scaling``: as
+    ``ModelConfig.rope_scaling``; the attention factor of ``yarn`` multiplies cosine and sine here."""
+    dims: int
+    base: float
+    scaling: tuple | None = None
+
+    def table(self) -> tuple[torch.Tensor, float]:
+        """(fp32 radians per position of every pair, factor on cosine and sine)."""
+        f = rope_inv_freq(self.dims, self.base, scaling=self.scaling, dtype=torch.float64).float()
+        return f, float(self.scaling[5]) if self.scaling and self.scaling[0] == "yarn" else 1.0
+
+
+@dataclass(frozen=True)
+class AttentionSpec(MixerSpec):
+    """Grouped-query attention with head norms and rotary pairs; a value is the raw key of its token."""
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    rotary: RotarySpec
+    window: int = 0              # 0: every earlier token
+    sink: float | None = 0.0     # score of a softmax entry without a value (None: none)
+    label = "attention"
+
+    @property
+    def width_padded(self) -> int:
+        """Columns of a cached key or value: the widths the attention kernels are built for."""
+        return round_up(self.dim, 64)
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.dim
+
+    def page_bytes(self, act_bytes: int) -> int:
+        return 16 * self.kv_heads * 2 * self.width_padded * act_bytes
+
+    def validate(self) -> None:
+        if min(self.heads, self.kv_heads, self.dim) <= 0 or self.heads % self.kv_heads or self.window < 0:
+            raise LayeredConfigError("attention heads are grouped evenly over positive key head counts and sizes")
+        if self.dim > MAX_HEAD:
+            raise LayeredConfigError(f"attention heads of up to {MAX_HEAD} channels are served")
+        r = self.rotary
+        if r.dims % 2 or not 0 <= r.dims <= self.dim or r.base <= 0:
+            raise LayeredConfigError("rotary channels come in pairs inside a head")
+
+
+@dataclass(frozen=True)
+class GatedLinearSpec(MixerSpec):
+    """Gated linear attention: decay per key channel, a state of [key channel, value channel] per head."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float                   # the decay is a sigmoid to the power 1 / tau
+    decay_rank: int = 0          # inner size of the low-rank decay projection
+    label = "gated_linear"
+
+    @property
+    def state_stride(self) -> int:
+        return round_up(self.dim, 4)
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    def state_bytes(self, act_bytes: int) -> int:
+        return self.heads * self.vdim * self.state_stride * 4
+
+    def validate(self) -> None:
+        if min(self.heads, self.dim, self.vdim) <= 0 or self.tau <= 0:
+            raise LayeredConfigError("gated linear attention sizes and tau are positive")
+        if self.dim > MAX_DELTA_DIM:
+            raise LayeredConfigError(f"gated linear attention takes key widths of up to {MAX_DELTA_DIM}")
+
+
+@dataclass(frozen=True)
+class SsdSpec(MixerSpec):
+    """State-space duality layer (Mamba-2): ``heads`` of ``vdim`` channels, B and C of ``state`` channels per group."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_groups: int
+    label = "mamba2"
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        """Convolved channels: x of the heads, B and C of the groups."""
+        return self.out_width + 2 * self.groups * self.state
+
+    @property
+    def conv_width(self) -> int:
+        return round_up(self.channels, 8)
+
+    @property
+    def state_stride(self) -> int:
+        return round_up(self.state, 4)
+
+    def state_bytes(self, act_bytes: int) -> int:
+        return self.heads * self.vdim * self.state_stride * 4 + round_up((self.conv - 1) * self.conv_width * act_bytes, 16)
+
+    def validate(self) -> None:
+        if min(self.heads, self.vdim, self.state, self.groups, self.conv, self.norm_groups) <= 0 or self.heads % self.groups \
+                or self.out_width % self.norm_groups:
+            raise LayeredConfigError("mamba2 heads are grouped evenly and the normed width is cut evenly")
+        if self.conv > MAX_CONV_TAPS or self.state > MAX_DELTA_DIM:
+            raise LayeredConfigError(f"mamba2 layers take up to {MAX_CONV_TAPS} convolution taps and state width {MAX_DELTA_DIM}")
+
+
+@dataclass(frozen=True)
+class PairSpec(MixerSpec):
+    """Two mixers side by side on the same input: ``left_scale * left + right_scale * right``."""
+    left: MixerSpec
+    right: MixerSpec
+    left_scale: float
+    right_scale: float
+
+    @property
+    def label(self) -> str:
+        return f"{self.left.label}+{self.right.label}"
+
+    @property
+    def parts(self) -> tuple[MixerSpec, ...]:
+        return (self.left, self.right)
+
+    @property
+    def right_off(self) -> int:
+        """Column of the right outputs in the operand of the joint output product."""
+        return round_up(self.left.out_width, 8)
+
+    @property
+    def out_width(self) -> int:
+        return self.right_off + self.right.out_width
+
+    def page_bytes(self, act_bytes: int) -> int:
+        return sum(p.page_bytes(act_bytes) for p in self.parts)
+
+    def state_bytes(self, act_bytes: int) -> int:
+        return sum(p.state_bytes(act_bytes) for p in self.parts)
+
+    def validate(self) -> None:
+        for p in self.parts:
+            p.validate()
+
+
+ATTENTION_SPECS, RECURRENT_SPECS = (LatentSpec, AttentionSpec), (DeltaSpec, GatedLinearSpec, SsdSpec)
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: object                # DeltaSpec | LatentSpec
-    ff: int = 0                  # feed-forward width (squared relu); 0 = none
+    mixer: MixerSpec
+    ff: int = 0                  # feed-forward width; 0 = none
 
 
 @dataclass(frozen=True)
@@ -119,8 +323,9 @@ class LayeredConfig:
     loop: tuple[int, int, int] | None = None      # (start, stop, times)
     dtype: str = "bfloat16"                       # activations and products: bfloat16 | float32
     architecture: str = ARCHITECTURES[0]
+    side_dim: int = 0                             # width of a layer's part of the token's side embedding; 0 = none
     family: str = "layered"
-    max_position: int = 1 << 20                   # no positions enter the model: only memory limits the context
+    max_position: int = 1 << 20                   # positions are rotary or none: only memory limits the context
     quant: QuantSpec = field(default_factory=lambda: QuantSpec("none", 16, 0))
     eos_token_id: int | None = None
 
@@ -134,9 +339,13 @@ class LayeredConfig:
         return len(self.layers)
 
     @property
+    def design(self) -> Design:
+        return DESIGNS[self.architecture]
+
+    @property
     def is_hybrid(self) -> bool:
         """Some layer keeps recurrent state per request."""
-        return any(isinstance(l.mixer, DeltaSpec) for l in self.layers)
+        return any(l.mixer.state_bytes(4) for l in self.layers)
 
     @property
     def act_bytes(self) -> int:
@@ -155,13 +364,15 @@ class LayeredConfig:
     @property
     def page_bytes(self) -> int:
         """One 16-token page of every attention run."""
-        return sum(16 * self.layers[i].mixer.rank_padded * self.act_bytes for i, _ in self.runs
-                   if isinstance(self.layers[i].mixer, LatentSpec))
+        return sum(self.layers[i].mixer.page_bytes(self.act_bytes) for i, _ in self.runs)
 
     @property
     def state_bytes_per_request(self) -> int:
-        return sum(self.layers[i].mixer.state_bytes(self.act_bytes) for i, _ in self.runs
-                   if isinstance(self.layers[i].mixer, DeltaSpec))
+        return sum(self.layers[i].mixer.state_bytes(self.act_bytes) for i, _ in self.runs)
+
+    def run_parts(self, kind: type | tuple[type, ...]) -> int:
+        """How many mixers of a kind the layer runs have (each with a cache or state of its own)."""
+        return sum(isinstance(p, kind) for i, _ in self.runs for p in self.layers[i].mixer.parts)
 
     def validate(self) -> None:
         if min(self.vocab_size, self.hidden_size, len(self.layers)) <= 0 or self.rms_eps < 0:
@@ -172,6 +383,8 @@ class LayeredConfig:
             l.mixer.validate()
             if l.ff < 0:
                 raise LayeredConfigError("feed-forward widths are positive")
+        if self.side_dim < 0 or (self.side_dim or self.design.sequential) and self.loop is not None:
+            raise LayeredConfigError("sequential layers are run once, and the side input of a layer has a positive width")
         if self.loop is not None:
             a, b, times = self.loop
             if not 0 <= a < b <= self.num_layers or times < 1:
@@ -179,26 +392,90 @@ class LayeredConfig:
 
     def to_config(self) -> dict:
         """The ``config.json`` object of this configuration."""
-        layers = []
-        for l in self.layers:
-            m = l.mixer
-            if isinstance(m, DeltaSpec):
-                kind = "channel_delta" if m.per_channel else "delta"
-                mix = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv}
-            else:
-                kind = "latent_attention"
-                mix = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "q_rank": m.q_rank, "kv_rank": m.kv_rank,
-                       "scale": m.scale, "mask": {"size": m.window} if m.window else None}
-            layers.append({"type": kind, "mixer": mix, "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None})
-        loop = None if self.loop is None else dict(zip(("start", "stop", "times"), self.loop))
-        return {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
-                "norm": {"eps": self.rms_eps}, "layers": layers, "loop": loop}
+        layers = [{**dict(zip(("type", "mixer"), _mixer_config(l.mixer))),
+                   "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None} for l in self.layers]
+        out = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
+               "norm": {"eps": self.rms_eps}, "layers": layers}
+        if self.design.sequential:
+            out["token_side"] = {"dim": self.side_dim} if self.side_dim else None
+        else:
+            out["loop"] = None if self.loop is None else dict(zip(("start", "stop", "times"), self.loop))
+        return out
+
+
+def _mask_config(window: int) -> dict | None:
+    return {"size": window} if window else None
+
+
+def _mixer_config(m: MixerSpec) -> tuple[str, dict]:
+    """(type, mixer object) of a layer's entry in ``config.json``."""
+    if isinstance(m, DeltaSpec):
+        return m.label, {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv}
+    if isinstance(m, LatentSpec):
+        return "latent_attention", {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "q_rank": m.q_rank, "kv_rank": m.kv_rank,
+                                    "scale": m.scale, "mask": _mask_config(m.window)}
+    if isinstance(m, SsdSpec):
+        return "mamba2", {"heads": m.heads, "vdim": m.vdim, "state": m.state, "groups": m.groups, "conv": m.conv,
+                          "norm_groups": m.norm_groups}
+    a, g, sc = m.left, m.right, m.left.rotary.scaling
+    rot = {"dims": a.rotary.dims, "base": a.rotary.base,
+           "scaling": dict(zip(("factor", "original", "fast", "slow"), sc[1:5])) if sc else None}
+    return "parallel", {"left": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.dim, "scale": a.scale,
+                                 "mask": _mask_config(a.window), "rot": rot},
+                        "right": {"heads": g.heads, "dim": g.dim, "vdim": g.vdim, "tau": g.tau},
+                        "left_scale": m.left_scale, "right_scale": m.right_scale}
 
 
 def architecture_of(raw: dict) -> str | None:
     """Architecture a configuration names when it is one of this family's, else None."""
     arch = raw.get("architecture")
     return arch if arch in ARCHITECTURES else None
+
+
+def _window(m: dict) -> int:
+    mask = m.get("mask")
+    if not mask:
+        return 0
+    if int(mask["size"]) < 1:
+        raise LayeredConfigError("an attention window holds at least the token itself")
+    return int(mask["size"])
+
+
+def _read_rotary(rot: dict | None) -> RotarySpec:
+    if not rot:
+        return RotarySpec(0, 1.0)
+    sc = rot.get("scaling")
+    if sc:
+        factor = float(sc["factor"])
+        sc = ("yarn", factor, float(sc["original"]), float(sc["fast"]), float(sc["slow"]), 0.1 * math.log(factor) + 1.0)
+    return RotarySpec(int(rot["dims"]), float(rot["base"]), sc or None)
+
+
+def _read_delta(m: dict, p: str, rank, per_channel: bool = False) -> DeltaSpec:
+    return DeltaSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]), per_channel,
+                     rank(f"{p}.a1") if per_channel else 0, rank(f"{p}.g1") if per_channel else 0)
+
+
+def _read_latent(m: dict, p: str, rank) -> LatentSpec:
+    return LatentSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["q_rank"]), int(m["kv_rank"]), float(m["scale"]),
+                      _window(m))
+
+
+def _read_mamba2(m: dict, p: str, rank) -> SsdSpec:
+    return SsdSpec(int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["groups"]), int(m["conv"]), int(m["norm_groups"]))
+
+
+def _read_parallel(m: dict, p: str, rank) -> PairSpec:
+    a, g = m["left"], m["right"]
+    if int(a.get("vdim", a["dim"])) != int(a["dim"]):
+        raise LayeredConfigError("the values of this attention are its keys: vdim equals dim")
+    left = AttentionSpec(int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), float(a["scale"]), _read_rotary(a.get("rot")), _window(a))
+    right = GatedLinearSpec(int(g["heads"]), int(g["dim"]), int(g["vdim"]), float(g["tau"]), rank(f"{p}.right.a1"))
+    return PairSpec(left, right, float(m["left_scale"]), float(m["right_scale"]))
+
+
+_MIXER_READERS = {"delta": _read_delta, "channel_delta": lambda m, p, rank: _read_delta(m, p, rank, True),
+                  "latent_attention": _read_latent, "mamba2": _read_mamba2, "parallel": _read_parallel}
 
 
 def parse_layered_config(raw: dict, shapes: dict[str, tuple[int, ...]] | None = None, name: str = "") -> LayeredConfig:
@@ -216,74 +493,94 @@ def parse_layered_config(raw: dict, shapes: dict[str, tuple[int, ...]] | None = 
 
     layers = []
     for i, l in enumerate(raw["layers"]):
-        m, kind = l["mixer"], l["type"]
-        if kind in ("delta", "channel_delta"):
-            ch = kind == "channel_delta"
-            mixer = DeltaSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]), ch,
-                              rank(f"l{i}.mix.a1") if ch else 0, rank(f"l{i}.mix.g1") if ch else 0)
-        elif kind == "latent_attention":
-            mask = m.get("mask")
-            mixer = LatentSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["q_rank"]), int(m["kv_rank"]),
-                               float(m["scale"]), int(mask["size"]) if mask else 0)
-            if mask and mixer.window < 1:
-                raise LayeredConfigError("an attention window holds at least the token itself")
-        else:
-            raise LayeredConfigError(f"layer {i}: unknown mixer {kind!r}")
+        if l["type"] not in DESIGNS[arch].mixers:
+            raise LayeredConfigError(f"layer {i}: unknown mixer {l['type']!r}")
+        mixer = _MIXER_READERS[l["type"]](l["mixer"], f"l{i}.mix", rank)
         mlp = l.get("mlp")
         if mlp and mlp.get("kind") != "dense":
             raise LayeredConfigError(f"layer {i}: unknown feed-forward {mlp.get('kind')!r}")
         layers.append(LayerSpec(mixer, int(mlp["ff"]) if mlp else 0))
-    loop = raw.get("loop")
+    loop, side = raw.get("loop"), raw.get("token_side")
     cfg = LayeredConfig(name or arch, int(raw["vocab"]), int(raw["width"]), tuple(layers), float(raw["norm"]["eps"]),
-                        (int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None, architecture=arch)
+                        (int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None, architecture=arch,
+                        side_dim=int(side["dim"]) if side else 0)
     cfg.validate()
     return cfg
 
 
 # ------------------------------------------------------------------ tensor inventory
+def _mixer_shapes(m: MixerSpec, p: str, W: int) -> dict[str, tuple[int, ...]]:
+    out: dict[str, tuple[int, ...]] = {}
+    if isinstance(m, PairSpec):
+        return {**_mixer_shapes(m.left, f"{p}.left", W), **_mixer_shapes(m.right, f"{p}.right", W)}
+    if isinstance(m, DeltaSpec):
+        for t, c in (("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.heads * m.vdim)):
+            out[f"{p}.{t}"] = (c, W)
+            out[f"{p}.{t}.conv"] = (c, m.conv)
+        out[f"{p}.b"] = (m.heads, W)
+        out[f"{p}.A_log"] = (m.heads,)
+        out[f"{p}.norm"] = (m.vdim,)
+        if m.per_channel:
+            out.update({f"{p}.a1": (m.decay_rank, W), f"{p}.a2": (m.heads * m.dim, m.decay_rank),
+                        f"{p}.dt_bias": (m.heads * m.dim,),
+                        f"{p}.g1": (m.gate_rank, W), f"{p}.g2": (m.heads * m.vdim, m.gate_rank)})
+        else:
+            out.update({f"{p}.a": (m.heads, W), f"{p}.dt_bias": (m.heads,), f"{p}.g": (m.heads * m.vdim, W)})
+    elif isinstance(m, LatentSpec):
+        out.update({f"{p}.dq": (m.q_rank, W), f"{p}.dq.norm": (m.q_rank,), f"{p}.uq": (m.heads * m.dim, m.q_rank),
+                    f"{p}.dkv": (m.kv_rank, W), f"{p}.dkv.norm": (m.kv_rank,), f"{p}.uk": (m.heads * m.dim, m.kv_rank),
+                    f"{p}.uv": (m.heads * m.vdim, m.kv_rank), f"{p}.g": (m.heads, W)})
+    elif isinstance(m, AttentionSpec):
+        out.update({f"{p}.q": (m.heads * m.dim, W), f"{p}.k": (m.kv_heads * m.dim, W), f"{p}.q.norm": (m.dim,),
+                    f"{p}.k.norm": (m.dim,)})
+    elif isinstance(m, GatedLinearSpec):
+        out.update({f"{p}.{t}": (m.heads * c, W) for t, c in (("q", m.dim), ("k", m.dim), ("v", m.vdim), ("g", m.vdim))})
+        out.update({f"{p}.norm": (m.vdim,), f"{p}.a1": (m.decay_rank, W), f"{p}.a2": (m.heads * m.dim, m.decay_rank),
+                    f"{p}.a2.b": (m.heads * m.dim,)})
+    else:
+        out.update({f"{p}.in": (m.out_width + m.channels + m.heads, W), f"{p}.conv": (m.channels, m.conv),
+                    f"{p}.conv.b": (m.channels,), f"{p}.dt_bias": (m.heads,), f"{p}.A_log": (m.heads,), f"{p}.D": (m.heads,),
+                    f"{p}.norm": (m.out_width,)})
+    out[f"{p}.o"] = (W, m.out_width)
+    return out
+
+
 def tensor_shapes(cfg: LayeredConfig) -> dict[str, tuple[int, ...]]:
     """Every tensor of a checkpoint of this configuration."""
-    W = cfg.hidden_size
-    out: dict[str, tuple[int, ...]] = {"embed": (cfg.vocab_size, W), "embed.norm": (W,), "final.norm": (W,),
-                                       "head": (cfg.vocab_size, W)}
+    W, d = cfg.hidden_size, cfg.design
+    out: dict[str, tuple[int, ...]] = {"embed": (cfg.vocab_size, W), "final.norm": (W,)}
+    if d.embed_norm:
+        out["embed.norm"] = (W,)
+    if not d.tied_head:
+        out["head"] = (cfg.vocab_size, W)
     if cfg.loop is not None:
         out["loop.in"] = (W, 2 * W)
+    if cfg.side_dim:
+        out["side.embed"] = (cfg.vocab_size, cfg.num_layers * cfg.side_dim)
     for i, l in enumerate(cfg.layers):
-        m, p = l.mixer, f"l{i}.mix"
         out[f"l{i}.norm1"] = (W,)
-        if isinstance(m, DeltaSpec):
-            for t, c in (("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.heads * m.vdim)):
-                out[f"{p}.{t}"] = (c, W)
-                out[f"{p}.{t}.conv"] = (c, m.conv)
-            out[f"{p}.b"] = (m.heads, W)
-            out[f"{p}.A_log"] = (m.heads,)
-            out[f"{p}.norm"] = (m.vdim,)
-            if m.per_channel:
-                out.update({f"{p}.a1": (m.decay_rank, W), f"{p}.a2": (m.heads * m.dim, m.decay_rank),
-                            f"{p}.dt_bias": (m.heads * m.dim,),
-                            f"{p}.g1": (m.gate_rank, W), f"{p}.g2": (m.heads * m.vdim, m.gate_rank)})
-            else:
-                out.update({f"{p}.a": (m.heads, W), f"{p}.dt_bias": (m.heads,), f"{p}.g": (m.heads * m.vdim, W)})
-        else:
-            out.update({f"{p}.dq": (m.q_rank, W), f"{p}.dq.norm": (m.q_rank,), f"{p}.uq": (m.heads * m.dim, m.q_rank),
-                        f"{p}.dkv": (m.kv_rank, W), f"{p}.dkv.norm": (m.kv_rank,), f"{p}.uk": (m.heads * m.dim, m.kv_rank),
-                        f"{p}.uv": (m.heads * m.vdim, m.kv_rank), f"{p}.g": (m.heads, W)})
-        out[f"{p}.o"] = (W, m.out_width)
+        out.update(_mixer_shapes(l.mixer, f"l{i}.mix", W))
         if l.ff:
+            if d.sequential:
+                out[f"l{i}.norm2"] = (W,)
+            if d.ff == "gelu_glu":
+                out[f"l{i}.mlp.gate"] = (l.ff, W)
             out[f"l{i}.mlp.up"] = (l.ff, W)
             out[f"l{i}.mlp.down"] = (W, l.ff)
+        if cfg.side_dim:
+            out.update({f"l{i}.side.gate": (cfg.side_dim, W), f"l{i}.side.proj": (W, cfg.side_dim), f"l{i}.side.norm": (W,)})
     return out
 
 
 def check_inventory(cfg: LayeredConfig, shapes: dict[str, tuple[int, ...]]) -> None:
-    """The checkpoint's tensors are exactly the configuration's."""
+    """The checkpoint's tensors are exactly the configuration's (a second norm without a feed-forward behind it is ignored)."""
     want = tensor_shapes(cfg)
     for n, s in want.items():
         if n not in shapes:
             raise LayeredConfigError(f"missing tensor {n}")
         if tuple(shapes[n]) != s:
             raise LayeredConfigError(f"{n}: shape {tuple(shapes[n])}, expected {s}")
-    extra = sorted(set(shapes) - set(want))
+    extra = sorted(set(shapes) - set(want) - {f"l{i}.norm2" for i, l in enumerate(cfg.layers) if cfg.design.sequential and not l.ff})
     if extra:
         raise LayeredConfigError(f"checkpoint has {len(extra)} tensors this configuration does not own, e.g. {extra[:3]}")
 
@@ -291,20 +588,21 @@ def check_inventory(cfg: LayeredConfig, shapes: dict[str, tuple[int, ...]]) -> N
 def random_tensors(cfg: LayeredConfig, seed: int = 0, device="cpu") -> dict[str, torch.Tensor]:
     """Random weights with the magnitudes of a trained model: unit-variance activations through every product."""
     g = torch.Generator(device=device).manual_seed(seed)
+    stream = ("norm", "norm1", "norm2")              # norms of the residual stream; the others are plain factors
     out = {}
     for n, s in tensor_shapes(cfg).items():
         z = torch.randn(s, generator=g, device=device)
-        if n.endswith((".dq.norm", ".dkv.norm", ".mix.norm")):
-            t = 1.0 + 0.1 * z                    # plain norm weights
-        elif n.endswith("norm") or n.endswith("norm1"):
-            t = 0.1 * z                          # stored around zero
-        elif n.endswith(".A_log"):
+        last = n.rsplit(".", 1)[-1]
+        if last in stream:
+            of_stream = n in ("embed.norm", "final.norm") or n.count(".") == 1
+            t = (1.0 - cfg.design.norm_offset if of_stream else 1.0) + 0.1 * z
+        elif last == "A_log":
             t = 0.5 * z - 2.0
-        elif n.endswith(".dt_bias"):
+        elif last in ("dt_bias", "b") and len(s) == 1:
             t = 0.5 * z
-        elif n.endswith(".conv"):
-            t = z / math.sqrt(s[1])
-        elif n == "embed":
+        elif last == "D":
+            t = 1.0 + 0.1 * z
+        elif n == "embed" and not cfg.design.tied_head or n == "side.embed":
             t = z
         else:
             t = z / math.sqrt(s[1])
@@ -385,36 +683,102 @@ class LatentWeights:
 
 
 @dataclass
+class AttentionWeights:
+    spec: AttentionSpec
+    q_norm: torch.Tensor
+    k_norm: torch.Tensor
+    freq: torch.Tensor               # fp32 [pairs] radians per position
+    rot_mult: float                  # factor on cosine and sine
+    q_off: int
+    k_off: int
+    out_scale: float = 1.0
+
+
+@dataclass
+class GatedLinearWeights:
+    spec: GatedLinearSpec
+    low: wq_pack.PackedWeight        # decay logits from the inner columns
+    bias: torch.Tensor
+    norm_w: torch.Tensor             # times what the mixer's output is scaled by
+    q_off: int
+    k_off: int
+    v_off: int
+    g_off: int
+    a_off: int
+
+
+@dataclass
+class SsdWeights:
+    spec: SsdSpec
+    conv_w: torch.Tensor             # fp32 [taps, conv_width], channels x | B | C
+    conv_b: torch.Tensor
+    a_log: torch.Tensor
+    dt_bias: torch.Tensor
+    d: torch.Tensor
+    norm_w: torch.Tensor
+    z_off: int
+    x_off: int
+    dt_off: int
+
+
+@dataclass
+class PairWeights:
+    spec: PairSpec
+    left: object
+    right: object
+
+
+@dataclass
+class SideWeights:
+    """A layer's input from the token's side embedding."""
+    gate: torch.Tensor               # bf16 [dim, W rounded up]
+    proj: wq_pack.PackedWeight
+    norm_w: torch.Tensor
+    col: int                         # first column of the layer's part of the side embedding
+
+
+@dataclass
 class LayerWeights:
-    norm: torch.Tensor               # fp32 factor 1 + w
-    proj: wq_pack.PackedWeight       # [mixer inputs | feed-forward up]
+    norm: torch.Tensor               # fp32 factor of the norm
+    proj: wq_pack.PackedWeight       # mixer inputs; parallel layers: [mixer inputs | feed-forward up]
     split: int                       # mixer columns
     ff: int
-    mixer: object                    # DeltaWeights | LatentWeights
-    out: wq_pack.PackedWeight        # [o | down]
-    out_off: int                     # first feed-forward column of ``out``'s input
+    mixer: object                    # DeltaWeights | LatentWeights | SsdWeights | PairWeights
+    out: wq_pack.PackedWeight        # mixer output; parallel layers: [o | down]
+    out_off: int                     # parallel layers: first feed-forward column of ``out``'s input
+    norm2: torch.Tensor | None = None            # sequential layers: the feed-forward's norm, products and width of its activation
+    gate_up: wq_pack.PackedWeight | None = None  # rows in the order of the fused gated activation
+    down: wq_pack.PackedWeight | None = None
+    side: SideWeights | None = None
+
+    def matrices(self) -> list[wq_pack.PackedWeight]:
+        """Every packed matrix of the layer."""
+        out = [self.proj, self.out]
+        for part in ((self.mixer.left, self.mixer.right) if isinstance(self.mixer, PairWeights) else (self.mixer,)):
+            if isinstance(part, LatentWeights):
+                out += [part.uq, part.absorb.w, part.value.w]
+            elif getattr(part, "low", None) is not None:
+                out.append(part.low)
+        out += [m for m in (self.gate_up, self.down) if m is not None]
+        return out + ([self.side.proj] if self.side is not None else [])
 
 
 @dataclass
 class LayeredWeights:
     embed: torch.Tensor
-    embed_norm: torch.Tensor
+    embed_norm: torch.Tensor | None
     loop_in: wq_pack.PackedWeight | None
     layers: list[LayerWeights]
     final_norm: torch.Tensor
     lm_head: wq_pack.PackedWeight
+    side_embed: torch.Tensor | None = None
     vocab_start: int = 0
 
     def nbytes(self) -> int:
         total = self.embed.numel() * 2 + self.lm_head.nbytes + (self.loop_in.nbytes if self.loop_in else 0)
-        for l in self.layers:
-            total += l.proj.nbytes + l.out.nbytes
-            m = l.mixer
-            if isinstance(m, LatentWeights):
-                total += m.uq.nbytes + m.absorb.w.nbytes + m.value.w.nbytes
-            elif m.low is not None:
-                total += m.low.nbytes
-        return total
+        if self.side_embed is not None:
+            total += self.side_embed.numel() * 2 + sum(l.side.gate.numel() * 2 for l in self.layers)
+        return total + sum(m.nbytes for l in self.layers for m in l.matrices())
 
 
 class _Rows:
@@ -442,71 +806,137 @@ class _Rows:
         return torch.cat(self.parts)
 
 
+def _f32(get, n: str) -> torch.Tensor:
+    return get(n).float().contiguous()
+
+
+def _pack_delta(m: DeltaSpec, p: str, rows: _Rows, get) -> DeltaWeights:
+    rows.add(get(f"{p}.q"), get(f"{p}.k"), get(f"{p}.v"))
+    b_off = rows.add(get(f"{p}.b"))
+    conv = torch.cat([get(f"{p}.{t}.conv") for t in "qkv"]).float()
+    conv_w = torch.zeros(m.conv, m.conv_width, device=conv.device)
+    conv_w[:, :m.channels] = conv.t()
+    common = dict(spec=m, conv_w=conv_w.contiguous(), a_log=_f32(get, f"{p}.A_log"), dt_bias=_f32(get, f"{p}.dt_bias"),
+                  norm_w=_f32(get, f"{p}.norm"), b_off=b_off)
+    if not m.per_channel:
+        a_off = rows.add(get(f"{p}.a"))
+        return DeltaWeights(**common, a_off=a_off, z_off=rows.add(get(f"{p}.g")))
+    inner = round_up(m.decay_rank + m.gate_rank, 64)
+    a_off = rows.add(get(f"{p}.a1"), get(f"{p}.g1"), align=64, size=inner)
+    low_z = round_up(m.heads * m.dim, 8)
+    low = torch.zeros(low_z + m.heads * m.vdim, inner, dtype=torch.bfloat16, device=conv.device)
+    low[:m.heads * m.dim, :m.decay_rank] = get(f"{p}.a2")
+    low[low_z:, m.decay_rank:m.decay_rank + m.gate_rank] = get(f"{p}.g2")
+    return DeltaWeights(**common, a_off=a_off, z_off=0, low=wq_pack.pack_bf16(low), low_z=low_z)
+
+
+def _pack_latent(m: LatentSpec, p: str, rows: _Rows, get) -> LatentWeights:
+    H, d, e, R, Rp = m.heads, m.dim, m.vdim, m.kv_rank, m.rank_padded
+    rows.add(get(f"{p}.dq"))
+    c_off = rows.add(get(f"{p}.dkv"))
+    g_off = rows.add(get(f"{p}.g"))
+    uk = torch.zeros(H, Rp, d, dtype=torch.bfloat16, device=get(f"{p}.uk").device)
+    uk[:, :R] = get(f"{p}.uk").view(H, d, R).transpose(1, 2)
+    absorb = BlockDiagonal.pack(uk)
+    uv = torch.zeros(H, e, Rp, dtype=torch.bfloat16, device=uk.device)
+    uv[:, :, :R] = get(f"{p}.uv").view(H, e, R)
+    # the query projection writes every head where its block of ``absorb`` reads it
+    hp, kg = absorb.heads, absorb.w.k
+    uq = torch.zeros(-(-H // hp) * kg, m.q_rank, dtype=torch.bfloat16, device=uk.device)
+    src = get(f"{p}.uq").view(H, d, m.q_rank)
+    for h in range(H):
+        c = (h // hp) * kg + (h % hp) * d
+        uq[c:c + d] = src[h]
+    return LatentWeights(m, _f32(get, f"{p}.dq.norm"), _f32(get, f"{p}.dkv.norm"), _matrix(uq), absorb, BlockDiagonal.pack(uv),
+                         c_off, g_off)
+
+
+def _pack_attention(m: AttentionSpec, p: str, rows: _Rows, get, out_scale: float = 1.0) -> AttentionWeights:
+    q_off = rows.add(get(f"{p}.q"))
+    k_off = rows.add(get(f"{p}.k"))
+    freq, mult = m.rotary.table()
+    q_norm = _f32(get, f"{p}.q.norm")
+    return AttentionWeights(m, q_norm, _f32(get, f"{p}.k.norm"), freq.to(q_norm.device).contiguous(), mult, q_off, k_off, out_scale)
+
+
+def _pack_gated_linear(m: GatedLinearSpec, p: str, rows: _Rows, get, out_scale: float = 1.0) -> GatedLinearWeights:
+    q_off, k_off, v_off, g_off = (rows.add(get(f"{p}.{t}")) for t in "qkvg")
+    inner = round_up(m.decay_rank, 64)
+    a_off = rows.add(get(f"{p}.a1"), align=64, size=inner)
+    return GatedLinearWeights(m, _matrix(get(f"{p}.a2").to(torch.bfloat16)), _f32(get, f"{p}.a2.b"),
+                              out_scale * _f32(get, f"{p}.norm"), q_off, k_off, v_off, g_off, a_off)
+
+
+def _pack_ssd(m: SsdSpec, p: str, rows: _Rows, get) -> SsdWeights:
+    z, x, dt = get(f"{p}.in").split([m.out_width, m.channels, m.heads])
+    z_off, x_off, dt_off = rows.add(z), rows.add(x), rows.add(dt)
+    conv_w = torch.zeros(m.conv, m.conv_width, device=x.device)
+    conv_w[:, :m.channels] = get(f"{p}.conv").float().t()
+    conv_b = torch.zeros(m.conv_width, device=x.device)
+    conv_b[:m.channels] = get(f"{p}.conv.b").float()
+    return SsdWeights(m, conv_w, conv_b, *(_f32(get, f"{p}.{t}") for t in ("A_log", "dt_bias", "D", "norm")), z_off, x_off, dt_off)
+
+
+def _pack_pair(m: PairSpec, p: str, rows: _Rows, get) -> PairWeights:
+    return PairWeights(m, _PACKERS[type(m.left)](m.left, f"{p}.left", rows, get, out_scale=m.left_scale),
+                       _PACKERS[type(m.right)](m.right, f"{p}.right", rows, get, out_scale=m.right_scale))
+
+
+_PACKERS = {DeltaSpec: _pack_delta, LatentSpec: _pack_latent, AttentionSpec: _pack_attention, GatedLinearSpec: _pack_gated_linear,
+            SsdSpec: _pack_ssd, PairSpec: _pack_pair}
+
+
+def _pack_output(m: MixerSpec, p: str, get, ff: int, W: int) -> tuple[torch.Tensor, int]:
+    """Output projections side by side, with room for ``ff`` feed-forward columns: (matrix, first of those columns)."""
+    off = round_up(m.out_width, 8)
+    parts = ((m.left, f"{p}.left", 0), (m.right, f"{p}.right", m.right_off)) if isinstance(m, PairSpec) else ((m, p, 0),)
+    out = torch.zeros(W, round_up(off + ff, 64), dtype=torch.bfloat16, device=get(f"{parts[0][1]}.o").device)
+    for part, prefix, col in parts:
+        out[:, col:col + part.out_width] = get(f"{prefix}.o")
+    return out, off
+
+
+def _pack_glu(gate: torch.Tensor, up: torch.Tensor) -> wq_pack.PackedWeight:
+    """[gate ; up] in the row order of the GEMM's gated activation; the width is padded to whole blocks of it."""
+    ff, k = gate.shape
+    both = torch.zeros(2, round_up(ff, 16), k, dtype=torch.bfloat16, device=gate.device)
+    both[0, :ff], both[1, :ff] = gate, up
+    return wq_pack.swiglu_interleave(_matrix(both.flatten(0, 1)))
+
+
 def pack_layer(cfg: LayeredConfig, i: int, get) -> LayerWeights:
     """``get(name)`` -> tensor on the target device."""
-    l, p = cfg.layers[i], f"l{i}.mix"
-    W, m = cfg.hidden_size, l.mixer
-
-    def f32(n):
-        return get(n).float().contiguous()
-
+    l, p, W, d = cfg.layers[i], f"l{i}", cfg.hidden_size, cfg.design
     rows = _Rows(W)
-    if isinstance(m, DeltaSpec):
-        rows.add(get(f"{p}.q"), get(f"{p}.k"), get(f"{p}.v"))
-        b_off = rows.add(get(f"{p}.b"))
-        conv = torch.cat([get(f"{p}.{t}.conv") for t in "qkv"]).float()
-        conv_w = torch.zeros(m.conv, m.conv_width, device=conv.device)
-        conv_w[:, :m.channels] = conv.t()
-        common = dict(spec=m, conv_w=conv_w.contiguous(), a_log=f32(f"{p}.A_log"), dt_bias=f32(f"{p}.dt_bias"),
-                      norm_w=f32(f"{p}.norm"), b_off=b_off)
-        if m.per_channel:
-            inner = round_up(m.decay_rank + m.gate_rank, 64)
-            a_off = rows.add(get(f"{p}.a1"), get(f"{p}.g1"), align=64, size=inner)
-            low_z = round_up(m.heads * m.dim, 8)
-            low = torch.zeros(low_z + m.heads * m.vdim, inner, dtype=torch.bfloat16, device=conv.device)
-            low[:m.heads * m.dim, :m.decay_rank] = get(f"{p}.a2")
-            low[low_z:, m.decay_rank:m.decay_rank + m.gate_rank] = get(f"{p}.g2")
-            mixer = DeltaWeights(**common, a_off=a_off, z_off=0, low=wq_pack.pack_bf16(low), low_z=low_z)
-        else:
-            a_off = rows.add(get(f"{p}.a"))
-            z_off = rows.add(get(f"{p}.g"))
-            mixer = DeltaWeights(**common, a_off=a_off, z_off=z_off)
-    else:
-        H, d, e, R, Rp = m.heads, m.dim, m.vdim, m.kv_rank, m.rank_padded
-        rows.add(get(f"{p}.dq"))
-        c_off = rows.add(get(f"{p}.dkv"))
-        g_off = rows.add(get(f"{p}.g"))
-        uk = torch.zeros(H, Rp, d, dtype=torch.bfloat16, device=get(f"{p}.uk").device)
-        uk[:, :R] = get(f"{p}.uk").view(H, d, R).transpose(1, 2)
-        absorb = BlockDiagonal.pack(uk)
-        uv = torch.zeros(H, e, Rp, dtype=torch.bfloat16, device=uk.device)
-        uv[:, :, :R] = get(f"{p}.uv").view(H, e, R)
-        # the query projection writes every head where its block of ``absorb`` reads it
-        hp, kg = absorb.heads, absorb.w.k
-        uq = torch.zeros(-(-H // hp) * kg, m.q_rank, dtype=torch.bfloat16, device=uk.device)
-        src = get(f"{p}.uq").view(H, d, m.q_rank)
-        for h in range(H):
-            c = (h // hp) * kg + (h % hp) * d
-            uq[c:c + d] = src[h]
-        mixer = LatentWeights(m, f32(f"{p}.dq.norm"), f32(f"{p}.dkv.norm"), _matrix(uq), absorb, BlockDiagonal.pack(uv),
-                              c_off, g_off)
-    mixer_rows = rows.end()
-    split = mixer_rows.shape[0]
-    out_off = round_up(m.out_width, 8)
-    out = torch.zeros(W, round_up(out_off + l.ff, 64), dtype=torch.bfloat16, device=mixer_rows.device)
-    out[:, :m.out_width] = get(f"{p}.o")
-    if l.ff:
-        mixer_rows = torch.cat([mixer_rows, get(f"l{i}.mlp.up").to(torch.bfloat16)])
-        out[:, out_off:out_off + l.ff] = get(f"l{i}.mlp.down")
-    return LayerWeights(1.0 + f32(f"l{i}.norm1"), _matrix(mixer_rows), split, l.ff, mixer, wq_pack.pack_bf16(out), out_off)
+    mixer = _PACKERS[type(l.mixer)](l.mixer, f"{p}.mix", rows, get)
+    proj = rows.end()
+    split = proj.shape[0]
+    joint = l.ff if not d.sequential else 0
+    out, out_off = _pack_output(l.mixer, f"{p}.mix", get, joint, W)
+    if joint:
+        proj = torch.cat([proj, get(f"{p}.mlp.up").to(torch.bfloat16)])
+        out[:, out_off:out_off + l.ff] = get(f"{p}.mlp.down")
+    lw = LayerWeights(d.norm_offset + _f32(get, f"{p}.norm1"), _matrix(proj), split, joint, mixer, wq_pack.pack_bf16(out), out_off)
+    if d.sequential and l.ff:
+        lw.norm2 = d.norm_offset + _f32(get, f"{p}.norm2")
+        lw.gate_up = _pack_glu(get(f"{p}.mlp.gate"), get(f"{p}.mlp.up"))
+        lw.down = _matrix(get(f"{p}.mlp.down").to(torch.bfloat16))
+    if cfg.side_dim:
+        gate = get(f"{p}.side.gate").to(torch.bfloat16)
+        lw.side = SideWeights(_pad(gate, gate.shape[0], round_up(W, 64)), _matrix(get(f"{p}.side.proj").to(torch.bfloat16)),
+                              _f32(get, f"{p}.side.norm"), i * cfg.side_dim)
+    return lw
 
 
 def pack_weights(cfg: LayeredConfig, get) -> LayeredWeights:
+    d = cfg.design
+    embed = get("embed").to(torch.bfloat16).contiguous()
     return LayeredWeights(
-        embed=get("embed").to(torch.bfloat16).contiguous(), embed_norm=1.0 + get("embed.norm").float(),
+        embed=embed, embed_norm=d.norm_offset + get("embed.norm").float() if d.embed_norm else None,
         loop_in=_matrix(get("loop.in")) if cfg.loop is not None else None,
         layers=[pack_layer(cfg, i, get) for i in range(cfg.num_layers)],
-        final_norm=1.0 + get("final.norm").float(), lm_head=_matrix(get("head")))
+        final_norm=d.norm_offset + get("final.norm").float(), lm_head=_matrix(embed if d.tied_head else get("head")),
+        side_embed=get("side.embed").to(torch.bfloat16).contiguous() if cfg.side_dim else None)
 
 
 def random_layered_weights(cfg: LayeredConfig, device="cuda", seed: int = 0, *_, **__) -> LayeredWeights:

@@ -1,14 +1,20 @@
 """Layered decoders on the native sm_100a kernels.
 
 ``LayeredRunner`` is the model body of ``models/layered.py`` checkpoints: it owns the packed weights, fixed-address
-buffers, one paged latent cache per attention run and the per-request state of every delta run, and serves the executor
+buffers, one paged cache per attention run and the per-request state of every recurrent run, and serves the executor
 through the same surface as ``DecoderRunner`` (``forward_hidden`` / ``forward_logits`` / ``run_step``, all capturable in a
-CUDA graph).  A layer run is
+CUDA graph).  A run of a parallel layer is
 
     norm(x) -> h                          fp32 residual in, activation type out
     [mixer inputs | relu^2(up)] = h W     one product; the up columns leave as the right half of the output's operand
     mixer -> left half of that operand
     x += [o | relu^2(up)] [W_o | W_down]  one product, accumulated into the fp32 residual
+
+and a sequential layer, whose h comes from the step before it,
+
+    mixer inputs = h W;  mixer -> operand;  x += operand W_o
+    norm2(x) -> h;  act = gelu(h W_gate) (h W_up), one product;  x += act W_down
+    side = gelu(x W_side) e, one kernel;  y = side W_proj;  x += norm(y) and h = norm1 of the next layer, one kernel
 
 ``cfg.dtype`` "float32" runs the same steps with fp32 activations and fp32 products.
 """
@@ -17,21 +23,30 @@ from __future__ import annotations
 import torch
 
 from ..ops import kernels as K
-from .layered import DeltaWeights, LatentWeights, LayeredConfig, LayeredWeights, round_up
+from .layered import (AttentionWeights, DeltaWeights, GatedLinearWeights, LatentWeights, LayeredConfig, LayeredWeights, PairWeights,
+                      SsdWeights, round_up)
 from .step_runner import StepRunner
 
 
-class _DeltaRun:
-    """Per-request state of one run of a delta layer: convolution history (activation type) and delta-rule state (fp32)."""
+class _StateRun:
+    """Per-request state of one run of a recurrent layer: recurrence state (fp32) and, with a convolution, its last inputs
+    (activation type)."""
 
-    def __init__(self, spec, rows: int, act: torch.dtype, device) -> None:
+    def __init__(self, rows: int, heads: int, vdim: int, stride: int, device, taps: int = 0, conv_width: int = 0,
+                 act: torch.dtype = torch.bfloat16) -> None:
         # a row is a multiple of 16 bytes (whole-row copies); the history's layout inside it is [taps - 1, channels]
-        self.conv = torch.zeros(rows, max(1, spec.conv - 1), spec.conv_width, dtype=act, device=device)
-        self.state = torch.zeros(rows, spec.heads, spec.vdim, spec.state_stride, dtype=torch.float32, device=device)
+        self.conv = torch.zeros(rows, max(1, taps - 1), conv_width, dtype=act, device=device) if taps else None
+        self.state = torch.zeros(rows, heads, vdim, stride, dtype=torch.float32, device=device)
 
     def copy(self, src, dst) -> None:
-        K.copy_rows(self.conv, src, dst)
+        if self.conv is not None:
+            K.copy_rows(self.conv, src, dst)
         K.copy_rows(self.state, src, dst)
+
+
+def _parts(m) -> tuple:
+    """The mixers a layer's weights consist of."""
+    return (m.left, m.right) if isinstance(m, PairWeights) else (m,)
 
 
 class LayeredRunner(StepRunner):
@@ -48,6 +63,7 @@ class LayeredRunner(StepRunner):
         self.act = act = torch.float32 if cfg.dtype == "float32" else torch.bfloat16
         self.logits_dtype = act
         self.ws = K.workspace(dev)
+        self.sequential = cfg.design.sequential
         T, W = max_tokens, cfg.hidden_size
 
         def buf(cols: int, dtype=act) -> torch.Tensor:
@@ -58,37 +74,59 @@ class LayeredRunner(StepRunner):
         self.x0 = buf(W, torch.float32) if cfg.loop is not None else None
         self.h = buf(round_up(W, 64))
         self.entry = buf(round_up(2 * W, 64)) if cfg.loop is not None else None
-        self.runs = []                         # per layer run: _DeltaRun or the latent cache of the run
-        self.kv = []                           # latent caches (copied page by page on copy-on-write)
-        for i, _ in cfg.runs:
-            m = cfg.layers[i].mixer
-            if isinstance(weights.layers[i].mixer, DeltaWeights):
-                self.runs.append(_DeltaRun(m, max_requests + state_checkpoints, act, dev))
-            else:
-                self.runs.append(torch.zeros(num_pages, 16, m.rank_padded, dtype=act, device=dev))
-                self.kv.append(self.runs[-1])
-        # operands of the output products ([mixer output | feed-forward]) by layout, scratch by width: layers share them
+        self.side = buf(round_up(cfg.side_dim, 64)) if cfg.side_dim else None
+        self.side_y = buf(round_up(W, 8)) if cfg.side_dim else None
+        self.kv = []                           # paged caches (copied page by page on copy-on-write)
+        self.states = []                       # recurrent states (copied row by row)
+        # per layer run: the cache or state of every mixer it consists of
+        self.runs = [tuple(self._store(p) for p in _parts(weights.layers[i].mixer)) for i, _ in cfg.runs]
+        # operands of the products by layout, scratch by width: layers share them
         self._operands: dict = {}
         self._scratch: dict = {}
-        delta = []
+        recurrent = []
         for l in weights.layers:
-            key = (l.mixer.spec.out_width, l.out_off, l.ff, l.out.k)
-            self._operands.setdefault(key, buf(l.out.k))
+            self._operands.setdefault(self._layout(l), buf(l.out.k))
             self._need("proj", l.split)
-            if isinstance(l.mixer, DeltaWeights):
-                m = l.mixer.spec
-                delta.append((m.heads, m.kv_heads, m.dim, m.vdim, m.per_channel))
-                if l.mixer.low is not None:
-                    self._need("low", l.mixer.low.n)
-            else:
-                m, mw = l.mixer.spec, l.mixer
-                self._need("cq%d" % m.q_rank, round_up(m.q_rank, 64))
-                self._need("q", mw.uq.n)
-                self._need("ql", m.heads * m.rank_padded)
-                self._need("ol", m.heads * m.rank_padded)
+            if l.down is not None:
+                self._operands.setdefault(("act", l.gate_up.n, l.down.k), buf(l.down.k))
+            for m in _parts(l.mixer):
+                s = m.spec
+                if isinstance(m, LatentWeights):
+                    self._need("cq%d" % s.q_rank, round_up(s.q_rank, 64))
+                    self._need("q", m.uq.n)
+                    self._need("ql", s.heads * s.rank_padded)
+                    self._need("ol", s.heads * s.rank_padded)
+                elif isinstance(m, AttentionWeights):
+                    self._need("q", s.heads * s.width_padded)
+                else:
+                    if isinstance(m, DeltaWeights):
+                        recurrent.append((s.heads, s.kv_heads, s.dim, s.vdim, s.per_channel))
+                    elif isinstance(m, SsdWeights):
+                        recurrent.append((s.heads, s.groups, s.state, s.vdim, False))
+                    else:
+                        recurrent.append((s.heads, s.heads, s.dim, s.vdim, True))
+                    if getattr(m, "low", None) is not None:
+                        self._need("low", m.low.n)
         self._scratch = {n: torch.zeros(T * c, dtype=act, device=dev) for n, c in self._scratch.items()}
-        self.delta = K.DeltaScratch(T, delta, act, dev) if delta else None
+        self.recurrence = K.RecurrenceScratch(T, recurrent, act, dev) if recurrent else None
         self.trace: list | None = None         # a list here receives a copy of the residual after every layer run
+
+    def _store(self, m):
+        """Cache or state of one run of a mixer."""
+        s, dev, rows = m.spec, self.device, self.max_requests + len(self.state_checkpoint_rows)
+        if isinstance(m, LatentWeights):
+            self.kv.append(torch.zeros(self.num_pages, 16, s.rank_padded, dtype=self.act, device=dev))
+            return self.kv[-1]
+        if isinstance(m, AttentionWeights):
+            self.kv.append(torch.zeros(self.num_pages, s.kv_heads, 2, 16, s.width_padded, dtype=self.act, device=dev))
+            return self.kv[-1]
+        conv = {} if isinstance(m, GatedLinearWeights) else dict(taps=s.conv, conv_width=s.conv_width, act=self.act)
+        self.states.append(_StateRun(rows, s.heads, s.vdim, s.state_stride, dev, **conv))
+        return self.states[-1]
+
+    def _layout(self, l) -> tuple:
+        """What an operand of a layer's output product is shared by: every column keeps its role."""
+        return (*(m.spec.out_width for m in _parts(l.mixer)), l.out_off, l.ff, l.out.k)
 
     def _need(self, name: str, cols: int) -> None:
         self._scratch[name] = max(self._scratch.get(name, 0), cols)
@@ -97,16 +135,18 @@ class LayeredRunner(StepRunner):
         return self._scratch[name][:T * cols].view(T, cols)
 
     def copy_state(self, src: torch.Tensor, dst: torch.Tensor) -> None:
-        """Whole recurrent-state rows ``src[i] -> dst[i]`` of every delta run."""
-        for r in self.runs:
-            if isinstance(r, _DeltaRun):
-                r.copy(src, dst)
+        """Whole recurrent-state rows ``src[i] -> dst[i]`` of every recurrent run."""
+        for r in self.states:
+            r.copy(src, dst)
 
     # ---------------------------------------------------------------- forward
     def forward_hidden(self, b) -> torch.Tensor:
-        cfg, w, T = self.cfg, self.w, b.num_tokens
         if b.segments is None:
             raise RuntimeError("layered decoders need the step's request segments (StepBatch.segments)")
+        return self._sequential(b) if self.sequential else self._parallel(b)
+
+    def _parallel(self, b) -> torch.Tensor:
+        cfg, w, T = self.cfg, self.w, b.num_tokens
         decode = T == b.segments.num           # every segment has at most one row
         x, x0, h = self.x[:T], None if self.x0 is None else self.x0[:T], self.h[:T]
         K.embed_norm(b.token_ids[:T], w.embed, w.embed_norm, x, cfg.rms_eps, x0)
@@ -119,21 +159,64 @@ class LayeredRunner(StepRunner):
                 K.wide_gemm(entry, w.loop_in, x, ws=self.ws)
                 n += 2
             K.row_norm(x, l.norm, h, cfg.rms_eps)
-            m = l.mixer
-            operand = self._operands[(m.spec.out_width, l.out_off, l.ff, l.out.k)][:T]
+            operand = self._operands[self._layout(l)][:T]
             proj = self._rows("proj", T, l.split)
             up = operand[:, l.out_off:l.out_off + l.ff] if l.ff else None
             K.wide_gemm(h, l.proj, proj, relu2=up, split=l.split, ws=self.ws)
-            mixed = operand[:, :m.spec.out_width]
-            n += 3 + (self._delta(m, proj, run, b, mixed, decode) if isinstance(m, DeltaWeights)
-                      else self._latent(m, proj, run, b, mixed, decode))
+            n += 3 + self._mix(l.mixer, proj, run, b, operand, decode)
             K.wide_gemm(operand, l.out, x, residual=x, ws=self.ws)
-            if self.trace is not None:
-                self.trace.append(x.clone())
+            self._after_layer(x)
         self.launches_per_step = n
         return x
 
-    def _delta(self, m: DeltaWeights, proj, run: _DeltaRun, b, out, decode: bool) -> int:
+    def _sequential(self, b) -> torch.Tensor:
+        cfg, w, T, eps = self.cfg, self.w, b.num_tokens, self.cfg.rms_eps
+        decode = T == b.segments.num
+        x, h = self.x[:T], self.h[:T]
+        K.embed_rows(b.token_ids[:T], w.embed, w.layers[0].norm, x, h, eps)
+        n, last = 1, len(w.layers) - 1
+        for i, (l, run) in enumerate(zip(w.layers, self.runs)):
+            operand, proj = self._operands[self._layout(l)][:T], self._rows("proj", T, l.split)
+            K.wide_gemm(h, l.proj, proj, ws=self.ws)
+            n += 2 + self._mix(l.mixer, proj, run, b, operand, decode)
+            K.wide_gemm(operand, l.out, x, residual=x, ws=self.ws)
+            if l.down is not None:
+                act = self._operands[("act", l.gate_up.n, l.down.k)][:T]
+                K.row_norm(x, l.norm2, h, eps)
+                K.wide_gemm(h, l.gate_up, act[:, :l.gate_up.n // 2], gelu_glu=True, ws=self.ws)
+                K.wide_gemm(act, l.down, x, residual=x, ws=self.ws)
+                n += 3
+            follow = None if i == last else w.layers[i + 1].norm       # the final norm reads the wanted rows only
+            if l.side is not None:
+                g, y = self.side[:T], self.side_y[:T, :cfg.hidden_size]
+                K.side_gate(x, l.side.gate, b.token_ids[:T], w.side_embed, l.side.col, g)
+                K.wide_gemm(g, l.side.proj, y, ws=self.ws)
+                K.add_norm_rows(y, l.side.norm_w, x, eps, follow, None if follow is None else h)
+                n += 3
+            elif follow is not None:
+                K.row_norm(x, follow, h, eps)
+                n += 1
+            self._after_layer(x)
+        self.launches_per_step = n
+        return x
+
+    def _after_layer(self, x: torch.Tensor) -> None:
+        if self.trace is not None:
+            self.trace.append(x.clone())
+
+    # ---------------------------------------------------------------- mixers: columns of ``proj`` -> columns of the operand
+    def _mix(self, m, proj, run, b, operand, decode: bool) -> int:
+        """Runs a layer's mixer; returns the launches made."""
+        if isinstance(m, PairWeights):
+            off = (0, m.spec.right_off)
+            return sum(self._one(p, proj, store, b, operand[:, c:c + p.spec.out_width], decode)
+                       for p, store, c in zip(_parts(m), run, off))
+        return self._one(m, proj, run[0], b, operand[:, :m.spec.out_width], decode)
+
+    def _one(self, m, proj, store, b, out, decode: bool) -> int:
+        return _MIXERS[type(m)](self, m, proj, store, b, out, decode)
+
+    def _delta(self, m: DeltaWeights, proj, run: _StateRun, b, out, decode: bool) -> int:
         s, T = m.spec, proj.shape[0]
         n = 1
         if m.low is not None:
@@ -144,8 +227,8 @@ class LayeredRunner(StepRunner):
         else:
             a, z = proj[:, m.a_off:m.a_off + s.heads], proj[:, m.z_off:m.z_off + s.out_width]
         K.delta_prepare(proj[:, :s.conv_width], proj[:, m.b_off:m.b_off + s.heads], a, m.conv_w, run.conv, m.a_log, m.dt_bias,
-                        b.segments, self.delta, s.heads, s.kv_heads, s.dim, s.vdim)
-        return n + K.delta_walk(z, m.norm_w, run.state, b.segments, out, self.delta, s.kv_heads, s.dim, self.cfg.rms_eps,
+                        b.segments, self.recurrence, s.heads, s.kv_heads, s.dim, s.vdim)
+        return n + K.delta_walk(z, m.norm_w, run.state, b.segments, out, self.recurrence, s.kv_heads, s.dim, self.cfg.rms_eps,
                                 s.per_channel, s.per_channel, decode)
 
     def _latent(self, m: LatentWeights, proj, cache: torch.Tensor, b, out, decode: bool) -> int:
@@ -161,6 +244,30 @@ class LayeredRunner(StepRunner):
         K.wide_gemm(ol, m.value.w, out, diag_rows=m.value.rows, ws=self.ws)
         return 5
 
+    def _attention(self, m: AttentionWeights, proj, cache: torch.Tensor, b, out, decode: bool) -> int:
+        s, T = m.spec, proj.shape[0]
+        q = self._rows("q", T, s.heads * s.width_padded)
+        K.gqa_prepare(proj, m.q_off, m.k_off, m.q_norm, m.k_norm, m.freq, m.rot_mult, b.positions[:T], b.slots[:T], q, cache, s.heads,
+                      s.dim, self.cfg.rms_eps)
+        return 1 + K.gqa_attention(q, cache, b.page_table, b.segments, out, s.heads, s.dim, s.window, s.scale, s.sink, m.out_scale,
+                                   decode=decode, ws=self.ws)
+
+    def _gated_linear(self, m: GatedLinearWeights, proj, run: _StateRun, b, out, decode: bool) -> int:
+        s, T = m.spec, proj.shape[0]
+        a = self._rows("low", T, m.low.n)
+        K.wide_gemm(proj[:, m.a_off:m.a_off + m.low.k], m.low, a, ws=self.ws)
+        K.gated_linear_prepare(proj, m.q_off, m.k_off, m.v_off, a, m.bias, 1.0 / s.tau, b.segments, self.recurrence, s.heads, s.dim,
+                               s.vdim)
+        return 2 + K.gated_linear_walk(proj[:, m.g_off:m.g_off + s.out_width], m.norm_w, run.state, b.segments, out, self.recurrence,
+                                       s.dim, self.cfg.rms_eps, decode)
+
+    def _ssd(self, m: SsdWeights, proj, run: _StateRun, b, out, decode: bool) -> int:
+        s = m.spec
+        K.ssd_prepare(proj[:, m.x_off:m.x_off + s.conv_width], proj[:, m.dt_off:m.dt_off + s.heads], m.conv_w, m.conv_b, run.conv,
+                      m.a_log, m.dt_bias, b.segments, self.recurrence, s.heads, s.groups, s.state, s.vdim)
+        return 1 + K.ssd_walk(proj[:, m.z_off:m.z_off + s.out_width], m.d, m.norm_w, s.norm_groups, run.state, b.segments, out,
+                              self.recurrence, s.groups, s.state, self.cfg.rms_eps, decode)
+
     def forward_logits(self, b, hidden: torch.Tensor, logits_out: torch.Tensor) -> torch.Tensor:
         """Final norm and output head of the selected rows."""
         R = b.num_logit_rows
@@ -169,3 +276,7 @@ class LayeredRunner(StepRunner):
         K.wide_gemm(h, self.w.lm_head, logits_out[:R], ws=self.ws)
         self.launches_per_step += 2
         return logits_out[:R]
+
+
+_MIXERS = {DeltaWeights: LayeredRunner._delta, LatentWeights: LayeredRunner._latent, AttentionWeights: LayeredRunner._attention,
+           GatedLinearWeights: LayeredRunner._gated_linear, SsdWeights: LayeredRunner._ssd}

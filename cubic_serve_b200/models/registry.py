@@ -78,15 +78,16 @@ def _builtin() -> None:
 
     def runner_layered(cfg, weights, **kw):
         from .layered_runner import LayeredRunner
-        kw.pop("k_bits", None), kw.pop("v_bits", None)          # latents are cached in the activation type
+        kw.pop("k_bits", None), kw.pop("v_bits", None)          # latents, keys and values are cached in the activation type
         if kw.pop("kv_rotation", False):
-            raise ModelRegistryError("cache rotation applies to quantized key / value caches, not to cached latents")
+            raise ModelRegistryError("cache rotation applies to quantized key / value caches, not to those of layered decoders")
         return LayeredRunner(cfg, weights, **kw)
 
     register(ModelDefinition("layered", LAYERED, parse_config=parse_layered, random_weights=random_layered_weights,
                              load_weights=load_layered_weights, build_runner=runner_layered,
-                             description="parallel layers with a mixer each (delta rule per head or per channel, windowed "
-                                         "latent attention), optional loop over a run of layers, fp32 residual"))
+                             description="layers with a mixer each (delta rule per head or per channel, windowed latent "
+                                         "attention, state-space recurrence, sink attention beside gated linear attention), "
+                                         "parallel or sequential, loops, token side inputs, fp32 residual"))
 
     def parse_q4(path: Path):
         from .qwen4_exp import parse_qwen4_exp_config_json

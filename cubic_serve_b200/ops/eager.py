@@ -26,14 +26,15 @@ def swiglu(gate_up: torch.Tensor) -> torch.Tensor:
     return torch.nn.functional.silu(g) * u
 
 
-def rope_inv_freq(rotary_dim: int, theta: float, device=None, scaling: tuple | None = None) -> torch.Tensor:
+def rope_inv_freq(rotary_dim: int, theta: float, device=None, scaling: tuple | None = None,
+                  dtype: torch.dtype = torch.float32) -> torch.Tensor:
     """Rotary frequencies.  ``scaling`` (``ModelConfig.rope_scaling``): ``("linear", factor)`` divides every frequency;
     ``("llama3", factor, low_freq_factor, high_freq_factor, original_max_position)`` keeps wavelengths below
     ``original / high`` as they are, divides those above ``original / low`` by ``factor`` and blends in between;
     ``("yarn", factor, original_max_position, beta_fast, beta_slow, attention_factor)`` blends by slot index (its
     attention factor is a softmax scale, ``ModelConfig.attention_scale``).  All are static, so the kernels see them only
     as another frequency table."""
-    inv = 1.0 / (theta ** (torch.arange(0, rotary_dim, 2, device=device, dtype=torch.float32) / rotary_dim))
+    inv = 1.0 / (theta ** (torch.arange(0, rotary_dim, 2, device=device, dtype=dtype) / rotary_dim))
     if scaling is None:
         return inv
     if scaling[0] == "linear":
@@ -45,7 +46,7 @@ def rope_inv_freq(rotary_dim: int, theta: float, device=None, scaling: tuple | N
         blended = (1 - smooth) * inv / factor + smooth * inv
         return torch.where(wavelen < original / high, inv, torch.where(wavelen > original / low, inv / factor, blended))
     if scaling[0] == "factors":                # one divisor per slot, as stored by GGUF exporters (``rope_freqs.weight``)
-        div = torch.tensor(scaling[1], device=device, dtype=torch.float32)
+        div = torch.tensor(scaling[1], device=device, dtype=dtype)
         if div.numel() != inv.numel():
             raise ValueError("the rotary divisor table does not match the rotary width")
         return inv / div
@@ -57,9 +58,7 @@ def rope_inv_freq(rotary_dim: int, theta: float, device=None, scaling: tuple | N
         def slot(turns: float) -> float:
             return rotary_dim * math.log(original / (turns * 2 * math.pi)) / (2 * math.log(theta))
         low, high = max(math.floor(slot(beta_fast)), 0), min(math.ceil(slot(beta_slow)), rotary_dim - 1)
-        if low == high:
-            high += 0.001
-        ramp = ((torch.arange(rotary_dim // 2, device=device, dtype=torch.float32) - low) / (high - low)).clamp(0, 1)
+        ramp = ((torch.arange(rotary_dim // 2, device=device, dtype=dtype) - low) / max(high - low, 0.001)).clamp(0, 1)
         return inv / factor * ramp + inv * (1 - ramp)
     raise ValueError(f"unknown rotary scaling {scaling[0]!r}")
 

@@ -725,17 +725,19 @@ def _seg(seg: GdnSegments) -> "native.GdnSegmentsStruct":
 
 def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: torch.Tensor | None = None,
               relu2: torch.Tensor | None = None, split: int = 0, diag_rows: int = 0, ws: Workspace | None = None,
-              stream_k: bool | None = None, splits: int | None = None) -> None:
+              stream_k: bool | None = None, splits: int | None = None, gelu_glu: bool = False) -> None:
     """``x @ W^T`` with bf16-stored weights through the wide epilogue.
 
     ``x`` fp32: everything is fp32 (``csrc/layered.cu``); ``x`` bf16: tcgen05 with fp32 accumulation.  ``out`` gets the
     product; an fp32 ``out`` may be added to ``residual`` (the same tensor: in-place accumulation).  With ``relu2`` the
-    features from ``split`` on leave there as ``max(v, 0)^2`` and ``out`` holds the first ``split``.  ``diag_rows``:
+    features from ``split`` on leave there as ``max(v, 0)^2`` and ``out`` holds the first ``split``.  ``gelu_glu``: the rows
+    of ``w`` are interleaved [gate ; up] and ``out`` gets ``gelu_tanh(gate) * up`` (``N / 2`` columns).  ``diag_rows``:
     block-diagonal weights, see ``models/layered.py::BlockDiagonal``.  ``x`` may have fewer columns than ``w.k``: the rest
     read as zero."""
     m, k = x.shape[0], w.k
     assert w.fmt == FMT_BF16 and x.stride(1) == 1 and out.stride(1) == 1 and out.shape[0] == m
-    assert out.shape[1] == (split if relu2 is not None else w.n), (out.shape, split, w.n)
+    assert gelu_glu == w.act_interleaved and not (gelu_glu and (relu2 is not None or residual is not None or diag_rows))
+    assert out.shape[1] == (split if relu2 is not None else w.n // 2 if gelu_glu else w.n), (out.shape, split, w.n)
     assert residual is None or (residual.dtype == torch.float32 and residual.stride(0) == out.stride(0))
     if relu2 is not None:
         assert relu2.dtype == x.dtype and relu2.stride(1) == 1 and relu2.shape == (m, w.n - split) and split % 4 == 0
@@ -745,11 +747,12 @@ def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: tor
         assert out.dtype == torch.float32
         a = native.F32GemmStruct(x.data_ptr(), x.stride(0), x_cols, w.codes.data_ptr(), out.data_ptr(), out.stride(0),
                                  _ptr(residual), _ptr(relu2), 0 if relu2 is None else relu2.stride(0), split, diag_rows, m,
-                                 w.n, k)
+                                 w.n, k, 2 if gelu_glu else 0)
         native.check(l.cb_f32_gemm(ctypes.byref(a), _stream()), "cb_f32_gemm")
         return
     wide32 = out.dtype == torch.float32
     assert residual is None or wide32
+    assert not (gelu_glu and wide32)
     ws = ws or workspace(x.device)
     if stream_k is None:
         stream_k = splits is None and not diag_rows and use_stream_k(m, w.n, FMT_BF16, sm_count(x.device), k)
@@ -761,7 +764,7 @@ def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: tor
     a = native.WideGemmStruct(x.data_ptr(), x.stride(0), x_cols, w.codes.data_ptr(), None if wide32 else out.data_ptr(),
                               out.data_ptr() if wide32 else None, out.stride(0), _ptr(residual), _ptr(relu2),
                               0 if relu2 is None else relu2.stride(0), split, diag_rows, m, w.n, k, int(stream_k), splits,
-                              active().gemm.stream_k_min_units)
+                              active().gemm.stream_k_min_units, 2 if gelu_glu else 0)
     code = l.cb_bf16_gemm_wide(ctypes.byref(a), ws.gemm.data_ptr(), ws.gemm.numel(), ws.gemm_counters.data_ptr(),
                                ws.status.data_ptr(), _stream())
     native.check(code, "cb_bf16_gemm_wide")
@@ -790,9 +793,39 @@ def concat_rows(x: torch.Tensor, x0: torch.Tensor, out: torch.Tensor) -> None:
                                              x.shape[1], int(out.dtype == torch.float32), _stream()), "cb_concat_rows")
 
 
-class DeltaScratch:
-    """Fixed-address buffers between the preparation and the recurrence of delta layers, for up to ``max_tokens`` rows of the
-    largest layer they are made for (layers share them)."""
+def embed_rows(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, h: torch.Tensor, eps: float) -> None:
+    """``x`` = embedding rows (fp32), ``h = x / rms(x) * weight`` in ``h``'s type."""
+    assert x.dtype == weight.dtype == torch.float32 and x.is_contiguous() and table.dtype == torch.bfloat16 and h.stride(1) == 1
+    native.check(native.lib().cb_embed_rows(ids.data_ptr(), table.data_ptr(), weight.data_ptr(), x.data_ptr(), h.data_ptr(),
+                                            h.stride(0), x.shape[0], x.shape[1], table.shape[0], float(eps),
+                                            int(h.dtype == torch.float32), _stream()), "cb_embed_rows")
+
+
+def add_norm_rows(y: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, eps: float, next_weight: torch.Tensor | None = None,
+                  h: torch.Tensor | None = None) -> None:
+    """``x += y / rms(y) * weight`` on the fp32 residual; with ``h`` also ``h = x / rms(x) * next_weight``, the norm that reads
+    the residual next."""
+    assert x.dtype == weight.dtype == torch.float32 and x.is_contiguous() and y.stride(1) == 1 and y.shape[1] == x.shape[1]
+    assert h is None or h.dtype == y.dtype and h.stride(1) == 1 and next_weight.dtype == torch.float32
+    native.check(native.lib().cb_add_norm_rows(y.data_ptr(), y.stride(0), weight.data_ptr(), x.data_ptr(), _ptr(next_weight), _ptr(h),
+                                               0 if h is None else h.stride(0), x.shape[0], x.shape[1], float(eps),
+                                               int(y.dtype == torch.float32), _stream()), "cb_add_norm_rows")
+
+
+def side_gate(x: torch.Tensor, gate: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col: int, out: torch.Tensor) -> None:
+    """``out[t, n] = gelu_tanh(x[t] . gate[n]) * table[ids[t], col + n]``: the fp32 residual gates a token's side embedding.
+    ``gate`` bf16 ``[dim, columns >= W]`` with zeros behind the width; fp32 ``out``: everything is fp32."""
+    dim = gate.shape[0]
+    assert x.dtype == torch.float32 and x.is_contiguous() and gate.dtype == table.dtype == torch.bfloat16 and gate.is_contiguous()
+    assert out.stride(1) == 1 and out.shape[1] >= dim and out.shape[0] == x.shape[0]
+    native.check(native.lib().cb_side_gate(x.data_ptr(), x.shape[1], gate.data_ptr(), gate.shape[1], ids.data_ptr(), table.data_ptr(),
+                                           table.shape[1], col, out.data_ptr(), out.stride(0), x.shape[0], dim, table.shape[0],
+                                           int(out.dtype == torch.float32), _stream()), "cb_side_gate")
+
+
+class RecurrenceScratch:
+    """Fixed-address buffers between the preparation and the recurrence of recurrent layers, for up to ``max_tokens`` rows of
+    the largest layer they are made for (layers share them)."""
 
     def __init__(self, max_tokens: int, sizes, act: torch.dtype, device) -> None:
         """``sizes``: (heads, key heads, key width, value width, per channel) of every layer."""
@@ -808,49 +841,111 @@ class DeltaScratch:
         self.raw = torch.zeros(T * most(lambda H, G, d, e, c: H * e), **f32)
 
 
-def delta_prepare(x: torch.Tensor, b: torch.Tensor, a: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor,
-                  a_log: torch.Tensor, dt_bias: torch.Tensor, seg: GdnSegments, sc: DeltaScratch, heads: int, kv_heads: int,
-                  dim: int, vdim: int) -> None:
-    """Everything of a delta layer's tokens that does not depend on its state (``csrc/delta_rule.cu``): causal depthwise
-    convolution + SiLU of ``x [T, q | k | v]`` with ``conv_w`` fp32 ``[taps, channels]`` (the last row multiplies the current
-    input) and the requests' last inputs ``conv_state [slots, taps - 1, channels]``, which are read and replaced; unit q / k;
-    step sizes and decays from the logits ``b`` and ``a``."""
-    taps, ldw = conv_w.shape
-    channel = dt_bias.numel() != heads
-    assert conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_state.dtype == x.dtype == a.dtype == b.dtype
-    assert conv_state.is_contiguous() and (taps == 1 or tuple(conv_state.shape[1:]) == (taps - 1, ldw))
-    assert x.shape[1] == ldw and x.stride(1) == b.stride(1) == a.stride(1) == 1 and dt_bias.numel() in (heads, heads * dim)
-    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (a_log, dt_bias))
-    ds, es = -(-dim // 4) * 4, -(-vdim // 8) * 8
+def _prepare(entry: str, x, a, dt_bias, seg: GdnSegments, sc: RecurrenceScratch, heads: int, kv_heads: int, dim: int, vdim: int,
+             channel: bool, offs: tuple[int, int, int], conv=None, b=None, a_log=None, rate: float = 0.0) -> None:
+    """Preparation of a recurrence's tokens (``csrc/recurrence.cuh``).  ``offs``: columns of q, k and v in ``x``; ``conv``:
+    (weights fp32 [taps, channels], bias or None, state [slots, taps - 1, channels])."""
     T = x.shape[0]
+    ds, es = -(-dim // 4) * 4, -(-vdim // 8) * 8
+    assert x.stride(1) == a.stride(1) == 1 and a.dtype == x.dtype
+    assert all(t is None or t.dtype == torch.float32 and t.is_contiguous() for t in (a_log, dt_bias))
     assert sc.q.numel() >= T * kv_heads * ds and sc.v.numel() >= T * heads * es and sc.v.dtype == x.dtype
     assert not channel or sc.g.numel() >= T * heads * ds
-    p = native.DeltaPrepStruct(x.data_ptr(), x.stride(0), b.data_ptr(), b.stride(0), a.data_ptr(), a.stride(0),
-                               conv_w.data_ptr(), ldw, taps, conv_state.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(),
-                               sc.q.data_ptr(), sc.k.data_ptr(), sc.kq.data_ptr(), sc.v.data_ptr(), sc.coef.data_ptr(),
-                               sc.g.data_ptr() if channel else None, heads, kv_heads, dim, vdim, ds, es, T,
-                               int(x.dtype == torch.float32))
+    w = bias = state = None
+    taps = ldw = 0
+    if conv is not None:
+        w, bias, state = conv
+        taps, ldw = w.shape
+        assert w.dtype == torch.float32 and w.is_contiguous() and state.dtype == x.dtype and state.is_contiguous()
+        assert taps == 1 or tuple(state.shape[1:]) == (taps - 1, ldw)
+        assert x.shape[1] == ldw and (bias is None or bias.dtype == torch.float32 and bias.numel() == ldw)
+    p = native.RecPrepStruct(x.data_ptr(), x.stride(0), _ptr(w), _ptr(bias), ldw, taps, _ptr(state), *offs, _ptr(b),
+                             0 if b is None else b.stride(0), a.data_ptr(), a.stride(0), _ptr(a_log), dt_bias.data_ptr(),
+                             float(rate), sc.q.data_ptr(), sc.k.data_ptr(), sc.kq.data_ptr(), sc.v.data_ptr(),
+                             sc.coef.data_ptr(), sc.g.data_ptr() if channel else None, heads, kv_heads, dim, vdim, ds, es, T,
+                             int(x.dtype == torch.float32))
     st = _seg(seg)
-    native.check(native.lib().cb_delta_prepare(ctypes.byref(p), ctypes.byref(st), _stream()), "cb_delta_prepare")
+    native.check(getattr(native.lib(), entry)(ctypes.byref(p), ctypes.byref(st), _stream()), entry)
+
+
+def delta_prepare(x: torch.Tensor, b: torch.Tensor, a: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor,
+                  a_log: torch.Tensor, dt_bias: torch.Tensor, seg: GdnSegments, sc: RecurrenceScratch, heads: int, kv_heads: int,
+                  dim: int, vdim: int) -> None:
+    """Everything of a delta layer's tokens that does not depend on its state: causal depthwise convolution + SiLU of
+    ``x [T, q | k | v]`` with ``conv_w`` fp32 ``[taps, channels]`` (the last row multiplies the current input) and the
+    requests' last inputs ``conv_state [slots, taps - 1, channels]``, which are read and replaced; unit q / k; step sizes and
+    decays from the logits ``b`` and ``a``."""
+    assert b.stride(1) == 1 and b.dtype == x.dtype and dt_bias.numel() in (heads, heads * dim)
+    _prepare("cb_delta_prepare", x, a, dt_bias, seg, sc, heads, kv_heads, dim, vdim, dt_bias.numel() != heads,
+             (0, kv_heads * dim, 2 * kv_heads * dim), (conv_w, None, conv_state), b, a_log)
+
+
+def gated_linear_prepare(x: torch.Tensor, q_off: int, k_off: int, v_off: int, a: torch.Tensor, bias: torch.Tensor, rate: float,
+                         seg: GdnSegments, sc: RecurrenceScratch, heads: int, dim: int, vdim: int) -> None:
+    """The tokens of gated linear attention: q times ``dim^-1/2``, k and v at their columns of ``x``; decays
+    ``sigmoid(a + bias)^rate`` per key channel."""
+    assert a.shape[1] == bias.numel() == heads * dim and x.stride(0) % 2 == 0
+    assert x.shape[1] >= max(q_off + heads * dim, k_off + heads * dim, v_off + heads * vdim)
+    _prepare("cb_gated_linear_prepare", x, a, bias, seg, sc, heads, heads, dim, vdim, True, (q_off, k_off, v_off), rate=rate)
+
+
+def ssd_prepare(x: torch.Tensor, dt: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, conv_state: torch.Tensor,
+                a_log: torch.Tensor, dt_bias: torch.Tensor, seg: GdnSegments, sc: RecurrenceScratch, heads: int, groups: int,
+                state: int, vdim: int) -> None:
+    """The tokens of a state-space layer: convolution with bias + SiLU of ``x [T, x | B | C]`` (state as in
+    ``delta_prepare``), step sizes ``softplus(dt + dt_bias)`` and decays."""
+    assert dt.shape[1] == a_log.numel() == dt_bias.numel() == heads and conv_b is not None
+    inner = heads * vdim
+    _prepare("cb_ssd_prepare", x, dt, dt_bias, seg, sc, heads, groups, state, vdim, False,
+             (inner + groups * state, inner, 0), (conv_w, conv_b, conv_state), a_log=a_log)
+
+
+def _walk(entry: str, T: int, z, norm_w, skip, state, seg: GdnSegments, out, sc: RecurrenceScratch, kv_heads: int, dim: int,
+          eps: float, sigmoid_gate: bool, channel: bool, decode: bool, f32: bool) -> None:
+    H, e, ds = state.shape[1:]
+    assert state.dtype == torch.float32 and state.is_contiguous() and ds == -(-dim // 4) * 4
+    assert (sc.v.dtype == torch.float32) == f32 and sc.raw.numel() >= T * H * e
+    assert z is None or z.dtype == out.dtype == sc.v.dtype and z.stride(1) == out.stride(1) == 1 and out.shape[1] == H * e
+    assert all(t is None or t.dtype == torch.float32 and t.is_contiguous() for t in (norm_w, skip))
+    p = native.RecWalkStruct(sc.q.data_ptr(), sc.k.data_ptr(), sc.kq.data_ptr(), sc.v.data_ptr(), sc.coef.data_ptr(),
+                             sc.g.data_ptr() if channel else None, _ptr(skip), _ptr(z), 0 if z is None else z.stride(0),
+                             _ptr(norm_w), state.data_ptr(), _ptr(out), 0 if out is None else out.stride(0), sc.raw.data_ptr(), H,
+                             kv_heads, dim, e, ds, -(-e // 8) * 8, float(eps), int(sigmoid_gate), int(decode), T, int(f32))
+    st = _seg(seg)
+    native.check(getattr(native.lib(), entry)(ctypes.byref(p), ctypes.byref(st), _stream()), entry)
 
 
 def delta_walk(z: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, seg: GdnSegments, out: torch.Tensor,
-               sc: DeltaScratch, kv_heads: int, dim: int, eps: float, sigmoid_gate: bool, channel: bool, decode: bool) -> int:
+               sc: RecurrenceScratch, kv_heads: int, dim: int, eps: float, sigmoid_gate: bool, channel: bool, decode: bool) -> int:
     """The recurrence over the rows prepared by ``delta_prepare`` and the gated norm of every head.  ``state`` fp32
     ``[slots, H, vdim, stride]`` is read and replaced; ``channel``: one decay per key channel; ``decode``: every segment has
     at most one row.  Returns the launches made (at most)."""
-    H, e, ds = state.shape[1:]
-    T = z.shape[0]
-    assert state.dtype == torch.float32 and state.is_contiguous() and ds == -(-dim // 4) * 4
-    assert z.dtype == out.dtype == sc.v.dtype and z.stride(1) == out.stride(1) == 1 and out.shape[1] == H * e
-    assert norm_w.dtype == torch.float32 and sc.raw.numel() >= T * H * e
-    p = native.DeltaWalkStruct(sc.q.data_ptr(), sc.k.data_ptr(), sc.kq.data_ptr(), sc.v.data_ptr(), sc.coef.data_ptr(),
-                               sc.g.data_ptr() if channel else None, z.data_ptr(), z.stride(0), norm_w.data_ptr(),
-                               state.data_ptr(), out.data_ptr(), out.stride(0), sc.raw.data_ptr(), H, kv_heads, dim, e, ds,
-                               -(-e // 8) * 8, float(eps), int(sigmoid_gate), int(decode), T, int(z.dtype == torch.float32))
-    st = _seg(seg)
-    native.check(native.lib().cb_delta_walk(ctypes.byref(p), ctypes.byref(st), _stream()), "cb_delta_walk")
+    _walk("cb_delta_walk", z.shape[0], z, norm_w, None, state, seg, out, sc, kv_heads, dim, eps, sigmoid_gate, channel, decode,
+          z.dtype == torch.float32)
     return 1 if decode else 2
+
+
+def gated_linear_walk(z: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, seg: GdnSegments, out: torch.Tensor,
+                      sc: RecurrenceScratch, dim: int, eps: float, decode: bool) -> int:
+    """Gated linear attention over the rows of ``gated_linear_prepare``: recurrence, norm of every head, times ``silu(z)``.
+    State and return value as in ``delta_walk``."""
+    _walk("cb_linear_walk", z.shape[0], z, norm_w, None, state, seg, out, sc, state.shape[1], dim, eps, False, True, decode,
+          z.dtype == torch.float32)
+    return 1 if decode else 2
+
+
+def ssd_walk(z: torch.Tensor, d: torch.Tensor, norm_w: torch.Tensor, parts: int, state: torch.Tensor, seg: GdnSegments,
+             out: torch.Tensor, sc: RecurrenceScratch, groups: int, dim: int, eps: float, decode: bool) -> int:
+    """State-space layer over the rows of ``ssd_prepare``: recurrence, ``d`` times the value rows, and the gated norm in
+    ``parts`` equal parts across the heads.  State and return value as in ``delta_walk``."""
+    T, f32 = z.shape[0], z.dtype == torch.float32
+    width = norm_w.numel() // parts
+    assert z.shape[1] == out.shape[1] == parts * width and z.dtype == out.dtype and d.numel() == state.shape[1]
+    _walk("cb_linear_walk", T, None, None, d, state, seg, None, sc, groups, dim, eps, False, False, decode, f32)
+    native.check(native.lib().cb_gated_parts_norm(sc.raw.data_ptr(), z.data_ptr(), z.stride(0), norm_w.data_ptr(), out.data_ptr(),
+                                                  out.stride(0), T, parts, width, float(eps), int(f32), _stream()),
+                 "cb_gated_parts_norm")
+    return 2
 
 
 def latent_prepare(proj: torch.Tensor, q_rank: int, c_off: int, rank: int, q_norm: torch.Tensor, c_norm: torch.Tensor,
@@ -896,3 +991,54 @@ def latent_attention(q: torch.Tensor, gate: torch.Tensor, cache: torch.Tensor, p
                                 int(decode), splits, partial)
     st = _seg(seg)
     native.check(l.cb_latent_attn(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_latent_attn")
+
+
+def gqa_prepare(x: torch.Tensor, q_off: int, k_off: int, q_norm: torch.Tensor, k_norm: torch.Tensor, freq: torch.Tensor,
+                mult: float, positions: torch.Tensor, slots: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, heads: int,
+                dim: int, eps: float) -> None:
+    """Query and key heads of ``x``'s rows: RMS norm of a head, rotary positions on its first ``2 len(freq)`` channels; queries to
+    ``q [T, H P]``, keys and the raw key heads (values) to their rows of ``cache [pages, G, 2, 16, P]``."""
+    G, P = cache.shape[1], cache.shape[4]
+    assert cache.is_contiguous() and cache.dtype == x.dtype == q.dtype and q.is_contiguous() and q.shape[1] == heads * P
+    assert x.stride(1) == 1 and slots.dtype == positions.dtype == torch.int32
+    assert q_norm.dtype == k_norm.dtype == freq.dtype == torch.float32
+    a = native.GqaPrepStruct(x.data_ptr(), x.stride(0), q_off, k_off, q_norm.data_ptr(), k_norm.data_ptr(), freq.data_ptr(),
+                             float(mult), positions.data_ptr(), slots.data_ptr(), q.data_ptr(), cache.data_ptr(), heads, G, dim, P,
+                             freq.numel(), float(eps), x.shape[0], int(x.dtype == torch.float32))
+    native.check(native.lib().cb_gqa_prepare(ctypes.byref(a), _stream()), "cb_gqa_prepare")
+
+
+def gqa_attention(q: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor, seg: GdnSegments, out: torch.Tensor, heads: int,
+                  dim: int, window: int, scale: float, sink: float | None = None, out_scale: float = 1.0, decode: bool = False,
+                  splits: int | None = None, ws: Workspace | None = None) -> int:
+    """Windowed grouped-query attention over the paged cache of ``gqa_prepare``, times ``out_scale``.  ``window`` 0: every
+    earlier token; ``sink``: score of a softmax entry without a value.  ``decode``: every segment has at most one row.
+    ``splits``: key splits of the bf16 decode form (None: as many as fill the device).  Returns the launches made."""
+    G, P = cache.shape[1], cache.shape[4]
+    T = q.shape[0]
+    assert q.is_contiguous() and q.shape[1] == heads * P and out.stride(1) == 1 and out.shape[1] == heads * dim
+    assert q.dtype == out.dtype == cache.dtype and page_table.dtype == torch.int32
+    f32 = q.dtype == torch.float32
+    l = native.lib()
+    partial = None
+    if f32 or not decode:
+        splits = 1
+    else:
+        if splits is None:
+            from .strategies import active
+            units = ctypes.c_int(0)
+            l.cb_gqa_attn_partial_floats(T, seg.num, heads, G, P, 1, 1, ctypes.byref(units))
+            a = active().attention
+            # a block walks four pages at a time: no more splits than the longest row has such strides
+            keys = page_table.shape[1] * PAGE_TOKENS if window <= 0 else min(window, page_table.shape[1] * PAGE_TOKENS)
+            splits = min(a.max_splits, -(-keys // 64), max(1, a.target_ctas // units.value))
+        if splits > 1:
+            ws = ws or workspace(q.device)
+            ws.ensure_attn(l.cb_gqa_attn_partial_floats(T, seg.num, heads, G, P, 1, splits, None))
+            partial = ws.attn.data_ptr()
+    a = native.GqaAttnStruct(q.data_ptr(), out.data_ptr(), out.stride(0), cache.data_ptr(), page_table.data_ptr(),
+                             page_table.shape[1], heads, G, dim, P, window, float(scale), float(out_scale),
+                             float("-inf") if sink is None else float(sink), T, int(f32), int(decode), splits, partial)
+    st = _seg(seg)
+    native.check(l.cb_gqa_attn(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_gqa_attn")
+    return 2 if splits > 1 else 1

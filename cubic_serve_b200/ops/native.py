@@ -267,14 +267,23 @@ def _declare(l: ctypes.CDLL) -> None:
     l.cb_row_norm.argtypes = [vp, vp, vp, vp, i, i, i, f, i, vp]
     l.cb_embed_norm.argtypes = [vp, vp, vp, vp, vp, i, i, i, f, vp]
     l.cb_concat_rows.argtypes = [vp, vp, vp, i, i, i, i, vp]
-    l.cb_delta_prepare.argtypes = [vp, vp, vp]
-    l.cb_delta_walk.argtypes = [vp, vp, vp]
+    for name in ("delta_prepare", "gated_linear_prepare", "ssd_prepare", "delta_walk", "linear_walk"):
+        getattr(l, f"cb_{name}").argtypes = [vp, vp, vp]
+        getattr(l, f"cb_{name}").restype = i
+    l.cb_gated_parts_norm.argtypes = [vp, vp, i, vp, vp, i, i, i, i, f, i, vp]
+    l.cb_embed_rows.argtypes = [vp, vp, vp, vp, vp, i, i, i, i, f, i, vp]
+    l.cb_add_norm_rows.argtypes = [vp, i, vp, vp, vp, vp, i, i, i, f, i, vp]
+    l.cb_side_gate.argtypes = [vp, i, vp, i, vp, vp, i, i, vp, i, i, i, i, i, vp]
+    l.cb_gqa_prepare.argtypes = [vp, vp]
+    l.cb_gqa_attn.argtypes = [vp, vp, vp]
+    l.cb_gqa_attn_partial_floats.argtypes = [i, i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
+    l.cb_gqa_attn_partial_floats.restype = ll
     l.cb_latent_prepare.argtypes = [vp, i, i, i, i, i, vp, vp, vp, i, vp, i, vp, i, f, i, vp]
     l.cb_latent_attn.argtypes = [vp, vp, vp]
     l.cb_latent_attn_partial_floats.argtypes = [i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
     l.cb_latent_attn_partial_floats.restype = ll
-    for name in ("bf16_gemm_wide", "f32_gemm", "row_norm", "embed_norm", "concat_rows", "delta_prepare", "delta_walk",
-                 "latent_prepare", "latent_attn"):
+    for name in ("bf16_gemm_wide", "f32_gemm", "row_norm", "embed_norm", "concat_rows", "latent_prepare",
+                 "latent_attn", "gated_parts_norm", "embed_rows", "add_norm_rows", "side_gate", "gqa_prepare", "gqa_attn"):
         getattr(l, f"cb_{name}").restype = i
     # fp8 (e4m3 x e4m3) tensor path: activation quantizers and the GEMM entries
     l.cb_fp8_quantize_rows.argtypes = [vp, i, vp, i, vp, i, i, vp]
@@ -319,7 +328,7 @@ class WideGemmStruct(ctypes.Structure):
                 ("y", ctypes.c_void_p), ("y32", ctypes.c_void_p), ("ldy", ctypes.c_int), ("residual32", ctypes.c_void_p),
                 ("y2", ctypes.c_void_p), ("ldy2", ctypes.c_int), ("n_split", ctypes.c_int), ("diag_n", ctypes.c_int),
                 ("M", ctypes.c_int), ("N", ctypes.c_int), ("K", ctypes.c_int), ("stream_k", ctypes.c_int),
-                ("splits", ctypes.c_int), ("min_units", ctypes.c_int)]
+                ("splits", ctypes.c_int), ("min_units", ctypes.c_int), ("glu", ctypes.c_int)]
 
 
 class F32GemmStruct(ctypes.Structure):
@@ -327,26 +336,27 @@ class F32GemmStruct(ctypes.Structure):
     _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("x_cols", ctypes.c_int), ("w", ctypes.c_void_p),
                 ("y", ctypes.c_void_p), ("ldy", ctypes.c_int), ("residual", ctypes.c_void_p), ("y2", ctypes.c_void_p),
                 ("ldy2", ctypes.c_int), ("n_split", ctypes.c_int), ("diag_n", ctypes.c_int), ("M", ctypes.c_int),
-                ("N", ctypes.c_int), ("K", ctypes.c_int)]
+                ("N", ctypes.c_int), ("K", ctypes.c_int), ("glu", ctypes.c_int)]
 
 
-class DeltaPrepStruct(ctypes.Structure):
-    """Mirror of ``CbDeltaPrep`` in ``csrc/delta_rule.cu``."""
-    _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("b", ctypes.c_void_p), ("ldb", ctypes.c_int),
-                ("a", ctypes.c_void_p), ("lda", ctypes.c_int), ("w", ctypes.c_void_p), ("ldw", ctypes.c_int),
-                ("taps", ctypes.c_int), ("state", ctypes.c_void_p), ("a_log", ctypes.c_void_p), ("dt_bias", ctypes.c_void_p),
-                ("q", ctypes.c_void_p), ("k", ctypes.c_void_p), ("kq", ctypes.c_void_p), ("v", ctypes.c_void_p),
-                ("coef", ctypes.c_void_p), ("g", ctypes.c_void_p), ("H", ctypes.c_int), ("G", ctypes.c_int),
-                ("d", ctypes.c_int), ("e", ctypes.c_int), ("ds", ctypes.c_int), ("es", ctypes.c_int),
+class RecPrepStruct(ctypes.Structure):
+    """Mirror of ``CbRecPrep`` in ``csrc/recurrence.cuh``."""
+    _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("w", ctypes.c_void_p), ("bias", ctypes.c_void_p),
+                ("ldw", ctypes.c_int), ("taps", ctypes.c_int), ("state", ctypes.c_void_p), ("q_off", ctypes.c_int),
+                ("k_off", ctypes.c_int), ("v_off", ctypes.c_int), ("b", ctypes.c_void_p), ("ldb", ctypes.c_int),
+                ("a", ctypes.c_void_p), ("lda", ctypes.c_int), ("a_log", ctypes.c_void_p), ("dt_bias", ctypes.c_void_p),
+                ("rate", ctypes.c_float), ("q", ctypes.c_void_p), ("k", ctypes.c_void_p), ("kq", ctypes.c_void_p),
+                ("v", ctypes.c_void_p), ("coef", ctypes.c_void_p), ("g", ctypes.c_void_p), ("H", ctypes.c_int),
+                ("G", ctypes.c_int), ("d", ctypes.c_int), ("e", ctypes.c_int), ("ds", ctypes.c_int), ("es", ctypes.c_int),
                 ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
 
 
-class DeltaWalkStruct(ctypes.Structure):
-    """Mirror of ``CbDeltaWalk`` in ``csrc/delta_rule.cu``."""
+class RecWalkStruct(ctypes.Structure):
+    """Mirror of ``CbRecWalk`` in ``csrc/recurrence.cuh``."""
     _fields_ = [("q", ctypes.c_void_p), ("k", ctypes.c_void_p), ("kq", ctypes.c_void_p), ("v", ctypes.c_void_p),
-                ("coef", ctypes.c_void_p), ("g", ctypes.c_void_p), ("z", ctypes.c_void_p), ("ldz", ctypes.c_int),
-                ("norm_w", ctypes.c_void_p), ("state", ctypes.c_void_p), ("out", ctypes.c_void_p), ("ldo", ctypes.c_int),
-                ("raw", ctypes.c_void_p), ("H", ctypes.c_int), ("G", ctypes.c_int), ("d", ctypes.c_int),
+                ("coef", ctypes.c_void_p), ("g", ctypes.c_void_p), ("skip", ctypes.c_void_p), ("z", ctypes.c_void_p),
+                ("ldz", ctypes.c_int), ("norm_w", ctypes.c_void_p), ("state", ctypes.c_void_p), ("out", ctypes.c_void_p),
+                ("ldo", ctypes.c_int), ("raw", ctypes.c_void_p), ("H", ctypes.c_int), ("G", ctypes.c_int), ("d", ctypes.c_int),
                 ("e", ctypes.c_int), ("ds", ctypes.c_int), ("es", ctypes.c_int), ("eps", ctypes.c_float),
                 ("sigmoid_gate", ctypes.c_int), ("decode", ctypes.c_int), ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
 
@@ -357,6 +367,24 @@ class LatentAttnStruct(ctypes.Structure):
                 ("ldg", ctypes.c_int), ("page_table", ctypes.c_void_p), ("max_pages", ctypes.c_int), ("H", ctypes.c_int),
                 ("Rp", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float), ("tokens", ctypes.c_int),
                 ("f32", ctypes.c_int), ("decode", ctypes.c_int), ("splits", ctypes.c_int), ("partial", ctypes.c_void_p)]
+
+
+class GqaPrepStruct(ctypes.Structure):
+    """Mirror of ``CbGqaPrep`` in ``csrc/gqa_attn.cu``."""
+    _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("q_off", ctypes.c_int), ("k_off", ctypes.c_int),
+                ("qw", ctypes.c_void_p), ("kw", ctypes.c_void_p), ("freq", ctypes.c_void_p), ("mult", ctypes.c_float),
+                ("positions", ctypes.c_void_p), ("slots", ctypes.c_void_p), ("q", ctypes.c_void_p), ("cache", ctypes.c_void_p),
+                ("H", ctypes.c_int), ("G", ctypes.c_int), ("d", ctypes.c_int), ("P", ctypes.c_int), ("pairs", ctypes.c_int),
+                ("eps", ctypes.c_float), ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
+
+
+class GqaAttnStruct(ctypes.Structure):
+    """Mirror of ``CbGqaAttn`` in ``csrc/gqa_attn.cu``."""
+    _fields_ = [("q", ctypes.c_void_p), ("out", ctypes.c_void_p), ("ldo", ctypes.c_int), ("cache", ctypes.c_void_p),
+                ("page_table", ctypes.c_void_p), ("max_pages", ctypes.c_int), ("H", ctypes.c_int), ("G", ctypes.c_int),
+                ("d", ctypes.c_int), ("P", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float),
+                ("out_scale", ctypes.c_float), ("sink", ctypes.c_float), ("tokens", ctypes.c_int), ("f32", ctypes.c_int),
+                ("decode", ctypes.c_int), ("splits", ctypes.c_int), ("partial", ctypes.c_void_p)]
 
 
 class ReduceNormStruct(ctypes.Structure):

@@ -176,7 +176,7 @@ def run_delta(c, shape, dtype, spans, conv_state, state, eps=1e-5, decode=None):
     w[:, :C] = c["conv"].t()
     dev = {k: v.to(DEV, dtype).contiguous() for k, v in c.items() if k in "baz"}
     f32 = {k: c[k].float().to(DEV).contiguous() for k in ("a_log", "dt", "norm")}
-    sc = K.DeltaScratch(T, [(H, G, d, e, per_channel)], dtype, DEV)
+    sc = K.RecurrenceScratch(T, [(H, G, d, e, per_channel)], dtype, DEV)
     seg = spans if not isinstance(spans, list) else segs(spans)
     out = torch.full((T, H * e + 8), 3.0, dtype=dtype, device=DEV)[:, :H * e]
     K.delta_prepare(x.to(DEV), dev["b"], dev["a"], w.to(DEV), conv_state, f32["a_log"], f32["dt"], seg, sc, H, G, d, e)
