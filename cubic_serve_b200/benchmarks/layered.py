@@ -2,8 +2,8 @@
 throughput of whole models (``bench.py --layered``).
 
 The closest model is the hybrid family (Gated DeltaNet layers with periodic full attention) with bf16 weights; its SwiGLU
-feed-forward has three matrices where the layered one has two, so its width is two thirds: equal parameters.  Weights are
-random, prompts are random ids, one GPU.  Kernel times are CUDA-event times inside CUDA graphs with L2 flushed; the roofline
+feed-forward has three matrices where a parallel layer's has two, so its width is two thirds of that: equal parameters (the
+sequential layers have the same three matrices).  Weights are random, prompts are random ids, one GPU.  Kernel times are CUDA-event times inside CUDA graphs with L2 flushed; the roofline
 of a kernel is the slower of its bytes over the copy bandwidth and its operations over the pipe that runs them.
 """
 from __future__ import annotations
@@ -14,7 +14,8 @@ from pathlib import Path
 import torch
 
 from ..models.config import ModelConfig, QuantSpec
-from ..models.layered import DeltaSpec, LatentSpec, LayeredConfig, LayerSpec
+from ..models.layered import (AttentionSpec, DeltaSpec, GatedLinearSpec, LatentSpec, LayeredConfig, LayerSpec, PairSpec, RotarySpec,
+                              SsdSpec)
 from ..ops import kernels as K, wq_pack
 from ..utils.kernel_bench import DEV, timeit_graph
 
@@ -37,6 +38,18 @@ def layered_config(width: int, layers: int) -> LayeredConfig:
     channel = LayerSpec(DeltaSpec(h, h, 128, 128, 4, True, 128, 128), ff)
     latent = LayerSpec(LatentSpec(h, 128, 128, 1536, 512, 128 ** -0.5, 1024), ff)
     return LayeredConfig(f"layered-{width}", 32768, width, (delta, channel, delta, latent) * (layers // 4), 1e-6)
+
+
+def sequential_config(width: int, layers: int) -> LayeredConfig:
+    """Real-model sequential layers at ``width``: attention heads of 128 (four per key head, window 1024) beside gated linear
+    heads of 128 over half the width; every fourth layer a state-space layer of twice the width (heads of 64, state 128)."""
+    h, ff = width // 128, 2 * width
+    rotary = RotarySpec(64, 1e6, ("yarn", 4.0, 8192.0, 32.0, 1.0, 1.14))
+    pair = LayerSpec(PairSpec(AttentionSpec(h, max(1, h // 4), 128, 128 ** -0.5, rotary, 1024), GatedLinearSpec(h // 2, 128, 128, 16.0, 64),
+                              1.0, 1.0), ff)
+    ssd = LayerSpec(SsdSpec(width // 32, 64, 128, 8, 4, 8), ff)
+    return LayeredConfig(f"sequential-{width}", 32768, width, (ssd, pair, pair, pair) * (layers // 4), 1e-6, architecture="Loduzen",
+                         side_dim=64)
 
 
 def hybrid_config(width: int, layers: int) -> ModelConfig:
@@ -111,6 +124,88 @@ def bench_gdn(requests: int, tokens: int, hv: int, hk: int, flush, pk) -> list[d
                   4 * 2.0 * T * hv * d * d, FP32_FLOPS, pk),
             _line(f"gdn_delta [{shape}]", delta, 2 * state.numel() * 4 + T * (C + 2 * hv * d + 2 * hv) * 2,
                   4 * 2.0 * T * hv * d * d, FP32_FLOPS, pk)]
+
+
+def bench_gated_linear(requests: int, tokens: int, heads: int, flush, pk) -> list[dict]:
+    d, T, H = 128, requests * tokens, heads
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    seg = _segments(requests, tokens, 5)
+    proj, a, bias = torch.randn(T, 4 * H * d, **bf), torch.randn(T, H * d, **bf), torch.zeros(H * d, device=DEV)
+    state, out = torch.randn(requests, H, d, d, device=DEV) * 0.01, torch.empty(T, H * d, **bf)
+    norm_w = torch.ones(d, device=DEV)
+    sc = K.RecurrenceScratch(T, [(H, H, d, d, True)], torch.bfloat16, DEV)
+    prep = timeit_graph(lambda: K.gated_linear_prepare(proj, 0, H * d, 2 * H * d, a, bias, 1 / 16, seg, sc, H, d, d), flush, launches=5)
+    walk = timeit_graph(lambda: K.gated_linear_walk(proj[:, 3 * H * d:], norm_w, state, seg, out, sc, d, 1e-6, tokens == 1), flush, launches=5)
+    shape = f"{requests} x {tokens} tokens, {H} heads of 128"
+    return [_line(f"gated_linear_prepare [{shape}]", prep, T * 4 * H * d * 2, 0, 1, pk),
+            _line(f"gated_linear_walk + norm [{shape}]", walk, 2 * state.numel() * 4 + T * 6 * H * d * 2, 3 * 2.0 * T * H * d * d, FP32_FLOPS, pk),
+            _line(f"gated linear both [{shape}]", prep + walk, 2 * state.numel() * 4 + T * 6 * H * d * 2, 3 * 2.0 * T * H * d * d, FP32_FLOPS, pk)]
+
+
+def bench_ssd(requests: int, tokens: int, heads: int, groups: int, flush, pk) -> list[dict]:
+    P, N, T, H, G = 64, 128, requests * tokens, heads, groups
+    C = H * P + 2 * G * N
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    seg = _segments(requests, tokens, 5)
+    proj, z, dt = torch.randn(T, C, **bf), torch.randn(T, H * P, **bf), torch.randn(T, H, **bf)
+    conv_w, conv_b, conv_state = torch.randn(4, C, device=DEV) * 0.3, torch.zeros(C, device=DEV), torch.zeros(requests, 3, C, **bf)
+    state, out = torch.randn(requests, H, P, N, device=DEV) * 0.01, torch.empty(T, H * P, **bf)
+    a_log, dt_bias, D, norm_w = torch.full((H,), -2.0, device=DEV), torch.zeros(H, device=DEV), torch.ones(H, device=DEV), torch.ones(H * P, device=DEV)
+    sc = K.RecurrenceScratch(T, [(H, G, N, P, False)], torch.bfloat16, DEV)
+    prep = timeit_graph(lambda: K.ssd_prepare(proj, dt, conv_w, conv_b, conv_state, a_log, dt_bias, seg, sc, H, G, N, P), flush, launches=5)
+    walk = timeit_graph(lambda: K.ssd_walk(z, D, norm_w, G, state, seg, out, sc, G, N, 1e-6, tokens == 1), flush, launches=5)
+    shape = f"{requests} x {tokens} tokens, {H} heads of 64, state 128"
+    conv_io = T * C * 4 + 2 * requests * 3 * C * 2
+    return [_line(f"ssd_prepare [{shape}]", prep, conv_io + T * H * 2, 0, 1, pk),
+            _line(f"ssd_walk + norm [{shape}]", walk, 2 * state.numel() * 4 + T * (C + 2 * H * P) * 2, 3 * 2.0 * T * H * P * N, FP32_FLOPS, pk),
+            _line(f"ssd both [{shape}]", prep + walk, 2 * state.numel() * 4 + conv_io + T * (2 * H * P + H) * 2, 3 * 2.0 * T * H * P * N,
+                  FP32_FLOPS, pk)]
+
+
+def bench_gqa(requests: int, tokens: int, ctx: int, heads: int, kv_heads: int, window: int, flush, pk) -> list[dict]:
+    d, T, per = 128, requests * tokens, -(-ctx // 16)
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    cache = torch.randn(requests * per + 1, kv_heads, 2, 16, d, **bf)
+    table = (torch.randperm(requests * per, device=DEV).to(torch.int32) + 1).view(requests, per)
+    x, q, out = torch.randn(T, (heads + kv_heads) * d, **bf), torch.empty(T, heads * d, **bf), torch.empty(T, heads * d, **bf)
+    qn, freq = torch.ones(d, device=DEV), torch.rand(32, device=DEV)
+    seg = _segments(requests, tokens, ctx - tokens)
+    pos = torch.arange(ctx - tokens, ctx, device=DEV, dtype=torch.int32).repeat(requests)
+    slots = (table.long().gather(1, (pos.view(requests, tokens) // 16).long()) * 16 + pos.view(requests, tokens) % 16).to(torch.int32).view(-1)
+    prep = timeit_graph(lambda: K.gqa_prepare(x, 0, heads * d, qn, qn, freq, 1.1, pos, slots, q, cache, heads, d, 1e-6), flush, launches=5)
+    ms = timeit_graph(lambda: K.gqa_attention(q, cache, table, seg, out, heads, d, window, 0.09, 0.0, decode=tokens == 1), flush, launches=5)
+    pairs = requests * _visible(tokens, ctx, window)
+    keys = requests * (min(ctx, window + tokens - 1) if window else ctx)
+    shape = f"{requests} x {tokens} at {ctx}, window {window}, {heads}/{kv_heads} heads"
+    return [_line(f"gqa_prepare [{shape}]", prep, T * (2 * heads + 3 * kv_heads) * d * 2, 0, 1, pk),
+            _line(f"gqa_attention [{shape}]", ms, keys * kv_heads * 2 * d * 2 + 2 * T * heads * d * 2, 4.0 * pairs * heads * d, pk["bf16"], pk)]
+
+
+def bench_sequential_rows(m: int, width: int, side: int, flush, pk) -> list[dict]:
+    """The gated product, the side input's steps and the fused norm, beside their plain counterparts."""
+    ff = 2 * width
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    h, x = torch.randn(m, width, **bf), torch.randn(m, width, device=DEV)
+    w = wq_pack.swiglu_interleave(wq_pack.pack_bf16(torch.randn(2 * ff, width, device=DEV) * 0.02))
+    act, nw = torch.empty(m, ff, **bf), torch.ones(width, device=DEV)
+    glu = timeit_graph(lambda: K.wide_gemm(h, w, act, gelu_glu=True), flush, launches=5)
+    silu = timeit_graph(lambda: K.wq_gemm_act(h, w, out=act), flush, launches=5)
+    gate, table = torch.randn(side, width, **bf), torch.randn(4096, 8 * side, **bf)
+    ids, g = torch.randint(0, 4096, (m,), device=DEV, dtype=torch.int32), torch.zeros(m, -(-side // 64) * 64, **bf)
+    proj, y = wq_pack.pack_bf16(torch.zeros(width, g.shape[1], **bf)), torch.randn(m, width, **bf)
+    sg = timeit_graph(lambda: K.side_gate(x, gate, ids, table, side, g), flush, launches=5)
+    sp = timeit_graph(lambda: K.wide_gemm(g, proj, y), flush, launches=5)
+    add = timeit_graph(lambda: K.add_norm_rows(y, nw, x, 1e-6, nw, h), flush, launches=5)
+    rn = timeit_graph(lambda: K.row_norm(x, nw, h, 1e-6), flush, launches=5)
+    K.workspace(torch.device(DEV)).check_status()
+    flops = 2.0 * m * 2 * ff * width
+    nbytes = (2 * ff * width + m * (width + ff)) * 2
+    return [_line(f"wide_gemm gate/up (gelu) [{m} x {2 * ff} x {width}]", glu, nbytes, flops, pk["bf16"], pk),
+            _line("wq_gemm_act bf16 (silu), same shape", silu, nbytes, flops, pk["bf16"], pk),
+            _line(f"side_gate [{m} x {side} x {width}]", sg, m * width * 4 + side * width * 2 + m * side * 4, 2.0 * m * side * width, pk["bf16"], pk),
+            _line(f"side projection [{m} x {width} x {g.shape[1]}]", sp, m * width * 2 + m * side * 2, 2.0 * m * side * width, pk["bf16"], pk),
+            _line(f"add_norm_rows [{m} x {width}]", add, m * width * 12, 0, 1, pk),
+            _line(f"row_norm fp32 in [{m} x {width}]", rn, m * width * 6, 0, 1, pk)]
 
 
 def _visible(tokens: int, ctx: int, window: int) -> int:
@@ -208,6 +303,23 @@ def kernels(width: int = 4096) -> list[dict]:
     return out
 
 
+def sequential_kernels(width: int = 4096) -> list[dict]:
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=DEV)
+    pk = peaks()
+    h = width // 128
+    out = []
+    for requests, tokens in ((256, 1), (8, 1024), (1, 4096)):
+        out += bench_gated_linear(requests, tokens, h // 2, flush, pk)
+        out += bench_ssd(requests, tokens, width // 32, 8, flush, pk)
+        out += bench_gdn(requests, tokens, h, h // 2, flush, pk)
+    for requests, tokens, ctx in ((256, 1, 1280), (1, 1, 4096), (8, 1024, 1024), (1, 4096, 4096)):
+        out += bench_gqa(requests, tokens, ctx, h, max(1, h // 4), 1024, flush, pk)
+        out += bench_paged(requests, tokens, ctx, h, max(1, h // 4), flush, pk)
+    for m in (16, 256, 4096):
+        out += bench_sequential_rows(m, width, 64, flush, pk)
+    return out
+
+
 # ------------------------------------------------------------------ whole models
 def model_throughput(cfg, concurrency: int, prompt: int, steps: int, warmup: int = 4, budget: int = 8192) -> dict:
     """Prefill and decode rates of a random model through the serving engine."""
@@ -267,11 +379,13 @@ def model_throughput(cfg, concurrency: int, prompt: int, steps: int, warmup: int
     return out
 
 
-def run(steps: int = 32) -> None:
-    """Prints one JSON line per measurement."""
-    for line in kernels():
+def run(steps: int = 32, designs: str = "all") -> None:
+    """Prints one JSON line per measurement.  ``designs``: all, or ``parallel`` / ``sequential`` layers only."""
+    both = designs == "all"
+    for line in (kernels() if both or designs == "parallel" else []) + (sequential_kernels() if both or designs == "sequential" else []):
         print(json.dumps(line), flush=True)
+    models = [c for d, c in (("parallel", layered_config), ("sequential", sequential_config)) if both or designs == d] + [hybrid_config]
     for width, layers in ((2048, 8), (4096, 8)):
         for concurrency, prompt in ((1, 4096), (16, 1024), (256, 1024)):
-            for cfg in (layered_config(width, layers), hybrid_config(width, layers)):
-                print(json.dumps(model_throughput(cfg, concurrency, prompt, steps)), flush=True)
+            for make in models:
+                print(json.dumps(model_throughput(make(width, layers), concurrency, prompt, steps)), flush=True)

@@ -46,12 +46,14 @@ gqa_prepare_kernel(const GqaPrep<T> p) {
   const size_t t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (static_cast<int>(threadIdx.x) < p.pairs) {
-    // the rounding error of the product is put back to first order: angles of far positions keep their fraction of a turn
+    // the rounding error e of the product is put back (|e| < 0.04 up to a million radians): angles of far positions keep their
+    // fraction of a turn
     const float pos = static_cast<float>(p.positions[t]), f = p.freq[threadIdx.x];
     const float a = pos * f, e = fmaf(pos, f, -a);
     float s, c;
     sincosf(a, &s, &c);
-    turn[threadIdx.x] = make_float2(fmaf(-e, s, c) * p.mult, fmaf(e, c, s) * p.mult);
+    const float ce = fmaf(-0.5f * e, e, 1.f), se = e * fmaf(e * (-1.f / 6.f), e, 1.f);
+    turn[threadIdx.x] = make_float2((c * ce - s * se) * p.mult, fmaf(s, ce, c * se) * p.mult);
   }
   __syncthreads();
   const int slot = p.slots[t];

@@ -970,7 +970,26 @@ def layered_8b_config() -> LayeredConfig:
     return LayeredConfig("layered-8b", 151936, 4096, (delta, channel, channel, latent) * 9, 1e-6, None)
 
 
-NAMED = {"layered-tiny": tiny_layered_config, "layered-8b": layered_8b_config}
+def tiny_sequential_config() -> LayeredConfig:
+    """A few small sequential layers of both kinds (tests and demonstrations)."""
+    pair = PairSpec(AttentionSpec(6, 2, 40, 0.2, RotarySpec(24, 10000.0, ("yarn", 4.0, 128.0, 16.0, 1.0, 0.1 * math.log(4.0) + 1.0)), 37),
+                    GatedLinearSpec(3, 24, 32, 8.0, 12), 0.8, 1.1)
+    ssd = SsdSpec(6, 24, 20, 2, 4, 3)
+    return LayeredConfig("layered-seq-tiny", 384, 192, (LayerSpec(ssd, 160), LayerSpec(pair, 160), LayerSpec(ssd, 96), LayerSpec(pair, 0)),
+                         1e-5, architecture="Loduzen", side_dim=20)
+
+
+def sequential_8b_config() -> LayeredConfig:
+    """Sequential layers of the size of an 8B model: one state-space layer in four, else windowed sink attention beside gated
+    linear attention."""
+    rotary = RotarySpec(64, 1e6, ("yarn", 8.0, 8192.0, 32.0, 1.0, 0.1 * math.log(8.0) + 1.0))
+    pair = LayerSpec(PairSpec(AttentionSpec(32, 8, 128, 128 ** -0.5, rotary, 1024), GatedLinearSpec(16, 128, 128, 16.0, 64), 1.0, 1.0), 12288)
+    ssd = LayerSpec(SsdSpec(128, 64, 128, 8, 4, 8), 12288)
+    return LayeredConfig("layered-seq-8b", 151936, 4096, (ssd, pair, pair, pair) * 8, 1e-6, architecture="Loduzen", side_dim=64)
+
+
+NAMED = {"layered-tiny": tiny_layered_config, "layered-8b": layered_8b_config, "layered-seq-tiny": tiny_sequential_config,
+         "layered-seq-8b": sequential_8b_config}
 
 
 def with_dtype(cfg: LayeredConfig, dtype: str) -> LayeredConfig:

@@ -42,6 +42,52 @@ CASES = {
     "wide": config(256, 128, [delta(2, 1, 128, 144, 4, 128), latent(40, 8, 8, 64, 136, 50, 0.35, 0),
                               channel(2, 1, 160, 64, 4, 96)], (2, 3, 1), 1e-6),
 }
+
+
+# ------------------------------------------------------------------ sequential layers (Loduzen)
+def parallel(left, right, scales, ff):
+    """``left``: (heads, kv heads, dim, window, scale, rotary dims, base, yarn (factor, original, fast, slow) or None);
+    ``right``: (heads, dim, vdim, tau)."""
+    H, G, d, size, scale, dims, base, yarn = left
+    rot = {"dims": dims, "base": base, "scaling": dict(zip(("factor", "original", "fast", "slow"), yarn)) if yarn else None}
+    return {"type": "parallel",
+            "mixer": {"left": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": scale, "rot": rot,
+                               "mask": {"size": size} if size else None},
+                      "right": dict(zip(("heads", "dim", "vdim", "tau"), right)),
+                      "left_scale": scales[0], "right_scale": scales[1]},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def mamba2(heads, vdim, state, groups, conv, norm_groups, ff):
+    return {"type": "mamba2", "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv,
+                                        "norm_groups": norm_groups},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def sequential(vocab, width, layers, side=0, eps=1e-5):
+    return {"architecture": "Loduzen", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": eps},
+            "token_side": {"dim": side} if side else None}
+
+
+SEQUENTIAL = {
+    # both mixers, grouped heads, stretched rotary pairs, parts of the norm, a layer without a feed-forward
+    "seq": sequential(210, 96, [parallel((6, 2, 24, 21, 0.3, 12, 1000.0, (3.0, 40, 4.0, 0.5)), (3, 20, 28, 8.0), (0.7, 1.3), 80),
+                                mamba2(4, 24, 20, 2, 4, 3, 96),
+                                parallel((4, 4, 32, 40, 0.25, 32, 5000.0, (2.0, 64, 8.0, 1.0)), (2, 32, 16, 16.0), (1.1, 0.6), 0),
+                                mamba2(2, 40, 16, 1, 3, 1, 64)], 12, 1e-6),
+    # single heads, a window of one token, one tap, no side input, plain rotation
+    "seq_small": sequential(71, 64, [mamba2(1, 16, 16, 1, 1, 1, 48),
+                                     parallel((1, 1, 16, 1, 0.25, 16, 100.0, None), (1, 16, 16, 1.0), (1.0, 1.0), 64)]),
+    # odd widths, many taps, three query heads per key head, every earlier token, no rotated channel in one layer
+    "seq_odd": sequential(123, 68, [parallel((9, 3, 13, 0, 0.4, 6, 50.0, (4.0, 30, 2.0, 1.0)), (2, 7, 9, 3.0), (0.5, 1.5), 44),
+                                    mamba2(6, 5, 7, 3, 6, 5, 36),
+                                    parallel((5, 1, 18, 33, 0.3, 0, 10.0, None), (3, 10, 12, 5.0), (1.2, 0.8), 20)], 5, 1e-4),
+    # wide heads, more query heads than a block has rows, windows over several pages
+    "seq_wide": sequential(256, 128, [parallel((40, 1, 72, 50, 0.15, 64, 10000.0, (8.0, 100, 32.0, 1.0)), (1, 144, 72, 16.0), (0.9, 1.2), 0),
+                                      mamba2(4, 130, 136, 1, 4, 4, 128),
+                                      parallel((3, 1, 200, 19, 0.1, 40, 300.0, None), (2, 96, 200, 4.0), (1.0, 0.5), 96)], 40),
+}
+ALL = {**CASES, **SEQUENTIAL}
 LOW_RANKS = (12, 20)          # inner sizes of the low-rank decay and gate projections
 
 
@@ -56,6 +102,9 @@ def tensors(cfg: dict, seed: int = 0) -> dict[str, torch.Tensor]:
         out[name] = (mean + std * torch.randn(n, generator=g)).to(torch.bfloat16)
 
     mat("embed", cfg["vocab"], W, math.sqrt(W))
+    if cfg["architecture"] == "Loduzen":
+        _sequential_tensors(cfg, mat, vec)
+        return out
     vec("embed.norm", W)
     vec("final.norm", W)
     mat("head", cfg["vocab"], W)
@@ -97,6 +146,52 @@ def tensors(cfg: dict, seed: int = 0) -> dict[str, torch.Tensor]:
             mat(f"l{i}.mlp.up", l["mlp"]["ff"], W)
             mat(f"l{i}.mlp.down", W, l["mlp"]["ff"])
     return out
+
+
+def _sequential_tensors(cfg: dict, mat, vec) -> None:
+    W = cfg["width"]
+    side = (cfg["token_side"] or {}).get("dim", 0)
+    vec("final.norm", W, 1.0)
+    if side:
+        mat("side.embed", cfg["vocab"], len(cfg["layers"]) * side, math.sqrt(len(cfg["layers"]) * side))
+    for i, l in enumerate(cfg["layers"]):
+        m, p = l["mixer"], f"l{i}.mix"
+        vec(f"l{i}.norm1", W, 1.0)
+        if l["type"] == "mamba2":
+            H, inner = m["heads"], m["heads"] * m["vdim"]
+            C = inner + 2 * m["groups"] * m["state"]
+            mat(f"{p}.in", inner + C + H, W)
+            mat(f"{p}.conv", C, m["conv"], 1.5)
+            vec(f"{p}.conv.b", C, 0.1, 0.3)
+            vec(f"{p}.dt_bias", H, -1.0, 0.7)
+            vec(f"{p}.A_log", H, -1.0, 0.7)
+            vec(f"{p}.D", H, 0.5, 0.5)
+            vec(f"{p}.norm", inner, 1.0)
+            mat(f"{p}.o", W, inner)
+        else:
+            a, g = m["left"], m["right"]
+            for t, n in (("q", a["heads"]), ("k", a["kv_heads"])):
+                mat(f"{p}.left.{t}", n * a["dim"], W)
+                vec(f"{p}.left.{t}.norm", a["dim"], 1.0, 0.3)
+            mat(f"{p}.left.o", W, a["heads"] * a["dim"])
+            H, d, e = g["heads"], g["dim"], g["vdim"]
+            for t, n in (("q", d), ("k", d), ("v", e), ("g", e)):
+                mat(f"{p}.right.{t}", H * n, W)
+            mat(f"{p}.right.o", W, H * e)
+            vec(f"{p}.right.norm", e, 1.0)
+            mat(f"{p}.right.a1", LOW_RANKS[0], W)
+            mat(f"{p}.right.a2", H * d, LOW_RANKS[0], 1.5)
+            vec(f"{p}.right.a2.b", H * d, 1.0, 0.5)
+        if l["mlp"]:
+            ff = l["mlp"]["ff"]
+            vec(f"l{i}.norm2", W, 1.0)
+            mat(f"l{i}.mlp.gate", ff, W)
+            mat(f"l{i}.mlp.up", ff, W)
+            mat(f"l{i}.mlp.down", W, ff)
+        if side:
+            mat(f"l{i}.side.gate", side, W)
+            mat(f"l{i}.side.proj", W, side)
+            vec(f"l{i}.side.norm", W, 0.3, 0.1)
 
 
 def write(path, cfg: dict, weights: dict[str, torch.Tensor]):

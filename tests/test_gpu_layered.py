@@ -6,9 +6,11 @@ from pathlib import Path
 import numpy as np
 import pytest
 import torch
+from torch.overrides import TorchFunctionMode
 
 sys.path.insert(0, str(Path(__file__).parent))
-from layered_cases import CASES, channel, config, delta, latent, prompt, tensors, write  # noqa: E402
+from layered_cases import (ALL, CASES, channel, config, delta, latent, mamba2, parallel, prompt, sequential,  # noqa: E402
+                           tensors, write)
 
 from cubic_serve_b200.models import layered_reference as R  # noqa: E402
 
@@ -386,7 +388,7 @@ WORST = {"float32": 2e-5, "bfloat16": 8e-2}
 
 def engine_for(tmp_path, name, dtype, max_tokens=512, requests=4, seed=1, raw=None):
     from cubic_serve_b200.utils.trace_run import build_engine
-    raw = raw or CASES[name]
+    raw = raw or ALL[name]
     w = tensors(raw, seed)
     return build_engine(str(write(tmp_path / "model", raw, w)), dtype, max_tokens, max_requests=requests), raw, w
 
@@ -397,47 +399,80 @@ def session_for(*a, **k):
     return ImposedSession(eng), raw, R.Oracle(raw, w, torch.float64)
 
 
-def off(got, want, dtype):
+class RoundedProducts(TorchFunctionMode):
+    """Operands and results of every matrix product rounded to bf16: the least a bf16 model rounds.  ``scale``: what is rounded
+    is this many times larger, so that other values round up and down."""
+
+    def __init__(self, scale):
+        super().__init__()
+        self.scale = scale
+
+    def __torch_function__(self, func, types, args=(), kwargs=None):
+        if func in (torch.Tensor.__matmul__, torch.Tensor.matmul, torch.matmul):
+            r = lambda t: (t * self.scale).to(torch.bfloat16).to(t.dtype) / self.scale      # noqa: E731
+            return r(func(r(args[0]), r(args[1])))
+        return func(*args, **(kwargs or {}))
+
+
+def error(got, want):
     d = torch.as_tensor(np.asarray(got)).double() - want
     d -= d.mean(-1, keepdim=True)
-    err = d.pow(2).mean(-1).sqrt() / want.pow(2).mean(-1).sqrt()
-    assert (err <= WORST[dtype]).all(), (float(err.max()), int(err.argmax()))
-    assert (err > LIMIT[dtype]).sum() <= max(1, len(err) // 20), sorted(err.tolist())[-12:]
+    return d.pow(2).mean(-1).sqrt() / want.pow(2).mean(-1).sqrt()
+
+
+def rounding(oracle, ids, want, dtype):
+    """What rounding alone does at every position: a norm over values that cancel amplifies it at some of them."""
+    if dtype == "float32":
+        return None
+    errs = []
+    for scale in (1.0, 1.19, 1.41, 1.68):
+        with RoundedProducts(scale):
+            errs.append(error(oracle.forward(ids)[0], want))
+    return torch.stack(errs).amax(0)
+
+
+def off(got, want, dtype, noise=None):
+    err = error(got, want)
+    own = torch.zeros_like(err) if noise is None else 3 * noise
+    assert (err <= own.clamp_min(WORST[dtype])).all(), (float(err.max()), int(err.argmax()))
+    assert (err > own.clamp_min(LIMIT[dtype])).sum() <= max(1, len(err) // 20), sorted(err.tolist())[-12:]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("name", list(CASES))
+@pytest.mark.parametrize("name", list(ALL))
 def test_prefill_portions_and_decode_agree(tmp_path, name, dtype):
     """A prompt in one step, in portions down to two tokens, and token by token through the decode graphs."""
     s, raw, oracle = session_for(tmp_path, name, dtype)
     ids = prompt(raw, 113, 4)
     want, _ = oracle.forward(ids)
+    noise = rounding(oracle, ids, want, dtype)
     for cuts in ([113], [2] * 6 + [101], [16, 17, 80], [50, 1, 1, 60, 1], [1] * 113, [3, 107, 2, 1]):
         got, i = [], 0
         for c in cuts:
             got.append(s.step([("a", ids[i:i + c], list(range(c)))])[0])
             i += c
         s.end(["a"])
-        off(np.concatenate(got), want, dtype)
+        off(np.concatenate(got), want, dtype, noise)
     s.engine.executor.runner.ws.check_status()
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-def test_residual_after_every_run(tmp_path, dtype):
-    s, raw, oracle = session_for(tmp_path, "all", dtype)
+@pytest.mark.parametrize("name, runs", [("all", 6), ("seq", 4)])
+def test_residual_after_every_run(tmp_path, name, runs, dtype):
+    s, raw, oracle = session_for(tmp_path, name, dtype)
     ids = prompt(raw, 40, 9)
     ref = []
     oracle.forward(ids, trace=ref)
     runner = s.engine.executor.runner
     runner.trace = []
     s.step([("a", ids, [])])
-    assert len(runner.trace) == len(ref) == 6
+    assert len(runner.trace) == len(ref) == runs
     for got, want in zip(runner.trace, ref):
         close(got, want, torch.float32, exact=1e-5 if dtype == "float32" else 3e-2)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("name", ["all", "odd"])
+@pytest.mark.parametrize("name", ["all", "odd", "seq", "seq_odd"])
 def test_unequal_requests_share_steps_pages_and_slots(tmp_path, name, dtype):
     """Up to four live requests, portions beside single tokens, requests that pause, end and make room for others in a pool
     that is too small for all of them."""
@@ -445,6 +480,7 @@ def test_unequal_requests_share_steps_pages_and_slots(tmp_path, name, dtype):
     lens = {"a": 100, "b": 37, "c": 1, "d": 60, "e": 90, "f": 33, "g": 16, "h": 130}
     ids = {r: prompt(raw, n, i) for i, (r, n) in enumerate(lens.items())}
     want = {r: oracle.forward(t)[0] for r, t in ids.items()}
+    noise = {r: rounding(oracle, t, want[r], dtype) for r, t in ids.items()}
     at = dict.fromkeys(lens, 0)
     rng = np.random.default_rng(3)
     live, todo = [], list(lens)
@@ -462,7 +498,8 @@ def test_unequal_requests_share_steps_pages_and_slots(tmp_path, name, dtype):
         if not entries:
             continue
         for (r, t, _), got in zip(entries, s.step(entries)):
-            off(got, want[r][at[r]:at[r] + len(t)], dtype)
+            here = slice(at[r], at[r] + len(t))
+            off(got, want[r][here], dtype, None if noise[r] is None else noise[r][here])
             at[r] += len(t)
         pages_seen |= {p for r in live if r in s.engine.requests for p in s.engine.requests[r].pages}
         done = [r for r in live if at[r] == lens[r]]
@@ -474,9 +511,13 @@ def test_unequal_requests_share_steps_pages_and_slots(tmp_path, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-def test_long_decoding_passes_the_window(tmp_path, dtype):
+@pytest.mark.parametrize("raw", [
+    config(90, 64, [latent(4, 16, 16, 32, 48, 70, 0.5, 64), delta(2, 1, 16, 32, 4, 64), latent(3, 16, 16, 32, 40, 17, 0.5, 0)], (0, 2, 2)),
+    sequential(90, 64, [parallel((4, 2, 16, 70, 0.5, 16, 300.0, (3.0, 60, 8.0, 1.0)), (2, 16, 24, 8.0), (1.0, 0.8), 64),
+                        mamba2(2, 24, 16, 1, 4, 2, 48), parallel((3, 1, 24, 17, 0.4, 8, 80.0, None), (1, 20, 16, 4.0), (0.8, 1.1), 0)], 8),
+], ids=["Bumodra", "Loduzen"])
+def test_long_decoding_passes_the_window(tmp_path, raw, dtype):
     """Decoded tokens move every window past the prompt; first tokens of the sequence included."""
-    raw = config(90, 64, [latent(4, 16, 16, 32, 48, 70, 0.5, 64), delta(2, 1, 16, 32, 4, 64), latent(3, 16, 16, 32, 40, 17, 0.5, 0)], (0, 2, 2))
     s, raw, oracle = session_for(tmp_path, "", dtype, raw=raw)
     ids = prompt(raw, 230, 2)
     want, _ = oracle.forward(ids)
@@ -486,13 +527,18 @@ def test_long_decoding_passes_the_window(tmp_path, dtype):
     off(np.concatenate(got), want, dtype)
 
 
-def test_far_token_reaches_through_the_state(tmp_path):
-    """With slow decays and nothing but delta layers, changing a token far back moves the logits as the oracle says."""
-    raw = config(80, 64, [channel(2, 1, 32, 32, 3, 64), delta(2, 2, 32, 32, 4, 64)])
+@pytest.mark.parametrize("raw", [
+    config(80, 64, [channel(2, 1, 32, 32, 3, 64), delta(2, 2, 32, 32, 4, 64)]),
+    sequential(80, 64, [mamba2(2, 32, 24, 2, 3, 1, 64), parallel((2, 1, 16, 9, 0.3, 8, 100.0, None), (2, 24, 24, 16.0), (0.8, 1.5), 64)], 8),
+], ids=["Bumodra", "Loduzen"])
+def test_far_token_reaches_through_the_state(tmp_path, raw):
+    """With slow decays and no attention that far back, changing an early token moves the logits as the oracle says."""
     w = tensors(raw, 3)
     for n in w:
         if n.endswith(".A_log"):
             w[n] = torch.full_like(w[n], -7.0)
+        elif n.endswith(".a2.b"):
+            w[n] = torch.full_like(w[n], 5.0)
     from cubic_serve_b200.runtime.imposed import ImposedSession
     from cubic_serve_b200.utils.trace_run import build_engine
     s = ImposedSession(build_engine(str(write(tmp_path, raw, w)), "float32", 512))
@@ -531,10 +577,13 @@ def serving_backend(model, *flags):
 
 
 @pytest.mark.parametrize("prefix", [False, True])
-def test_greedy_generation_through_the_serving_stack(tmp_path, prefix):
+@pytest.mark.parametrize("raw", [
+    config(300, 64, [delta(2, 1, 16, 16, 3, 64), latent(2, 16, 16, 24, 32, 20, 0.25, 0), channel(2, 2, 16, 16, 2, 48)], (0, 2, 2)),
+    sequential(300, 64, [mamba2(2, 16, 8, 1, 3, 2, 48), parallel((4, 2, 16, 20, 0.3, 8, 90.0, (2.0, 50, 4.0, 1.0)), (2, 12, 16, 8.0), (0.9, 0.8), 64)], 8),
+], ids=["Bumodra", "Loduzen"])
+def test_greedy_generation_through_the_serving_stack(tmp_path, raw, prefix):
     """``cubic serve`` with --dtype float32: scheduler, prefix cache with state snapshots, overlapped decode graphs, sampler."""
     from cubic_serve_b200.runtime.scheduler import SamplingParams
-    raw = config(300, 64, [delta(2, 1, 16, 16, 3, 64), latent(2, 16, 16, 24, 32, 20, 0.25, 0), channel(2, 2, 16, 16, 2, 48)], (0, 2, 2))
     w = tensors(raw, 5)
     eng = serving_backend(write(tmp_path, raw, w), "--dtype", "float32", "--prefix-cache" if prefix else "--no-prefix-cache")
     oracle = R.Oracle(raw, w, torch.float64)
@@ -548,7 +597,8 @@ def test_greedy_generation_through_the_serving_stack(tmp_path, prefix):
     eng.executor.runner.ws.check_status()
 
 
-def test_bf16_serving_samples_and_preempts(tmp_path):
+@pytest.mark.parametrize("name", ["all", "seq"])
+def test_bf16_serving_samples_and_preempts(tmp_path, name):
     """bf16 through the same stack: greedy tokens are the oracle's wherever its margin is clear, seeded sampling repeats, and a
     pool that is too small for all requests recomputes the preempted ones to the same tokens."""
     from cubic_serve_b200.executor.gpu_executor import GpuExecutor
@@ -556,7 +606,7 @@ def test_bf16_serving_samples_and_preempts(tmp_path):
     from cubic_serve_b200.models.checkpoint import admit_checkpoint
     from cubic_serve_b200.runtime.engine import LLMEngine
     from cubic_serve_b200.runtime.scheduler import SamplingParams, SchedulerConfig
-    raw = CASES["all"]
+    raw = ALL[name]
     w = tensors(raw, 6)
     ck = admit_checkpoint(write(tmp_path, raw, w))
     defn = registry.get("layered")
@@ -582,11 +632,12 @@ def test_bf16_serving_samples_and_preempts(tmp_path):
         assert same > 8                                         # recomputed context: equal to rounding
 
 
-def test_trace_run_program(tmp_path):
+@pytest.mark.parametrize("name", ["small", "seq_small"])
+def test_trace_run_program(tmp_path, name):
     """The program itself: lines in, files out, two requests in one step, exit code 0."""
     import json
     import subprocess
-    raw = CASES["small"]
+    raw = ALL[name]
     w = tensors(raw, 2)
     write(tmp_path / "m", raw, w)
     a, b = prompt(raw, 30, 1), prompt(raw, 21, 2)

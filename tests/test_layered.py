@@ -10,7 +10,8 @@ import pytest
 import torch
 
 sys.path.insert(0, str(Path(__file__).parent))
-from layered_cases import CASES, LOW_RANKS, channel, config, delta, latent, prompt, tensors, write  # noqa: E402
+from layered_cases import (ALL, CASES, LOW_RANKS, SEQUENTIAL, channel, config, delta, latent, mamba2, parallel,  # noqa: E402
+                           prompt, sequential, tensors, write)
 
 from cubic_serve_b200.models import layered as L  # noqa: E402
 from cubic_serve_b200.models import layered_reference as R  # noqa: E402
@@ -18,21 +19,21 @@ from cubic_serve_b200.models.checkpoint import CheckpointError, admit_checkpoint
 
 
 def parsed(name):
-    w = tensors(CASES[name])
-    return L.parse_layered_config(CASES[name], {n: tuple(t.shape) for n, t in w.items()}), w
+    w = tensors(ALL[name])
+    return L.parse_layered_config(ALL[name], {n: tuple(t.shape) for n, t in w.items()}), w
 
 
 # ------------------------------------------------------------------ configuration and inventory
-@pytest.mark.parametrize("name", list(CASES))
+@pytest.mark.parametrize("name", list(ALL))
 def test_config_and_inventory(name):
     cfg, w = parsed(name)
     L.check_inventory(cfg, {n: tuple(t.shape) for n, t in w.items()})
     back = L.parse_layered_config(cfg.to_config(), {n: tuple(t.shape) for n, t in w.items()}, name=cfg.name)
     assert back == cfg
-    loop = CASES[name]["loop"]
+    loop = ALL[name].get("loop")
     runs = len(cfg.layers) + ((loop["times"] - 1) * (loop["stop"] - loop["start"]) if loop else 0)
-    assert len(cfg.runs) == runs == len(R.layer_schedule(CASES[name]))
-    assert [i for i, _ in cfg.runs] == [i for i, _ in R.layer_schedule(CASES[name])]
+    assert len(cfg.runs) == runs == len(R.layer_schedule(ALL[name]))
+    assert [i for i, _ in cfg.runs] == [i for i, _ in R.layer_schedule(ALL[name])]
     assert sum(enters for _, enters in cfg.runs) == (loop["times"] if loop else 0)
 
 
@@ -58,6 +59,56 @@ def test_bad_configurations_are_refused(change, message):
     change(c)
     with pytest.raises(L.LayeredConfigError, match=message):
         L.parse_layered_config(c, {n: tuple(t.shape) for n, t in tensors(CASES["all"]).items()})
+
+
+@pytest.mark.parametrize("change, message", [
+    (lambda c: c["layers"][0].update(type="delta"), "unknown mixer"),
+    (lambda c: c["layers"][0]["mixer"]["left"].update(vdim=8), "values of this attention are its keys"),
+    (lambda c: c["layers"][0]["mixer"]["left"].update(kv_heads=4), "grouped evenly"),
+    (lambda c: c["layers"][0]["mixer"]["left"]["rot"].update(dims=26), "inside a head"),
+    (lambda c: c["layers"][0]["mixer"]["left"].update(mask={"size": 0}), "at least the token itself"),
+    (lambda c: c["layers"][0]["mixer"]["right"].update(tau=0), "tau are positive"),
+    (lambda c: c["layers"][1]["mixer"].update(norm_groups=5), "cut evenly"),
+    (lambda c: c["layers"][1]["mixer"].update(groups=3), "grouped evenly"),
+    (lambda c: c["layers"][1]["mixer"].update(state=300), "state width"),
+    (lambda c: c.update(loop={"start": 0, "stop": 1, "times": 2}), "run once"),
+])
+def test_bad_sequential_configurations_are_refused(change, message):
+    c = copy.deepcopy(SEQUENTIAL["seq"])
+    change(c)
+    with pytest.raises(L.LayeredConfigError, match=message):
+        L.parse_layered_config(c, {n: tuple(t.shape) for n, t in tensors(SEQUENTIAL["seq"]).items()})
+
+
+def test_sequential_checkpoint_admission(tmp_path):
+    from cubic_serve_b200.contracts.model import ModelSpec
+    from cubic_serve_b200.contracts.plan import decoder_step_operators
+    from cubic_serve_b200.models import registry
+    raw, w = SEQUENTIAL["seq"], tensors(SEQUENTIAL["seq"])
+    ck = admit_checkpoint(write(tmp_path / "good", raw, w))
+    assert ck.cfg.family == "layered" and registry.for_architecture("Loduzen").family == "layered" and ck.cfg.side_dim == 12
+    info = inspect_checkpoint(tmp_path / "good")
+    assert info["mixers"] == {"attention+gated_linear": 2, "mamba2": 2} and info["architecture"] == "Loduzen"
+    # a second norm without a feed-forward behind it is tolerated, anything else is not
+    admit_checkpoint(write(tmp_path / "spare", raw, {**w, "l2.norm2": w["l1.norm2"].clone()}))
+    with pytest.raises(CheckpointError, match="does not own"):
+        admit_checkpoint(write(tmp_path / "head", raw, {**w, "head": w["embed"].clone()}))
+    with pytest.raises(CheckpointError, match="missing tensor side.embed"):
+        admit_checkpoint(write(tmp_path / "missing", raw, {n: t for n, t in w.items() if n != "side.embed"}))
+    # caches and states of the parts: 2 attentions (keys and values of 64 padded channels), 2 gated linear and 2 mamba2 states
+    spec = ModelSpec.from_layered(ck.cfg)
+    assert spec.cache.runs == 2 and spec.state.runs == 4 and spec.cache.page_bytes == (2 + 4) * 2 * 16 * 64 * 2
+    conv = (3 * (96 + 80) + 2 * (80 + 32)) * 2
+    assert ck.cfg.state_bytes_per_request == 4 * (3 * 28 * 20 + 2 * 16 * 32 + 4 * 24 * 20 + 2 * 40 * 16) + conv
+    assert {o.semantic_op for o in decoder_step_operators(ck.cfg, 8)} >= {"attention.gqa", "linear_recurrence.head",
+                                                                          "linear_recurrence.channel", "token_side"}
+
+
+def test_random_weights_of_both_designs_are_admitted(tmp_path):
+    for name in ("layered-tiny", "layered-seq-tiny"):
+        cfg = L.NAMED[name]()
+        back = admit_checkpoint(L.write_checkpoint(tmp_path / name, cfg, L.random_tensors(cfg, 3))).cfg
+        assert (back.layers, back.side_dim, back.loop) == (cfg.layers, cfg.side_dim, cfg.loop)
 
 
 def test_checkpoint_admission(tmp_path):
@@ -129,7 +180,113 @@ def test_projection_sections_are_aligned_and_complete():
                 assert off % 8 == 0 and torch.equal(rows[off:off + t.shape[0]], t.float())
 
 
+def test_sequential_packing():
+    """Sections of the joint projection and of the joint output product, gated rows in the GEMM's order, folded scales."""
+    from cubic_serve_b200.ops import wq_pack
+    cfg, w = parsed("seq")
+    W = cfg.hidden_size
+    p = L.pack_layer(cfg, 0, w.__getitem__)
+    left, right = p.mixer.left, p.mixer.right
+    rows = p.proj.codes.float()[:, :W]
+    for name, off in (("left.q", left.q_off), ("left.k", left.k_off), ("right.q", right.q_off), ("right.k", right.k_off),
+                      ("right.v", right.v_off), ("right.g", right.g_off), ("right.a1", right.a_off)):
+        t = w[f"l0.mix.{name}"]
+        assert off % 8 == 0 and torch.equal(rows[off:off + t.shape[0]], t.float())
+    assert right.a_off + right.low.k <= p.split == p.proj.n and p.ff == 0
+    out = p.out.codes.float()
+    assert torch.equal(out[:, :144], w["l0.mix.left.o"].float()) and torch.equal(out[:, 144:228], w["l0.mix.right.o"].float())
+    assert left.out_scale == 0.7 and torch.allclose(right.norm_w, 1.3 * w["l0.mix.right.norm"].float())
+    assert torch.equal(p.norm, w["l0.norm1"].float()) and torch.equal(p.norm2, w["l0.norm2"].float())
+    order = wq_pack.swiglu_row_order(80)
+    both = torch.cat([w["l0.mlp.gate"], w["l0.mlp.up"]]).float()
+    assert torch.equal(p.gate_up.codes.float()[:, :W], both[order]) and p.gate_up.act_interleaved
+    assert torch.equal(p.down.codes.float()[:, :80], w["l0.mlp.down"].float()) and p.down.k == 128
+    assert p.side.col == 0 and L.pack_layer(cfg, 3, w.__getitem__).side.col == 36
+    m = L.pack_layer(cfg, 1, w.__getitem__)
+    rows, s = m.proj.codes.float()[:, :W], m.mixer
+    for off, (a, b) in ((s.z_off, (0, 96)), (s.x_off, (96, 96 + 176)), (s.dt_off, (272, 276))):
+        assert off % 8 == 0 and torch.equal(rows[off:off + b - a], w["l1.mix.in"].float()[a:b])
+    assert torch.equal(s.conv_w[:, :176].t(), w["l1.mix.conv"].float()) and (s.conv_w[:, 176:] == 0).all()
+    # a feed-forward width that is no multiple of the activation's block gets zero features
+    odd, wo = parsed("seq_odd")
+    q = L.pack_layer(odd, 0, wo.__getitem__)
+    assert q.gate_up.n == 96 and q.down.k == 64 and (q.down.codes.float()[:, 44:] == 0).all()
+    assert L.pack_layer(cfg, 2, w.__getitem__).down is None
+    packed = L.pack_weights(cfg, w.__getitem__)
+    assert torch.equal(packed.lm_head.codes.float()[:, :W], w["embed"].float()) and packed.embed_norm is None
+
+
 # ------------------------------------------------------------------ the oracle's mechanisms, against element-wise loops
+def test_rotary_table_equals_the_oracle():
+    """Frequencies of the product and of the oracle, stretched and plain; the ramp's ends, also where it has no width."""
+    for raw in (*SEQUENTIAL.values(),):
+        for l in raw["layers"]:
+            if l["type"] == "parallel":
+                rot = l["mixer"]["left"]["rot"]
+                f, mult = L._read_rotary(rot).table()
+                g, m2 = R.rotary_frequencies(rot)
+                assert torch.allclose(f.double(), g, rtol=1e-7) and abs(mult - m2) < 1e-12
+    for fast, slow in ((32, 1), (1, 1), (1000, 0.001), (0.01, 0.001), (5000, 4000)):
+        rot = {"dims": 16, "base": 700.0, "scaling": {"factor": 5.0, "original": 90, "fast": fast, "slow": slow}}
+        f, _ = L._read_rotary(rot).table()
+        g, _ = R.rotary_frequencies(rot)
+        assert torch.allclose(f.double(), g, rtol=1e-7), (fast, slow)
+        plain = torch.tensor([700.0 ** (-i / 8) for i in range(8)], dtype=torch.float64)
+        ratio = g / plain
+        assert ((ratio <= 1 + 1e-12) & (ratio >= 0.2 - 1e-12)).all() and (ratio[1:] <= ratio[:-1] + 1e-12).all()
+
+
+def test_oracle_rotation_and_sink():
+    x = torch.randn(4, 2, 7, dtype=torch.float64)
+    freq = torch.tensor([0.9, 0.05], dtype=torch.float64)
+    y = R.rotate_pairs(x, 5, freq, 1.3)
+    for t in range(4):
+        for h in range(2):
+            for i in range(2):
+                a = (5 + t) * float(freq[i])
+                u, v = float(x[t, h, 2 * i]), float(x[t, h, 2 * i + 1])
+                assert abs(float(y[t, h, 2 * i]) - 1.3 * (u * np.cos(a) - v * np.sin(a))) < 1e-12
+                assert abs(float(y[t, h, 2 * i + 1]) - 1.3 * (v * np.cos(a) + u * np.sin(a))) < 1e-12
+    assert torch.equal(y[:, :, 4:], x[:, :, 4:])
+    q, k, v = torch.randn(6, 4, 3), torch.randn(6, 2, 3), torch.randn(6, 2, 5)
+    o = R.sink_attention(q, k, v, 0, 3, 0.8)
+    for i in range(6):
+        for h in range(4):
+            js = [j for j in range(6) if 0 <= i - j < 3]
+            e = [np.exp(0.8 * float(q[i, h] @ k[j, h // 2])) for j in js]
+            want = sum(w * v[j, h // 2] for w, j in zip(e, js)) / (1 + sum(e))
+            assert torch.allclose(o[i, h], want, atol=1e-5)
+
+
+def test_oracle_linear_step_and_parts_norm():
+    H, d, e = 2, 3, 4
+    S, q, k, v, decay = torch.randn(H, d, e), torch.randn(H, d), torch.randn(H, d), torch.randn(H, e), torch.rand(H, d)
+    o, S2 = R.linear_step(S, q, k, v, decay)
+    for h in range(H):
+        for j in range(e):
+            col = [float(decay[h, i] * S[h, i, j] + k[h, i] * v[h, j]) for i in range(d)]
+            assert np.allclose(col, S2[h, :, j].numpy(), atol=1e-5)
+            assert abs(sum(c * float(q[h, i]) for i, c in enumerate(col)) - float(o[h, j])) < 1e-5
+    y, z, w = torch.randn(2, 6, dtype=torch.float64), torch.randn(2, 6, dtype=torch.float64), torch.randn(6, dtype=torch.float64)
+    out = R.gated_parts_norm(y, z, w, 3, 0.01)
+    for t in range(2):
+        u = [float(y[t, c] * z[t, c]) / (1 + np.exp(-float(z[t, c]))) for c in range(6)]
+        for c in range(6):
+            part = u[c // 2 * 2:c // 2 * 2 + 2]
+            assert abs(float(out[t, c]) - u[c] / (sum(p * p for p in part) / 2 + 0.01) ** 0.5 * float(w[c])) < 1e-9
+    x = torch.linspace(-4, 4, 9, dtype=torch.float64)
+    assert torch.allclose(R.gelu_tanh(x), torch.nn.functional.gelu(x, approximate="tanh"))
+
+
+def test_oracle_convolution_bias():
+    x, w, b = torch.randn(5, 3), torch.randn(3, 2), torch.randn(3)
+    y, past = R.short_conv(x, w, torch.zeros(1, 3), b)
+    for t in range(5):
+        s = b + w[:, 1] * x[t] + (w[:, 0] * x[t - 1] if t else 0)
+        assert torch.allclose(y[t], s / (1 + torch.exp(-s)), atol=1e-6)
+    assert torch.equal(past, x[4:])
+
+
 def test_oracle_norms_and_activations():
     x, w = torch.randn(3, 5, dtype=torch.float64), torch.randn(5, dtype=torch.float64)
     for r in range(3):
@@ -187,10 +344,10 @@ def test_oracle_window_edges(window):
             assert [i for i in range(n) if moved[i]] == [i for i in seen if i >= first]
 
 
-@pytest.mark.parametrize("name", list(CASES))
+@pytest.mark.parametrize("name", list(ALL))
 def test_oracle_portions_equal_one_pass(name):
-    o = R.Oracle(CASES[name], tensors(CASES[name]), torch.float64)
-    ids = prompt(CASES[name], 61, 0)
+    o = R.Oracle(ALL[name], tensors(ALL[name]), torch.float64)
+    ids = prompt(ALL[name], 61, 0)
     whole, _ = o.forward(ids)
     for cuts in ([1] * 61, [2, 2, 57], [40, 1, 20], [16, 16, 16, 13]):
         st, parts, i = None, [], 0
@@ -321,9 +478,12 @@ def backend_of(args, tp=1):
     return build_backend(args, list(range(tp)), tp, parse_speculative_config(args.speculative_config), 8, 8)
 
 
-def test_eager_mode_generates_like_the_oracle(tmp_path):
+@pytest.mark.parametrize("raw", [
+    config(300, 64, [delta(2, 1, 16, 16, 3, 64), latent(2, 16, 16, 24, 32, 20, 0.25, 0), channel(2, 2, 16, 16, 2, 48)], (0, 2, 2)),
+    sequential(300, 64, [mamba2(2, 16, 8, 1, 3, 2, 48), parallel((4, 2, 16, 20, 0.3, 8, 90.0, (2.0, 50, 4.0, 1.0)), (2, 12, 16, 8.0), (0.9, 0.8), 64)], 8),
+], ids=["Bumodra", "Loduzen"])
+def test_eager_mode_generates_like_the_oracle(tmp_path, raw):
     from cubic_serve_b200.runtime.scheduler import SamplingParams
-    raw = config(300, 64, [delta(2, 1, 16, 16, 3, 64), latent(2, 16, 16, 24, 32, 20, 0.25, 0), channel(2, 2, 16, 16, 2, 48)], (0, 2, 2))
     w = tensors(raw, 5)
     backend, _ = backend_of(serve_args(write(tmp_path, raw, w), "--execution-mode", "eager", "--prefill-chunk-tokens", "16",
                                        "--token-budget", "32"))
