@@ -175,6 +175,12 @@ gqa_row_kernel(const GqaAttn<float> p) {
 // ------------------------------------------------------------------ bf16, prompts and mixed steps
 using bf16 = __nv_bfloat16;
 
+__device__ __forceinline__ float ex2(float x) {       // 2^x, zero for -inf
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+
 struct GqaMma {
   GqaAttn<bf16> a;
   int hb, qb;                 // heads and tokens of a block (hb * qb rows at most)
@@ -192,15 +198,17 @@ __device__ __forceinline__ void store_pair(bf16* row, int c, int d, float x, flo
   }
 }
 
-// NW warps of 16 rows each, row = token * hb + head; key tiles of 64 keys in two buffers, 16-byte chunks XOR-swizzled by the row.
-// A warp keeps its rows' scores, weights and outputs in registers: no exchange between warps.
-template <int NW, int NCH>
-__global__ void __launch_bounds__(32 * NW)
+// Four warps of 16 rows each, row = token * hb + head; key tiles of 64 keys in two buffers, 16-byte chunks XOR-swizzled by the
+// row.  A warp keeps its rows' scores, weights and outputs in registers: no exchange between warps.
+static constexpr int kGqaWarps = 4;
+template <int NCH>
+__global__ void __launch_bounds__(32 * kGqaWarps, NCH <= 2 ? 3 : 1)
 gqa_prefill_kernel(const GqaMma p) {
-  constexpr int P = NCH * 64, ROWB = P * 2, MR = 16 * NW, KT = 64, CH = P / 8, NT = P / 8;
+  constexpr int P = NCH * 64, ROWB = P * 2, NW = kGqaWarps, MR = 16 * NW, KT = 64, CH = P / 8, NT = P / 8;
   extern __shared__ __align__(128) uint8_t lsm[];
-  uint8_t* qs = lsm;                                  // [MR][ROWB]
-  uint8_t* kvs = qs + MR * ROWB;                      // [2 buffers][key, value][KT][ROWB]
+  constexpr bool QREG = NCH <= 2;                     // query fragments in registers; the rows pass through the second buffer
+  uint8_t* kvs = lsm + (QREG ? 0 : MR * ROWB);        // [2 buffers][key, value][KT][ROWB]
+  uint8_t* qs = QREG ? kvs + 2 * KT * ROWB : lsm;     // [MR][ROWB]
   pdl_wait();
   pdl_launch_dependents();
   const GqaAttn<bf16>& a = p.a;
@@ -272,6 +280,14 @@ gqa_prefill_kernel(const GqaMma p) {
     k_at[i] = ((lane & 7) + ((lane >> 4) << 3)) * ROWB + (((i * 2 + ((lane >> 3) & 1)) ^ (lane & 7)) << 4);
     v_at[i] = (lane & 15) * ROWB + (((i * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
   }
+  uint32_t qr[QREG ? P / 16 : 1][4];
+  if constexpr (QREG) {
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < P / 16; ++kk) ldsm4(qr[kk], q_at[kk & 3] + (kk >> 2) * 128);
+    __syncthreads();
+  }
   for (int t = 0; t < tiles; ++t) {
     const int b = t & 1;
     if (t + 1 < tiles) load_tile(t + 1, b ^ 1);       // its buffer was released by the barrier that ended the last turn
@@ -289,7 +305,8 @@ gqa_prefill_kernel(const GqaMma p) {
 #pragma unroll
       for (int kk = 0; kk < P / 16; ++kk) {
         uint32_t qa[4];
-        ldsm4(qa, q_at[kk & 3] + (kk >> 2) * 128);
+        if constexpr (QREG) { qa[0] = qr[kk][0]; qa[1] = qr[kk][1]; qa[2] = qr[kk][2]; qa[3] = qr[kk][3]; }
+        else ldsm4(qa, q_at[kk & 3] + (kk >> 2) * 128);
 #pragma unroll
         for (int j = 0; j < 8; j += 2) {
           uint32_t cb[4];
@@ -314,7 +331,7 @@ gqa_prefill_kernel(const GqaMma p) {
         mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
         mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
         use[i] = mx[i] == -INFINITY ? 0.f : mx[i];
-        al[i] = exp2f(m2[i] - use[i]);
+        al[i] = ex2(m2[i] - use[i]);
         m2[i] = mx[i];
         l2[i] *= al[i];
       }
@@ -322,7 +339,7 @@ gqa_prefill_kernel(const GqaMma p) {
       for (int j = 0; j < 8; ++j)
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          sf[j][c] = exp2f(sf[j][c] - use[c >> 1]);
+          sf[j][c] = ex2(sf[j][c] - use[c >> 1]);
           l2[c >> 1] += sf[j][c];
         }
 #pragma unroll
@@ -350,7 +367,7 @@ gqa_prefill_kernel(const GqaMma p) {
     const int r = warp * 16 + g + 8 * i;
     const int tok = r / p.hb, h = r - tok * p.hb;
     if (tok >= toks || h >= heads) continue;
-    const float f = a.out_scale / (l2[i] + exp2f(a.sink * kLog2e - m2[i]));
+    const float f = a.out_scale / (l2[i] + ex2(a.sink * kLog2e - m2[i]));
     bf16* row = a.out + (row0 + tok) * a.ldo + (h0 + h) * a.d;
 #pragma unroll
     for (int j = 0; j < NT; ++j) store_pair(row, j * 8 + 2 * t4, a.d, o[j][2 * i] * f, o[j][2 * i + 1] * f);
@@ -449,7 +466,7 @@ gqa_decode_kernel(const GqaMma p) {
       mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
       mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
       use[i] = mx[i] == -INFINITY ? 0.f : mx[i];
-      al[i] = exp2f(m2[i] - use[i]);
+      al[i] = ex2(m2[i] - use[i]);
     }
     if (__any_sync(0xffffffffu, mx[0] > m2[0] || mx[1] > m2[1])) {
 #pragma unroll
@@ -464,7 +481,7 @@ gqa_decode_kernel(const GqaMma p) {
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        sf[j][c] = exp2f(sf[j][c] - use[c >> 1]);
+        sf[j][c] = ex2(sf[j][c] - use[c >> 1]);
         l2[c >> 1] += sf[j][c];
       }
     const uint32_t pa[4] = {pack_bf16x2(sf[0][0], sf[0][1]), pack_bf16x2(sf[0][2], sf[0][3]), pack_bf16x2(sf[1][0], sf[1][1]),
@@ -504,11 +521,11 @@ gqa_decode_kernel(const GqaMma p) {
     const float use = mx == -INFINITY ? 0.f : mx;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
-      f[w] = exp2f(res[(w * 16 + r) * LD + P] - use);
+      f[w] = ex2(res[(w * 16 + r) * LD + P] - use);
       l += f[w] * res[(w * 16 + r) * LD + P + 1];
     }
     float* part = p.partial + ((unit * p.splits + blockIdx.z) * 16 + r) * LD;
-    const float scale = p.splits > 1 ? 1.f : a.out_scale / (l + exp2f(a.sink * kLog2e - use));
+    const float scale = p.splits > 1 ? 1.f : a.out_scale / (l + ex2(a.sink * kLog2e - use));
 #pragma unroll
     for (int i = 0; i < P / 64; ++i) {
       const int c = 2 * (lane + 32 * i);
@@ -543,12 +560,12 @@ gqa_merge_kernel(const GqaMma p) {
   constexpr int step = 16 * LD;
   float mx = a.sink * kLog2e;
   for (int z = 0; z < p.splits; ++z) mx = fmaxf(mx, part[z * step + P]);
-  float l = exp2f(a.sink * kLog2e - mx);
+  float l = ex2(a.sink * kLog2e - mx);
   float2 v[NCH];
 #pragma unroll
   for (int i = 0; i < NCH; ++i) v[i] = make_float2(0.f, 0.f);
   for (int z = 0; z < p.splits; ++z) {
-    const float f = exp2f(part[z * step + P] - mx);   // 0 for a split that saw no key
+    const float f = ex2(part[z * step + P] - mx);   // 0 for a split that saw no key
     l += f * part[z * step + P + 1];
 #pragma unroll
     for (int i = 0; i < NCH; ++i) {
@@ -576,10 +593,11 @@ static int gqa_go(K kernel, dim3 grid, int threads, size_t smem, const GqaMma& p
   return static_cast<int>(launch(kernel, grid, dim3(threads), smem, st, p));
 }
 
-template <int NW, int NCH>
+template <int NCH>
 static int gqa_prefill(const GqaMma& p, dim3 grid, cudaStream_t st) {
   static bool configured[64] = {};
-  return gqa_go(gqa_prefill_kernel<NW, NCH>, grid, 32 * NW, static_cast<size_t>(16 * NW + 256) * NCH * 128, p, configured, st);
+  return gqa_go(gqa_prefill_kernel<NCH>, grid, 32 * kGqaWarps, static_cast<size_t>((NCH <= 2 ? 0 : 16 * kGqaWarps) + 256) * NCH * 128, p,
+                configured, st);
 }
 
 template <int NCH>
@@ -588,18 +606,6 @@ static int gqa_decode(const GqaMma& p, dim3 grid, cudaStream_t st) {
   const int rc = gqa_go(gqa_decode_kernel<NCH>, grid, 128, static_cast<size_t>(4) * kRing * 2 * kGqaPage * NCH * 128, p, configured, st);
   if (rc || p.splits == 1) return rc;
   return static_cast<int>(launch(gqa_merge_kernel<NCH>, dim3(grid.x, grid.y, 4), dim3(128), 0, st, p));
-}
-
-// Rows of a block of the prompt form: 128 when the step then still has enough blocks, else 64.
-static void gqa_shape(int tokens, int segs, int H, int G, int& nw, int& hb, int& qb, int& head_tiles) {
-  const int R = H / G;
-  for (nw = 8; nw >= 4; nw -= 4) {
-    hb = R < 16 * nw ? R : 16 * nw;
-    qb = 16 * nw / hb;
-    head_tiles = (R + hb - 1) / hb;
-    if (static_cast<long long>(max_tiles(tokens, segs, qb)) * G * head_tiles >= 296) return;
-  }
-  nw = 4;
 }
 
 }  // namespace cb
@@ -705,20 +711,18 @@ int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
     }
     return gqa_decode<4>(p, grid, st);
   }
-  int nw;
-  gqa_shape(a->tokens, seg->num, a->H, a->G, nw, p.hb, p.qb, p.head_tiles);
+  const int R = a->H / a->G;
+  p.hb = min(R, 16 * kGqaWarps);
+  p.qb = 16 * kGqaWarps / p.hb;
+  p.head_tiles = (R + p.hb - 1) / p.hb;
   const dim3 grid(max_tiles(a->tokens, seg->num, p.qb), a->G * p.head_tiles);
   if (grid.y > 65535) return -11;
-  switch (a->P / 64 * 10 + nw) {
-    case 14: return gqa_prefill<4, 1>(p, grid, st);
-    case 18: return gqa_prefill<8, 1>(p, grid, st);
-    case 24: return gqa_prefill<4, 2>(p, grid, st);
-    case 28: return gqa_prefill<8, 2>(p, grid, st);
-    case 34: return gqa_prefill<4, 3>(p, grid, st);
-    case 38: return gqa_prefill<8, 3>(p, grid, st);
-    case 44: return gqa_prefill<4, 4>(p, grid, st);
+  switch (a->P / 64) {
+    case 1: return gqa_prefill<1>(p, grid, st);
+    case 2: return gqa_prefill<2>(p, grid, st);
+    case 3: return gqa_prefill<3>(p, grid, st);
   }
-  return gqa_prefill<8, 4>(p, grid, st);
+  return gqa_prefill<4>(p, grid, st);
 }
 
 }  // extern "C"

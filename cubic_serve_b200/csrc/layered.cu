@@ -300,7 +300,10 @@ side_gate_mma_kernel(const SideGate p) {
     float z = 0.f;
     if (cluster > 1) {
       const uint32_t at = smem_u32(&part[0][r][n]);
-      for (int c = 0; c < cluster; ++c) z += ld_cluster_f32(cluster_map(at, c));
+      float v[8];
+#pragma unroll
+      for (int c = 0; c < 8; ++c) v[c] = c < cluster ? ld_cluster_f32(cluster_map(at, c)) : 0.f;
+      z = ((v[0] + v[1]) + (v[2] + v[3])) + ((v[4] + v[5]) + (v[6] + v[7]));
     } else {
 #pragma unroll
       for (int w = 0; w < kSideWarps; ++w) z += part[w][r][n];
@@ -331,6 +334,244 @@ side_gate_f32_kernel(const SideGate p) {
       static_cast<float*>(p.out)[t * p.ldo + n] =
           gelu_tanh(z) * __bfloat162float(p.table[static_cast<size_t>(id) * p.ldt + p.col + n]);
   }
+}
+
+// ------------------------------------------------------------------ a layer's whole side input in one kernel
+// g = gelu_tanh(x Wg) e;  y = g Wp;  x += y * norm_w / rms(y);  h = x * next_w / rms(x)   (bf16 models, up to 64 side channels)
+// A cluster takes 16 tokens, each of its blocks a slice of 64 NTW columns of x: the slices' partial gates and the two row sums of
+// squares meet through distributed shared memory, everything else stays in registers and x passes through once.
+struct SideInput {
+  SideGate s;
+  float* x;                               // the gate's input, written back
+  const __nv_bfloat16* proj; int ldp;     // [W, ldp], zero columns behind dim
+  const float* norm_w;
+  const float* next_w;                    // null: no h
+  __nv_bfloat16* h; int ldh;
+  float eps;
+};
+
+template <int NB, int NTW>
+__global__ void __launch_bounds__(32 * kSideWarps, 2)
+side_input_kernel(const SideInput p) {
+  constexpr int KC = (NB * 8 + 31) / 32, LDG = 32 * KC + 8;
+  __shared__ float part[kSideWarps][16][NB * 8 + 1];
+  __shared__ __align__(16) __nv_bfloat16 gs[16][LDG];
+  __shared__ float red[kSideWarps][16], sums[2][16], total[16];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+  const int t0 = blockIdx.x * 16, W = p.s.W, T = p.s.T, cluster = gridDim.z;
+  const int c_lo = blockIdx.z * 64 * NTW;
+  // the slice's weights on their way into L2 while the kernel before this one ends
+  for (int i = threadIdx.x; i < 64 * NTW * KC / 2; i += 32 * kSideWarps) {        // a row of the projection is 64 KC bytes
+    const int n = c_lo + (KC == 1 ? 2 * i : i);
+    if (n < W) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.proj + static_cast<size_t>(n) * p.ldp));
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  // a thread's share of the gates, two neighbouring ones at a time, and their factors from the side embedding
+  constexpr int PAIRS = 16 * NB * 4, ITER = (PAIRS + 32 * kSideWarps - 1) / (32 * kSideWarps);
+  const int share = PAIRS / cluster;                       // PAIRS and the cluster are powers of two
+  float e[ITER][2];
+#pragma unroll
+  for (int it = 0; it < ITER; ++it) {
+    const int i = threadIdx.x + it * 32 * kSideWarps, idx = blockIdx.z * share + i, t = t0 + idx / (NB * 4), n = 2 * (idx % (NB * 4));
+    e[it][0] = e[it][1] = 0.f;
+    if (i < share && t < T) {
+      const __nv_bfloat16* er = p.s.table + static_cast<size_t>(min(max(p.s.ids[t], 0), p.s.vocab - 1)) * p.s.ldt + p.s.col;
+      if (n < p.s.dim) e[it][0] = __bfloat162float(er[n]);
+      if (n + 1 < p.s.dim) e[it][1] = __bfloat162float(er[n + 1]);
+    }
+  }
+  auto meet = [&]() {                     // barrier of everybody who works on the tokens
+    __syncwarp();
+    if (cluster > 1) cluster_sync_all();
+    else __syncthreads();
+  };
+  // ---- partial gates of this slice
+  {
+    float acc[NB][4] = {};
+#pragma unroll
+    for (int j = 0; j < 2 * NTW / kSideWarps; ++j) {
+      const int ch = warp + j * kSideWarps;
+      const int k = c_lo + ch * 32 + 8 * t4;               // W is a multiple of 8: all of a lane's columns exist, or none
+      float a[2][8];
+      uint4 b[NB];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        float4 u = make_float4(0.f, 0.f, 0.f, 0.f), v = u;
+        if (t0 + g + 8 * i < T && k < W) {
+          const float* xr = p.x + static_cast<size_t>(t0 + g + 8 * i) * W + k;
+          u = *reinterpret_cast<const float4*>(xr);
+          v = *reinterpret_cast<const float4*>(xr + 4);
+        }
+        a[i][0] = u.x; a[i][1] = u.y; a[i][2] = u.z; a[i][3] = u.w;
+        a[i][4] = v.x; a[i][5] = v.y; a[i][6] = v.z; a[i][7] = v.w;
+      }
+#pragma unroll
+      for (int n = 0; n < NB; ++n)
+        b[n] = n * 8 + g < p.s.dim && k < W ? *reinterpret_cast<const uint4*>(p.s.w + static_cast<size_t>(n * 8 + g) * p.s.ldw + k)
+                                            : make_uint4(0, 0, 0, 0);
+      const uint32_t a0[4] = {pack_bf16x2(a[0][0], a[0][1]), pack_bf16x2(a[1][0], a[1][1]), pack_bf16x2(a[0][2], a[0][3]), pack_bf16x2(a[1][2], a[1][3])};
+      const uint32_t a1[4] = {pack_bf16x2(a[0][4], a[0][5]), pack_bf16x2(a[1][4], a[1][5]), pack_bf16x2(a[0][6], a[0][7]), pack_bf16x2(a[1][6], a[1][7])};
+#pragma unroll
+      for (int n = 0; n < NB; ++n) {
+        mma_bf16(acc[n], a0, b[n].x, b[n].y);
+        mma_bf16(acc[n], a1, b[n].z, b[n].w);
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < NB; ++n)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) part[warp][g + 8 * (c >> 1)][n * 8 + 2 * t4 + (c & 1)] = acc[n][c];
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < 16 * NB * 8; i += 32 * kSideWarps) {
+    const int r = i / (NB * 8), n = i % (NB * 8);
+    float z = 0.f;
+#pragma unroll
+    for (int w = 0; w < kSideWarps; ++w) z += part[w][r][n];
+    part[0][r][n] = z;
+  }
+  meet();
+  // every block finishes its share of the gates and hands them to all of the cluster
+  {
+#pragma unroll
+    for (int it = 0; it < ITER; ++it) {
+      const int i = threadIdx.x + it * 32 * kSideWarps, idx = blockIdx.z * share + i, r = idx / (NB * 4), n = 2 * (idx % (NB * 4));
+      if (i >= share) break;
+      float v[2][8];
+      const uint32_t at = smem_u32(&part[0][r][n]);
+#pragma unroll
+      for (int c = 0; c < 8; ++c) {                        // all in flight at once
+        const bool there = cluster > 1 && c < cluster;
+        v[0][c] = there ? ld_cluster_f32(cluster_map(at, c)) : 0.f;
+        v[1][c] = there ? ld_cluster_f32(cluster_map(at, c) + 4) : 0.f;
+      }
+      float z[2];
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        z[k] = cluster > 1 ? ((v[k][0] + v[k][1]) + (v[k][2] + v[k][3])) + ((v[k][4] + v[k][5]) + (v[k][6] + v[k][7])) : part[0][r][n + k];
+        z[k] = gelu_tanh_fast(z[k]) * e[it][k];
+      }
+      const uint32_t both = pack_bf16x2(z[0], z[1]), dst = smem_u32(&gs[r][n]);
+      if (cluster > 1)
+        for (int c = 0; c < cluster; ++c) st_cluster_u32(cluster_map(dst, c), both);
+      else
+        *reinterpret_cast<uint32_t*>(&gs[r][n]) = both;
+    }
+    if constexpr (NB * 8 < 32 * KC) {                      // columns behind the gates
+      constexpr int REST = 32 * KC - NB * 8;
+      for (int i = threadIdx.x; i < 16 * REST; i += 32 * kSideWarps) gs[i / REST][NB * 8 + i % REST] = __float2bfloat16(0.f);
+    }
+  }
+  meet();
+  // ---- y of this slice: a warp's 8 NTW columns in registers
+  uint4 ga[KC][2];
+#pragma unroll
+  for (int c = 0; c < KC; ++c)
+#pragma unroll
+    for (int i = 0; i < 2; ++i) ga[c][i] = *reinterpret_cast<const uint4*>(&gs[g + 8 * i][32 * c + 8 * t4]);
+  const int c_w = c_lo + warp * 8 * NTW;
+  float y[NTW][4], ss[2] = {0.f, 0.f};
+#pragma unroll
+  for (int j = 0; j < NTW; ++j) {
+    const int n = c_w + 8 * j + g;
+#pragma unroll
+    for (int c = 0; c < 4; ++c) y[j][c] = 0.f;
+#pragma unroll
+    for (int c = 0; c < KC; ++c) {
+      const uint4 b = n < W ? *reinterpret_cast<const uint4*>(p.proj + static_cast<size_t>(n) * p.ldp + 32 * c + 8 * t4) : make_uint4(0, 0, 0, 0);
+      const uint32_t a0[4] = {ga[c][0].x, ga[c][1].x, ga[c][0].y, ga[c][1].y}, a1[4] = {ga[c][0].z, ga[c][1].z, ga[c][0].w, ga[c][1].w};
+      mma_bf16(y[j], a0, b.x, b.y);
+      mma_bf16(y[j], a1, b.z, b.w);
+    }
+    ss[0] = fmaf(y[j][0], y[j][0], fmaf(y[j][1], y[j][1], ss[0]));
+    ss[1] = fmaf(y[j][2], y[j][2], fmaf(y[j][3], y[j][3], ss[1]));
+  }
+  // 1 / rms of the thread's two rows from their sums of squares
+  auto inv_rms = [&](int which, float (&q)[2]) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      q[i] += __shfl_xor_sync(0xffffffffu, q[i], 1);
+      q[i] += __shfl_xor_sync(0xffffffffu, q[i], 2);
+      if (t4 == 0) red[warp][g + 8 * i] = q[i];
+    }
+    __syncthreads();
+    if (threadIdx.x < 16) {
+      float z = 0.f;
+#pragma unroll
+      for (int w = 0; w < kSideWarps; ++w) z += red[w][threadIdx.x];
+      sums[which][threadIdx.x] = z;
+    }
+    meet();
+    if (cluster > 1) {                                     // eight lanes add a row's parts
+      if (threadIdx.x < 128) {
+        const int r = threadIdx.x >> 3, c = threadIdx.x & 7;
+        float z = c < cluster ? ld_cluster_f32(cluster_map(smem_u32(&sums[which][r]), c)) : 0.f;
+        z += __shfl_xor_sync(0xffffffffu, z, 1);
+        z += __shfl_xor_sync(0xffffffffu, z, 2);
+        z += __shfl_xor_sync(0xffffffffu, z, 4);
+        if (c == 0) total[r] = z;
+      }
+      __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      q[i] = 1.f / sqrtf((cluster > 1 ? total : sums[which])[g + 8 * i] / static_cast<float>(W) + p.eps);
+  };
+  // x in the products' layout, eight column tiles at a time: all loads of a batch before its stores
+  float2 xv[8][2];
+  auto load_x = [&](int j0) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int c = c_w + 8 * (j0 + j) + 2 * t4, t = t0 + g + 8 * i;
+        xv[j][i] = make_float2(0.f, 0.f);
+        if (c < W && t < T) xv[j][i] = *reinterpret_cast<const float2*>(p.x + static_cast<size_t>(t) * W + c);
+      }
+  };
+  auto weight2 = [&](const float* w, int c) { return c < W ? __ldg(reinterpret_cast<const float2*>(w + c)) : make_float2(0.f, 0.f); };
+  load_x(0);
+  inv_rms(0, ss);
+  float s2[2] = {0.f, 0.f};
+#pragma unroll
+  for (int j0 = 0; j0 < NTW; j0 += 8) {
+    if (j0) load_x(j0);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int c = c_w + 8 * (j0 + j) + 2 * t4;
+      const float2 w = weight2(p.norm_w, c);
+      float (&yj)[4] = y[j0 + j];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int t = t0 + g + 8 * i;
+        yj[2 * i] = fmaf(yj[2 * i] * ss[i], w.x, xv[j][i].x);
+        yj[2 * i + 1] = fmaf(yj[2 * i + 1] * ss[i], w.y, xv[j][i].y);
+        if (c < W && t < T) *reinterpret_cast<float2*>(p.x + static_cast<size_t>(t) * W + c) = make_float2(yj[2 * i], yj[2 * i + 1]);
+        s2[i] = fmaf(yj[2 * i], yj[2 * i], fmaf(yj[2 * i + 1], yj[2 * i + 1], s2[i]));
+      }
+    }
+  }
+  if (p.next_w) {
+    inv_rms(1, s2);
+    __syncwarp();
+    if (cluster > 1) cluster_arrive();    // this block has read what it needs of the others
+#pragma unroll
+    for (int j = 0; j < NTW; ++j) {
+      const int c = c_w + 8 * j + 2 * t4;
+      const float2 w = weight2(p.next_w, c);
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        if (c < W && t0 + g + 8 * i < T)
+          *reinterpret_cast<uint32_t*>(p.h + static_cast<size_t>(t0 + g + 8 * i) * p.ldh + c) =
+              pack_bf16x2(y[j][2 * i] * s2[i] * w.x, y[j][2 * i + 1] * s2[i] * w.y);
+    }
+  } else if (cluster > 1) {
+    __syncwarp();
+    cluster_arrive();
+  }
+  __syncwarp();
+  if (cluster > 1) cluster_wait();        // nobody leaves while others read its sums
 }
 
 // ------------------------------------------------------------------ fp32 matrix product
@@ -512,6 +753,49 @@ int cb_side_gate(const void* x, int W, const void* w, int ldw, const void* ids, 
     case 4: return static_cast<int>(launch(side_gate_mma_kernel<4>, grid, dim3(32 * kSideWarps), 0, st, shape, p));
   }
   return static_cast<int>(launch(side_gate_mma_kernel<8>, grid, dim3(32 * kSideWarps), 0, st, shape, p));
+}
+
+struct CbSideInput {
+  void* x;
+  const void* gate; int ldw;
+  const void* ids;
+  const void* table; int ldt, col, vocab;
+  const void* proj; int ldp;
+  const void* norm_w;
+  const void* next_w;         // null: no h
+  void* h; int ldh;
+  int n, W, dim;
+  float eps;
+};
+
+// Widths and side channels the one-kernel form takes.
+int cb_side_input_fits(int W, int dim) { return W > 0 && dim > 0 && (W & 7) == 0 && W <= 8192 && dim <= 64; }
+
+int cb_side_input(const CbSideInput* a, void* stream) {
+  using namespace cb;
+  if (!a || a->n <= 0) return 0;
+  if (!cb_side_input_fits(a->W, a->dim) || a->vocab <= 0 || a->ldw < a->W || (a->ldw & 7) || a->ldp < (a->dim + 31) / 32 * 32 || (a->ldp & 7) ||
+      a->col < 0 || a->col + a->dim > a->ldt || (a->next_w && (!a->h || a->ldh < a->W || (a->ldh & 1))))
+    return -10;
+  SideInput p;
+  p.s.x = static_cast<const float*>(a->x); p.s.W = a->W;
+  p.s.w = static_cast<const __nv_bfloat16*>(a->gate); p.s.ldw = a->ldw;
+  p.s.ids = static_cast<const int*>(a->ids);
+  p.s.table = static_cast<const __nv_bfloat16*>(a->table); p.s.ldt = a->ldt; p.s.col = a->col; p.s.vocab = a->vocab;
+  p.s.out = nullptr; p.s.ldo = 0; p.s.T = a->n; p.s.dim = a->dim;
+  p.x = static_cast<float*>(a->x);
+  p.proj = static_cast<const __nv_bfloat16*>(a->proj); p.ldp = a->ldp;
+  p.norm_w = static_cast<const float*>(a->norm_w); p.next_w = static_cast<const float*>(a->next_w);
+  p.h = static_cast<__nv_bfloat16*>(a->h); p.ldh = a->ldh; p.eps = a->eps;
+  // prompts: fewer blocks share the tokens, and each has more columns to hide its waits behind
+  const int ntw = a->W > 4096 || (a->n + 15) / 16 * ((a->W + 511) / 512) > 296 ? 16 : 8;
+  int cluster = 1;
+  while (cluster * 64 * ntw < a->W) cluster *= 2;
+  const dim3 grid((a->n + 15) / 16, 1, cluster), shape(1, 1, cluster);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  auto go = [&](auto kernel) { return static_cast<int>(launch(kernel, grid, dim3(32 * kSideWarps), 0, st, shape, p)); };
+  if (ntw == 16) return a->dim <= 16 ? go(side_input_kernel<2, 16>) : a->dim <= 32 ? go(side_input_kernel<4, 16>) : go(side_input_kernel<8, 16>);
+  return a->dim <= 16 ? go(side_input_kernel<2, 8>) : a->dim <= 32 ? go(side_input_kernel<4, 8>) : go(side_input_kernel<8, 8>);
 }
 
 struct CbF32Gemm {

@@ -41,10 +41,12 @@ gated_parts_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, in
 
 extern "C" {
 
-// Gated linear attention: q, k [H d] and v [H e] at their columns of x; a: decay logits [H d].
+// Gated linear attention: q, k [H d] and v [H e] at their columns of x; a: decay logits [H d], or with `low` the inner columns of
+// their low-rank projection (low_k of them readable, zero from low_rank on).
 int cb_gated_linear_prepare(const CbRecPrep* a, const CbSegments* seg, void* stream) {
   if (!a || !seg || seg->num <= 0 || a->tokens <= 0) return 0;
   if (!cb::recurrence_sizes_ok(a->H, a->G, a->d, a->e, a->ds, a->es, seg) || a->G != a->H || !a->g || (a->ldx & 1)) return -10;
+  if (a->low && (a->f32 || (a->lda & 7) || (a->low_k & 7) || a->low_rank <= 0 || a->low_rank > a->low_k || (a->low_k & 31))) return -11;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return a->f32 ? cb::prep_typed<float, cb::kGated>(a, seg, st) : cb::prep_typed<__nv_bfloat16, cb::kGated>(a, seg, st);
 }

@@ -236,6 +236,8 @@ __device__ __forceinline__ uint32_t cluster_map(uint32_t smem_addr, uint32_t ran
   return r;
 }
 // All threads of all CTAs of the cluster (the hardware barrier: it waits only for threads that exist and run).
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
 __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
@@ -279,6 +281,9 @@ __device__ __forceinline__ float ld_cluster_f32(uint32_t cluster_addr) {
   float v;
   asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(cluster_addr) : "memory");
   return v;
+}
+__device__ __forceinline__ void st_cluster_u32(uint32_t cluster_addr, uint32_t v) {
+  asm volatile("st.shared::cluster.u32 [%0], %1;" ::"r"(cluster_addr), "r"(v) : "memory");
 }
 // 16 bytes from the shared memory of a CTA of the cluster (address from cluster_map)
 __device__ __forceinline__ float4 ld_cluster_f4(uint32_t cluster_addr) {

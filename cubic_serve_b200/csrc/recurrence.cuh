@@ -16,6 +16,7 @@
 // which keep the activation type.
 #pragma once
 #include "launch.cuh"
+#include "mma.cuh"
 #include "short_conv.cuh"
 
 namespace cb {
@@ -46,25 +47,69 @@ struct RecPrep {
   T* v;                       // [T, H, es]
   float2* coef;               // [T, H] {step size, decay per head (1 with channel decays)}
   float* g;                   // [T, H, ds] channel decays or null
+  const T* low;               // kGated, bf16: [H d, low_k]: a holds low_rank inner columns of the logits, this makes the logits; or null
+  int low_k, low_rank;
   int H, G, d, e, ds, es;
   Segments sg;
 };
 
-// A warp per (slot, tile of kPrepRows tokens): slots [0, G) are key heads (q and k), [G, G + H) value heads (v, step size,
-// decay per head), [G + H, G + 2 H) channel decays.  NP: channel pairs per lane of a key head (d <= 64 NP).  STEP: segments of
-// one token (decode): nothing is read ahead, which leaves registers for more warps.
+// The channel decays of a head for up to 16 tokens from the inner columns of their low-rank logits (bf16 models): the second
+// product runs here on the tensor cores, its result stays fp32.  Lane (g, t4) feeds the columns 8 t4 .. + 7 of a chunk of 32 to
+// two steps: which column goes to which place of a step is the same for both operands, so 16-byte loads make the fragments.
+template <typename F>
+__device__ __forceinline__ void low_rank_decays(const RecPrep<__nv_bfloat16>& p, int h, size_t row, int tokens, F decay_of) {
+  const int lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+  const __nv_bfloat16* w = p.low + static_cast<size_t>(h) * p.d * p.low_k;
+  for (int n0 = 0; n0 < p.ds; n0 += 32) {
+    float acc[4][4] = {};
+    for (int kc = 0; kc < p.low_rank; kc += 32) {              // the whole warp together; low_k is a multiple of 32
+      const int k = kc + 8 * t4;
+      uint4 a[2], b[4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        a[i] = g + 8 * i < tokens ? *reinterpret_cast<const uint4*>(p.a + (row + g + 8 * i) * p.lda + k) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        b[j] = n0 + 8 * j + g < p.d ? *reinterpret_cast<const uint4*>(w + static_cast<size_t>(n0 + 8 * j + g) * p.low_k + k) : make_uint4(0, 0, 0, 0);
+      const uint32_t a0[4] = {a[0].x, a[1].x, a[0].y, a[1].y}, a1[4] = {a[0].z, a[1].z, a[0].w, a[1].w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        mma_bf16(acc[j], a0, b[j].x, b[j].y);
+        mma_bf16(acc[j], a1, b[j].z, b[j].w);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = n0 + 8 * j + 2 * t4;
+      if (c >= p.ds) continue;                                 // ds is a multiple of 4
+      const float b0 = c < p.d ? p.dt_bias[h * p.d + c] : 0.f, b1 = c + 1 < p.d ? p.dt_bias[h * p.d + c + 1] : 0.f;
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        if (g + 8 * i < tokens)
+          *reinterpret_cast<float2*>(p.g + ((row + g + 8 * i) * p.H + h) * p.ds + c) =
+              make_float2(c < p.d ? decay_of(acc[j][2 * i] + b0) : 0.f, c + 1 < p.d ? decay_of(acc[j][2 * i + 1] + b1) : 0.f);
+    }
+  }
+}
+
+// A warp per (slot, tile of kPrepRows tokens).  The first G slots are key heads (q and k), then come value channels (64 VP of them
+// a slot), step sizes and decays (32 heads a slot) and the heads of channel decays.  NP: channel pairs per lane of a key head
+// (d <= 64 NP).  STEP: segments of one token (decode): nothing is read ahead, which leaves registers for more channels at once.
+template <bool STEP> constexpr int value_pairs() { return STEP ? 4 : 2; }
 template <typename T, int NP, int TAPS, bool STEP, int RULE>
 __global__ void __launch_bounds__(32 * kPrepWarps)
 recurrence_prepare_kernel(const RecPrep<T> p) {
   using Pair = ConvPair<T, TAPS, RULE == kSsd>;
+  constexpr int VP = value_pairs<STEP>();
   const ShortConv<T>& cvp = p.cv;
+  const int vslots = (p.H * p.e + 64 * VP - 1) / (64 * VP), cslots = (p.H + 31) / 32;
   pdl_wait();
   pdl_launch_dependents();
   int s, off;
   if (!find_tile(p.sg, kPrepRows, blockIdx.y, s, off)) return;
   const int slot = blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
-  if (slot >= p.G + (p.g ? 2 : 1) * p.H) return;
+  if (slot >= p.G + vslots + cslots + (p.g ? p.H : 0)) return;
   const int count = p.sg.count[s], end = min(count, off + kPrepRows);
   const bool fresh = p.sg.pos0[s] == 0;
   const size_t row0 = p.sg.row0[s];
@@ -138,55 +183,82 @@ recurrence_prepare_kernel(const RecPrep<T> p) {
         conv_state(cvp, xr, st, fresh, count, kb, p.d);
       }
     }
-  } else if (slot < p.G + p.H) {
-    const int h = slot - p.G, vb = p.v_off + h * p.e;
+  } else if (slot < p.G + vslots) {
+    // 64 VP neighbouring value channels, whatever heads they belong to
+    const int c0 = (slot - p.G) * 64 * VP, lim = p.H * p.e;
     constexpr int AH = STEP ? 1 : 4;
-    for (int c0 = 2 * lane; c0 < p.e; c0 += 128) {             // two pairs at a time
-      Pair cv[2];
+    Pair cv[VP];
+    int at0[VP], at1[VP];                                      // places of the pair's channels in a row of v
 #pragma unroll
-      for (int i = 0; i < 2; ++i) cv[i].begin(cvp, xr, st, fresh, vb, c0 + 64 * i, p.e, off);
-      for (int t0 = off; t0 < end; t0 += AH) {
-        float2 xv[AH][2];
+    for (int i = 0; i < VP; ++i) {
+      const int c = c0 + 2 * lane + 64 * i;
+      cv[i].begin(cvp, xr, st, fresh, p.v_off, c, lim, off);
+      at0[i] = p.es == p.e ? c : c / p.e * p.es + c % p.e;
+      at1[i] = p.es == p.e || (p.e & 1) == 0 ? at0[i] + 1 : (c + 1) / p.e * p.es + (c + 1) % p.e;
+    }
+    for (int t0 = off; t0 < end; t0 += AH) {
+      float2 xv[AH][VP];
 #pragma unroll
-        for (int u = 0; u < AH; ++u)
+      for (int u = 0; u < AH; ++u)
 #pragma unroll
-          for (int i = 0; i < 2; ++i) xv[u][i] = cv[i].ahead(t0 + u, end);
+        for (int i = 0; i < VP; ++i) xv[u][i] = cv[i].ahead(t0 + u, end);
 #pragma unroll
-        for (int u = 0; u < AH; ++u) {
-          const int t = t0 + u;
-          if (t >= end) break;
+      for (int u = 0; u < AH; ++u) {
+        const int t = t0 + u;
+        if (t >= end) break;
+        T* dst = p.v + (row0 + t) * p.H * p.es;
 #pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            const float2 v = cv[i].token(t, xv[u][i]);
-            T* dst = p.v + ((row0 + t) * p.H + h) * p.es + c0 + 64 * i;      // es is even: the pair's second column exists
-            if (!cv[i].ok) continue;
-            if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(v.x, v.y);
-            else *reinterpret_cast<float2*>(dst) = v;
+        for (int i = 0; i < VP; ++i) {
+          const float2 v = cv[i].token(t, xv[u][i]);
+          if (!cv[i].ok) continue;
+          if constexpr (Pair::ODD) {
+            dst[at0[i]] = from_f<T>(v.x);
+            if (cv[i].ok1) dst[at1[i]] = from_f<T>(v.y);
+          } else if constexpr (sizeof(T) == 2) {
+            *reinterpret_cast<uint32_t*>(dst + at0[i]) = pack_bf16x2(v.x, v.y);
+          } else {
+            *reinterpret_cast<float2*>(dst + at0[i]) = v;
           }
         }
       }
-      if (TAPS > 0 && off == 0) {
-#pragma unroll
-        for (int i = 0; i < 2; ++i) cv[i].save(st, count, end == count);
-      }
     }
-    if (off + lane < end && lane < kPrepRows) {
-      const size_t r = row0 + off + lane;
+    if constexpr (TAPS > 0) {
+      if (off == 0) {
+#pragma unroll
+        for (int i = 0; i < VP; ++i) cv[i].save(st, count, end == count);
+      }
+    } else if constexpr (TAPS == 0) {
+      if (off == 0) conv_state(cvp, xr, st, fresh, count, p.v_off + c0, min(64 * VP, lim - c0));
+    }
+  } else if (slot < p.G + vslots + cslots) {
+    // step sizes and decays of 32 heads
+    const int h = (slot - p.G - vslots) * 32 + lane;
+    if (h >= p.H) return;
+    const float rate = RULE == kGated ? 0.f : -expf(p.a_log[h]);
+    const float bias = RULE == kGated || p.g ? 0.f : p.dt_bias[h];
+    for (int t = off; t < end; ++t) {
+      const size_t r = row0 + t;
       float beta = 1.f, decay = 1.f;
       if constexpr (RULE == kSsd) {
-        beta = softplus_of<float>(to_f(p.a[r * p.lda + h]) + p.dt_bias[h]);
-        decay = expf(-expf(p.a_log[h]) * beta);
+        beta = softplus_of<float>(to_f(p.a[r * p.lda + h]) + bias);
+        decay = expf(rate * beta);
       } else if constexpr (RULE == kDelta) {
         beta = 1.f / (1.f + expf(-to_f(p.b[r * p.ldb + h])));
-        if (!p.g) decay = expf(-expf(p.a_log[h]) * softplus_of<float>(to_f(p.a[r * p.lda + h]) + p.dt_bias[h]));
+        if (!p.g) decay = expf(rate * softplus_of<float>(to_f(p.a[r * p.lda + h]) + bias));
       }
       p.coef[r * p.H + h] = make_float2(beta, decay);
     }
-    if (TAPS == 0 && off == 0) conv_state(cvp, xr, st, fresh, count, vb, p.e);
   } else if constexpr (RULE != kSsd) {
-    const int h = slot - p.G - p.H;
+    const int h = slot - p.G - vslots - cslots;
     // sigmoid(x)^rate = exp(-rate softplus(-x))
     const float rate = RULE == kGated ? -p.rate : -expf(p.a_log[h]), sign = RULE == kGated ? -1.f : 1.f;
+    auto decay_of = [&](float logit) { return exp_of<T>(rate * softplus_of<T>(sign * logit)); };
+    if constexpr (RULE == kGated && sizeof(T) == 2) {
+      if (p.low) {
+        low_rank_decays(p, h, row0 + off, end - off, decay_of);
+        return;
+      }
+    }
     constexpr int AH = STEP ? 1 : 4;
     for (int c0 = lane; c0 < p.ds; c0 += 128) {                // four channels x AH tokens read at once
       float dt[4];
@@ -206,8 +278,7 @@ recurrence_prepare_kernel(const RecPrep<T> p) {
 #pragma unroll
           for (int i = 0; i < 4; ++i)
             if (t0 + u < end && c0 + 32 * i < p.ds)
-              dst[static_cast<size_t>(t0 + u) * p.H * p.ds + 32 * i] =
-                  c0 + 32 * i < p.d ? exp_of<T>(rate * softplus_of<T>(sign * (v[u][i] + dt[i]))) : 0.f;
+              dst[static_cast<size_t>(t0 + u) * p.H * p.ds + 32 * i] = c0 + 32 * i < p.d ? decay_of(v[u][i] + dt[i]) : 0.f;
       }
     }
   }
@@ -654,6 +725,7 @@ struct CbRecPrep {
   void* v;
   void* coef;
   void* g;
+  const void* low; int low_k, low_rank;
   int H, G, d, e, ds, es, tokens, f32;
 };
 
@@ -696,6 +768,7 @@ static RecPrep<T> rec_prep(const CbRecPrep* a, const CbSegments* seg) {
   p.v = static_cast<T*>(a->v);
   p.coef = static_cast<float2*>(a->coef);
   p.g = static_cast<float*>(a->g);
+  p.low = static_cast<const T*>(a->low); p.low_k = a->low_k; p.low_rank = a->low_rank;
   p.H = a->H; p.G = a->G; p.d = a->d; p.e = a->e; p.ds = a->ds; p.es = a->es;
   p.sg = make_segments(seg, a->tokens);
   return p;
@@ -723,10 +796,12 @@ static RecWalk<T> rec_walk(const CbRecWalk* a, const CbSegments* seg) {
 // The preparation kernel of key width NP * 64 for every supported tap count of the rule.
 template <typename T, int NP, int TAPS, int RULE>
 static int prep_go(const RecPrep<T>& p, int tiles, cudaStream_t st) {
-  const dim3 grid((p.G + (p.g ? 2 : 1) * p.H + kPrepWarps - 1) / kPrepWarps, tiles);
-  if (p.sg.single)
-    return static_cast<int>(launch(recurrence_prepare_kernel<T, NP, TAPS, true, RULE>, grid, dim3(32 * kPrepWarps), 0, st, p));
-  return static_cast<int>(launch(recurrence_prepare_kernel<T, NP, TAPS, false, RULE>, grid, dim3(32 * kPrepWarps), 0, st, p));
+  auto go = [&](auto kernel, int vp) {
+    const int slots = p.G + (p.H * p.e + 64 * vp - 1) / (64 * vp) + (p.H + 31) / 32 + (p.g ? p.H : 0);
+    return static_cast<int>(launch(kernel, dim3((slots + kPrepWarps - 1) / kPrepWarps, tiles), dim3(32 * kPrepWarps), 0, st, p));
+  };
+  if (p.sg.single) return go(recurrence_prepare_kernel<T, NP, TAPS, true, RULE>, value_pairs<true>());
+  return go(recurrence_prepare_kernel<T, NP, TAPS, false, RULE>, value_pairs<false>());
 }
 template <typename T, int NP, int RULE>
 static int prep_taps(const RecPrep<T>& p, int tiles, cudaStream_t st) {

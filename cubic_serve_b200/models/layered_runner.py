@@ -188,11 +188,8 @@ class LayeredRunner(StepRunner):
                 n += 3
             follow = None if i == last else w.layers[i + 1].norm       # the final norm reads the wanted rows only
             if l.side is not None:
-                g, y = self.side[:T], self.side_y[:T, :cfg.hidden_size]
-                K.side_gate(x, l.side.gate, b.token_ids[:T], w.side_embed, l.side.col, g)
-                K.wide_gemm(g, l.side.proj, y, ws=self.ws)
-                K.add_norm_rows(y, l.side.norm_w, x, eps, follow, None if follow is None else h)
-                n += 3
+                n += K.side_input(x, l.side.gate, b.token_ids[:T], w.side_embed, l.side.col, l.side.proj, l.side.norm_w, eps, follow,
+                                  None if follow is None else h, self.side[:T], self.side_y[:T, :cfg.hidden_size], self.ws)
             elif follow is not None:
                 K.row_norm(x, follow, h, eps)
                 n += 1
@@ -253,12 +250,17 @@ class LayeredRunner(StepRunner):
                                    decode=decode, ws=self.ws)
 
     def _gated_linear(self, m: GatedLinearWeights, proj, run: _StateRun, b, out, decode: bool) -> int:
-        s, T = m.spec, proj.shape[0]
-        a = self._rows("low", T, m.low.n)
-        K.wide_gemm(proj[:, m.a_off:m.a_off + m.low.k], m.low, a, ws=self.ws)
+        s, T, n = m.spec, proj.shape[0], 1
+        low, a = m.low, proj[:, m.a_off:m.a_off + m.low.k]
+        # the preparation makes the decay logits itself, 16 tokens of a request at a time; steps of many single tokens and 32-bit
+        # models leave it to a product
+        if proj.dtype != torch.bfloat16 or decode and T > 64:
+            z = self._rows("low", T, low.n)
+            K.wide_gemm(a, low, z, ws=self.ws)
+            low, a, n = None, z, 2
         K.gated_linear_prepare(proj, m.q_off, m.k_off, m.v_off, a, m.bias, 1.0 / s.tau, b.segments, self.recurrence, s.heads, s.dim,
-                               s.vdim)
-        return 2 + K.gated_linear_walk(proj[:, m.g_off:m.g_off + s.out_width], m.norm_w, run.state, b.segments, out, self.recurrence,
+                               s.vdim, low, s.decay_rank)
+        return n + K.gated_linear_walk(proj[:, m.g_off:m.g_off + s.out_width], m.norm_w, run.state, b.segments, out, self.recurrence,
                                        s.dim, self.cfg.rms_eps, decode)
 
     def _ssd(self, m: SsdWeights, proj, run: _StateRun, b, out, decode: bool) -> int:

@@ -823,6 +823,26 @@ def side_gate(x: torch.Tensor, gate: torch.Tensor, ids: torch.Tensor, table: tor
                                            int(out.dtype == torch.float32), _stream()), "cb_side_gate")
 
 
+def side_input(x: torch.Tensor, gate: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col: int, proj: PackedWeight,
+               norm_w: torch.Tensor, eps: float, next_w: torch.Tensor | None, h: torch.Tensor | None, g: torch.Tensor, y: torch.Tensor,
+               ws: Workspace | None = None) -> int:
+    """A layer's whole side input: ``side_gate`` into ``g``, the product with ``proj`` into ``y``, ``add_norm_rows``.  One kernel
+    for bf16 rows of the widths it takes, which leaves ``g`` and ``y`` alone.  Returns the launches made."""
+    W, dim = x.shape[1], gate.shape[0]
+    if y.dtype == torch.float32 or not native.lib().cb_side_input_fits(W, dim):
+        side_gate(x, gate, ids, table, col, g)
+        wide_gemm(g, proj, y, ws=ws)
+        add_norm_rows(y, norm_w, x, eps, next_w, h)
+        return 3
+    assert x.dtype == norm_w.dtype == torch.float32 and x.is_contiguous() and gate.dtype == table.dtype == torch.bfloat16
+    assert proj.fmt == FMT_BF16 and proj.n == W and (h is None) == (next_w is None) and (h is None or h.dtype == torch.bfloat16)
+    a = native.SideInputStruct(x.data_ptr(), gate.data_ptr(), gate.shape[1], ids.data_ptr(), table.data_ptr(), table.shape[1], col,
+                               table.shape[0], proj.codes.data_ptr(), proj.k, norm_w.data_ptr(), _ptr(next_w), _ptr(h),
+                               0 if h is None else h.stride(0), x.shape[0], W, dim, float(eps))
+    native.check(native.lib().cb_side_input(ctypes.byref(a), _stream()), "cb_side_input")
+    return 1
+
+
 class RecurrenceScratch:
     """Fixed-address buffers between the preparation and the recurrence of recurrent layers, for up to ``max_tokens`` rows of
     the largest layer they are made for (layers share them)."""
@@ -842,7 +862,8 @@ class RecurrenceScratch:
 
 
 def _prepare(entry: str, x, a, dt_bias, seg: GdnSegments, sc: RecurrenceScratch, heads: int, kv_heads: int, dim: int, vdim: int,
-             channel: bool, offs: tuple[int, int, int], conv=None, b=None, a_log=None, rate: float = 0.0) -> None:
+             channel: bool, offs: tuple[int, int, int], conv=None, b=None, a_log=None, rate: float = 0.0,
+             low: PackedWeight | None = None, low_rank: int = 0) -> None:
     """Preparation of a recurrence's tokens (``csrc/recurrence.cuh``).  ``offs``: columns of q, k and v in ``x``; ``conv``:
     (weights fp32 [taps, channels], bias or None, state [slots, taps - 1, channels])."""
     T = x.shape[0]
@@ -862,8 +883,8 @@ def _prepare(entry: str, x, a, dt_bias, seg: GdnSegments, sc: RecurrenceScratch,
     p = native.RecPrepStruct(x.data_ptr(), x.stride(0), _ptr(w), _ptr(bias), ldw, taps, _ptr(state), *offs, _ptr(b),
                              0 if b is None else b.stride(0), a.data_ptr(), a.stride(0), _ptr(a_log), dt_bias.data_ptr(),
                              float(rate), sc.q.data_ptr(), sc.k.data_ptr(), sc.kq.data_ptr(), sc.v.data_ptr(),
-                             sc.coef.data_ptr(), sc.g.data_ptr() if channel else None, heads, kv_heads, dim, vdim, ds, es, T,
-                             int(x.dtype == torch.float32))
+                             sc.coef.data_ptr(), sc.g.data_ptr() if channel else None, None if low is None else low.codes.data_ptr(),
+                             0 if low is None else low.k, low_rank, heads, kv_heads, dim, vdim, ds, es, T, int(x.dtype == torch.float32))
     st = _seg(seg)
     native.check(getattr(native.lib(), entry)(ctypes.byref(p), ctypes.byref(st), _stream()), entry)
 
@@ -881,12 +902,20 @@ def delta_prepare(x: torch.Tensor, b: torch.Tensor, a: torch.Tensor, conv_w: tor
 
 
 def gated_linear_prepare(x: torch.Tensor, q_off: int, k_off: int, v_off: int, a: torch.Tensor, bias: torch.Tensor, rate: float,
-                         seg: GdnSegments, sc: RecurrenceScratch, heads: int, dim: int, vdim: int) -> None:
+                         seg: GdnSegments, sc: RecurrenceScratch, heads: int, dim: int, vdim: int, low: PackedWeight | None = None,
+                         low_rank: int = 0) -> None:
     """The tokens of gated linear attention: q times ``dim^-1/2``, k and v at their columns of ``x``; decays
-    ``sigmoid(a + bias)^rate`` per key channel."""
-    assert a.shape[1] == bias.numel() == heads * dim and x.stride(0) % 2 == 0
+    ``sigmoid(a + bias)^rate`` per key channel.  With ``low`` (bf16 rows) ``a`` holds the ``low.k`` inner columns of the low-rank
+    logits, zero from ``low_rank`` on, and the logits ``a low^T`` are made on the way, in fp32."""
+    assert bias.numel() == heads * dim and x.stride(0) % 2 == 0
+    if low is None:
+        assert a.shape[1] == heads * dim
+    else:
+        assert low.fmt == FMT_BF16 and low.n == heads * dim and a.shape[1] == low.k and a.dtype == torch.bfloat16
+        assert a.data_ptr() % 16 == 0 and a.stride(0) % 8 == 0
     assert x.shape[1] >= max(q_off + heads * dim, k_off + heads * dim, v_off + heads * vdim)
-    _prepare("cb_gated_linear_prepare", x, a, bias, seg, sc, heads, heads, dim, vdim, True, (q_off, k_off, v_off), rate=rate)
+    _prepare("cb_gated_linear_prepare", x, a, bias, seg, sc, heads, heads, dim, vdim, True, (q_off, k_off, v_off), rate=rate,
+             low=low, low_rank=low_rank)
 
 
 def ssd_prepare(x: torch.Tensor, dt: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, conv_state: torch.Tensor,

@@ -274,6 +274,9 @@ def _declare(l: ctypes.CDLL) -> None:
     l.cb_embed_rows.argtypes = [vp, vp, vp, vp, vp, i, i, i, i, f, i, vp]
     l.cb_add_norm_rows.argtypes = [vp, i, vp, vp, vp, vp, i, i, i, f, i, vp]
     l.cb_side_gate.argtypes = [vp, i, vp, i, vp, vp, i, i, vp, i, i, i, i, i, vp]
+    l.cb_side_input.argtypes = [vp, vp]
+    l.cb_side_input_fits.argtypes = [i, i]
+    l.cb_side_input_fits.restype = i
     l.cb_gqa_prepare.argtypes = [vp, vp]
     l.cb_gqa_attn.argtypes = [vp, vp, vp]
     l.cb_gqa_attn_partial_floats.argtypes = [i, i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
@@ -283,7 +286,8 @@ def _declare(l: ctypes.CDLL) -> None:
     l.cb_latent_attn_partial_floats.argtypes = [i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
     l.cb_latent_attn_partial_floats.restype = ll
     for name in ("bf16_gemm_wide", "f32_gemm", "row_norm", "embed_norm", "concat_rows", "latent_prepare",
-                 "latent_attn", "gated_parts_norm", "embed_rows", "add_norm_rows", "side_gate", "gqa_prepare", "gqa_attn"):
+                 "latent_attn", "gated_parts_norm", "embed_rows", "add_norm_rows", "side_gate", "side_input",
+                 "gqa_prepare", "gqa_attn"):
         getattr(l, f"cb_{name}").restype = i
     # fp8 (e4m3 x e4m3) tensor path: activation quantizers and the GEMM entries
     l.cb_fp8_quantize_rows.argtypes = [vp, i, vp, i, vp, i, i, vp]
@@ -346,9 +350,9 @@ class RecPrepStruct(ctypes.Structure):
                 ("k_off", ctypes.c_int), ("v_off", ctypes.c_int), ("b", ctypes.c_void_p), ("ldb", ctypes.c_int),
                 ("a", ctypes.c_void_p), ("lda", ctypes.c_int), ("a_log", ctypes.c_void_p), ("dt_bias", ctypes.c_void_p),
                 ("rate", ctypes.c_float), ("q", ctypes.c_void_p), ("k", ctypes.c_void_p), ("kq", ctypes.c_void_p),
-                ("v", ctypes.c_void_p), ("coef", ctypes.c_void_p), ("g", ctypes.c_void_p), ("H", ctypes.c_int),
-                ("G", ctypes.c_int), ("d", ctypes.c_int), ("e", ctypes.c_int), ("ds", ctypes.c_int), ("es", ctypes.c_int),
-                ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
+                ("v", ctypes.c_void_p), ("coef", ctypes.c_void_p), ("g", ctypes.c_void_p), ("low", ctypes.c_void_p),
+                ("low_k", ctypes.c_int), ("low_rank", ctypes.c_int), ("H", ctypes.c_int), ("G", ctypes.c_int),
+                ("d", ctypes.c_int), ("e", ctypes.c_int), ("ds", ctypes.c_int), ("es", ctypes.c_int), ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
 
 
 class RecWalkStruct(ctypes.Structure):
@@ -367,6 +371,15 @@ class LatentAttnStruct(ctypes.Structure):
                 ("ldg", ctypes.c_int), ("page_table", ctypes.c_void_p), ("max_pages", ctypes.c_int), ("H", ctypes.c_int),
                 ("Rp", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float), ("tokens", ctypes.c_int),
                 ("f32", ctypes.c_int), ("decode", ctypes.c_int), ("splits", ctypes.c_int), ("partial", ctypes.c_void_p)]
+
+
+class SideInputStruct(ctypes.Structure):
+    """Mirror of ``CbSideInput`` in ``csrc/layered.cu``."""
+    _fields_ = [("x", ctypes.c_void_p), ("gate", ctypes.c_void_p), ("ldw", ctypes.c_int), ("ids", ctypes.c_void_p),
+                ("table", ctypes.c_void_p), ("ldt", ctypes.c_int), ("col", ctypes.c_int), ("vocab", ctypes.c_int),
+                ("proj", ctypes.c_void_p), ("ldp", ctypes.c_int), ("norm_w", ctypes.c_void_p), ("next_w", ctypes.c_void_p),
+                ("h", ctypes.c_void_p), ("ldh", ctypes.c_int), ("n", ctypes.c_int), ("W", ctypes.c_int), ("dim", ctypes.c_int),
+                ("eps", ctypes.c_float)]
 
 
 class GqaPrepStruct(ctypes.Structure):

@@ -95,6 +95,41 @@ def test_side_gate(dtype, T, W, dim):
     assert (out[:, dim:] == 9).all()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T, W, dim", [(1, 64, 16), (5, 72, 5), (17, 68, 8), (300, 520, 40), (1, 2048, 64), (33, 4096, 24), (40, 1024, 130),
+                                       (600, 96, 12), (16, 8192, 33), (19, 6144, 64), (4, 8704, 16)])
+def test_side_input(dtype, T, W, dim):
+    """The whole step, in one kernel (clusters of one to eight blocks) where the sizes allow it: residual, next norm, and neither
+    of them touched where there is no next norm."""
+    from cubic_serve_b200.ops import kernels as K, wq_pack
+    g = torch.Generator().manual_seed(T + W)
+    x, w = torch.randn(T, W, generator=g), (torch.randn(dim, W, generator=g) / W ** 0.5).to(torch.bfloat16)
+    table, ids = torch.randn(19, 3 * dim + 2, generator=g).to(torch.bfloat16), torch.randint(0, 19, (T,), generator=g).to(torch.int32)
+    gate = torch.zeros(dim, -(-W // 64) * 64, dtype=torch.bfloat16)
+    gate[:, :W] = w
+    kp = -(-dim // 64) * 64
+    proj = torch.zeros(W, kp, dtype=torch.bfloat16)
+    proj[:, :dim] = (torch.randn(W, dim, generator=g) / dim ** 0.5).to(torch.bfloat16)
+    nw, nx = torch.randn(W, generator=g), 1 + 0.2 * torch.randn(W, generator=g)
+    e = table.double()[ids.long(), dim + 1:2 * dim + 1]
+    y = (R.gelu_tanh(x.double() @ w.double().t()) * e) @ proj[:, :dim].double().t()
+    want = x.double() + R.rms(y, 1e-3) * nw.double()
+    packed = wq_pack.pack_bf16(proj).to(DEV)
+    for follow in (True, False):
+        xd = x.to(DEV)
+        h = torch.full((T, -(-W // 64) * 64), 9.0, dtype=dtype, device=DEV)
+        gs, ys = torch.zeros(T, kp, dtype=dtype, device=DEV), torch.zeros(T, -(-W // 8) * 8, dtype=dtype, device=DEV)
+        n = K.side_input(xd, gate.to(DEV), ids.to(DEV), table.to(DEV), dim + 1, packed, nw.to(DEV), 1e-3, nx.to(DEV) if follow else None,
+                         h if follow else None, gs, ys[:, :W])
+        assert n == (1 if dtype == torch.bfloat16 and dim <= 64 and W % 8 == 0 and W <= 8192 else 3)
+        close(xd, want, torch.float32, exact=2e-5 if dtype == torch.float32 else 1e-2)
+        if follow:
+            close(h[:, :W], R.rms(want, 1e-3) * nx.double(), dtype, exact=2e-5, rough=1.5e-2)
+            assert (h[:, W:] == 9).all()
+        else:
+            assert (h == 9).all()
+
+
 # ------------------------------------------------------------------ sink attention
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H, G, d, pairs", [(6, 2, 24, 6), (3, 1, 13, 3), (4, 4, 64, 32), (2, 1, 200, 20), (5, 5, 18, 0), (40, 1, 128, 64)])
@@ -415,6 +450,28 @@ def test_recurrence_batches(dtype, layer):
         want, state = layer.oracle(rows_of(cs[i], lens[i], lens[i] + 1), oracle[i][1])
         close(out[j:j + 1], want, dtype, exact=5e-5)
         layer.check_state(states, slots[i], state, dtype)
+
+
+@pytest.mark.parametrize("layer, rank", [(GatedLinear(3, 20, 28), 12), (GatedLinear(2, 128, 64, 16.0), 64), (GatedLinear(2, 7, 9, 3.0), 33),
+                                         (GatedLinear(1, 160, 16), 100)], ids=["20", "128", "7", "160"])
+def test_low_rank_decays(layer, rank):
+    """Decay logits made by the preparation from their inner columns equal the product done before it, in prompts and decoding."""
+    from cubic_serve_b200.ops import kernels as K, wq_pack
+    H, d, T, kp = layer.H, layer.d, 37, -(-rank // 64) * 64
+    c = layer.case(T, 3)
+    g = torch.Generator().manual_seed(rank)
+    inner, w = torch.randn(T, rank, generator=g).to(torch.bfloat16), (2 * torch.randn(H * d, rank, generator=g) / rank ** 0.5).to(torch.bfloat16)
+    z = inner.double() @ w.double().t() + c["bias"].double()
+    want = (1 / (1 + torch.exp(-z))) ** (1 / layer.tau)
+    a, low = torch.zeros(T, kp + 8, dtype=torch.bfloat16), torch.zeros(H * d, kp, dtype=torch.bfloat16)
+    a[:, :rank], low[:, :rank] = inner, w
+    ds = -(-d // 4) * 4
+    for spans in ([(T, 0, 0)], [(5, 0, 0), (1, 1, 3), (31, 2, 0)], [(1, t, 4) for t in range(T)]):
+        sc = K.RecurrenceScratch(T, [(H, H, d, layer.e, True)], torch.bfloat16, DEV)
+        K.gated_linear_prepare(c["x"].to(DEV), *layer.offs, a.to(DEV)[:, :kp], c["bias"].to(DEV), 1 / layer.tau, segs(spans), sc, H, d,
+                               layer.e, wq_pack.pack_bf16(low).to(DEV), rank)
+        got = sc.g[:T * H * ds].view(T, H, ds)
+        assert (got[:, :, :d].double().cpu() - want.view(T, H, d)).abs().max() < 5e-6 and (got[:, :, d:] == 0).all()
 
 
 def test_decay_of_every_channel_counts():
