@@ -29,6 +29,7 @@ REF_DIR = os.path.join(os.path.dirname(os.path.abspath(__file__)), "_ref")
 
 def _timeit_graph(torch, fn, flush, launches: int = 5, repeats: int = 3) -> float:
     stream = torch.cuda.Stream()
+    stream.wait_stream(torch.cuda.current_stream())      # the caller's inputs are written there
     graphs = []
     with torch.cuda.stream(stream):
         fn()

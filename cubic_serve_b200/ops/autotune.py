@@ -73,6 +73,7 @@ def _random_weight(fmt: int, n: int, k: int, act: bool, device) -> wq_pack.Packe
 def _time_graph(fn, flush: torch.Tensor, launches: int = 6, repeats: int = 3) -> float:
     """Device microseconds per call inside a CUDA graph, L2 flushed before every call (flush time subtracted)."""
     stream = torch.cuda.Stream()
+    stream.wait_stream(torch.cuda.current_stream())      # the caller's inputs are written there
     times = []
     with torch.cuda.stream(stream):
         fn()

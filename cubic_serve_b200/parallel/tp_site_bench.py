@@ -76,6 +76,7 @@ def main(argv=None) -> None:
     gu = torch.empty(M, 2 * I // size, dtype=torch.bfloat16, device=dev)
     flush = torch.empty(192 << 20, dtype=torch.uint8, device=dev)
     stream = torch.cuda.Stream(dev)
+    stream.wait_stream(torch.cuda.current_stream(dev))   # the operands are written there
     report = {"ranks": size, "m": M, "hidden": H, "inter": I, "sites_per_graph": args.sites,
               "nvls": os.environ.get("CUBIC_SERVE_NVLS", "gather")}
 

@@ -45,6 +45,7 @@ def timeit_graph(fn, flush: torch.Tensor, launches: int = 10, repeats: int = 3) 
     {write a buffer larger than L2, call}; the same graph without the calls is timed too and subtracted.
     """
     stream = torch.cuda.Stream()
+    stream.wait_stream(torch.cuda.current_stream())      # the caller's inputs (page tables, segments) are written there
     graphs = []
     with torch.cuda.stream(stream):
         fn()
