@@ -132,19 +132,11 @@ def bench_gated_linear(requests: int, tokens: int, heads: int, flush, pk) -> lis
     seg = _segments(requests, tokens, 5)
     proj, bias = torch.randn(T, 4 * H * d + 64, **bf), torch.zeros(H * d, device=DEV)
     a, low = proj[:, 4 * H * d:], wq_pack.pack_bf16(torch.randn(H * d, 64, device=DEV) / 8)      # rank 64
-    logits = torch.empty(T, H * d, **bf)
     state, out = torch.randn(requests, H, d, d, device=DEV) * 0.01, torch.empty(T, H * d, **bf)
     norm_w = torch.ones(d, device=DEV)
     sc = K.RecurrenceScratch(T, [(H, H, d, d, True)], torch.bfloat16, DEV)
-
-    def prepare():
-        if tokens == 1 and T > 64:                       # as the runner does
-            K.wide_gemm(a, low, logits)
-            K.gated_linear_prepare(proj, 0, H * d, 2 * H * d, logits, bias, 1 / 16, seg, sc, H, d, d)
-        else:
-            K.gated_linear_prepare(proj, 0, H * d, 2 * H * d, a, bias, 1 / 16, seg, sc, H, d, d, low, 64)
-
-    prep = timeit_graph(prepare, flush, launches=5)
+    prep = timeit_graph(lambda: K.gated_linear_prepare(proj, 0, H * d, 2 * H * d, a, bias, 1 / 16, seg, sc, H, d, d, low, 64), flush,
+                        launches=5)
     walk = timeit_graph(lambda: K.gated_linear_walk(proj[:, 3 * H * d:4 * H * d], norm_w, state, seg, out, sc, d, 1e-6, tokens == 1), flush, launches=5)
     shape = f"{requests} x {tokens} tokens, {H} heads of 128"
     return [_line(f"gated_linear_prepare with decay logits [{shape}]", prep, T * (3 * H * d + 64) * 2, 0, 1, pk),

@@ -53,47 +53,54 @@ struct RecPrep {
   Segments sg;
 };
 
-// The channel decays of a head for up to 16 tokens from the inner columns of their low-rank logits (bf16 models): the second
-// product runs here on the tensor cores, its result stays fp32.  Lane (g, t4) feeds the columns 8 t4 .. + 7 of a chunk of 32 to
-// two steps: which column goes to which place of a step is the same for both operands, so 16-byte loads make the fragments.
+// 32 channel decays (from channel n0 of head h on) of up to 16 tokens from the inner columns of their low-rank logits (bf16
+// models): the second product runs here on the tensor cores, its result stays fp32.  Lane (g, t4) feeds the columns 8 t4 .. + 7 of
+// a chunk of 32 to two steps: which column goes to which place of a step is the same for both operands, so 16-byte loads make the
+// fragments.
 template <typename F>
-__device__ __forceinline__ void low_rank_decays(const RecPrep<__nv_bfloat16>& p, int h, size_t row, int tokens, F decay_of) {
+__device__ __forceinline__ void low_rank_decays(const RecPrep<__nv_bfloat16>& p, int h, int n0, size_t row, int tokens, F decay_of) {
   const int lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
   const __nv_bfloat16* w = p.low + static_cast<size_t>(h) * p.d * p.low_k;
-  for (int n0 = 0; n0 < p.ds; n0 += 32) {
-    float acc[4][4] = {};
-    for (int kc = 0; kc < p.low_rank; kc += 32) {              // the whole warp together; low_k is a multiple of 32
-      const int k = kc + 8 * t4;
-      uint4 a[2], b[4];
+  float acc[4][4] = {};
+  for (int kc = 0; kc < p.low_rank; kc += 64) {                // the whole warp together; two chunks' loads in flight
+    uint4 a[2][2], b[2][4];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int k = kc + 32 * u + 8 * t4;
+      const bool there = kc + 32 * u < p.low_rank;             // low_k is a multiple of 32
 #pragma unroll
       for (int i = 0; i < 2; ++i)
-        a[i] = g + 8 * i < tokens ? *reinterpret_cast<const uint4*>(p.a + (row + g + 8 * i) * p.lda + k) : make_uint4(0, 0, 0, 0);
+        a[u][i] = there && g + 8 * i < tokens ? *reinterpret_cast<const uint4*>(p.a + (row + g + 8 * i) * p.lda + k) : make_uint4(0, 0, 0, 0);
 #pragma unroll
       for (int j = 0; j < 4; ++j)
-        b[j] = n0 + 8 * j + g < p.d ? *reinterpret_cast<const uint4*>(w + static_cast<size_t>(n0 + 8 * j + g) * p.low_k + k) : make_uint4(0, 0, 0, 0);
-      const uint32_t a0[4] = {a[0].x, a[1].x, a[0].y, a[1].y}, a1[4] = {a[0].z, a[1].z, a[0].w, a[1].w};
+        b[u][j] = there && n0 + 8 * j + g < p.d ? *reinterpret_cast<const uint4*>(w + static_cast<size_t>(n0 + 8 * j + g) * p.low_k + k)
+                                                : make_uint4(0, 0, 0, 0);
+    }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const uint32_t a0[4] = {a[u][0].x, a[u][1].x, a[u][0].y, a[u][1].y}, a1[4] = {a[u][0].z, a[u][1].z, a[u][0].w, a[u][1].w};
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        mma_bf16(acc[j], a0, b[j].x, b[j].y);
-        mma_bf16(acc[j], a1, b[j].z, b[j].w);
+        mma_bf16(acc[j], a0, b[u][j].x, b[u][j].y);
+        mma_bf16(acc[j], a1, b[u][j].z, b[u][j].w);
       }
     }
+  }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int c = n0 + 8 * j + 2 * t4;
-      if (c >= p.ds) continue;                                 // ds is a multiple of 4
-      const float b0 = c < p.d ? p.dt_bias[h * p.d + c] : 0.f, b1 = c + 1 < p.d ? p.dt_bias[h * p.d + c + 1] : 0.f;
+  for (int j = 0; j < 4; ++j) {
+    const int c = n0 + 8 * j + 2 * t4;
+    if (c >= p.ds) continue;                                   // ds is a multiple of 4
+    const float b0 = c < p.d ? p.dt_bias[h * p.d + c] : 0.f, b1 = c + 1 < p.d ? p.dt_bias[h * p.d + c + 1] : 0.f;
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
-        if (g + 8 * i < tokens)
-          *reinterpret_cast<float2*>(p.g + ((row + g + 8 * i) * p.H + h) * p.ds + c) =
-              make_float2(c < p.d ? decay_of(acc[j][2 * i] + b0) : 0.f, c + 1 < p.d ? decay_of(acc[j][2 * i + 1] + b1) : 0.f);
-    }
+    for (int i = 0; i < 2; ++i)
+      if (g + 8 * i < tokens)
+        *reinterpret_cast<float2*>(p.g + ((row + g + 8 * i) * p.H + h) * p.ds + c) =
+            make_float2(c < p.d ? decay_of(acc[j][2 * i] + b0) : 0.f, c + 1 < p.d ? decay_of(acc[j][2 * i + 1] + b1) : 0.f);
   }
 }
 
 // A warp per (slot, tile of kPrepRows tokens).  The first G slots are key heads (q and k), then come value channels (64 VP of them
-// a slot), step sizes and decays (32 heads a slot) and the heads of channel decays.  NP: channel pairs per lane of a key head
+// a slot), step sizes and decays (32 heads a slot) and the channel decays (a head a slot, with low-rank logits 32 channels of one).  NP: channel pairs per lane of a key head
 // (d <= 64 NP).  STEP: segments of one token (decode): nothing is read ahead, which leaves registers for more channels at once.
 template <bool STEP> constexpr int value_pairs() { return STEP ? 4 : 2; }
 template <typename T, int NP, int TAPS, bool STEP, int RULE>
@@ -105,11 +112,24 @@ recurrence_prepare_kernel(const RecPrep<T> p) {
   const int vslots = (p.H * p.e + 64 * VP - 1) / (64 * VP), cslots = (p.H + 31) / 32;
   pdl_wait();
   pdl_launch_dependents();
+  const int slot = blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
+  auto low_rank_slot = [&](size_t row, int tokens) {
+    if constexpr (RULE == kGated && sizeof(T) == 2) {
+      const int chunks = (p.ds + 31) / 32, i = slot - p.G - vslots - cslots;
+      if (i < p.H * chunks)
+        low_rank_decays(p, i / chunks, i % chunks * 32, row, tokens,
+                        [&](float logit) { return exp_of<T>(-p.rate * softplus_of<T>(-logit)); });
+    }
+  };
+  if (RULE == kGated && STEP && p.low && slot >= p.G + vslots + cslots) {
+    // decays do not depend on what request a token belongs to: 16 rows of the step at a time
+    if ((blockIdx.y & 15) == 0) low_rank_slot(blockIdx.y, min(16, p.sg.num - static_cast<int>(blockIdx.y)));
+    return;
+  }
   int s, off;
   if (!find_tile(p.sg, kPrepRows, blockIdx.y, s, off)) return;
-  const int slot = blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
-  if (slot >= p.G + vslots + cslots + (p.g ? p.H : 0)) return;
+  if (slot >= p.G + vslots + cslots + (p.g ? p.H * (p.low ? (p.ds + 31) / 32 : 1) : 0)) return;
   const int count = p.sg.count[s], end = min(count, off + kPrepRows);
   const bool fresh = p.sg.pos0[s] == 0;
   const size_t row0 = p.sg.row0[s];
@@ -248,17 +268,13 @@ recurrence_prepare_kernel(const RecPrep<T> p) {
       }
       p.coef[r * p.H + h] = make_float2(beta, decay);
     }
+  } else if (RULE == kGated && p.low) {
+    low_rank_slot(row0 + off, end - off);
   } else if constexpr (RULE != kSsd) {
     const int h = slot - p.G - vslots - cslots;
     // sigmoid(x)^rate = exp(-rate softplus(-x))
     const float rate = RULE == kGated ? -p.rate : -expf(p.a_log[h]), sign = RULE == kGated ? -1.f : 1.f;
     auto decay_of = [&](float logit) { return exp_of<T>(rate * softplus_of<T>(sign * logit)); };
-    if constexpr (RULE == kGated && sizeof(T) == 2) {
-      if (p.low) {
-        low_rank_decays(p, h, row0 + off, end - off, decay_of);
-        return;
-      }
-    }
     constexpr int AH = STEP ? 1 : 4;
     for (int c0 = lane; c0 < p.ds; c0 += 128) {                // four channels x AH tokens read at once
       float dt[4];
@@ -797,7 +813,7 @@ static RecWalk<T> rec_walk(const CbRecWalk* a, const CbSegments* seg) {
 template <typename T, int NP, int TAPS, int RULE>
 static int prep_go(const RecPrep<T>& p, int tiles, cudaStream_t st) {
   auto go = [&](auto kernel, int vp) {
-    const int slots = p.G + (p.H * p.e + 64 * vp - 1) / (64 * vp) + (p.H + 31) / 32 + (p.g ? p.H : 0);
+    const int slots = p.G + (p.H * p.e + 64 * vp - 1) / (64 * vp) + (p.H + 31) / 32 + (p.g ? p.H * (p.low ? (p.ds + 31) / 32 : 1) : 0);
     return static_cast<int>(launch(kernel, dim3((slots + kPrepWarps - 1) / kPrepWarps, tiles), dim3(32 * kPrepWarps), 0, st, p));
   };
   if (p.sg.single) return go(recurrence_prepare_kernel<T, NP, TAPS, true, RULE>, value_pairs<true>());

@@ -105,7 +105,7 @@ class LayeredRunner(StepRunner):
                         recurrent.append((s.heads, s.groups, s.state, s.vdim, False))
                     else:
                         recurrent.append((s.heads, s.heads, s.dim, s.vdim, True))
-                    if getattr(m, "low", None) is not None:
+                    if getattr(m, "low", None) is not None and (isinstance(m, DeltaWeights) or act == torch.float32):
                         self._need("low", m.low.n)
         self._scratch = {n: torch.zeros(T * c, dtype=act, device=dev) for n, c in self._scratch.items()}
         self.recurrence = K.RecurrenceScratch(T, recurrent, act, dev) if recurrent else None
@@ -252,9 +252,7 @@ class LayeredRunner(StepRunner):
     def _gated_linear(self, m: GatedLinearWeights, proj, run: _StateRun, b, out, decode: bool) -> int:
         s, T, n = m.spec, proj.shape[0], 1
         low, a = m.low, proj[:, m.a_off:m.a_off + m.low.k]
-        # the preparation makes the decay logits itself, 16 tokens of a request at a time; steps of many single tokens and 32-bit
-        # models leave it to a product
-        if proj.dtype != torch.bfloat16 or decode and T > 64:
+        if proj.dtype != torch.bfloat16:       # bf16: the preparation makes the decay logits itself
             z = self._rows("low", T, low.n)
             K.wide_gemm(a, low, z, ws=self.ws)
             low, a, n = None, z, 2
