@@ -190,7 +190,7 @@ def bench_sequential_rows(m: int, width: int, side: int, flush, pk) -> list[dict
     h, x = torch.randn(m, width, **bf), torch.randn(m, width, device=DEV)
     w = wq_pack.swiglu_interleave(wq_pack.pack_bf16(torch.randn(2 * ff, width, device=DEV) * 0.02))
     act, nw = torch.empty(m, ff, **bf), torch.ones(width, device=DEV)
-    glu = timeit_graph(lambda: K.wide_gemm(h, w, act, gelu_glu=True), flush, launches=5)
+    glu = timeit_graph(lambda: K.wide_gemm(h, w, act, glu="gelu"), flush, launches=5)
     silu = timeit_graph(lambda: K.wq_gemm_act(h, w, out=act), flush, launches=5)
     gate, table = torch.randn(side, width, **bf), torch.randn(4096, 8 * side, **bf)
     ids, g = torch.randint(0, 4096, (m,), device=DEV, dtype=torch.int32), torch.zeros(m, -(-side // 64) * 64, **bf)

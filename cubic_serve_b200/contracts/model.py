@@ -91,7 +91,7 @@ class LatentCacheSpec:
 
 @dataclass(frozen=True)
 class DeltaStateSpec:
-    """Recurrent state of a layered decoder's recurrent runs (fp32 state and convolution inputs)."""
+    """State of a layered decoder's runs that keep some per request (fp32 recurrences, convolution inputs)."""
     runs: int
     bytes_per_request: int
 
@@ -149,9 +149,9 @@ class ModelSpec:
     @staticmethod
     def from_layered(cfg, manifest: WeightManifest | None = None) -> "ModelSpec":
         """Of a layered decoder (``models/layered.py``): every layer RUN has its own cache or state."""
-        from ..models.layered import ATTENTION_SPECS, RECURRENT_SPECS
-        attn, recurrent = cfg.run_parts(ATTENTION_SPECS), cfg.run_parts(RECURRENT_SPECS)
-        state = DeltaStateSpec(recurrent, cfg.state_bytes_per_request) if recurrent else None
+        from ..models.layered import ATTENTION_SPECS
+        attn, stateful = cfg.run_parts(ATTENTION_SPECS), cfg.state_runs
+        state = DeltaStateSpec(stateful, cfg.state_bytes_per_request) if stateful else None
         return ModelSpec(cfg.name, cfg.family, digest_of(dataclasses.asdict(cfg)), LatentCacheSpec(cfg.page_bytes, attn), state,
                          manifest)
 

@@ -362,7 +362,7 @@ def decoder_step_operators(cfg, rows: int, tp_size: int = 1, topology_id: str = 
 
 def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple[OpSignature, ...]:
     """Operator signatures of one decode step of a layered decoder: the distinct operators of its layer runs."""
-    from ..models.layered import AttentionSpec, DeltaSpec, LatentSpec, SsdSpec
+    from ..models.layered import AttentionSpec, BiasedAttentionSpec, ConvAttentionSpec, DeltaSpec, LatentSpec, SsdSpec
     W, act = cfg.hidden_size, "fp32" if cfg.dtype == "float32" else "bf16"
     ops: dict[tuple, OpSignature] = {}
 
@@ -384,6 +384,10 @@ def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple
             elif isinstance(m, AttentionSpec):
                 add("attention.gqa", "paged", m.out_width, (m.heads + m.kv_heads) * m.dim, heads=m.heads,
                     window=m.window or cfg.max_position)
+            elif isinstance(m, (ConvAttentionSpec, BiasedAttentionSpec)):
+                k = (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim
+                extra = {"taps": m.conv, "keep": m.keep} if isinstance(m, ConvAttentionSpec) else {"buckets": m.buckets}
+                add("attention.gqa", "paged", m.out_width, k, heads=m.heads, window=m.window or cfg.max_position, **extra)
             elif isinstance(m, DeltaSpec):
                 add("delta_rule." + ("channel" if m.per_channel else "head"), "state32", m.out_width, m.channels, heads=m.heads,
                     taps=m.conv)
@@ -398,6 +402,15 @@ def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple
                 add("linear.bf16", "down", W, l.ff)
         else:
             add("linear.bf16", "parallel_out", W, l.mixer.out_width + l.ff)
+        if l.routed is not None:
+            r = l.routed
+            add("moe.route", f"top{r.top}", W, W, experts=r.experts, identity=r.identity)
+            add("linear.bf16", "experts_up", r.ff, W, experts=r.experts)
+            add("linear.bf16", "experts_down", W, r.ff, experts=r.experts)
+            if r.shared_ff:
+                add("linear.bf16", "down", W, r.shared_ff)
+        if cfg.streams > 1:
+            add("residual.streams", "residual32", W, W, streams=cfg.streams)
         if cfg.side_dim:
             add("token_side", "residual32", W, cfg.side_dim)
     add("linear.bf16", "lm_head", cfg.vocab_size, W)

@@ -1,15 +1,16 @@
-// Grouped-query attention of the layered decoders over a paged cache in the activation type: head norms, rotary pairs, a sliding
-// window and a softmax entry without a value (sink).  A value is the raw key of its token, as projected.
+// Grouped-query attention of the layered decoders over a paged cache in the activation type: a sliding window, first tokens that
+// stay visible behind it, a bias per distance and head, and a softmax entry without a value (sink).
 //
 //   gqa_prepare_kernel    RMS norm of every query and key head, rotary positions on neighbouring channel pairs; keys and values
-//                         to their page
+//                         to their page, where a value is the raw key of its token, as projected (qkv_prepare.cu has the others)
 //   gqa_prefill_kernel    bf16: blocks of (token, head) rows of one key head on the tensor cores
 //   gqa_decode_kernel,    bf16, one token per segment: the query heads of a key head are the rows, a warp walks whole pages;
 //   gqa_merge_kernel      key splits are merged in split order
 //   gqa_row_kernel        fp32 models: a warp per (token, head)
 //
-// The cache is [pages][key head][key, value][16][P], P the head width rounded up to 64, zero columns behind the head.  Scores,
-// softmax weights and sums are fp32; the weights are rounded to bf16 as the operand of the second product of the bf16 kernels.
+// The cache is [pages][key head][key, value][16][P], P the wider of the key and value widths rounded up to 64, zero columns behind
+// the head.  Scores, softmax weights and sums are fp32; the weights are rounded to bf16 as the operand of the second product of the bf16 kernels.
+#include <climits>
 #include <type_traits>
 
 #include "segments.cuh"
@@ -116,10 +117,22 @@ struct GqaAttn {
   const T* cache;
   const int* page_table;      // [slots, max_pages]
   int max_pages;
-  int H, G, d, P, window;     // window <= 0: every earlier token
+  int H, G, e, P, window;     // e: width of a value; window <= 0: every earlier token
+  int keep;                   // the first tokens, visible whatever the window (0 without a window)
   float scale, out_scale;
   float sink;                 // score of the entry without a value, -inf: none
+  const float* bias;          // [bias_far + 1, H] added to the scaled score by distance (the last row from bias_far on), null: none
+  int bias_far;
   Segments sg;
+};
+
+// Keys of a query tile [pos0, pos0 + toks): the window's from `kmin` (a page's first key) on, and the kept ones below it, [0, kept)
+struct GqaSpan {
+  int kmin, kept;
+  __device__ __forceinline__ GqaSpan(int window, int keep, int pos0) {
+    kmin = window > 0 ? max(0, pos0 - window + 1) & ~(kGqaPage - 1) : 0;
+    kept = min(keep, kmin);
+  }
 };
 
 // ------------------------------------------------------------------ fp32
@@ -146,7 +159,9 @@ gqa_row_kernel(const GqaAttn<float> p) {
     acc[i] = 0.f;
   }
   float m = p.sink, l = p.sink == -INFINITY ? 0.f : 1.f;
-  for (int j = lo; j <= pos; ++j) {
+  const int kept = min(p.keep, lo);
+  for (int i = 0; i < kept + pos + 1 - lo; ++i) {
+    const int j = i < kept ? i : lo + i - kept;
     const float* kr = p.cache + ((static_cast<size_t>(pages[j / kGqaPage]) * p.G + kh) * 2 * kGqaPage + j % kGqaPage) * p.P;
     const float* vr = kr + kGqaPage * p.P;
     float v[NR], sdot = 0.f;
@@ -156,6 +171,7 @@ gqa_row_kernel(const GqaAttn<float> p) {
       sdot = fmaf(q[i], kr[lane + 32 * i], sdot);
     }
     sdot = warp_sum(sdot);
+    if (p.bias) sdot += __ldg(p.bias + static_cast<size_t>(min(pos - j, p.bias_far)) * p.H + h);
     const float mn = fmaxf(m, sdot);
     const float f = expf(m - mn), w = expf(sdot - mn);
     m = mn;
@@ -164,11 +180,11 @@ gqa_row_kernel(const GqaAttn<float> p) {
     for (int i = 0; i < NR; ++i) acc[i] = fmaf(w, v[i], acc[i] * f);
   }
   const float g = p.out_scale / l;
-  float* orow = p.out + row * p.ldo + h * p.d;
+  float* orow = p.out + row * p.ldo + h * p.e;
 #pragma unroll
   for (int i = 0; i < NR; ++i) {
     const int c = lane + 32 * i;
-    if (c < p.d) orow[c] = acc[i] * g;
+    if (c < p.e) orow[c] = acc[i] * g;
   }
 }
 
@@ -186,6 +202,7 @@ struct GqaMma {
   int hb, qb;                 // heads and tokens of a block (hb * qb rows at most)
   int head_tiles;             // blocks of hb heads that share a key head
   int splits;
+  int bias_rows;              // prompts: rows of the bias table kept in shared memory (bias_far + 1), 0: read in place
   float* partial;             // decode: [segment][key head tile][split][16][P + 2]
 };
 
@@ -201,7 +218,8 @@ __device__ __forceinline__ void store_pair(bf16* row, int c, int d, float x, flo
 // Four warps of 16 rows each, row = token * hb + head; key tiles of 64 keys in two buffers, 16-byte chunks XOR-swizzled by the
 // row.  A warp keeps its rows' scores, weights and outputs in registers: no exchange between warps.
 static constexpr int kGqaWarps = 4;
-template <int NCH>
+static constexpr int kGqaBiasBytes = 11 << 10;      // three blocks of two column groups and their tables fit on an SM
+template <int NCH, bool BIAS>
 __global__ void __launch_bounds__(32 * kGqaWarps, NCH <= 2 ? 3 : 1)
 gqa_prefill_kernel(const GqaMma p) {
   constexpr int P = NCH * 64, ROWB = P * 2, NW = kGqaWarps, MR = 16 * NW, KT = 64, CH = P / 8, NT = P / 8;
@@ -209,6 +227,7 @@ gqa_prefill_kernel(const GqaMma p) {
   constexpr bool QREG = NCH <= 2;                     // query fragments in registers; the rows pass through the second buffer
   uint8_t* kvs = lsm + (QREG ? 0 : MR * ROWB);        // [2 buffers][key, value][KT][ROWB]
   uint8_t* qs = QREG ? kvs + 2 * KT * ROWB : lsm;     // [MR][ROWB]
+  float* table = reinterpret_cast<float*>(kvs + 4 * KT * ROWB);        // [bias_rows][hb], times log2 e
   pdl_wait();
   pdl_launch_dependents();
   const GqaAttn<bf16>& a = p.a;
@@ -221,9 +240,12 @@ gqa_prefill_kernel(const GqaMma p) {
   const size_t row0 = static_cast<size_t>(a.sg.row0[s]) + off;
   const int pos0 = a.sg.pos0[s] + off;
   const int* pages = a.page_table + static_cast<size_t>(a.sg.slot[s]) * a.max_pages;
-  const int kmin = a.window > 0 ? max(0, pos0 - a.window + 1) & ~(kGqaPage - 1) : 0;
+  const GqaSpan span(a.window, a.keep, pos0);
+  const int kmin = span.kmin, kept_tiles = (span.kept + KT - 1) / KT;
   const int kend = pos0 + toks;
-  const int tiles = (kend - kmin + KT - 1) / KT;
+  const int tiles = kept_tiles + (kend - kmin + KT - 1) / KT;
+  // tiles of kept tokens come first; a tile's first key and the end of its keys
+  auto tile_key = [&](int t) { return t < kept_tiles ? t * KT : kmin + (t - kept_tiles) * KT; };
 
   auto load_tile = [&](int t, int b) {
     const uint32_t dst0 = smem_u32(kvs + b * 2 * KT * ROWB);
@@ -231,8 +253,8 @@ gqa_prefill_kernel(const GqaMma p) {
     for (int i = 0; i < KT * CH / (32 * NW); ++i) {
       const int idx = tid + i * 32 * NW;
       const int r = idx / CH, c = idx % CH;
-      const int key = kmin + t * KT + r;
-      const bool ok = key < kend;
+      const int key = tile_key(t) + r;
+      const bool ok = key < (t < kept_tiles ? span.kept : kend);
       const int page = ok ? pages[key / kGqaPage] : 0;
       const bf16* src = a.cache + ((static_cast<size_t>(page) * a.G + kh) * 2 * kGqaPage + key % kGqaPage) * P + c * 8;
       const uint32_t at = dst0 + r * ROWB + ((c ^ (r & 7)) << 4);
@@ -240,6 +262,12 @@ gqa_prefill_kernel(const GqaMma p) {
       cp_async16(at + KT * ROWB, src + kGqaPage * P, ok);
     }
   };
+  if constexpr (BIAS) {
+    for (int idx = tid; idx < p.bias_rows * p.hb; idx += 32 * NW) {
+      const int n = idx / p.hb, h = idx - n * p.hb;
+      table[idx] = h < heads ? __ldg(a.bias + static_cast<size_t>(n) * a.H + h0 + h) * kLog2e : 0.f;
+    }
+  }
   for (int idx = tid; idx < MR * CH; idx += 32 * NW) {
     const int r = idx / CH, c = idx % CH;
     const int tok = r / p.hb, h = r - tok * p.hb;
@@ -252,12 +280,19 @@ gqa_prefill_kernel(const GqaMma p) {
 
   // visible keys of the thread's two rows; rows without a query see none
   int lim_lo[2], lim_hi[2];
+  int row_pos[2], row_h[2];                            // for the bias: position and head of the two rows
+  float far[2];                                        // bias from bias_far on
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int r = warp * 16 + g + 8 * i;
     const int tok = r / p.hb, h = r - tok * p.hb;
     lim_hi[i] = tok < toks && h < heads ? pos0 + tok : -1;
     lim_lo[i] = a.window > 0 ? pos0 + tok - a.window + 1 : 0;
+    if constexpr (BIAS) {
+      row_pos[i] = pos0 + tok;
+      row_h[i] = h < heads ? h : 0;
+      far[i] = __ldg(a.bias + static_cast<size_t>(a.bias_far) * a.H + h0 + row_h[i]) * kLog2e;
+    }
   }
   // of the whole warp
   const int tok_a = min(warp * 16 / p.hb, toks - 1), tok_b = min((warp * 16 + 15) / p.hb, toks - 1);
@@ -294,8 +329,9 @@ gqa_prefill_kernel(const GqaMma p) {
     asm volatile("cp.async.commit_group;" ::: "memory");
     asm volatile("cp.async.wait_group 1;" ::: "memory");
     __syncthreads();
-    const int key_t = kmin + t * KT;
-    if (!idle && key_t <= see_hi && key_t + KT > see_lo) {
+    const int key_t = tile_key(t);
+    const bool kept = t < kept_tiles;
+    if (!idle && key_t <= see_hi && (key_t + KT > see_lo || key_t < a.keep)) {
       const uint32_t k_base = smem_u32(kvs + b * 2 * KT * ROWB), v_base = k_base + KT * ROWB;
       float sf[8][4];
 #pragma unroll
@@ -317,12 +353,35 @@ gqa_prefill_kernel(const GqaMma p) {
       }
       const bool whole = key_t >= all_lo && key_t + KT - 1 <= all_hi;
       float mx[2] = {m2[0], m2[1]};
+      // a key is seen behind the window's start, or among the first tokens; a kept tile has no others
+      const int seen_low = kept ? span.kept : a.keep;
+      const int seen_from[2] = {kept ? INT_MAX : lim_lo[0], kept ? INT_MAX : lim_lo[1]};
+      if constexpr (BIAS) {
+        if (pos0 + tok_a - (key_t + KT - 1) >= a.bias_far) {             // the same for every distance of the tile
+#pragma unroll
+          for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) sf[j][c] = fmaf(sf[j][c], sc, far[c >> 1]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+              const int key = key_t + j * 8 + 2 * t4 + (c & 1), i = c >> 1;
+              const int n = min(max(row_pos[i] - key, 0), a.bias_far);
+              const float b = p.bias_rows ? table[n * p.hb + row_h[i]]
+                                          : __ldg(a.bias + static_cast<size_t>(n) * a.H + h0 + row_h[i]) * kLog2e;
+              sf[j][c] = fmaf(sf[j][c], sc, b);
+            }
+        }
+      }
 #pragma unroll
       for (int j = 0; j < 8; ++j)
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           const int key = key_t + j * 8 + 2 * t4 + (c & 1), i = c >> 1;
-          sf[j][c] = whole || (key >= lim_lo[i] && key <= lim_hi[i]) ? sf[j][c] * sc : -INFINITY;
+          const float v = BIAS ? sf[j][c] : sf[j][c] * sc;
+          sf[j][c] = whole || ((key >= seen_from[i] || key < seen_low) && key <= lim_hi[i]) ? v : -INFINITY;
           mx[i] = fmaxf(mx[i], sf[j][c]);
         }
       float al[2], use[2];
@@ -368,9 +427,9 @@ gqa_prefill_kernel(const GqaMma p) {
     const int tok = r / p.hb, h = r - tok * p.hb;
     if (tok >= toks || h >= heads) continue;
     const float f = a.out_scale / (l2[i] + ex2(a.sink * kLog2e - m2[i]));
-    bf16* row = a.out + (row0 + tok) * a.ldo + (h0 + h) * a.d;
+    bf16* row = a.out + (row0 + tok) * a.ldo + (h0 + h) * a.e;
 #pragma unroll
-    for (int j = 0; j < NT; ++j) store_pair(row, j * 8 + 2 * t4, a.d, o[j][2 * i] * f, o[j][2 * i + 1] * f);
+    for (int j = 0; j < NT; ++j) store_pair(row, j * 8 + 2 * t4, a.e, o[j][2 * i] * f, o[j][2 * i + 1] * f);
   }
 }
 
@@ -379,7 +438,7 @@ gqa_prefill_kernel(const GqaMma p) {
 // a product are the query heads of the key head (up to 16 of them).
 static constexpr int kRing = 3;
 
-template <int NCH>
+template <int NCH, bool BIAS>
 __global__ void __launch_bounds__(128)
 gqa_decode_kernel(const GqaMma p) {
   constexpr int P = NCH * 64, ROWB = P * 2, CH = P / 8, NT = P / 8, PAGEB = 2 * kGqaPage * ROWB;
@@ -396,13 +455,16 @@ gqa_decode_kernel(const GqaMma p) {
   const int pos = a.sg.pos0[s];
   const int* pages = a.page_table + static_cast<size_t>(a.sg.slot[s]) * a.max_pages;
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-  const int pg_all = pos / kGqaPage + 1, pg_first = lo / kGqaPage, per = (pg_all - pg_first + p.splits - 1) / p.splits;
-  const int pg_lo = min(pg_all, pg_first + static_cast<int>(blockIdx.z) * per), pg_hi = min(pg_all, pg_lo + per);
+  // the pages to walk: those with kept tokens below the window, then the window's
+  const int pg_first = lo / kGqaPage, kept_pages = (min(a.keep, pg_first * kGqaPage) + kGqaPage - 1) / kGqaPage;
+  const int skip = pg_first - kept_pages;             // pages between the two
+  const int pg_all = pos / kGqaPage + 1 - skip, per = (pg_all + p.splits - 1) / p.splits;
+  const int pg_lo = min(pg_all, static_cast<int>(blockIdx.z) * per), pg_hi = min(pg_all, pg_lo + per);
   uint8_t* ring = lsm + warp * kRing * PAGEB;
 
-  auto load_page = [&](int pg, int b) {               // nothing behind the last page
-    if (pg < pg_hi) {
-      const bf16* src = a.cache + (static_cast<size_t>(pages[pg]) * a.G + kh) * 2 * kGqaPage * P;
+  auto load_page = [&](int at, int b) {               // nothing behind the last page
+    if (at < pg_hi) {
+      const bf16* src = a.cache + (static_cast<size_t>(pages[at < kept_pages ? at : at + skip]) * a.G + kh) * 2 * kGqaPage * P;
       const uint32_t dst0 = smem_u32(ring + b * PAGEB);
 #pragma unroll
       for (int i = 0; i < 2 * kGqaPage * CH / 32; ++i) {
@@ -437,8 +499,32 @@ gqa_decode_kernel(const GqaMma p) {
     v_at[i] = (lane & 15) * ROWB + (((i * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
   }
   int b = 0;
-  for (int pg = pg_lo + warp; pg < pg_hi; pg += 4) {
-    load_page(pg + 4 * (kRing - 1), (b + kRing - 1) % kRing);
+  int bias_h[2] = {0, 0};
+  float far[2] = {0.f, 0.f};
+  if constexpr (BIAS) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      bias_h[i] = h0 + min(g + 8 * i, heads - 1);
+      far[i] = __ldg(a.bias + static_cast<size_t>(a.bias_far) * a.H + bias_h[i]) * kLog2e;
+    }
+  }
+  for (int at = pg_lo + warp; at < pg_hi; at += 4) {
+    const int pg = at < kept_pages ? at : at + skip;
+    load_page(at + 4 * (kRing - 1), (b + kRing - 1) % kRing);
+    float bv[2][4];
+    if constexpr (BIAS) {
+      const bool near = pos - (pg * kGqaPage + kGqaPage - 1) < a.bias_far;
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          bv[j][c] = far[c >> 1];
+          if (near) {
+            const int n = min(max(pos - (pg * kGqaPage + j * 8 + 2 * t4 + (c & 1)), 0), a.bias_far);
+            bv[j][c] = __ldg(a.bias + static_cast<size_t>(n) * a.H + bias_h[c >> 1]) * kLog2e;
+          }
+        }
+    }
     asm volatile("cp.async.wait_group %0;" ::"n"(kRing - 1) : "memory");
     __syncwarp();
     const uint32_t k_base = smem_u32(ring + b * PAGEB), v_base = k_base + kGqaPage * ROWB;
@@ -457,7 +543,8 @@ gqa_decode_kernel(const GqaMma p) {
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int key = pg * kGqaPage + j * 8 + 2 * t4 + (c & 1);
-        sf[j][c] = key >= lo && key <= pos ? (sf[j][c] + s2[j][c]) * sc : -INFINITY;
+        const float v = sf[j][c] + s2[j][c];
+        sf[j][c] = (key >= lo || key < a.keep) && key <= pos ? (BIAS ? fmaf(v, sc, bv[j][c]) : v * sc) : -INFINITY;
         mx[c >> 1] = fmaxf(mx[c >> 1], sf[j][c]);
       }
     float use[2], al[2];
@@ -537,7 +624,7 @@ gqa_decode_kernel(const GqaMma p) {
         v.y = fmaf(f[w], u.y, v.y);
       }
       if (p.splits > 1) *reinterpret_cast<float2*>(part + c) = v;
-      else store_pair(a.out + row * a.ldo + (h0 + r) * a.d, c, a.d, v.x * scale, v.y * scale);
+      else store_pair(a.out + row * a.ldo + (h0 + r) * a.e, c, a.e, v.x * scale, v.y * scale);
     }
     if (p.splits > 1 && lane == 0) *reinterpret_cast<float2*>(part + P) = make_float2(mx, l);
   }
@@ -575,9 +662,9 @@ gqa_merge_kernel(const GqaMma p) {
     }
   }
   const float f = a.out_scale / l;
-  bf16* row = a.out + static_cast<size_t>(a.sg.row0[s]) * a.ldo + (kh * R + hq0 + r) * a.d;
+  bf16* row = a.out + static_cast<size_t>(a.sg.row0[s]) * a.ldo + (kh * R + hq0 + r) * a.e;
 #pragma unroll
-  for (int i = 0; i < NCH; ++i) store_pair(row, 2 * (lane + 32 * i), a.d, v[i].x * f, v[i].y * f);
+  for (int i = 0; i < NCH; ++i) store_pair(row, 2 * (lane + 32 * i), a.e, v[i].x * f, v[i].y * f);
 }
 
 // ------------------------------------------------------------------ host
@@ -593,19 +680,29 @@ static int gqa_go(K kernel, dim3 grid, int threads, size_t smem, const GqaMma& p
   return static_cast<int>(launch(kernel, grid, dim3(threads), smem, st, p));
 }
 
-template <int NCH>
+template <int NCH, bool BIAS>
 static int gqa_prefill(const GqaMma& p, dim3 grid, cudaStream_t st) {
   static bool configured[64] = {};
-  return gqa_go(gqa_prefill_kernel<NCH>, grid, 32 * kGqaWarps, static_cast<size_t>((NCH <= 2 ? 0 : 16 * kGqaWarps) + 256) * NCH * 128, p,
-                configured, st);
+  const size_t rows = static_cast<size_t>((NCH <= 2 ? 0 : 16 * kGqaWarps) + 256) * NCH * 128;
+  return gqa_go(gqa_prefill_kernel<NCH, BIAS>, grid, 32 * kGqaWarps, rows + (BIAS ? kGqaBiasBytes : 0), p, configured, st);
 }
 
-template <int NCH>
+template <int NCH, bool BIAS>
 static int gqa_decode(const GqaMma& p, dim3 grid, cudaStream_t st) {
   static bool configured[64] = {};
-  const int rc = gqa_go(gqa_decode_kernel<NCH>, grid, 128, static_cast<size_t>(4) * kRing * 2 * kGqaPage * NCH * 128, p, configured, st);
+  const int rc = gqa_go(gqa_decode_kernel<NCH, BIAS>, grid, 128, static_cast<size_t>(4) * kRing * 2 * kGqaPage * NCH * 128, p, configured, st);
   if (rc || p.splits == 1) return rc;
   return static_cast<int>(launch(gqa_merge_kernel<NCH>, dim3(grid.x, grid.y, 4), dim3(128), 0, st, p));
+}
+
+template <bool BIAS>
+static int gqa_mma(const GqaMma& p, int nch, bool decode, dim3 grid, cudaStream_t st) {
+  switch (nch) {
+    case 1: return decode ? gqa_decode<1, BIAS>(p, grid, st) : gqa_prefill<1, BIAS>(p, grid, st);
+    case 2: return decode ? gqa_decode<2, BIAS>(p, grid, st) : gqa_prefill<2, BIAS>(p, grid, st);
+    case 3: return decode ? gqa_decode<3, BIAS>(p, grid, st) : gqa_prefill<3, BIAS>(p, grid, st);
+  }
+  return decode ? gqa_decode<4, BIAS>(p, grid, st) : gqa_prefill<4, BIAS>(p, grid, st);
 }
 
 }  // namespace cb
@@ -632,8 +729,10 @@ struct CbGqaAttn {
   void* out; int ldo;
   const void* cache;
   const void* page_table;
-  int max_pages, H, G, d, P, window;
+  int max_pages, H, G, e, P, window, keep;
   float scale, out_scale, sink;
+  const void* bias;           // fp32 [bias_far + 1, H] or null
+  int bias_far;
   int tokens, f32;
   int decode;                 // every segment has at most one row, row s belongs to segment s
   int splits;                 // key splits of the decode form (1 = none)
@@ -671,7 +770,8 @@ int cb_gqa_prepare(const CbGqaPrep* a, void* stream) {
 int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
   using namespace cb;
   if (!a || !seg || seg->num <= 0 || a->tokens <= 0) return 0;
-  if (a->H <= 0 || a->G <= 0 || (a->H % a->G) || a->d <= 0 || a->P < a->d || a->P > 256 || (a->P & 63) || a->ldo < a->H * a->d) return -10;
+  if (a->H <= 0 || a->G <= 0 || (a->H % a->G) || a->e <= 0 || a->P < a->e || a->P > 256 || (a->P & 63) || a->ldo < a->H * a->e) return -10;
+  if (a->keep < 0 || (a->bias && a->bias_far < 0)) return -13;
   if (a->splits > 1 && (!a->decode || !a->partial || a->splits > 65535)) return -12;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   auto fill = [&](auto& p) {
@@ -680,7 +780,9 @@ int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
     p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
     p.cache = static_cast<const T*>(a->cache);
     p.page_table = static_cast<const int*>(a->page_table); p.max_pages = a->max_pages;
-    p.H = a->H; p.G = a->G; p.d = a->d; p.P = a->P; p.window = a->window;
+    p.H = a->H; p.G = a->G; p.e = a->e; p.P = a->P; p.window = a->window;
+    p.keep = a->window > 0 ? a->keep : 0;
+    p.bias = static_cast<const float*>(a->bias); p.bias_far = a->bias_far;
     p.scale = a->scale; p.out_scale = a->out_scale; p.sink = a->sink;
     p.sg = make_segments(seg, a->tokens);
   };
@@ -698,18 +800,14 @@ int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
   GqaMma p;
   fill(p.a);
   p.splits = a->splits > 1 ? a->splits : 1;
+  p.bias_rows = 0;
   p.partial = static_cast<float*>(a->partial);
   if (a->decode) {
     p.hb = 16; p.qb = 1;
     p.head_tiles = (a->H / a->G + 15) / 16;
     const dim3 grid(seg->num, a->G * p.head_tiles, p.splits);
     if (grid.y > 65535) return -11;
-    switch (a->P / 64) {
-      case 1: return gqa_decode<1>(p, grid, st);
-      case 2: return gqa_decode<2>(p, grid, st);
-      case 3: return gqa_decode<3>(p, grid, st);
-    }
-    return gqa_decode<4>(p, grid, st);
+    return a->bias ? gqa_mma<true>(p, a->P / 64, true, grid, st) : gqa_mma<false>(p, a->P / 64, true, grid, st);
   }
   const int R = a->H / a->G;
   p.hb = min(R, 16 * kGqaWarps);
@@ -717,12 +815,9 @@ int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
   p.head_tiles = (R + p.hb - 1) / p.hb;
   const dim3 grid(max_tiles(a->tokens, seg->num, p.qb), a->G * p.head_tiles);
   if (grid.y > 65535) return -11;
-  switch (a->P / 64) {
-    case 1: return gqa_prefill<1>(p, grid, st);
-    case 2: return gqa_prefill<2>(p, grid, st);
-    case 3: return gqa_prefill<3>(p, grid, st);
-  }
-  return gqa_prefill<4>(p, grid, st);
+  const long long rows = static_cast<long long>(a->bias_far) + 1;
+  p.bias_rows = a->bias && rows * p.hb * 4 <= kGqaBiasBytes ? static_cast<int>(rows) : 0;
+  return a->bias ? gqa_mma<true>(p, a->P / 64, false, grid, st) : gqa_mma<false>(p, a->P / 64, false, grid, st);
 }
 
 }  // extern "C"

@@ -585,7 +585,8 @@ struct F32Gemm {
   const float* residual;
   float* y2; int ldy2, n_split, diag_n;
   int M, N, K;
-  int glu;                    // gated gelu: 16 gate rows and 16 up rows of w in turn, y gets N / 2 features
+  int glu;                    // gated silu (1) or gelu (2): 16 gate rows and 16 up rows of w in turn, y gets N / 2 features
+  const int* tiles;           // grouped: work list {count, then {expert, first row, up to 64 rows}}, w stacks the experts; null: one matrix
 };
 
 __global__ void __launch_bounds__(256)
@@ -593,19 +594,28 @@ f32_gemm_kernel(const F32Gemm p) {
   constexpr int BM = 64, BN = 64, BK = 16;
   __shared__ float xs[BK][BM + 4];
   __shared__ float ws[BK][BN + 4];
-  const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
+  const int n0 = blockIdx.x * BN;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   pdl_wait();
   pdl_launch_dependents();
+  int m0 = blockIdx.y * BM, m_end = p.M;
+  const __nv_bfloat16* wm = p.w;
+  if (p.tiles) {
+    const int item = blockIdx.y;
+    if (item >= p.tiles[0]) return;
+    wm += static_cast<size_t>(p.tiles[1 + 3 * item]) * p.N * p.K;
+    m0 = p.tiles[2 + 3 * item];
+    m_end = min(p.M, m0 + min(BM, p.tiles[3 + 3 * item]));
+  }
   const int xc0 = p.diag_n ? (n0 / p.diag_n) * p.K : 0;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < p.K; k0 += BK) {
     for (int i = threadIdx.x; i < BM * BK; i += 256) {
       const int r = i / BK, k = i % BK;
       const int m = m0 + r, c = xc0 + k0 + k;
-      xs[k][r] = (m < p.M && k0 + k < p.K && c < p.x_cols) ? p.x[static_cast<size_t>(m) * p.ldx + c] : 0.f;
+      xs[k][r] = (m < m_end && k0 + k < p.K && c < p.x_cols) ? p.x[static_cast<size_t>(m) * p.ldx + c] : 0.f;
       const int n = n0 + r;
-      ws[k][r] = (n < p.N && k0 + k < p.K) ? __bfloat162float(p.w[static_cast<size_t>(n) * p.K + k0 + k]) : 0.f;
+      ws[k][r] = (n < p.N && k0 + k < p.K) ? __bfloat162float(wm[static_cast<size_t>(n) * p.K + k0 + k]) : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -630,7 +640,8 @@ f32_gemm_kernel(const F32Gemm p) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float u = __shfl_down_sync(0xffffffffu, acc[i][j], 4);
-        if (!(tx & 4) && m < p.M && f + j < (p.N >> 1)) p.y[static_cast<size_t>(m) * p.ldy + f + j] = gelu_tanh(acc[i][j]) * u;
+        if (!(tx & 4) && m < m_end && f + j < (p.N >> 1))
+          p.y[static_cast<size_t>(m) * p.ldy + f + j] = (p.glu == 1 ? acc[i][j] / (1.f + expf(-acc[i][j])) : gelu_tanh(acc[i][j])) * u;
       }
     }
     return;
@@ -638,7 +649,7 @@ f32_gemm_kernel(const F32Gemm p) {
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
-    if (m >= p.M) continue;
+    if (m >= m_end) continue;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
@@ -806,6 +817,7 @@ struct CbF32Gemm {
   void* y2; int ldy2, n_split, diag_n;
   int M, N, K;
   int glu;
+  const void* tiles; int max_items;       // grouped form (see F32Gemm)
 };
 
 int cb_f32_gemm(const CbF32Gemm* a, void* stream) {
@@ -820,8 +832,10 @@ int cb_f32_gemm(const CbF32Gemm* a, void* stream) {
   p.y2 = static_cast<float*>(a->y2); p.ldy2 = a->ldy2; p.n_split = a->n_split; p.diag_n = a->diag_n;
   p.M = a->M; p.N = a->N; p.K = a->K;
   p.glu = a->glu;
-  if (p.glu && (p.glu != 2 || p.y2 || p.residual || p.diag_n || (p.N % 32) != 0 || p.ldy < p.N / 2)) return -13;
-  const dim3 grid((a->N + 63) / 64, (a->M + 63) / 64);
+  p.tiles = static_cast<const int*>(a->tiles);
+  if (p.tiles && (a->max_items <= 0 || a->diag_n || a->glu || a->residual)) return -14;
+  if (p.glu && (p.glu < 1 || p.glu > 2 || p.y2 || p.residual || p.diag_n || (p.N % 32) != 0 || p.ldy < p.N / 2)) return -13;
+  const dim3 grid((a->N + 63) / 64, p.tiles ? a->max_items : (a->M + 63) / 64);
   if (grid.y > 65535) return -12;
   return static_cast<int>(launch(f32_gemm_kernel, grid, dim3(256), 0, static_cast<cudaStream_t>(stream), p));
 }

@@ -14,6 +14,7 @@
 // kernels serve EP = 1 and the EP shards whose partial outputs are then reduced
 // like any row-parallel partial sum.
 #include "ptx.cuh"
+#include "launch.cuh"
 
 namespace cb {
 
@@ -173,9 +174,199 @@ moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ 
   }
 }
 
+// ------------------------------------------------------------------ scored routing (layered decoders)
+// Router logits and everything up to the weights are fp32: s = softmax(z) over all `outputs` (more than `experts`: the rest return
+// the token itself), the `top` largest s + correction are chosen (lowest id on ties), their weights are s over the sum of the
+// chosen.  A route's rank among its expert's comes from the expert's counter.
+struct ScoredRoute {
+  const float* z; int ldz;    // [T, ldz]
+  const float* correction;    // [outputs]
+  int T, experts, outputs, top;
+  int* ids;                   // [T, top] expert, -1: none (the token itself)
+  int* rank;                  // [T, top] in: nothing, out: rank among the expert's routes
+  float* weight;              // [T, top]
+  float* self;                // [T] summed weight of the token itself
+  int* counts;                // [experts], zero on entry
+};
+
+static constexpr int kMaxScoredTop = 32;
+
+__global__ void __launch_bounds__(128)
+scored_route_kernel(const ScoredRoute p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= p.T) return;
+  float s[8], c[8], mx = -INFINITY;
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int e = lane + 32 * j;
+    s[j] = e < p.outputs ? p.z[static_cast<size_t>(t) * p.ldz + e] : -INFINITY;
+    if (!(s[j] == s[j])) s[j] = -INFINITY;
+    mx = fmaxf(mx, s[j]);
+  }
+  mx = warp_max(mx);
+  if (mx == -INFINITY) mx = 0.f;
+  float sum = 0.f;
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    s[j] = expf(s[j] - mx);
+    sum += s[j];
+  }
+  sum = warp_sum(sum);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int e = lane + 32 * j;
+    s[j] /= sum;
+    c[j] = e < p.outputs ? s[j] + __ldg(p.correction + e) : -INFINITY;
+    if (e < p.outputs && !(c[j] > -INFINITY)) c[j] = -3.0e38f;           // never chosen before a real score, always a valid id
+  }
+  float mine = 0.f;                                                      // lane r holds the r-th choice
+  int expert = -1;
+  for (int r = 0; r < p.top; ++r) {
+    float bv = -INFINITY, bs = 0.f;
+    int be = 0x7fffffff;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int e = lane + 32 * j;
+      if (e < p.outputs && (c[j] > bv || (c[j] == bv && c[j] > -INFINITY && e < be))) { bv = c[j]; be = e; bs = s[j]; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o), os = __shfl_xor_sync(0xffffffffu, bs, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+      if (ov > bv || (ov == bv && oe < be)) { bv = ov; be = oe; bs = os; }
+    }
+    if (lane == r) { mine = bs; expert = be; }
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+      if (lane + 32 * j == be) c[j] = -INFINITY;
+  }
+  const float w = mine / (warp_sum(mine) + 1e-20f);
+  const bool routed = lane < p.top && expert >= 0 && expert < p.experts;
+  const float own = warp_sum(lane < p.top && !routed ? w : 0.f);
+  if (lane == 0) p.self[t] = own;
+  if (lane < p.top) {
+    const size_t i = static_cast<size_t>(t) * p.top + lane;
+    p.ids[i] = routed ? expert : -1;
+    p.weight[i] = w;
+    p.rank[i] = routed ? atomicAdd(p.counts + expert, 1) : -1;
+  }
+}
+
+struct RouteScatter {
+  const void* x; int ldx;     // [T, ldx] elements of `elem` bytes, W of them are copied
+  void* xs; int ldxs;         // [routes, ldxs] rows by expert
+  int T, W, elem, top, experts, mb;
+  const int* ids;
+  int* pos;                   // in: rank, out: place in xs (-1: none)
+  int* counts;                // zero again on exit
+  int* done;                  // blocks that are through, zero on entry and exit
+  int* tiles;                 // work list of the grouped products: {count, then {expert, first row, rows}}
+};
+
+// Every block derives the experts' first rows from the counts; block 0 writes the work list.  A warp copies a route's row.
+__global__ void __launch_bounds__(256)
+route_scatter_kernel(const RouteScatter p) {
+  __shared__ int rows[256], items[256];
+  __shared__ int last;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int e = threadIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int cnt = e < p.experts ? p.counts[e] : 0, nt = (cnt + p.mb - 1) / p.mb;
+  rows[e] = cnt;
+  items[e] = nt;
+  __syncthreads();
+  for (int o = 1; o < p.experts; o <<= 1) {
+    const int a = e >= o ? rows[e - o] : 0, b = e >= o ? items[e - o] : 0;
+    __syncthreads();
+    rows[e] += a;
+    items[e] += b;
+    __syncthreads();
+  }
+  const int first = rows[e] - cnt, t0 = items[e] - nt;
+  __syncthreads();
+  rows[e] = first;
+  if (blockIdx.x == 0) {
+    for (int i = 0; i < nt; ++i) {
+      p.tiles[1 + 3 * (t0 + i)] = e;
+      p.tiles[2 + 3 * (t0 + i)] = first + i * p.mb;
+      p.tiles[3 + 3 * (t0 + i)] = min(p.mb, cnt - i * p.mb);
+    }
+    if (e == p.experts - 1) p.tiles[0] = t0 + nt;
+  }
+  __syncthreads();
+  const size_t bytes = static_cast<size_t>(p.W) * p.elem;
+  const bool vec = (bytes & 15) == 0 && ((static_cast<size_t>(p.ldx) * p.elem) & 15) == 0 && ((static_cast<size_t>(p.ldxs) * p.elem) & 15) == 0;
+  for (int route = blockIdx.x * 8 + warp; route < p.T * p.top; route += 8 * gridDim.x) {
+    const int ex = p.ids[route];
+    if (ex < 0) continue;                                                // its place is -1 already
+    const int at = rows[ex] + p.pos[route];
+    const char* src = static_cast<const char*>(p.x) + static_cast<size_t>(route / p.top) * p.ldx * p.elem;
+    char* dst = static_cast<char*>(p.xs) + static_cast<size_t>(at) * p.ldxs * p.elem;
+    if (vec) {
+      for (size_t i = lane; i < (bytes >> 4); i += 32) reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+    } else if (p.elem == 2) {
+      for (int i = lane; i < p.W; i += 32) reinterpret_cast<uint16_t*>(dst)[i] = reinterpret_cast<const uint16_t*>(src)[i];
+    } else {
+      for (int i = lane; i < p.W; i += 32) reinterpret_cast<uint32_t*>(dst)[i] = reinterpret_cast<const uint32_t*>(src)[i];
+    }
+    __syncwarp();
+    if (lane == 0) p.pos[route] = at;
+  }
+  // the last block through leaves the counters as it found them: every block has read them by then
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    __threadfence();
+    last = atomicAdd(p.done, 1) == static_cast<int>(gridDim.x) - 1;
+  }
+  __syncthreads();
+  if (last) {
+    if (e < p.experts) p.counts[e] = 0;
+    if (e == 0) *p.done = 0;
+  }
+}
+
 }  // namespace cb
 
 extern "C" {
+
+struct CbScoredMoe {
+  const void* z; int ldz;
+  const void* correction;
+  const void* x; int ldx;
+  void* xs; int ldxs;
+  int T, W, elem, experts, outputs, top, mb;
+  void* ids;
+  void* pos;
+  void* weight;
+  void* self;
+  void* counts;               // int [experts + 1], zero between launches
+  void* tiles;                // int [1 + 3 (ceil(T top / mb) + experts)]
+};
+
+// Routing from fp32 logits and permutation of the rows to their experts (see ScoredRoute and RouteScatter).
+int cb_scored_moe_route(const CbScoredMoe* a, void* stream) {
+  using namespace cb;
+  if (!a || a->T <= 0) return 0;
+  if (a->experts < 1 || a->outputs < a->experts || a->outputs > 256 || a->top < 1 || a->top > kMaxScoredTop || a->top > a->outputs) return -10;
+  if (a->W <= 0 || (a->elem != 2 && a->elem != 4) || a->ldx < a->W || a->ldxs < a->W || a->mb <= 0 || a->ldz < a->outputs) return -11;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  ScoredRoute r;
+  r.z = static_cast<const float*>(a->z); r.ldz = a->ldz; r.correction = static_cast<const float*>(a->correction);
+  r.T = a->T; r.experts = a->experts; r.outputs = a->outputs; r.top = a->top;
+  r.ids = static_cast<int*>(a->ids); r.rank = static_cast<int*>(a->pos); r.weight = static_cast<float*>(a->weight);
+  r.self = static_cast<float*>(a->self); r.counts = static_cast<int*>(a->counts);
+  cudaError_t e = launch(scored_route_kernel, dim3((a->T + 3) / 4), dim3(128), 0, st, r);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  RouteScatter s;
+  s.x = a->x; s.ldx = a->ldx; s.xs = a->xs; s.ldxs = a->ldxs;
+  s.T = a->T; s.W = a->W; s.elem = a->elem; s.top = a->top; s.experts = a->experts; s.mb = a->mb;
+  s.ids = r.ids; s.pos = r.rank; s.counts = r.counts; s.done = r.counts + a->experts; s.tiles = static_cast<int*>(a->tiles);
+  const long long routes = static_cast<long long>(a->T) * a->top;
+  const int blocks = static_cast<int>(routes / 8 + 1 < 148 * 8 ? (routes + 7) / 8 : 148 * 8);
+  return static_cast<int>(launch(route_scatter_kernel, dim3(blocks), dim3(256), 0, st, s));
+}
 
 // Routing + permutation in one call: zeroes the counts, selects the top-k, scans, scatters the rows.
 // Buffers: topk_ids [T,k] i32, topk_w [T,k] f32, counts/offsets/cursors [expert_count] i32, total [1] i32,

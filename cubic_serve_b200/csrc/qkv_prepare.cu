@@ -1,0 +1,408 @@
+// Queries, keys and values of the layered decoders' attention on their way from the projection to the padded queries and the paged
+// cache of gqa_attn.cu (values of their own; gqa_attn.cu prepares the layers whose values are raw keys).
+//
+//   conv_qkv_kernel   short causal convolution over time on every channel, rotary positions on the halves of a head's first
+//                     channels, every query and key head over its root mean square
+//   norm_qkv_kernel   queries and keys of a token over the root mean square of their whole projection, times a weight per channel;
+//                     queries times a factor that grows with the position
+//
+// A warp takes a head, lane l the channels 4 l .. and 128 + 4 l ..; everything between the projection and the stored row is fp32.
+#include <type_traits>
+
+#include "segments.cuh"
+#include "launch.cuh"
+
+namespace cb {
+
+static constexpr int kQkvPage = 16;
+static constexpr int kQkvWarps = 4;
+static constexpr int kQkvTokens = 16;       // of a conv_qkv_kernel block; at least the convolution's history (taps - 1)
+
+// Four channels c .. c + 3 of a row of d; `vec`: rows start at multiples of four elements and d is one
+__device__ __forceinline__ float4 load_four(const float* p, int c, int d, bool vec) {
+  if (vec) return c < d ? *reinterpret_cast<const float4*>(p + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  return make_float4(c < d ? p[c] : 0.f, c + 1 < d ? p[c + 1] : 0.f, c + 2 < d ? p[c + 2] : 0.f, c + 3 < d ? p[c + 3] : 0.f);
+}
+__device__ __forceinline__ float4 load_four(const __nv_bfloat16* p, int c, int d, bool vec) {
+  if (vec) {
+    uint2 u = make_uint2(0u, 0u);
+    if (c < d) u = *reinterpret_cast<const uint2*>(p + c);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+  return make_float4(c < d ? to_f(p[c]) : 0.f, c + 1 < d ? to_f(p[c + 1]) : 0.f, c + 2 < d ? to_f(p[c + 2]) : 0.f,
+                     c + 3 < d ? to_f(p[c + 3]) : 0.f);
+}
+__device__ __forceinline__ void store_four(float* p, int c, float4 v) { *reinterpret_cast<float4*>(p + c) = v; }
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, int c, float4 v) {
+  *reinterpret_cast<uint2*>(p + c) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+__device__ __forceinline__ float4 fma_four(float4 a, float4 b, float4 c) {
+  return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w));
+}
+__device__ __forceinline__ float4 mul_four(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
+__device__ __forceinline__ float dot_four(float4 a, float4 b) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w))); }
+
+template <typename T>
+struct QkvPrep {
+  const T* x; int ldx;        // projections
+  int q_off, k_off, v_off;    // columns of q [H d], k [G d] and v [G e]
+  T* q;                       // [T, H, P]
+  T* cache;                   // [pages][G][key, value][16][P]
+  const int* slots;           // [T] cache row, < 0: none
+  int H, G, d, e, P;
+  float eps;
+  int vec;                    // four channels at a time
+
+  // Where token t's row of item `it` (H queries, G keys, G values) goes, null: nowhere
+  __device__ __forceinline__ T* row(int it, size_t t, int slot) const {
+    if (it < H) return q + (t * H + it) * P;
+    if (slot < 0) return nullptr;
+    const bool value = it >= H + G;
+    const int g = it - H - (value ? G : 0);
+    return cache + (((static_cast<size_t>(slot / kQkvPage) * G + g) * 2 + value) * kQkvPage + slot % kQkvPage) * P;
+  }
+  __device__ __forceinline__ int col(int it) const { return it < H ? q_off + it * d : it < H + G ? k_off + (it - H) * d : v_off + (it - H - G) * e; }
+  __device__ __forceinline__ int width(int it) const { return it < H + G ? d : e; }
+};
+
+template <typename T>
+struct ConvQkv {
+  QkvPrep<T> a;
+  const float* w;             // [taps][ldw], column 0 is the first query's; the last row multiplies the current input
+  int ldw, taps;
+  T* state;                   // [slots, taps - 1, ldw]: a request's last inputs
+  const float* freq;          // [2][pairs] radians per position, and what they were rounded by
+  int pairs;
+  const int* positions;
+  Segments sg;
+};
+
+// A block takes a tile of tokens of one segment and the heads blockIdx.y, + gridDim.y, ... by warps.  TAPS: 0 any number.  NJ: 128-channel
+// chunks of a head.
+template <typename T, int TAPS, int NJ>
+__global__ void __launch_bounds__(32 * kQkvWarps)
+conv_qkv_kernel(const ConvQkv<T> p) {
+  constexpr int R = TAPS > 0 ? TAPS : 1, BATCH = NJ == 1 ? 4 : 2;
+  extern __shared__ __align__(16) float2 turn[];                       // [tokens][pairs] cosine and sine, then the warps' rows
+  pdl_wait();
+  pdl_launch_dependents();
+  int s, off;
+  if (!find_tile(p.sg, kQkvTokens, blockIdx.x, s, off)) return;
+  const QkvPrep<T>& a = p.a;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int count = p.sg.count[s], toks = min(kQkvTokens, count - off);
+  const size_t row0 = p.sg.row0[s];                                    // first row of the segment
+  const bool fresh = p.sg.pos0[s] == 0;
+  const int hist_rows = p.taps - 1;
+  T* st = p.state + static_cast<size_t>(p.sg.slot[s]) * hist_rows * p.ldw;
+  const int half = p.pairs, dims = 2 * half;
+  for (int i = threadIdx.x; i < toks * half; i += 32 * kQkvWarps) {
+    const int t = i / half, j = i - t * half;
+    // the rounding error of the product is put back: angles of far positions keep their fraction of a turn
+    const float pos = static_cast<float>(p.positions[row0 + off + t]), f = p.freq[j];
+    const float ang = pos * f, e = fmaf(pos, f, -ang) + pos * p.freq[half + j];
+    float sn, cs;
+    sincosf(ang, &sn, &cs);
+    const float ce = fmaf(-0.5f * e, e, 1.f), se = e * fmaf(e * (-1.f / 6.f), e, 1.f);
+    turn[i] = make_float2(cs * ce - sn * se, fmaf(sn, ce, cs * se));
+  }
+  __syncthreads();
+  float* swap = reinterpret_cast<float*>(turn + kQkvTokens * half + (half * kQkvTokens & 1)) + warp * 256;
+  const bool vec = a.vec, vec_turn = (half & 3) == 0;
+  for (int it = blockIdx.y * kQkvWarps + warp; it < a.H + 2 * a.G; it += kQkvWarps * gridDim.y) {
+    const int d = a.width(it), col = a.col(it), wc = col - a.q_off;
+    const bool value = it >= a.H + a.G;
+    const T* xr = a.x + row0 * a.ldx + col;
+    // input at token t of the segment (t >= -(taps - 1)), channels of chunk j
+    auto input = [&](int t, int j) {
+      const int c = 4 * lane + 128 * j;
+      if (t >= 0) return load_four(xr + static_cast<size_t>(t) * a.ldx, c, d, vec);
+      if (fresh) return make_float4(0.f, 0.f, 0.f, 0.f);
+      return load_four(st + static_cast<size_t>(t + hist_rows) * p.ldw + wc, c, d, vec);
+    };
+    auto tap = [&](int k, int j) { return load_four(p.w + static_cast<size_t>(k) * p.ldw + wc, 4 * lane + 128 * j, d, vec); };
+    float4 w[R][NJ], hist[R][NJ];
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int k = 0; k < TAPS; ++k)
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) w[k][j] = tap(k, j);
+#pragma unroll
+      for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) hist[k][j] = input(off + k - (TAPS - 1), j);
+    }
+    for (int t0 = 0; t0 < toks; t0 += BATCH) {
+      float4 in[BATCH][NJ];
+      if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int b = 0; b < BATCH; ++b)                                // several tokens in flight; nothing behind the tile
+#pragma unroll
+          for (int j = 0; j < NJ; ++j)
+            in[b][j] = t0 + b < toks ? input(off + t0 + b, j) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll
+      for (int b = 0; b < BATCH; ++b) {
+        const int t = t0 + b;
+        if (t >= toks) break;
+        float4 v[NJ];
+        if constexpr (TAPS > 0) {
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) {
+            float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int k = 0; k < TAPS - 1; ++k) acc = fma_four(w[k][j], hist[k][j], acc);
+            v[j] = fma_four(w[TAPS - 1][j], in[b][j], acc);
+#pragma unroll
+            for (int k = 0; k + 1 < TAPS - 1; ++k) hist[k][j] = hist[k + 1][j];
+            if constexpr (TAPS > 1) hist[TAPS - 2][j] = in[b][j];
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) {
+            v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 1
+            for (int k = 0; k < p.taps; ++k) v[j] = fma_four(tap(k, j), input(off + t - hist_rows + k, j), v[j]);
+          }
+        }
+        if (!value) {
+          if (half) {
+            __syncwarp();                                              // the row before this one was read
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) store_four(swap, 4 * lane + 128 * j, v[j]);
+            __syncwarp();
+            const float2* tr = turn + t * half;
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) {
+              const int c = 4 * lane + 128 * j;
+              if (c >= dims) continue;
+              if (vec_turn) {                                          // four channels turn with four neighbours
+                const bool hi = c >= half;
+                const float4 o = *reinterpret_cast<const float4*>(swap + (hi ? c - half : c + half));
+                const float4 r0 = *reinterpret_cast<const float4*>(tr + (hi ? c - half : c));
+                const float4 r1 = *reinterpret_cast<const float4*>(tr + (hi ? c - half : c) + 2);
+                const float sg = hi ? 1.f : -1.f;
+                v[j] = make_float4(fmaf(v[j].x, r0.x, sg * o.x * r0.y), fmaf(v[j].y, r0.z, sg * o.y * r0.w),
+                                   fmaf(v[j].z, r1.x, sg * o.z * r1.y), fmaf(v[j].w, r1.z, sg * o.w * r1.w));
+              } else {
+                float* vp = &v[j].x;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                  const int ch = c + i;
+                  if (ch >= dims) continue;
+                  const bool hi = ch >= half;
+                  const float2 r = tr[hi ? ch - half : ch];
+                  const float o = swap[hi ? ch - half : ch + half];
+                  vp[i] = fmaf(vp[i], r.x, (hi ? o : -o) * r.y);
+                }
+              }
+            }
+          }
+          float ss = 0.f;
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) ss += dot_four(v[j], v[j]);
+          const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(d) + a.eps);
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) v[j] = mul_four(v[j], inv);
+        }
+        const size_t tok = row0 + off + t;
+        T* dst = a.row(it, tok, a.slots[tok]);
+        if (!dst) continue;
+#pragma unroll
+        for (int j = 0; j < NJ; ++j)
+          if (4 * lane + 128 * j < a.P) store_four(dst, 4 * lane + 128 * j, v[j]);
+      }
+    }
+    // The last inputs become the state: by the tile with the segment's first tokens, the only reader of the old one.  A lane reads
+    // and writes its own channels; entry k takes entry k + count, which is read before it is written.
+    if (off == 0) {
+#pragma unroll 1
+      for (int k = 0; k < hist_rows; ++k)
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const int c = 4 * lane + 128 * j;
+          if (c >= d) continue;
+          const float4 n = input(count - hist_rows + k, j);
+          T* dst = st + static_cast<size_t>(k) * p.ldw + wc;
+          if (vec) {
+            store_four(dst, c, n);
+          } else {
+            dst[c] = from_f<T>(n.x);
+            if (c + 1 < d) dst[c + 1] = from_f<T>(n.y);
+            if (c + 2 < d) dst[c + 2] = from_f<T>(n.z);
+            if (c + 3 < d) dst[c + 3] = from_f<T>(n.w);
+          }
+        }
+    }
+  }
+}
+
+template <typename T>
+struct NormQkv {
+  QkvPrep<T> a;
+  const float* qw;            // [H d]
+  const float* kw;            // [G d]
+  const int* positions;
+  float coef;                 // queries times 1 + coef ln(floor((position + 1) / every) + 1); every 0: no factor
+  int every;
+};
+
+static constexpr int kNormWarps = 8;
+
+// A block takes a token.
+template <typename T>
+__global__ void __launch_bounds__(32 * kNormWarps)
+norm_qkv_kernel(const NormQkv<T> p) {
+  __shared__ float part[2][kNormWarps];
+  pdl_wait();
+  pdl_launch_dependents();
+  const QkvPrep<T>& a = p.a;
+  const size_t t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* xr = a.x + t * a.ldx;
+  const bool vec = a.vec;
+  const int nq = a.H * a.d, nk = a.G * a.d;
+  float ss[2] = {0.f, 0.f};
+  for (int c = 4 * threadIdx.x; c < nq; c += 128 * kNormWarps) { const float4 v = load_four(xr + a.q_off, c, nq, vec); ss[0] += dot_four(v, v); }
+  for (int c = 4 * threadIdx.x; c < nk; c += 128 * kNormWarps) { const float4 v = load_four(xr + a.k_off, c, nk, vec); ss[1] += dot_four(v, v); }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    ss[i] = warp_sum(ss[i]);
+    if (lane == 0) part[i][warp] = ss[i];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < 2; ++i) ss[i] = warp_sum(lane < kNormWarps ? part[i][lane] : 0.f);
+  float fq = 1.f / sqrtf(ss[0] / static_cast<float>(nq) + a.eps);
+  const float fk = 1.f / sqrtf(ss[1] / static_cast<float>(nk) + a.eps);
+  if (p.every > 0) fq *= fmaf(p.coef, logf(static_cast<float>((p.positions[t] + 1) / p.every + 1)), 1.f);
+  const int slot = a.slots[t];
+  for (int it = warp; it < a.H + 2 * a.G; it += kNormWarps) {
+    T* dst = a.row(it, t, slot);
+    if (!dst) continue;
+    const int d = a.width(it);
+    const T* src = xr + a.col(it);
+    const float f = it < a.H ? fq : fk;
+    const float* w = it < a.H ? p.qw + it * a.d : p.kw + (it - a.H) * a.d;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int c = 4 * lane + 128 * j;
+      if (c >= a.P) continue;
+      float4 v = load_four(src, c, d, vec);
+      if (it < a.H + a.G) {
+        const float4 g = load_four(w, c, d, vec);
+        v = make_float4(v.x * f * g.x, v.y * f * g.y, v.z * f * g.z, v.w * f * g.w);
+      }
+      store_four(dst, c, v);
+    }
+  }
+}
+
+}  // namespace cb
+
+extern "C" {
+
+struct CbQkvPrep {
+  const void* x; int ldx, q_off, k_off, v_off;
+  void* q;
+  void* cache;
+  const void* slots;
+  const void* positions;
+  int H, G, d, e, P;
+  float eps;
+  int tokens, f32;
+};
+
+struct CbConvQkv {
+  CbQkvPrep a;
+  const void* w; int ldw, taps;
+  void* state;
+  const void* freq; int pairs;
+};
+
+struct CbNormQkv {
+  CbQkvPrep a;
+  const void* qw;
+  const void* kw;
+  float coef; int every;
+};
+
+}  // extern "C"
+
+namespace cb {
+
+static int qkv_check(const CbQkvPrep& a) {
+  if (a.H <= 0 || a.G <= 0 || a.d <= 0 || a.e <= 0 || a.P < a.d || a.P < a.e || a.P > 256 || (a.P & 63)) return -10;
+  if (a.q_off < 0 || a.k_off < a.q_off + a.H * a.d || a.v_off < a.k_off + a.G * a.d || a.ldx < a.v_off + a.G * a.e) return -11;
+  return 0;
+}
+
+template <typename T>
+static QkvPrep<T> qkv_fill(const CbQkvPrep& a) {
+  QkvPrep<T> p;
+  p.x = static_cast<const T*>(a.x); p.ldx = a.ldx; p.q_off = a.q_off; p.k_off = a.k_off; p.v_off = a.v_off;
+  p.q = static_cast<T*>(a.q); p.cache = static_cast<T*>(a.cache); p.slots = static_cast<const int*>(a.slots);
+  p.H = a.H; p.G = a.G; p.d = a.d; p.e = a.e; p.P = a.P; p.eps = a.eps;
+  p.vec = ((a.d | a.e | a.ldx | a.q_off | a.k_off | a.v_off) & 3) == 0;
+  return p;
+}
+
+}  // namespace cb
+
+extern "C" {
+
+int cb_conv_qkv(const CbConvQkv* c, const CbSegments* seg, void* stream) {
+  using namespace cb;
+  if (!c || !seg || seg->num <= 0 || c->a.tokens <= 0) return 0;
+  if (const int rc = qkv_check(c->a)) return rc;
+  if (c->taps < 1 || c->taps - 1 > kQkvTokens || c->pairs < 0 || 2 * c->pairs > c->a.d) return -12;
+  if (c->ldw < c->a.v_off - c->a.q_off + c->a.G * c->a.e || (c->taps > 1 && !c->state) || !c->w || (c->pairs && !c->freq)) return -13;
+  const int tiles = max_tiles(c->a.tokens, seg->num, kQkvTokens), items = c->a.H + 2 * c->a.G;
+  // enough warps for the device: at most one head each
+  const int groups = (items + kQkvWarps - 1) / kQkvWarps;
+  const int ny = min(groups, max(1, 148 * 12 / tiles));
+  const size_t smem = (static_cast<size_t>(kQkvTokens) * c->pairs + 1) * 8 + kQkvWarps * 256 * 4;
+  auto go = [&](auto kernel, auto p) {
+    using T = std::remove_pointer_t<decltype(p.a.q)>;
+    p.a = qkv_fill<T>(c->a);
+    p.a.vec = p.a.vec && (c->ldw & 3) == 0;
+    p.w = static_cast<const float*>(c->w); p.ldw = c->ldw; p.taps = c->taps;
+    p.state = static_cast<T*>(c->state);
+    p.freq = static_cast<const float*>(c->freq); p.pairs = c->pairs;
+    p.positions = static_cast<const int*>(c->a.positions);
+    p.sg = make_segments(seg, c->a.tokens);
+    return static_cast<int>(launch(kernel, dim3(tiles, ny), dim3(32 * kQkvWarps), smem, static_cast<cudaStream_t>(stream), p));
+  };
+  auto pick = [&](auto p) {
+    using T = std::remove_pointer_t<decltype(p.a.q)>;
+    const bool one = c->a.P <= 128;
+    switch (c->taps) {
+      case 1: return one ? go(conv_qkv_kernel<T, 1, 1>, p) : go(conv_qkv_kernel<T, 1, 2>, p);
+      case 2: return one ? go(conv_qkv_kernel<T, 2, 1>, p) : go(conv_qkv_kernel<T, 2, 2>, p);
+      case 3: return one ? go(conv_qkv_kernel<T, 3, 1>, p) : go(conv_qkv_kernel<T, 3, 2>, p);
+      case 4: return one ? go(conv_qkv_kernel<T, 4, 1>, p) : go(conv_qkv_kernel<T, 4, 2>, p);
+    }
+    return go(conv_qkv_kernel<T, 0, 2>, p);
+  };
+  return c->a.f32 ? pick(ConvQkv<float>{}) : pick(ConvQkv<__nv_bfloat16>{});
+}
+
+int cb_norm_qkv(const CbNormQkv* c, void* stream) {
+  using namespace cb;
+  if (!c || c->a.tokens <= 0) return 0;
+  if (const int rc = qkv_check(c->a)) return rc;
+  if (!c->qw || !c->kw || c->every < 0) return -12;
+  auto go = [&](auto kernel, auto p) {
+    using T = std::remove_pointer_t<decltype(p.a.q)>;
+    p.a = qkv_fill<T>(c->a);
+    p.qw = static_cast<const float*>(c->qw); p.kw = static_cast<const float*>(c->kw);
+    p.positions = static_cast<const int*>(c->a.positions);
+    p.coef = c->coef; p.every = c->every;
+    return static_cast<int>(launch(kernel, dim3(c->a.tokens), dim3(32 * kNormWarps), 0, static_cast<cudaStream_t>(stream), p));
+  };
+  return c->a.f32 ? go(norm_qkv_kernel<float>, NormQkv<float>{}) : go(norm_qkv_kernel<__nv_bfloat16>, NormQkv<__nv_bfloat16>{});
+}
+
+}  // extern "C"

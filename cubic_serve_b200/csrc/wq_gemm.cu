@@ -798,6 +798,7 @@ struct WqLaunchOpts {
   int swiglu = 0;                      // fused SwiGLU epilogue (gate / up rows interleaved)
   int cluster_splitk = -1;             // -1: the process default; 0 / 1: workspace / cluster reduction for this launch
   bool stream_k = false;
+  int squared_relu = 0;                // bf16 weights: every feature leaves through the squared relu
   int min_units = 0;
   long long workspace_bytes = 0;
   const struct CbWideGemm* wide = nullptr;   // bf16 weights: wide epilogue and block-diagonal weights
@@ -936,7 +937,7 @@ static int wq_gemm_dispatch(int fmt, const void* x, int ldx, const void* codes, 
   if (o.wide) {
     const CbWideGemm& g = *o.wide;
     if (fmt != kFmtBf16 || residual || link || o.swiglu || o.tiles || g.x_cols <= 0 || g.x_cols > ldx) return -61;
-    if ((!g.y && !g.y32) || (g.y && g.y32) || (g.y2 && (g.y32 || (g.n_split & 3) || g.n_split < 0))) return -62;
+    if ((!g.y && !g.y32) || (g.y && g.y32) || (g.y2 && ((g.n_split & 3) || g.n_split < 0 || (g.y32 && g.residual32)))) return -62;
     if (g.glu && (!g.y || g.y2 || g.diag_n || g.glu < 0 || g.glu > kGluGelu || (N % 32) != 0 || ldy < N / 2)) return -64;
     p.swiglu = g.glu;
     if (g.diag_n && (stream_k || g.diag_n < 0 || (g.diag_n % kTileN) != 0)) return -63;
@@ -946,6 +947,13 @@ static int wq_gemm_dispatch(int fmt, const void* x, int ldx, const void* codes, 
     p.y2 = static_cast<__nv_bfloat16*>(g.y2);
     p.ldy2 = g.ldy2; p.n_split = g.n_split; p.diag_n = g.diag_n;
     x_cols = static_cast<uint64_t>(g.x_cols);
+  }
+  if (o.squared_relu) {
+    if (fmt != kFmtBf16 || o.wide || o.swiglu || residual || link) return -65;
+    p.wide = 1;
+    p.y2 = p.y;
+    p.ldy2 = ldy;
+    p.n_split = 0;
   }
   if (p.swiglu && (residual || (link && (link->mode & kTpScatterPush)))) return -51;
   p.tp.mode = kTpNone;
@@ -1100,7 +1108,7 @@ int cb_wq_gemm_resident_pairs(int fmt) { return cb::streamk_resident_pairs(fmt);
 static int wq_gemm_grouped_launch(int fmt, const void* x, int ldx, const void* codes, const void* meta, void* y, int ldy,
                                   float alpha, int total_rows, int N, int K, int group_k, const void* tiles,
                                   int max_items, int mb, int num_experts, long long code_stride, long long meta_stride,
-                                  void* status, void* stream, int swiglu) {
+                                  void* status, void* stream, int swiglu, int squared_relu = 0) {
   if (!tiles || max_items <= 0 || mb <= 0 || mb > 256 || (mb % 16) != 0 || num_experts <= 0) return -40;
   WqLaunchOpts o;
   o.num_experts = num_experts;
@@ -1110,6 +1118,7 @@ static int wq_gemm_grouped_launch(int fmt, const void* x, int ldx, const void* c
   o.max_items = max_items;
   o.mb_hint = mb;
   o.swiglu = swiglu;
+  o.squared_relu = squared_relu;
   o.stream_k = g_grouped_persistent.load(std::memory_order_relaxed) != 0;
   // the tensor map spans all rows; every work item starts at its own row offset
   return wq_gemm_dispatch(fmt, x, ldx, codes, meta, y, ldy, nullptr, alpha, total_rows, N, K, group_k, 1, nullptr,
@@ -1132,6 +1141,14 @@ int cb_wq_gemm_grouped(int fmt, const void* x, int ldx, const void* codes, const
                        void* stream) {
   return wq_gemm_grouped_launch(fmt, x, ldx, codes, meta, y, ldy, alpha, total_rows, N, K, group_k, tiles, max_items, mb,
                                 num_experts, code_stride, meta_stride, status, stream, 0);
+}
+
+// Grouped projection of bf16 experts whose features leave as max(v, 0)^2.
+int cb_wq_gemm_grouped_relu2(const void* x, int ldx, const void* w, void* y, int ldy, int total_rows, int N, int K, const void* tiles,
+                             int max_items, int mb, int num_experts, void* status, void* stream) {
+  if (ldy < N) return -50;
+  return wq_gemm_grouped_launch(cb::kFmtBf16, x, ldx, w, nullptr, y, ldy, 1.f, total_rows, N, K, K, tiles, max_items, mb, num_experts, 0, 0,
+                                status, stream, 0, 1);
 }
 
 // W8A8 on the fp8 tensor-core path (tcgen05.mma.kind::f8f6f4, e4m3 x e4m3, fp32 accumulate):

@@ -194,7 +194,8 @@ __device__ __forceinline__ void store_act4(const WqGemmParams& p, int m, int n_t
 __device__ __forceinline__ void store_wide4(const WqGemmParams& p, int m, int n0, float (&v)[4]) {
   if (n0 >= p.N) return;
   const bool whole = n0 + 3 < p.N;
-  if (p.y32) {
+  const bool second = p.y2 && n0 >= p.n_split;
+  if (p.y32 && !second) {
     const size_t off = static_cast<size_t>(m) * p.ldy + n0;
     if (whole && (p.ldy & 3) == 0) {
       float4 o = make_float4(v[0], v[1], v[2], v[3]);
@@ -212,7 +213,7 @@ __device__ __forceinline__ void store_wide4(const WqGemmParams& p, int m, int n0
   }
   __nv_bfloat16* dst;
   bool vec;
-  if (p.y2 && n0 >= p.n_split) {
+  if (second) {
     // the projection is rounded to bf16 before the activation, as a separate activation kernel would read it
 #pragma unroll
     for (int j = 0; j < 4; ++j) {

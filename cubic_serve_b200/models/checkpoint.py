@@ -338,6 +338,7 @@ def inspect_checkpoint(path: str | Path) -> dict:
         return {"model": c.name, "family": c.family, "architecture": c.architecture, "layers": c.num_layers,
                 "layer_runs": len(c.runs), "hidden": c.hidden_size, "vocab": c.vocab_size,
                 "mixers": {k: mixers.count(k) for k in sorted(set(mixers))}, "loop": c.loop, "side_dim": c.side_dim,
+                "residual_streams": c.streams, "routed_layers": sum(l.routed is not None for l in c.layers),
                 "cache_bytes_per_token": c.page_bytes // 16, "state_bytes_per_request": c.state_bytes_per_request,
                 "tensors": len(ck.store.tensors), "elements": sum(math.prod(t.shape) for t in ck.store.tensors.values()),
                 "manifest_digest": WeightManifest.from_store(ck.store).digest}

@@ -7,7 +7,10 @@ the layers of an architecture have in common is its entry in ``DESIGNS``:
   {start, stop, times} runs the layers ``start .. stop - 1`` ``times`` times with the same weights, each pass with its own
   cache and state; a pass starts with a projection of [residual ; embedding output];
 * ``Loduzen``: sequential layers (mixer, then feed-forward, each behind a norm of its own), tied output head; ``token_side`` =
-  {dim} adds, after the feed-forward, what the layer takes from its part of a second embedding of the token.
+  {dim} adds, after the feed-forward, what the layer takes from its part of a second embedding of the token;
+* ``Vimelorn``: sequential sublayers on ``streams`` residual streams (hyper-connections: every sublayer reads a weighted sum of
+  them, its result is added to all of them while they are mixed), scaled embedding; feed-forwards are dense or routed: experts
+  chosen by score plus correction, some of which return the token itself, and a gated shared expert.
 
 Mixers (another one is a spec, a reader in ``_MIXER_READERS``, an inventory entry, a ``_pack_*`` function and a method of
 ``models/layered_runner.py``):
@@ -16,7 +19,9 @@ Mixers (another one is a spec, a reader in ``_MIXER_READERS``, an inventory entr
 * ``latent_attention``: attention over cached latents with a sliding window and a gate per head;
 * ``mamba2``: short convolution, scalar-decay linear recurrence (state-space duality), gated norm in equal parts;
 * ``parallel``: two mixers that read the same norm, each scaled: sliding-window grouped-query attention with head norms,
-  rotary pairs, a softmax sink and values that are the raw keys; and gated linear attention with a decay per key channel.
+  rotary pairs, a softmax sink and values that are the raw keys; and gated linear attention with a decay per key channel;
+* ``attention``: short convolutions of q, k and v, rotary halves, unit root mean squares, a window beside kept first tokens;
+* ``attention_2``: q and k normed over their whole projections, queries warmer with their position, a bias per distance and head.
 
 ONE matrix holds all projections that read a layer's norm and ONE the output projections side by side, whatever the mixer is:
 with parallel layers the first also has the feed-forward's up rows and the second its down columns ([o | down]).  Rows and
@@ -36,6 +41,7 @@ from ..ops.eager import rope_inv_freq
 from .config import QuantSpec
 
 MAX_CONV_TAPS, MAX_DELTA_DIM, MAX_LATENT, MAX_HEAD = 16, 256, 1024, 256      # limits of the kernels
+MAX_STREAMS, MAX_ROUTER, MAX_TOP = 8, 256, 32
 
 
 @dataclass(frozen=True)
@@ -46,12 +52,14 @@ class Design:
     norm_offset: float           # a norm's factor is this plus its stored weight
     embed_norm: bool             # the embedding is normed before the first layer
     tied_head: bool              # the output head is the embedding table
-    ff: str                      # "squared_relu" (up, down) or "gelu_glu" (gate, up, down)
+    ff: str                      # "squared_relu" (up, down) or gated (gate, up, down): "gelu_glu", "silu_glu"
+    streams: bool = False        # several residual streams, a scaled embedding, routed feed-forwards
 
 
 DESIGNS = {
     "Bumodra": Design(("delta", "channel_delta", "latent_attention"), False, 1.0, True, False, "squared_relu"),
     "Loduzen": Design(("parallel", "mamba2"), True, 0.0, False, True, "gelu_glu"),
+    "Vimelorn": Design(("attention", "attention_2"), True, 0.0, False, False, "silu_glu", True),
 }
 ARCHITECTURES = tuple(DESIGNS)
 
@@ -304,13 +312,141 @@ class PairSpec(MixerSpec):
             p.validate()
 
 
-ATTENTION_SPECS, RECURRENT_SPECS = (LatentSpec, AttentionSpec), (DeltaSpec, GatedLinearSpec, SsdSpec)
+class _QkvSpec(MixerSpec):
+    """Grouped-query attention with keys and values of their own (columns [q | k | v] of the projection)."""
+
+    @property
+    def width_padded(self) -> int:
+        """Columns of a cached key or value: the widths the attention kernels are built for."""
+        return round_up(max(self.dim, self.vdim), 64)
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def offsets(self) -> tuple[int, int, int]:
+        """First columns of q, k and v from the first of them on."""
+        k = round_up(self.heads * self.dim, 8)
+        return 0, k, k + round_up(self.kv_heads * self.dim, 8)
+
+    def page_bytes(self, act_bytes: int) -> int:
+        return 16 * self.kv_heads * 2 * self.width_padded * act_bytes
+
+    def validate(self) -> None:
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) <= 0 or self.heads % self.kv_heads:
+            raise LayeredConfigError("attention heads are grouped evenly over positive key head counts and sizes")
+        if max(self.dim, self.vdim) > MAX_HEAD:
+            raise LayeredConfigError(f"attention heads of up to {MAX_HEAD} channels are served")
+
+
+@dataclass(frozen=True)
+class ConvAttentionSpec(_QkvSpec):
+    """Short convolutions of q, k and v, rotary halves, heads over their root mean square, a window beside kept first tokens."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    scale: float
+    rotary: "RotarySpec"
+    window: int = 0              # 0: every earlier token
+    keep: int = 0                # first tokens that stay visible behind the window
+    label = "conv_attention"
+
+    @property
+    def conv_width(self) -> int:
+        """Convolved columns of the projection."""
+        return round_up(self.offsets[2] + self.kv_heads * self.vdim, 8)
+
+    def state_bytes(self, act_bytes: int) -> int:
+        return round_up((self.conv - 1) * self.conv_width * act_bytes, 16)
+
+    def validate(self) -> None:
+        super().validate()
+        r = self.rotary
+        if not 1 <= self.conv <= MAX_CONV_TAPS:
+            raise LayeredConfigError(f"attention takes 1 to {MAX_CONV_TAPS} convolution taps")
+        if r.dims % 2 or not 0 <= r.dims <= self.dim or r.base <= 0:
+            raise LayeredConfigError("rotary channels come in pairs inside a head")
+        if self.window < 0 or self.keep < 0:
+            raise LayeredConfigError("an attention window and the tokens kept before it are not negative")
+
+
+@dataclass(frozen=True)
+class BiasedAttentionSpec(_QkvSpec):
+    """q and k normed over their whole projections, queries times ``1 + coef ln(floor((position + 1) / every) + 1)``, a learned
+    bias by bucket of distance and head."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    buckets: int                 # rows of the bias table
+    bias_max: int                # distance at which the last bucket's steps end
+    temp_coef: float = 0.0
+    temp_every: int = 0          # 0: no factor
+    window = 0
+    label = "biased_attention"
+
+    def bucket(self, n: int) -> int:
+        """Row of distance n: a row each for the first half, equal steps of the logarithm up to ``bias_max`` for the rest.  In
+        integers, so that no rounding moves a border."""
+        B = self.buckets
+        half = B // 2
+        if n < half:
+            return n
+        k = 0
+        while k < B - half and n ** (B - half) * half ** (k + 1) >= self.bias_max ** (k + 1) * half ** (B - half):
+            k += 1
+        return min(B - 1, half + k)
+
+    def bucket_of_distance(self) -> torch.Tensor:
+        """Rows of the distances 0 .. ``bias_max``; farther ones share the last."""
+        return torch.tensor([self.bucket(n) for n in range(self.bias_max + 1)])
+
+    def validate(self) -> None:
+        super().validate()
+        if self.buckets < 2 or self.bias_max <= self.buckets // 2:
+            raise LayeredConfigError("distance biases have two rows or more and a largest distance behind their first half")
+        if self.temp_every < 0:
+            raise LayeredConfigError("the query factor grows every positive number of positions")
+
+
+ATTENTION_SPECS = (LatentSpec, AttentionSpec, ConvAttentionSpec, BiasedAttentionSpec)
+
+
+@dataclass(frozen=True)
+class RoutedSpec:
+    """Squared-relu experts of which a token uses ``top``, ``identity`` more that return the token itself, and a gated shared
+    expert.  Scores are a softmax over all; the choice adds a correction, the weights do not and sum to one."""
+    experts: int
+    top: int
+    ff: int
+    identity: int = 0
+    shared_ff: int = 0           # 0: no shared expert
+
+    @property
+    def outputs(self) -> int:
+        """Outputs of the router."""
+        return self.experts + self.identity
+
+    def validate(self) -> None:
+        if min(self.experts, self.top, self.ff) <= 0 or min(self.identity, self.shared_ff) < 0 or self.top > self.outputs:
+            raise LayeredConfigError("experts, their widths and routes of a token are positive, with no more routes than outputs")
+        if self.outputs > MAX_ROUTER or self.top > MAX_TOP:
+            raise LayeredConfigError(f"routers of up to {MAX_ROUTER} outputs and {MAX_TOP} routes are served")
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: MixerSpec
     ff: int = 0                  # feed-forward width; 0 = none
+    routed: RoutedSpec | None = None     # instead of a dense feed-forward
+
+    @property
+    def has_ff(self) -> bool:
+        return self.ff > 0 or self.routed is not None
 
 
 @dataclass(frozen=True)
@@ -324,6 +460,8 @@ class LayeredConfig:
     dtype: str = "bfloat16"                       # activations and products: bfloat16 | float32
     architecture: str = ARCHITECTURES[0]
     side_dim: int = 0                             # width of a layer's part of the token's side embedding; 0 = none
+    streams: int = 1                              # residual streams
+    embed_scale: float = 1.0
     family: str = "layered"
     max_position: int = 1 << 20                   # positions are rotary or none: only memory limits the context
     quant: QuantSpec = field(default_factory=lambda: QuantSpec("none", 16, 0))
@@ -370,6 +508,11 @@ class LayeredConfig:
     def state_bytes_per_request(self) -> int:
         return sum(self.layers[i].mixer.state_bytes(self.act_bytes) for i, _ in self.runs)
 
+    @property
+    def state_runs(self) -> int:
+        """Mixers of the layer runs that keep state per request."""
+        return sum(p.state_bytes(self.act_bytes) > 0 for i, _ in self.runs for p in self.layers[i].mixer.parts)
+
     def run_parts(self, kind: type | tuple[type, ...]) -> int:
         """How many mixers of a kind the layer runs have (each with a cache or state of its own)."""
         return sum(isinstance(p, kind) for i, _ in self.runs for p in self.layers[i].mixer.parts)
@@ -381,8 +524,14 @@ class LayeredConfig:
             raise LayeredConfigError(f"dtype {self.dtype!r} is not bfloat16 or float32")
         for l in self.layers:
             l.mixer.validate()
-            if l.ff < 0:
+            if l.ff < 0 or l.ff and l.routed:
                 raise LayeredConfigError("feed-forward widths are positive")
+            if l.routed is not None:
+                if not self.design.streams:
+                    raise LayeredConfigError(f"{self.architecture} layers have dense feed-forwards")
+                l.routed.validate()
+        if not 1 <= self.streams <= MAX_STREAMS or self.streams > 1 and not self.design.streams:
+            raise LayeredConfigError(f"1 to {MAX_STREAMS} residual streams are served, more than one in designs that mix them")
         if self.side_dim < 0 or (self.side_dim or self.design.sequential) and self.loop is not None:
             raise LayeredConfigError("sequential layers are run once, and the side input of a layer has a positive width")
         if self.loop is not None:
@@ -392,11 +541,12 @@ class LayeredConfig:
 
     def to_config(self) -> dict:
         """The ``config.json`` object of this configuration."""
-        layers = [{**dict(zip(("type", "mixer"), _mixer_config(l.mixer))),
-                   "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None} for l in self.layers]
+        layers = [{**dict(zip(("type", "mixer"), _mixer_config(l.mixer))), "mlp": _ff_config(l)} for l in self.layers]
         out = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
                "norm": {"eps": self.rms_eps}, "layers": layers}
-        if self.design.sequential:
+        if self.design.streams:
+            out.update(streams=self.streams, embedding={"scale": self.embed_scale})
+        elif self.design.sequential:
             out["token_side"] = {"dim": self.side_dim} if self.side_dim else None
         else:
             out["loop"] = None if self.loop is None else dict(zip(("start", "stop", "times"), self.loop))
@@ -405,6 +555,15 @@ class LayeredConfig:
 
 def _mask_config(window: int) -> dict | None:
     return {"size": window} if window else None
+
+
+def _ff_config(l: LayerSpec) -> dict | None:
+    """Feed-forward object of a layer's entry in ``config.json``."""
+    if l.routed is None:
+        return {"kind": "dense", "ff": l.ff} if l.ff else None
+    r = l.routed
+    return {"kind": "moe", "expert": {"ff": r.ff}, "router": {"experts": r.experts, "identity": r.identity, "top": r.top},
+            "shared": {"ff": r.shared_ff} if r.shared_ff else None}
 
 
 def _mixer_config(m: MixerSpec) -> tuple[str, dict]:
@@ -417,6 +576,14 @@ def _mixer_config(m: MixerSpec) -> tuple[str, dict]:
     if isinstance(m, SsdSpec):
         return "mamba2", {"heads": m.heads, "vdim": m.vdim, "state": m.state, "groups": m.groups, "conv": m.conv,
                           "norm_groups": m.norm_groups}
+    if isinstance(m, ConvAttentionSpec):
+        return "attention", {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv, "scale": m.scale,
+                             "rot": {"dims": m.rotary.dims, "base": m.rotary.base},
+                             "mask": {"size": m.window, "keep_first": m.keep} if m.window else None}
+    if isinstance(m, BiasedAttentionSpec):
+        return "attention_2", {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
+                               "bias_max": m.bias_max,
+                               "q_temp": {"coef": m.temp_coef, "every": m.temp_every} if m.temp_every else None}
     a, g, sc = m.left, m.right, m.left.rotary.scaling
     rot = {"dims": a.rotary.dims, "base": a.rotary.base,
            "scaling": dict(zip(("factor", "original", "fast", "slow"), sc[1:5])) if sc else None}
@@ -474,8 +641,37 @@ def _read_parallel(m: dict, p: str, rank) -> PairSpec:
     return PairSpec(left, right, float(m["left_scale"]), float(m["right_scale"]))
 
 
+def _read_conv_attention(m: dict, p: str, rank) -> ConvAttentionSpec:
+    mask = m.get("mask") or {}
+    return ConvAttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m.get("conv") or 1),
+                             float(m["scale"]), _read_rotary(m.get("rot")), _window(m), int(mask.get("keep_first") or 0))
+
+
+def _read_biased_attention(m: dict, p: str, rank) -> BiasedAttentionSpec:
+    temp = m.get("q_temp") or {}
+    if temp and int(temp["every"]) < 1:
+        raise LayeredConfigError("the query factor grows every positive number of positions")
+    return BiasedAttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), rank(f"{p}.rel"),
+                               int(m["bias_max"]), float(temp.get("coef", 0.0)), int(temp.get("every", 0)))
+
+
+def _read_ff(mlp: dict | None, i: int, d: Design) -> dict:
+    """Feed-forward fields of a ``LayerSpec``."""
+    if not mlp:
+        return {}
+    kind = mlp.get("kind")
+    if kind == "dense":
+        return {"ff": int(mlp["ff"])}
+    if kind != "moe" or not d.streams:
+        raise LayeredConfigError(f"layer {i}: unknown feed-forward {kind!r}")
+    r, shared = mlp["router"], mlp.get("shared")
+    return {"routed": RoutedSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), int(r.get("identity") or 0),
+                                 int(shared["ff"]) if shared else 0)}
+
+
 _MIXER_READERS = {"delta": _read_delta, "channel_delta": lambda m, p, rank: _read_delta(m, p, rank, True),
-                  "latent_attention": _read_latent, "mamba2": _read_mamba2, "parallel": _read_parallel}
+                  "latent_attention": _read_latent, "mamba2": _read_mamba2, "parallel": _read_parallel,
+                  "attention": _read_conv_attention, "attention_2": _read_biased_attention}
 
 
 def parse_layered_config(raw: dict, shapes: dict[str, tuple[int, ...]] | None = None, name: str = "") -> LayeredConfig:
@@ -496,14 +692,14 @@ def parse_layered_config(raw: dict, shapes: dict[str, tuple[int, ...]] | None = 
         if l["type"] not in DESIGNS[arch].mixers:
             raise LayeredConfigError(f"layer {i}: unknown mixer {l['type']!r}")
         mixer = _MIXER_READERS[l["type"]](l["mixer"], f"l{i}.mix", rank)
-        mlp = l.get("mlp")
-        if mlp and mlp.get("kind") != "dense":
-            raise LayeredConfigError(f"layer {i}: unknown feed-forward {mlp.get('kind')!r}")
-        layers.append(LayerSpec(mixer, int(mlp["ff"]) if mlp else 0))
+        layers.append(LayerSpec(mixer, **_read_ff(l.get("mlp"), i, DESIGNS[arch])))
     loop, side = raw.get("loop"), raw.get("token_side")
+    streams = {}
+    if DESIGNS[arch].streams:
+        streams = dict(streams=int(raw.get("streams") or 1), embed_scale=float((raw.get("embedding") or {}).get("scale", 1.0)))
     cfg = LayeredConfig(name or arch, int(raw["vocab"]), int(raw["width"]), tuple(layers), float(raw["norm"]["eps"]),
                         (int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None, architecture=arch,
-                        side_dim=int(side["dim"]) if side else 0)
+                        side_dim=int(side["dim"]) if side else 0, **streams)
     cfg.validate()
     return cfg
 
@@ -533,6 +729,13 @@ def _mixer_shapes(m: MixerSpec, p: str, W: int) -> dict[str, tuple[int, ...]]:
     elif isinstance(m, AttentionSpec):
         out.update({f"{p}.q": (m.heads * m.dim, W), f"{p}.k": (m.kv_heads * m.dim, W), f"{p}.q.norm": (m.dim,),
                     f"{p}.k.norm": (m.dim,)})
+    elif isinstance(m, _QkvSpec):
+        sizes = {"q": m.heads * m.dim, "k": m.kv_heads * m.dim, "v": m.kv_heads * m.vdim}
+        out.update({f"{p}.{t}": (n, W) for t, n in sizes.items()})
+        if isinstance(m, ConvAttentionSpec):
+            out.update({f"{p}.{t}.conv": (n, m.conv) for t, n in sizes.items()})
+        else:
+            out.update({f"{p}.q.norm": (sizes["q"],), f"{p}.k.norm": (sizes["k"],), f"{p}.rel": (m.buckets, m.heads)})
     elif isinstance(m, GatedLinearSpec):
         out.update({f"{p}.{t}": (m.heads * c, W) for t, c in (("q", m.dim), ("k", m.dim), ("v", m.vdim), ("g", m.vdim))})
         out.update({f"{p}.norm": (m.vdim,), f"{p}.a1": (m.decay_rank, W), f"{p}.a2": (m.heads * m.dim, m.decay_rank),
@@ -560,10 +763,21 @@ def tensor_shapes(cfg: LayeredConfig) -> dict[str, tuple[int, ...]]:
     for i, l in enumerate(cfg.layers):
         out[f"l{i}.norm1"] = (W,)
         out.update(_mixer_shapes(l.mixer, f"l{i}.mix", W))
+        if d.sequential and l.has_ff:
+            out[f"l{i}.norm2"] = (W,)
+        if d.streams:
+            for q in (1, 2) if l.has_ff else (1,):
+                out.update({f"l{i}.hc{q}.in": (cfg.streams,), f"l{i}.hc{q}.out": (cfg.streams,),
+                            f"l{i}.hc{q}.mix": (cfg.streams, cfg.streams)})
+        if l.routed is not None:
+            r, p = l.routed, f"l{i}.mlp"
+            for e in range(r.experts):
+                out.update({f"{p}.e{e}.up": (r.ff, W), f"{p}.e{e}.down": (W, r.ff)})
+            out.update({f"{p}.router": (r.outputs, W), f"{p}.correction": (r.outputs,)})
+            if r.shared_ff:
+                out.update({f"{p}.shared.up": (r.shared_ff, W), f"{p}.shared.down": (W, r.shared_ff), f"{p}.shared.sg": (1, W)})
         if l.ff:
-            if d.sequential:
-                out[f"l{i}.norm2"] = (W,)
-            if d.ff == "gelu_glu":
+            if d.ff.endswith("_glu"):
                 out[f"l{i}.mlp.gate"] = (l.ff, W)
             out[f"l{i}.mlp.up"] = (l.ff, W)
             out[f"l{i}.mlp.down"] = (W, l.ff)
@@ -573,14 +787,16 @@ def tensor_shapes(cfg: LayeredConfig) -> dict[str, tuple[int, ...]]:
 
 
 def check_inventory(cfg: LayeredConfig, shapes: dict[str, tuple[int, ...]]) -> None:
-    """The checkpoint's tensors are exactly the configuration's (a second norm without a feed-forward behind it is ignored)."""
+    """The checkpoint's tensors are exactly the configuration's (what a missing feed-forward would need is ignored)."""
     want = tensor_shapes(cfg)
     for n, s in want.items():
         if n not in shapes:
             raise LayeredConfigError(f"missing tensor {n}")
         if tuple(shapes[n]) != s:
             raise LayeredConfigError(f"{n}: shape {tuple(shapes[n])}, expected {s}")
-    extra = sorted(set(shapes) - set(want) - {f"l{i}.norm2" for i, l in enumerate(cfg.layers) if cfg.design.sequential and not l.ff})
+    idle = {f"l{i}.{t}" for i, l in enumerate(cfg.layers) if cfg.design.sequential and not l.has_ff
+            for t in ("norm2", "hc2.in", "hc2.out", "hc2.mix")}
+    extra = sorted(set(shapes) - set(want) - idle)
     if extra:
         raise LayeredConfigError(f"checkpoint has {len(extra)} tensors this configuration does not own, e.g. {extra[:3]}")
 
@@ -596,6 +812,14 @@ def random_tensors(cfg: LayeredConfig, seed: int = 0, device="cpu") -> dict[str,
         if last in stream:
             of_stream = n in ("embed.norm", "final.norm") or n.count(".") == 1
             t = (1.0 - cfg.design.norm_offset if of_stream else 1.0) + 0.1 * z
+        elif ".hc" in n:                             # streams that stay alike, each sublayer's input and result of about their size
+            t = 0.1 * z + {"in": 1.0 / cfg.streams, "out": 1.0}.get(last, torch.eye(cfg.streams, device=device) if last == "mix" else 0.0)
+        elif last == "rel":
+            t = 0.5 * z
+        elif last == "correction":
+            t = 0.02 * z
+        elif n == "embed" and cfg.design.streams:
+            t = z / cfg.embed_scale
         elif last == "A_log":
             t = 0.5 * z - 2.0
         elif last in ("dt_bias", "b") and len(s) == 1:
@@ -729,6 +953,44 @@ class PairWeights:
 
 
 @dataclass
+class ConvAttentionWeights:
+    spec: ConvAttentionSpec
+    conv_w: torch.Tensor             # fp32 [taps, conv_width]
+    freq: torch.Tensor               # fp32 [2, pairs] radians per position, and what rounding took from them
+    q_off: int
+
+
+@dataclass
+class BiasedAttentionWeights:
+    spec: BiasedAttentionSpec
+    q_norm: torch.Tensor             # fp32 [H d]
+    k_norm: torch.Tensor             # fp32 [G d]
+    bias: torch.Tensor               # fp32 [bias_max + 1, H] by distance
+    q_off: int
+
+
+@dataclass
+class StreamWeights:
+    """How a sublayer reads and writes the residual streams (fp32)."""
+    read: torch.Tensor               # [streams]
+    write: torch.Tensor              # [streams]
+    mix: torch.Tensor                # [streams, streams] from, to
+
+
+@dataclass
+class RoutedWeights:
+    """ONE matrix reads the feed-forward's norm for everybody: [router | shared expert's gate] in fp32, then the shared expert's
+    up rows behind the squared relu."""
+    spec: RoutedSpec
+    head: wq_pack.PackedWeight
+    split: int                       # fp32 columns of its output
+    correction: torch.Tensor
+    up: wq_pack.PackedWeight         # experts stacked
+    down: wq_pack.PackedWeight
+    shared_down: wq_pack.PackedWeight | None
+
+
+@dataclass
 class SideWeights:
     """A layer's input from the token's side embedding."""
     gate: torch.Tensor               # bf16 [dim, W rounded up]
@@ -750,6 +1012,8 @@ class LayerWeights:
     gate_up: wq_pack.PackedWeight | None = None  # rows in the order of the fused gated activation
     down: wq_pack.PackedWeight | None = None
     side: SideWeights | None = None
+    streams: tuple[StreamWeights, ...] = ()      # of the mixer and of the feed-forward
+    routed: RoutedWeights | None = None
 
     def matrices(self) -> list[wq_pack.PackedWeight]:
         """Every packed matrix of the layer."""
@@ -760,6 +1024,8 @@ class LayerWeights:
             elif getattr(part, "low", None) is not None:
                 out.append(part.low)
         out += [m for m in (self.gate_up, self.down) if m is not None]
+        if self.routed is not None:
+            out += [m for m in (self.routed.head, self.routed.up, self.routed.down, self.routed.shared_down) if m is not None]
         return out + ([self.side.proj] if self.side is not None else [])
 
 
@@ -859,6 +1125,32 @@ def _pack_attention(m: AttentionSpec, p: str, rows: _Rows, get, out_scale: float
     return AttentionWeights(m, q_norm, _f32(get, f"{p}.k.norm"), freq.to(q_norm.device).contiguous(), mult, q_off, k_off, out_scale)
 
 
+def _add_qkv(m: _QkvSpec, p: str, rows: _Rows, get) -> int:
+    q_off = rows.add(get(f"{p}.q"))
+    offs = q_off, rows.add(get(f"{p}.k")), rows.add(get(f"{p}.v"))
+    assert tuple(o - q_off for o in offs) == m.offsets
+    return q_off
+
+
+def _pack_conv_attention(m: ConvAttentionSpec, p: str, rows: _Rows, get) -> ConvAttentionWeights:
+    q_off = _add_qkv(m, p, rows, get)
+    dev = get(f"{p}.q").device
+    conv_w = torch.zeros(m.conv, m.conv_width, device=dev)
+    for t, off in zip("qkv", m.offsets):
+        w = get(f"{p}.{t}.conv").float()
+        conv_w[:, off:off + w.shape[0]] = w.t()
+    exact = rope_inv_freq(m.rotary.dims, m.rotary.base, dtype=torch.float64)
+    freq = torch.stack([exact.float(), (exact - exact.float().double()).float()])
+    return ConvAttentionWeights(m, conv_w, freq.to(dev).contiguous(), q_off)
+
+
+def _pack_biased_attention(m: BiasedAttentionSpec, p: str, rows: _Rows, get) -> BiasedAttentionWeights:
+    q_off = _add_qkv(m, p, rows, get)
+    rel = _f32(get, f"{p}.rel")
+    return BiasedAttentionWeights(m, _f32(get, f"{p}.q.norm"), _f32(get, f"{p}.k.norm"),
+                                  rel[m.bucket_of_distance().to(rel.device)].contiguous(), q_off)
+
+
 def _pack_gated_linear(m: GatedLinearSpec, p: str, rows: _Rows, get, out_scale: float = 1.0) -> GatedLinearWeights:
     q_off, k_off, v_off, g_off = (rows.add(get(f"{p}.{t}")) for t in "qkvg")
     inner = round_up(m.decay_rank, 64)
@@ -883,7 +1175,8 @@ def _pack_pair(m: PairSpec, p: str, rows: _Rows, get) -> PairWeights:
 
 
 _PACKERS = {DeltaSpec: _pack_delta, LatentSpec: _pack_latent, AttentionSpec: _pack_attention, GatedLinearSpec: _pack_gated_linear,
-            SsdSpec: _pack_ssd, PairSpec: _pack_pair}
+            SsdSpec: _pack_ssd, PairSpec: _pack_pair, ConvAttentionSpec: _pack_conv_attention,
+            BiasedAttentionSpec: _pack_biased_attention}
 
 
 def _pack_output(m: MixerSpec, p: str, get, ff: int, W: int) -> tuple[torch.Tensor, int]:
@@ -904,6 +1197,30 @@ def _pack_glu(gate: torch.Tensor, up: torch.Tensor) -> wq_pack.PackedWeight:
     return wq_pack.swiglu_interleave(_matrix(both.flatten(0, 1)))
 
 
+def _stack(mats) -> wq_pack.PackedWeight:
+    """Equal matrices along a leading axis, each as ``_matrix`` packs it."""
+    packed = [_matrix(t.to(torch.bfloat16)) for t in mats]
+    return replace(packed[0], codes=torch.stack([w.codes for w in packed]))
+
+
+def _pack_routed(r: RoutedSpec, p: str, W: int, get) -> RoutedWeights:
+    rows = _Rows(W)
+    rows.add(get(f"{p}.router"))
+    if r.shared_ff:
+        rows.add(get(f"{p}.shared.sg"), align=1)
+    rows.end()
+    split = rows.n
+    if r.shared_ff:
+        rows.add(get(f"{p}.shared.up"))
+    return RoutedWeights(r, _matrix(rows.end(1)), split, _f32(get, f"{p}.correction"),
+                         _stack(get(f"{p}.e{e}.up") for e in range(r.experts)), _stack(get(f"{p}.e{e}.down") for e in range(r.experts)),
+                         _matrix(get(f"{p}.shared.down").to(torch.bfloat16)) if r.shared_ff else None)
+
+
+def _pack_streams(p: str, get) -> StreamWeights:
+    return StreamWeights(*(_f32(get, f"{p}.{t}") for t in ("in", "out", "mix")))
+
+
 def pack_layer(cfg: LayeredConfig, i: int, get) -> LayerWeights:
     """``get(name)`` -> tensor on the target device."""
     l, p, W, d = cfg.layers[i], f"l{i}", cfg.hidden_size, cfg.design
@@ -911,14 +1228,19 @@ def pack_layer(cfg: LayeredConfig, i: int, get) -> LayerWeights:
     mixer = _PACKERS[type(l.mixer)](l.mixer, f"{p}.mix", rows, get)
     proj = rows.end()
     split = proj.shape[0]
-    joint = l.ff if not d.sequential else 0
+    joint = 0 if d.sequential else l.ff
     out, out_off = _pack_output(l.mixer, f"{p}.mix", get, joint, W)
     if joint:
         proj = torch.cat([proj, get(f"{p}.mlp.up").to(torch.bfloat16)])
         out[:, out_off:out_off + l.ff] = get(f"{p}.mlp.down")
     lw = LayerWeights(d.norm_offset + _f32(get, f"{p}.norm1"), _matrix(proj), split, joint, mixer, wq_pack.pack_bf16(out), out_off)
-    if d.sequential and l.ff:
+    if d.streams:
+        lw.streams = tuple(_pack_streams(f"{p}.hc{q}", get) for q in ((1, 2) if l.has_ff else (1,)))
+    if d.sequential and l.has_ff:
         lw.norm2 = d.norm_offset + _f32(get, f"{p}.norm2")
+    if l.routed is not None:
+        lw.routed = _pack_routed(l.routed, f"{p}.mlp", W, get)
+    if d.sequential and l.ff:
         lw.gate_up = _pack_glu(get(f"{p}.mlp.gate"), get(f"{p}.mlp.up"))
         lw.down = _matrix(get(f"{p}.mlp.down").to(torch.bfloat16))
     if cfg.side_dim:
@@ -988,7 +1310,26 @@ def sequential_8b_config() -> LayeredConfig:
     return LayeredConfig("layered-seq-8b", 151936, 4096, (ssd, pair, pair, pair) * 8, 1e-6, architecture="Loduzen", side_dim=64)
 
 
-NAMED = {"layered-tiny": tiny_layered_config, "layered-8b": layered_8b_config, "layered-seq-tiny": tiny_sequential_config,
+def tiny_streams_config() -> LayeredConfig:
+    """A few small layers of both attentions and both feed-forwards on three residual streams (tests and demonstrations)."""
+    near = ConvAttentionSpec(6, 2, 40, 24, 4, 0.2, RotarySpec(24, 10000.0), 37, 5)
+    far = BiasedAttentionSpec(4, 4, 32, 48, 0.2, 12, 50, 0.3, 20)
+    routed = RoutedSpec(6, 3, 80, 2, 96)
+    return LayeredConfig("layered-streams-tiny", 384, 192, (LayerSpec(near, 160), LayerSpec(far, routed=routed), LayerSpec(near, routed=routed),
+                                                            LayerSpec(far)), 1e-5, architecture="Vimelorn", streams=3, embed_scale=13.0)
+
+
+def streams_moe_config() -> LayeredConfig:
+    """Layers of the size of a mixture-of-experts model with 4 of 64 experts: three windowed attention layers and one of every
+    earlier token in turn, every second feed-forward routed, two residual streams."""
+    near = ConvAttentionSpec(32, 8, 128, 128, 4, 1.0, RotarySpec(128, 1e6), 1024, 8)
+    far = BiasedAttentionSpec(32, 8, 128, 128, 128 ** -0.5, 32, 512, 0.1, 4096)
+    routed = RoutedSpec(64, 4, 1024, 8, 1024)
+    group = (LayerSpec(near, 8192), LayerSpec(near, routed=routed), LayerSpec(near, 8192), LayerSpec(far, routed=routed))
+    return LayeredConfig("layered-streams-moe", 151936, 4096, group * 8, 1e-6, architecture="Vimelorn", streams=2, embed_scale=64.0)
+
+
+NAMED = {"layered-streams-tiny": tiny_streams_config, "layered-streams-moe": streams_moe_config, "layered-tiny": tiny_layered_config, "layered-8b": layered_8b_config, "layered-seq-tiny": tiny_sequential_config,
          "layered-seq-8b": sequential_8b_config}
 
 

@@ -1,4 +1,4 @@
-"""Plain model of the layered decoders (``Bumodra`` and ``Loduzen`` checkpoints): the oracle of the native runner and the
+"""Plain model of the layered decoders (``Bumodra``, ``Loduzen`` and ``Vimelorn`` checkpoints): the oracle of the native runner and the
 model of the eager execution mode.
 
 Everything is written from the equations, token by token where the mechanism is a recurrence, one function per
@@ -132,6 +132,72 @@ def sink_attention(q, k, v, first: int, window: int | None, scale: float) -> tor
     s = s.masked_fill(~seen, float("-inf"))
     s = torch.cat([s, torch.zeros(H, n, 1, dtype=s.dtype)], -1)
     return torch.einsum("hnm,mhe->nhe", torch.softmax(s, -1)[..., :m], v[:, rep])
+
+
+def plain_short_conv(x: torch.Tensor, w: torch.Tensor, past: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    """``short_conv`` without the activation."""
+    taps, n = w.shape[1], x.shape[0]
+    ext = torch.cat([past, x])
+    out = sum(w[:, j] * ext[j:j + n] for j in range(taps))
+    return out, ext[ext.shape[0] - (taps - 1):].clone()
+
+
+def rotate_halves(x: torch.Tensor, first: int, dims: int, base: float) -> torch.Tensor:
+    """Rotary positions ``first ..`` on ``x`` [n, H, d]: channel i of the first ``dims`` turns with channel ``i + dims / 2``."""
+    n, half = x.shape[0], dims // 2
+    f = torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(half)], dtype=torch.float64)
+    a = torch.arange(first, first + n, dtype=torch.float64).view(n, 1, 1) * f
+    c, s = torch.cos(a).to(x.dtype), torch.sin(a).to(x.dtype)
+    u, v = x[..., :half], x[..., half:dims]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], -1)
+
+
+def kept_window(first: int, n: int, m: int, size: int | None, keep: int) -> torch.Tensor:
+    """[n, m] which of m keys the queries at positions ``first ..`` see: the last ``size`` and the first ``keep``."""
+    i, j = torch.arange(first, first + n).unsqueeze(1), torch.arange(m).unsqueeze(0)
+    near = (i - j) < size if size is not None else torch.ones(n, m, dtype=torch.bool)
+    return (j <= i) & (near | (j < keep))
+
+
+def distance_bucket(n: int, rows: int, most: int) -> int:
+    """Row of a distance table with ``rows`` rows: the first half one distance each, the others in equal steps of the distance's
+    logarithm up to ``most``.  Decided in integers: the largest k with ``(n / half) ** (rows - half) >= (most / half) ** k``."""
+    half = rows // 2
+    if n < half:
+        return n
+    steps = rows - half
+    passed = max(k for k in range(steps + 1) if n ** steps * half ** k >= most ** k * half ** steps)
+    return min(rows - 1, half + passed)
+
+
+def masked_attention(q, k, v, seen, scale: float, bias=None) -> torch.Tensor:
+    """Softmax attention over the keys ``seen`` [n, m]; query head h uses key head ``h // (H / G)``; ``bias`` [H, n, m] is added
+    to the scaled scores."""
+    rep = torch.arange(q.shape[1]) // (q.shape[1] // k.shape[1])
+    s = torch.einsum("nhd,mhd->hnm", q, k[:, rep]) * scale
+    if bias is not None:
+        s = s + bias
+    s = s.masked_fill(~seen, float("-inf"))
+    return torch.einsum("hnm,mhe->nhe", torch.softmax(s, -1), v[:, rep])
+
+
+def route(z: torch.Tensor, correction: torch.Tensor, top: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """Chosen experts [n, top] and their weights from router logits ``z`` [n, E]: softmax scores, the choice by score plus
+    correction, the weights the chosen scores over their sum."""
+    s = torch.softmax(z, -1)
+    chosen = torch.argsort(-(s + correction), dim=-1, stable=True)[:, :top]
+    picked = s.gather(1, chosen)
+    return chosen, picked / (picked.sum(-1, keepdim=True) + 1e-20)
+
+
+def stream_read(xs: torch.Tensor, w_in: torch.Tensor) -> torch.Tensor:
+    """Input of a sublayer from the residual streams ``xs`` [s, n, W]."""
+    return torch.einsum("s,snw->nw", w_in, xs)
+
+
+def stream_write(xs: torch.Tensor, mix: torch.Tensor, out: torch.Tensor, y: torch.Tensor) -> torch.Tensor:
+    """Streams after a sublayer with result ``y``: old streams mixed ([from, to]) and ``y`` added to each by its factor."""
+    return torch.einsum("st,snw->tnw", mix, xs) + out.view(-1, 1, 1) * y
 
 
 def linear_step(S: torch.Tensor, q, k, v, decay) -> tuple[torch.Tensor, torch.Tensor]:
@@ -269,6 +335,70 @@ def token_side(w, p: str, x, e, eps: float) -> torch.Tensor:
 SEQUENTIAL_MIXERS = {"parallel": parallel_mixer, "mamba2": ssd_mixer}
 
 
+def conv_attention(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    """Attention behind short convolutions of q, k and v: rotary halves, then unit root mean squares; a window and kept first
+    tokens."""
+    H, G, d, e = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    n = h.shape[0]
+    if not st:
+        for t, c in (("q", H * d), ("k", G * d), ("v", G * e)):
+            st[f"past_{t}"] = torch.zeros(m["conv"] - 1, c, dtype=h.dtype)
+        st["k"], st["v"] = torch.zeros(0, G, d, dtype=h.dtype), torch.zeros(0, G, e, dtype=h.dtype)
+    first, new = st["k"].shape[0], {}
+    for t in "qkv":
+        new[t], st[f"past_{t}"] = plain_short_conv(h @ w[f"{p}.{t}"].T, w[f"{p}.{t}.conv"], st[f"past_{t}"])
+    rot = m["rot"]
+    q, k = (rms(rotate_halves(new[t].view(n, -1, d), first, rot["dims"], rot["base"]), eps) for t in "qk")
+    st["k"], st["v"] = torch.cat([st["k"], k]), torch.cat([st["v"], new["v"].view(n, G, e)])
+    mask = m.get("mask") or {}
+    seen = kept_window(first, n, first + n, mask.get("size"), mask.get("keep_first", 0))
+    return masked_attention(q, st["k"], st["v"], seen, m["scale"]).reshape(n, H * e) @ w[f"{p}.o"].T
+
+
+def biased_attention(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    """Attention without rotation: q and k normed over their whole projection, queries warmer with their position, a learned
+    bias per bucket of distance and head."""
+    H, G, d, e = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    n = h.shape[0]
+    if not st:
+        st["k"], st["v"] = torch.zeros(0, G, d, dtype=h.dtype), torch.zeros(0, G, e, dtype=h.dtype)
+    first = st["k"].shape[0]
+    q, k = (rms(h @ w[f"{p}.{t}"].T, eps) * w[f"{p}.{t}.norm"] for t in "qk")
+    if m.get("q_temp"):
+        warm = [1.0 + m["q_temp"]["coef"] * math.log((pos + 1) // m["q_temp"]["every"] + 1) for pos in range(first, first + n)]
+        q = q * torch.tensor(warm, dtype=h.dtype).unsqueeze(1)
+    st["k"] = torch.cat([st["k"], k.view(n, G, d)])
+    st["v"] = torch.cat([st["v"], (h @ w[f"{p}.v"].T).view(n, G, e)])
+    rel, total = w[f"{p}.rel"], first + n
+    by_distance = rel[torch.tensor([distance_bucket(i, rel.shape[0], m["bias_max"]) for i in range(total)])]
+    seen = kept_window(first, n, total, None, 0)
+    gap = (torch.arange(first, total).unsqueeze(1) - torch.arange(total)).clamp(min=0)
+    return masked_attention(q.view(n, H, d), st["k"], st["v"], seen, m["scale"], by_distance[gap].permute(2, 0, 1)).reshape(n, H * e) \
+        @ w[f"{p}.o"].T
+
+
+STREAM_MIXERS = {"attention": conv_attention, "attention_2": biased_attention}
+
+
+def routed_feed_forward(w, p: str, mlp: dict, h) -> torch.Tensor:
+    """Squared-relu experts with identity experts behind them, and a gated shared expert."""
+    r = mlp["router"]
+    chosen, weight = route(h @ w[f"{p}.router"].T, w[f"{p}.correction"], r["top"])
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, g in zip(chosen[t].tolist(), weight[t]):
+            y = h[t] if e >= r["experts"] else squared_relu(h[t] @ w[f"{p}.e{e}.up"].T) @ w[f"{p}.e{e}.down"].T
+            out[t] += g * y
+    if mlp.get("shared"):
+        gate = 1.0 / (1.0 + torch.exp(-(h @ w[f"{p}.shared.sg"].T)))
+        out = out + gate * (squared_relu(h @ w[f"{p}.shared.up"].T) @ w[f"{p}.shared.down"].T)
+    return out
+
+
+def silu_feed_forward(w, p: str, h) -> torch.Tensor:
+    return (silu(h @ w[f"{p}.gate"].T) * (h @ w[f"{p}.up"].T)) @ w[f"{p}.down"].T
+
+
 def layer_schedule(cfg: dict) -> list[tuple[int, bool]]:
     """The layer runs in order: (layer index, whether the pass's entry projection comes right before it)."""
     loop = cfg.get("loop")
@@ -298,6 +428,8 @@ class Oracle:
         ids = torch.as_tensor(list(tokens), dtype=torch.long)
         if cfg["architecture"] == "Loduzen":
             return self._sequential(ids, state, eps, last_only, trace)
+        if cfg["architecture"] == "Vimelorn":
+            return self._streams(ids, state, eps, last_only, trace)
         x0 = rms_around_zero(w["embed"][ids], w["embed.norm"], eps)
         x = x0
         for (i, enters), st in zip(self.schedule, state.runs):
@@ -343,6 +475,29 @@ class Oracle:
         if last_only:
             x = x[-1:]
         return (rms(x, eps) * w["final.norm"]) @ w["embed"].T, state
+
+
+    def _streams(self, ids, state, eps: float, last_only: bool, trace):
+        """Pre-norm sublayers that read and write several residual streams; a scaled embedding, untied head."""
+        w, cfg = self.w, self.cfg
+        xs = (w["embed"][ids] * cfg["embedding"]["scale"]).repeat(cfg["streams"], 1, 1)
+        for i, (layer, st) in enumerate(zip(cfg["layers"], state.runs)):
+            p, mlp = f"l{i}", layer.get("mlp")
+            subs = [(1, lambda h: STREAM_MIXERS[layer["type"]](w, f"{p}.mix", layer["mixer"], h, st, eps))]
+            if mlp:
+                subs.append((2, lambda h: silu_feed_forward(w, f"{p}.mlp", h) if mlp["kind"] == "dense"
+                             else routed_feed_forward(w, f"{p}.mlp", mlp, h)))
+            for q, sub in subs:
+                u = stream_read(xs, w[f"{p}.hc{q}.in"])
+                y = sub(rms(u, eps) * w[f"{p}.norm{q}"])
+                xs = stream_write(xs, w[f"{p}.hc{q}.mix"], w[f"{p}.hc{q}.out"], y)
+            if trace is not None:
+                trace.append(xs.sum(0))
+        state.length += len(ids)
+        x = xs.sum(0)
+        if last_only:
+            x = x[-1:]
+        return (rms(x, eps) * w["final.norm"]) @ w["head"].T, state
 
 
 class OracleState:

@@ -16,6 +16,15 @@ and a sequential layer, whose h comes from the step before it,
     norm2(x) -> h;  act = gelu(h W_gate) (h W_up), one product;  x += act W_down
     side = gelu(x W_side) e, one kernel;  y = side W_proj;  x += norm(y) and h = norm1 of the next layer, one kernel
 
+and of a layer on several residual streams x_s, whose h is the norm of their weighted sum,
+
+    mixer inputs = h W;  mixer -> operand;  y = operand W_o
+    x_t <- sum_s mix[s, t] x_s + out[t] y and h = norm2 of the next weighted sum, one kernel
+    dense:   act = silu(h W_gate) (h W_up), one product;  y = act W_down
+    routed:  [router, gate | relu^2(shared up)] = h W, one product;  routes, rows to their experts
+             relu^2(rows W_up), rows W_down, one product each over all experts;  y = shared W_down
+    the same kernel as above puts a routed y together from the places of the token's routes
+
 ``cfg.dtype`` "float32" runs the same steps with fp32 activations and fp32 products.
 """
 from __future__ import annotations
@@ -23,25 +32,26 @@ from __future__ import annotations
 import torch
 
 from ..ops import kernels as K
-from .layered import (AttentionWeights, DeltaWeights, GatedLinearWeights, LatentWeights, LayeredConfig, LayeredWeights, PairWeights,
-                      SsdWeights, round_up)
+from .layered import (AttentionWeights, BiasedAttentionWeights, ConvAttentionWeights, DeltaWeights, GatedLinearWeights, LatentWeights,
+                      LayeredConfig, LayeredWeights, PairWeights, RoutedWeights, SsdWeights, round_up)
 from .step_runner import StepRunner
 
 
 class _StateRun:
-    """Per-request state of one run of a recurrent layer: recurrence state (fp32) and, with a convolution, its last inputs
-    (activation type)."""
+    """Per-request state of one run of a layer: recurrence state (fp32; none with ``heads`` 0) and, with a convolution, its last
+    inputs (activation type)."""
 
     def __init__(self, rows: int, heads: int, vdim: int, stride: int, device, taps: int = 0, conv_width: int = 0,
                  act: torch.dtype = torch.bfloat16) -> None:
         # a row is a multiple of 16 bytes (whole-row copies); the history's layout inside it is [taps - 1, channels]
         self.conv = torch.zeros(rows, max(1, taps - 1), conv_width, dtype=act, device=device) if taps else None
-        self.state = torch.zeros(rows, heads, vdim, stride, dtype=torch.float32, device=device)
+        self.state = torch.zeros(rows, heads, vdim, stride, dtype=torch.float32, device=device) if heads else None
 
     def copy(self, src, dst) -> None:
         if self.conv is not None:
             K.copy_rows(self.conv, src, dst)
-        K.copy_rows(self.state, src, dst)
+        if self.state is not None:
+            K.copy_rows(self.state, src, dst)
 
 
 def _parts(m) -> tuple:
@@ -70,12 +80,13 @@ class LayeredRunner(StepRunner):
             # zero-filled: padding columns are multiplied by zero weights, and must be finite for that
             return torch.zeros(T, cols, dtype=dtype, device=dev)
 
-        self.x = buf(W, torch.float32)         # residual stream
+        self.x = buf(cfg.streams * W, torch.float32)      # residual stream, or streams
         self.x0 = buf(W, torch.float32) if cfg.loop is not None else None
         self.h = buf(round_up(W, 64))
         self.entry = buf(round_up(2 * W, 64)) if cfg.loop is not None else None
         self.side = buf(round_up(cfg.side_dim, 64)) if cfg.side_dim else None
         self.side_y = buf(round_up(W, 8)) if cfg.side_dim else None
+        self.y = buf(round_up(W, 8))[:, :W] if cfg.design.streams else None       # a sublayer's result
         self.kv = []                           # paged caches (copied page by page on copy-on-write)
         self.states = []                       # recurrent states (copied row by row)
         # per layer run: the cache or state of every mixer it consists of
@@ -96,7 +107,7 @@ class LayeredRunner(StepRunner):
                     self._need("q", m.uq.n)
                     self._need("ql", s.heads * s.rank_padded)
                     self._need("ol", s.heads * s.rank_padded)
-                elif isinstance(m, AttentionWeights):
+                elif isinstance(m, (AttentionWeights, ConvAttentionWeights, BiasedAttentionWeights)):
                     self._need("q", s.heads * s.width_padded)
                 else:
                     if isinstance(m, DeltaWeights):
@@ -107,6 +118,7 @@ class LayeredRunner(StepRunner):
                         recurrent.append((s.heads, s.heads, s.dim, s.vdim, True))
                     if getattr(m, "low", None) is not None and (isinstance(m, DeltaWeights) or act == torch.float32):
                         self._need("low", m.low.n)
+        self._routing()
         self._scratch = {n: torch.zeros(T * c, dtype=act, device=dev) for n, c in self._scratch.items()}
         self.recurrence = K.RecurrenceScratch(T, recurrent, act, dev) if recurrent else None
         self.trace: list | None = None         # a list here receives a copy of the residual after every layer run
@@ -117,12 +129,31 @@ class LayeredRunner(StepRunner):
         if isinstance(m, LatentWeights):
             self.kv.append(torch.zeros(self.num_pages, 16, s.rank_padded, dtype=self.act, device=dev))
             return self.kv[-1]
-        if isinstance(m, AttentionWeights):
+        if isinstance(m, (AttentionWeights, ConvAttentionWeights, BiasedAttentionWeights)):
             self.kv.append(torch.zeros(self.num_pages, s.kv_heads, 2, 16, s.width_padded, dtype=self.act, device=dev))
-            return self.kv[-1]
+            if not isinstance(m, ConvAttentionWeights):
+                return self.kv[-1]
+            if s.conv == 1:
+                return self.kv[-1], None
+            self.states.append(_StateRun(rows, 0, 0, 0, dev, taps=s.conv, conv_width=s.conv_width, act=self.act))
+            return self.kv[-1], self.states[-1].conv
         conv = {} if isinstance(m, GatedLinearWeights) else dict(taps=s.conv, conv_width=s.conv_width, act=self.act)
         self.states.append(_StateRun(rows, s.heads, s.vdim, s.state_stride, dev, **conv))
         return self.states[-1]
+
+    def _routing(self) -> None:
+        """Buffers of routed feed-forwards; layers of equal sizes share them."""
+        T, W, dev = self.max_tokens, self.cfg.hidden_size, self.device
+        routed = [l.routed for l in self.w.layers if l.routed is not None]
+        self._z = torch.zeros(T * max((r.split for r in routed), default=0), dtype=torch.float32, device=dev)
+        self._routes: dict = {}
+        for r in routed:
+            key = (r.spec.top, r.spec.experts)
+            if key not in self._routes:
+                self._routes[key] = K.ScoredScratch(T, r.spec.top, r.spec.experts, W, r.up.k, self.act, dev)
+            for name, rows, m, used in (("expert", T * r.spec.top, r.down, r.spec.ff), ("shared", T, r.shared_down, r.spec.shared_ff)):
+                if m is not None and (name, used, rows, m.k) not in self._operands:
+                    self._operands[(name, used, rows, m.k)] = torch.zeros(rows, m.k, dtype=self.act, device=dev)
 
     def _layout(self, l) -> tuple:
         """What an operand of a layer's output product is shared by: every column keeps its role."""
@@ -143,6 +174,8 @@ class LayeredRunner(StepRunner):
     def forward_hidden(self, b) -> torch.Tensor:
         if b.segments is None:
             raise RuntimeError("layered decoders need the step's request segments (StepBatch.segments)")
+        if self.cfg.design.streams:
+            return self._streams(b)
         return self._sequential(b) if self.sequential else self._parallel(b)
 
     def _parallel(self, b) -> torch.Tensor:
@@ -183,7 +216,7 @@ class LayeredRunner(StepRunner):
             if l.down is not None:
                 act = self._operands[("act", l.gate_up.n, l.down.k)][:T]
                 K.row_norm(x, l.norm2, h, eps)
-                K.wide_gemm(h, l.gate_up, act[:, :l.gate_up.n // 2], gelu_glu=True, ws=self.ws)
+                K.wide_gemm(h, l.gate_up, act[:, :l.gate_up.n // 2], glu="gelu", ws=self.ws)
                 K.wide_gemm(act, l.down, x, residual=x, ws=self.ws)
                 n += 3
             follow = None if i == last else w.layers[i + 1].norm       # the final norm reads the wanted rows only
@@ -196,6 +229,58 @@ class LayeredRunner(StepRunner):
             self._after_layer(x)
         self.launches_per_step = n
         return x
+
+    def _streams(self, b) -> torch.Tensor:
+        cfg, w, T, eps = self.cfg, self.w, b.num_tokens, self.cfg.rms_eps
+        decode = T == b.segments.num
+        x, h, y = self.x[:T].view(T, cfg.streams, cfg.hidden_size), self.h[:T], self.y[:T]
+        # what every sublayer reads: its weights of the streams and its norm; nothing behind the last
+        reads = [(s.read, norm) for l in w.layers for s, norm in zip(l.streams, (l.norm, l.norm2))] + [(None, None)]
+        K.stream_embed(b.token_ids[:T], w.embed, cfg.embed_scale, x, *reads[0], h, eps)
+        n, at = 1, 0
+        for l, run in zip(w.layers, self.runs):
+            operand, proj = self._operands[self._layout(l)][:T], self._rows("proj", T, l.split)
+            K.wide_gemm(h, l.proj, proj, ws=self.ws)
+            n += 3 + self._mix(l.mixer, proj, run, b, operand, decode)
+            K.wide_gemm(operand, l.out, y, ws=self.ws)
+            for q, s in enumerate(l.streams):
+                result, routes = y, None
+                if q and l.routed is not None:
+                    result, routes, made = self._routed(l.routed, h, y)
+                    n += 1 + made
+                elif q:
+                    act = self._operands[("act", l.gate_up.n, l.down.k)][:T]
+                    K.wide_gemm(h, l.gate_up, act[:, :l.gate_up.n // 2], glu="silu", ws=self.ws)
+                    K.wide_gemm(act, l.down, y, ws=self.ws)
+                    n += 3
+                at += 1
+                K.stream_step(x, result, s.mix, s.write, h, eps, *reads[at], routes)
+            self._after_layer(x.sum(1) if self.trace is not None else x)
+        self.launches_per_step = n
+        return self.x[:T]
+
+    def _routed(self, m: RoutedWeights, h, y) -> tuple:
+        """A routed feed-forward of ``h`` up to its combination: (shared expert's result, what the experts left, launches made)."""
+        s, T = m.spec, h.shape[0]
+        sc = self._routes[(s.top, s.experts)]
+        z = self._z[:T * m.split].view(T, m.split)
+        shared = None
+        if s.shared_ff:
+            shared = self._operands[("shared", s.shared_ff, self.max_tokens, m.shared_down.k)][:T]
+            K.wide_gemm(h, m.head, z, relu2=shared[:, :s.shared_ff], split=m.split, ws=self.ws)
+        else:
+            K.wide_gemm(h, m.head, z, ws=self.ws)
+        mb = K.scored_route(z, m.correction, h, self.cfg.hidden_size, s.experts, s.top, sc)
+        rows = T * s.top
+        act = self._operands[("expert", s.ff, self.max_tokens * s.top, m.down.k)]
+        out = sc.ys[:, :self.cfg.hidden_size]
+        K.grouped_gemm(sc.xs, m.up, act[:, :s.ff], sc, rows, mb, relu2=True, ws=self.ws)
+        K.grouped_gemm(act, m.down, out, sc, rows, mb, ws=self.ws)
+        if shared is not None:
+            K.wide_gemm(shared, m.shared_down, y, ws=self.ws)
+        gate = z[:, s.outputs:s.outputs + 1] if s.shared_ff else None
+        routes = K.RoutedResult(out, sc.pos, sc.weight, sc.self_weight if s.identity else None, gate, s.top)
+        return (None if shared is None else y), routes, 5 + (shared is not None)
 
     def _after_layer(self, x: torch.Tensor) -> None:
         if self.trace is not None:
@@ -249,6 +334,22 @@ class LayeredRunner(StepRunner):
         return 1 + K.gqa_attention(q, cache, b.page_table, b.segments, out, s.heads, s.dim, s.window, s.scale, s.sink, m.out_scale,
                                    decode=decode, ws=self.ws)
 
+    def _conv_attention(self, m: ConvAttentionWeights, proj, store, b, out, decode: bool) -> int:
+        s, T, (cache, history) = m.spec, proj.shape[0], store
+        q = self._rows("q", T, s.heads * s.width_padded)
+        K.conv_qkv(proj, tuple(m.q_off + o for o in s.offsets), m.conv_w, history, m.freq, b.positions[:T], b.slots[:T], b.segments, q,
+                   cache, s.heads, s.dim, s.vdim, self.cfg.rms_eps)
+        return 1 + K.gqa_attention(q, cache, b.page_table, b.segments, out, s.heads, s.vdim, s.window, s.scale, decode=decode, ws=self.ws,
+                                   keep=s.keep)
+
+    def _biased_attention(self, m: BiasedAttentionWeights, proj, cache: torch.Tensor, b, out, decode: bool) -> int:
+        s, T = m.spec, proj.shape[0]
+        q = self._rows("q", T, s.heads * s.width_padded)
+        K.norm_qkv(proj, tuple(m.q_off + o for o in s.offsets), m.q_norm, m.k_norm, b.positions[:T], b.slots[:T], q, cache, s.heads,
+                   s.dim, s.vdim, self.cfg.rms_eps, (s.temp_coef, s.temp_every))
+        return 1 + K.gqa_attention(q, cache, b.page_table, b.segments, out, s.heads, s.vdim, s.window, s.scale, decode=decode, ws=self.ws,
+                                   bias=m.bias)
+
     def _gated_linear(self, m: GatedLinearWeights, proj, run: _StateRun, b, out, decode: bool) -> int:
         s, T, n = m.spec, proj.shape[0], 1
         low, a = m.low, proj[:, m.a_off:m.a_off + m.low.k]
@@ -272,11 +373,16 @@ class LayeredRunner(StepRunner):
         """Final norm and output head of the selected rows."""
         R = b.num_logit_rows
         h = self.h[:R]                         # free once the last layer has run
-        K.row_norm(hidden, self.w.final_norm, h, self.cfg.rms_eps, rows=b.logit_rows[:R])
+        if self.cfg.design.streams:
+            K.stream_norm(hidden.view(-1, self.cfg.streams, self.cfg.hidden_size), self.w.final_norm, h, self.cfg.rms_eps,
+                          rows=b.logit_rows[:R])
+        else:
+            K.row_norm(hidden, self.w.final_norm, h, self.cfg.rms_eps, rows=b.logit_rows[:R])
         K.wide_gemm(h, self.w.lm_head, logits_out[:R], ws=self.ws)
         self.launches_per_step += 2
         return logits_out[:R]
 
 
 _MIXERS = {DeltaWeights: LayeredRunner._delta, LatentWeights: LayeredRunner._latent, AttentionWeights: LayeredRunner._attention,
-           GatedLinearWeights: LayeredRunner._gated_linear, SsdWeights: LayeredRunner._ssd}
+           GatedLinearWeights: LayeredRunner._gated_linear, SsdWeights: LayeredRunner._ssd,
+           ConvAttentionWeights: LayeredRunner._conv_attention, BiasedAttentionWeights: LayeredRunner._biased_attention}

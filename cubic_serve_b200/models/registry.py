@@ -86,8 +86,9 @@ def _builtin() -> None:
     register(ModelDefinition("layered", LAYERED, parse_config=parse_layered, random_weights=random_layered_weights,
                              load_weights=load_layered_weights, build_runner=runner_layered,
                              description="layers with a mixer each (delta rule per head or per channel, windowed latent "
-                                         "attention, state-space recurrence, sink attention beside gated linear attention), "
-                                         "parallel or sequential, loops, token side inputs, fp32 residual"))
+                                         "attention, state-space recurrence, sink attention beside gated linear attention, "
+                                         "convolved or biased attention), parallel or sequential, loops, token side inputs, "
+                                         "routed experts, fp32 residual streams"))
 
     def parse_q4(path: Path):
         from .qwen4_exp import parse_qwen4_exp_config_json

@@ -723,21 +723,24 @@ def _seg(seg: GdnSegments) -> "native.GdnSegmentsStruct":
     return seg.struct()
 
 
+GLU = {None: 0, "silu": 1, "gelu": 2}       # Glu in csrc/wq_gemm_common.cuh
+
+
 def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: torch.Tensor | None = None,
               relu2: torch.Tensor | None = None, split: int = 0, diag_rows: int = 0, ws: Workspace | None = None,
-              stream_k: bool | None = None, splits: int | None = None, gelu_glu: bool = False) -> None:
+              stream_k: bool | None = None, splits: int | None = None, glu: str | None = None) -> None:
     """``x @ W^T`` with bf16-stored weights through the wide epilogue.
 
     ``x`` fp32: everything is fp32 (``csrc/layered.cu``); ``x`` bf16: tcgen05 with fp32 accumulation.  ``out`` gets the
     product; an fp32 ``out`` may be added to ``residual`` (the same tensor: in-place accumulation).  With ``relu2`` the
-    features from ``split`` on leave there as ``max(v, 0)^2`` and ``out`` holds the first ``split``.  ``gelu_glu``: the rows
-    of ``w`` are interleaved [gate ; up] and ``out`` gets ``gelu_tanh(gate) * up`` (``N / 2`` columns).  ``diag_rows``:
+    features from ``split`` on leave there as ``max(v, 0)^2`` and ``out`` holds the first ``split``.  ``glu`` "gelu" / "silu": the
+    rows of ``w`` are interleaved [gate ; up] and ``out`` gets ``gelu_tanh(gate) * up`` / ``silu(gate) * up`` (``N / 2`` columns).  ``diag_rows``:
     block-diagonal weights, see ``models/layered.py::BlockDiagonal``.  ``x`` may have fewer columns than ``w.k``: the rest
     read as zero."""
     m, k = x.shape[0], w.k
     assert w.fmt == FMT_BF16 and x.stride(1) == 1 and out.stride(1) == 1 and out.shape[0] == m
-    assert gelu_glu == w.act_interleaved and not (gelu_glu and (relu2 is not None or residual is not None or diag_rows))
-    assert out.shape[1] == (split if relu2 is not None else w.n // 2 if gelu_glu else w.n), (out.shape, split, w.n)
+    assert (glu is not None) == w.act_interleaved and not (glu and (relu2 is not None or residual is not None or diag_rows))
+    assert out.shape[1] == (split if relu2 is not None else w.n // 2 if glu else w.n), (out.shape, split, w.n)
     assert residual is None or (residual.dtype == torch.float32 and residual.stride(0) == out.stride(0))
     if relu2 is not None:
         assert relu2.dtype == x.dtype and relu2.stride(1) == 1 and relu2.shape == (m, w.n - split) and split % 4 == 0
@@ -747,12 +750,12 @@ def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: tor
         assert out.dtype == torch.float32
         a = native.F32GemmStruct(x.data_ptr(), x.stride(0), x_cols, w.codes.data_ptr(), out.data_ptr(), out.stride(0),
                                  _ptr(residual), _ptr(relu2), 0 if relu2 is None else relu2.stride(0), split, diag_rows, m,
-                                 w.n, k, 2 if gelu_glu else 0)
+                                 w.n, k, GLU[glu], None, 0)
         native.check(l.cb_f32_gemm(ctypes.byref(a), _stream()), "cb_f32_gemm")
         return
     wide32 = out.dtype == torch.float32
     assert residual is None or wide32
-    assert not (gelu_glu and wide32)
+    assert not (glu and wide32)
     ws = ws or workspace(x.device)
     if stream_k is None:
         stream_k = splits is None and not diag_rows and use_stream_k(m, w.n, FMT_BF16, sm_count(x.device), k)
@@ -764,7 +767,7 @@ def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: tor
     a = native.WideGemmStruct(x.data_ptr(), x.stride(0), x_cols, w.codes.data_ptr(), None if wide32 else out.data_ptr(),
                               out.data_ptr() if wide32 else None, out.stride(0), _ptr(residual), _ptr(relu2),
                               0 if relu2 is None else relu2.stride(0), split, diag_rows, m, w.n, k, int(stream_k), splits,
-                              active().gemm.stream_k_min_units, 2 if gelu_glu else 0)
+                              active().gemm.stream_k_min_units, GLU[glu])
     code = l.cb_bf16_gemm_wide(ctypes.byref(a), ws.gemm.data_ptr(), ws.gemm.numel(), ws.gemm_counters.data_ptr(),
                                ws.status.data_ptr(), _stream())
     native.check(code, "cb_bf16_gemm_wide")
@@ -1039,14 +1042,17 @@ def gqa_prepare(x: torch.Tensor, q_off: int, k_off: int, q_norm: torch.Tensor, k
 
 def gqa_attention(q: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor, seg: GdnSegments, out: torch.Tensor, heads: int,
                   dim: int, window: int, scale: float, sink: float | None = None, out_scale: float = 1.0, decode: bool = False,
-                  splits: int | None = None, ws: Workspace | None = None) -> int:
-    """Windowed grouped-query attention over the paged cache of ``gqa_prepare``, times ``out_scale``.  ``window`` 0: every
-    earlier token; ``sink``: score of a softmax entry without a value.  ``decode``: every segment has at most one row.
+                  splits: int | None = None, ws: Workspace | None = None, keep: int = 0, bias: torch.Tensor | None = None) -> int:
+    """Windowed grouped-query attention over the paged cache of ``gqa_prepare``, ``conv_qkv`` or ``norm_qkv`` with values of
+    ``dim`` channels, times ``out_scale``.  ``window`` 0: every earlier token; ``keep``: the first tokens stay visible behind the
+    window; ``bias`` fp32 ``[distances, H]`` is added to the scaled scores, its last row from the last distance on; ``sink``:
+    score of a softmax entry without a value.  ``decode``: every segment has at most one row.
     ``splits``: key splits of the bf16 decode form (None: as many as fill the device).  Returns the launches made."""
     G, P = cache.shape[1], cache.shape[4]
     T = q.shape[0]
     assert q.is_contiguous() and q.shape[1] == heads * P and out.stride(1) == 1 and out.shape[1] == heads * dim
     assert q.dtype == out.dtype == cache.dtype and page_table.dtype == torch.int32
+    assert bias is None or bias.dtype == torch.float32 and bias.is_contiguous() and bias.shape[1] == heads
     f32 = q.dtype == torch.float32
     l = native.lib()
     partial = None
@@ -1059,15 +1065,173 @@ def gqa_attention(q: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor
             l.cb_gqa_attn_partial_floats(T, seg.num, heads, G, P, 1, 1, ctypes.byref(units))
             a = active().attention
             # a block walks four pages at a time: no more splits than the longest row has such strides
-            keys = page_table.shape[1] * PAGE_TOKENS if window <= 0 else min(window, page_table.shape[1] * PAGE_TOKENS)
+            keys = page_table.shape[1] * PAGE_TOKENS if window <= 0 else min(window + keep, page_table.shape[1] * PAGE_TOKENS)
             splits = min(a.max_splits, -(-keys // 64), max(1, a.target_ctas // units.value))
         if splits > 1:
             ws = ws or workspace(q.device)
             ws.ensure_attn(l.cb_gqa_attn_partial_floats(T, seg.num, heads, G, P, 1, splits, None))
             partial = ws.attn.data_ptr()
     a = native.GqaAttnStruct(q.data_ptr(), out.data_ptr(), out.stride(0), cache.data_ptr(), page_table.data_ptr(),
-                             page_table.shape[1], heads, G, dim, P, window, float(scale), float(out_scale),
-                             float("-inf") if sink is None else float(sink), T, int(f32), int(decode), splits, partial)
+                             page_table.shape[1], heads, G, dim, P, window, keep, float(scale), float(out_scale),
+                             float("-inf") if sink is None else float(sink), _ptr(bias), 0 if bias is None else bias.shape[0] - 1, T, int(f32), int(decode), splits, partial)
     st = _seg(seg)
     native.check(l.cb_gqa_attn(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_gqa_attn")
     return 2 if splits > 1 else 1
+
+
+def _qkv(x: torch.Tensor, offs: tuple[int, int, int], positions: torch.Tensor, slots: torch.Tensor, q: torch.Tensor,
+         cache: torch.Tensor, heads: int, dim: int, vdim: int, eps: float) -> "native.QkvPrepStruct":
+    G, P = cache.shape[1], cache.shape[4]
+    assert cache.is_contiguous() and cache.dtype == x.dtype == q.dtype and q.is_contiguous() and q.shape[1] == heads * P
+    assert x.stride(1) == 1 and slots.dtype == positions.dtype == torch.int32 and x.shape[1] >= offs[2] + G * vdim
+    return native.QkvPrepStruct(x.data_ptr(), x.stride(0), *offs, q.data_ptr(), cache.data_ptr(), slots.data_ptr(), positions.data_ptr(),
+                                heads, G, dim, vdim, P, float(eps), x.shape[0], int(x.dtype == torch.float32))
+
+
+def conv_qkv(x: torch.Tensor, offs: tuple[int, int, int], conv_w: torch.Tensor, state: torch.Tensor | None, freq: torch.Tensor,
+             positions: torch.Tensor, slots: torch.Tensor, seg: GdnSegments, q: torch.Tensor, cache: torch.Tensor, heads: int, dim: int,
+             vdim: int, eps: float) -> None:
+    """Queries, keys and values at the columns ``offs`` of ``x``: causal depthwise convolution over the tokens of a request
+    (``conv_w`` fp32 ``[taps, channels]`` over the columns from ``offs[0]`` on, the last row multiplies the current input; the
+    requests' last inputs ``state [slots, taps - 1, channels]`` are read and replaced), rotary positions of channel i with channel
+    ``i + pairs`` (``freq`` fp32 ``[2, pairs]``: radians per position and what rounding took from them), queries and keys of a
+    head over their root mean square.  Queries to ``q [T, H P]``, keys and values to ``cache [pages, G, 2, 16, P]``."""
+    taps, ldw = conv_w.shape
+    assert conv_w.dtype == freq.dtype == torch.float32 and conv_w.is_contiguous() and freq.is_contiguous() and freq.shape[0] == 2
+    assert taps == 1 or state.dtype == x.dtype and state.is_contiguous() and tuple(state.shape[1:]) == (taps - 1, ldw)
+    a = native.ConvQkvStruct(_qkv(x, offs, positions, slots, q, cache, heads, dim, vdim, eps), conv_w.data_ptr(), ldw, taps,
+                             _ptr(state), freq.data_ptr(), freq.shape[1])
+    st = _seg(seg)
+    native.check(native.lib().cb_conv_qkv(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_conv_qkv")
+
+
+def norm_qkv(x: torch.Tensor, offs: tuple[int, int, int], q_norm: torch.Tensor, k_norm: torch.Tensor, positions: torch.Tensor,
+             slots: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, heads: int, dim: int, vdim: int, eps: float,
+             temp: tuple[float, int] = (0.0, 0)) -> None:
+    """Like ``conv_qkv`` without convolution and rotation: the queries of a token together, and its keys, over their root mean
+    square and times a weight per channel; queries times ``1 + coef ln(floor((position + 1) / every) + 1)`` with ``temp`` =
+    (coef, every), every 0: no factor."""
+    assert q_norm.dtype == k_norm.dtype == torch.float32 and q_norm.numel() == heads * dim and k_norm.numel() == cache.shape[1] * dim
+    a = native.NormQkvStruct(_qkv(x, offs, positions, slots, q, cache, heads, dim, vdim, eps), q_norm.data_ptr(), k_norm.data_ptr(),
+                             float(temp[0]), int(temp[1]))
+    native.check(native.lib().cb_norm_qkv(ctypes.byref(a), _stream()), "cb_norm_qkv")
+
+
+# ------------------------------------------------------------------ several residual streams
+def stream_embed(ids: torch.Tensor, table: torch.Tensor, scale: float, x: torch.Tensor, w_in: torch.Tensor, norm_w: torch.Tensor,
+                 h: torch.Tensor, eps: float) -> None:
+    """All streams of ``x`` fp32 ``[T, S, W]`` = ``scale`` times the embedding rows; ``h`` = norm of their sum weighted by ``w_in``."""
+    _stream_norm(x, w_in, norm_w, h, eps, x.shape[0], None, ids, table, scale)
+
+
+def stream_norm(x: torch.Tensor, norm_w: torch.Tensor, h: torch.Tensor, eps: float, rows: torch.Tensor | None = None,
+                w_in: torch.Tensor | None = None) -> None:
+    """``h[i]`` = norm of row i's streams, summed with weights ``w_in`` (None: ones); ``rows`` int64: the rows taken."""
+    _stream_norm(x, w_in, norm_w, h, eps, x.shape[0] if rows is None else rows.numel(), rows, None, None, 1.0)
+
+
+def _stream_norm(x, w_in, norm_w, h, eps, n, rows, ids, table, scale) -> None:
+    assert x.dtype == norm_w.dtype == torch.float32 and x.is_contiguous() and x.dim() == 3 and h.stride(1) == 1 and h.shape[0] >= n
+    assert w_in is None or w_in.dtype == torch.float32 and w_in.numel() == x.shape[1]
+    assert table is None or table.dtype == torch.bfloat16 and table.shape[1] == x.shape[2]
+    a = native.StreamNormStruct(_ptr(ids), _ptr(table), 0 if table is None else table.shape[0], float(scale), x.data_ptr(), _ptr(rows),
+                                _ptr(w_in), norm_w.data_ptr(), h.data_ptr(), h.stride(0), n, x.shape[1], x.shape[2], float(eps),
+                                int(h.dtype == torch.float32))
+    native.check(native.lib().cb_stream_norm(ctypes.byref(a), _stream()), "cb_stream_norm")
+
+
+def stream_step(x: torch.Tensor, y: torch.Tensor | None, mix: torch.Tensor, out: torch.Tensor, h: torch.Tensor, eps: float,
+                next_in: torch.Tensor | None = None, next_w: torch.Tensor | None = None, routes: "RoutedResult | None" = None) -> None:
+    """A sublayer's result ``y`` joins the streams ``x`` fp32 ``[T, S, W]``: ``x_t <- sum_s mix[s, t] x_s + out[t] y``.  ``routes``:
+    the result is what the token's experts left, plus ``y`` times the shared expert's gate, plus the sublayer's input ``h`` times
+    the weight of the experts that return it.  With ``next_w`` ``h`` becomes the next sublayer's input, the norm of
+    ``sum_s next_in[s] x_s``."""
+    T, S, W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and h.stride(1) == 1 and h.shape[0] >= T
+    assert y is None or y.dtype == h.dtype and y.stride(1) == 1 and y.shape[1] >= W
+    r = routes
+    assert all(t is None or t.dtype == torch.float32 for t in (mix, out, next_in, next_w)) and mix.numel() == S * S and out.numel() == S
+    a = native.StreamStepStruct(
+        x.data_ptr(), _ptr(y), 0 if y is None else y.stride(0), None if r is None else r.rows.data_ptr(), 0 if r is None else r.rows.stride(0),
+        None if r is None else r.pos.data_ptr(), None if r is None else r.weight.data_ptr(), None if r is None else _ptr(r.self_weight),
+        0 if r is None else r.top, None if r is None else _ptr(r.gate), 0 if r is None or r.gate is None else r.gate.stride(0),
+        mix.data_ptr(), out.data_ptr(), _ptr(next_in), _ptr(next_w), h.data_ptr(), h.stride(0), T, S, W, float(eps),
+        int(h.dtype == torch.float32))
+    native.check(native.lib().cb_stream_step(ctypes.byref(a), _stream()), "cb_stream_step")
+
+
+# ------------------------------------------------------------------ scored experts
+@dataclass
+class RoutedResult:
+    """What ``stream_step`` puts a routed feed-forward's result together from."""
+    rows: torch.Tensor               # [routes, W] results of the experts, by place
+    pos: torch.Tensor                # int32 [T, top] places, -1: none
+    weight: torch.Tensor             # fp32 [T, top]
+    self_weight: torch.Tensor | None # fp32 [T] weight of the token itself
+    gate: torch.Tensor | None        # fp32 [T, 1] logits of the shared expert's gate (any row stride)
+    top: int
+
+
+class ScoredScratch:
+    """Fixed-address buffers between routing and combination for up to ``max_tokens`` tokens of layers with ``experts`` experts of
+    which a token uses ``top``."""
+
+    def __init__(self, max_tokens: int, top: int, experts: int, width: int, k: int, act: torch.dtype, device) -> None:
+        """``k``: columns of an expert's operand (``width`` rounded up, the rest stays zero)."""
+        routes = max_tokens * top
+        i32 = dict(dtype=torch.int32, device=device)
+        self.ids, self.pos = torch.zeros(routes, **i32), torch.zeros(routes, **i32)
+        self.weight = torch.zeros(routes, dtype=torch.float32, device=device)
+        self.self_weight = torch.zeros(max_tokens, dtype=torch.float32, device=device)
+        self.counts = torch.zeros(experts + 1, **i32)
+        self.tiles = torch.zeros(1 + 3 * (-(-routes // 16) + experts), **i32)
+        self.xs = torch.zeros(routes, k, dtype=act, device=device)
+        self.ys = torch.zeros(routes, -(-width // 8) * 8, dtype=act, device=device)
+
+
+def rows_per_item(tokens: int, top: int, experts: int, f32: bool) -> int:
+    """Rows of a work item of the grouped products: about twice an expert's average share (one item for most experts)."""
+    if f32:
+        return 64                                      # the fp32 product's tile
+    share = 2 * tokens * top // experts
+    return 32 if share <= 32 else 64 if share <= 64 else 128 if share <= 128 else 256
+
+
+def scored_route(z: torch.Tensor, correction: torch.Tensor, h: torch.Tensor, width: int, experts: int, top: int, sc: ScoredScratch) -> int:
+    """Routes ``h``'s rows by the fp32 logits ``z [T, >= outputs]`` (outputs = ``correction.numel()``; those from ``experts`` on
+    return the token itself) and copies them to their experts' places in ``sc.xs``.  Returns the rows of a work item."""
+    T = z.shape[0]
+    assert z.dtype == correction.dtype == torch.float32 and z.stride(1) == 1 and h.dtype == sc.xs.dtype and h.stride(1) == 1
+    assert sc.counts.numel() == experts + 1 and T * top <= sc.ids.numel()
+    mb = rows_per_item(T, top, experts, h.dtype == torch.float32)
+    a = native.ScoredMoeStruct(z.data_ptr(), z.stride(0), correction.data_ptr(), h.data_ptr(), h.stride(0), sc.xs.data_ptr(), sc.xs.stride(0),
+                               T, width, h.element_size(), experts, correction.numel(), top, mb, sc.ids.data_ptr(), sc.pos.data_ptr(),
+                               sc.weight.data_ptr(), sc.self_weight.data_ptr(), sc.counts.data_ptr(), sc.tiles.data_ptr())
+    native.check(native.lib().cb_scored_moe_route(ctypes.byref(a), _stream()), "cb_scored_moe_route")
+    return mb
+
+
+def grouped_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, sc: ScoredScratch, rows: int, mb: int, relu2: bool = False,
+                 ws: Workspace | None = None) -> None:
+    """``out[rows of e] = x[rows of e] @ W_e^T`` (``relu2``: ``max(v, 0)^2`` of it) over the work list of ``scored_route`` for bf16
+    experts stacked in ``w``; ``rows``: tokens times routes of a token.  fp32 ``x``: everything is fp32."""
+    E = w.codes.shape[0]
+    assert w.fmt == FMT_BF16 and w.codes.dim() == 3 and x.shape[1] == w.k and out.shape[1] == w.n and out.dtype == x.dtype
+    assert x.stride(1) == out.stride(1) == 1
+    items = -(-rows // mb) + E
+    l = native.lib()
+    if x.dtype == torch.float32:
+        # with relu2 every feature leaves through the second output, from feature 0 on
+        a = native.F32GemmStruct(x.data_ptr(), x.stride(0), x.shape[1], w.codes.data_ptr(), out.data_ptr(), out.stride(0), None,
+                                 out.data_ptr() if relu2 else None, out.stride(0) if relu2 else 0, 0, 0, rows, w.n, w.k, 0,
+                                 sc.tiles.data_ptr(), items)
+        native.check(l.cb_f32_gemm(ctypes.byref(a), _stream()), "cb_f32_gemm")
+        return
+    ws = ws or workspace(x.device)
+    if relu2:
+        code = l.cb_wq_gemm_grouped_relu2(x.data_ptr(), x.stride(0), w.codes.data_ptr(), out.data_ptr(), out.stride(0), rows, w.n, w.k,
+                                          sc.tiles.data_ptr(), items, mb, E, ws.status.data_ptr(), _stream())
+    else:
+        code = l.cb_wq_gemm_grouped(FMT_BF16, x.data_ptr(), x.stride(0), w.codes.data_ptr(), None, out.data_ptr(), out.stride(0), 1.0, rows,
+                                    w.n, w.k, w.k, sc.tiles.data_ptr(), items, mb, E, 0, 0, ws.status.data_ptr(), _stream())
+    native.check(code, "cb_wq_gemm_grouped")

@@ -281,13 +281,18 @@ def _declare(l: ctypes.CDLL) -> None:
     l.cb_gqa_attn.argtypes = [vp, vp, vp]
     l.cb_gqa_attn_partial_floats.argtypes = [i, i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
     l.cb_gqa_attn_partial_floats.restype = ll
+    l.cb_conv_qkv.argtypes = [vp, vp, vp]
+    for name in ("norm_qkv", "stream_step", "stream_norm", "scored_moe_route"):
+        getattr(l, f"cb_{name}").argtypes = [vp, vp]
+    l.cb_wq_gemm_grouped_relu2.argtypes = [vp, i, vp, vp, i, i, i, i, vp, i, i, i, vp, vp]
     l.cb_latent_prepare.argtypes = [vp, i, i, i, i, i, vp, vp, vp, i, vp, i, vp, i, f, i, vp]
     l.cb_latent_attn.argtypes = [vp, vp, vp]
     l.cb_latent_attn_partial_floats.argtypes = [i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
     l.cb_latent_attn_partial_floats.restype = ll
     for name in ("bf16_gemm_wide", "f32_gemm", "row_norm", "embed_norm", "concat_rows", "latent_prepare",
                  "latent_attn", "gated_parts_norm", "embed_rows", "add_norm_rows", "side_gate", "side_input",
-                 "gqa_prepare", "gqa_attn"):
+                 "gqa_prepare", "gqa_attn", "conv_qkv", "norm_qkv", "stream_step", "stream_norm", "scored_moe_route",
+                 "wq_gemm_grouped_relu2"):
         getattr(l, f"cb_{name}").restype = i
     # fp8 (e4m3 x e4m3) tensor path: activation quantizers and the GEMM entries
     l.cb_fp8_quantize_rows.argtypes = [vp, i, vp, i, vp, i, i, vp]
@@ -340,7 +345,8 @@ class F32GemmStruct(ctypes.Structure):
     _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("x_cols", ctypes.c_int), ("w", ctypes.c_void_p),
                 ("y", ctypes.c_void_p), ("ldy", ctypes.c_int), ("residual", ctypes.c_void_p), ("y2", ctypes.c_void_p),
                 ("ldy2", ctypes.c_int), ("n_split", ctypes.c_int), ("diag_n", ctypes.c_int), ("M", ctypes.c_int),
-                ("N", ctypes.c_int), ("K", ctypes.c_int), ("glu", ctypes.c_int)]
+                ("N", ctypes.c_int), ("K", ctypes.c_int), ("glu", ctypes.c_int), ("tiles", ctypes.c_void_p),
+                ("max_items", ctypes.c_int)]
 
 
 class RecPrepStruct(ctypes.Structure):
@@ -395,9 +401,60 @@ class GqaAttnStruct(ctypes.Structure):
     """Mirror of ``CbGqaAttn`` in ``csrc/gqa_attn.cu``."""
     _fields_ = [("q", ctypes.c_void_p), ("out", ctypes.c_void_p), ("ldo", ctypes.c_int), ("cache", ctypes.c_void_p),
                 ("page_table", ctypes.c_void_p), ("max_pages", ctypes.c_int), ("H", ctypes.c_int), ("G", ctypes.c_int),
-                ("d", ctypes.c_int), ("P", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float),
-                ("out_scale", ctypes.c_float), ("sink", ctypes.c_float), ("tokens", ctypes.c_int), ("f32", ctypes.c_int),
+                ("e", ctypes.c_int), ("P", ctypes.c_int), ("window", ctypes.c_int), ("keep", ctypes.c_int),
+                ("scale", ctypes.c_float), ("out_scale", ctypes.c_float), ("sink", ctypes.c_float), ("bias", ctypes.c_void_p),
+                ("bias_far", ctypes.c_int), ("tokens", ctypes.c_int), ("f32", ctypes.c_int),
                 ("decode", ctypes.c_int), ("splits", ctypes.c_int), ("partial", ctypes.c_void_p)]
+
+
+class QkvPrepStruct(ctypes.Structure):
+    """Mirror of ``CbQkvPrep`` in ``csrc/qkv_prepare.cu``."""
+    _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("q_off", ctypes.c_int), ("k_off", ctypes.c_int),
+                ("v_off", ctypes.c_int), ("q", ctypes.c_void_p), ("cache", ctypes.c_void_p),
+                ("slots", ctypes.c_void_p), ("positions", ctypes.c_void_p), ("H", ctypes.c_int), ("G", ctypes.c_int),
+                ("d", ctypes.c_int), ("e", ctypes.c_int), ("P", ctypes.c_int), ("eps", ctypes.c_float),
+                ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
+
+
+class ConvQkvStruct(ctypes.Structure):
+    """Mirror of ``CbConvQkv`` in ``csrc/qkv_prepare.cu``."""
+    _fields_ = [("a", QkvPrepStruct), ("w", ctypes.c_void_p), ("ldw", ctypes.c_int), ("taps", ctypes.c_int),
+                ("state", ctypes.c_void_p), ("freq", ctypes.c_void_p), ("pairs", ctypes.c_int)]
+
+
+class NormQkvStruct(ctypes.Structure):
+    """Mirror of ``CbNormQkv`` in ``csrc/qkv_prepare.cu``."""
+    _fields_ = [("a", QkvPrepStruct), ("qw", ctypes.c_void_p), ("kw", ctypes.c_void_p), ("coef", ctypes.c_float),
+                ("every", ctypes.c_int)]
+
+
+class StreamStepStruct(ctypes.Structure):
+    """Mirror of ``CbStreamStep`` in ``csrc/streams.cu``."""
+    _fields_ = [("x", ctypes.c_void_p), ("y", ctypes.c_void_p), ("ldy", ctypes.c_int), ("rows", ctypes.c_void_p),
+                ("ld_rows", ctypes.c_int), ("pos", ctypes.c_void_p), ("weight", ctypes.c_void_p),
+                ("self_w", ctypes.c_void_p), ("top", ctypes.c_int), ("gate", ctypes.c_void_p), ("ldg", ctypes.c_int),
+                ("mix", ctypes.c_void_p), ("out", ctypes.c_void_p), ("in_w", ctypes.c_void_p), ("w", ctypes.c_void_p),
+                ("h", ctypes.c_void_p), ("ldh", ctypes.c_int), ("n", ctypes.c_int), ("S", ctypes.c_int),
+                ("W", ctypes.c_int), ("eps", ctypes.c_float), ("f32", ctypes.c_int)]
+
+
+class StreamNormStruct(ctypes.Structure):
+    """Mirror of ``CbStreamNorm`` in ``csrc/streams.cu``."""
+    _fields_ = [("ids", ctypes.c_void_p), ("table", ctypes.c_void_p), ("vocab", ctypes.c_int),
+                ("scale", ctypes.c_float), ("x", ctypes.c_void_p), ("rows", ctypes.c_void_p),
+                ("in_w", ctypes.c_void_p), ("w", ctypes.c_void_p), ("h", ctypes.c_void_p), ("ldh", ctypes.c_int),
+                ("n", ctypes.c_int), ("S", ctypes.c_int), ("W", ctypes.c_int), ("eps", ctypes.c_float),
+                ("f32", ctypes.c_int)]
+
+
+class ScoredMoeStruct(ctypes.Structure):
+    """Mirror of ``CbScoredMoe`` in ``csrc/moe.cu``."""
+    _fields_ = [("z", ctypes.c_void_p), ("ldz", ctypes.c_int), ("correction", ctypes.c_void_p), ("x", ctypes.c_void_p),
+                ("ldx", ctypes.c_int), ("xs", ctypes.c_void_p), ("ldxs", ctypes.c_int), ("T", ctypes.c_int),
+                ("W", ctypes.c_int), ("elem", ctypes.c_int), ("experts", ctypes.c_int), ("outputs", ctypes.c_int),
+                ("top", ctypes.c_int), ("mb", ctypes.c_int), ("ids", ctypes.c_void_p), ("pos", ctypes.c_void_p),
+                ("weight", ctypes.c_void_p), ("self_w", ctypes.c_void_p), ("counts", ctypes.c_void_p),
+                ("tiles", ctypes.c_void_p)]
 
 
 class ReduceNormStruct(ctypes.Structure):

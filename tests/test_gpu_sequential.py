@@ -28,7 +28,7 @@ def test_gated_gelu_product(dtype, m, ff, k, how):
     w = wq_pack.pack_bf16(torch.cat([gate, up]))
     want = R.gelu_tanh(x.double() @ w.codes[:ff].double().t()) * (x.double() @ w.codes[ff:].double().t())
     out = torch.full((m, ff + 16), 7.0, dtype=dtype, device=DEV)
-    K.wide_gemm(x.to(DEV), wq_pack.swiglu_interleave(w).to(DEV), out[:, 8:8 + ff], gelu_glu=True, **how)
+    K.wide_gemm(x.to(DEV), wq_pack.swiglu_interleave(w).to(DEV), out[:, 8:8 + ff], glu="gelu", **how)
     close(out[:, 8:8 + ff], want, dtype, exact=1e-5, rough=1e-2)
     assert (out[:, :8] == 7).all() and (out[:, 8 + ff:] == 7).all()
     K.workspace(torch.device(DEV)).check_status()
@@ -43,7 +43,7 @@ def test_gated_gelu_extremes(dtype):
     w = torch.zeros(32, 64)
     w[:16, 0], w[16:, 0] = 1.0, 0.5
     out = torch.zeros(4, 16, dtype=dtype, device=DEV)
-    K.wide_gemm(x.to(DEV), wq_pack.swiglu_interleave(wq_pack.pack_bf16(w)).to(DEV), out, gelu_glu=True)
+    K.wide_gemm(x.to(DEV), wq_pack.swiglu_interleave(wq_pack.pack_bf16(w)).to(DEV), out, glu="gelu")
     v = x[:, 0].double()
     got, want = out.double().cpu(), (R.gelu_tanh(v) * 0.5 * v).unsqueeze(1).expand(4, 16)
     assert torch.isfinite(got).all() and ((got - want).abs() <= (1e-5 if dtype == torch.float32 else 1e-2) * (want.abs() + 0.1)).all()
