@@ -386,8 +386,9 @@ def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple
                     window=m.window or cfg.max_position)
             elif isinstance(m, (ConvAttentionSpec, BiasedAttentionSpec)):
                 k = (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim
-                extra = {"taps": m.conv, "keep": m.keep} if isinstance(m, ConvAttentionSpec) else {"buckets": m.buckets}
-                add("attention.gqa", "paged", m.out_width, k, heads=m.heads, window=m.window or cfg.max_position, **extra)
+                extra = {"taps": m.conv} if isinstance(m, ConvAttentionSpec) else {"buckets": m.buckets}
+                kept = {"keep": m.keep} if getattr(m, "keep", 0) else {}
+                add("attention.gqa", "paged", m.out_width, k, heads=m.heads, window=m.window or cfg.max_position, **extra, **kept)
             elif isinstance(m, DeltaSpec):
                 add("delta_rule." + ("channel" if m.per_channel else "head"), "state32", m.out_width, m.channels, heads=m.heads,
                     taps=m.conv)
@@ -404,7 +405,7 @@ def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple
             add("linear.bf16", "parallel_out", W, l.mixer.out_width + l.ff)
         if l.routed is not None:
             r = l.routed
-            add("moe.route", f"top{r.top}", W, W, experts=r.experts, identity=r.identity)
+            add("moe.route", f"top{r.top}", W, W, experts=r.experts, outputs=r.outputs)
             add("linear.bf16", "experts_up", r.ff, W, experts=r.experts)
             add("linear.bf16", "experts_down", W, r.ff, experts=r.experts)
             if r.shared_ff:

@@ -87,7 +87,68 @@ SEQUENTIAL = {
                                       mamba2(4, 130, 136, 1, 4, 4, 128),
                                       parallel((3, 1, 200, 19, 0.1, 40, 300.0, None), (2, 96, 200, 4.0), (1.0, 0.5), 96)], 40),
 }
-ALL = {**CASES, **SEQUENTIAL}
+
+
+# ------------------------------------------------------------------ several residual streams (Vimelorn)
+def ff_of(mlp):
+    """``mlp``: width of a dense feed-forward, 0 for none, or ``routed(...)``."""
+    return mlp if isinstance(mlp, dict) else {"kind": "dense", "ff": mlp} if mlp else None
+
+
+def routed(experts, top, ff, identity=0, shared=0):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": identity, "top": top},
+            "shared": {"ff": shared} if shared else None}
+
+
+def near(heads, kv_heads, dim, vdim, conv, scale, dims, base, size, keep, mlp):
+    """Convolved attention with rotary halves; ``size`` 0: no window."""
+    return {"type": "attention",
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv, "scale": scale,
+                      "rot": {"dims": dims, "base": base}, "mask": {"size": size, "keep_first": keep} if size else None},
+            "mlp": ff_of(mlp)}
+
+
+def far(heads, kv_heads, dim, vdim, scale, bias_max, temp, mlp, rows=8):
+    """Attention with a bias by distance (a table of ``rows`` rows); ``temp``: (coef, every) or None."""
+    return {"type": "attention_2", "rows": rows,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "bias_max": bias_max,
+                      "q_temp": dict(zip(("coef", "every"), temp)) if temp else None},
+            "mlp": ff_of(mlp)}
+
+
+class StreamConfig(dict):
+    """A configuration with the rows of its layers' bias tables, which only the tensors state."""
+    bias_rows: list[int]
+    close_calls = False          # the choice of experts may hang on rounding
+
+
+def streams(vocab, width, layers, count, scale=1.0, eps=1e-5, close_calls=False):
+    rows = [l.pop("rows", 0) for l in layers]
+    cfg = StreamConfig(architecture="Vimelorn", vocab=vocab, width=width, layers=layers, norm={"eps": eps}, streams=count,
+                       embedding={"scale": scale})
+    cfg.bias_rows, cfg.close_calls = rows, close_calls
+    return cfg
+
+
+STREAMS = {
+    # both attentions and both feed-forwards, grouped heads, key and value widths that differ, a layer without a feed-forward
+    "str": streams(210, 96, [near(6, 2, 24, 40, 3, 0.5, 12, 1000.0, 21, 5, 80), far(4, 2, 20, 28, 0.3, 30, (0.5, 16), routed(5, 3, 48, 3, 64)),
+                             near(4, 4, 32, 16, 2, 0.4, 32, 5000.0, 40, 18, 0), far(2, 1, 32, 32, 0.25, 70, None, routed(7, 2, 40), 11),
+                             near(3, 1, 16, 24, 4, 0.5, 8, 100.0, 17, 0, routed(3, 2, 56, 1, 32))], 2, 9.5, 1e-6),
+    # one stream, single heads, a window of one token, one tap, no rotated channel, the smallest table, a single expert
+    "str_small": streams(71, 64, [near(1, 1, 16, 16, 1, 0.5, 0, 10.0, 1, 0, routed(1, 1, 32)),
+                                  far(1, 1, 16, 16, 0.25, 2, (1.0, 1), 48, 2), near(2, 1, 16, 16, 1, 0.4, 16, 100.0, 1, 1, routed(2, 1, 16, 1, 16))], 1),
+    # a choice of experts per token
+    "str_select": streams(150, 64, [near(4, 2, 16, 16, 3, 0.5, 16, 200.0, 30, 4, routed(9, 3, 32, 3, 32)), far(2, 2, 16, 16, 0.3, 40, (0.3, 20), routed(6, 2, 24, 2), 10),
+                                    near(4, 1, 16, 24, 2, 0.4, 8, 200.0, 25, 2, routed(16, 4, 16, 0, 16))], 2, 2.0, close_calls=True),
+    # odd widths, more taps than the unrolled forms have, three query heads per key head, every earlier token, three streams
+    "str_odd": streams(123, 68, [near(9, 3, 13, 9, 6, 0.6, 6, 50.0, 0, 0, 44), far(6, 2, 7, 13, 0.5, 25, (0.2, 7), routed(4, 4, 20, 2, 36), 9),
+                                 near(5, 1, 18, 21, 7, 0.5, 10, 300.0, 33, 7, routed(6, 5, 12, 4))], 3, 2.5, 1e-4),
+    # wide heads, more query heads than a block has rows, kept tokens over several pages, many experts, four streams
+    "str_wide": streams(256, 128, [near(40, 1, 72, 136, 4, 0.2, 64, 10000.0, 50, 35, routed(40, 6, 64, 9, 128)),
+                                   far(20, 1, 200, 64, 0.1, 60, (0.3, 30), 96, 16), near(3, 1, 200, 256, 3, 0.1, 40, 300.0, 19, 65, 0)], 4, 3.0),
+}
+ALL = {**CASES, **SEQUENTIAL, **STREAMS}
 LOW_RANKS = (12, 20)          # inner sizes of the low-rank decay and gate projections
 
 
@@ -104,6 +165,9 @@ def tensors(cfg: dict, seed: int = 0) -> dict[str, torch.Tensor]:
     mat("embed", cfg["vocab"], W, math.sqrt(W))
     if cfg["architecture"] == "Loduzen":
         _sequential_tensors(cfg, mat, vec)
+        return out
+    if cfg["architecture"] == "Vimelorn":
+        _stream_tensors(cfg, mat, vec, out, g)
         return out
     vec("embed.norm", W)
     vec("final.norm", W)
@@ -192,6 +256,53 @@ def _sequential_tensors(cfg: dict, mat, vec) -> None:
             mat(f"l{i}.side.gate", side, W)
             mat(f"l{i}.side.proj", W, side)
             vec(f"l{i}.side.norm", W, 0.3, 0.1)
+
+
+def _stream_tensors(cfg: dict, mat, vec, out: dict, g) -> None:
+    W, S = cfg["width"], cfg["streams"]
+    rows = cfg.bias_rows
+    out["embed"] = (out["embed"].float() / cfg["embedding"]["scale"]).to(torch.bfloat16)
+    vec("final.norm", W, 1.0)
+    mat("head", cfg["vocab"], W)
+    for i, l in enumerate(cfg["layers"]):
+        m, p, mlp = l["mixer"], f"l{i}.mix", l["mlp"]
+        vec(f"l{i}.norm1", W, 1.0)
+        sizes = {"q": m["heads"] * m["dim"], "k": m["kv_heads"] * m["dim"], "v": m["kv_heads"] * m["vdim"]}
+        for t, n in sizes.items():
+            mat(f"{p}.{t}", n, W)
+            if l["type"] == "attention":
+                mat(f"{p}.{t}.conv", n, m["conv"])
+            elif t != "v":
+                vec(f"{p}.{t}.norm", n, 1.0, 0.3)
+        if l["type"] == "attention_2":
+            out[f"{p}.rel"] = torch.randn(rows[i], m["heads"], generator=g).to(torch.bfloat16)
+        mat(f"{p}.o", W, m["heads"] * m["vdim"])
+        for q in (1, 2) if mlp else (1,):
+            vec(f"l{i}.hc{q}.in", S, 1.0 / S, 0.2)
+            vec(f"l{i}.hc{q}.out", S, 1.0, 0.3)
+            out[f"l{i}.hc{q}.mix"] = (torch.eye(S) + 0.15 * torch.randn(S, S, generator=g)).to(torch.bfloat16)
+        if not mlp:
+            continue
+        p = f"l{i}.mlp"
+        vec(f"l{i}.norm2", W, 1.0)
+        if mlp["kind"] == "dense":
+            for t in ("gate", "up"):
+                mat(f"{p}.{t}", mlp["ff"], W)
+            mat(f"{p}.down", W, mlp["ff"])
+            continue
+        r = mlp["router"]
+        n = r["experts"] + r["identity"]
+        for e in range(r["experts"]):
+            mat(f"{p}.e{e}.up", mlp["expert"]["ff"], W)
+            mat(f"{p}.e{e}.down", W, mlp["expert"]["ff"])
+        # corrections farther apart than any two scores: the choice of a token's experts does not hang on rounding, their weights
+        # follow the scores; or close together: every token has experts of its own, and some tokens a close call
+        mat(f"{p}.router", n, W, 3.0)
+        out[f"{p}.correction"] = ((0.3 / n if cfg.close_calls else 1.5) * torch.randperm(n, generator=g)).to(torch.bfloat16)
+        if mlp["shared"]:
+            mat(f"{p}.shared.up", mlp["shared"]["ff"], W)
+            mat(f"{p}.shared.down", W, mlp["shared"]["ff"])
+            mat(f"{p}.shared.sg", 1, W)
 
 
 def write(path, cfg: dict, weights: dict[str, torch.Tensor]):

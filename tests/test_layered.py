@@ -10,8 +10,8 @@ import pytest
 import torch
 
 sys.path.insert(0, str(Path(__file__).parent))
-from layered_cases import (ALL, CASES, LOW_RANKS, SEQUENTIAL, channel, config, delta, latent, mamba2, parallel,  # noqa: E402
-                           prompt, sequential, tensors, write)
+from layered_cases import (ALL, CASES, LOW_RANKS, SEQUENTIAL, STREAMS, channel, config, delta, far, latent, mamba2, near,  # noqa: E402
+                           parallel, prompt, routed, sequential, streams, tensors, write)
 
 from cubic_serve_b200.models import layered as L  # noqa: E402
 from cubic_serve_b200.models import layered_reference as R  # noqa: E402
@@ -104,11 +104,68 @@ def test_sequential_checkpoint_admission(tmp_path):
                                                                           "linear_recurrence.channel", "token_side"}
 
 
-def test_random_weights_of_both_designs_are_admitted(tmp_path):
-    for name in ("layered-tiny", "layered-seq-tiny"):
+def test_random_weights_of_all_designs_are_admitted(tmp_path):
+    for name in ("layered-tiny", "layered-seq-tiny", "layered-streams-tiny"):
         cfg = L.NAMED[name]()
         back = admit_checkpoint(L.write_checkpoint(tmp_path / name, cfg, L.random_tensors(cfg, 3))).cfg
         assert (back.layers, back.side_dim, back.loop) == (cfg.layers, cfg.side_dim, cfg.loop)
+        assert (back.streams, back.embed_scale) == (cfg.streams, cfg.embed_scale)
+
+
+@pytest.mark.parametrize("change, message", [
+    (lambda c: c["layers"][0].update(type="latent_attention"), "unknown mixer"),
+    (lambda c: c["layers"][1]["mlp"].update(kind="experts"), "unknown feed-forward"),
+    (lambda c: c["layers"][0]["mixer"].update(kv_heads=4), "grouped evenly"),
+    (lambda c: c["layers"][0]["mixer"].update(vdim=300), "up to 256 channels"),
+    (lambda c: c["layers"][0]["mixer"].update(conv=17), "convolution taps"),
+    (lambda c: c["layers"][0]["mixer"]["rot"].update(dims=26), "inside a head"),
+    (lambda c: c["layers"][0]["mixer"]["mask"].update(size=0), "at least the token itself"),
+    (lambda c: c["layers"][0]["mixer"]["mask"].update(keep_first=-1), "not negative"),
+    (lambda c: c["layers"][1]["mixer"].update(bias_max=4), "behind their first half"),
+    (lambda c: c["layers"][1]["mixer"]["q_temp"].update(every=0), "positive number of positions"),
+    (lambda c: c["layers"][1]["mlp"]["router"].update(top=9), "no more routes than outputs"),
+    (lambda c: c["layers"][1]["mlp"]["router"].update(experts=255), "256 outputs"),
+    (lambda c: c.update(streams=9), "residual streams"),
+])
+def test_bad_stream_configurations_are_refused(change, message):
+    c = copy.deepcopy(STREAMS["str"])
+    change(c)
+    with pytest.raises(L.LayeredConfigError, match=message):
+        L.parse_layered_config(c, {n: tuple(t.shape) for n, t in tensors(STREAMS["str"]).items()})
+
+
+def test_routed_feed_forwards_belong_to_designs_with_streams():
+    c = copy.deepcopy(SEQUENTIAL["seq"])
+    c["layers"][0]["mlp"] = routed(4, 2, 16)
+    with pytest.raises(L.LayeredConfigError, match="unknown feed-forward"):
+        L.parse_layered_config(c, {n: tuple(t.shape) for n, t in tensors(SEQUENTIAL["seq"]).items()})
+
+
+def test_stream_checkpoint_admission(tmp_path):
+    from cubic_serve_b200.contracts.model import ModelSpec
+    from cubic_serve_b200.contracts.plan import decoder_step_operators
+    from cubic_serve_b200.models import registry
+    raw, w = STREAMS["str"], tensors(STREAMS["str"])
+    ck = admit_checkpoint(write(tmp_path / "good", raw, w))
+    assert ck.cfg.family == "layered" and registry.for_architecture("Vimelorn").family == "layered" and ck.cfg.streams == 2
+    info = inspect_checkpoint(tmp_path / "good")
+    assert info["mixers"] == {"biased_attention": 2, "conv_attention": 3} and info["residual_streams"] == 2 and info["routed_layers"] == 3
+    # what a missing feed-forward would need is tolerated, anything else is not
+    admit_checkpoint(write(tmp_path / "spare", raw, {**w, "l2.norm2": w["l1.norm2"].clone(), "l2.hc2.in": w["l1.hc2.in"].clone()}))
+    with pytest.raises(CheckpointError, match="does not own"):
+        admit_checkpoint(write(tmp_path / "extra", raw, {**w, "l1.mlp.e5.up": w["l1.mlp.e0.up"].clone()}))
+    with pytest.raises(CheckpointError, match="missing tensor l0.hc2.mix"):
+        admit_checkpoint(write(tmp_path / "missing", raw, {n: t for n, t in w.items() if n != "l0.hc2.mix"}))
+    with pytest.raises(CheckpointError, match="l1.mix.rel is stated"):
+        admit_checkpoint(write(tmp_path / "rel", raw, {n: t for n, t in w.items() if n != "l1.mix.rel"}))
+    # keys and values of 64 padded channels for every layer; convolution inputs of the three convolved ones
+    spec = ModelSpec.from_layered(ck.cfg)
+    assert spec.cache.runs == 5 and spec.cache.page_bytes == (2 + 2 + 4 + 1 + 1) * 2 * 16 * 64 * 2
+    conv = (2 * (144 + 48 + 80), 1 * (128 + 128 + 64), 3 * (48 + 16 + 24))
+    assert spec.state.runs == 3 and ck.cfg.state_bytes_per_request == 2 * sum(conv) and ck.cfg.is_hybrid
+    assert {o.semantic_op for o in decoder_step_operators(ck.cfg, 8)} >= {"attention.gqa", "moe.route", "residual.streams"}
+    plain, _ = parsed("str_small")
+    assert not plain.is_hybrid and ModelSpec.from_layered(plain).state is None          # one tap: nothing to remember
 
 
 def test_checkpoint_admission(tmp_path):
@@ -216,7 +273,137 @@ def test_sequential_packing():
     assert torch.equal(packed.lm_head.codes.float()[:, :W], w["embed"].float()) and packed.embed_norm is None
 
 
+def test_stream_packing():
+    """Sections of the projection and the convolution's columns, distance biases, the routed feed-forward's joint matrix."""
+    cfg, w = parsed("str")
+    W = cfg.hidden_size
+    p = L.pack_layer(cfg, 0, w.__getitem__)
+    rows, s = p.proj.codes.float()[:, :W], p.mixer.spec
+    for t, off in zip("qkv", s.offsets):
+        n = w[f"l0.mix.{t}"].shape[0]
+        assert off % 8 == 0 and torch.equal(rows[p.mixer.q_off + off:p.mixer.q_off + off + n], w[f"l0.mix.{t}"].float())
+        assert torch.equal(p.mixer.conv_w[:, off:off + n].t(), w[f"l0.mix.{t}.conv"].float())
+    assert torch.equal(p.out.codes.float()[:, :s.out_width], w["l0.mix.o"].float())
+    exact = torch.tensor([1000.0 ** (-i / 6) for i in range(6)], dtype=torch.float64)
+    assert torch.equal(p.mixer.freq[0].double(), exact.float().double())
+    assert (p.mixer.freq.double().sum(0) - exact).abs().max() < 1e-14
+    assert p.streams[0].read.tolist() == w["l0.hc1.in"].float().tolist() and torch.equal(p.streams[1].mix, w["l0.hc2.mix"].float())
+    assert p.gate_up.act_interleaved and p.gate_up.n == 160 and p.routed is None
+    q = L.pack_layer(cfg, 1, w.__getitem__)
+    bias, rel = q.mixer.bias, w["l1.mix.rel"].float()
+    assert bias.shape == (31, 4) and all(torch.equal(bias[n], rel[R.distance_bucket(n, 8, 30)]) for n in range(31))
+    r, head = q.routed, q.routed.head.codes.float()[:, :W]
+    assert r.split == 16 and torch.equal(head[:8], w["l1.mlp.router"].float()) and torch.equal(head[8:9], w["l1.mlp.shared.sg"].float())
+    assert torch.equal(head[16:80], w["l1.mlp.shared.up"].float()) and head.shape[0] == 80
+    assert r.up.codes.shape == (5, 48, 128) and r.down.codes.shape == (5, 96, 64) and q.gate_up is None
+    assert all(torch.equal(r.down.codes[e, :, :48].float(), w[f"l1.mlp.e{e}.down"].float()) for e in range(5))
+    last = L.pack_layer(cfg, 2, w.__getitem__)
+    assert last.norm2 is None and len(last.streams) == 1 and last.routed is None
+    packed = L.pack_weights(cfg, w.__getitem__)
+    assert torch.equal(packed.lm_head.codes.float()[:, :W], w["head"].float()) and packed.nbytes() > 0
+
+
+@pytest.mark.parametrize("rows, most", [(2, 2), (2, 50), (3, 9), (8, 30), (9, 128), (11, 70), (16, 120), (16, 128), (32, 512), (33, 100)])
+def test_distance_buckets(rows, most):
+    """The product's table and the oracle's buckets: the formula wherever floating point decides it, every row up to the last."""
+    half = rows // 2
+    spec = L.BiasedAttentionSpec(1, 1, 8, 8, 1.0, rows, most)
+    table = spec.bucket_of_distance().tolist()
+    assert table == [R.distance_bucket(n, rows, most) for n in range(most + 1)]
+    assert table[:half] == list(range(half)) and table[-1] == rows - 1 and sorted(table) == table
+    assert R.distance_bucket(most * 7, rows, most) == rows - 1
+    for n in range(half, most + 1):
+        at = np.log(n / half) / np.log(most / half) * (rows - half)
+        if abs(at - round(at)) > 1e-9:
+            assert table[n] == min(rows - 1, half + int(np.floor(at)))
+        else:
+            assert table[n] == min(rows - 1, half + round(at))                          # a border is the next row's
+
+
 # ------------------------------------------------------------------ the oracle's mechanisms, against element-wise loops
+def test_oracle_rotation_of_halves_and_kept_window():
+    x = torch.randn(4, 2, 7, dtype=torch.float64)
+    y = R.rotate_halves(x, 5, 6, 50.0)
+    for t in range(4):
+        for h in range(2):
+            for i in range(3):
+                a = (5 + t) * 50.0 ** (-2 * i / 6)
+                u, v = float(x[t, h, i]), float(x[t, h, i + 3])
+                assert abs(float(y[t, h, i]) - (u * np.cos(a) - v * np.sin(a))) < 1e-12
+                assert abs(float(y[t, h, i + 3]) - (v * np.cos(a) + u * np.sin(a))) < 1e-12
+    assert torch.equal(y[:, :, 6:], x[:, :, 6:]) and torch.equal(R.rotate_halves(x, 5, 0, 9.0), x)
+    for size, keep in ((3, 2), (1, 0), (None, 0), (4, 20)):
+        seen = R.kept_window(6, 5, 11, size, keep)
+        for i in range(5):
+            for j in range(11):
+                p = 6 + i
+                assert bool(seen[i, j]) == (j <= p and (size is None or p - j < size or j < keep))
+
+
+def test_oracle_masked_attention_with_bias():
+    q, k, v, b = torch.randn(5, 4, 3), torch.randn(5, 2, 3), torch.randn(5, 2, 6), torch.randn(4, 5, 5)
+    seen = R.kept_window(0, 5, 5, 2, 1)
+    o = R.masked_attention(q, k, v, seen, 0.8, b)
+    for i in range(5):
+        for h in range(4):
+            js = [j for j in range(5) if j <= i and (i - j < 2 or j < 1)]
+            e = [np.exp(0.8 * float(q[i, h] @ k[j, h // 2]) + float(b[h, i, j])) for j in js]
+            assert torch.allclose(o[i, h], sum(w * v[j, h // 2] for w, j in zip(e, js)) / sum(e), atol=1e-5)
+
+
+def test_oracle_routing():
+    """Choice by score plus correction, weights by score alone, ties to the first; an expert that returns the token."""
+    z, corr = torch.tensor([[1.0, 1.0, 0.0, 2.0], [0.0, 0.0, 0.0, 0.0]], dtype=torch.float64), torch.tensor([0.0, 0.0, 0.6, 0.0])
+    chosen, weight = R.route(z, corr, 2)
+    s = torch.exp(z[0]) / torch.exp(z[0]).sum()
+    assert chosen.tolist() == [[2, 3], [2, 0]]
+    assert torch.allclose(weight[0], s[[2, 3]] / s[[2, 3]].sum()) and torch.allclose(weight[1], torch.tensor([0.5, 0.5], dtype=torch.float64))
+    w = {"p.router": torch.zeros(3, 4), "p.correction": torch.tensor([0.0, 0.2, 0.1]), "p.e0.up": torch.randn(5, 4), "p.e0.down": torch.randn(4, 5),
+         "p.e1.up": torch.randn(5, 4), "p.e1.down": torch.randn(4, 5), "p.shared.up": torch.randn(3, 4), "p.shared.down": torch.randn(4, 3),
+         "p.shared.sg": torch.randn(1, 4)}
+    h = torch.randn(2, 4)
+    out = R.routed_feed_forward(w, "p", routed(2, 2, 5, 1, 3), h)
+    for t in range(2):
+        e1 = w["p.e1.down"] @ (w["p.e1.up"] @ h[t]).clamp_min(0) ** 2
+        sh = w["p.shared.down"] @ (w["p.shared.up"] @ h[t]).clamp_min(0) ** 2
+        want = 0.5 * e1 + 0.5 * h[t] + sh / (1 + torch.exp(-(w["p.shared.sg"] @ h[t])))
+        assert torch.allclose(out[t], want, atol=1e-5)
+
+
+def test_oracle_streams():
+    xs, w_in, mix, out, y = torch.randn(3, 2, 4), torch.randn(3), torch.randn(3, 3), torch.randn(3), torch.randn(2, 4)
+    assert torch.allclose(R.stream_read(xs, w_in), sum(w_in[s] * xs[s] for s in range(3)), atol=1e-6)
+    new = R.stream_write(xs, mix, out, y)
+    for t in range(3):
+        assert torch.allclose(new[t], sum(mix[s, t] * xs[s] for s in range(3)) + out[t] * y, atol=1e-6)
+
+
+@pytest.mark.parametrize("taps", [1, 2, 5])
+def test_oracle_plain_convolution(taps):
+    x, w = torch.randn(6, 3), torch.randn(3, taps)
+    y, past = R.plain_short_conv(x, w, torch.zeros(taps - 1, 3))
+    for t in range(6):
+        assert torch.allclose(y[t], sum(w[:, taps - 1 - d] * x[t - d] for d in range(taps) if t - d >= 0), atol=1e-5)
+    a, p1 = R.plain_short_conv(x[:1], w, torch.zeros(taps - 1, 3))
+    b, p2 = R.plain_short_conv(x[1:], w, p1)
+    assert torch.allclose(torch.cat([a, b]), y, atol=1e-6) and torch.equal(p2, past)
+
+
+def test_oracle_query_factor():
+    """The factor steps where the position after a token is a multiple of ``every``; a query scaled alone moves the weights."""
+    raw = streams(30, 16, [far(1, 1, 8, 8, 2.0, 4, (0.7, 3), 0, 2)], 1)
+    w = {n: t.double() for n, t in tensors(raw, 1).items()}
+    m, h = raw["layers"][0]["mixer"], torch.randn(9, 16, dtype=torch.float64)
+    got = R.biased_attention(w, "l0.mix", m, h, {}, 1e-5)
+    q, k = (R.rms(h @ w[f"l0.mix.{t}"].T, 1e-5) * w[f"l0.mix.{t}.norm"] for t in "qk")
+    v = h @ w["l0.mix.v"].T
+    for i in range(9):
+        f = 1 + 0.7 * np.log((i + 1) // 3 + 1)
+        sc = [2.0 * f * float(q[i] @ k[j]) + float(w["l0.mix.rel"][min(i - j, 1), 0]) for j in range(i + 1)]
+        e = np.exp(np.array(sc) - max(sc))
+        assert torch.allclose(got[i], w["l0.mix.o"] @ sum(a * v[j] for j, a in enumerate(e / e.sum())), atol=1e-9)
+
+
 def test_rotary_table_equals_the_oracle():
     """Frequencies of the product and of the oracle, stretched and plain; the ramp's ends, also where it has no width."""
     for raw in (*SEQUENTIAL.values(),):
@@ -481,7 +668,8 @@ def backend_of(args, tp=1):
 @pytest.mark.parametrize("raw", [
     config(300, 64, [delta(2, 1, 16, 16, 3, 64), latent(2, 16, 16, 24, 32, 20, 0.25, 0), channel(2, 2, 16, 16, 2, 48)], (0, 2, 2)),
     sequential(300, 64, [mamba2(2, 16, 8, 1, 3, 2, 48), parallel((4, 2, 16, 20, 0.3, 8, 90.0, (2.0, 50, 4.0, 1.0)), (2, 12, 16, 8.0), (0.9, 0.8), 64)], 8),
-], ids=["Bumodra", "Loduzen"])
+    streams(300, 64, [near(4, 2, 16, 24, 3, 0.5, 8, 90.0, 20, 3, routed(4, 2, 32, 1, 24)), far(2, 1, 16, 16, 0.3, 20, (0.4, 8), 48)], 2, 3.0),
+], ids=["Bumodra", "Loduzen", "Vimelorn"])
 def test_eager_mode_generates_like_the_oracle(tmp_path, raw):
     from cubic_serve_b200.runtime.scheduler import SamplingParams
     w = tensors(raw, 5)
