@@ -3,7 +3,8 @@ throughput of whole models (``bench.py --layered``).
 
 The closest model is the hybrid family (Gated DeltaNet layers with periodic full attention) with bf16 weights; its SwiGLU
 feed-forward has three matrices where a parallel layer's has two, so its width is two thirds of that: equal parameters (the
-sequential layers have the same three matrices).  Weights are random, prompts are random ids, one GPU.  Kernel times are CUDA-event times inside CUDA graphs with L2 flushed; the roofline
+sequential layers have the same three matrices).  For the layers on several residual streams it is the family of grouped-query
+decoders with routed experts: an expert there has three matrices where one here has two, so its width is two thirds.  Weights are random, prompts are random ids, one GPU.  Kernel times are CUDA-event times inside CUDA graphs with L2 flushed; the roofline
 of a kernel is the slower of its bytes over the copy bandwidth and its operations over the pipe that runs them.
 """
 from __future__ import annotations
@@ -14,8 +15,8 @@ from pathlib import Path
 import torch
 
 from ..models.config import ModelConfig, QuantSpec
-from ..models.layered import (AttentionSpec, DeltaSpec, GatedLinearSpec, LatentSpec, LayeredConfig, LayerSpec, PairSpec, RotarySpec,
-                              SsdSpec)
+from ..models.layered import (AttentionSpec, BiasedAttentionSpec, ConvAttentionSpec, DeltaSpec, GatedLinearSpec, LatentSpec,
+                              LayeredConfig, LayerSpec, PairSpec, RotarySpec, RoutedSpec, SsdSpec)
 from ..ops import kernels as K, wq_pack
 from ..utils.kernel_bench import DEV, timeit_graph
 
@@ -50,6 +51,29 @@ def sequential_config(width: int, layers: int) -> LayeredConfig:
     ssd = LayerSpec(SsdSpec(width // 32, 64, 128, 8, 4, 8), ff)
     return LayeredConfig(f"sequential-{width}", 32768, width, (ssd, pair, pair, pair) * (layers // 4), 1e-6, architecture="Loduzen",
                          side_dim=64)
+
+
+EXPERTS, TOP = 64, 4
+
+
+def streams_config(width: int, layers: int) -> LayeredConfig:
+    """Real-model layers on two residual streams at ``width``: attention heads of 128 (four per key head), three windowed layers
+    and one of every earlier token in turn, all feed-forwards routed with a shared expert."""
+    h = width // 128
+    ff = 3 * width // 8
+    routed = RoutedSpec(EXPERTS, TOP, ff, 8, ff)
+    near = LayerSpec(ConvAttentionSpec(h, max(1, h // 4), 128, 128, 4, 1.0, RotarySpec(128, 1e6), 1024, 8), routed=routed)
+    far = LayerSpec(BiasedAttentionSpec(h, max(1, h // 4), 128, 128, 128 ** -0.5, 32, 512, 0.1, 4096), routed=routed)
+    return LayeredConfig(f"streams-{width}", 32768, width, (near, near, near, far) * (layers // 4), 1e-6, architecture="Vimelorn",
+                         streams=2, embed_scale=width ** 0.5)
+
+
+def experts_config(width: int, layers: int) -> ModelConfig:
+    h = width // 128
+    return ModelConfig(name=f"experts-{width}", family="gqa_moe", num_layers=layers, hidden_size=width, num_q_heads=h,
+                       num_kv_heads=max(1, h // 4), head_dim=128, intermediate_size=width // 4, vocab_size=32768, rope_theta=1e6,
+                       qk_norm=True, num_experts=EXPERTS, experts_per_token=TOP, moe_intermediate_size=width // 4,
+                       shared_intermediate_size=width // 4, quant=QuantSpec("none", 16, 0))
 
 
 def hybrid_config(width: int, layers: int) -> ModelConfig:
@@ -209,9 +233,104 @@ def bench_sequential_rows(m: int, width: int, side: int, flush, pk) -> list[dict
             _line(f"row_norm fp32 in [{m} x {width}]", rn, m * width * 6, 0, 1, pk)]
 
 
-def _visible(tokens: int, ctx: int, window: int) -> int:
+def _visible(tokens: int, ctx: int, window: int, keep: int = 0) -> int:
     """Keys seen by the ``tokens`` last positions of a context of ``ctx`` tokens."""
-    return sum(min(p + 1, window) if window else p + 1 for p in range(ctx - tokens, ctx))
+    return sum(min(p + 1, window + keep) if window else p + 1 for p in range(ctx - tokens, ctx))
+
+
+def bench_qkv(requests: int, tokens: int, ctx: int, heads: int, kv_heads: int, flush, pk) -> list[dict]:
+    """Preparation of both attentions and the attentions themselves, beside the rotation kernel of the int8-cached decoders."""
+    d, T, per = 128, requests * tokens, -(-ctx // 16)
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    C = (heads + 2 * kv_heads) * d
+    offs = (0, heads * d, (heads + kv_heads) * d)
+    cache = torch.randn(requests * per + 1, kv_heads, 2, 16, d, **bf)
+    table = (torch.randperm(requests * per, device=DEV).to(torch.int32) + 1).view(requests, per)
+    x, q, out = torch.randn(T, C, **bf), torch.empty(T, heads * d, **bf), torch.empty(T, heads * d, **bf)
+    seg = _segments(requests, tokens, ctx - tokens)
+    pos = torch.arange(ctx - tokens, ctx, device=DEV, dtype=torch.int32).repeat(requests)
+    slots = (table.long().gather(1, (pos.view(requests, tokens) // 16).long()) * 16 + pos.view(requests, tokens) % 16).to(torch.int32).view(-1)
+    conv_w, state, freq = torch.randn(4, C, device=DEV) * 0.5, torch.zeros(requests, 3, C, **bf), torch.rand(2, 64, device=DEV)
+    freq[1] = 0
+    qn, kn, bias = torch.ones(heads * d, device=DEV), torch.ones(kv_heads * d, device=DEV), torch.randn(513, heads, device=DEV)
+    decode = tokens == 1
+    cv = timeit_graph(lambda: K.conv_qkv(x, offs, conv_w, state, freq, pos, slots, seg, q, cache, heads, d, d, 1e-6), flush, launches=5)
+    nm = timeit_graph(lambda: K.norm_qkv(x, offs, qn, kn, pos, slots, q, cache, heads, d, d, 1e-6, (0.1, 4096)), flush, launches=5)
+    near = timeit_graph(lambda: K.gqa_attention(q, cache, table, seg, out, heads, d, 1024, 0.09, decode=decode, keep=8), flush, launches=5)
+    far = timeit_graph(lambda: K.gqa_attention(q, cache, table, seg, out, heads, d, 0, 0.09, decode=decode, bias=bias), flush, launches=5)
+    blob = torch.zeros(requests * per + 1, kv_heads, K.kv_blob_bytes(d, 8, 8), dtype=torch.uint8, device=DEV)
+    q8, w = torch.empty(T, heads, d, **bf), torch.ones(d, **bf)
+    rope = timeit_graph(lambda: K.rope_kv_write(x, q8, blob, pos, slots, freq[0], heads, kv_heads, d, 8, 8, w, w), flush, launches=5)
+    shape = f"{requests} x {tokens} at {ctx}, {heads}/{kv_heads} heads"
+    io = T * 2 * C * 2
+    attn = lambda window, keep: (requests * (min(ctx, window + keep + tokens - 1) if window else ctx) * kv_heads * 2 * d * 2      # noqa: E731
+                                 + 2 * T * heads * d * 2, 4.0 * requests * _visible(tokens, ctx, window, keep) * heads * d)
+    return [_line(f"conv_qkv [{shape}]", cv, io + 2 * requests * 3 * C * 2, 0, 1, pk), _line(f"norm_qkv [{shape}]", nm, io, 0, 1, pk),
+            _line(f"rope_kv_write int8 with norms [{shape}]", rope, T * (C + heads * d) * 2 + T * 2 * kv_heads * (d + 16), 0, 1, pk),
+            _line(f"gqa_attention window 1024, 8 kept [{shape}]", near, *attn(1024, 8), pk["bf16"], pk),
+            _line(f"gqa_attention biased [{shape}]", far, *attn(0, 0), pk["bf16"], pk)]
+
+
+def bench_streams(m: int, width: int, flush, pk) -> list[dict]:
+    """A step between two sublayers on two streams, with a plain and a routed result, beside the norm that adds a residual and the
+    combination of the other routed decoders."""
+    S, top = 2, TOP
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    x, h, y, w = torch.randn(m, S, width, device=DEV), torch.randn(m, width, **bf), torch.randn(m, width, **bf), torch.ones(width, device=DEV)
+    mix, out = torch.eye(S, device=DEV), torch.full((S,), 1e-3, device=DEV)
+    rows = torch.randn(m * top, width, **bf)
+    routes = K.RoutedResult(rows, torch.randperm(m * top, device=DEV).to(torch.int32), torch.rand(m * top, device=DEV),
+                            torch.zeros(m, device=DEV), torch.randn(m, 1, device=DEV), top)
+    plain = timeit_graph(lambda: K.stream_step(x, y, mix, out, h, 1e-6, out, w), flush, launches=5)
+    full = timeit_graph(lambda: K.stream_step(x, y, mix, out, h, 1e-6, out, w, routes), flush, launches=5)
+    res, wb = torch.randn(m, width, **bf), torch.ones(width, **bf)
+    norm = timeit_graph(lambda: K.rmsnorm(y, wb, 1e-6, out=h, residual=res), flush, launches=5)
+    sc = K.MoeScratch(m, top, width, 128, EXPERTS, 32, DEV)
+    sc.route_pos.copy_(routes.pos.view(m, top))
+    sc.topk_w.copy_(routes.weight.view(m, top))
+    comb = timeit_graph(lambda: K.moe_combine(rows, sc, m, y, res), flush, launches=5)
+    row = m * width
+    return [_line(f"stream_step [{m} x {S} x {width}]", plain, row * (8 * S + 4), 0, 1, pk),
+            _line(f"stream_step routed, top {top} [{m} x {S} x {width}]", full, row * (8 * S + 4 + 2 * top), 0, 1, pk),
+            _line(f"rmsnorm + residual bf16 [{m} x {width}]", norm, row * 8, 0, 1, pk),
+            _line(f"moe_combine + residual, top {top} [{m} x {width}]", comb, row * (4 + 2 * top), 0, 1, pk)]
+
+
+def bench_experts(m: int, width: int, flush, pk) -> list[dict]:
+    """Routing and the products of all experts, beside those of the gated experts of equal size."""
+    from ..models.moe import MoeLayer, stack_experts
+    E, top, bf = EXPERTS, TOP, dict(dtype=torch.bfloat16, device=DEV)
+    ff, gf = 3 * width // 8, width // 4
+    h, z, corr = torch.randn(m, width, **bf), torch.randn(m, E, device=DEV), torch.zeros(E, device=DEV)
+    sc = K.ScoredScratch(m, top, E, width, width, torch.bfloat16, DEV)
+    stack = lambda n, k: wq_pack.PackedWeight(wq_pack.FMT_BF16, n, k, k, torch.randn(E, n, k, **bf) * 0.02, None)      # noqa: E731
+    up, down, act = stack(ff, width), stack(width, ff), torch.zeros(m * top, ff, **bf)
+    route = timeit_graph(lambda: K.scored_route(z, corr, h, width, E, top, sc), flush, launches=5)
+    mb = K.scored_route(z, corr, h, width, E, top, sc)
+    used = len(set(sc.ids[:m * top].tolist()))
+    u = timeit_graph(lambda: K.grouped_gemm(sc.xs, up, act, sc, m * top, mb, relu2=True), flush, launches=5)
+    dn = timeit_graph(lambda: K.grouped_gemm(act, down, sc.ys, sc, m * top, mb), flush, launches=5)
+    del up, down
+    gu, cs, ms = stack_experts([wq_pack.pack_bf16(torch.randn(2 * gf, width, **bf) * 0.02) for _ in range(E)])
+    dg, ds, dm = stack_experts([wq_pack.pack_bf16(torch.randn(width, gf, **bf) * 0.02) for _ in range(E)])
+    layer = MoeLayer(wq_pack.pack_bf16(torch.randn(E, width, **bf)), gu, dg, (cs, ms, ds, dm), E, top, 0, E)
+    layer.fuse_activation()
+    old = layer.ensure_scratch(m, width, torch.device(DEV))
+    zb = z.to(torch.bfloat16)
+    r2 = timeit_graph(lambda: K.moe_route(zb, h, top, old), flush, launches=5)
+    K.moe_route(zb, h, top, old)
+    g2 = timeit_graph(lambda: K.wq_gemm_grouped(old.xs, layer.gate_up, old.act, m * top, old, cs, ms, swiglu=True), flush, launches=5)
+    d2 = timeit_graph(lambda: K.wq_gemm_grouped(old.act, layer.down, old.y, m * top, old, ds, dm), flush, launches=5)
+    K.workspace(torch.device(DEV)).check_status()
+    R = m * top
+    io = lambda n, k: (used * n * k + R * (n + k)) * 2                                   # noqa: E731
+    shape = f"{m} tokens, {top} of {E}, width {width}"
+    return [_line(f"scored_route [{shape}]", route, m * E * 4 + (m + R) * width * 2, 0, 1, pk),
+            _line(f"moe_route [{shape}]", r2, m * E * 2 + (m + R) * width * 2, 0, 1, pk),
+            _line(f"grouped up relu^2 [{shape}, {ff}]", u, io(ff, width), 2.0 * R * ff * width, pk["bf16"], pk),
+            _line(f"wq_gemm_grouped gate/up bf16 [{shape}, {gf}]", g2, (used * 2 * gf * width + R * (gf + width)) * 2, 4.0 * R * gf * width, pk["bf16"], pk),
+            _line(f"grouped down [{shape}, {ff}]", dn, io(width, ff), 2.0 * R * ff * width, pk["bf16"], pk),
+            _line(f"wq_gemm_grouped down bf16 [{shape}, {gf}]", d2, io(width, gf), 2.0 * R * gf * width, pk["bf16"], pk)]
 
 
 def bench_latent(requests: int, tokens: int, ctx: int, heads: int, rank: int, window: int, flush, pk) -> list[dict]:
@@ -321,6 +440,20 @@ def sequential_kernels(width: int = 4096) -> list[dict]:
     return out
 
 
+def streams_kernels(width: int = 4096) -> list[dict]:
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=DEV)
+    pk = peaks()
+    h = width // 128
+    out = []
+    for requests, tokens, ctx in ((256, 1, 1280), (1, 1, 4096), (8, 1024, 1024), (1, 4096, 4096)):
+        out += bench_qkv(requests, tokens, ctx, h, max(1, h // 4), flush, pk)
+        out += bench_paged(requests, tokens, ctx, h, max(1, h // 4), flush, pk)
+    for m in (16, 256, 4096):
+        out += bench_streams(m, width, flush, pk)
+        out += bench_experts(m, width, flush, pk)
+    return out
+
+
 # ------------------------------------------------------------------ whole models
 def model_throughput(cfg, concurrency: int, prompt: int, steps: int, warmup: int = 4, budget: int = 8192) -> dict:
     """Prefill and decode rates of a random model through the serving engine."""
@@ -380,12 +513,18 @@ def model_throughput(cfg, concurrency: int, prompt: int, steps: int, warmup: int
     return out
 
 
+KERNELS = {"parallel": kernels, "sequential": sequential_kernels, "streams": streams_kernels}
+MODELS = {"parallel": (layered_config, hybrid_config), "sequential": (sequential_config, hybrid_config),
+          "streams": (streams_config, experts_config)}
+
+
 def run(steps: int = 32, designs: str = "all") -> None:
-    """Prints one JSON line per measurement.  ``designs``: all, or ``parallel`` / ``sequential`` layers only."""
-    both = designs == "all"
-    for line in (kernels() if both or designs == "parallel" else []) + (sequential_kernels() if both or designs == "sequential" else []):
-        print(json.dumps(line), flush=True)
-    models = [c for d, c in (("parallel", layered_config), ("sequential", sequential_config)) if both or designs == d] + [hybrid_config]
+    """Prints one JSON line per measurement.  ``designs``: all, or one of ``KERNELS``."""
+    chosen = list(KERNELS) if designs == "all" else [designs]
+    for d in chosen:
+        for line in KERNELS[d]():
+            print(json.dumps(line), flush=True)
+    models = list(dict.fromkeys(make for d in chosen for make in MODELS[d]))
     for width, layers in ((2048, 8), (4096, 8)):
         for concurrency, prompt in ((1, 4096), (16, 1024), (256, 1024)):
             for make in models:

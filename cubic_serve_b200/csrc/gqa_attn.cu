@@ -280,8 +280,9 @@ gqa_prefill_kernel(const GqaMma p) {
 
   // visible keys of the thread's two rows; rows without a query see none
   int lim_lo[2], lim_hi[2];
-  int row_pos[2], row_h[2];                            // for the bias: position and head of the two rows
-  float far[2];                                        // bias from bias_far on
+  // entries of the bias table (the one in shared memory, or the layer's): the rows' at distance 0 plus their position's, and the last
+  const int bias_step = BIAS ? (p.bias_rows ? p.hb : a.H) : 0;
+  int bias_at[2], bias_last[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int r = warp * 16 + g + 8 * i;
@@ -289,9 +290,9 @@ gqa_prefill_kernel(const GqaMma p) {
     lim_hi[i] = tok < toks && h < heads ? pos0 + tok : -1;
     lim_lo[i] = a.window > 0 ? pos0 + tok - a.window + 1 : 0;
     if constexpr (BIAS) {
-      row_pos[i] = pos0 + tok;
-      row_h[i] = h < heads ? h : 0;
-      far[i] = __ldg(a.bias + static_cast<size_t>(a.bias_far) * a.H + h0 + row_h[i]) * kLog2e;
+      const int head = (h < heads ? h : 0) + (p.bias_rows ? 0 : h0);
+      bias_at[i] = (pos0 + tok) * bias_step + head;
+      bias_last[i] = a.bias_far * bias_step + head;
     }
   }
   // of the whole warp
@@ -359,20 +360,40 @@ gqa_prefill_kernel(const GqaMma p) {
       if constexpr (BIAS) {
         if (pos0 + tok_a - (key_t + KT - 1) >= a.bias_far) {             // the same for every distance of the tile
 #pragma unroll
-          for (int j = 0; j < 8; ++j)
+          for (int i = 0; i < 2; ++i) {
+            const float far = p.bias_rows ? table[bias_last[i]] : __ldg(a.bias + bias_last[i]) * kLog2e;
 #pragma unroll
-            for (int c = 0; c < 4; ++c) sf[j][c] = fmaf(sf[j][c], sc, far[c >> 1]);
+            for (int j = 0; j < 8; ++j) {
+              sf[j][2 * i] = fmaf(sf[j][2 * i], sc, far);
+              sf[j][2 * i + 1] = fmaf(sf[j][2 * i + 1], sc, far);
+            }
+          }
+        } else if (p.bias_rows && key_t + KT - 1 <= pos0 + tok_a && pos0 + (warp * 16 + 15) / p.hb - key_t <= a.bias_far) {
+          // every distance has a row of its own: neighbouring keys are hb entries apart
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const float* row = table + bias_at[i] - (key_t + 2 * t4) * bias_step;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+              sf[j][2 * i] = fmaf(sf[j][2 * i], sc, row[0]);
+              sf[j][2 * i + 1] = fmaf(sf[j][2 * i + 1], sc, row[-bias_step]);
+              row -= 8 * bias_step;
+            }
+          }
         } else {
 #pragma unroll
-          for (int j = 0; j < 8; ++j)
+          for (int i = 0; i < 2; ++i) {
+            int at = bias_at[i] - (key_t + 2 * t4) * bias_step;          // negative for keys that are not seen yet
 #pragma unroll
-            for (int c = 0; c < 4; ++c) {
-              const int key = key_t + j * 8 + 2 * t4 + (c & 1), i = c >> 1;
-              const int n = min(max(row_pos[i] - key, 0), a.bias_far);
-              const float b = p.bias_rows ? table[n * p.hb + row_h[i]]
-                                          : __ldg(a.bias + static_cast<size_t>(n) * a.H + h0 + row_h[i]) * kLog2e;
-              sf[j][c] = fmaf(sf[j][c], sc, b);
+            for (int j = 0; j < 8; ++j) {
+              const int n0 = min(max(at, 0), bias_last[i]), n1 = min(max(at - bias_step, 0), bias_last[i]);
+              const float b0 = p.bias_rows ? table[n0] : __ldg(a.bias + n0) * kLog2e;
+              const float b1 = p.bias_rows ? table[n1] : __ldg(a.bias + n1) * kLog2e;
+              sf[j][2 * i] = fmaf(sf[j][2 * i], sc, b0);
+              sf[j][2 * i + 1] = fmaf(sf[j][2 * i + 1], sc, b1);
+              at -= 8 * bias_step;
             }
+          }
         }
       }
 #pragma unroll
@@ -668,12 +689,13 @@ gqa_merge_kernel(const GqaMma p) {
 }
 
 // ------------------------------------------------------------------ host
+// `most`: shared memory of the largest launch (0: of every launch)
 template <typename K>
-static int gqa_go(K kernel, dim3 grid, int threads, size_t smem, const GqaMma& p, bool (&configured)[64], cudaStream_t st) {
+static int gqa_go(K kernel, dim3 grid, int threads, size_t smem, const GqaMma& p, bool (&configured)[64], cudaStream_t st, size_t most = 0) {
   int dev = 0;                                        // dynamic shared memory is configured once per device
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -18;
   if (!configured[dev]) {
-    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(most ? most : smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev] = true;
   }
@@ -684,7 +706,8 @@ template <int NCH, bool BIAS>
 static int gqa_prefill(const GqaMma& p, dim3 grid, cudaStream_t st) {
   static bool configured[64] = {};
   const size_t rows = static_cast<size_t>((NCH <= 2 ? 0 : 16 * kGqaWarps) + 256) * NCH * 128;
-  return gqa_go(gqa_prefill_kernel<NCH, BIAS>, grid, 32 * kGqaWarps, rows + (BIAS ? kGqaBiasBytes : 0), p, configured, st);
+  return gqa_go(gqa_prefill_kernel<NCH, BIAS>, grid, 32 * kGqaWarps, rows + (BIAS ? static_cast<size_t>(p.bias_rows) * p.hb * 4 : 0), p, configured,
+                st, rows + (BIAS ? kGqaBiasBytes : 0));
 }
 
 template <int NCH, bool BIAS>

@@ -268,24 +268,23 @@ struct RouteScatter {
 // Every block derives the experts' first rows from the counts; block 0 writes the work list.  A warp copies a route's row.
 __global__ void __launch_bounds__(256)
 route_scatter_kernel(const RouteScatter p) {
-  __shared__ int rows[256], items[256];
+  __shared__ int rows[256], sums[2][8];
   __shared__ int last;
   pdl_wait();
   pdl_launch_dependents();
   const int e = threadIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int cnt = e < p.experts ? p.counts[e] : 0, nt = (cnt + p.mb - 1) / p.mb;
-  rows[e] = cnt;
-  items[e] = nt;
-  __syncthreads();
-  for (int o = 1; o < p.experts; o <<= 1) {
-    const int a = e >= o ? rows[e - o] : 0, b = e >= o ? items[e - o] : 0;
-    __syncthreads();
-    rows[e] += a;
-    items[e] += b;
-    __syncthreads();
+  int first = cnt, t0 = nt;                                              // sums up to here, then without this one
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int a = __shfl_up_sync(0xffffffffu, first, o), b = __shfl_up_sync(0xffffffffu, t0, o);
+    if (lane >= o) { first += a; t0 += b; }
   }
-  const int first = rows[e] - cnt, t0 = items[e] - nt;
+  if (lane == 31) { sums[0][warp] = first; sums[1][warp] = t0; }
   __syncthreads();
+  for (int w = 0; w < warp; ++w) { first += sums[0][w]; t0 += sums[1][w]; }
+  first -= cnt;
+  t0 -= nt;
   rows[e] = first;
   if (blockIdx.x == 0) {
     for (int i = 0; i < nt; ++i) {

@@ -23,17 +23,28 @@ __device__ __forceinline__ float4 load_four(const float* p, int c, int d, bool v
   if (vec) return c < d ? *reinterpret_cast<const float4*>(p + c) : make_float4(0.f, 0.f, 0.f, 0.f);
   return make_float4(c < d ? p[c] : 0.f, c + 1 < d ? p[c + 1] : 0.f, c + 2 < d ? p[c + 2] : 0.f, c + 3 < d ? p[c + 3] : 0.f);
 }
-__device__ __forceinline__ float4 load_four(const __nv_bfloat16* p, int c, int d, bool vec) {
+// ... of an activation row as they are stored, and as numbers
+__device__ __forceinline__ float4 load_raw(const float* p, int c, int d, bool vec) { return load_four(p, c, d, vec); }
+__device__ __forceinline__ uint2 load_raw(const __nv_bfloat16* p, int c, int d, bool vec) {
+  uint2 u = make_uint2(0u, 0u);
   if (vec) {
-    uint2 u = make_uint2(0u, 0u);
     if (c < d) u = *reinterpret_cast<const uint2*>(p + c);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-    return make_float4(a.x, a.y, b.x, b.y);
+  } else {
+    u.x = pack_bf16x2(c < d ? to_f(p[c]) : 0.f, c + 1 < d ? to_f(p[c + 1]) : 0.f);
+    u.y = pack_bf16x2(c + 2 < d ? to_f(p[c + 2]) : 0.f, c + 3 < d ? to_f(p[c + 3]) : 0.f);
   }
-  return make_float4(c < d ? to_f(p[c]) : 0.f, c + 1 < d ? to_f(p[c + 1]) : 0.f, c + 2 < d ? to_f(p[c + 2]) : 0.f,
-                     c + 3 < d ? to_f(p[c + 3]) : 0.f);
+  return u;
 }
+__device__ __forceinline__ float4 unpack_four(float4 v) { return v; }
+__device__ __forceinline__ float4 unpack_four(uint2 u) {
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename T> struct RawFour;
+template <> struct RawFour<float> { using type = float4; };
+template <> struct RawFour<__nv_bfloat16> { using type = uint2; };
+__device__ __forceinline__ float4 load_four(const __nv_bfloat16* p, int c, int d, bool vec) { return unpack_four(load_raw(p, c, d, vec)); }
 __device__ __forceinline__ void store_four(float* p, int c, float4 v) { *reinterpret_cast<float4*>(p + c) = v; }
 __device__ __forceinline__ void store_four(__nv_bfloat16* p, int c, float4 v) {
   *reinterpret_cast<uint2*>(p + c) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
@@ -80,161 +91,221 @@ struct ConvQkv {
 };
 
 // A block takes a tile of tokens of one segment and the heads blockIdx.y, + gridDim.y, ... by warps.  TAPS: 0 any number.  NJ: 128-channel
-// chunks of a head.
-template <typename T, int TAPS, int NJ>
-__global__ void __launch_bounds__(32 * kQkvWarps)
+// chunks of a head.  BATCH: tokens a warp has in flight (1: steps of one token per segment).
+template <typename T, int TAPS, int NJ, int BATCH>
+__global__ void __launch_bounds__(32 * kQkvWarps, NJ == 1 && BATCH > 1 ? 5 : 1)
 conv_qkv_kernel(const ConvQkv<T> p) {
-  constexpr int R = TAPS > 0 ? TAPS : 1, BATCH = NJ == 1 ? 4 : 2;
-  extern __shared__ __align__(16) float2 turn[];                       // [tokens][pairs] cosine and sine, then the warps' rows
+  constexpr int R = TAPS > 0 ? TAPS : 1, ROW = 128 * NJ, TOKS = BATCH == 1 ? 1 : kQkvTokens;
+  using Raw = typename RawFour<T>::type;
+  extern __shared__ __align__(16) float lsm[];                         // cosines and sines [tokens][half], then the warps' rows
+  __shared__ long long place[TOKS];                                    // first element of a token's first key in the cache, -1: none
   pdl_wait();
   pdl_launch_dependents();
   int s, off;
   if (!find_tile(p.sg, kQkvTokens, blockIdx.x, s, off)) return;
   const QkvPrep<T>& a = p.a;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int count = p.sg.count[s], toks = min(kQkvTokens, count - off);
+  const int count = p.sg.count[s], toks = BATCH == 1 ? 1 : min(kQkvTokens, count - off);
   const size_t row0 = p.sg.row0[s];                                    // first row of the segment
   const bool fresh = p.sg.pos0[s] == 0;
   const int hist_rows = p.taps - 1;
   T* st = p.state + static_cast<size_t>(p.sg.slot[s]) * hist_rows * p.ldw;
-  const int half = p.pairs, dims = 2 * half;
+  const int half = p.pairs, dims = 2 * half, hp = (half + 3) & ~3;     // hp: a token's cosines start at multiples of 16 bytes
+  float* cosine = lsm;
+  float* sine = lsm + TOKS * hp;
   for (int i = threadIdx.x; i < toks * half; i += 32 * kQkvWarps) {
-    const int t = i / half, j = i - t * half;
+    const int t = BATCH == 1 ? 0 : i / half, j = i - t * half;
     // the rounding error of the product is put back: angles of far positions keep their fraction of a turn
     const float pos = static_cast<float>(p.positions[row0 + off + t]), f = p.freq[j];
     const float ang = pos * f, e = fmaf(pos, f, -ang) + pos * p.freq[half + j];
     float sn, cs;
     sincosf(ang, &sn, &cs);
     const float ce = fmaf(-0.5f * e, e, 1.f), se = e * fmaf(e * (-1.f / 6.f), e, 1.f);
-    turn[i] = make_float2(cs * ce - sn * se, fmaf(sn, ce, cs * se));
+    cosine[t * hp + j] = cs * ce - sn * se;
+    sine[t * hp + j] = fmaf(sn, ce, cs * se);
+  }
+  if (static_cast<int>(threadIdx.x) < toks) {
+    const int slot = a.slots[row0 + off + threadIdx.x];
+    place[threadIdx.x] = slot < 0 ? -1 : (static_cast<long long>(slot / kQkvPage) * a.G * 2 * kQkvPage + slot % kQkvPage) * a.P;
   }
   __syncthreads();
-  float* swap = reinterpret_cast<float*>(turn + kQkvTokens * half + (half * kQkvTokens & 1)) + warp * 256;
+  float* swap = lsm + 2 * TOKS * hp + warp * BATCH * ROW;
   const bool vec = a.vec, vec_turn = (half & 3) == 0;
   for (int it = blockIdx.y * kQkvWarps + warp; it < a.H + 2 * a.G; it += kQkvWarps * gridDim.y) {
     const int d = a.width(it), col = a.col(it), wc = col - a.q_off;
-    const bool value = it >= a.H + a.G;
+    const bool query = it < a.H, value = it >= a.H + a.G;
     const T* xr = a.x + row0 * a.ldx + col;
+    const float inv_d = 1.f / static_cast<float>(d);
+    // where token t's row goes, by its entry of `place`
+    T* const dst0 = query ? a.q + ((row0 + off) * a.H + it) * a.P
+                          : a.cache + static_cast<size_t>(2 * (it - a.H - (value ? a.G : 0)) + value) * kQkvPage * a.P;
     // input at token t of the segment (t >= -(taps - 1)), channels of chunk j
+    auto raw = [&](int t, int j) { return load_raw(xr + static_cast<size_t>(t) * a.ldx, 4 * lane + 128 * j, d, vec); };
     auto input = [&](int t, int j) {
-      const int c = 4 * lane + 128 * j;
-      if (t >= 0) return load_four(xr + static_cast<size_t>(t) * a.ldx, c, d, vec);
+      if (t >= 0) return unpack_four(raw(t, j));
       if (fresh) return make_float4(0.f, 0.f, 0.f, 0.f);
-      return load_four(st + static_cast<size_t>(t + hist_rows) * p.ldw + wc, c, d, vec);
+      return load_four(st + static_cast<size_t>(t + hist_rows) * p.ldw + wc, 4 * lane + 128 * j, d, vec);
     };
     auto tap = [&](int k, int j) { return load_four(p.w + static_cast<size_t>(k) * p.ldw + wc, 4 * lane + 128 * j, d, vec); };
     float4 w[R][NJ], hist[R][NJ];
+    Raw next[BATCH][NJ];                                               // the inputs of the tokens that come next
     if constexpr (TAPS > 0) {
-#pragma unroll
-      for (int k = 0; k < TAPS; ++k)
-#pragma unroll
-        for (int j = 0; j < NJ; ++j) w[k][j] = tap(k, j);
 #pragma unroll
       for (int k = 0; k < TAPS - 1; ++k)
 #pragma unroll
         for (int j = 0; j < NJ; ++j) hist[k][j] = input(off + k - (TAPS - 1), j);
+#pragma unroll
+      for (int b = 0; b < BATCH; ++b)
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) next[b][j] = raw(off + min(b, toks - 1), j);
+#pragma unroll
+      for (int k = 0; k < TAPS; ++k)
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) w[k][j] = tap(k, j);
     }
-    for (int t0 = 0; t0 < toks; t0 += BATCH) {
-      float4 in[BATCH][NJ];
+    // tokens t0 .. + BATCH - 1 of the tile; FULL: all of them exist
+    auto batch = [&](int t0, auto full) {
+      constexpr bool FULL = decltype(full)::value;
+      float4 v[BATCH][NJ];
       if constexpr (TAPS > 0) {
 #pragma unroll
-        for (int b = 0; b < BATCH; ++b)                                // several tokens in flight; nothing behind the tile
-#pragma unroll
-          for (int j = 0; j < NJ; ++j)
-            in[b][j] = t0 + b < toks ? input(off + t0 + b, j) : make_float4(0.f, 0.f, 0.f, 0.f);
-      }
-#pragma unroll
-      for (int b = 0; b < BATCH; ++b) {
-        const int t = t0 + b;
-        if (t >= toks) break;
-        float4 v[NJ];
-        if constexpr (TAPS > 0) {
+        for (int b = 0; b < BATCH; ++b) {
 #pragma unroll
           for (int j = 0; j < NJ; ++j) {
+            const float4 in = unpack_four(next[b][j]);
             float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
             for (int k = 0; k < TAPS - 1; ++k) acc = fma_four(w[k][j], hist[k][j], acc);
-            v[j] = fma_four(w[TAPS - 1][j], in[b][j], acc);
+            v[b][j] = fma_four(w[TAPS - 1][j], in, acc);
+            if (FULL || t0 + b < toks) {
 #pragma unroll
-            for (int k = 0; k + 1 < TAPS - 1; ++k) hist[k][j] = hist[k + 1][j];
-            if constexpr (TAPS > 1) hist[TAPS - 2][j] = in[b][j];
-          }
-        } else {
-#pragma unroll
-          for (int j = 0; j < NJ; ++j) {
-            v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 1
-            for (int k = 0; k < p.taps; ++k) v[j] = fma_four(tap(k, j), input(off + t - hist_rows + k, j), v[j]);
+              for (int k = 0; k + 1 < TAPS - 1; ++k) hist[k][j] = hist[k + 1][j];
+              if constexpr (TAPS > 1) hist[TAPS - 2][j] = in;
+            }
           }
         }
-        if (!value) {
-          if (half) {
-            __syncwarp();                                              // the row before this one was read
+        if (t0 + BATCH < toks) {                                       // nothing behind the tile
 #pragma unroll
-            for (int j = 0; j < NJ; ++j) store_four(swap, 4 * lane + 128 * j, v[j]);
-            __syncwarp();
-            const float2* tr = turn + t * half;
+          for (int b = 0; b < BATCH; ++b)
 #pragma unroll
-            for (int j = 0; j < NJ; ++j) {
-              const int c = 4 * lane + 128 * j;
-              if (c >= dims) continue;
-              if (vec_turn) {                                          // four channels turn with four neighbours
-                const bool hi = c >= half;
-                const float4 o = *reinterpret_cast<const float4*>(swap + (hi ? c - half : c + half));
-                const float4 r0 = *reinterpret_cast<const float4*>(tr + (hi ? c - half : c));
-                const float4 r1 = *reinterpret_cast<const float4*>(tr + (hi ? c - half : c) + 2);
-                const float sg = hi ? 1.f : -1.f;
-                v[j] = make_float4(fmaf(v[j].x, r0.x, sg * o.x * r0.y), fmaf(v[j].y, r0.z, sg * o.y * r0.w),
-                                   fmaf(v[j].z, r1.x, sg * o.z * r1.y), fmaf(v[j].w, r1.z, sg * o.w * r1.w));
-              } else {
-                float* vp = &v[j].x;
+            for (int j = 0; j < NJ; ++j) next[b][j] = raw(off + min(t0 + BATCH + b, toks - 1), j);
+        }
+      } else {
+#pragma unroll
+        for (int b = 0; b < BATCH; ++b)
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) {
+            v[b][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (!FULL && t0 + b >= toks) continue;
+#pragma unroll 1
+            for (int k = 0; k < p.taps; ++k) v[b][j] = fma_four(tap(k, j), input(off + t0 + b - hist_rows + k, j), v[b][j]);
+          }
+      }
+      if (!value) {
+        if (half) {
+          __syncwarp();                                                // the rows before these were read
+#pragma unroll
+          for (int b = 0; b < BATCH; ++b)
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) store_four(swap, b * ROW + 4 * lane + 128 * j, v[b][j]);
+          __syncwarp();
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) {
+            const int c = 4 * lane + 128 * j;
+            if (c >= dims) continue;
+            if (vec_turn) {                                            // four channels turn with four neighbours
+              const bool hi = c >= half;
+              const float sg = hi ? 1.f : -1.f;
+              const int other = hi ? c - half : c + half, low = hi ? c - half : c;
+#pragma unroll
+              for (int b = 0; b < BATCH; ++b) {
+                const int at = (FULL || t0 + b < toks ? t0 + b : 0) * hp + low;
+                const float4 o = *reinterpret_cast<const float4*>(swap + b * ROW + other);
+                const float4 cs = *reinterpret_cast<const float4*>(cosine + at), sn = *reinterpret_cast<const float4*>(sine + at);
+                float4& u = v[b][j];
+                u = make_float4(fmaf(u.x, cs.x, sg * o.x * sn.x), fmaf(u.y, cs.y, sg * o.y * sn.y), fmaf(u.z, cs.z, sg * o.z * sn.z),
+                                fmaf(u.w, cs.w, sg * o.w * sn.w));
+              }
+            } else {
+#pragma unroll
+              for (int b = 0; b < BATCH; ++b) {
+                const int at = (FULL || t0 + b < toks ? t0 + b : 0) * hp;
+                float* vp = &v[b][j].x;
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                   const int ch = c + i;
                   if (ch >= dims) continue;
                   const bool hi = ch >= half;
-                  const float2 r = tr[hi ? ch - half : ch];
-                  const float o = swap[hi ? ch - half : ch + half];
-                  vp[i] = fmaf(vp[i], r.x, (hi ? o : -o) * r.y);
+                  const int low = hi ? ch - half : ch;
+                  const float o = swap[b * ROW + (hi ? low : ch + half)];
+                  vp[i] = fmaf(vp[i], cosine[at + low], (hi ? o : -o) * sine[at + low]);
                 }
               }
             }
           }
-          float ss = 0.f;
-#pragma unroll
-          for (int j = 0; j < NJ; ++j) ss += dot_four(v[j], v[j]);
-          const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(d) + a.eps);
-#pragma unroll
-          for (int j = 0; j < NJ; ++j) v[j] = mul_four(v[j], inv);
         }
-        const size_t tok = row0 + off + t;
-        T* dst = a.row(it, tok, a.slots[tok]);
-        if (!dst) continue;
+        float ss[BATCH];
+#pragma unroll
+        for (int b = 0; b < BATCH; ++b) {
+          ss[b] = 0.f;
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) ss[b] += dot_four(v[b][j], v[b][j]);
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+          for (int b = 0; b < BATCH; ++b) ss[b] += __shfl_xor_sync(0xffffffffu, ss[b], o);
+#pragma unroll
+        for (int b = 0; b < BATCH; ++b) {
+          const float inv = rsqrtf(fmaf(ss[b], inv_d, a.eps));
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) v[b][j] = mul_four(v[b][j], inv);
+        }
+      }
+#pragma unroll
+      for (int b = 0; b < BATCH; ++b) {
+        if (!FULL && t0 + b >= toks) continue;
+        const long long at = query ? static_cast<long long>(t0 + b) * a.H * a.P : place[t0 + b];
+        if (at < 0) continue;
 #pragma unroll
         for (int j = 0; j < NJ; ++j)
-          if (4 * lane + 128 * j < a.P) store_four(dst, 4 * lane + 128 * j, v[j]);
+          if (4 * lane + 128 * j < a.P) store_four(dst0 + at, 4 * lane + 128 * j, v[b][j]);
       }
+    };
+#pragma unroll 1
+    for (int t0 = 0; t0 < toks; t0 += BATCH) {
+      if (t0 + BATCH <= toks) batch(t0, std::true_type{});
+      else batch(t0, std::false_type{});
     }
     // The last inputs become the state: by the tile with the segment's first tokens, the only reader of the old one.  A lane reads
-    // and writes its own channels; entry k takes entry k + count, which is read before it is written.
+    // and writes its own channels.  They are in the registers when the tile has the segment's last tokens too; else entry k takes
+    // entry k + count, which is read before it is written.
     if (off == 0) {
-#pragma unroll 1
-      for (int k = 0; k < hist_rows; ++k)
-#pragma unroll
-        for (int j = 0; j < NJ; ++j) {
-          const int c = 4 * lane + 128 * j;
-          if (c >= d) continue;
-          const float4 n = input(count - hist_rows + k, j);
-          T* dst = st + static_cast<size_t>(k) * p.ldw + wc;
-          if (vec) {
-            store_four(dst, c, n);
-          } else {
-            dst[c] = from_f<T>(n.x);
-            if (c + 1 < d) dst[c + 1] = from_f<T>(n.y);
-            if (c + 2 < d) dst[c + 2] = from_f<T>(n.z);
-            if (c + 3 < d) dst[c + 3] = from_f<T>(n.w);
-          }
+      auto save = [&](int k, int j, float4 n) {
+        const int c = 4 * lane + 128 * j;
+        if (c >= d) return;
+        T* dst = st + static_cast<size_t>(k) * p.ldw + wc;
+        if (vec) {
+          store_four(dst, c, n);
+        } else {
+          dst[c] = from_f<T>(n.x);
+          if (c + 1 < d) dst[c + 1] = from_f<T>(n.y);
+          if (c + 2 < d) dst[c + 2] = from_f<T>(n.z);
+          if (c + 3 < d) dst[c + 3] = from_f<T>(n.w);
         }
+      };
+      if (TAPS > 0 && toks == count) {
+#pragma unroll
+        for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) save(k, j, hist[k][j]);
+      } else {
+#pragma unroll 1
+        for (int k = 0; k < hist_rows; ++k)
+#pragma unroll
+          for (int j = 0; j < NJ; ++j)
+            if (4 * lane + 128 * j < d) save(k, j, input(count - hist_rows + k, j));
+      }
     }
   }
 }
@@ -360,10 +431,12 @@ int cb_conv_qkv(const CbConvQkv* c, const CbSegments* seg, void* stream) {
   if (c->taps < 1 || c->taps - 1 > kQkvTokens || c->pairs < 0 || 2 * c->pairs > c->a.d) return -12;
   if (c->ldw < c->a.v_off - c->a.q_off + c->a.G * c->a.e || (c->taps > 1 && !c->state) || !c->w || (c->pairs && !c->freq)) return -13;
   const int tiles = max_tiles(c->a.tokens, seg->num, kQkvTokens), items = c->a.H + 2 * c->a.G;
-  // enough warps for the device: at most one head each
+  // a head per warp where the tiles alone do not fill the device; the cosines are made once per block
   const int groups = (items + kQkvWarps - 1) / kQkvWarps;
-  const int ny = min(groups, max(1, 148 * 12 / tiles));
-  const size_t smem = (static_cast<size_t>(kQkvTokens) * c->pairs + 1) * 8 + kQkvWarps * 256 * 4;
+  const bool one = c->a.P <= 128, single = c->a.tokens == seg->num;
+  const int ny = min(groups, max(1, 148 * 24 / tiles));
+  const int batch = c->taps > 4 ? 2 : single ? 1 : one ? 4 : 2, row = one && c->taps <= 4 ? 128 : 256;
+  const size_t smem = (static_cast<size_t>(batch == 1 ? 1 : kQkvTokens) * 2 * ((c->pairs + 3) & ~3) + static_cast<size_t>(kQkvWarps) * batch * row) * 4;
   auto go = [&](auto kernel, auto p) {
     using T = std::remove_pointer_t<decltype(p.a.q)>;
     p.a = qkv_fill<T>(c->a);
@@ -377,14 +450,13 @@ int cb_conv_qkv(const CbConvQkv* c, const CbSegments* seg, void* stream) {
   };
   auto pick = [&](auto p) {
     using T = std::remove_pointer_t<decltype(p.a.q)>;
-    const bool one = c->a.P <= 128;
-    switch (c->taps) {
-      case 1: return one ? go(conv_qkv_kernel<T, 1, 1>, p) : go(conv_qkv_kernel<T, 1, 2>, p);
-      case 2: return one ? go(conv_qkv_kernel<T, 2, 1>, p) : go(conv_qkv_kernel<T, 2, 2>, p);
-      case 3: return one ? go(conv_qkv_kernel<T, 3, 1>, p) : go(conv_qkv_kernel<T, 3, 2>, p);
-      case 4: return one ? go(conv_qkv_kernel<T, 4, 1>, p) : go(conv_qkv_kernel<T, 4, 2>, p);
-    }
-    return go(conv_qkv_kernel<T, 0, 2>, p);
+#define CB_TAPS(N)                                                                                            \
+  case N:                                                                                                     \
+    if (single) return one ? go(conv_qkv_kernel<T, N, 1, 1>, p) : go(conv_qkv_kernel<T, N, 2, 1>, p);         \
+    return one ? go(conv_qkv_kernel<T, N, 1, 4>, p) : go(conv_qkv_kernel<T, N, 2, 2>, p);
+    switch (c->taps) { CB_TAPS(1) CB_TAPS(2) CB_TAPS(3) CB_TAPS(4) }
+#undef CB_TAPS
+    return go(conv_qkv_kernel<T, 0, 2, 2>, p);
   };
   return c->a.f32 ? pick(ConvQkv<float>{}) : pick(ConvQkv<__nv_bfloat16>{});
 }
