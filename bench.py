@@ -59,7 +59,8 @@ def parse_args():
                     help="forced per-depth acceptance probability of speculative rounds (random weights never agree)")
     ap.add_argument("--layered", nargs="?", const="all", choices=("all", "parallel", "sequential", "streams"), default=None,
                     help="instead of the headline workload: the layered decoders (with parallel layers, sequential layers, "
-                         "residual streams, or all) beside the closest existing model at equal size, one JSON line per kernel and per model (one GPU)")
+                         "residual streams, or all) beside the closest existing model at equal size, one JSON line per kernel "
+                         "and per model (one GPU)")
     return ap.parse_args()
 
 

@@ -4,8 +4,10 @@ throughput of whole models (``bench.py --layered``).
 The closest model is the hybrid family (Gated DeltaNet layers with periodic full attention) with bf16 weights; its SwiGLU
 feed-forward has three matrices where a parallel layer's has two, so its width is two thirds of that: equal parameters (the
 sequential layers have the same three matrices).  For the layers on several residual streams it is the family of grouped-query
-decoders with routed experts: an expert there has three matrices where one here has two, so its width is two thirds.  Weights are random, prompts are random ids, one GPU.  Kernel times are CUDA-event times inside CUDA graphs with L2 flushed; the roofline
-of a kernel is the slower of its bytes over the copy bandwidth and its operations over the pipe that runs them.
+decoders with routed experts: an expert there has three matrices where one here has two, so its width is two thirds.
+
+Weights are random, prompts are random ids, one GPU.  Kernel times are CUDA-event times inside CUDA graphs with L2 flushed; the
+roofline of a kernel is the slower of its bytes over the copy bandwidth and its operations over the pipe that runs them.
 """
 from __future__ import annotations
 
@@ -328,7 +330,8 @@ def bench_experts(m: int, width: int, flush, pk) -> list[dict]:
     return [_line(f"scored_route [{shape}]", route, m * E * 4 + (m + R) * width * 2, 0, 1, pk),
             _line(f"moe_route [{shape}]", r2, m * E * 2 + (m + R) * width * 2, 0, 1, pk),
             _line(f"grouped up relu^2 [{shape}, {ff}]", u, io(ff, width), 2.0 * R * ff * width, pk["bf16"], pk),
-            _line(f"wq_gemm_grouped gate/up bf16 [{shape}, {gf}]", g2, (used * 2 * gf * width + R * (gf + width)) * 2, 4.0 * R * gf * width, pk["bf16"], pk),
+            _line(f"wq_gemm_grouped gate/up bf16 [{shape}, {gf}]", g2, (used * 2 * gf * width + R * (gf + width)) * 2,
+                  4.0 * R * gf * width, pk["bf16"], pk),
             _line(f"grouped down [{shape}, {ff}]", dn, io(width, ff), 2.0 * R * ff * width, pk["bf16"], pk),
             _line(f"wq_gemm_grouped down bf16 [{shape}, {gf}]", d2, io(width, gf), 2.0 * R * gf * width, pk["bf16"], pk)]
 

@@ -436,7 +436,8 @@ int cb_conv_qkv(const CbConvQkv* c, const CbSegments* seg, void* stream) {
   const bool one = c->a.P <= 128, single = c->a.tokens == seg->num;
   const int ny = min(groups, max(1, 148 * 24 / tiles));
   const int batch = c->taps > 4 ? 2 : single ? 1 : one ? 4 : 2, row = one && c->taps <= 4 ? 128 : 256;
-  const size_t smem = (static_cast<size_t>(batch == 1 ? 1 : kQkvTokens) * 2 * ((c->pairs + 3) & ~3) + static_cast<size_t>(kQkvWarps) * batch * row) * 4;
+  const size_t turns = static_cast<size_t>(batch == 1 ? 1 : kQkvTokens) * 2 * ((c->pairs + 3) & ~3);
+  const size_t smem = (turns + static_cast<size_t>(kQkvWarps) * batch * row) * 4;
   auto go = [&](auto kernel, auto p) {
     using T = std::remove_pointer_t<decltype(p.a.q)>;
     p.a = qkv_fill<T>(c->a);

@@ -1329,8 +1329,8 @@ def streams_moe_config() -> LayeredConfig:
     return LayeredConfig("layered-streams-moe", 151936, 4096, group * 8, 1e-6, architecture="Vimelorn", streams=2, embed_scale=64.0)
 
 
-NAMED = {"layered-streams-tiny": tiny_streams_config, "layered-streams-moe": streams_moe_config, "layered-tiny": tiny_layered_config, "layered-8b": layered_8b_config, "layered-seq-tiny": tiny_sequential_config,
-         "layered-seq-8b": sequential_8b_config}
+NAMED = {"layered-tiny": tiny_layered_config, "layered-8b": layered_8b_config, "layered-seq-tiny": tiny_sequential_config,
+         "layered-seq-8b": sequential_8b_config, "layered-streams-tiny": tiny_streams_config, "layered-streams-moe": streams_moe_config}
 
 
 def with_dtype(cfg: LayeredConfig, dtype: str) -> LayeredConfig:

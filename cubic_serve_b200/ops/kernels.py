@@ -1073,7 +1073,8 @@ def gqa_attention(q: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor
             partial = ws.attn.data_ptr()
     a = native.GqaAttnStruct(q.data_ptr(), out.data_ptr(), out.stride(0), cache.data_ptr(), page_table.data_ptr(),
                              page_table.shape[1], heads, G, dim, P, window, keep, float(scale), float(out_scale),
-                             float("-inf") if sink is None else float(sink), _ptr(bias), 0 if bias is None else bias.shape[0] - 1, T, int(f32), int(decode), splits, partial)
+                             float("-inf") if sink is None else float(sink), _ptr(bias), 0 if bias is None else bias.shape[0] - 1, T,
+                             int(f32), int(decode), splits, partial)
     st = _seg(seg)
     native.check(l.cb_gqa_attn(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_gqa_attn")
     return 2 if splits > 1 else 1
