@@ -93,18 +93,18 @@ struct ConvQkv {
 // A block takes a tile of tokens of one segment and the heads blockIdx.y, + gridDim.y, ... by warps.  TAPS: 0 any number.  NJ: 128-channel
 // chunks of a head.  BATCH: tokens a warp has in flight (1: steps of one token per segment).
 template <typename T, int TAPS, int NJ, int BATCH>
-__global__ void __launch_bounds__(32 * kQkvWarps, NJ == 1 && BATCH > 1 ? 5 : 1)
+__global__ void __launch_bounds__(32 * kQkvWarps, NJ > 1 ? 1 : BATCH > 1 ? 5 : 8)
 conv_qkv_kernel(const ConvQkv<T> p) {
   constexpr int R = TAPS > 0 ? TAPS : 1, ROW = 128 * NJ, TOKS = BATCH == 1 ? 1 : kQkvTokens;
   using Raw = typename RawFour<T>::type;
   extern __shared__ __align__(16) float lsm[];                         // cosines and sines [tokens][half], then the warps' rows
   __shared__ long long place[TOKS];                                    // first element of a token's first key in the cache, -1: none
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_wait();
   pdl_launch_dependents();
   int s, off;
   if (!find_tile(p.sg, kQkvTokens, blockIdx.x, s, off)) return;
   const QkvPrep<T>& a = p.a;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int count = p.sg.count[s], toks = BATCH == 1 ? 1 : min(kQkvTokens, count - off);
   const size_t row0 = p.sg.row0[s];                                    // first row of the segment
   const bool fresh = p.sg.pos0[s] == 0;
@@ -272,10 +272,14 @@ conv_qkv_kernel(const ConvQkv<T> p) {
           if (4 * lane + 128 * j < a.P) store_four(dst0 + at, 4 * lane + 128 * j, v[b][j]);
       }
     };
+    if constexpr (BATCH == 1) {
+      batch(0, std::true_type{});
+    } else {
 #pragma unroll 1
-    for (int t0 = 0; t0 < toks; t0 += BATCH) {
-      if (t0 + BATCH <= toks) batch(t0, std::true_type{});
-      else batch(t0, std::false_type{});
+      for (int t0 = 0; t0 < toks; t0 += BATCH) {
+        if (t0 + BATCH <= toks) batch(t0, std::true_type{});
+        else batch(t0, std::false_type{});
+      }
     }
     // The last inputs become the state: by the tile with the segment's first tokens, the only reader of the old one.  A lane reads
     // and writes its own channels.  They are in the registers when the tile has the segment's last tokens too; else entry k takes
