@@ -1,4 +1,4 @@
-"""Plain model of the layered decoders (``Bumodra``, ``Loduzen`` and ``Vimelorn`` checkpoints): the oracle of the native runner and the
+"""Plain model of the layered decoders (``Bumodra``, ``Loduzen``, ``Vimelorn`` and ``Fovunex`` checkpoints): the oracle of the native runner and the
 model of the eager execution mode.
 
 Everything is written from the equations, token by token where the mechanism is a recurrence, one function per
@@ -399,6 +399,78 @@ def silu_feed_forward(w, p: str, h) -> torch.Tensor:
     return (silu(h @ w[f"{p}.gate"].T) * (h @ w[f"{p}.up"].T)) @ w[f"{p}.down"].T
 
 
+def sigmoid(x: torch.Tensor) -> torch.Tensor:
+    return 1.0 / (1.0 + torch.exp(-x))
+
+
+def same_chunk(first: int, n: int, m: int, size: int | None) -> torch.Tensor:
+    """[n, m] which of m keys the queries at positions ``first ..`` see: the earlier ones of their own chunk of ``size`` positions."""
+    i, j = torch.arange(first, first + n).unsqueeze(1), torch.arange(m).unsqueeze(0)
+    seen = j <= i
+    return seen if size is None else seen & (torch.div(i, size, rounding_mode="floor") == torch.div(j, size, rounding_mode="floor"))
+
+
+def rotated_latent_attention(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    """Latent attention whose scores have two parts: per head from the latent, and rotated from a key all heads share."""
+    H, d, r, e, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    n = h.shape[0]
+    q = (h @ w[f"{p}.q"].T).view(n, H, d + r)
+    down = h @ w[f"{p}.dkv"].T
+    first = st["c"].shape[0] if st else 0
+    freq, mult = rotary_frequencies(m["rot"])
+    c = rms(down[:, :R], eps) * w[f"{p}.dkv.norm"]
+    shared = rotate_pairs(down[:, R:].unsqueeze(1), first, freq, mult)[:, 0]
+    turned = rotate_pairs(q[..., d:], first, freq, mult)
+    st["c"] = torch.cat([st["c"], c]) if st else c
+    st["r"] = torch.cat([st["r"], shared]) if "r" in st else shared
+    k = (st["c"] @ w[f"{p}.uk"].T).view(-1, H, d)
+    v = (st["c"] @ w[f"{p}.uv"].T).view(-1, H, e)
+    k = torch.cat([k, st["r"].unsqueeze(1).expand(-1, H, r)], -1)
+    o = masked_attention(torch.cat([q[..., :d], turned], -1), k, v, same_chunk(first, n, first + n, None), m["scale"])
+    return o.reshape(n, H * e) @ w[f"{p}.o"].T
+
+
+def differential_attention(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    """Two attention maps per head over the same values, the second subtracted with a learned factor; heads normed and gated."""
+    H, G, d, e = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    n = h.shape[0]
+    first = st["k"].shape[0] if st else 0
+    rot = m["rot"]
+    q, k = (rms((h @ w[f"{p}.{t}"].T).view(n, -1, d), eps) * w[f"{p}.{t}.norm"] for t in "qk")
+    q, k = (rotate_halves(t, first, rot["dims"], rot["base"]).view(n, -1, 2, d) for t in (q, k))
+    v = (h @ w[f"{p}.v"].T).view(n, G, e)
+    st["k"] = torch.cat([st["k"], k]) if st else k
+    st["v"] = torch.cat([st["v"], v]) if "v" in st else v
+    mask = m.get("mask")
+    seen = same_chunk(first, n, first + n, mask["size"] if mask else None)
+    a1, a2 = (masked_attention(q[:, :, i], st["k"][:, :, i], st["v"], seen, m["scale"]) for i in range(2))
+    less = torch.exp((w[f"{p}.lq1"] * w[f"{p}.lk1"]).sum()) - torch.exp((w[f"{p}.lq2"] * w[f"{p}.lk2"]).sum()) + m["diff"]
+    o = rms(a1 - less * a2, eps) * (1.0 - m["diff"])
+    return (o.reshape(n, H * e) * sigmoid(h @ w[f"{p}.g"].T)) @ w[f"{p}.o"].T
+
+
+def mingru_mixer(w, p: str, m: dict, h, st: dict, eps: float) -> torch.Tensor:
+    """Element-wise recurrence whose gate and candidate read the current token only."""
+    z = sigmoid(h @ w[f"{p}.z"].T + w[f"{p}.z.b"])
+    u = h @ w[f"{p}.x"].T + w[f"{p}.x.b"]
+    candidate = torch.where(u >= 0, u + 0.5, sigmoid(u))
+    S = st["S"] if st else torch.zeros(m["width"], dtype=h.dtype)
+    out = torch.empty_like(u)
+    for t in range(h.shape[0]):
+        S = (1.0 - z[t]) * S + z[t] * candidate[t]
+        out[t] = S
+    st["S"] = S
+    return (out * silu(h @ w[f"{p}.g"].T)) @ w[f"{p}.o"].T
+
+
+GATED_MIXERS = {"latent_attention": rotated_latent_attention, "attention": differential_attention, "mingru": mingru_mixer}
+
+
+def clamped_feed_forward(w, p: str, h, limit: float) -> torch.Tensor:
+    g, u = torch.clamp(h @ w[f"{p}.gate"].T, max=limit), torch.clamp(h @ w[f"{p}.up"].T, -limit, limit)
+    return (g * sigmoid(1.702 * g) * (u + 1.0)) @ w[f"{p}.down"].T
+
+
 def layer_schedule(cfg: dict) -> list[tuple[int, bool]]:
     """The layer runs in order: (layer index, whether the pass's entry projection comes right before it)."""
     loop = cfg.get("loop")
@@ -430,6 +502,8 @@ class Oracle:
             return self._sequential(ids, state, eps, last_only, trace)
         if cfg["architecture"] == "Vimelorn":
             return self._streams(ids, state, eps, last_only, trace)
+        if cfg["architecture"] == "Fovunex":
+            return self._gated(ids, state, eps, last_only, trace)
         x0 = rms_around_zero(w["embed"][ids], w["embed.norm"], eps)
         x = x0
         for (i, enters), st in zip(self.schedule, state.runs):
@@ -495,6 +569,32 @@ class Oracle:
                 trace.append(xs.sum(0))
         state.length += len(ids)
         x = xs.sum(0)
+        if last_only:
+            x = x[-1:]
+        return (rms(x, eps) * w["final.norm"]) @ w["head"].T, state
+
+
+    def _gated(self, ids, state, eps: float, last_only: bool, trace):
+        """Pre-norm layers whose results pass a gate per channel that reads the same normed input; norms with one number; the
+        embedding output is added again before every later pass of the loop."""
+        w, cfg = self.w, self.cfg
+        x0 = w["embed"][ids] * cfg["embedding"]["scale"]
+        x, passes = x0, 0
+        for (i, enters), st in zip(self.schedule, state.runs):
+            if enters:
+                passes += 1
+                x = x + x0 if passes > 1 else x
+            layer, p = cfg["layers"][i], f"l{i}"
+            h = rms(x, eps) * w[f"{p}.norm1"]
+            y = GATED_MIXERS[layer["type"]](w, f"{p}.mix", layer["mixer"], h, st, eps)
+            x = x + y * sigmoid(h @ w[f"{p}.rg1"].T + w[f"{p}.rg1.b"])
+            if layer.get("mlp"):
+                h = rms(x, eps) * w[f"{p}.norm2"]
+                y = clamped_feed_forward(w, f"{p}.mlp", h, layer["mlp"]["limit"])
+                x = x + y * sigmoid(h @ w[f"{p}.rg2"].T + w[f"{p}.rg2.b"])
+            if trace is not None:
+                trace.append(x.clone())
+        state.length += len(ids)
         if last_only:
             x = x[-1:]
         return (rms(x, eps) * w["final.norm"]) @ w["head"].T, state
