@@ -362,7 +362,8 @@ def decoder_step_operators(cfg, rows: int, tp_size: int = 1, topology_id: str = 
 
 def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple[OpSignature, ...]:
     """Operator signatures of one decode step of a layered decoder: the distinct operators of its layer runs."""
-    from ..models.layered import AttentionSpec, BiasedAttentionSpec, ConvAttentionSpec, DeltaSpec, LatentSpec, SsdSpec
+    from ..models.layered import (AttentionSpec, BiasedAttentionSpec, ConvAttentionSpec, DeltaSpec, DifferentialSpec, LatentSpec, MinGruSpec,
+                                  SsdSpec)
     W, act = cfg.hidden_size, "fp32" if cfg.dtype == "float32" else "bf16"
     ops: dict[tuple, OpSignature] = {}
 
@@ -374,13 +375,22 @@ def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple
                                    "fp32", layout, tuple(sorted(shape.items())), topology_id)
 
     add("norm.rms", "residual32", W, W)
-    if cfg.loop is not None:
+    if cfg.loop is not None and cfg.design.loop == "project":
         add("linear.bf16", "loop_entry", W, 2 * W)
+    elif cfg.loop is not None:
+        add("norm.rms", "residual32_entry", W, W)
     for i, _ in cfg.runs:
         l = cfg.layers[i]
         for m in l.mixer.parts:
             if isinstance(m, LatentSpec):
-                add("attention.latent", "paged", m.out_width, m.q_rank + m.kv_rank, heads=m.heads, window=m.window or cfg.max_position)
+                rotated = {"rotated": m.rot_dim} if m.rot_dim else {}
+                add("attention.latent", "paged", m.out_width, (m.q_rank or m.heads * m.dim) + m.kv_rank, heads=m.heads,
+                    window=m.window or cfg.max_position, **rotated)
+            elif isinstance(m, DifferentialSpec):
+                add("attention.differential", "paged", m.out_width, 2 * (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim, heads=m.heads,
+                    chunk=m.chunk or cfg.max_position)
+            elif isinstance(m, MinGruSpec):
+                add("linear_recurrence.elementwise", "state32", m.width, 3 * m.width)
             elif isinstance(m, AttentionSpec):
                 add("attention.gqa", "paged", m.out_width, (m.heads + m.kv_heads) * m.dim, heads=m.heads,
                     window=m.window or cfg.max_position)
@@ -397,6 +407,8 @@ def layered_step_operators(cfg, rows: int, topology_id: str = "single") -> tuple
             else:
                 add("linear_recurrence.channel", "state32", m.out_width, 2 * m.heads * m.dim, heads=m.heads)
         if cfg.design.sequential:
+            if cfg.design.gated:
+                add("residual.gate", "residual32", W, W)
             add("linear.bf16", "out", W, l.mixer.out_width)
             if l.ff:
                 add("linear.bf16", "gate_up", 2 * l.ff, W)

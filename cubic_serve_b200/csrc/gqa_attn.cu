@@ -1,5 +1,6 @@
 // Grouped-query attention of the layered decoders over a paged cache in the activation type: a sliding window, first tokens that
-// stay visible behind it, a bias per distance and head, and a softmax entry without a value (sink).
+// stay visible behind it, or chunks of positions; a bias per distance and head, a softmax entry without a value (sink), and the
+// difference of two attention maps over the same values.
 //
 //   gqa_prepare_kernel    RMS norm of every query and key head, rotary positions on neighbouring channel pairs; keys and values
 //                         to their page, where a value is the raw key of its token, as projected (qkv_prepare.cu has the others)
@@ -9,7 +10,9 @@
 //   gqa_row_kernel        fp32 models: a warp per (token, head)
 //
 // The cache is [pages][key head][key, value][16][P], P the wider of the key and value widths rounded up to 64, zero columns behind
-// the head.  Scores, softmax weights and sums are fp32; the weights are rounded to bf16 as the operand of the second product of the bf16 kernels.
+// the head.  With two maps (MAPS 2) a query or key row holds both, half of its columns each (P is 64, 128 or 256), and every (token,
+// head) has a row of scores per map: rows of both maps share the keys and values a block has loaded, and the maps' outputs meet in
+// the epilogue, where the difference is normed over the head and gated per channel.  Scores, softmax weights and sums are fp32; the weights are rounded to bf16 as the operand of the second product of the bf16 kernels.
 #include <climits>
 #include <type_traits>
 
@@ -119,24 +122,35 @@ struct GqaAttn {
   int max_pages;
   int H, G, e, P, window;     // e: width of a value; window <= 0: every earlier token
   int keep;                   // the first tokens, visible whatever the window (0 without a window)
+  int chunk;                  // > 0: a token sees its own chunk of positions only (no window then)
   float scale, out_scale;
   float sink;                 // score of the entry without a value, -inf: none
   const float* bias;          // [bias_far + 1, H] added to the scaled score by distance (the last row from bias_far on), null: none
   int bias_far;
+  float less;                 // two maps: the second's output times this is taken from the first's, the difference o leaves as
+  float eps;                  // o / sqrt(mean(o^2) + eps) * out_scale * sigmoid(gate)
+  const T* gate; int ldg;     // [T, H e] logits
   Segments sg;
+
+  // First key the token at `pos` sees (kept ones aside); it never decreases with the position
+  __device__ __forceinline__ int first_key(int pos) const {
+    return chunk > 0 ? pos - pos % chunk : window > 0 ? max(0, pos - window + 1) : 0;
+  }
 };
 
-// Keys of a query tile [pos0, pos0 + toks): the window's from `kmin` (a page's first key) on, and the kept ones below it, [0, kept)
+// Keys of a query tile from position pos0 on: the visible ones from `kmin` (a page's first key) on, and the kept ones below it, [0, kept)
 struct GqaSpan {
   int kmin, kept;
-  __device__ __forceinline__ GqaSpan(int window, int keep, int pos0) {
-    kmin = window > 0 ? max(0, pos0 - window + 1) & ~(kGqaPage - 1) : 0;
+  __device__ __forceinline__ GqaSpan(int first_key, int keep) {
+    kmin = first_key & ~(kGqaPage - 1);
     kept = min(keep, kmin);
   }
 };
 
+__device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + expf(-z)); }
+
 // ------------------------------------------------------------------ fp32
-template <int NR>
+template <int NR, int MAPS>
 __global__ void __launch_bounds__(128)
 gqa_row_kernel(const GqaAttn<float> p) {
   pdl_wait();
@@ -149,42 +163,65 @@ gqa_row_kernel(const GqaAttn<float> p) {
   const int kh = h / (p.H / p.G);
   const size_t row = static_cast<size_t>(p.sg.row0[s]) + off;
   const int pos = p.sg.pos0[s] + off;
-  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int lo = p.first_key(pos);
   const int* pages = p.page_table + static_cast<size_t>(p.sg.slot[s]) * p.max_pages;
   const float* qr = p.q + (row * p.H + h) * p.P;
-  float q[NR], acc[NR];
+  float q[NR], acc[MAPS][NR], m[MAPS], l[MAPS];
 #pragma unroll
-  for (int i = 0; i < NR; ++i) {
-    q[i] = qr[lane + 32 * i] * p.scale;
-    acc[i] = 0.f;
+  for (int i = 0; i < NR; ++i) q[i] = qr[lane + 32 * i] * p.scale;
+#pragma unroll
+  for (int k = 0; k < MAPS; ++k) {
+#pragma unroll
+    for (int i = 0; i < NR; ++i) acc[k][i] = 0.f;
+    m[k] = p.sink;
+    l[k] = p.sink == -INFINITY ? 0.f : 1.f;
   }
-  float m = p.sink, l = p.sink == -INFINITY ? 0.f : 1.f;
   const int kept = min(p.keep, lo);
   for (int i = 0; i < kept + pos + 1 - lo; ++i) {
     const int j = i < kept ? i : lo + i - kept;
     const float* kr = p.cache + ((static_cast<size_t>(pages[j / kGqaPage]) * p.G + kh) * 2 * kGqaPage + j % kGqaPage) * p.P;
     const float* vr = kr + kGqaPage * p.P;
-    float v[NR], sdot = 0.f;
+    float v[NR], sdot[MAPS] = {};
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
       v[i] = vr[lane + 32 * i];
-      sdot = fmaf(q[i], kr[lane + 32 * i], sdot);
+      sdot[i * MAPS / NR] = fmaf(q[i], kr[lane + 32 * i], sdot[i * MAPS / NR]);
     }
-    sdot = warp_sum(sdot);
-    if (p.bias) sdot += __ldg(p.bias + static_cast<size_t>(min(pos - j, p.bias_far)) * p.H + h);
-    const float mn = fmaxf(m, sdot);
-    const float f = expf(m - mn), w = expf(sdot - mn);
-    m = mn;
-    l = l * f + w;
 #pragma unroll
-    for (int i = 0; i < NR; ++i) acc[i] = fmaf(w, v[i], acc[i] * f);
+    for (int k = 0; k < MAPS; ++k) {
+      sdot[k] = warp_sum(sdot[k]);
+      if (p.bias) sdot[k] += __ldg(p.bias + static_cast<size_t>(min(pos - j, p.bias_far)) * p.H + h);
+      const float mn = fmaxf(m[k], sdot[k]);
+      const float f = expf(m[k] - mn), w = expf(sdot[k] - mn);
+      m[k] = mn;
+      l[k] = l[k] * f + w;
+#pragma unroll
+      for (int i = 0; i < NR; ++i) acc[k][i] = fmaf(w, v[i], acc[k][i] * f);
+    }
   }
-  const float g = p.out_scale / l;
   float* orow = p.out + row * p.ldo + h * p.e;
+  if constexpr (MAPS == 2) {
+    const float i1 = 1.f / l[0], i2 = p.less / l[1];
+    float ss = 0.f;                                     // columns behind the value are zero
 #pragma unroll
-  for (int i = 0; i < NR; ++i) {
-    const int c = lane + 32 * i;
-    if (c < p.e) orow[c] = acc[i] * g;
+    for (int i = 0; i < NR; ++i) {
+      acc[0][i] = acc[0][i] * i1 - acc[1][i] * i2;
+      ss = fmaf(acc[0][i], acc[0][i], ss);
+    }
+    const float g = p.out_scale / sqrtf(warp_sum(ss) / static_cast<float>(p.e) + p.eps);
+    const float* gr = p.gate + row * p.ldg + h * p.e;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int c = lane + 32 * i;
+      if (c < p.e) orow[c] = acc[0][i] * g * sigmoid_of(gr[c]);
+    }
+  } else {
+    const float g = p.out_scale / l[0];
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int c = lane + 32 * i;
+      if (c < p.e) orow[c] = acc[0][i] * g;
+    }
   }
 }
 
@@ -205,6 +242,8 @@ struct GqaMma {
   int bias_rows;              // prompts: rows of the bias table kept in shared memory (bias_far + 1), 0: read in place
   float* partial;             // decode: [segment][key head tile][split][16][P + 2]
 };
+// Decode rows of a block are 16: the heads of a key head, with two maps eight heads' first maps and their second maps
+template <int MAPS> constexpr int decode_heads() { return 16 / MAPS; }
 
 __device__ __forceinline__ void store_pair(bf16* row, int c, int d, float x, float y) {
   if (c + 1 < d && (d & 1) == 0) {
@@ -215,14 +254,29 @@ __device__ __forceinline__ void store_pair(bf16* row, int c, int d, float x, flo
   }
 }
 
+// Two channels of the normed and gated difference of two maps, written to a row of outputs (`gate`: the head's logits of the row)
+__device__ __forceinline__ void store_gated_pair(bf16* row, const bf16* gate, int c, int e, float x, float y) {
+  if (c + 1 < e && (e & 1) == 0) {
+    const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + c));
+    *reinterpret_cast<uint32_t*>(row + c) = pack_bf16x2(x * sigmoid_of(z.x), y * sigmoid_of(z.y));
+  } else {
+    if (c < e) row[c] = __float2bfloat16(x * sigmoid_of(to_f(gate[c])));
+    if (c + 1 < e) row[c + 1] = __float2bfloat16(y * sigmoid_of(to_f(gate[c + 1])));
+  }
+}
+
 // Four warps of 16 rows each, row = token * hb + head; key tiles of 64 keys in two buffers, 16-byte chunks XOR-swizzled by the
-// row.  A warp keeps its rows' scores, weights and outputs in registers: no exchange between warps.
+// row.  A warp keeps its rows' scores, weights and outputs in registers: no exchange between warps.  With two maps the first two
+// warps have the first map's rows, the others the second's of the same (token, head); a warp's products run over its map's half of
+// the columns, and the second map's outputs pass through shared memory once at the end.
 static constexpr int kGqaWarps = 4;
 static constexpr int kGqaBiasBytes = 11 << 10;      // three blocks of two column groups and their tables fit on an SM
-template <int NCH, bool BIAS>
+template <int NCH, bool BIAS, int MAPS>
 __global__ void __launch_bounds__(32 * kGqaWarps, NCH <= 2 ? 3 : 1)
 gqa_prefill_kernel(const GqaMma p) {
-  constexpr int P = NCH * 64, ROWB = P * 2, NW = kGqaWarps, MR = 16 * NW, KT = 64, CH = P / 8, NT = P / 8;
+  constexpr int P = NCH * 64, ROWB = P * 2, NW = kGqaWarps, MR = 16 * NW / MAPS, KT = 64, CH = P / 8, NT = P / 8;
+  constexpr int KS = P / 16 / MAPS;                   // steps of a product over a map's columns
+  static_assert(MAPS == 1 || (!BIAS && NCH != 3), "two maps take half of a row each");
   extern __shared__ __align__(128) uint8_t lsm[];
   constexpr bool QREG = NCH <= 2;                     // query fragments in registers; the rows pass through the second buffer
   uint8_t* kvs = lsm + (QREG ? 0 : MR * ROWB);        // [2 buffers][key, value][KT][ROWB]
@@ -233,14 +287,15 @@ gqa_prefill_kernel(const GqaMma p) {
   const GqaAttn<bf16>& a = p.a;
   int s, off;
   if (!find_tile(a.sg, p.qb, blockIdx.x, s, off)) return;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int tid = threadIdx.x, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int warp = MAPS == 2 ? (tid >> 5) & 1 : tid >> 5, map = MAPS == 2 ? tid >> 6 : 0;     // warp: of the rows
   const int R = a.H / a.G, kh = blockIdx.y / p.head_tiles, hq0 = (blockIdx.y % p.head_tiles) * p.hb;
   const int heads = min(p.hb, R - hq0), h0 = kh * R + hq0;
   const int toks = min(p.qb, a.sg.count[s] - off);
   const size_t row0 = static_cast<size_t>(a.sg.row0[s]) + off;
   const int pos0 = a.sg.pos0[s] + off;
   const int* pages = a.page_table + static_cast<size_t>(a.sg.slot[s]) * a.max_pages;
-  const GqaSpan span(a.window, a.keep, pos0);
+  const GqaSpan span(a.first_key(pos0), a.keep);
   const int kmin = span.kmin, kept_tiles = (span.kept + KT - 1) / KT;
   const int kend = pos0 + toks;
   const int tiles = kept_tiles + (kend - kmin + KT - 1) / KT;
@@ -288,7 +343,7 @@ gqa_prefill_kernel(const GqaMma p) {
     const int r = warp * 16 + g + 8 * i;
     const int tok = r / p.hb, h = r - tok * p.hb;
     lim_hi[i] = tok < toks && h < heads ? pos0 + tok : -1;
-    lim_lo[i] = a.window > 0 ? pos0 + tok - a.window + 1 : 0;
+    lim_lo[i] = a.first_key(pos0 + tok);
     if constexpr (BIAS) {
       const int head = (h < heads ? h : 0) + (p.bias_rows ? 0 : h0);
       bias_at[i] = (pos0 + tok) * bias_step + head;
@@ -298,8 +353,8 @@ gqa_prefill_kernel(const GqaMma p) {
   // of the whole warp
   const int tok_a = min(warp * 16 / p.hb, toks - 1), tok_b = min((warp * 16 + 15) / p.hb, toks - 1);
   const bool idle = warp * 16 / p.hb >= toks;
-  const int see_lo = a.window > 0 ? pos0 + tok_a - a.window + 1 : 0, see_hi = pos0 + tok_b;     // some row sees these
-  const int all_lo = a.window > 0 ? pos0 + tok_b - a.window + 1 : 0, all_hi = pos0 + tok_a;     // every row sees these
+  const int see_lo = a.first_key(pos0 + tok_a), see_hi = pos0 + tok_b;     // some row sees these
+  const int all_lo = a.first_key(pos0 + tok_b), all_hi = pos0 + tok_a;     // every row sees these
   const float sc = a.scale * kLog2e;
   float m2[2] = {-INFINITY, -INFINITY}, l2[2] = {0.f, 0.f};
   float o[NT][4];
@@ -315,13 +370,17 @@ gqa_prefill_kernel(const GqaMma p) {
     q_at[i] = q_base + (((i * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
     k_at[i] = ((lane & 7) + ((lane >> 4) << 3)) * ROWB + (((i * 2 + ((lane >> 3) & 1)) ^ (lane & 7)) << 4);
     v_at[i] = (lane & 15) * ROWB + (((i * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
+    if (MAPS == 2 && map) {                           // the second half of a row: four chunks, or whole 128-byte groups, on
+      q_at[i] = NCH == 1 ? q_at[i] ^ 64 : q_at[i] + NCH * 64;
+      k_at[i] = NCH == 1 ? k_at[i] ^ 64 : k_at[i] + NCH * 64;
+    }
   }
-  uint32_t qr[QREG ? P / 16 : 1][4];
+  uint32_t qr[QREG ? KS : 1][4];
   if constexpr (QREG) {
     asm volatile("cp.async.wait_all;" ::: "memory");
     __syncthreads();
 #pragma unroll
-    for (int kk = 0; kk < P / 16; ++kk) ldsm4(qr[kk], q_at[kk & 3] + (kk >> 2) * 128);
+    for (int kk = 0; kk < KS; ++kk) ldsm4(qr[kk], q_at[kk & 3] + (kk >> 2) * 128);
     __syncthreads();
   }
   for (int t = 0; t < tiles; ++t) {
@@ -340,7 +399,7 @@ gqa_prefill_kernel(const GqaMma p) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) sf[j][c] = 0.f;
 #pragma unroll
-      for (int kk = 0; kk < P / 16; ++kk) {
+      for (int kk = 0; kk < KS; ++kk) {
         uint32_t qa[4];
         if constexpr (QREG) { qa[0] = qr[kk][0]; qa[1] = qr[kk][1]; qa[2] = qr[kk][2]; qa[3] = qr[kk][3]; }
         else ldsm4(qa, q_at[kk & 3] + (kk >> 2) * 128);
@@ -440,6 +499,49 @@ gqa_prefill_kernel(const GqaMma p) {
     __syncthreads();                                  // the tile's buffer is free again
   }
   asm volatile("cp.async.wait_all;" ::: "memory");
+  if constexpr (MAPS == 2) {
+    constexpr int LD = P + 8;
+    float* other = reinterpret_cast<float*>(kvs);      // [MR][LD]: what is taken away; nobody reads keys or values any more
+    if (map) {
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        l2[i] += __shfl_xor_sync(0xffffffffu, l2[i], 1);
+        l2[i] += __shfl_xor_sync(0xffffffffu, l2[i], 2);
+        const float f = a.less / l2[i];
+        float* row = other + (warp * 16 + g + 8 * i) * LD + 2 * t4;
+#pragma unroll
+        for (int j = 0; j < NT; ++j) *reinterpret_cast<float2*>(row + j * 8) = make_float2(o[j][2 * i] * f, o[j][2 * i + 1] * f);
+      }
+    }
+    __syncthreads();
+    if (map) return;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      l2[i] += __shfl_xor_sync(0xffffffffu, l2[i], 1);
+      l2[i] += __shfl_xor_sync(0xffffffffu, l2[i], 2);
+      const int r = warp * 16 + g + 8 * i;
+      const int tok = r / p.hb, h = r - tok * p.hb;
+      const float f = 1.f / l2[i];
+      const float* sub = other + r * LD + 2 * t4;
+      float ss = 0.f;                                  // columns behind the value are zero
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const float2 u = *reinterpret_cast<const float2*>(sub + j * 8);
+        o[j][2 * i] = o[j][2 * i] * f - u.x;
+        o[j][2 * i + 1] = o[j][2 * i + 1] * f - u.y;
+        ss = fmaf(o[j][2 * i], o[j][2 * i], fmaf(o[j][2 * i + 1], o[j][2 * i + 1], ss));
+      }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      if (tok >= toks || h >= heads) continue;
+      const float n = a.out_scale / sqrtf(ss / static_cast<float>(a.e) + a.eps);
+      bf16* row = a.out + (row0 + tok) * a.ldo + (h0 + h) * a.e;
+      const bf16* gate = a.gate + (row0 + tok) * a.ldg + (h0 + h) * a.e;
+#pragma unroll
+      for (int j = 0; j < NT; ++j) store_gated_pair(row, gate, j * 8 + 2 * t4, a.e, o[j][2 * i] * n, o[j][2 * i + 1] * n);
+    }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     l2[i] += __shfl_xor_sync(0xffffffffu, l2[i], 1);
@@ -456,10 +558,28 @@ gqa_prefill_kernel(const GqaMma p) {
 
 // ------------------------------------------------------------------ bf16, one token per segment
 // Four warps deal the pages of a (segment, key head, split) among themselves; each has its own ring of kRing pages.  The rows of
-// a product are the query heads of the key head (up to 16 of them).
+// a product are the query heads of the key head (up to 16 of them); with two maps a query's row of the first map is zero in the
+// second's columns and the other way round, so that one product makes both maps' scores.
 static constexpr int kRing = 3;
 
-template <int NCH, bool BIAS>
+// A head's output from its maps' outputs x1, x2 (columns 2 (lane + 32 i) of a warp) and their factors
+template <int NCH>
+__device__ __forceinline__ void store_difference(const GqaAttn<bf16>& a, size_t t, int h, int lane, const float2 (&x1)[NCH], float f1,
+                                                 const float2 (&x2)[NCH], float f2) {
+  float2 v[NCH];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NCH; ++i) {
+    v[i] = make_float2(x1[i].x * f1 - x2[i].x * f2, x1[i].y * f1 - x2[i].y * f2);
+    ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, ss));
+  }
+  const float n = a.out_scale / sqrtf(warp_sum(ss) / static_cast<float>(a.e) + a.eps);
+#pragma unroll
+  for (int i = 0; i < NCH; ++i)
+    store_gated_pair(a.out + t * a.ldo + h * a.e, a.gate + t * a.ldg + h * a.e, 2 * (lane + 32 * i), a.e, v[i].x * n, v[i].y * n);
+}
+
+template <int NCH, bool BIAS, int MAPS>
 __global__ void __launch_bounds__(128)
 gqa_decode_kernel(const GqaMma p) {
   constexpr int P = NCH * 64, ROWB = P * 2, CH = P / 8, NT = P / 8, PAGEB = 2 * kGqaPage * ROWB;
@@ -470,12 +590,13 @@ gqa_decode_kernel(const GqaMma p) {
   const int s = blockIdx.x;
   if (a.sg.count[s] <= 0) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-  const int R = a.H / a.G, kh = blockIdx.y / p.head_tiles, hq0 = (blockIdx.y % p.head_tiles) * 16;
-  const int heads = min(16, R - hq0), h0 = kh * R + hq0;
+  constexpr int HB = decode_heads<MAPS>();
+  const int R = a.H / a.G, kh = blockIdx.y / p.head_tiles, hq0 = (blockIdx.y % p.head_tiles) * HB;
+  const int heads = min(HB, R - hq0), h0 = kh * R + hq0;
   const size_t row = a.sg.row0[s];
   const int pos = a.sg.pos0[s];
   const int* pages = a.page_table + static_cast<size_t>(a.sg.slot[s]) * a.max_pages;
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int lo = a.first_key(pos);
   // the pages to walk: those with kept tokens below the window, then the window's
   const int pg_first = lo / kGqaPage, kept_pages = (min(a.keep, pg_first * kGqaPage) + kGqaPage - 1) / kGqaPage;
   const int skip = pg_first - kept_pages;             // pages between the two
@@ -503,8 +624,9 @@ gqa_decode_kernel(const GqaMma p) {
   for (int kk = 0; kk < P / 16; ++kk)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      const int h = g + 8 * (i & 1), c = kk * 16 + 2 * t4 + 8 * (i >> 1);
-      qa[kk][i] = h < heads ? *reinterpret_cast<const uint32_t*>(a.q + (row * a.H + h0 + h) * P + c) : 0u;
+      const int h = MAPS == 2 ? g : g + 8 * (i & 1), c = kk * 16 + 2 * t4 + 8 * (i >> 1);
+      const bool in = MAPS == 1 || (kk >= P / 32) == ((i & 1) != 0);      // rows 8 .. 15 are the second maps
+      qa[kk][i] = in && h < heads ? *reinterpret_cast<const uint32_t*>(a.q + (row * a.H + h0 + h) * P + c) : 0u;
     }
   const float sc = a.scale * kLog2e;
   float m2[2] = {-INFINITY, -INFINITY}, l2[2] = {0.f, 0.f};
@@ -622,16 +744,51 @@ gqa_decode_kernel(const GqaMma p) {
   }
   __syncthreads();
   const size_t unit = static_cast<size_t>(s) * gridDim.y + blockIdx.y;
-  for (int r = warp; r < heads; r += 4) {
-    float mx = -INFINITY, f[4], l = 0.f;
+  // the warps' results of row r: maximum, sum and factors
+  auto merge = [&](int r, float& mx, float& use, float& l, float (&f)[4]) {
+    mx = -INFINITY;
+    l = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) mx = fmaxf(mx, res[(w * 16 + r) * LD + P]);
-    const float use = mx == -INFINITY ? 0.f : mx;
+    use = mx == -INFINITY ? 0.f : mx;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       f[w] = ex2(res[(w * 16 + r) * LD + P] - use);
       l += f[w] * res[(w * 16 + r) * LD + P + 1];
     }
+  };
+  if constexpr (MAPS == 2) {
+    for (int r = warp; r < heads; r += 4) {
+      float2 v[2][NCH];
+      float l[2];
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        float mx, use, f[4];
+        merge(r + 8 * k, mx, use, l[k], f);
+#pragma unroll
+        for (int i = 0; i < NCH; ++i) {
+          v[k][i] = make_float2(0.f, 0.f);
+#pragma unroll
+          for (int w = 0; w < 4; ++w) {
+            const float2 u = *reinterpret_cast<const float2*>(res + (w * 16 + r + 8 * k) * LD + 2 * (lane + 32 * i));
+            v[k][i].x = fmaf(f[w], u.x, v[k][i].x);
+            v[k][i].y = fmaf(f[w], u.y, v[k][i].y);
+          }
+        }
+        if (p.splits > 1) {
+          float* part = p.partial + ((unit * p.splits + blockIdx.z) * 16 + r + 8 * k) * LD;
+#pragma unroll
+          for (int i = 0; i < NCH; ++i) *reinterpret_cast<float2*>(part + 2 * (lane + 32 * i)) = v[k][i];
+          if (lane == 0) *reinterpret_cast<float2*>(part + P) = make_float2(mx, l[k]);
+        }
+      }
+      if (p.splits == 1) store_difference<NCH>(a, row, h0 + r, lane, v[0], 1.f / l[0], v[1], a.less / l[1]);
+    }
+    return;
+  }
+  for (int r = warp; r < heads; r += 4) {
+    float mx, use, l, f[4];
+    merge(r, mx, use, l, f);
     float* part = p.partial + ((unit * p.splits + blockIdx.z) * 16 + r) * LD;
     const float scale = p.splits > 1 ? 1.f : a.out_scale / (l + ex2(a.sink * kLog2e - use));
 #pragma unroll
@@ -652,7 +809,7 @@ gqa_decode_kernel(const GqaMma p) {
 }
 
 // A warp per row of a unit.
-template <int NCH>
+template <int NCH, int MAPS>
 __global__ void __launch_bounds__(128)
 gqa_merge_kernel(const GqaMma p) {
   constexpr int P = NCH * 64, LD = P + 2;
@@ -661,31 +818,45 @@ gqa_merge_kernel(const GqaMma p) {
   const GqaAttn<bf16>& a = p.a;
   const int s = blockIdx.x, lane = threadIdx.x & 31, r = blockIdx.z * 4 + (threadIdx.x >> 5);
   if (a.sg.count[s] <= 0) return;
-  const int R = a.H / a.G, kh = blockIdx.y / p.head_tiles, hq0 = (blockIdx.y % p.head_tiles) * 16;
-  if (r >= min(16, R - hq0)) return;
+  constexpr int HB = decode_heads<MAPS>();
+  const int R = a.H / a.G, kh = blockIdx.y / p.head_tiles, hq0 = (blockIdx.y % p.head_tiles) * HB;
+  if (r >= min(HB, R - hq0)) return;
   const size_t unit = static_cast<size_t>(s) * gridDim.y + blockIdx.y;
-  const float* part = p.partial + (unit * p.splits * 16 + r) * LD;
   constexpr int step = 16 * LD;
-  float mx = a.sink * kLog2e;
-  for (int z = 0; z < p.splits; ++z) mx = fmaxf(mx, part[z * step + P]);
-  float l = ex2(a.sink * kLog2e - mx);
-  float2 v[NCH];
+  // row `at` of the unit: sum over the splits, returns the sum of the weights
+  auto merge = [&](int at, float2 (&v)[NCH]) {
+    const float* part = p.partial + (unit * p.splits * 16 + at) * LD;
+    float mx = a.sink * kLog2e;
+    for (int z = 0; z < p.splits; ++z) mx = fmaxf(mx, part[z * step + P]);
+    float l = ex2(a.sink * kLog2e - mx);
 #pragma unroll
-  for (int i = 0; i < NCH; ++i) v[i] = make_float2(0.f, 0.f);
-  for (int z = 0; z < p.splits; ++z) {
-    const float f = ex2(part[z * step + P] - mx);   // 0 for a split that saw no key
-    l += f * part[z * step + P + 1];
+    for (int i = 0; i < NCH; ++i) v[i] = make_float2(0.f, 0.f);
+    for (int z = 0; z < p.splits; ++z) {
+      const float f = ex2(part[z * step + P] - mx);   // 0 for a split that saw no key
+      l += f * part[z * step + P + 1];
 #pragma unroll
-    for (int i = 0; i < NCH; ++i) {
-      const float2 u = *reinterpret_cast<const float2*>(part + z * step + 2 * (lane + 32 * i));
-      v[i].x = fmaf(f, u.x, v[i].x);
-      v[i].y = fmaf(f, u.y, v[i].y);
+      for (int i = 0; i < NCH; ++i) {
+        const float2 u = *reinterpret_cast<const float2*>(part + z * step + 2 * (lane + 32 * i));
+        v[i].x = fmaf(f, u.x, v[i].x);
+        v[i].y = fmaf(f, u.y, v[i].y);
+      }
     }
-  }
-  const float f = a.out_scale / l;
-  bf16* row = a.out + static_cast<size_t>(a.sg.row0[s]) * a.ldo + (kh * R + hq0 + r) * a.e;
+    return l;
+  };
+  const size_t t = static_cast<size_t>(a.sg.row0[s]);
+  const int h = kh * R + hq0 + r;
+  float2 v[NCH];
+  const float l = merge(r, v);
+  if constexpr (MAPS == 2) {
+    float2 v2[NCH];
+    const float l2 = merge(r + 8, v2);
+    store_difference<NCH>(a, t, h, lane, v, 1.f / l, v2, a.less / l2);
+  } else {
+    const float f = a.out_scale / l;
+    bf16* row = a.out + t * a.ldo + h * a.e;
 #pragma unroll
-  for (int i = 0; i < NCH; ++i) store_pair(row, 2 * (lane + 32 * i), a.e, v[i].x * f, v[i].y * f);
+    for (int i = 0; i < NCH; ++i) store_pair(row, 2 * (lane + 32 * i), a.e, v[i].x * f, v[i].y * f);
+  }
 }
 
 // ------------------------------------------------------------------ host
@@ -702,30 +873,36 @@ static int gqa_go(K kernel, dim3 grid, int threads, size_t smem, const GqaMma& p
   return static_cast<int>(launch(kernel, grid, dim3(threads), smem, st, p));
 }
 
-template <int NCH, bool BIAS>
+template <int NCH, bool BIAS, int MAPS>
 static int gqa_prefill(const GqaMma& p, dim3 grid, cudaStream_t st) {
   static bool configured[64] = {};
-  const size_t rows = static_cast<size_t>((NCH <= 2 ? 0 : 16 * kGqaWarps) + 256) * NCH * 128;
-  return gqa_go(gqa_prefill_kernel<NCH, BIAS>, grid, 32 * kGqaWarps, rows + (BIAS ? static_cast<size_t>(p.bias_rows) * p.hb * 4 : 0), p, configured,
-                st, rows + (BIAS ? kGqaBiasBytes : 0));
+  const size_t rows = static_cast<size_t>((NCH <= 2 ? 0 : 16 * kGqaWarps / MAPS) + 256) * NCH * 128;
+  return gqa_go(gqa_prefill_kernel<NCH, BIAS, MAPS>, grid, 32 * kGqaWarps, rows + (BIAS ? static_cast<size_t>(p.bias_rows) * p.hb * 4 : 0), p,
+                configured, st, rows + (BIAS ? kGqaBiasBytes : 0));
 }
 
-template <int NCH, bool BIAS>
+template <int NCH, bool BIAS, int MAPS>
 static int gqa_decode(const GqaMma& p, dim3 grid, cudaStream_t st) {
   static bool configured[64] = {};
-  const int rc = gqa_go(gqa_decode_kernel<NCH, BIAS>, grid, 128, static_cast<size_t>(4) * kRing * 2 * kGqaPage * NCH * 128, p, configured, st);
+  const int rc = gqa_go(gqa_decode_kernel<NCH, BIAS, MAPS>, grid, 128, static_cast<size_t>(4) * kRing * 2 * kGqaPage * NCH * 128, p, configured, st);
   if (rc || p.splits == 1) return rc;
-  return static_cast<int>(launch(gqa_merge_kernel<NCH>, dim3(grid.x, grid.y, 4), dim3(128), 0, st, p));
+  return static_cast<int>(launch(gqa_merge_kernel<NCH, MAPS>, dim3(grid.x, grid.y, 4 / MAPS), dim3(128), 0, st, p));
 }
 
-template <bool BIAS>
+template <bool BIAS, int MAPS>
 static int gqa_mma(const GqaMma& p, int nch, bool decode, dim3 grid, cudaStream_t st) {
   switch (nch) {
-    case 1: return decode ? gqa_decode<1, BIAS>(p, grid, st) : gqa_prefill<1, BIAS>(p, grid, st);
-    case 2: return decode ? gqa_decode<2, BIAS>(p, grid, st) : gqa_prefill<2, BIAS>(p, grid, st);
-    case 3: return decode ? gqa_decode<3, BIAS>(p, grid, st) : gqa_prefill<3, BIAS>(p, grid, st);
+    case 1: return decode ? gqa_decode<1, BIAS, MAPS>(p, grid, st) : gqa_prefill<1, BIAS, MAPS>(p, grid, st);
+    case 2: return decode ? gqa_decode<2, BIAS, MAPS>(p, grid, st) : gqa_prefill<2, BIAS, MAPS>(p, grid, st);
+    case 3:
+      if constexpr (MAPS == 1) return decode ? gqa_decode<3, BIAS, 1>(p, grid, st) : gqa_prefill<3, BIAS, 1>(p, grid, st);
+      return -15;
   }
-  return decode ? gqa_decode<4, BIAS>(p, grid, st) : gqa_prefill<4, BIAS>(p, grid, st);
+  return decode ? gqa_decode<4, BIAS, MAPS>(p, grid, st) : gqa_prefill<4, BIAS, MAPS>(p, grid, st);
+}
+static int gqa_mma_any(const GqaMma& p, int nch, bool decode, dim3 grid, cudaStream_t st) {
+  if (p.a.gate) return gqa_mma<false, 2>(p, nch, decode, grid, st);
+  return p.a.bias ? gqa_mma<true, 1>(p, nch, decode, grid, st) : gqa_mma<false, 1>(p, nch, decode, grid, st);
 }
 
 }  // namespace cb
@@ -752,10 +929,12 @@ struct CbGqaAttn {
   void* out; int ldo;
   const void* cache;
   const void* page_table;
-  int max_pages, H, G, e, P, window, keep;
+  int max_pages, H, G, e, P, window, keep, chunk;
   float scale, out_scale, sink;
   const void* bias;           // fp32 [bias_far + 1, H] or null
   int bias_far;
+  const void* gate; int ldg;  // two maps: gate logits [T, H e] of their difference (null: one map), see GqaAttn
+  float less, eps;
   int tokens, f32;
   int decode;                 // every segment has at most one row, row s belongs to segment s
   int splits;                 // key splits of the decode form (1 = none)
@@ -763,9 +942,10 @@ struct CbGqaAttn {
 };
 
 // Scratch of a split decode launch; `units` receives the blocks of one split.
-long long cb_gqa_attn_partial_floats(int tokens, int segs, int H, int G, int P, int decode, int splits, int* units) {
+long long cb_gqa_attn_partial_floats(int tokens, int segs, int H, int G, int P, int maps, int decode, int splits, int* units) {
   if (!decode) return 0;
-  const long long n = static_cast<long long>(segs) * G * ((H / G + 15) / 16);
+  const int hb = 16 / maps;
+  const long long n = static_cast<long long>(segs) * G * ((H / G + hb - 1) / hb);
   if (units) *units = static_cast<int>(n);
   return splits > 1 ? n * splits * 16 * (P + 2) : 0;
 }
@@ -794,7 +974,9 @@ int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
   using namespace cb;
   if (!a || !seg || seg->num <= 0 || a->tokens <= 0) return 0;
   if (a->H <= 0 || a->G <= 0 || (a->H % a->G) || a->e <= 0 || a->P < a->e || a->P > 256 || (a->P & 63) || a->ldo < a->H * a->e) return -10;
-  if (a->keep < 0 || (a->bias && a->bias_far < 0)) return -13;
+  if (a->keep < 0 || (a->bias && a->bias_far < 0) || a->chunk < 0 || (a->chunk && (a->window > 0 || a->keep))) return -13;
+  if (a->gate && (a->bias || a->P == 192 || a->ldg < a->H * a->e || a->sink != -INFINITY)) return -14;
+  const int maps = a->gate ? 2 : 1;
   if (a->splits > 1 && (!a->decode || !a->partial || a->splits > 65535)) return -12;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   auto fill = [&](auto& p) {
@@ -805,6 +987,8 @@ int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
     p.page_table = static_cast<const int*>(a->page_table); p.max_pages = a->max_pages;
     p.H = a->H; p.G = a->G; p.e = a->e; p.P = a->P; p.window = a->window;
     p.keep = a->window > 0 ? a->keep : 0;
+    p.chunk = a->chunk;
+    p.gate = static_cast<const T*>(a->gate); p.ldg = a->ldg; p.less = a->less; p.eps = a->eps;
     p.bias = static_cast<const float*>(a->bias); p.bias_far = a->bias_far;
     p.scale = a->scale; p.out_scale = a->out_scale; p.sink = a->sink;
     p.sg = make_segments(seg, a->tokens);
@@ -813,12 +997,13 @@ int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
     GqaAttn<float> p;
     fill(p);
     const dim3 grid(a->tokens, (a->H + 3) / 4);
+    auto row = [&](auto one, auto two) { return static_cast<int>(launch(maps == 2 ? two : one, grid, dim3(128), 0, st, p)); };
     switch (a->P / 64) {
-      case 1: return static_cast<int>(launch(gqa_row_kernel<2>, grid, dim3(128), 0, st, p));
-      case 2: return static_cast<int>(launch(gqa_row_kernel<4>, grid, dim3(128), 0, st, p));
-      case 3: return static_cast<int>(launch(gqa_row_kernel<6>, grid, dim3(128), 0, st, p));
+      case 1: return row(gqa_row_kernel<2, 1>, gqa_row_kernel<2, 2>);
+      case 2: return row(gqa_row_kernel<4, 1>, gqa_row_kernel<4, 2>);
+      case 3: return static_cast<int>(launch(gqa_row_kernel<6, 1>, grid, dim3(128), 0, st, p));
     }
-    return static_cast<int>(launch(gqa_row_kernel<8>, grid, dim3(128), 0, st, p));
+    return row(gqa_row_kernel<8, 1>, gqa_row_kernel<8, 2>);
   }
   GqaMma p;
   fill(p.a);
@@ -826,21 +1011,21 @@ int cb_gqa_attn(const CbGqaAttn* a, const CbSegments* seg, void* stream) {
   p.bias_rows = 0;
   p.partial = static_cast<float*>(a->partial);
   if (a->decode) {
-    p.hb = 16; p.qb = 1;
-    p.head_tiles = (a->H / a->G + 15) / 16;
+    p.hb = 16 / maps; p.qb = 1;
+    p.head_tiles = (a->H / a->G + p.hb - 1) / p.hb;
     const dim3 grid(seg->num, a->G * p.head_tiles, p.splits);
     if (grid.y > 65535) return -11;
-    return a->bias ? gqa_mma<true>(p, a->P / 64, true, grid, st) : gqa_mma<false>(p, a->P / 64, true, grid, st);
+    return gqa_mma_any(p, a->P / 64, true, grid, st);
   }
   const int R = a->H / a->G;
-  p.hb = min(R, 16 * kGqaWarps);
-  p.qb = 16 * kGqaWarps / p.hb;
+  p.hb = min(R, 16 * kGqaWarps / maps);
+  p.qb = 16 * kGqaWarps / maps / p.hb;
   p.head_tiles = (R + p.hb - 1) / p.hb;
   const dim3 grid(max_tiles(a->tokens, seg->num, p.qb), a->G * p.head_tiles);
   if (grid.y > 65535) return -11;
   const long long rows = static_cast<long long>(a->bias_far) + 1;
   p.bias_rows = a->bias && rows * p.hb * 4 <= kGqaBiasBytes ? static_cast<int>(rows) : 0;
-  return a->bias ? gqa_mma<true>(p, a->P / 64, false, grid, st) : gqa_mma<false>(p, a->P / 64, false, grid, st);
+  return gqa_mma_any(p, a->P / 64, false, grid, st);
 }
 
 }  // extern "C"

@@ -128,11 +128,11 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, int c, float4 v) {
   reinterpret_cast<uint2*>(p)[c] = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
 }
 
-// x[t] = table[ids[t]] (fp32) and h[t] = x[t] * w / rms(x[t])
+// x[t] = scale * table[ids[t]] (fp32), added to what x[t] holds with `add`, and h[t] = x[t] * w / rms(x[t])
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
 embed_rows_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__ table, const float* __restrict__ w,
-                  float* __restrict__ x, T* __restrict__ h, int ldh, int W, int vocab, float eps) {
+                  float* __restrict__ x, T* __restrict__ h, int ldh, int W, int vocab, float eps, float scale, int add) {
   __shared__ float red[8];
   pdl_wait();
   pdl_launch_dependents();
@@ -144,7 +144,16 @@ embed_rows_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__
   float ss = 0.f;
   if ((W & 3) == 0 && W <= 32 * kRowThreads) {
     Row8 r;
-    r.each(W, [&](int c, float4& v) { v = load4(e, c); ss += dot4(v, v); store4(xr, c, v); });
+    r.each(W, [&](int c, float4& v) {
+      v = load4(e, c);
+      v = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+      if (add) {
+        const float4 u = load4(xr, c);
+        v = make_float4(v.x + u.x, v.y + u.y, v.z + u.z, v.w + u.w);
+      }
+      ss += dot4(v, v);
+      store4(xr, c, v);
+    });
     const float inv = 1.f / sqrtf(row_sum(ss, red) / static_cast<float>(W) + eps);
     r.each(W, [&](int c, float4& v) {
       const float4 g = load4(w, c);
@@ -153,12 +162,12 @@ embed_rows_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__
     return;
   }
   for (int c = threadIdx.x; c < W; c += kRowThreads) {
-    const float v = __bfloat162float(e[c]);
+    const float v = fmaf(__bfloat162float(e[c]), scale, add ? xr[c] : 0.f);
     ss = fmaf(v, v, ss);
     xr[c] = v;
   }
   const float inv = 1.f / sqrtf(row_sum(ss, red) / static_cast<float>(W) + eps);
-  for (int c = threadIdx.x; c < W; c += kRowThreads) hr[c] = from_f<T>(__bfloat162float(e[c]) * inv * w[c]);
+  for (int c = threadIdx.x; c < W; c += kRowThreads) hr[c] = from_f<T>(xr[c] * inv * w[c]);
 }
 
 // x[t] += y[t] * w / rms(y[t]); then, with h, h[t] = x[t] * w2 / rms(x[t]): a normed addition to the residual and the norm that
@@ -585,7 +594,11 @@ struct F32Gemm {
   const float* residual;
   float* y2; int ldy2, n_split, diag_n;
   int M, N, K;
-  int glu;                    // gated silu (1) or gelu (2): 16 gate rows and 16 up rows of w in turn, y gets N / 2 features
+  int glu;                    // gated silu (1), gelu (2) or clamped (3): 16 gate rows and 16 up rows of w in turn, y gets N / 2 features;
+                              // with y2 only the rows below n_split are, and the others leave to y2 as they are
+  float glu_limit;
+  const float* rgate; int ldrg;     // [M, ldrg] or null: a feature times sigmoid(rgate[m, n] + rgate_b[n]) joins the residual
+  const float* rgate_b;       // [N]
   const int* tiles;           // grouped: work list {count, then {expert, first row, up to 64 rows}}, w stacks the experts; null: one matrix
 };
 
@@ -630,7 +643,7 @@ f32_gemm_kernel(const F32Gemm p) {
     }
     __syncthreads();
   }
-  if (p.glu) {
+  if (p.glu && !(p.y2 && n0 >= p.n_split)) {
     // a thread's four columns are gate columns of features f .. f + 3 (tx & 4 clear) or their up columns, which the thread
     // four places on holds
     const int f = (n0 >> 1) + (tx >> 3) * 16 + (tx & 3) * 4;
@@ -639,9 +652,15 @@ f32_gemm_kernel(const F32Gemm p) {
       const int m = m0 + ty * 4 + i;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const float u = __shfl_down_sync(0xffffffffu, acc[i][j], 4);
-        if (!(tx & 4) && m < m_end && f + j < (p.N >> 1))
-          p.y[static_cast<size_t>(m) * p.ldy + f + j] = (p.glu == 1 ? acc[i][j] / (1.f + expf(-acc[i][j])) : gelu_tanh(acc[i][j])) * u;
+        float g = acc[i][j], u = __shfl_down_sync(0xffffffffu, g, 4);
+        if (p.glu == 3) {
+          g = fminf(g, p.glu_limit);
+          u = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
+          u = (u + 1.f) / (1.f + expf(-1.702f * g));
+        } else {
+          g = p.glu == 1 ? g / (1.f + expf(-g)) : gelu_tanh(g);
+        }
+        if (!(tx & 4) && m < m_end && f + j < ((p.y2 ? p.n_split : p.N) >> 1)) p.y[static_cast<size_t>(m) * p.ldy + f + j] = g * u;
       }
     }
     return;
@@ -656,10 +675,14 @@ f32_gemm_kernel(const F32Gemm p) {
       if (n >= p.N) continue;
       float v = acc[i][j];
       if (p.y2 && n >= p.n_split) {
-        v = fmaxf(v, 0.f);
-        p.y2[static_cast<size_t>(m) * p.ldy2 + n - p.n_split] = v * v;
+        if (!p.glu) {
+          v = fmaxf(v, 0.f);
+          v *= v;
+        }
+        p.y2[static_cast<size_t>(m) * p.ldy2 + n - p.n_split] = v;
       } else {
         const size_t o = static_cast<size_t>(m) * p.ldy + n;
+        if (p.rgate) v /= 1.f + expf(-(p.rgate[static_cast<size_t>(m) * p.ldrg + n] + p.rgate_b[n]));
         p.y[o] = p.residual ? v + p.residual[o] : v;
       }
     }
@@ -710,14 +733,14 @@ int cb_concat_rows(const void* x, const void* x0, void* out, int ldo, int n, int
 }
 
 int cb_embed_rows(const void* ids, const void* table, const void* w, void* x, void* h, int ldh, int n, int W, int vocab, float eps,
-                  int f32, void* stream) {
+                  float scale, int add, int f32, void* stream) {
   using namespace cb;
   if (n <= 0) return 0;
   if (W <= 0 || vocab <= 0 || ldh < W || (ldh & 3)) return -10;
   auto go = [&](auto kernel, auto* out) {
     return static_cast<int>(launch(kernel, dim3(n), dim3(kRowThreads), 0, static_cast<cudaStream_t>(stream),
                                    static_cast<const int*>(ids), static_cast<const __nv_bfloat16*>(table),
-                                   static_cast<const float*>(w), static_cast<float*>(x), out, ldh, W, vocab, eps));
+                                   static_cast<const float*>(w), static_cast<float*>(x), out, ldh, W, vocab, eps, scale, add));
   };
   return f32 ? go(embed_rows_kernel<float>, static_cast<float*>(h)) : go(embed_rows_kernel<__nv_bfloat16>, static_cast<__nv_bfloat16*>(h));
 }
@@ -818,6 +841,9 @@ struct CbF32Gemm {
   int M, N, K;
   int glu;
   const void* tiles; int max_items;       // grouped form (see F32Gemm)
+  float glu_limit;
+  const void* rgate; int ldrg;
+  const void* rgate_b;
 };
 
 int cb_f32_gemm(const CbF32Gemm* a, void* stream) {
@@ -834,7 +860,13 @@ int cb_f32_gemm(const CbF32Gemm* a, void* stream) {
   p.glu = a->glu;
   p.tiles = static_cast<const int*>(a->tiles);
   if (p.tiles && (a->max_items <= 0 || a->diag_n || a->glu || a->residual)) return -14;
-  if (p.glu && (p.glu < 1 || p.glu > 2 || p.y2 || p.residual || p.diag_n || (p.N % 32) != 0 || p.ldy < p.N / 2)) return -13;
+  p.glu_limit = a->glu_limit;
+  p.rgate = static_cast<const float*>(a->rgate); p.ldrg = a->ldrg;
+  p.rgate_b = static_cast<const float*>(a->rgate_b);
+  const int glu_rows = p.y2 ? p.n_split : p.N;
+  if (p.glu && (p.glu < 1 || p.glu > 3 || p.residual || p.diag_n || (glu_rows % 32) != 0 || glu_rows > p.N || p.ldy < glu_rows / 2)) return -13;
+  if (p.glu && p.y2 && ((glu_rows % 64) != 0 || p.ldy2 < p.N - glu_rows)) return -15;
+  if (p.rgate && (p.y2 || p.glu || !p.rgate_b || p.ldrg < p.N)) return -16;
   const dim3 grid((a->N + 63) / 64, p.tiles ? a->max_items : (a->M + 63) / 64);
   if (grid.y > 65535) return -12;
   return static_cast<int>(launch(f32_gemm_kernel, grid, dim3(256), 0, static_cast<cudaStream_t>(stream), p));

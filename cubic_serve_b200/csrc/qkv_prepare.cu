@@ -5,8 +5,11 @@
 //                     channels, every query and key head over its root mean square
 //   norm_qkv_kernel   queries and keys of a token over the root mean square of their whole projection, times a weight per channel;
 //                     queries times a factor that grows with the position
+//   head_qkv_kernel   every query and key head, or map of it, over its root mean square, times a weight per channel, rotary positions
+//                     on the halves of its first channels
 //
-// A warp takes a head, lane l the channels 4 l .. and 128 + 4 l ..; everything between the projection and the stored row is fp32.
+// In the first two a warp takes a head, lane l the channels 4 l .. and 128 + 4 l ..; in the last, rows of 32 or 64 columns share a
+// warp.  Everything between the projection and the stored row is fp32.
 #include <type_traits>
 
 #include "segments.cuh"
@@ -375,6 +378,124 @@ norm_qkv_kernel(const NormQkv<T> p) {
   }
 }
 
+template <typename T>
+struct HeadQkv {
+  QkvPrep<T> a;
+  const float* qw;            // [d]
+  const float* kw;
+  const float* freq;          // [2][pairs] radians per position, and what they were rounded by
+  int pairs;
+  const int* positions;
+  int maps;                   // rows of d channels a head consists of; they share its P columns evenly
+  int tokens;
+};
+
+static constexpr int kHeadBatch = 4;        // rows a group of lanes has in flight
+
+// A block takes TOKS tokens and every gridDim.y-th of their rows; L lanes of four channels each take a row of 4 L columns (a query's
+// or key's map) at a time.  Values are copied at the end.
+template <typename T, int L, int TOKS>
+__global__ void __launch_bounds__(32 * kQkvWarps)
+head_qkv_kernel(const HeadQkv<T> p) {
+  using Raw = typename RawFour<T>::type;
+  extern __shared__ __align__(16) float lsm[];                         // cosines [TOKS][hp], sines
+  constexpr int GROUPS = 32 * kQkvWarps / L, COLS = 4 * L;
+  pdl_wait();
+  pdl_launch_dependents();
+  const QkvPrep<T>& a = p.a;
+  const int t_first = blockIdx.x * TOKS, toks = min(TOKS, p.tokens - t_first);
+  const int half = p.pairs, dims = 2 * half, hp = (half + 3) & ~3;
+  float* cosine = lsm;
+  float* sine = lsm + TOKS * hp;
+  for (int i = threadIdx.x; i < toks * half; i += 32 * kQkvWarps) {
+    const int t = TOKS == 1 ? 0 : i / half, j = i - t * half;
+    // the rounding error of the product is put back: angles of far positions keep their fraction of a turn
+    const float pos = static_cast<float>(p.positions[t_first + t]), f = p.freq[j];
+    const float ang = pos * f, e = fmaf(pos, f, -ang) + pos * p.freq[half + j];
+    float sn, cs;
+    sincosf(ang, &sn, &cs);
+    const float ce = fmaf(-0.5f * e, e, 1.f), se = e * fmaf(e * (-1.f / 6.f), e, 1.f);
+    cosine[t * hp + j] = cs * ce - sn * se;
+    sine[t * hp + j] = fmaf(sn, ce, cs * se);
+  }
+  __syncthreads();
+  const int sub = threadIdx.x % L, group = threadIdx.x / L;
+  const int lane0 = (threadIdx.x & 31) - sub;                          // first lane of the group
+  const int c = 4 * sub;
+  const bool vec = a.vec, vec_turn = (half & 3) == 0;
+  const float inv_d = 1.f / static_cast<float>(a.d);
+  const int nq = a.H * p.maps, rows = nq + a.G * p.maps;               // of a token
+  const int stride = GROUPS * gridDim.y, first = blockIdx.y * GROUPS + group;
+  // this lane's weights, and where its channels turn
+  const float4 wq = load_four(p.qw, c, a.d, vec), wk = load_four(p.kw, c, a.d, vec);
+  const bool hi = c >= half;
+  const int low = hi ? c - half : c;
+  // every group makes the same turns: its lanes exchange by shuffles
+  const int units = toks * rows, turns = (units - static_cast<int>(blockIdx.y) * GROUPS + stride * kHeadBatch - 1) / (stride * kHeadBatch);
+  for (int turn = 0; turn < turns; ++turn) {
+    Raw raw[kHeadBatch];
+    int tok[kHeadBatch], row[kHeadBatch];
+#pragma unroll
+    for (int b = 0; b < kHeadBatch; ++b) {
+      const int u = first + (turn * kHeadBatch + b) * stride;
+      const bool ok = u < units;
+      tok[b] = ok ? (TOKS == 1 ? 0 : u / rows) : 0;
+      row[b] = ok ? u - tok[b] * rows : -1;
+      const int r = ok ? row[b] : 0;
+      raw[b] = load_raw(a.x + static_cast<size_t>(t_first + tok[b]) * a.ldx + (r < nq ? a.q_off + r * a.d : a.k_off + (r - nq) * a.d), c, a.d, vec);
+    }
+#pragma unroll
+    for (int b = 0; b < kHeadBatch; ++b) {
+      float4 v = unpack_four(raw[b]);
+      float ss = dot_four(v, v);
+#pragma unroll
+      for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float inv = 1.f / sqrtf(fmaf(ss, inv_d, a.eps));
+      const bool query = row[b] < nq;
+      const float4 w = query ? wq : wk;
+      v = make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w);
+      const float* cs = cosine + tok[b] * hp;
+      const float* sn = sine + tok[b] * hp;
+      if (vec_turn) {                                                  // four channels turn with four neighbours
+        const int other = lane0 + (c < dims ? (hi ? c - half : c + half) >> 2 : sub);
+        const float4 o = make_float4(__shfl_sync(0xffffffffu, v.x, other), __shfl_sync(0xffffffffu, v.y, other),
+                                     __shfl_sync(0xffffffffu, v.z, other), __shfl_sync(0xffffffffu, v.w, other));
+        if (c < dims) {
+          const float sg = hi ? 1.f : -1.f;
+          const float4 x = *reinterpret_cast<const float4*>(cs + low), y = *reinterpret_cast<const float4*>(sn + low);
+          v = make_float4(fmaf(v.x, x.x, sg * o.x * y.x), fmaf(v.y, x.y, sg * o.y * y.y), fmaf(v.z, x.z, sg * o.z * y.z),
+                          fmaf(v.w, x.w, sg * o.w * y.w));
+        }
+      } else {
+        const float4 u = v;
+        float* vp = &v.x;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int ch = c + i;
+          const bool up = ch >= half;
+          const int partner = ch < dims ? (up ? ch - half : ch + half) : ch, from = lane0 + (partner >> 2);
+          const float o0 = __shfl_sync(0xffffffffu, u.x, from), o1 = __shfl_sync(0xffffffffu, u.y, from);
+          const float o2 = __shfl_sync(0xffffffffu, u.z, from), o3 = __shfl_sync(0xffffffffu, u.w, from);
+          if (ch >= dims) continue;
+          const int e = partner & 3, j = up ? ch - half : ch;
+          const float o = e == 0 ? o0 : e == 1 ? o1 : e == 2 ? o2 : o3;
+          vp[i] = fmaf(vp[i], cs[j], (up ? o : -o) * sn[j]);
+        }
+      }
+      if (row[b] < 0) continue;
+      const int r = query ? row[b] : row[b] - nq, head = r / p.maps, map = r - head * p.maps;
+      T* dst = a.row(query ? head : a.H + head, t_first + tok[b], a.slots[t_first + tok[b]]);
+      if (dst) store_four(dst + map * COLS, c, v);
+    }
+  }
+  const int quads = a.P >> 2;                                          // four columns of a value row at a time
+  for (int i = blockIdx.y * 32 * kQkvWarps + threadIdx.x; i < toks * a.G * quads; i += 32 * kQkvWarps * gridDim.y) {
+    const int qd = i % quads, tg = i / quads, g = tg % a.G, t = tg / a.G;
+    T* dst = a.row(a.H + a.G + g, t_first + t, a.slots[t_first + t]);
+    if (dst) store_four(dst, 4 * qd, load_four(a.x + static_cast<size_t>(t_first + t) * a.ldx + a.v_off + g * a.e, 4 * qd, a.e, vec));
+  }
+}
+
 }  // namespace cb
 
 extern "C" {
@@ -404,13 +525,21 @@ struct CbNormQkv {
   float coef; int every;
 };
 
+struct CbHeadQkv {
+  CbQkvPrep a;                // d: channels of a map
+  const void* qw;
+  const void* kw;
+  const void* freq; int pairs;
+  int maps;
+};
+
 }  // extern "C"
 
 namespace cb {
 
-static int qkv_check(const CbQkvPrep& a) {
-  if (a.H <= 0 || a.G <= 0 || a.d <= 0 || a.e <= 0 || a.P < a.d || a.P < a.e || a.P > 256 || (a.P & 63)) return -10;
-  if (a.q_off < 0 || a.k_off < a.q_off + a.H * a.d || a.v_off < a.k_off + a.G * a.d || a.ldx < a.v_off + a.G * a.e) return -11;
+static int qkv_check(const CbQkvPrep& a, int maps = 1) {
+  if (a.H <= 0 || a.G <= 0 || a.d <= 0 || a.e <= 0 || a.P < maps * a.d || a.P < a.e || a.P > 256 || (a.P & 63)) return -10;
+  if (a.q_off < 0 || a.k_off < a.q_off + a.H * maps * a.d || a.v_off < a.k_off + a.G * maps * a.d || a.ldx < a.v_off + a.G * a.e) return -11;
   return 0;
 }
 
@@ -480,6 +609,38 @@ int cb_norm_qkv(const CbNormQkv* c, void* stream) {
     return static_cast<int>(launch(kernel, dim3(c->a.tokens), dim3(32 * kNormWarps), 0, static_cast<cudaStream_t>(stream), p));
   };
   return c->a.f32 ? go(norm_qkv_kernel<float>, NormQkv<float>{}) : go(norm_qkv_kernel<__nv_bfloat16>, NormQkv<__nv_bfloat16>{});
+}
+
+int cb_head_qkv(const CbHeadQkv* c, void* stream) {
+  using namespace cb;
+  if (!c || c->a.tokens <= 0) return 0;
+  if (c->maps < 1 || c->maps > 2) return -12;
+  if (const int rc = qkv_check(c->a, c->maps)) return rc;
+  const int cols = c->a.P / c->maps;
+  if (cols != 32 && cols != 64 && cols != 128) return -14;
+  if (c->pairs < 0 || 2 * c->pairs > c->a.d || !c->qw || !c->kw || (c->pairs && !c->freq)) return -13;
+  // few tokens: a token per block, and more blocks per token
+  const bool single = c->a.tokens < 592;
+  const int toks = single ? 1 : 8, tiles = (c->a.tokens + toks - 1) / toks;
+  const int rows = (c->a.H + c->a.G) * c->maps * toks, groups = 32 * kQkvWarps / (cols / 4);
+  const int ny = min((rows + groups * kHeadBatch - 1) / (groups * kHeadBatch), max(1, 148 * 8 / tiles));
+  const size_t smem = static_cast<size_t>(toks) * 2 * ((c->pairs + 3) & ~3) * 4;
+  auto go = [&](auto kernel, auto p) {
+    using T = std::remove_pointer_t<decltype(p.a.q)>;
+    p.a = qkv_fill<T>(c->a);
+    p.qw = static_cast<const float*>(c->qw); p.kw = static_cast<const float*>(c->kw);
+    p.freq = static_cast<const float*>(c->freq); p.pairs = c->pairs;
+    p.positions = static_cast<const int*>(c->a.positions);
+    p.maps = c->maps; p.tokens = c->a.tokens;
+    return static_cast<int>(launch(kernel, dim3(tiles, ny), dim3(32 * kQkvWarps), smem, static_cast<cudaStream_t>(stream), p));
+  };
+  auto pick = [&](auto p) {
+    using T = std::remove_pointer_t<decltype(p.a.q)>;
+    if (cols == 32) return single ? go(head_qkv_kernel<T, 8, 1>, p) : go(head_qkv_kernel<T, 8, 8>, p);
+    if (cols == 64) return single ? go(head_qkv_kernel<T, 16, 1>, p) : go(head_qkv_kernel<T, 16, 8>, p);
+    return single ? go(head_qkv_kernel<T, 32, 1>, p) : go(head_qkv_kernel<T, 32, 8>, p);
+  };
+  return c->a.f32 ? pick(HeadQkv<float>{}) : pick(HeadQkv<__nv_bfloat16>{});
 }
 
 }  // extern "C"

@@ -426,7 +426,7 @@ wq_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
         const int rows_here = min(p.mb, m_end - m0);
         const int n_base = n_tile * kTileN;
         const bool vec_ok = (p.ldy & 7) == 0 && (p.N & 7) == 0;
-        if (p.swiglu) {
+        if (glu_tile(p, n_tile)) {
           // 64 activation features per tile row: 16 items of four
           for (int idx = dq; idx < rows_here * 16; idx += kNumDequantWarps * 32) {
             const int mm = idx >> 4, j0 = (idx & 15) * 4;
@@ -530,7 +530,7 @@ wq_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
         // L2 (.cg), 8-byte bf16 stores
         const int rows_here = min(p.mb, m_end - m0);
         const int n_base = n_tile * kTileN;
-        if (p.swiglu) {
+        if (glu_tile(p, n_tile)) {
           for (int idx = dq; idx < rows_here * 16; idx += kNumDequantWarps * 32) {
             const int mm = idx >> 4, j0 = (idx & 15) * 4;
             const size_t e = static_cast<size_t>(mm) * kTileN + act_gate_col(j0);
@@ -604,7 +604,7 @@ wq_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
       const int row_lo = rank * chunk, row_hi = min(rows_here, row_lo + chunk);
       const uint32_t stg0 = smem_u32(smem);
       const int n_base = n_tile * kTileN;
-      if (p.swiglu) {
+      if (glu_tile(p, n_tile)) {
         for (int idx = dq; idx < (row_hi - row_lo) * 16; idx += kNumDequantWarps * 32) {
           const int mm = row_lo + (idx >> 4), j0 = (idx & 15) * 4;
           const uint32_t off = static_cast<uint32_t>(mm * kTileN + act_gate_col(j0)) * 4u;
@@ -784,7 +784,11 @@ struct CbWideGemm {
   int ldy2, n_split, diag_n;
   int M, N, K;
   int stream_k, splits, min_units;
-  int glu;                    // gated activation (Glu): w's rows are interleaved, y [M, ldy] gets N / 2 features
+  int glu;                    // gated activation (Glu): w's rows are interleaved, y [M, ldy] gets N / 2 features; with y2 only the
+                              // rows below n_split are, and the others leave to y2 as they are
+  float glu_limit;            // kGluClamped
+  const void* rgate; int ldrg;      // bf16 [M, ldrg] or null: y32 = residual32 + sigmoid(rgate + rgate_b) * product
+  const void* rgate_b;        // fp32 [N]
 };
 
 // Per-launch options of the common launcher.  Everything that steers ONE launch travels in this struct (not in
@@ -938,8 +942,19 @@ static int wq_gemm_dispatch(int fmt, const void* x, int ldx, const void* codes, 
     const CbWideGemm& g = *o.wide;
     if (fmt != kFmtBf16 || residual || link || o.swiglu || o.tiles || g.x_cols <= 0 || g.x_cols > ldx) return -61;
     if ((!g.y && !g.y32) || (g.y && g.y32) || (g.y2 && ((g.n_split & 3) || g.n_split < 0 || (g.y32 && g.residual32)))) return -62;
-    if (g.glu && (!g.y || g.y2 || g.diag_n || g.glu < 0 || g.glu > kGluGelu || (N % 32) != 0 || ldy < N / 2)) return -64;
+    if (g.glu) {
+      const int rows = g.y2 ? g.n_split : N;
+      if (!g.y || g.diag_n || g.glu < 0 || g.glu > kGluClamped || (rows % 32) != 0 || rows > N || ldy < rows / 2) return -64;
+      if (g.y2 && ((rows % kTileN) != 0 || g.ldy2 < N - rows)) return -66;
+    }
+    if (g.rgate && (!g.y32 || g.y2 || !g.rgate_b || g.ldrg < N || (g.ldrg & 3) || (reinterpret_cast<uintptr_t>(g.rgate) & 7) ||
+                    (reinterpret_cast<uintptr_t>(g.rgate_b) & 15)))
+      return -67;
     p.swiglu = g.glu;
+    p.glu_limit = g.glu_limit;
+    p.rgate = static_cast<const __nv_bfloat16*>(g.rgate);
+    p.rgate_b = static_cast<const float*>(g.rgate_b);
+    p.ldrg = g.ldrg;
     if (g.diag_n && (stream_k || g.diag_n < 0 || (g.diag_n % kTileN) != 0)) return -63;
     p.wide = 1;
     p.y32 = static_cast<float*>(g.y32);

@@ -89,8 +89,10 @@ struct WqGemmParams {
   // fused SwiGLU epilogue (gate/up projection): the weight rows were interleaved at load time so that a
   // 128-row tile holds 64 output features as four blocks of {16 gate rows, 16 up rows}; the epilogue writes
   // act[m, 64 * n_tile + 16 * q + i] = silu(tile row 32 q + i) * (tile row 32 q + 16 + i), ldy = row stride of act;
-  // kGluGelu: the tanh form of gelu instead of silu
+  // kGluGelu: the tanh form of gelu instead of silu; kGluClamped: see glu_mul.  With a second buffer y2 the rows from n_split on
+  // (a multiple of the 128-row tile) are not interleaved: they leave there as they are
   int swiglu;
+  float glu_limit;          // kGluClamped
   // persistent kernel on CTA pairs (cta_group::2): the schedule's tile is a PAIR of adjacent weight tiles, CTA rank r of
   // the pair owns weight tile 2 * pair_tile + r and loads batch rows [m0 + r * mb / 2, + mb / 2) of the activation tile
   int pair;
@@ -98,10 +100,14 @@ struct WqGemmParams {
   // tiles through distributed shared memory (no workspace, no fences, no arrival counter)
   int cluster_splitk;
   // wide epilogue (store_wide4): results leave as fp32, added to an fp32 residual stream, or the features from n_split on
-  // leave through the squared relu into a second buffer (a projection whose rows are [mixer inputs | feed-forward up])
+  // leave through the squared relu into a second buffer (a projection whose rows are [mixer inputs | feed-forward up]).  With
+  // `rgate` a feature is multiplied by sigmoid(rgate[m, n] + rgate_b[n]) before it joins the residual
   int wide;
   float* y32;               // fp32 [M, ldy] instead of y
   const float* residual32;  // added to y32 (may be y32 itself)
+  const __nv_bfloat16* rgate;     // [M, ldrg], ldrg a multiple of 4
+  const float* rgate_b;           // [N]
+  int ldrg;
   __nv_bfloat16* y2;        // [M, ldy2]: feature n >= n_split goes to y2[m, n - n_split]
   int ldy2, n_split;        // n_split is a multiple of 4
   // block-diagonal weights (per-tile kernel): weight rows [g diag_n, (g + 1) diag_n) multiply x columns [g K, (g + 1) K);
@@ -162,22 +168,28 @@ __device__ __forceinline__ bool wait_counter_gpu(const uint32_t* p, uint32_t tar
   }
 }
 
-enum Glu : int { kGluNone = 0, kGluSilu = 1, kGluGelu = 2 };
+enum Glu : int { kGluNone = 0, kGluSilu = 1, kGluGelu = 2, kGluClamped = 3 };
 
 // Gated activation on a pair of accumulators, with the rounding points of the unfused path (the projection's output is
 // rounded to bf16, the activation is computed in fp32 from those and rounded once)
-__device__ __forceinline__ float glu_mul(int kind, float g, float u) {
+__device__ __forceinline__ float glu_mul(int kind, float limit, float g, float u) {
   g = __bfloat162float(__float2bfloat16(g));
   u = __bfloat162float(__float2bfloat16(u));
+  if (kind == kGluClamped) {            // the gate is bounded from above, the other factor on both sides and moved by one
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return __fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f);
+  }
   return (kind == kGluGelu ? gelu_tanh_fast(g) : silu_fast(g)) * u;
 }
 // Four consecutive activation features j0..j0+3 (j0 % 4 == 0) of tile `n_tile` for row m from the fp32 gate / up
 // values of the tile row (already scaled by alpha)
 __device__ __forceinline__ void store_act4(const WqGemmParams& p, int m, int n_tile, int j0, const float4 g, const float4 u) {
-  const int n_out = p.N >> 1;
+  const int n_out = (p.y2 ? p.n_split : p.N) >> 1;
   const int n0 = n_tile * 64 + j0;
   if (n0 >= n_out) return;
-  const float a[4] = {glu_mul(p.swiglu, g.x, u.x), glu_mul(p.swiglu, g.y, u.y), glu_mul(p.swiglu, g.z, u.z), glu_mul(p.swiglu, g.w, u.w)};
+  const float a[4] = {glu_mul(p.swiglu, p.glu_limit, g.x, u.x), glu_mul(p.swiglu, p.glu_limit, g.y, u.y),
+                      glu_mul(p.swiglu, p.glu_limit, g.z, u.z), glu_mul(p.swiglu, p.glu_limit, g.w, u.w)};
   __nv_bfloat16* dst = p.y + static_cast<size_t>(m) * p.ldy + n0;
   if ((p.ldy & 3) == 0 && n0 + 3 < n_out) {
     uint2 ov;
@@ -190,6 +202,10 @@ __device__ __forceinline__ void store_act4(const WqGemmParams& p, int m, int n_t
       if (n0 + j < n_out) dst[j] = __float2bfloat16(a[j]);
   }
 }
+// Whether the features of a weight tile leave through the gated activation
+__device__ __forceinline__ bool glu_tile(const WqGemmParams& p, int n_tile) {
+  return p.swiglu && !(p.y2 && n_tile * kTileN >= p.n_split);
+}
 // Four consecutive output features n0..n0+3 (n0 % 4 == 0) of row m, already scaled, through the wide epilogue.
 __device__ __forceinline__ void store_wide4(const WqGemmParams& p, int m, int n0, float (&v)[4]) {
   if (n0 >= p.N) return;
@@ -197,6 +213,23 @@ __device__ __forceinline__ void store_wide4(const WqGemmParams& p, int m, int n0
   const bool second = p.y2 && n0 >= p.n_split;
   if (p.y32 && !second) {
     const size_t off = static_cast<size_t>(m) * p.ldy + n0;
+    if (p.rgate) {
+      const __nv_bfloat16* gr = p.rgate + static_cast<size_t>(m) * p.ldrg + n0;
+      if (whole) {
+        const uint2 u = *reinterpret_cast<const uint2*>(gr);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+        const float4 c = *reinterpret_cast<const float4*>(p.rgate_b + n0);
+        v[0] = __fdividef(v[0], 1.f + __expf(-(a.x + c.x)));
+        v[1] = __fdividef(v[1], 1.f + __expf(-(a.y + c.y)));
+        v[2] = __fdividef(v[2], 1.f + __expf(-(b.x + c.z)));
+        v[3] = __fdividef(v[3], 1.f + __expf(-(b.y + c.w)));
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (n0 + j < p.N) v[j] = __fdividef(v[j], 1.f + __expf(-(__bfloat162float(gr[j]) + p.rgate_b[n0 + j])));
+      }
+    }
     if (whole && (p.ldy & 3) == 0) {
       float4 o = make_float4(v[0], v[1], v[2], v[3]);
       if (p.residual32) {
@@ -213,7 +246,10 @@ __device__ __forceinline__ void store_wide4(const WqGemmParams& p, int m, int n0
   }
   __nv_bfloat16* dst;
   bool vec;
-  if (second) {
+  if (second && p.swiglu) {
+    dst = p.y2 + static_cast<size_t>(m) * p.ldy2 + (n0 - p.n_split);
+    vec = (p.ldy2 & 3) == 0;
+  } else if (second) {
     // the projection is rounded to bf16 before the activation, as a separate activation kernel would read it
 #pragma unroll
     for (int j = 0; j < 4; ++j) {

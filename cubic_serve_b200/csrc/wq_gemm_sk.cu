@@ -298,7 +298,7 @@ __device__ __forceinline__ void sk_reduce_write(const WqGemmParams& p, const SkS
   const int parts = seg.parts;
   const int own_part = own ? seg.part : -1;
   const float* slots = p.workspace + static_cast<size_t>(g_first) * 2 * part_elems;   // part q > 0 at + q * stride * part_elems
-  if (p.swiglu) {
+  if (glu_tile(p, n_base / kTileN)) {
     sk_reduce_write_act(p, slots, parts, own_part, own, tid, nthreads, m0, row_lo, row_hi, n_base / kTileN);
     return;
   }
@@ -618,7 +618,7 @@ wq_gemm_sk_kernel(const __grid_constant__ CUtensorMap tmap_x,
       tail_bar();
       bool finalized = whole;
       if (whole) {
-        if (ok && p.swiglu) {
+        if (ok && glu_tile(p, n_base / kTileN)) {
           for (int idx = tt; idx < rows_here * 16; idx += nthr) {
             const int mm = idx >> 4, j0 = (idx & 15) * 4;
             const float* gp = stg + mm * kTileN + act_gate_col(j0);
@@ -850,7 +850,7 @@ wq_gemm_sk_kernel(const __grid_constant__ CUtensorMap tmap_x,
 #pragma unroll
             for (int j = 0; j < 16; ++j) scr[j * 32 + lane] = __uint_as_float(acc[j]);
             __syncwarp();
-            if (whole && p.swiglu) {
+            if (whole && glu_tile(p, n_base / kTileN)) {
               // this warp's 32 tile rows are 16 gate + 16 up rows of the same 16 features: lane L owns rows
               // (L >> 2) + 8 i, features 4 (L & 3) .. + 3 (all 32 lanes busy, 32 contiguous bytes per row)
               const int a4 = (lane & 3) * 4;

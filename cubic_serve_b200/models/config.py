@@ -293,6 +293,7 @@ def _layered(name: str):
     return layered.NAMED[name]()
 
 
-for _name in ("layered-tiny", "layered-8b", "layered-seq-tiny", "layered-seq-8b", "layered-streams-tiny", "layered-streams-moe"):
+for _name in ("layered-tiny", "layered-8b", "layered-seq-tiny", "layered-seq-8b", "layered-streams-tiny", "layered-streams-moe",
+              "layered-gated-tiny", "layered-gated-8b"):
     NAMED_CONFIGS[_name] = lambda name=_name: _layered(name)
 NAMED_CONFIGS["qwen4-exp-tiny"] = _qwen4_exp_tiny          # served by the eager executor of ``models/qwen4_exp.py``

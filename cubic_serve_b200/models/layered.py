@@ -10,22 +10,29 @@ the layers of an architecture have in common is its entry in ``DESIGNS``:
   {dim} adds, after the feed-forward, what the layer takes from its part of a second embedding of the token;
 * ``Vimelorn``: sequential sublayers on ``streams`` residual streams (hyper-connections: every sublayer reads a weighted sum of
   them, its result is added to all of them while they are mixed), scaled embedding; feed-forwards are dense or routed: experts
-  chosen by score plus correction, some of which return the token itself, and a gated shared expert.
+  chosen by score plus correction, some of which return the token itself, and a gated shared expert;
+* ``Fovunex``: sequential layers whose results pass a gate per channel that reads the same normed input, norms with one number,
+  scaled embedding, clamped gated feed-forward; a loop, before whose later passes the embedding output is added again.
 
 Mixers (another one is a spec, a reader in ``_MIXER_READERS``, an inventory entry, a ``_pack_*`` function and a method of
 ``models/layered_runner.py``):
 
 * ``delta`` / ``channel_delta``: short convolution, gated delta rule with one decay per head / per (head, key channel);
-* ``latent_attention``: attention over cached latents with a sliding window and a gate per head;
+* ``latent_attention``: attention over cached latents, with a sliding window, low-rank queries and a gate per head (``Bumodra``), or
+  with a rotated key part that all heads share (``Fovunex``);
 * ``mamba2``: short convolution, scalar-decay linear recurrence (state-space duality), gated norm in equal parts;
 * ``parallel``: two mixers that read the same norm, each scaled: sliding-window grouped-query attention with head norms,
   rotary pairs, a softmax sink and values that are the raw keys; and gated linear attention with a decay per key channel;
-* ``attention``: short convolutions of q, k and v, rotary halves, unit root mean squares, a window beside kept first tokens;
-* ``attention_2``: q and k normed over their whole projections, queries warmer with their position, a bias per distance and head.
+* ``attention``: short convolutions of q, k and v, rotary halves, unit root mean squares, a window beside kept first tokens
+  (``Vimelorn``); or the difference of two attention maps over the same values inside chunks of positions, heads normed and gated
+  (``Fovunex``);
+* ``attention_2``: q and k normed over their whole projections, queries warmer with their position, a bias per distance and head;
+* ``mingru``: an element-wise recurrence whose gate and candidate read the current token only.
 
 ONE matrix holds all projections that read a layer's norm and ONE the output projections side by side, whatever the mixer is:
-with parallel layers the first also has the feed-forward's up rows and the second its down columns ([o | down]).  Rows and
-columns are padded with zeros to what the GEMM asks for.
+with parallel layers the first also has the feed-forward's up rows and the second its down columns ([o | down]); with gated
+residuals the matrices that read a norm end with the rows of the gate.  Rows and columns are padded with zeros to what the GEMM
+asks for.
 """
 from __future__ import annotations
 
@@ -42,24 +49,34 @@ from .config import QuantSpec
 
 MAX_CONV_TAPS, MAX_DELTA_DIM, MAX_LATENT, MAX_HEAD = 16, 256, 1024, 256      # limits of the kernels
 MAX_STREAMS, MAX_ROUTER, MAX_TOP = 8, 256, 32
+LATENT_WIDTHS = ((64, 64), (128, 128), (192, 128), (256, 256), (320, 256), (512, 512), (576, 512))   # of latent_attn.cu
 
 
 @dataclass(frozen=True)
 class Design:
     """What the layers of an architecture have in common."""
-    mixers: tuple[str, ...]
+    mixers: dict[str, str]       # type in ``config.json`` -> entry of ``_MIXER_READERS``
     sequential: bool             # mixer and feed-forward one after the other, each with a norm; else in parallel behind one
     norm_offset: float           # a norm's factor is this plus its stored weight
     embed_norm: bool             # the embedding is normed before the first layer
     tied_head: bool              # the output head is the embedding table
-    ff: str                      # "squared_relu" (up, down) or gated (gate, up, down): "gelu_glu", "silu_glu"
-    streams: bool = False        # several residual streams, a scaled embedding, routed feed-forwards
+    ff: str                      # "squared_relu" (up, down) or gated (gate, up, down): "gelu_glu", "silu_glu", "clamped_glu"
+    streams: bool = False        # several residual streams, routed feed-forwards
+    embed_scale: bool = False    # the embedding is scaled
+    scalar_norm: bool = False    # a norm of the residual has one number for all channels
+    gated: bool = False          # a sublayer's result passes a sigmoid gate per channel that reads the sublayer's input
+    loop: str = ""               # a loop of layers: passes start with a projection of [residual ; embedding output] ("project"),
+                                 # or later passes with their sum ("add"); "": none
 
 
 DESIGNS = {
-    "Bumodra": Design(("delta", "channel_delta", "latent_attention"), False, 1.0, True, False, "squared_relu"),
-    "Loduzen": Design(("parallel", "mamba2"), True, 0.0, False, True, "gelu_glu"),
-    "Vimelorn": Design(("attention", "attention_2"), True, 0.0, False, False, "silu_glu", True),
+    "Bumodra": Design({"delta": "delta", "channel_delta": "channel_delta", "latent_attention": "latent"}, False, 1.0, True, False,
+                      "squared_relu", loop="project"),
+    "Loduzen": Design({"parallel": "parallel", "mamba2": "mamba2"}, True, 0.0, False, True, "gelu_glu"),
+    "Vimelorn": Design({"attention": "conv_attention", "attention_2": "biased_attention"}, True, 0.0, False, False, "silu_glu",
+                       streams=True, embed_scale=True),
+    "Fovunex": Design({"latent_attention": "rotated_latent", "attention": "differential", "mingru": "mingru"}, True, 0.0, False, False,
+                      "clamped_glu", embed_scale=True, scalar_norm=True, gated=True, loop="add"),
 }
 ARCHITECTURES = tuple(DESIGNS)
 
@@ -132,47 +149,88 @@ class DeltaSpec(MixerSpec):
 
 
 @dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions on the first ``dims`` channels.  ``scaling``: as ``ModelConfig.rope_scaling``; the attention factor of
+    ``yarn`` multiplies cosine and sine here."""
+    dims: int
+    base: float
+    scaling: tuple | None = None
+
+    def validate(self, width: int) -> None:
+        if self.dims % 2 or not 0 <= self.dims <= width or self.base <= 0:
+            raise LayeredConfigError("rotary channels come in pairs inside a head")
+
+    def _exact(self) -> torch.Tensor:
+        return rope_inv_freq(self.dims, self.base, scaling=self.scaling, dtype=torch.float64)
+
+    @property
+    def factor(self) -> float:
+        """On cosine and sine."""
+        return float(self.scaling[5]) if self.scaling and self.scaling[0] == "yarn" else 1.0
+
+    def table(self) -> tuple[torch.Tensor, float]:
+        """(fp32 radians per position of every pair, factor on cosine and sine)."""
+        return self._exact().float(), self.factor
+
+    def split_table(self) -> torch.Tensor:
+        """fp32 ``[2, pairs]``: radians per position, and what rounding took from them."""
+        exact = self._exact()
+        return torch.stack([exact.float(), (exact - exact.float().double()).float()])
+
+
+@dataclass(frozen=True)
 class LatentSpec(MixerSpec):
     heads: int
     dim: int
     vdim: int
-    q_rank: int
+    q_rank: int                  # inner size of the low-rank query projection; 0: one full matrix
     kv_rank: int
     scale: float
     window: int = 0              # 0: every earlier token
+    rot_dim: int = 0             # rotated channels of a query head, beside ``dim``; the rotated key is shared by all heads
+    rotary: RotarySpec | None = None
+    gated: bool = True           # a sigmoid gate per head
     label = "latent"
 
     def page_bytes(self, act_bytes: int) -> int:
-        return 16 * self.rank_padded * act_bytes
+        return 16 * self.row_padded * act_bytes
+
+    @property
+    def rot_col(self) -> int:
+        """Column of the rotated part in a cached row, behind the latent."""
+        return round_up(self.kv_rank, 8) if self.rot_dim else self.kv_rank
+
+    @property
+    def _padded(self) -> tuple[int, int]:
+        """Columns of (a cached row, its latent part read as values): pairs the attention kernels are built for."""
+        for row, rank in LATENT_WIDTHS:
+            if self.rot_col + self.rot_dim <= row and self.kv_rank <= rank:
+                return row, rank
+        return MAX_LATENT, MAX_LATENT
+
+    @property
+    def row_padded(self) -> int:
+        return self._padded[0]
 
     @property
     def rank_padded(self) -> int:
-        """Columns of a cached latent: the widths the attention kernels are built for."""
-        return next((p for p in (64, 128, 256, 512) if self.kv_rank <= p), MAX_LATENT)
+        return self._padded[1]
 
     @property
     def out_width(self) -> int:
         return self.heads * self.vdim
 
     def validate(self) -> None:
-        if min(self.heads, self.dim, self.vdim, self.q_rank, self.kv_rank) <= 0 or self.window < 0:
+        if min(self.heads, self.dim, self.vdim, self.kv_rank) <= 0 or min(self.q_rank, self.window, self.rot_dim) < 0:
             raise LayeredConfigError("latent attention sizes are positive")
-        if self.kv_rank > MAX_LATENT:
-            raise LayeredConfigError(f"latents of up to {MAX_LATENT} channels are served")
-
-
-@dataclass(frozen=True)
-class RotarySpec:
-    """Rotary positions on neighbouring channel pairs of the first ``dims`` channels.  ``scaling``: as
-    ``ModelConfig.rope_scaling``; the attention factor of ``yarn`` multiplies cosine and sine here."""
-    dims: int
-    base: float
-    scaling: tuple | None = None
-
-    def table(self) -> tuple[torch.Tensor, float]:
-        """(fp32 radians per position of every pair, factor on cosine and sine)."""
-        f = rope_inv_freq(self.dims, self.base, scaling=self.scaling, dtype=torch.float64).float()
-        return f, float(self.scaling[5]) if self.scaling and self.scaling[0] == "yarn" else 1.0
+        if self.rot_col + self.rot_dim > MAX_LATENT or self.rot_dim > MAX_HEAD:
+            raise LayeredConfigError(f"latents of up to {MAX_LATENT} channels with their rotated part are served")
+        if bool(self.rot_dim) != (self.rotary is not None):
+            raise LayeredConfigError("rotated channels and their frequencies come together")
+        if self.rotary is not None:
+            self.rotary.validate(self.rot_dim)
+            if self.rotary.dims != self.rot_dim:
+                raise LayeredConfigError("the rotated part of latent attention is rotated as a whole")
 
 
 @dataclass(frozen=True)
@@ -204,9 +262,7 @@ class AttentionSpec(MixerSpec):
             raise LayeredConfigError("attention heads are grouped evenly over positive key head counts and sizes")
         if self.dim > MAX_HEAD:
             raise LayeredConfigError(f"attention heads of up to {MAX_HEAD} channels are served")
-        r = self.rotary
-        if r.dims % 2 or not 0 <= r.dims <= self.dim or r.base <= 0:
-            raise LayeredConfigError("rotary channels come in pairs inside a head")
+        self.rotary.validate(self.dim)
 
 
 @dataclass(frozen=True)
@@ -364,11 +420,9 @@ class ConvAttentionSpec(_QkvSpec):
 
     def validate(self) -> None:
         super().validate()
-        r = self.rotary
         if not 1 <= self.conv <= MAX_CONV_TAPS:
             raise LayeredConfigError(f"attention takes 1 to {MAX_CONV_TAPS} convolution taps")
-        if r.dims % 2 or not 0 <= r.dims <= self.dim or r.base <= 0:
-            raise LayeredConfigError("rotary channels come in pairs inside a head")
+        self.rotary.validate(self.dim)
         if self.window < 0 or self.keep < 0:
             raise LayeredConfigError("an attention window and the tokens kept before it are not negative")
 
@@ -413,7 +467,64 @@ class BiasedAttentionSpec(_QkvSpec):
             raise LayeredConfigError("the query factor grows every positive number of positions")
 
 
-ATTENTION_SPECS = (LatentSpec, AttentionSpec, ConvAttentionSpec, BiasedAttentionSpec)
+@dataclass(frozen=True)
+class DifferentialSpec(_QkvSpec):
+    """Two attention maps per head over the same values: the second's output times a learned factor is taken from the first's, the
+    difference normed per head and gated per channel.  Head norms and rotary halves on every map; ``chunk``: a token sees its own
+    chunk of positions only."""
+    heads: int
+    kv_heads: int
+    dim: int                     # of a map
+    vdim: int
+    scale: float
+    rotary: RotarySpec
+    diff: float                  # constant part of the factor
+    chunk: int = 0               # 0: every earlier token
+    label = "differential"
+
+    @property
+    def width_padded(self) -> int:
+        """Columns of a cached key (both maps, half of them each) or value: the widths the kernels are built for."""
+        return next((p for p in (64, 128) if max(2 * self.dim, self.vdim) <= p), 256)
+
+    @property
+    def offsets(self) -> tuple[int, int, int]:
+        k = round_up(self.heads * 2 * self.dim, 8)
+        return 0, k, k + round_up(self.kv_heads * 2 * self.dim, 8)
+
+    def validate(self) -> None:
+        super().validate()
+        if 2 * self.dim > MAX_HEAD:
+            raise LayeredConfigError(f"maps of up to {MAX_HEAD // 2} channels are served")
+        self.rotary.validate(self.dim)
+        if self.chunk < 0:
+            raise LayeredConfigError("a chunk holds a positive number of positions")
+
+
+@dataclass(frozen=True)
+class MinGruSpec(MixerSpec):
+    """Element-wise recurrence of ``width`` channels: ``S <- (1 - z) S + z candidate``, gate and candidate from the current token."""
+    width: int
+    label = "mingru"
+
+    @property
+    def out_width(self) -> int:
+        return self.width
+
+    @property
+    def padded(self) -> int:
+        """Channels of the state: whole 16-byte rows."""
+        return round_up(self.width, 4)
+
+    def state_bytes(self, act_bytes: int) -> int:
+        return self.padded * 4
+
+    def validate(self) -> None:
+        if self.width <= 0:
+            raise LayeredConfigError("a recurrence has a positive width")
+
+
+ATTENTION_SPECS = (LatentSpec, AttentionSpec, ConvAttentionSpec, BiasedAttentionSpec, DifferentialSpec)
 
 
 @dataclass(frozen=True)
@@ -443,6 +554,7 @@ class LayerSpec:
     mixer: MixerSpec
     ff: int = 0                  # feed-forward width; 0 = none
     routed: RoutedSpec | None = None     # instead of a dense feed-forward
+    limit: float = 0.0           # of a clamped feed-forward
 
     @property
     def has_ff(self) -> bool:
@@ -499,6 +611,10 @@ class LayeredConfig:
         return (tuple((i, False) for i in range(a)) + tuple((i, i == a) for _ in range(times) for i in range(a, b))
                 + tuple((i, False) for i in range(b, n)))
 
+    def reenters(self, run: int) -> bool:
+        """Whether a later pass of the loop, one that adds the embedding output, starts right before this layer run."""
+        return self.design.loop == "add" and self.runs[run][1] and run > self.loop[0]
+
     @property
     def page_bytes(self) -> int:
         """One 16-token page of every attention run."""
@@ -526,14 +642,16 @@ class LayeredConfig:
             l.mixer.validate()
             if l.ff < 0 or l.ff and l.routed:
                 raise LayeredConfigError("feed-forward widths are positive")
+            if l.ff and self.design.ff == "clamped_glu" and l.limit <= 0:
+                raise LayeredConfigError("a clamped feed-forward has a positive limit")
             if l.routed is not None:
                 if not self.design.streams:
                     raise LayeredConfigError(f"{self.architecture} layers have dense feed-forwards")
                 l.routed.validate()
         if not 1 <= self.streams <= MAX_STREAMS or self.streams > 1 and not self.design.streams:
             raise LayeredConfigError(f"1 to {MAX_STREAMS} residual streams are served, more than one in designs that mix them")
-        if self.side_dim < 0 or (self.side_dim or self.design.sequential) and self.loop is not None:
-            raise LayeredConfigError("sequential layers are run once, and the side input of a layer has a positive width")
+        if self.side_dim < 0 or (self.side_dim or not self.design.loop) and self.loop is not None:
+            raise LayeredConfigError("layers of this design are run once, and the side input of a layer has a positive width")
         if self.loop is not None:
             a, b, times = self.loop
             if not 0 <= a < b <= self.num_layers or times < 1:
@@ -542,15 +660,23 @@ class LayeredConfig:
     def to_config(self) -> dict:
         """The ``config.json`` object of this configuration."""
         layers = [{**dict(zip(("type", "mixer"), _mixer_config(l.mixer))), "mlp": _ff_config(l)} for l in self.layers]
+        loop = None if self.loop is None else dict(zip(("start", "stop", "times"), self.loop))
         out = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
                "norm": {"eps": self.rms_eps}, "layers": layers}
+        if self.design.embed_scale:
+            out["embedding"] = {"scale": self.embed_scale}
         if self.design.streams:
-            out.update(streams=self.streams, embedding={"scale": self.embed_scale})
-        elif self.design.sequential:
-            out["token_side"] = {"dim": self.side_dim} if self.side_dim else None
+            out["streams"] = self.streams
+        elif self.design.loop:
+            out["loop"] = loop
         else:
-            out["loop"] = None if self.loop is None else dict(zip(("start", "stop", "times"), self.loop))
+            out["token_side"] = {"dim": self.side_dim} if self.side_dim else None
         return out
+
+
+def _rotary_config(r: RotarySpec) -> dict:
+    scaling = {"scaling": dict(zip(("factor", "original", "fast", "slow"), r.scaling[1:5]))} if r.scaling else {}
+    return {"dims": r.dims, "base": r.base, **scaling}
 
 
 def _mask_config(window: int) -> dict | None:
@@ -560,7 +686,8 @@ def _mask_config(window: int) -> dict | None:
 def _ff_config(l: LayerSpec) -> dict | None:
     """Feed-forward object of a layer's entry in ``config.json``."""
     if l.routed is None:
-        return {"kind": "dense", "ff": l.ff} if l.ff else None
+        limit = {"limit": l.limit} if l.limit else {}
+        return {"kind": "dense", "ff": l.ff, **limit} if l.ff else None
     r = l.routed
     return {"kind": "moe", "expert": {"ff": r.ff}, "router": {"experts": r.experts, "identity": r.identity, "top": r.top},
             "shared": {"ff": r.shared_ff} if r.shared_ff else None}
@@ -570,6 +697,9 @@ def _mixer_config(m: MixerSpec) -> tuple[str, dict]:
     """(type, mixer object) of a layer's entry in ``config.json``."""
     if isinstance(m, DeltaSpec):
         return m.label, {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv}
+    if isinstance(m, LatentSpec) and m.rot_dim:
+        return "latent_attention", {"heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank,
+                                    "scale": m.scale, "rot": _rotary_config(m.rotary)}
     if isinstance(m, LatentSpec):
         return "latent_attention", {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "q_rank": m.q_rank, "kv_rank": m.kv_rank,
                                     "scale": m.scale, "mask": _mask_config(m.window)}
@@ -584,9 +714,13 @@ def _mixer_config(m: MixerSpec) -> tuple[str, dict]:
         return "attention_2", {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
                                "bias_max": m.bias_max,
                                "q_temp": {"coef": m.temp_coef, "every": m.temp_every} if m.temp_every else None}
-    a, g, sc = m.left, m.right, m.left.rotary.scaling
-    rot = {"dims": a.rotary.dims, "base": a.rotary.base,
-           "scaling": dict(zip(("factor", "original", "fast", "slow"), sc[1:5])) if sc else None}
+    if isinstance(m, DifferentialSpec):
+        return "attention", {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale, "diff": m.diff,
+                             "rot": _rotary_config(m.rotary), "mask": _mask_config(m.chunk)}
+    if isinstance(m, MinGruSpec):
+        return "mingru", {"width": m.width}
+    a, g = m.left, m.right
+    rot = {"scaling": None, **_rotary_config(a.rotary)}
     return "parallel", {"left": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.dim, "scale": a.scale,
                                  "mask": _mask_config(a.window), "rot": rot},
                         "right": {"heads": g.heads, "dim": g.dim, "vdim": g.vdim, "tau": g.tau},
@@ -628,6 +762,20 @@ def _read_latent(m: dict, p: str, rank) -> LatentSpec:
                       _window(m))
 
 
+def _read_rotated_latent(m: dict, p: str, rank) -> LatentSpec:
+    return LatentSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), 0, int(m["kv_rank"]), float(m["scale"]), 0, int(m["rot_dim"]),
+                      _read_rotary(m["rot"]), False)
+
+
+def _read_differential(m: dict, p: str, rank) -> DifferentialSpec:
+    return DifferentialSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                            _read_rotary(m.get("rot")), float(m["diff"]), _window(m))
+
+
+def _read_mingru(m: dict, p: str, rank) -> MinGruSpec:
+    return MinGruSpec(int(m["width"]))
+
+
 def _read_mamba2(m: dict, p: str, rank) -> SsdSpec:
     return SsdSpec(int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["groups"]), int(m["conv"]), int(m["norm_groups"]))
 
@@ -661,7 +809,7 @@ def _read_ff(mlp: dict | None, i: int, d: Design) -> dict:
         return {}
     kind = mlp.get("kind")
     if kind == "dense":
-        return {"ff": int(mlp["ff"])}
+        return {"ff": int(mlp["ff"]), **({"limit": float(mlp["limit"])} if d.ff == "clamped_glu" else {})}
     if kind != "moe" or not d.streams:
         raise LayeredConfigError(f"layer {i}: unknown feed-forward {kind!r}")
     r, shared = mlp["router"], mlp.get("shared")
@@ -670,8 +818,9 @@ def _read_ff(mlp: dict | None, i: int, d: Design) -> dict:
 
 
 _MIXER_READERS = {"delta": _read_delta, "channel_delta": lambda m, p, rank: _read_delta(m, p, rank, True),
-                  "latent_attention": _read_latent, "mamba2": _read_mamba2, "parallel": _read_parallel,
-                  "attention": _read_conv_attention, "attention_2": _read_biased_attention}
+                  "latent": _read_latent, "rotated_latent": _read_rotated_latent, "mamba2": _read_mamba2, "parallel": _read_parallel,
+                  "conv_attention": _read_conv_attention, "biased_attention": _read_biased_attention,
+                  "differential": _read_differential, "mingru": _read_mingru}
 
 
 def parse_layered_config(raw: dict, shapes: dict[str, tuple[int, ...]] | None = None, name: str = "") -> LayeredConfig:
@@ -691,15 +840,17 @@ def parse_layered_config(raw: dict, shapes: dict[str, tuple[int, ...]] | None = 
     for i, l in enumerate(raw["layers"]):
         if l["type"] not in DESIGNS[arch].mixers:
             raise LayeredConfigError(f"layer {i}: unknown mixer {l['type']!r}")
-        mixer = _MIXER_READERS[l["type"]](l["mixer"], f"l{i}.mix", rank)
+        mixer = _MIXER_READERS[DESIGNS[arch].mixers[l["type"]]](l["mixer"], f"l{i}.mix", rank)
         layers.append(LayerSpec(mixer, **_read_ff(l.get("mlp"), i, DESIGNS[arch])))
     loop, side = raw.get("loop"), raw.get("token_side")
-    streams = {}
+    more = {}
     if DESIGNS[arch].streams:
-        streams = dict(streams=int(raw.get("streams") or 1), embed_scale=float((raw.get("embedding") or {}).get("scale", 1.0)))
+        more["streams"] = int(raw.get("streams") or 1)
+    if DESIGNS[arch].embed_scale:
+        more["embed_scale"] = float((raw.get("embedding") or {}).get("scale", 1.0))
     cfg = LayeredConfig(name or arch, int(raw["vocab"]), int(raw["width"]), tuple(layers), float(raw["norm"]["eps"]),
                         (int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None, architecture=arch,
-                        side_dim=int(side["dim"]) if side else 0, **streams)
+                        side_dim=int(side["dim"]) if side else 0, **more)
     cfg.validate()
     return cfg
 
@@ -722,6 +873,16 @@ def _mixer_shapes(m: MixerSpec, p: str, W: int) -> dict[str, tuple[int, ...]]:
                         f"{p}.g1": (m.gate_rank, W), f"{p}.g2": (m.heads * m.vdim, m.gate_rank)})
         else:
             out.update({f"{p}.a": (m.heads, W), f"{p}.dt_bias": (m.heads,), f"{p}.g": (m.heads * m.vdim, W)})
+    elif isinstance(m, LatentSpec) and m.rot_dim:
+        out.update({f"{p}.q": (m.heads * (m.dim + m.rot_dim), W), f"{p}.dkv": (m.kv_rank + m.rot_dim, W), f"{p}.dkv.norm": (m.kv_rank,),
+                    f"{p}.uk": (m.heads * m.dim, m.kv_rank), f"{p}.uv": (m.heads * m.vdim, m.kv_rank)})
+    elif isinstance(m, DifferentialSpec):
+        out.update({f"{p}.q": (m.heads * 2 * m.dim, W), f"{p}.k": (m.kv_heads * 2 * m.dim, W), f"{p}.v": (m.kv_heads * m.vdim, W),
+                    f"{p}.g": (m.out_width, W)})
+        out.update({f"{p}.{t}": (m.dim,) for t in ("q.norm", "k.norm", "lq1", "lk1", "lq2", "lk2")})
+    elif isinstance(m, MinGruSpec):
+        out.update({f"{p}.{t}": (m.width, W) for t in "zxg"})
+        out.update({f"{p}.{t}.b": (m.width,) for t in "zx"})
     elif isinstance(m, LatentSpec):
         out.update({f"{p}.dq": (m.q_rank, W), f"{p}.dq.norm": (m.q_rank,), f"{p}.uq": (m.heads * m.dim, m.q_rank),
                     f"{p}.dkv": (m.kv_rank, W), f"{p}.dkv.norm": (m.kv_rank,), f"{p}.uk": (m.heads * m.dim, m.kv_rank),
@@ -751,20 +912,24 @@ def _mixer_shapes(m: MixerSpec, p: str, W: int) -> dict[str, tuple[int, ...]]:
 def tensor_shapes(cfg: LayeredConfig) -> dict[str, tuple[int, ...]]:
     """Every tensor of a checkpoint of this configuration."""
     W, d = cfg.hidden_size, cfg.design
-    out: dict[str, tuple[int, ...]] = {"embed": (cfg.vocab_size, W), "final.norm": (W,)}
+    norm = () if d.scalar_norm else (W,)
+    out: dict[str, tuple[int, ...]] = {"embed": (cfg.vocab_size, W), "final.norm": norm}
     if d.embed_norm:
         out["embed.norm"] = (W,)
     if not d.tied_head:
         out["head"] = (cfg.vocab_size, W)
-    if cfg.loop is not None:
+    if cfg.loop is not None and d.loop == "project":
         out["loop.in"] = (W, 2 * W)
     if cfg.side_dim:
         out["side.embed"] = (cfg.vocab_size, cfg.num_layers * cfg.side_dim)
     for i, l in enumerate(cfg.layers):
-        out[f"l{i}.norm1"] = (W,)
+        out[f"l{i}.norm1"] = norm
         out.update(_mixer_shapes(l.mixer, f"l{i}.mix", W))
         if d.sequential and l.has_ff:
-            out[f"l{i}.norm2"] = (W,)
+            out[f"l{i}.norm2"] = norm
+        if d.gated:
+            for q in (1, 2) if l.has_ff else (1,):
+                out.update({f"l{i}.rg{q}": (W, W), f"l{i}.rg{q}.b": (W,)})
         if d.streams:
             for q in (1, 2) if l.has_ff else (1,):
                 out.update({f"l{i}.hc{q}.in": (cfg.streams,), f"l{i}.hc{q}.out": (cfg.streams,),
@@ -795,7 +960,7 @@ def check_inventory(cfg: LayeredConfig, shapes: dict[str, tuple[int, ...]]) -> N
         if tuple(shapes[n]) != s:
             raise LayeredConfigError(f"{n}: shape {tuple(shapes[n])}, expected {s}")
     idle = {f"l{i}.{t}" for i, l in enumerate(cfg.layers) if cfg.design.sequential and not l.has_ff
-            for t in ("norm2", "hc2.in", "hc2.out", "hc2.mix")}
+            for t in ("norm2", "hc2.in", "hc2.out", "hc2.mix", "rg2", "rg2.b")}
     extra = sorted(set(shapes) - set(want) - idle)
     if extra:
         raise LayeredConfigError(f"checkpoint has {len(extra)} tensors this configuration does not own, e.g. {extra[:3]}")
@@ -818,8 +983,10 @@ def random_tensors(cfg: LayeredConfig, seed: int = 0, device="cpu") -> dict[str,
             t = 0.5 * z
         elif last == "correction":
             t = 0.02 * z
-        elif n == "embed" and cfg.design.streams:
+        elif n == "embed" and cfg.design.embed_scale:
             t = z / cfg.embed_scale
+        elif last in ("lq1", "lk1", "lq2", "lk2"):
+            t = 0.3 * z / s[0] ** 0.25
         elif last == "A_log":
             t = 0.5 * z - 2.0
         elif last in ("dt_bias", "b") and len(s) == 1:
@@ -897,13 +1064,18 @@ class DeltaWeights:
 @dataclass
 class LatentWeights:
     spec: LatentSpec
-    q_norm: torch.Tensor
+    q_norm: torch.Tensor | None      # low-rank queries
     c_norm: torch.Tensor
-    uq: wq_pack.PackedWeight         # rows in the column layout of ``absorb``'s input
+    uq: wq_pack.PackedWeight | None  # rows in the column layout of ``absorb``'s input; None: the projection writes them at ``q_off``
     absorb: BlockDiagonal            # queries -> latent space
     value: BlockDiagonal             # latent outputs -> head outputs
     c_off: int
-    g_off: int
+    g_off: int = -1                  # gates of the heads (< 0: none)
+    q_off: int = 0                   # low-rank queries, or full ones
+    qr_off: int = 0                  # rotated part of the queries [H, rot_dim]
+    r_off: int = 0                   # ... of the shared key
+    freq: torch.Tensor | None = None # fp32 [2, pairs] radians per position, and what rounding took from them
+    rot_mult: float = 1.0
 
 
 @dataclass
@@ -970,6 +1142,26 @@ class BiasedAttentionWeights:
 
 
 @dataclass
+class DifferentialWeights:
+    spec: DifferentialSpec
+    q_norm: torch.Tensor             # fp32 [d]
+    k_norm: torch.Tensor
+    freq: torch.Tensor               # fp32 [2, pairs]
+    less: float                      # what the second map is multiplied by before it is taken away
+    q_off: int
+    g_off: int
+
+
+@dataclass
+class MinGruWeights:
+    spec: MinGruSpec
+    bias: torch.Tensor               # fp32 [2, width] of gate and candidate
+    z_off: int
+    x_off: int
+    g_off: int
+
+
+@dataclass
 class StreamWeights:
     """How a sublayer reads and writes the residual streams (fp32)."""
     read: torch.Tensor               # [streams]
@@ -1014,13 +1206,17 @@ class LayerWeights:
     side: SideWeights | None = None
     streams: tuple[StreamWeights, ...] = ()      # of the mixer and of the feed-forward
     routed: RoutedWeights | None = None
+    rg_off: int = 0                  # gated residuals: columns of the gate's logits in the output of ``proj``,
+    rg: tuple[torch.Tensor, ...] = ()            # biases (fp32 [W]) of the mixer's and of the feed-forward's gate; the latter's
+    ff_rows: int = 0                 # logits follow these rows of ``gate_up``
+    limit: float = 0.0               # of a clamped feed-forward
 
     def matrices(self) -> list[wq_pack.PackedWeight]:
         """Every packed matrix of the layer."""
         out = [self.proj, self.out]
         for part in ((self.mixer.left, self.mixer.right) if isinstance(self.mixer, PairWeights) else (self.mixer,)):
             if isinstance(part, LatentWeights):
-                out += [part.uq, part.absorb.w, part.value.w]
+                out += [m for m in (part.uq, part.absorb.w, part.value.w) if m is not None]
             elif getattr(part, "low", None) is not None:
                 out.append(part.low)
         out += [m for m in (self.gate_up, self.down) if m is not None]
@@ -1097,24 +1293,36 @@ def _pack_delta(m: DeltaSpec, p: str, rows: _Rows, get) -> DeltaWeights:
 
 
 def _pack_latent(m: LatentSpec, p: str, rows: _Rows, get) -> LatentWeights:
-    H, d, e, R, Rp = m.heads, m.dim, m.vdim, m.kv_rank, m.rank_padded
-    rows.add(get(f"{p}.dq"))
-    c_off = rows.add(get(f"{p}.dkv"))
-    g_off = rows.add(get(f"{p}.g"))
+    H, d, e, r, R, Rp = m.heads, m.dim, m.vdim, m.rot_dim, m.kv_rank, m.row_padded
     uk = torch.zeros(H, Rp, d, dtype=torch.bfloat16, device=get(f"{p}.uk").device)
     uk[:, :R] = get(f"{p}.uk").view(H, d, R).transpose(1, 2)
     absorb = BlockDiagonal.pack(uk)
-    uv = torch.zeros(H, e, Rp, dtype=torch.bfloat16, device=uk.device)
+    uv = torch.zeros(H, e, m.rank_padded, dtype=torch.bfloat16, device=uk.device)
     uv[:, :, :R] = get(f"{p}.uv").view(H, e, R)
+    value = BlockDiagonal.pack(uv)
     # the query projection writes every head where its block of ``absorb`` reads it
     hp, kg = absorb.heads, absorb.w.k
-    uq = torch.zeros(-(-H // hp) * kg, m.q_rank, dtype=torch.bfloat16, device=uk.device)
-    src = get(f"{p}.uq").view(H, d, m.q_rank)
-    for h in range(H):
-        c = (h // hp) * kg + (h % hp) * d
-        uq[c:c + d] = src[h]
-    return LatentWeights(m, _f32(get, f"{p}.dq.norm"), _f32(get, f"{p}.dkv.norm"), _matrix(uq), absorb, BlockDiagonal.pack(uv),
-                         c_off, g_off)
+
+    def spread(src: torch.Tensor) -> torch.Tensor:
+        out = torch.zeros(-(-H // hp) * kg, src.shape[-1], dtype=torch.bfloat16, device=uk.device)
+        for h in range(H):
+            c = (h // hp) * kg + (h % hp) * d
+            out[c:c + d] = src[h]
+        return out
+    c_norm = _f32(get, f"{p}.dkv.norm")
+    if m.rot_dim:
+        q = get(f"{p}.q").view(H, d + r, -1)
+        q_off = rows.add(spread(q[:, :d]))
+        qr_off = rows.add(q[:, d:].flatten(0, 1))
+        down = get(f"{p}.dkv")
+        c_off, r_off = rows.add(down[:R]), rows.add(down[R:])
+        return LatentWeights(m, None, c_norm, None, absorb, value, c_off, q_off=q_off, qr_off=qr_off, r_off=r_off,
+                             freq=m.rotary.split_table().to(uk.device).contiguous(), rot_mult=m.rotary.factor)
+    q_off = rows.add(get(f"{p}.dq"))
+    c_off = rows.add(get(f"{p}.dkv"))
+    g_off = rows.add(get(f"{p}.g"))
+    uq = spread(get(f"{p}.uq").view(H, d, m.q_rank))
+    return LatentWeights(m, _f32(get, f"{p}.dq.norm"), c_norm, _matrix(uq), absorb, value, c_off, g_off, q_off)
 
 
 def _pack_attention(m: AttentionSpec, p: str, rows: _Rows, get, out_scale: float = 1.0) -> AttentionWeights:
@@ -1139,9 +1347,7 @@ def _pack_conv_attention(m: ConvAttentionSpec, p: str, rows: _Rows, get) -> Conv
     for t, off in zip("qkv", m.offsets):
         w = get(f"{p}.{t}.conv").float()
         conv_w[:, off:off + w.shape[0]] = w.t()
-    exact = rope_inv_freq(m.rotary.dims, m.rotary.base, dtype=torch.float64)
-    freq = torch.stack([exact.float(), (exact - exact.float().double()).float()])
-    return ConvAttentionWeights(m, conv_w, freq.to(dev).contiguous(), q_off)
+    return ConvAttentionWeights(m, conv_w, m.rotary.split_table().to(dev).contiguous(), q_off)
 
 
 def _pack_biased_attention(m: BiasedAttentionSpec, p: str, rows: _Rows, get) -> BiasedAttentionWeights:
@@ -1149,6 +1355,20 @@ def _pack_biased_attention(m: BiasedAttentionSpec, p: str, rows: _Rows, get) -> 
     rel = _f32(get, f"{p}.rel")
     return BiasedAttentionWeights(m, _f32(get, f"{p}.q.norm"), _f32(get, f"{p}.k.norm"),
                                   rel[m.bucket_of_distance().to(rel.device)].contiguous(), q_off)
+
+
+def _pack_differential(m: DifferentialSpec, p: str, rows: _Rows, get) -> DifferentialWeights:
+    q_off = _add_qkv(m, p, rows, get)
+    g_off = rows.add(get(f"{p}.g"))
+    dot = [float((get(f"{p}.lq{i}").double() * get(f"{p}.lk{i}").double()).sum()) for i in (1, 2)]
+    q_norm = _f32(get, f"{p}.q.norm")
+    return DifferentialWeights(m, q_norm, _f32(get, f"{p}.k.norm"), m.rotary.split_table().to(q_norm.device).contiguous(),
+                               math.exp(dot[0]) - math.exp(dot[1]) + m.diff, q_off, g_off)
+
+
+def _pack_mingru(m: MinGruSpec, p: str, rows: _Rows, get) -> MinGruWeights:
+    z_off, x_off, g_off = (rows.add(get(f"{p}.{t}")) for t in "zxg")
+    return MinGruWeights(m, torch.stack([_f32(get, f"{p}.{t}.b") for t in "zx"]).contiguous(), z_off, x_off, g_off)
 
 
 def _pack_gated_linear(m: GatedLinearSpec, p: str, rows: _Rows, get, out_scale: float = 1.0) -> GatedLinearWeights:
@@ -1176,7 +1396,7 @@ def _pack_pair(m: PairSpec, p: str, rows: _Rows, get) -> PairWeights:
 
 _PACKERS = {DeltaSpec: _pack_delta, LatentSpec: _pack_latent, AttentionSpec: _pack_attention, GatedLinearSpec: _pack_gated_linear,
             SsdSpec: _pack_ssd, PairSpec: _pack_pair, ConvAttentionSpec: _pack_conv_attention,
-            BiasedAttentionSpec: _pack_biased_attention}
+            BiasedAttentionSpec: _pack_biased_attention, DifferentialSpec: _pack_differential, MinGruSpec: _pack_mingru}
 
 
 def _pack_output(m: MixerSpec, p: str, get, ff: int, W: int) -> tuple[torch.Tensor, int]:
@@ -1189,12 +1409,17 @@ def _pack_output(m: MixerSpec, p: str, get, ff: int, W: int) -> tuple[torch.Tens
     return out, off
 
 
-def _pack_glu(gate: torch.Tensor, up: torch.Tensor) -> wq_pack.PackedWeight:
-    """[gate ; up] in the row order of the GEMM's gated activation; the width is padded to whole blocks of it."""
+def _pack_glu(gate: torch.Tensor, up: torch.Tensor, rest: torch.Tensor | None = None) -> tuple[wq_pack.PackedWeight, int]:
+    """[gate ; up] in the row order of the GEMM's gated activation, the width padded to whole blocks of it, or, with ``rest`` rows
+    behind them, to whole tiles: (matrix, rows of the gated activation)."""
     ff, k = gate.shape
-    both = torch.zeros(2, round_up(ff, 16), k, dtype=torch.bfloat16, device=gate.device)
+    both = torch.zeros(2, round_up(ff, 16 if rest is None else wq_pack.TILE_N // 2), k, dtype=torch.bfloat16, device=gate.device)
     both[0, :ff], both[1, :ff] = gate, up
-    return wq_pack.swiglu_interleave(_matrix(both.flatten(0, 1)))
+    w = wq_pack.swiglu_interleave(_matrix(both.flatten(0, 1)))
+    if rest is None:
+        return w, w.n
+    codes = torch.cat([w.codes, _pad(rest, rest.shape[0], w.k)])
+    return replace(w, n=codes.shape[0], codes=codes), w.n
 
 
 def _stack(mats) -> wq_pack.PackedWeight:
@@ -1221,11 +1446,17 @@ def _pack_streams(p: str, get) -> StreamWeights:
     return StreamWeights(*(_f32(get, f"{p}.{t}") for t in ("in", "out", "mix")))
 
 
+def _norm_factor(cfg: LayeredConfig, get, name: str) -> torch.Tensor:
+    """fp32 factor per channel of a norm of the residual."""
+    return (cfg.design.norm_offset + _f32(get, name)).expand(cfg.hidden_size).contiguous()
+
+
 def pack_layer(cfg: LayeredConfig, i: int, get) -> LayerWeights:
     """``get(name)`` -> tensor on the target device."""
     l, p, W, d = cfg.layers[i], f"l{i}", cfg.hidden_size, cfg.design
     rows = _Rows(W)
     mixer = _PACKERS[type(l.mixer)](l.mixer, f"{p}.mix", rows, get)
+    rg_off = rows.add(get(f"{p}.rg1")) if d.gated else 0
     proj = rows.end()
     split = proj.shape[0]
     joint = 0 if d.sequential else l.ff
@@ -1233,15 +1464,18 @@ def pack_layer(cfg: LayeredConfig, i: int, get) -> LayerWeights:
     if joint:
         proj = torch.cat([proj, get(f"{p}.mlp.up").to(torch.bfloat16)])
         out[:, out_off:out_off + l.ff] = get(f"{p}.mlp.down")
-    lw = LayerWeights(d.norm_offset + _f32(get, f"{p}.norm1"), _matrix(proj), split, joint, mixer, wq_pack.pack_bf16(out), out_off)
+    lw = LayerWeights(_norm_factor(cfg, get, f"{p}.norm1"), _matrix(proj), split, joint, mixer, wq_pack.pack_bf16(out), out_off)
     if d.streams:
         lw.streams = tuple(_pack_streams(f"{p}.hc{q}", get) for q in ((1, 2) if l.has_ff else (1,)))
     if d.sequential and l.has_ff:
-        lw.norm2 = d.norm_offset + _f32(get, f"{p}.norm2")
+        lw.norm2 = _norm_factor(cfg, get, f"{p}.norm2")
+    if d.gated:
+        lw.rg_off, lw.rg, lw.limit = rg_off, tuple(_f32(get, f"{p}.rg{q}.b") for q in ((1, 2) if l.has_ff else (1,))), l.limit
     if l.routed is not None:
         lw.routed = _pack_routed(l.routed, f"{p}.mlp", W, get)
     if d.sequential and l.ff:
-        lw.gate_up = _pack_glu(get(f"{p}.mlp.gate"), get(f"{p}.mlp.up"))
+        lw.gate_up, lw.ff_rows = _pack_glu(get(f"{p}.mlp.gate"), get(f"{p}.mlp.up"),
+                                           get(f"{p}.rg2").to(torch.bfloat16) if d.gated else None)
         lw.down = _matrix(get(f"{p}.mlp.down").to(torch.bfloat16))
     if cfg.side_dim:
         gate = get(f"{p}.side.gate").to(torch.bfloat16)
@@ -1254,10 +1488,10 @@ def pack_weights(cfg: LayeredConfig, get) -> LayeredWeights:
     d = cfg.design
     embed = get("embed").to(torch.bfloat16).contiguous()
     return LayeredWeights(
-        embed=embed, embed_norm=d.norm_offset + get("embed.norm").float() if d.embed_norm else None,
-        loop_in=_matrix(get("loop.in")) if cfg.loop is not None else None,
+        embed=embed, embed_norm=_norm_factor(cfg, get, "embed.norm") if d.embed_norm else None,
+        loop_in=_matrix(get("loop.in")) if cfg.loop is not None and d.loop == "project" else None,
         layers=[pack_layer(cfg, i, get) for i in range(cfg.num_layers)],
-        final_norm=d.norm_offset + get("final.norm").float(), lm_head=_matrix(embed if d.tied_head else get("head")),
+        final_norm=_norm_factor(cfg, get, "final.norm"), lm_head=_matrix(embed if d.tied_head else get("head")),
         side_embed=get("side.embed").to(torch.bfloat16).contiguous() if cfg.side_dim else None)
 
 
@@ -1329,8 +1563,28 @@ def streams_moe_config() -> LayeredConfig:
     return LayeredConfig("layered-streams-moe", 151936, 4096, group * 8, 1e-6, architecture="Vimelorn", streams=2, embed_scale=64.0)
 
 
+def tiny_gated_config() -> LayeredConfig:
+    """A few small layers of every kind with gated residuals and a loop (tests and demonstrations)."""
+    latent = LatentSpec(5, 24, 40, 0, 72, 0.2, 0, 20, RotarySpec(20, 10000.0, ("yarn", 4.0, 128.0, 16.0, 1.0, 0.1 * math.log(4.0) + 1.0)), False)
+    pair = DifferentialSpec(6, 2, 24, 40, 0.2, RotarySpec(16, 10000.0), 0.4, 37)
+    return LayeredConfig("layered-gated-tiny", 384, 192, (LayerSpec(latent, 160, limit=2.0), LayerSpec(MinGruSpec(224), 128, limit=2.0),
+                                                          LayerSpec(pair, 160, limit=2.0), LayerSpec(MinGruSpec(160))),
+                         1e-5, (1, 3, 2), architecture="Fovunex", embed_scale=0.7)
+
+
+def gated_8b_config() -> LayeredConfig:
+    """Layers of the size of an 8B model with gated residuals: latent attention over every earlier token, differential attention in
+    chunks and element-wise recurrences in turn."""
+    yarn = ("yarn", 8.0, 8192.0, 32.0, 1.0, 0.1 * math.log(8.0) + 1.0)
+    latent = LayerSpec(LatentSpec(32, 128, 128, 0, 512, 192 ** -0.5, 0, 64, RotarySpec(64, 1e6, yarn), False), 12288, limit=7.0)
+    pair = LayerSpec(DifferentialSpec(32, 8, 64, 128, 64 ** -0.5, RotarySpec(64, 1e6), 0.6, 4096), 12288, limit=7.0)
+    gru = LayerSpec(MinGruSpec(6144), 12288, limit=7.0)
+    return LayeredConfig("layered-gated-8b", 151936, 4096, (pair, gru, pair, latent) * 8, 1e-6, architecture="Fovunex", embed_scale=1.0)
+
+
 NAMED = {"layered-tiny": tiny_layered_config, "layered-8b": layered_8b_config, "layered-seq-tiny": tiny_sequential_config,
-         "layered-seq-8b": sequential_8b_config, "layered-streams-tiny": tiny_streams_config, "layered-streams-moe": streams_moe_config}
+         "layered-seq-8b": sequential_8b_config, "layered-streams-tiny": tiny_streams_config, "layered-streams-moe": streams_moe_config,
+         "layered-gated-tiny": tiny_gated_config, "layered-gated-8b": gated_8b_config}
 
 
 def with_dtype(cfg: LayeredConfig, dtype: str) -> LayeredConfig:

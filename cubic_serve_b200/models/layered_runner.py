@@ -16,7 +16,13 @@ and a sequential layer, whose h comes from the step before it,
     norm2(x) -> h;  act = gelu(h W_gate) (h W_up), one product;  x += act W_down
     side = gelu(x W_side) e, one kernel;  y = side W_proj;  x += norm(y) and h = norm1 of the next layer, one kernel
 
-and of a layer on several residual streams x_s, whose h is the norm of their weighted sum,
+with gated residuals the matrices that read a norm also make the logits of the gate, which the products that join the residual
+take in their epilogue (and the feed-forward's product is [act | gate] = h [W_gate, W_up ; W_rg]),
+
+    x += sigmoid(gate) (operand W_o);  x += sigmoid(gate) (act W_down)
+
+and a pass of a loop that adds the embedding output starts with x += scale E and h = norm1 of its first layer, one kernel.  A layer on
+several residual streams x_s, whose h is the norm of their weighted sum, runs
 
     mixer inputs = h W;  mixer -> operand;  y = operand W_o
     x_t <- sum_s mix[s, t] x_s + out[t] y and h = norm2 of the next weighted sum, one kernel
@@ -32,9 +38,13 @@ from __future__ import annotations
 import torch
 
 from ..ops import kernels as K
-from .layered import (AttentionWeights, BiasedAttentionWeights, ConvAttentionWeights, DeltaWeights, GatedLinearWeights, LatentWeights,
-                      LayeredConfig, LayeredWeights, PairWeights, RoutedWeights, SsdWeights, round_up)
+from .layered import (AttentionWeights, BiasedAttentionWeights, ConvAttentionWeights, DeltaWeights, DifferentialWeights,
+                      GatedLinearWeights, LatentWeights, LayeredConfig, LayeredWeights, MinGruWeights, PairWeights, RoutedWeights,
+                      SsdWeights, round_up)
 from .step_runner import StepRunner
+
+
+_PAGED = (AttentionWeights, ConvAttentionWeights, BiasedAttentionWeights, DifferentialWeights)      # keys and values in pages
 
 
 class _StateRun:
@@ -81,9 +91,12 @@ class LayeredRunner(StepRunner):
             return torch.zeros(T, cols, dtype=dtype, device=dev)
 
         self.x = buf(cfg.streams * W, torch.float32)      # residual stream, or streams
-        self.x0 = buf(W, torch.float32) if cfg.loop is not None else None
+        project = cfg.loop is not None and cfg.design.loop == "project"
+        self.x0 = buf(W, torch.float32) if project else None
         self.h = buf(round_up(W, 64))
-        self.entry = buf(round_up(2 * W, 64)) if cfg.loop is not None else None
+        self.entry = buf(round_up(2 * W, 64)) if project else None
+        # logits of the feed-forward's gate
+        self.rg = buf(round_up(W, 8))[:, :W] if cfg.design.gated else None
         self.side = buf(round_up(cfg.side_dim, 64)) if cfg.side_dim else None
         self.side_y = buf(round_up(W, 8)) if cfg.side_dim else None
         self.y = buf(round_up(W, 8))[:, :W] if cfg.design.streams else None       # a sublayer's result
@@ -99,17 +112,18 @@ class LayeredRunner(StepRunner):
             self._operands.setdefault(self._layout(l), buf(l.out.k))
             self._need("proj", l.split)
             if l.down is not None:
-                self._operands.setdefault(("act", l.gate_up.n, l.down.k), buf(l.down.k))
+                self._operands.setdefault(("act", l.ff_rows, l.down.k), buf(l.down.k))
             for m in _parts(l.mixer):
                 s = m.spec
                 if isinstance(m, LatentWeights):
-                    self._need("cq%d" % s.q_rank, round_up(s.q_rank, 64))
-                    self._need("q", m.uq.n)
-                    self._need("ql", s.heads * s.rank_padded)
+                    if m.uq is not None:
+                        self._need("cq%d" % s.q_rank, round_up(s.q_rank, 64))
+                        self._need("q", m.uq.n)
+                    self._need("ql", s.heads * s.row_padded)
                     self._need("ol", s.heads * s.rank_padded)
-                elif isinstance(m, (AttentionWeights, ConvAttentionWeights, BiasedAttentionWeights)):
+                elif isinstance(m, _PAGED):
                     self._need("q", s.heads * s.width_padded)
-                else:
+                elif not isinstance(m, MinGruWeights):
                     if isinstance(m, DeltaWeights):
                         recurrent.append((s.heads, s.kv_heads, s.dim, s.vdim, s.per_channel))
                     elif isinstance(m, SsdWeights):
@@ -127,9 +141,12 @@ class LayeredRunner(StepRunner):
         """Cache or state of one run of a mixer."""
         s, dev, rows = m.spec, self.device, self.max_requests + len(self.state_checkpoint_rows)
         if isinstance(m, LatentWeights):
-            self.kv.append(torch.zeros(self.num_pages, 16, s.rank_padded, dtype=self.act, device=dev))
+            self.kv.append(torch.zeros(self.num_pages, 16, s.row_padded, dtype=self.act, device=dev))
             return self.kv[-1]
-        if isinstance(m, (AttentionWeights, ConvAttentionWeights, BiasedAttentionWeights)):
+        if isinstance(m, MinGruWeights):
+            self.states.append(_StateRun(rows, 1, 1, s.padded, dev))
+            return self.states[-1]
+        if isinstance(m, _PAGED):
             self.kv.append(torch.zeros(self.num_pages, s.kv_heads, 2, 16, s.width_padded, dtype=self.act, device=dev))
             if not isinstance(m, ConvAttentionWeights):
                 return self.kv[-1]
@@ -205,28 +222,33 @@ class LayeredRunner(StepRunner):
     def _sequential(self, b) -> torch.Tensor:
         cfg, w, T, eps = self.cfg, self.w, b.num_tokens, self.cfg.rms_eps
         decode = T == b.segments.num
-        x, h = self.x[:T], self.h[:T]
-        K.embed_rows(b.token_ids[:T], w.embed, w.layers[0].norm, x, h, eps)
-        n, last = 1, len(w.layers) - 1
-        for i, (l, run) in enumerate(zip(w.layers, self.runs)):
+        x, h, W = self.x[:T], self.h[:T], cfg.hidden_size
+        K.embed_rows(b.token_ids[:T], w.embed, w.layers[0].norm, x, h, eps, cfg.embed_scale)
+        n, last = 1, len(cfg.runs) - 1
+        for at, ((i, enters), run) in enumerate(zip(cfg.runs, self.runs)):
+            l = w.layers[i]
             operand, proj = self._operands[self._layout(l)][:T], self._rows("proj", T, l.split)
             K.wide_gemm(h, l.proj, proj, ws=self.ws)
             n += 2 + self._mix(l.mixer, proj, run, b, operand, decode)
-            K.wide_gemm(operand, l.out, x, residual=x, ws=self.ws)
+            K.wide_gemm(operand, l.out, x, residual=x, gate=(proj[:, l.rg_off:l.rg_off + W], l.rg[0]) if l.rg else None, ws=self.ws)
             if l.down is not None:
-                act = self._operands[("act", l.gate_up.n, l.down.k)][:T]
+                act = self._operands[("act", l.ff_rows, l.down.k)][:T]
+                rest = dict(rest=self.rg[:T], split=l.ff_rows, limit=l.limit) if l.rg else {}
                 K.row_norm(x, l.norm2, h, eps)
-                K.wide_gemm(h, l.gate_up, act[:, :l.gate_up.n // 2], glu="gelu", ws=self.ws)
-                K.wide_gemm(act, l.down, x, residual=x, ws=self.ws)
+                K.wide_gemm(h, l.gate_up, act[:, :l.ff_rows // 2], glu=cfg.design.ff[:-len("_glu")], ws=self.ws, **rest)
+                K.wide_gemm(act, l.down, x, residual=x, gate=(self.rg[:T], l.rg[1]) if l.rg else None, ws=self.ws)
                 n += 3
-            follow = None if i == last else w.layers[i + 1].norm       # the final norm reads the wanted rows only
+            follow = None if at == last else w.layers[cfg.runs[at + 1][0]].norm      # the final norm reads the wanted rows only
             if l.side is not None:
                 n += K.side_input(x, l.side.gate, b.token_ids[:T], w.side_embed, l.side.col, l.side.proj, l.side.norm_w, eps, follow,
-                                  None if follow is None else h, self.side[:T], self.side_y[:T, :cfg.hidden_size], self.ws)
-            elif follow is not None:
-                K.row_norm(x, follow, h, eps)
-                n += 1
+                                  None if follow is None else h, self.side[:T], self.side_y[:T, :W], self.ws)
             self._after_layer(x)
+            if l.side is None and follow is not None:
+                if cfg.reenters(at + 1):
+                    K.embed_rows(b.token_ids[:T], w.embed, follow, x, h, eps, cfg.embed_scale, add=True)
+                else:
+                    K.row_norm(x, follow, h, eps)
+                n += 1
         self.launches_per_step = n
         return x
 
@@ -249,8 +271,8 @@ class LayeredRunner(StepRunner):
                     result, routes, made = self._routed(l.routed, h, y)
                     n += 1 + made
                 elif q:
-                    act = self._operands[("act", l.gate_up.n, l.down.k)][:T]
-                    K.wide_gemm(h, l.gate_up, act[:, :l.gate_up.n // 2], glu="silu", ws=self.ws)
+                    act = self._operands[("act", l.ff_rows, l.down.k)][:T]
+                    K.wide_gemm(h, l.gate_up, act[:, :l.ff_rows // 2], glu=cfg.design.ff[:-len("_glu")], ws=self.ws)
                     K.wide_gemm(act, l.down, y, ws=self.ws)
                     n += 3
                 at += 1
@@ -314,17 +336,21 @@ class LayeredRunner(StepRunner):
                                 s.per_channel, s.per_channel, decode)
 
     def _latent(self, m: LatentWeights, proj, cache: torch.Tensor, b, out, decode: bool) -> int:
-        s, T = m.spec, proj.shape[0]
-        wide = s.heads * s.rank_padded
-        cq = self._rows("cq%d" % s.q_rank, T, round_up(s.q_rank, 64))
-        q, ql, ol = self._rows("q", T, m.uq.n), self._rows("ql", T, wide), self._rows("ol", T, wide)
-        K.latent_prepare(proj, s.q_rank, m.c_off, s.kv_rank, m.q_norm, m.c_norm, cq, cache, b.slots, self.cfg.rms_eps)
-        K.wide_gemm(cq, m.uq, q, ws=self.ws)
-        K.wide_gemm(q, m.absorb.w, ql, diag_rows=m.absorb.rows, ws=self.ws)
-        K.latent_attention(ql, proj[:, m.g_off:m.g_off + s.heads], cache, b.page_table, b.segments, ol, s.heads, s.window,
-                           s.scale, decode=decode, ws=self.ws)
+        s, T, eps = m.spec, proj.shape[0], self.cfg.rms_eps
+        ql, ol = self._rows("ql", T, s.heads * s.row_padded), self._rows("ol", T, s.heads * s.rank_padded)
+        if m.uq is not None:
+            cq, q = self._rows("cq%d" % s.q_rank, T, round_up(s.q_rank, 64)), self._rows("q", T, m.uq.n)
+            K.latent_prepare(proj, m.c_off, s.kv_rank, m.c_norm, cache, b.slots, eps, low=(m.q_off, s.q_rank, m.q_norm, cq))
+            K.wide_gemm(cq, m.uq, q, ws=self.ws)
+            K.wide_gemm(q, m.absorb.w, ql, diag_rows=m.absorb.rows, ws=self.ws)
+        else:                                  # the product writes zeros where the rotated part follows
+            K.wide_gemm(proj[:, m.q_off:m.qr_off], m.absorb.w, ql, diag_rows=m.absorb.rows, ws=self.ws)
+            K.latent_prepare(proj, m.c_off, s.kv_rank, m.c_norm, cache, b.slots, eps,
+                             rotated=(m.qr_off, m.r_off, s.rot_col, m.freq, m.rot_mult, b.positions[:T], ql, s.heads))
+        K.latent_attention(ql, proj[:, m.g_off:m.g_off + s.heads] if s.gated else None, cache, b.page_table, b.segments, ol, s.heads,
+                           s.window, s.scale, decode=decode, ws=self.ws)
         K.wide_gemm(ol, m.value.w, out, diag_rows=m.value.rows, ws=self.ws)
-        return 5
+        return 5 if m.uq is not None else 4
 
     def _attention(self, m: AttentionWeights, proj, cache: torch.Tensor, b, out, decode: bool) -> int:
         s, T = m.spec, proj.shape[0]
@@ -349,6 +375,19 @@ class LayeredRunner(StepRunner):
                    s.dim, s.vdim, self.cfg.rms_eps, (s.temp_coef, s.temp_every))
         return 1 + K.gqa_attention(q, cache, b.page_table, b.segments, out, s.heads, s.vdim, s.window, s.scale, decode=decode, ws=self.ws,
                                    bias=m.bias)
+
+    def _differential(self, m: DifferentialWeights, proj, cache: torch.Tensor, b, out, decode: bool) -> int:
+        s, T = m.spec, proj.shape[0]
+        q = self._rows("q", T, s.heads * s.width_padded)
+        K.head_qkv(proj, tuple(m.q_off + o for o in s.offsets), m.q_norm, m.k_norm, m.freq, b.positions[:T], b.slots[:T], q, cache,
+                   s.heads, s.dim, s.vdim, self.cfg.rms_eps, maps=2)
+        return 1 + K.gqa_attention(q, cache, b.page_table, b.segments, out, s.heads, s.vdim, 0, s.scale, out_scale=1.0 - s.diff,
+                                   decode=decode, ws=self.ws, chunk=s.chunk,
+                                   pair=(proj[:, m.g_off:m.g_off + s.out_width], m.less, self.cfg.rms_eps))
+
+    def _mingru(self, m: MinGruWeights, proj, run: _StateRun, b, out, decode: bool) -> int:
+        K.mingru(proj, m.z_off, m.x_off, m.g_off, m.bias, run.state[:, 0, 0], b.segments, out)
+        return 1
 
     def _gated_linear(self, m: GatedLinearWeights, proj, run: _StateRun, b, out, decode: bool) -> int:
         s, T, n = m.spec, proj.shape[0], 1
@@ -385,4 +424,5 @@ class LayeredRunner(StepRunner):
 
 _MIXERS = {DeltaWeights: LayeredRunner._delta, LatentWeights: LayeredRunner._latent, AttentionWeights: LayeredRunner._attention,
            GatedLinearWeights: LayeredRunner._gated_linear, SsdWeights: LayeredRunner._ssd,
-           ConvAttentionWeights: LayeredRunner._conv_attention, BiasedAttentionWeights: LayeredRunner._biased_attention}
+           ConvAttentionWeights: LayeredRunner._conv_attention, BiasedAttentionWeights: LayeredRunner._biased_attention,
+           DifferentialWeights: LayeredRunner._differential, MinGruWeights: LayeredRunner._mingru}

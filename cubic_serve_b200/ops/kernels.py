@@ -723,24 +723,36 @@ def _seg(seg: GdnSegments) -> "native.GdnSegmentsStruct":
     return seg.struct()
 
 
-GLU = {None: 0, "silu": 1, "gelu": 2}       # Glu in csrc/wq_gemm_common.cuh
+GLU = {None: 0, "silu": 1, "gelu": 2, "clamped": 3}       # Glu in csrc/wq_gemm_common.cuh
 
 
 def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: torch.Tensor | None = None,
               relu2: torch.Tensor | None = None, split: int = 0, diag_rows: int = 0, ws: Workspace | None = None,
-              stream_k: bool | None = None, splits: int | None = None, glu: str | None = None) -> None:
+              stream_k: bool | None = None, splits: int | None = None, glu: str | None = None, limit: float = 0.0,
+              rest: torch.Tensor | None = None, gate: tuple[torch.Tensor, torch.Tensor] | None = None) -> None:
     """``x @ W^T`` with bf16-stored weights through the wide epilogue.
 
     ``x`` fp32: everything is fp32 (``csrc/layered.cu``); ``x`` bf16: tcgen05 with fp32 accumulation.  ``out`` gets the
     product; an fp32 ``out`` may be added to ``residual`` (the same tensor: in-place accumulation).  With ``relu2`` the
     features from ``split`` on leave there as ``max(v, 0)^2`` and ``out`` holds the first ``split``.  ``glu`` "gelu" / "silu": the
-    rows of ``w`` are interleaved [gate ; up] and ``out`` gets ``gelu_tanh(gate) * up`` / ``silu(gate) * up`` (``N / 2`` columns).  ``diag_rows``:
-    block-diagonal weights, see ``models/layered.py::BlockDiagonal``.  ``x`` may have fewer columns than ``w.k``: the rest
+    rows of ``w`` are interleaved [gate ; up] and ``out`` gets ``gelu_tanh(gate) * up`` / ``silu(gate) * up`` (``N / 2`` columns); "clamped":
+    ``g sigmoid(1.702 g) (u + 1)`` with ``g = min(gate, limit)`` and ``u`` clamped to ``limit``.  With ``rest`` only the first ``split``
+    rows are interleaved, and the other features leave there as they are.  ``gate``: (logits ``[M, N]`` in ``x``'s type, bias fp32
+    ``[N]``): the product times the sigmoid of their sum joins ``residual``.  ``diag_rows``: block-diagonal weights, see ``models/layered.py::BlockDiagonal``.  ``x`` may have fewer columns than ``w.k``: the rest
     read as zero."""
     m, k = x.shape[0], w.k
     assert w.fmt == FMT_BF16 and x.stride(1) == 1 and out.stride(1) == 1 and out.shape[0] == m
     assert (glu is not None) == w.act_interleaved and not (glu and (relu2 is not None or residual is not None or diag_rows))
-    assert out.shape[1] == (split if relu2 is not None else w.n // 2 if glu else w.n), (out.shape, split, w.n)
+    assert rest is None or glu and rest.dtype == x.dtype and rest.stride(1) == 1 and rest.shape == (m, w.n - split)
+    assert out.shape[1] == (split if relu2 is not None else (w.n if rest is None else split) // 2 if glu else w.n), (out.shape, split, w.n)
+    g = b = None
+    if gate is not None:
+        g, b = gate
+        assert residual is not None and relu2 is None and g.dtype == x.dtype and g.stride(1) == 1 and g.shape == (m, w.n)
+        assert b.dtype == torch.float32 and b.is_contiguous() and b.numel() == w.n
+    ldg = 0 if g is None else g.stride(0)
+    second = relu2 if rest is None else rest
+    ld2 = 0 if second is None else second.stride(0)
     assert residual is None or (residual.dtype == torch.float32 and residual.stride(0) == out.stride(0))
     if relu2 is not None:
         assert relu2.dtype == x.dtype and relu2.stride(1) == 1 and relu2.shape == (m, w.n - split) and split % 4 == 0
@@ -749,8 +761,8 @@ def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: tor
     if x.dtype == torch.float32:
         assert out.dtype == torch.float32
         a = native.F32GemmStruct(x.data_ptr(), x.stride(0), x_cols, w.codes.data_ptr(), out.data_ptr(), out.stride(0),
-                                 _ptr(residual), _ptr(relu2), 0 if relu2 is None else relu2.stride(0), split, diag_rows, m,
-                                 w.n, k, GLU[glu], None, 0)
+                                 _ptr(residual), _ptr(second), ld2, split, diag_rows, m, w.n, k, GLU[glu], None, 0, float(limit),
+                                 _ptr(g), ldg, _ptr(b))
         native.check(l.cb_f32_gemm(ctypes.byref(a), _stream()), "cb_f32_gemm")
         return
     wide32 = out.dtype == torch.float32
@@ -765,9 +777,9 @@ def wide_gemm(x: torch.Tensor, w: PackedWeight, out: torch.Tensor, residual: tor
         splits = 1
     from .strategies import active
     a = native.WideGemmStruct(x.data_ptr(), x.stride(0), x_cols, w.codes.data_ptr(), None if wide32 else out.data_ptr(),
-                              out.data_ptr() if wide32 else None, out.stride(0), _ptr(residual), _ptr(relu2),
-                              0 if relu2 is None else relu2.stride(0), split, diag_rows, m, w.n, k, int(stream_k), splits,
-                              active().gemm.stream_k_min_units, GLU[glu])
+                              out.data_ptr() if wide32 else None, out.stride(0), _ptr(residual), _ptr(second), ld2, split,
+                              diag_rows, m, w.n, k, int(stream_k), splits, active().gemm.stream_k_min_units, GLU[glu], float(limit),
+                              _ptr(g), ldg, _ptr(b))
     code = l.cb_bf16_gemm_wide(ctypes.byref(a), ws.gemm.data_ptr(), ws.gemm.numel(), ws.gemm_counters.data_ptr(),
                                ws.status.data_ptr(), _stream())
     native.check(code, "cb_bf16_gemm_wide")
@@ -796,11 +808,13 @@ def concat_rows(x: torch.Tensor, x0: torch.Tensor, out: torch.Tensor) -> None:
                                              x.shape[1], int(out.dtype == torch.float32), _stream()), "cb_concat_rows")
 
 
-def embed_rows(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, h: torch.Tensor, eps: float) -> None:
-    """``x`` = embedding rows (fp32), ``h = x / rms(x) * weight`` in ``h``'s type."""
+def embed_rows(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, h: torch.Tensor, eps: float,
+               scale: float = 1.0, add: bool = False) -> None:
+    """``x`` = ``scale`` times the embedding rows (fp32), added to what it holds with ``add``; ``h = x / rms(x) * weight`` in ``h``'s
+    type."""
     assert x.dtype == weight.dtype == torch.float32 and x.is_contiguous() and table.dtype == torch.bfloat16 and h.stride(1) == 1
     native.check(native.lib().cb_embed_rows(ids.data_ptr(), table.data_ptr(), weight.data_ptr(), x.data_ptr(), h.data_ptr(),
-                                            h.stride(0), x.shape[0], x.shape[1], table.shape[0], float(eps),
+                                            h.stride(0), x.shape[0], x.shape[1], table.shape[0], float(eps), float(scale), int(add),
                                             int(h.dtype == torch.float32), _stream()), "cb_embed_rows")
 
 
@@ -980,34 +994,46 @@ def ssd_walk(z: torch.Tensor, d: torch.Tensor, norm_w: torch.Tensor, parts: int,
     return 2
 
 
-def latent_prepare(proj: torch.Tensor, q_rank: int, c_off: int, rank: int, q_norm: torch.Tensor, c_norm: torch.Tensor,
-                   cq: torch.Tensor, cache: torch.Tensor, slots: torch.Tensor, eps: float) -> None:
-    """RMS norms of the query latent (columns ``[0, q_rank)`` of ``proj``) into ``cq`` and of the cache latent (columns
-    ``[c_off, c_off + rank)``) into its page of ``cache`` ``[pages, 16, rank padded]``."""
-    assert cache.is_contiguous() and cache.dtype == proj.dtype == cq.dtype and slots.dtype == torch.int32
-    native.check(native.lib().cb_latent_prepare(proj.data_ptr(), proj.stride(0), 0, q_rank, c_off, rank, q_norm.data_ptr(),
-                                                c_norm.data_ptr(), cq.data_ptr(), cq.stride(0), cache.data_ptr(),
-                                                cache.shape[2], slots.data_ptr(), proj.shape[0], float(eps),
-                                                int(proj.dtype == torch.float32), _stream()), "cb_latent_prepare")
+def latent_prepare(proj: torch.Tensor, c_off: int, rank: int, c_norm: torch.Tensor, cache: torch.Tensor, slots: torch.Tensor, eps: float,
+                   low: tuple[int, int, torch.Tensor, torch.Tensor] | None = None,
+                   rotated: tuple[int, int, int, torch.Tensor, float, torch.Tensor, torch.Tensor, int] | None = None) -> None:
+    """RMS norm of the cache latent (columns ``[c_off, c_off + rank)`` of ``proj``) into its page of ``cache`` ``[pages, 16, padded]``.
+    ``low`` = (first column, rank, norm weight, destination): the same for a query latent.  ``rotated`` = (first column of the
+    queries' rotated parts, of the shared key's, column of a row they go to, ``freq`` fp32 ``[2, pairs]``, factor on cosine and sine,
+    positions, latent-space queries ``[T, H padded]``, heads): neighbouring channels turn with the position, queries beside their
+    latent part and the key into the cached row."""
+    assert cache.is_contiguous() and cache.dtype == proj.dtype and slots.dtype == torch.int32 and proj.stride(1) == 1
+    q_off, q_rank, q_norm, cq = low or (0, 0, None, None)
+    qr_off, r_off, col, freq, mult, positions, ql, heads = rotated or (0, 0, 0, None, 1.0, None, None, 0)
+    if low:
+        assert cq.dtype == proj.dtype and cq.stride(1) == 1
+    if rotated:
+        assert ql.dtype == proj.dtype and ql.is_contiguous() and ql.shape[1] == heads * cache.shape[2] and positions.dtype == torch.int32
+        assert freq.dtype == torch.float32 and freq.is_contiguous() and freq.shape[0] == 2
+    a = native.LatentPrepStruct(proj.data_ptr(), proj.stride(0), q_off, q_rank, c_off, rank, _ptr(q_norm), c_norm.data_ptr(), _ptr(cq),
+                                0 if cq is None else cq.stride(0), cache.data_ptr(), cache.shape[2], slots.data_ptr(), qr_off, r_off, col,
+                                0 if freq is None else freq.shape[1], _ptr(freq), float(mult), _ptr(positions), _ptr(ql), heads,
+                                proj.shape[0], float(eps), int(proj.dtype == torch.float32))
+    native.check(native.lib().cb_latent_prepare(ctypes.byref(a), _stream()), "cb_latent_prepare")
 
 
-def latent_attention(q: torch.Tensor, gate: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor, seg: GdnSegments,
+def latent_attention(q: torch.Tensor, gate: torch.Tensor | None, cache: torch.Tensor, page_table: torch.Tensor, seg: GdnSegments,
                      out: torch.Tensor, heads: int, window: int, scale: float, decode: bool = False, splits: int | None = None,
                      ws: Workspace | None = None) -> None:
-    """Windowed softmax attention of latent-space queries ``q [T, H Rp]`` over the paged latents, times the heads' sigmoid
-    gates (``gate [T, H]`` logits).  ``window`` 0: every earlier token.  ``decode``: every segment has at most one row.
-    ``splits``: key splits of the bf16 form (None: as many as fill the device)."""
-    T, rp = q.shape[0], cache.shape[2]
-    assert q.shape[1] == out.shape[1] == heads * rp and q.is_contiguous() and out.is_contiguous()
-    assert q.dtype == out.dtype == gate.dtype == cache.dtype and page_table.dtype == torch.int32
+    """Windowed softmax attention of latent-space queries ``q [T, H Rp]`` over the paged rows; a row's first columns are its value too
+    (``out [T, H Rv]``).  ``gate``: logits ``[T, H]`` of a sigmoid per head, or None.  ``window`` 0: every earlier token.
+    ``decode``: every segment has at most one row.  ``splits``: key splits of the bf16 form (None: as many as fill the device)."""
+    T, rp, rv = q.shape[0], cache.shape[2], out.shape[1] // heads
+    assert q.shape[1] == heads * rp and out.shape[1] == heads * rv and rv <= rp and q.is_contiguous() and out.is_contiguous()
+    assert q.dtype == out.dtype == cache.dtype and page_table.dtype == torch.int32 and (gate is None or gate.dtype == q.dtype)
     f32 = q.dtype == torch.float32
     l = native.lib()
     partial = None
-    if f32 or rp > 512:
+    if f32 or not l.cb_latent_attn_mma(rp, rv):
         splits = 1
     else:
         units = ctypes.c_int(0)
-        l.cb_latent_attn_partial_floats(T, seg.num, heads, rp, int(decode), 1, ctypes.byref(units))
+        l.cb_latent_attn_partial_floats(T, seg.num, heads, rv, int(decode), 1, ctypes.byref(units))
         if splits is None:
             from .strategies import active
             a = active().attention
@@ -1016,10 +1042,10 @@ def latent_attention(q: torch.Tensor, gate: torch.Tensor, cache: torch.Tensor, p
             splits = min(a.max_splits, -(-keys // 64), max(1, a.target_ctas // (1 if decode else 2) // units.value))
         if splits > 1:
             ws = ws or workspace(q.device)
-            ws.ensure_attn(l.cb_latent_attn_partial_floats(T, seg.num, heads, rp, int(decode), splits, None))
+            ws.ensure_attn(l.cb_latent_attn_partial_floats(T, seg.num, heads, rv, int(decode), splits, None))
             partial = ws.attn.data_ptr()
-    a = native.LatentAttnStruct(q.data_ptr(), out.data_ptr(), cache.data_ptr(), gate.data_ptr(), gate.stride(0),
-                                page_table.data_ptr(), page_table.shape[1], heads, rp, window, float(scale), T, int(f32),
+    a = native.LatentAttnStruct(q.data_ptr(), out.data_ptr(), cache.data_ptr(), _ptr(gate), 0 if gate is None else gate.stride(0),
+                                page_table.data_ptr(), page_table.shape[1], heads, rp, rv, window, float(scale), T, int(f32),
                                 int(decode), splits, partial)
     st = _seg(seg)
     native.check(l.cb_latent_attn(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_latent_attn")
@@ -1042,17 +1068,24 @@ def gqa_prepare(x: torch.Tensor, q_off: int, k_off: int, q_norm: torch.Tensor, k
 
 def gqa_attention(q: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor, seg: GdnSegments, out: torch.Tensor, heads: int,
                   dim: int, window: int, scale: float, sink: float | None = None, out_scale: float = 1.0, decode: bool = False,
-                  splits: int | None = None, ws: Workspace | None = None, keep: int = 0, bias: torch.Tensor | None = None) -> int:
+                  splits: int | None = None, ws: Workspace | None = None, keep: int = 0, bias: torch.Tensor | None = None,
+                  chunk: int = 0, pair: tuple[torch.Tensor, float, float] | None = None) -> int:
     """Windowed grouped-query attention over the paged cache of ``gqa_prepare``, ``conv_qkv`` or ``norm_qkv`` with values of
     ``dim`` channels, times ``out_scale``.  ``window`` 0: every earlier token; ``keep``: the first tokens stay visible behind the
     window; ``bias`` fp32 ``[distances, H]`` is added to the scaled scores, its last row from the last distance on; ``sink``:
-    score of a softmax entry without a value.  ``decode``: every segment has at most one row.
+    score of a softmax entry without a value.  ``chunk`` > 0 (instead of a window): a token sees its own chunk of positions, counted
+    from the sequence's first.  ``pair`` = (gate logits ``[T, H dim]``, factor, eps): query and key rows hold two maps, half of their
+    columns each, over the same values; the second map's output times the factor is taken from the first's, and the difference goes
+    over its root mean square, times ``out_scale`` and the sigmoid of the gate.  ``decode``: every segment has at most one row.
     ``splits``: key splits of the bf16 decode form (None: as many as fill the device).  Returns the launches made."""
     G, P = cache.shape[1], cache.shape[4]
     T = q.shape[0]
     assert q.is_contiguous() and q.shape[1] == heads * P and out.stride(1) == 1 and out.shape[1] == heads * dim
     assert q.dtype == out.dtype == cache.dtype and page_table.dtype == torch.int32
     assert bias is None or bias.dtype == torch.float32 and bias.is_contiguous() and bias.shape[1] == heads
+    gate, less, eps = pair or (None, 0.0, 0.0)
+    assert gate is None or gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == out.shape
+    maps = 1 if pair is None else 2
     f32 = q.dtype == torch.float32
     l = native.lib()
     partial = None
@@ -1062,19 +1095,21 @@ def gqa_attention(q: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor
         if splits is None:
             from .strategies import active
             units = ctypes.c_int(0)
-            l.cb_gqa_attn_partial_floats(T, seg.num, heads, G, P, 1, 1, ctypes.byref(units))
+            l.cb_gqa_attn_partial_floats(T, seg.num, heads, G, P, maps, 1, 1, ctypes.byref(units))
             a = active().attention
             # a block walks four pages at a time: no more splits than the longest row has such strides
-            keys = page_table.shape[1] * PAGE_TOKENS if window <= 0 else min(window + keep, page_table.shape[1] * PAGE_TOKENS)
+            most = chunk or (window + keep if window > 0 else 0)
+            keys = min(most or page_table.shape[1] * PAGE_TOKENS, page_table.shape[1] * PAGE_TOKENS)
             splits = min(a.max_splits, -(-keys // 64), max(1, a.target_ctas // units.value))
         if splits > 1:
             ws = ws or workspace(q.device)
-            ws.ensure_attn(l.cb_gqa_attn_partial_floats(T, seg.num, heads, G, P, 1, splits, None))
+            ws.ensure_attn(l.cb_gqa_attn_partial_floats(T, seg.num, heads, G, P, maps, 1, splits, None))
             partial = ws.attn.data_ptr()
     a = native.GqaAttnStruct(q.data_ptr(), out.data_ptr(), out.stride(0), cache.data_ptr(), page_table.data_ptr(),
-                             page_table.shape[1], heads, G, dim, P, window, keep, float(scale), float(out_scale),
-                             float("-inf") if sink is None else float(sink), _ptr(bias), 0 if bias is None else bias.shape[0] - 1, T,
-                             int(f32), int(decode), splits, partial)
+                             page_table.shape[1], heads, G, dim, P, window, keep, chunk, float(scale), float(out_scale),
+                             float("-inf") if sink is None else float(sink), _ptr(bias), 0 if bias is None else bias.shape[0] - 1,
+                             _ptr(gate), 0 if gate is None else gate.stride(0), float(less), float(eps), T, int(f32), int(decode), splits,
+                             partial)
     st = _seg(seg)
     native.check(l.cb_gqa_attn(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_gqa_attn")
     return 2 if splits > 1 else 1
@@ -1087,6 +1122,35 @@ def _qkv(x: torch.Tensor, offs: tuple[int, int, int], positions: torch.Tensor, s
     assert x.stride(1) == 1 and slots.dtype == positions.dtype == torch.int32 and x.shape[1] >= offs[2] + G * vdim
     return native.QkvPrepStruct(x.data_ptr(), x.stride(0), *offs, q.data_ptr(), cache.data_ptr(), slots.data_ptr(), positions.data_ptr(),
                                 heads, G, dim, vdim, P, float(eps), x.shape[0], int(x.dtype == torch.float32))
+
+
+def head_qkv(x: torch.Tensor, offs: tuple[int, int, int], q_norm: torch.Tensor, k_norm: torch.Tensor, freq: torch.Tensor,
+             positions: torch.Tensor, slots: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, heads: int, dim: int, vdim: int,
+             eps: float, maps: int = 1) -> None:
+    """Queries, keys and values at the columns ``offs`` of ``x``: every head (and map of it) of queries and keys over its root mean
+    square, times a weight per channel, then rotary positions of channel i with channel ``i + pairs`` (``freq`` fp32 ``[2, pairs]``:
+    radians per position and what rounding took from them).  Queries to ``q [T, H P]``, keys and values to
+    ``cache [pages, G, 2, 16, P]``; the maps of a head share its row of ``P`` columns evenly."""
+    assert q_norm.dtype == k_norm.dtype == freq.dtype == torch.float32 and q_norm.numel() == k_norm.numel() == dim
+    assert freq.is_contiguous() and freq.shape[0] == 2
+    a = native.HeadQkvStruct(_qkv(x, offs, positions, slots, q, cache, heads, dim, vdim, eps), q_norm.data_ptr(), k_norm.data_ptr(),
+                             freq.data_ptr(), freq.shape[1], maps)
+    native.check(native.lib().cb_head_qkv(ctypes.byref(a), _stream()), "cb_head_qkv")
+
+
+def mingru(x: torch.Tensor, z_off: int, x_off: int, g_off: int, bias: torch.Tensor, state: torch.Tensor, seg: GdnSegments,
+           out: torch.Tensor) -> None:
+    """Element-wise recurrence of ``out``'s channels: ``S <- (1 - z) S + z c`` with ``z`` = sigmoid of the columns ``z_off`` of ``x`` plus
+    ``bias[0]`` and the candidate ``c`` from the columns ``x_off`` plus ``bias[1]`` (``u + 1/2`` of ``u >= 0``, else its sigmoid);
+    ``out`` = ``S silu(x[:, g_off:])``.  ``state`` fp32 ``[slots, channels or more]`` is read (zero at position 0) and replaced."""
+    T, width = out.shape
+    assert x.dtype == out.dtype and x.stride(1) == out.stride(1) == 1 and x.shape[1] >= max(z_off, x_off, g_off) + width
+    assert state.dtype == bias.dtype == torch.float32 and bias.is_contiguous() and tuple(bias.shape) == (2, width)
+    assert state.stride(-1) == 1 and state.dim() == 2 and state.shape[1] >= width
+    a = native.MinGruStruct(x.data_ptr(), x.stride(0), z_off, x_off, g_off, bias.data_ptr(), state.data_ptr(), state.stride(0),
+                            out.data_ptr(), out.stride(0), width, T, int(x.dtype == torch.float32))
+    st = _seg(seg)
+    native.check(native.lib().cb_mingru(ctypes.byref(a), ctypes.byref(st), _stream()), "cb_mingru")
 
 
 def conv_qkv(x: torch.Tensor, offs: tuple[int, int, int], conv_w: torch.Tensor, state: torch.Tensor | None, freq: torch.Tensor,

@@ -271,7 +271,7 @@ def _declare(l: ctypes.CDLL) -> None:
         getattr(l, f"cb_{name}").argtypes = [vp, vp, vp]
         getattr(l, f"cb_{name}").restype = i
     l.cb_gated_parts_norm.argtypes = [vp, vp, i, vp, vp, i, i, i, i, f, i, vp]
-    l.cb_embed_rows.argtypes = [vp, vp, vp, vp, vp, i, i, i, i, f, i, vp]
+    l.cb_embed_rows.argtypes = [vp, vp, vp, vp, vp, i, i, i, i, f, f, i, i, vp]
     l.cb_add_norm_rows.argtypes = [vp, i, vp, vp, vp, vp, i, i, i, f, i, vp]
     l.cb_side_gate.argtypes = [vp, i, vp, i, vp, vp, i, i, vp, i, i, i, i, i, vp]
     l.cb_side_input.argtypes = [vp, vp]
@@ -279,19 +279,23 @@ def _declare(l: ctypes.CDLL) -> None:
     l.cb_side_input_fits.restype = i
     l.cb_gqa_prepare.argtypes = [vp, vp]
     l.cb_gqa_attn.argtypes = [vp, vp, vp]
-    l.cb_gqa_attn_partial_floats.argtypes = [i, i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
+    l.cb_gqa_attn_partial_floats.argtypes = [i, i, i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
     l.cb_gqa_attn_partial_floats.restype = ll
-    l.cb_conv_qkv.argtypes = [vp, vp, vp]
-    for name in ("norm_qkv", "stream_step", "stream_norm", "scored_moe_route"):
+    for name in ("conv_qkv", "mingru"):
+        getattr(l, f"cb_{name}").argtypes = [vp, vp, vp]
+        getattr(l, f"cb_{name}").restype = i
+    for name in ("head_qkv", "norm_qkv", "stream_step", "stream_norm", "scored_moe_route"):
         getattr(l, f"cb_{name}").argtypes = [vp, vp]
     l.cb_wq_gemm_grouped_relu2.argtypes = [vp, i, vp, vp, i, i, i, i, vp, i, i, i, vp, vp]
-    l.cb_latent_prepare.argtypes = [vp, i, i, i, i, i, vp, vp, vp, i, vp, i, vp, i, f, i, vp]
+    l.cb_latent_prepare.argtypes = [vp, vp]
+    l.cb_latent_attn_mma.argtypes = [i, i]
+    l.cb_latent_attn_mma.restype = i
     l.cb_latent_attn.argtypes = [vp, vp, vp]
     l.cb_latent_attn_partial_floats.argtypes = [i, i, i, i, i, i, ctypes.POINTER(ctypes.c_int)]
     l.cb_latent_attn_partial_floats.restype = ll
     for name in ("bf16_gemm_wide", "f32_gemm", "row_norm", "embed_norm", "concat_rows", "latent_prepare",
                  "latent_attn", "gated_parts_norm", "embed_rows", "add_norm_rows", "side_gate", "side_input",
-                 "gqa_prepare", "gqa_attn", "conv_qkv", "norm_qkv", "stream_step", "stream_norm", "scored_moe_route",
+                 "gqa_prepare", "gqa_attn", "head_qkv", "norm_qkv", "stream_step", "stream_norm", "scored_moe_route",
                  "wq_gemm_grouped_relu2"):
         getattr(l, f"cb_{name}").restype = i
     # fp8 (e4m3 x e4m3) tensor path: activation quantizers and the GEMM entries
@@ -337,7 +341,8 @@ class WideGemmStruct(ctypes.Structure):
                 ("y", ctypes.c_void_p), ("y32", ctypes.c_void_p), ("ldy", ctypes.c_int), ("residual32", ctypes.c_void_p),
                 ("y2", ctypes.c_void_p), ("ldy2", ctypes.c_int), ("n_split", ctypes.c_int), ("diag_n", ctypes.c_int),
                 ("M", ctypes.c_int), ("N", ctypes.c_int), ("K", ctypes.c_int), ("stream_k", ctypes.c_int),
-                ("splits", ctypes.c_int), ("min_units", ctypes.c_int), ("glu", ctypes.c_int)]
+                ("splits", ctypes.c_int), ("min_units", ctypes.c_int), ("glu", ctypes.c_int), ("glu_limit", ctypes.c_float),
+                ("rgate", ctypes.c_void_p), ("ldrg", ctypes.c_int), ("rgate_b", ctypes.c_void_p)]
 
 
 class F32GemmStruct(ctypes.Structure):
@@ -346,7 +351,8 @@ class F32GemmStruct(ctypes.Structure):
                 ("y", ctypes.c_void_p), ("ldy", ctypes.c_int), ("residual", ctypes.c_void_p), ("y2", ctypes.c_void_p),
                 ("ldy2", ctypes.c_int), ("n_split", ctypes.c_int), ("diag_n", ctypes.c_int), ("M", ctypes.c_int),
                 ("N", ctypes.c_int), ("K", ctypes.c_int), ("glu", ctypes.c_int), ("tiles", ctypes.c_void_p),
-                ("max_items", ctypes.c_int)]
+                ("max_items", ctypes.c_int), ("glu_limit", ctypes.c_float), ("rgate", ctypes.c_void_p), ("ldrg", ctypes.c_int),
+                ("rgate_b", ctypes.c_void_p)]
 
 
 class RecPrepStruct(ctypes.Structure):
@@ -371,12 +377,22 @@ class RecWalkStruct(ctypes.Structure):
                 ("sigmoid_gate", ctypes.c_int), ("decode", ctypes.c_int), ("tokens", ctypes.c_int), ("f32", ctypes.c_int)]
 
 
+class LatentPrepStruct(ctypes.Structure):
+    """Mirror of ``CbLatentPrep`` in ``csrc/latent_attn.cu``."""
+    _fields_ = [("proj", ctypes.c_void_p), ("ldp", ctypes.c_int), ("q_off", ctypes.c_int), ("q_rank", ctypes.c_int),
+                ("c_off", ctypes.c_int), ("R", ctypes.c_int), ("qw", ctypes.c_void_p), ("cw", ctypes.c_void_p),
+                ("cq", ctypes.c_void_p), ("ldq", ctypes.c_int), ("cache", ctypes.c_void_p), ("Rp", ctypes.c_int),
+                ("slots", ctypes.c_void_p), ("qr_off", ctypes.c_int), ("r_off", ctypes.c_int), ("col", ctypes.c_int),
+                ("pairs", ctypes.c_int), ("freq", ctypes.c_void_p), ("mult", ctypes.c_float), ("positions", ctypes.c_void_p),
+                ("ql", ctypes.c_void_p), ("H", ctypes.c_int), ("tokens", ctypes.c_int), ("eps", ctypes.c_float), ("f32", ctypes.c_int)]
+
+
 class LatentAttnStruct(ctypes.Structure):
     """Mirror of ``CbLatentAttn`` in ``csrc/latent_attn.cu``."""
     _fields_ = [("q", ctypes.c_void_p), ("out", ctypes.c_void_p), ("cache", ctypes.c_void_p), ("gate", ctypes.c_void_p),
                 ("ldg", ctypes.c_int), ("page_table", ctypes.c_void_p), ("max_pages", ctypes.c_int), ("H", ctypes.c_int),
-                ("Rp", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float), ("tokens", ctypes.c_int),
-                ("f32", ctypes.c_int), ("decode", ctypes.c_int), ("splits", ctypes.c_int), ("partial", ctypes.c_void_p)]
+                ("Rp", ctypes.c_int), ("Rv", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float),
+                ("tokens", ctypes.c_int), ("f32", ctypes.c_int), ("decode", ctypes.c_int), ("splits", ctypes.c_int), ("partial", ctypes.c_void_p)]
 
 
 class SideInputStruct(ctypes.Structure):
@@ -402,8 +418,9 @@ class GqaAttnStruct(ctypes.Structure):
     _fields_ = [("q", ctypes.c_void_p), ("out", ctypes.c_void_p), ("ldo", ctypes.c_int), ("cache", ctypes.c_void_p),
                 ("page_table", ctypes.c_void_p), ("max_pages", ctypes.c_int), ("H", ctypes.c_int), ("G", ctypes.c_int),
                 ("e", ctypes.c_int), ("P", ctypes.c_int), ("window", ctypes.c_int), ("keep", ctypes.c_int),
-                ("scale", ctypes.c_float), ("out_scale", ctypes.c_float), ("sink", ctypes.c_float), ("bias", ctypes.c_void_p),
-                ("bias_far", ctypes.c_int), ("tokens", ctypes.c_int), ("f32", ctypes.c_int),
+                ("chunk", ctypes.c_int), ("scale", ctypes.c_float), ("out_scale", ctypes.c_float), ("sink", ctypes.c_float),
+                ("bias", ctypes.c_void_p), ("bias_far", ctypes.c_int), ("gate", ctypes.c_void_p), ("ldg", ctypes.c_int),
+                ("less", ctypes.c_float), ("eps", ctypes.c_float), ("tokens", ctypes.c_int), ("f32", ctypes.c_int),
                 ("decode", ctypes.c_int), ("splits", ctypes.c_int), ("partial", ctypes.c_void_p)]
 
 
@@ -426,6 +443,20 @@ class NormQkvStruct(ctypes.Structure):
     """Mirror of ``CbNormQkv`` in ``csrc/qkv_prepare.cu``."""
     _fields_ = [("a", QkvPrepStruct), ("qw", ctypes.c_void_p), ("kw", ctypes.c_void_p), ("coef", ctypes.c_float),
                 ("every", ctypes.c_int)]
+
+
+class HeadQkvStruct(ctypes.Structure):
+    """Mirror of ``CbHeadQkv`` in ``csrc/qkv_prepare.cu``."""
+    _fields_ = [("a", QkvPrepStruct), ("qw", ctypes.c_void_p), ("kw", ctypes.c_void_p), ("freq", ctypes.c_void_p),
+                ("pairs", ctypes.c_int), ("maps", ctypes.c_int)]
+
+
+class MinGruStruct(ctypes.Structure):
+    """Mirror of ``CbMinGru`` in ``csrc/mingru.cu``."""
+    _fields_ = [("x", ctypes.c_void_p), ("ldx", ctypes.c_int), ("z_off", ctypes.c_int), ("x_off", ctypes.c_int),
+                ("g_off", ctypes.c_int), ("bias", ctypes.c_void_p), ("state", ctypes.c_void_p), ("lds", ctypes.c_int),
+                ("out", ctypes.c_void_p), ("ldo", ctypes.c_int), ("width", ctypes.c_int), ("tokens", ctypes.c_int),
+                ("f32", ctypes.c_int)]
 
 
 class StreamStepStruct(ctypes.Structure):
