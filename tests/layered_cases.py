@@ -148,7 +148,57 @@ STREAMS = {
     "str_wide": streams(256, 128, [near(40, 1, 72, 136, 4, 0.2, 64, 10000.0, 50, 35, routed(40, 6, 64, 9, 128)),
                                    far(20, 1, 200, 64, 0.1, 60, (0.3, 30), 96, 16), near(3, 1, 200, 256, 3, 0.1, 40, 300.0, 19, 65, 0)], 4, 3.0),
 }
-ALL = {**CASES, **SEQUENTIAL, **STREAMS}
+
+
+# ------------------------------------------------------------------ gated residuals (Fovunex)
+def clamped(ff, limit=2.0):
+    return {"kind": "dense", "ff": ff, "limit": limit} if ff else None
+
+
+def rotated(heads, dim, rot_dim, vdim, kv_rank, scale, base, yarn, mlp):
+    """Latent attention with a rotated key part; ``yarn``: (factor, original, fast, slow) or None."""
+    rot = {"dims": rot_dim, "base": base}
+    if yarn:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), yarn))
+    return {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank,
+                                                  "scale": scale, "rot": rot}, "mlp": mlp}
+
+
+def differential(heads, kv_heads, dim, vdim, scale, dims, base, diff, size, mlp):
+    """``size`` 0: every earlier token."""
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "diff": diff,
+                                           "rot": {"dims": dims, "base": base}, "mask": {"size": size} if size else None}, "mlp": mlp}
+
+
+def mingru(width, mlp):
+    return {"type": "mingru", "mixer": {"width": width}, "mlp": mlp}
+
+
+def gated(vocab, width, layers, loop=None, scale=1.0, eps=1e-5):
+    return {"architecture": "Fovunex", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": eps}, "embedding": {"scale": scale},
+            "loop": dict(zip(("start", "stop", "times"), loop)) if loop else None}
+
+
+GATED = {
+    # every mixer, a loop in the middle, grouped heads, stretched pairs, a layer without a feed-forward
+    "gat": gated(210, 96, [rotated(5, 16, 12, 40, 72, 0.3, 1000.0, (3.0, 40, 4.0, 0.5), clamped(80, 1.2)), mingru(72, clamped(96, 3.0)),
+                           differential(6, 2, 24, 40, 0.3, 12, 5000.0, 0.4, 37, clamped(72)), mingru(130, None),
+                           rotated(3, 24, 8, 16, 40, 0.25, 300.0, None, None)], (1, 3, 2), 0.7, 1e-6),
+    # single heads, unit sizes, a chunk of one token, a loop that runs once from the first layer on
+    "gat_small": gated(71, 64, [differential(1, 1, 16, 16, 0.25, 16, 100.0, 0.2, 1, clamped(48)), rotated(1, 16, 2, 16, 16, 0.25, 50.0, None, clamped(64, 0.5)),
+                                mingru(16, None)], (0, 2, 1)),
+    # odd widths, three query heads per key head, few rotated channels, every earlier token, the whole model looped three times
+    "gat_odd": gated(123, 68, [differential(9, 3, 13, 9, 0.5, 6, 50.0, 0.7, 0, clamped(44)), rotated(3, 20, 6, 13, 19, 0.35, 80.0, (4.0, 30, 2.0, 1.0), clamped(36, 0.8)),
+                               mingru(37, clamped(20)), differential(4, 1, 7, 21, 0.6, 0, 10.0, 0.1, 33, None)], (0, 4, 3), 2.5, 1e-4),
+    # wide heads, more query heads than a block has rows, latents of several widths, chunks over several pages
+    "gat_wide": gated(256, 128, [differential(40, 1, 72, 136, 0.15, 64, 10000.0, 0.5, 50, clamped(128)), rotated(40, 24, 64, 16, 512, 0.1, 10000.0, (8.0, 100, 32.0, 1.0), None),
+                                 rotated(2, 32, 100, 40, 500, 0.1, 500.0, None, clamped(96)), mingru(300, None),
+                                 differential(3, 3, 100, 250, 0.1, 40, 300.0, 0.3, 19, clamped(64))], (2, 4, 2), 3.0),
+    # a latent beside a rotated part that adds a group of columns, and one that fits in
+    "gat_latent": gated(150, 64, [rotated(4, 16, 32, 24, 120, 0.2, 700.0, None, clamped(40)), rotated(33, 8, 40, 8, 250, 0.2, 90.0, (2.0, 64, 8.0, 1.0), None),
+                                  rotated(6, 48, 16, 8, 44, 0.2, 2000.0, None, clamped(32))], None, 1.5),
+}
+ALL = {**CASES, **SEQUENTIAL, **STREAMS, **GATED}
 LOW_RANKS = (12, 20)          # inner sizes of the low-rank decay and gate projections
 
 
@@ -168,6 +218,9 @@ def tensors(cfg: dict, seed: int = 0) -> dict[str, torch.Tensor]:
         return out
     if cfg["architecture"] == "Vimelorn":
         _stream_tensors(cfg, mat, vec, out, g)
+        return out
+    if cfg["architecture"] == "Fovunex":
+        _gated_tensors(cfg, mat, vec, out, g)
         return out
     vec("embed.norm", W)
     vec("final.norm", W)
@@ -303,6 +356,50 @@ def _stream_tensors(cfg: dict, mat, vec, out: dict, g) -> None:
             mat(f"{p}.shared.up", mlp["shared"]["ff"], W)
             mat(f"{p}.shared.down", W, mlp["shared"]["ff"])
             mat(f"{p}.shared.sg", 1, W)
+
+
+def _gated_tensors(cfg: dict, mat, vec, out: dict, g) -> None:
+    W = cfg["width"]
+
+    def one(name):
+        out[name] = (1.0 + 0.3 * torch.randn((), generator=g)).to(torch.bfloat16)
+
+    out["embed"] = (out["embed"].float() / cfg["embedding"]["scale"]).to(torch.bfloat16)
+    one("final.norm")
+    mat("head", cfg["vocab"], W)
+    for i, l in enumerate(cfg["layers"]):
+        m, p, mlp = l["mixer"], f"l{i}.mix", l["mlp"]
+        for q in (1, 2) if mlp else (1,):
+            one(f"l{i}.norm{q}")
+            mat(f"l{i}.rg{q}", W, W, 1.5)
+            vec(f"l{i}.rg{q}.b", W, 0.3, 0.7)
+        if l["type"] == "latent_attention":
+            H, R = m["heads"], m["kv_rank"]
+            mat(f"{p}.q", H * (m["dim"] + m["rot_dim"]), W, 2.0)
+            mat(f"{p}.dkv", R + m["rot_dim"], W, 2.0)
+            vec(f"{p}.dkv.norm", R, 1.0, 0.3)
+            mat(f"{p}.uk", H * m["dim"], R, 2.0)
+            mat(f"{p}.uv", H * m["vdim"], R)
+            mat(f"{p}.o", W, H * m["vdim"])
+        elif l["type"] == "attention":
+            d = m["dim"]
+            for t, n in (("q", m["heads"] * 2 * d), ("k", m["kv_heads"] * 2 * d), ("v", m["kv_heads"] * m["vdim"]), ("g", m["heads"] * m["vdim"])):
+                mat(f"{p}.{t}", n, W)
+            for t in ("q", "k"):
+                vec(f"{p}.{t}.norm", d, 1.2, 0.4)
+            for t in ("lq1", "lk1", "lq2", "lk2"):
+                vec(f"{p}.{t}", d, 0.0, 0.7 / d ** 0.25)
+            mat(f"{p}.o", W, m["heads"] * m["vdim"])
+        else:
+            for t in "zxg":
+                mat(f"{p}.{t}", m["width"], W)
+            vec(f"{p}.z.b", m["width"], -2.0, 1.0)
+            vec(f"{p}.x.b", m["width"], 0.0, 0.5)
+            mat(f"{p}.o", W, m["width"])
+        if mlp:
+            for t in ("gate", "up"):
+                mat(f"l{i}.mlp.{t}", mlp["ff"], W, 1.5)
+            mat(f"l{i}.mlp.down", W, mlp["ff"])
 
 
 def write(path, cfg: dict, weights: dict[str, torch.Tensor]):

@@ -9,8 +9,8 @@ import torch
 from torch.overrides import TorchFunctionMode
 
 sys.path.insert(0, str(Path(__file__).parent))
-from layered_cases import (ALL, channel, config, delta, far, latent, mamba2, near, parallel, prompt, routed, sequential,  # noqa: E402
-                           streams, tensors, write)
+from layered_cases import (ALL, channel, clamped, config, delta, differential, far, gated, latent, mamba2, mingru, near,  # noqa: E402
+                           parallel, prompt, rotated, routed, sequential, streams, tensors, write)
 
 from cubic_serve_b200.models import layered_reference as R  # noqa: E402
 
@@ -368,7 +368,7 @@ def test_latent_prepare_norms_and_pages(dtype):
     cq = torch.zeros(T, 64, dtype=dtype, device=DEV)
     cache = torch.zeros(4, 16, rp, dtype=dtype, device=DEV)
     slots = torch.tensor([17, 63, -1, 0, 32], dtype=torch.int32)
-    K.latent_prepare(proj.to(DEV), qr, off, rank, qn.to(DEV), cn.to(DEV), cq, cache, slots.to(DEV), 1e-4)
+    K.latent_prepare(proj.to(DEV), off, rank, cn.to(DEV), cache, slots.to(DEV), 1e-4, low=(0, qr, qn.to(DEV), cq))
     p = proj.double()
     close(cq[:, :qr], R.rms(p[:, :qr], 1e-4) * qn.double(), dtype, exact=1e-6, rough=6e-3)
     assert (cq[:, qr:] == 0).all()
@@ -459,7 +459,7 @@ def test_prefill_portions_and_decode_agree(tmp_path, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("name, runs", [("all", 6), ("seq", 4), ("str", 5)])
+@pytest.mark.parametrize("name, runs", [("all", 6), ("seq", 4), ("str", 5), ("gat", 7), ("gat_odd", 12)])
 def test_residual_after_every_run(tmp_path, name, runs, dtype):
     s, raw, oracle = session_for(tmp_path, name, dtype)
     ids = prompt(raw, 40, 9)
@@ -474,7 +474,7 @@ def test_residual_after_every_run(tmp_path, name, runs, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("name", ["all", "odd", "seq", "seq_odd", "str", "str_odd", "str_select"])
+@pytest.mark.parametrize("name", ["all", "odd", "seq", "seq_odd", "str", "str_odd", "str_select", "gat", "gat_odd"])
 def test_unequal_requests_share_steps_pages_and_slots(tmp_path, name, dtype):
     """Up to four live requests, portions beside single tokens, requests that pause, end and make room for others in a pool
     that is too small for all of them."""
@@ -521,7 +521,9 @@ def test_unequal_requests_share_steps_pages_and_slots(tmp_path, name, dtype):
                         mamba2(2, 24, 16, 1, 4, 2, 48), parallel((3, 1, 24, 17, 0.4, 8, 80.0, None), (1, 20, 16, 4.0), (0.8, 1.1), 0)], 8),
     streams(90, 64, [near(4, 2, 16, 24, 4, 0.6, 16, 300.0, 70, 9, routed(4, 2, 32, 1, 32)), far(3, 1, 16, 16, 0.5, 60, (0.5, 32), 64, 12),
                      near(3, 3, 24, 16, 2, 0.5, 8, 80.0, 17, 33, 0)], 2, 3.0),
-], ids=["Bumodra", "Loduzen", "Vimelorn"])
+    gated(90, 64, [differential(4, 2, 16, 24, 0.5, 16, 300.0, 0.4, 70, clamped(64)), mingru(48, clamped(48, 1.0)),
+                   rotated(3, 16, 8, 16, 40, 0.4, 300.0, (3.0, 60, 8.0, 1.0), None), differential(3, 3, 24, 16, 0.5, 8, 80.0, 0.2, 17, None)], (1, 3, 2), 0.8),
+], ids=["Bumodra", "Loduzen", "Vimelorn", "Fovunex"])
 def test_long_decoding_passes_the_window(tmp_path, raw, dtype):
     """Decoded tokens move every window past the prompt; first tokens of the sequence included."""
     s, raw, oracle = session_for(tmp_path, "", dtype, raw=raw)
@@ -563,7 +565,8 @@ def test_far_tokens_reach_through_kept_places_and_the_biased_layer(tmp_path):
 @pytest.mark.parametrize("raw", [
     config(80, 64, [channel(2, 1, 32, 32, 3, 64), delta(2, 2, 32, 32, 4, 64)]),
     sequential(80, 64, [mamba2(2, 32, 24, 2, 3, 1, 64), parallel((2, 1, 16, 9, 0.3, 8, 100.0, None), (2, 24, 24, 16.0), (0.8, 1.5), 64)], 8),
-], ids=["Bumodra", "Loduzen"])
+    gated(80, 64, [mingru(96, clamped(64)), differential(2, 1, 16, 24, 0.3, 8, 100.0, 0.3, 9, clamped(64))], (0, 1, 2)),
+], ids=["Bumodra", "Loduzen", "Fovunex"])
 def test_far_token_reaches_through_the_state(tmp_path, raw):
     """With slow decays and no attention that far back, changing an early token moves the logits as the oracle says."""
     w = tensors(raw, 3)
@@ -572,6 +575,8 @@ def test_far_token_reaches_through_the_state(tmp_path, raw):
             w[n] = torch.full_like(w[n], -7.0)
         elif n.endswith(".a2.b"):
             w[n] = torch.full_like(w[n], 5.0)
+        elif n.endswith(".z.b"):
+            w[n] = torch.full_like(w[n], -6.0)
     from cubic_serve_b200.runtime.imposed import ImposedSession
     from cubic_serve_b200.utils.trace_run import build_engine
     s = ImposedSession(build_engine(str(write(tmp_path, raw, w)), "float32", 512))
@@ -614,7 +619,9 @@ def serving_backend(model, *flags):
     config(300, 64, [delta(2, 1, 16, 16, 3, 64), latent(2, 16, 16, 24, 32, 20, 0.25, 0), channel(2, 2, 16, 16, 2, 48)], (0, 2, 2)),
     sequential(300, 64, [mamba2(2, 16, 8, 1, 3, 2, 48), parallel((4, 2, 16, 20, 0.3, 8, 90.0, (2.0, 50, 4.0, 1.0)), (2, 12, 16, 8.0), (0.9, 0.8), 64)], 8),
     streams(300, 64, [near(4, 2, 16, 24, 3, 0.5, 8, 90.0, 20, 3, routed(4, 2, 32, 1, 24)), far(2, 1, 16, 16, 0.3, 20, (0.4, 8), 48)], 2, 3.0),
-], ids=["Bumodra", "Loduzen", "Vimelorn"])
+    gated(300, 64, [rotated(2, 16, 8, 16, 32, 0.3, 90.0, (2.0, 50, 4.0, 1.0), clamped(64)), mingru(48, None),
+                    differential(4, 2, 16, 24, 0.3, 8, 90.0, 0.4, 20, clamped(48))], (1, 3, 2), 0.5),
+], ids=["Bumodra", "Loduzen", "Vimelorn", "Fovunex"])
 def test_greedy_generation_through_the_serving_stack(tmp_path, raw, prefix):
     """``cubic serve`` with --dtype float32: scheduler, prefix cache with state snapshots, overlapped decode graphs, sampler."""
     from cubic_serve_b200.runtime.scheduler import SamplingParams
@@ -631,7 +638,7 @@ def test_greedy_generation_through_the_serving_stack(tmp_path, raw, prefix):
     eng.executor.runner.ws.check_status()
 
 
-@pytest.mark.parametrize("name", ["all", "seq", "str"])
+@pytest.mark.parametrize("name", ["all", "seq", "str", "gat"])
 def test_bf16_serving_samples_and_preempts(tmp_path, name):
     """bf16 through the same stack: greedy tokens are the oracle's wherever its margin is clear, seeded sampling repeats, and a
     pool that is too small for all requests recomputes the preempted ones to the same tokens."""
