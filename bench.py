@@ -57,9 +57,9 @@ def parse_args():
     ap.add_argument("--no-check", action="store_true", help="skip the untimed multi-GPU logit check")
     ap.add_argument("--accept", type=float, default=0.7,
                     help="forced per-depth acceptance probability of speculative rounds (random weights never agree)")
-    ap.add_argument("--layered", nargs="?", const="all", choices=("all", "parallel", "sequential", "streams"), default=None,
+    ap.add_argument("--layered", nargs="?", const="all", choices=("all", "parallel", "sequential", "streams", "gated"), default=None,
                     help="instead of the headline workload: the layered decoders (with parallel layers, sequential layers, "
-                         "residual streams, or all) beside the closest existing model at equal size, one JSON line per kernel "
+                         "residual streams, gated residuals, or all) beside the closest existing model at equal size, one JSON line per kernel "
                          "and per model (one GPU)")
     return ap.parse_args()
 

@@ -4,7 +4,8 @@ throughput of whole models (``bench.py --layered``).
 The closest model is the hybrid family (Gated DeltaNet layers with periodic full attention) with bf16 weights; its SwiGLU
 feed-forward has three matrices where a parallel layer's has two, so its width is two thirds of that: equal parameters (the
 sequential layers have the same three matrices).  For the layers on several residual streams it is the family of grouped-query
-decoders with routed experts: an expert there has three matrices where one here has two, so its width is two thirds.
+decoders with routed experts: an expert there has three matrices where one here has two, so its width is two thirds.  The layers with
+gated residuals have two square matrices more each: their feed-forwards are narrower by that.
 
 Weights are random, prompts are random ids, one GPU.  Kernel times are CUDA-event times inside CUDA graphs with L2 flushed; the
 roofline of a kernel is the slower of its bytes over the copy bandwidth and its operations over the pipe that runs them.
@@ -17,8 +18,8 @@ from pathlib import Path
 import torch
 
 from ..models.config import ModelConfig, QuantSpec
-from ..models.layered import (AttentionSpec, BiasedAttentionSpec, ConvAttentionSpec, DeltaSpec, GatedLinearSpec, LatentSpec,
-                              LayeredConfig, LayerSpec, PairSpec, RotarySpec, RoutedSpec, SsdSpec)
+from ..models.layered import (AttentionSpec, BiasedAttentionSpec, ConvAttentionSpec, DeltaSpec, DifferentialSpec, GatedLinearSpec,
+                              LatentSpec, LayeredConfig, LayerSpec, MinGruSpec, PairSpec, RotarySpec, RoutedSpec, SsdSpec)
 from ..ops import kernels as K, wq_pack
 from ..utils.kernel_bench import DEV, timeit_graph
 
@@ -68,6 +69,21 @@ def streams_config(width: int, layers: int) -> LayeredConfig:
     far = LayerSpec(BiasedAttentionSpec(h, max(1, h // 4), 128, 128, 128 ** -0.5, 32, 512, 0.1, 4096), routed=routed)
     return LayeredConfig(f"streams-{width}", 32768, width, (near, near, near, far) * (layers // 4), 1e-6, architecture="Vimelorn",
                          streams=2, embed_scale=width ** 0.5)
+
+
+YARN = ("yarn", 4.0, 8192.0, 32.0, 1.0, 1.14)
+
+
+def gated_config(width: int, layers: int) -> LayeredConfig:
+    """Real-model layers with gated residuals at ``width``: differential attention (two maps of 64 over values of 128, four heads per
+    key head, chunks of 2048), an element-wise recurrence of 1.5 x width, latent attention over every earlier token (latents of 512
+    beside a rotated part of 64)."""
+    h, ff = width // 128, 5 * width // 4
+    pair = LayerSpec(DifferentialSpec(h, max(1, h // 4), 64, 128, 0.125, RotarySpec(64, 1e6), 0.6, 2048), ff, limit=7.0)
+    gru = LayerSpec(MinGruSpec(3 * width // 2), ff, limit=7.0)
+    latent = LayerSpec(LatentSpec(h, 128, 128, 0, 512, 192 ** -0.5, 0, 64, RotarySpec(64, 1e6, YARN), False), ff, limit=7.0)
+    return LayeredConfig(f"gated-{width}", 32768, width, (pair, gru, pair, latent) * (layers // 4), 1e-6, architecture="Fovunex",
+                         embed_scale=1.0)
 
 
 def experts_config(width: int, layers: int) -> ModelConfig:
@@ -352,6 +368,103 @@ def bench_latent(requests: int, tokens: int, ctx: int, heads: int, rank: int, wi
                   keys * rank * 2 + 2 * T * heads * rank * 2, 4.0 * pairs * heads * rank, pk["bf16"], pk)]
 
 
+def _paged(requests: int, tokens: int, ctx: int):
+    """Shuffled pages, positions and cache rows of the last ``tokens`` of ``ctx`` tokens of every request."""
+    per = -(-ctx // 16)
+    table = (torch.randperm(requests * per, device=DEV).to(torch.int32) + 1).view(requests, per)
+    pos = torch.arange(ctx - tokens, ctx, device=DEV, dtype=torch.int32).repeat(requests)
+    at = pos.view(requests, tokens)
+    return table, pos, (table.long().gather(1, (at // 16).long()) * 16 + at % 16).to(torch.int32).view(-1)
+
+
+def bench_rotated(requests: int, tokens: int, ctx: int, heads: int, flush, pk) -> list[dict]:
+    """Latents of 512 beside a rotated part of 64, and the same attention over latents alone."""
+    rank, rot, T = 512, 64, requests * tokens
+    spec = LatentSpec(heads, 128, 128, 0, rank, 1.0, 0, rot, RotarySpec(rot, 1e6, YARN), False)
+    rp, rv = spec.row_padded, spec.rank_padded
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    table, pos, slots = _paged(requests, tokens, ctx)
+    seg = _segments(requests, tokens, ctx - tokens)
+    cache = torch.randn(table.numel() + 1, 16, rp, **bf)
+    proj, cn, freq = torch.randn(T, heads * rot + rank + rot, **bf), torch.ones(rank, device=DEV), spec.rotary.split_table().to(DEV)
+    q, out = torch.randn(T, heads * rp, **bf) * 0.05, torch.empty(T, heads * rv, **bf)
+    prep = timeit_graph(lambda: K.latent_prepare(proj, heads * rot, rank, cn, cache, slots, 1e-6,
+                                                 rotated=(0, heads * rot + rank, rank, freq, 1.14, pos, q, heads)), flush, launches=5)
+    decode = tokens == 1
+    ms = timeit_graph(lambda: K.latent_attention(q, None, cache, table, seg, out, heads, 0, 0.1, decode=decode), flush, launches=5)
+    pairs, keys = requests * _visible(tokens, ctx, 0), requests * ctx
+    shape = f"{requests} x {tokens} at {ctx}, {heads} heads"
+    res = [_line(f"latent_prepare rotated [{shape}]", prep, T * 2 * (2 * heads * rot + 2 * (rank + rot)), 0, 1, pk),
+           _line(f"latent_attn rank 512 + 64 rotated [{shape}]", ms, keys * rp * 2 + T * heads * (rp + rv) * 2, 2.0 * pairs * heads * (rp + rv), pk["bf16"], pk)]
+    del q, out, cache
+    lowq, cq = torch.randn(T, 1536 + rank, **bf), torch.empty(T, 1536, **bf)
+    plain = torch.randn(table.numel() + 1, 16, rank, **bf)
+    qn = torch.ones(1536, device=DEV)
+    lp = timeit_graph(lambda: K.latent_prepare(lowq, 1536, rank, cn, plain, slots, 1e-6, low=(0, 1536, qn, cq)), flush, launches=5)
+    del plain
+    return res + [_line(f"latent_prepare low-rank queries [{shape}]", lp, T * 4 * (1536 + rank), 0, 1, pk),
+                  *bench_latent(requests, tokens, ctx, heads, rank, 0, flush, pk)]
+
+
+def bench_pair(requests: int, tokens: int, ctx: int, heads: int, kv_heads: int, flush, pk) -> list[dict]:
+    """Differential attention in chunks of 2048 and its preparation, beside attention with one map over as many keys."""
+    d, e, chunk, T = 64, 128, 2048, requests * tokens
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    table, pos, slots = _paged(requests, tokens, ctx)
+    seg = _segments(requests, tokens, ctx - tokens)
+    cache = torch.randn(table.numel() + 1, kv_heads, 2, 16, 128, **bf)
+    offs = (0, heads * 128, (heads + kv_heads) * 128)
+    x, q, out, gate = torch.randn(T, (heads + 2 * kv_heads) * 128, **bf), torch.empty(T, heads * 128, **bf), torch.empty(T, heads * e, **bf), torch.randn(T, heads * e, **bf)
+    w, freq = torch.ones(d, device=DEV), RotarySpec(d, 1e6).split_table().to(DEV)
+    decode = tokens == 1
+    prep = timeit_graph(lambda: K.head_qkv(x, offs, w, w, freq, pos, slots, q, cache, heads, d, e, 1e-6, 2), flush, launches=5)
+    ms = timeit_graph(lambda: K.gqa_attention(q, cache, table, seg, out, heads, e, 0, 0.125, out_scale=0.4, decode=decode, chunk=chunk,
+                                              pair=(gate, 0.8, 1e-6)), flush, launches=5)
+    one = timeit_graph(lambda: K.gqa_attention(q, cache, table, seg, out, heads, e, 0, 0.09, decode=decode, chunk=chunk), flush, launches=5)
+    pairs = requests * sum(p % chunk + 1 for p in range(ctx - tokens, ctx))
+    lo = (ctx - tokens) // chunk * chunk
+    kv = requests * (ctx - lo) * kv_heads * 2 * 128 * 2
+    shape = f"{requests} x {tokens} at {ctx}, {heads}/{kv_heads} heads"
+    return [_line(f"head_qkv two maps [{shape}]", prep, T * 2 * (heads + 2 * kv_heads) * 128 * 2, 0, 1, pk),
+            _line(f"gqa_attention differential [{shape}]", ms, kv + T * heads * 3 * 128 * 2, 2.0 * pairs * heads * 2 * (d + e), pk["bf16"], pk),
+            _line(f"gqa_attention one map, same keys [{shape}]", one, kv + T * heads * 2 * 128 * 2, 4.0 * pairs * heads * 128, pk["bf16"], pk),
+            *bench_qkv(requests, tokens, ctx, heads, kv_heads, flush, pk)[:3]]
+
+
+def bench_mingru(requests: int, tokens: int, width: int, flush, pk) -> list[dict]:
+    T = requests * tokens
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    x, out, bias, state = torch.randn(T, 3 * width, **bf), torch.empty(T, width, **bf), torch.zeros(2, width, device=DEV), torch.zeros(requests, width, device=DEV)
+    seg = _segments(requests, tokens, 5)
+    ms = timeit_graph(lambda: K.mingru(x, 0, width, 2 * width, bias, state, seg, out), flush, launches=5)
+    return [_line(f"mingru [{requests} x {tokens} tokens, width {width}]", ms, T * width * 8 + requests * width * 8, 0, 1, pk)]
+
+
+def bench_gated_products(m: int, width: int, flush, pk) -> list[dict]:
+    """Products whose epilogues gate, clamp and add, beside the plain ones of the same shapes; the entry of a loop's later pass."""
+    ff = 2 * width
+    bf = dict(dtype=torch.bfloat16, device=DEV)
+    h, x = torch.randn(m, width, **bf), torch.randn(m, width, device=DEV)
+    w = wq_pack.swiglu_interleave(wq_pack.pack_bf16(torch.randn(2 * ff, width, **bf) * 0.02))
+    both = wq_pack.PackedWeight(w.fmt, w.n + width, w.k, w.k, torch.cat([w.codes, torch.randn(width, width, **bf) * 0.02]), None, act_interleaved=True)
+    plain = wq_pack.pack_bf16(both.codes)
+    act, rg, y = torch.empty(m, ff, **bf), torch.randn(m, width, **bf), torch.empty(m, both.n, **bf)
+    down, bias, yo = wq_pack.pack_bf16(torch.randn(width, ff, **bf) * 0.02), torch.zeros(width, device=DEV), torch.empty(m, width, **bf)
+    table, ids, nw = torch.randn(4096, width, **bf), torch.randint(0, 4096, (m,), device=DEV, dtype=torch.int32), torch.ones(width, device=DEV)
+    out = []
+    for name, fn, n, k, extra in (
+            ("wide_gemm [gate, up | residual gate] (clamped)", lambda: K.wide_gemm(h, both, act, glu="clamped", limit=7.0, rest=rg, split=2 * ff), both.n, width, -m * ff * 2),
+            ("wq_gemm bf16, same shape", lambda: K.wq_gemm(h, plain, out=y), both.n, width, 0),
+            ("wide_gemm down (gated fp32 residual)", lambda: K.wide_gemm(act, down, x, residual=x, gate=(rg, bias)), width, ff, m * width * 8),
+            ("wq_gemm bf16, same shape", lambda: K.wq_gemm(act, down, out=yo), width, ff, 0)):
+        out.append(_line(f"{name} [{m} x {n} x {k}]", timeit_graph(fn, flush, launches=5), (n * k + m * (n + k)) * 2 + extra, 2.0 * m * n * k, pk["bf16"], pk))
+    again = timeit_graph(lambda: K.embed_rows(ids, table, nw, x, h, 1e-6, 0.0, add=True), flush, launches=5)
+    rn = timeit_graph(lambda: K.row_norm(x, nw, h, 1e-6), flush, launches=5)
+    K.workspace(torch.device(DEV)).check_status()
+    return out + [_line(f"embedding added + norm [{m} x {width}]", again, m * width * 12, 0, 1, pk),
+                  _line(f"row_norm fp32 in [{m} x {width}]", rn, m * width * 6, 0, 1, pk)]
+
+
 def bench_paged(requests: int, tokens: int, ctx: int, hq: int, hkv: int, flush, pk) -> list[dict]:
     from ..ops import eager
     d, T, per = 128, requests * tokens, -(-ctx // 16)
@@ -457,6 +570,24 @@ def streams_kernels(width: int = 4096) -> list[dict]:
     return out
 
 
+def gated_kernels(width: int = 4096) -> list[dict]:
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=DEV)
+    pk = peaks()
+    h = width // 128
+    out = []
+    for requests, tokens in ((256, 1), (8, 1024), (1, 4096)):
+        out += bench_mingru(requests, tokens, 3 * width // 2, flush, pk)
+        out += bench_gated_linear(requests, tokens, h // 2, flush, pk)
+        out += bench_gdn(requests, tokens, h, h // 2, flush, pk)
+    for requests, tokens, ctx in ((256, 1, 1280), (1, 1, 4096), (8, 1024, 1024), (1, 4096, 4096)):
+        out += bench_pair(requests, tokens, ctx, h, max(1, h // 4), flush, pk)
+        out += bench_rotated(requests, tokens, ctx, h, flush, pk)
+        out += bench_paged(requests, tokens, ctx, h, max(1, h // 4), flush, pk)
+    for m in (16, 256, 4096):
+        out += bench_gated_products(m, width, flush, pk)
+    return out
+
+
 # ------------------------------------------------------------------ whole models
 def model_throughput(cfg, concurrency: int, prompt: int, steps: int, warmup: int = 4, budget: int = 8192) -> dict:
     """Prefill and decode rates of a random model through the serving engine."""
@@ -516,9 +647,9 @@ def model_throughput(cfg, concurrency: int, prompt: int, steps: int, warmup: int
     return out
 
 
-KERNELS = {"parallel": kernels, "sequential": sequential_kernels, "streams": streams_kernels}
+KERNELS = {"parallel": kernels, "sequential": sequential_kernels, "streams": streams_kernels, "gated": gated_kernels}
 MODELS = {"parallel": (layered_config, hybrid_config), "sequential": (sequential_config, hybrid_config),
-          "streams": (streams_config, experts_config)}
+          "streams": (streams_config, experts_config), "gated": (gated_config, hybrid_config)}
 
 
 def run(steps: int = 32, designs: str = "all") -> None:

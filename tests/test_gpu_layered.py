@@ -673,7 +673,7 @@ def test_bf16_serving_samples_and_preempts(tmp_path, name):
         assert same > 8                                         # recomputed context: equal to rounding
 
 
-@pytest.mark.parametrize("name", ["small", "seq_small", "str_small"])
+@pytest.mark.parametrize("name", ["small", "seq_small", "str_small", "gat_small"])
 def test_trace_run_program(tmp_path, name):
     """The program itself: lines in, files out, two requests in one step, exit code 0."""
     import json

@@ -10,8 +10,9 @@ import pytest
 import torch
 
 sys.path.insert(0, str(Path(__file__).parent))
-from layered_cases import (ALL, CASES, LOW_RANKS, SEQUENTIAL, STREAMS, channel, config, delta, far, latent, mamba2, near,  # noqa: E402
-                           parallel, prompt, routed, sequential, streams, tensors, write)
+from layered_cases import (ALL, CASES, GATED, LOW_RANKS, SEQUENTIAL, STREAMS, channel, clamped, config, delta, differential,  # noqa: E402
+                           far, gated, latent, mamba2, mingru, near, parallel, prompt, rotated, routed, sequential, streams, tensors,
+                           write)
 
 from cubic_serve_b200.models import layered as L  # noqa: E402
 from cubic_serve_b200.models import layered_reference as R  # noqa: E402
@@ -105,7 +106,7 @@ def test_sequential_checkpoint_admission(tmp_path):
 
 
 def test_random_weights_of_all_designs_are_admitted(tmp_path):
-    for name in ("layered-tiny", "layered-seq-tiny", "layered-streams-tiny"):
+    for name in ("layered-tiny", "layered-seq-tiny", "layered-streams-tiny", "layered-gated-tiny"):
         cfg = L.NAMED[name]()
         back = admit_checkpoint(L.write_checkpoint(tmp_path / name, cfg, L.random_tensors(cfg, 3))).cfg
         assert (back.layers, back.side_dim, back.loop) == (cfg.layers, cfg.side_dim, cfg.loop)
@@ -166,6 +167,71 @@ def test_stream_checkpoint_admission(tmp_path):
     assert {o.semantic_op for o in decoder_step_operators(ck.cfg, 8)} >= {"attention.gqa", "moe.route", "residual.streams"}
     plain, _ = parsed("str_small")
     assert not plain.is_hybrid and ModelSpec.from_layered(plain).state is None          # one tap: nothing to remember
+
+
+@pytest.mark.parametrize("change, message", [
+    (lambda c: c["layers"][0].update(type="delta"), "unknown mixer"),
+    (lambda c: c["layers"][0]["mlp"].update(kind="moe"), "unknown feed-forward"),
+    (lambda c: c["layers"][0]["mlp"].update(limit=0), "positive limit"),
+    (lambda c: c["layers"][0]["mixer"]["rot"].update(dims=10), "rotated as a whole"),
+    (lambda c: c["layers"][0]["mixer"].update(kv_rank=1020), "with their rotated part"),
+    (lambda c: c["layers"][0]["mixer"].update(rot_dim=0), "come together"),
+    (lambda c: c["layers"][2]["mixer"].update(kv_heads=4), "grouped evenly"),
+    (lambda c: c["layers"][2]["mixer"].update(dim=129), "128 channels"),
+    (lambda c: c["layers"][2]["mixer"].update(vdim=257), "256 channels"),
+    (lambda c: c["layers"][2]["mixer"]["rot"].update(dims=26), "inside a head"),
+    (lambda c: c["layers"][2]["mixer"]["mask"].update(size=0), "at least the token itself"),
+    (lambda c: c["layers"][1]["mixer"].update(width=0), "positive width"),
+    (lambda c: c["loop"].update(start=3), "loop needs"),
+])
+def test_bad_gated_configurations_are_refused(change, message):
+    c = copy.deepcopy(GATED["gat"])
+    change(c)
+    with pytest.raises(L.LayeredConfigError, match=message):
+        L.parse_layered_config(c, {n: tuple(t.shape) for n, t in tensors(GATED["gat"]).items()})
+
+
+def test_gated_checkpoint_admission(tmp_path):
+    from cubic_serve_b200.contracts.model import ModelSpec
+    from cubic_serve_b200.contracts.plan import decoder_step_operators
+    from cubic_serve_b200.models import registry
+    raw, w = GATED["gat"], tensors(GATED["gat"])
+    ck = admit_checkpoint(write(tmp_path / "good", raw, w))
+    assert ck.cfg.family == "layered" and registry.for_architecture("Fovunex").family == "layered" and ck.cfg.embed_scale == 0.7
+    info = inspect_checkpoint(tmp_path / "good")
+    assert info["mixers"] == {"differential": 1, "latent": 2, "mingru": 2} and tuple(info["loop"]) == (1, 3, 2) and info["layer_runs"] == 7
+    # what a missing feed-forward would need is tolerated, anything else is not
+    admit_checkpoint(write(tmp_path / "spare", raw, {**w, "l3.norm2": w["l1.norm2"].clone(), "l3.rg2": w["l1.rg2"].clone()}))
+    with pytest.raises(CheckpointError, match="does not own"):
+        admit_checkpoint(write(tmp_path / "extra", raw, {**w, "loop.in": w["l0.rg1"].clone()}))
+    with pytest.raises(CheckpointError, match="missing tensor l1.rg1.b"):
+        admit_checkpoint(write(tmp_path / "missing", raw, {n: t for n, t in w.items() if n != "l1.rg1.b"}))
+    with pytest.raises(CheckpointError, match="expected \\(\\)"):
+        admit_checkpoint(write(tmp_path / "norm", raw, {**w, "l0.norm1": torch.ones(96).to(torch.bfloat16)}))
+    # rows of [72 | 12] and [40 | 8] in 128 and 64 columns, keys of two maps and values of 64; the looped layers' states and caches twice
+    spec = ModelSpec.from_layered(ck.cfg)
+    assert spec.cache.runs == 4 and spec.cache.page_bytes == 16 * 2 * (128 + 64 + 2 * 2 * 2 * 64)
+    assert spec.state.runs == 3 and ck.cfg.state_bytes_per_request == 4 * (2 * 72 + 132) and ck.cfg.is_hybrid
+    assert {o.semantic_op for o in decoder_step_operators(ck.cfg, 8)} >= {"attention.latent", "attention.differential", "residual.gate",
+                                                                          "linear_recurrence.elementwise"}
+
+
+@pytest.mark.parametrize("rank, rot, widths", [(72, 12, (128, 128)), (120, 8, (128, 128)), (121, 6, (192, 128)), (128, 64, (192, 128)), (129, 8, (256, 256)),
+                                               (256, 64, (320, 256)), (256, 66, (512, 512)), (512, 64, (576, 512)), (512, 66, (1024, 1024)),
+                                               (44, 16, (64, 64)), (449, 8, (512, 512))])
+def test_widths_of_rotated_rows(rank, rot, widths):
+    m = L.LatentSpec(1, 8, 8, 0, rank, 1.0, 0, rot, L.RotarySpec(rot, 10.0), False)
+    m.validate()
+    assert (m.row_padded, m.rank_padded) == widths and m.rot_col % 8 == 0 and m.rot_col >= rank
+
+
+def test_passes_of_a_loop_add_the_embedding_before_all_but_the_first():
+    cfg, _ = parsed("gat")
+    assert [i for i, _ in cfg.runs] == [0, 1, 2, 1, 2, 3, 4] and [r for r in range(7) if cfg.reenters(r)] == [3]
+    first, _ = parsed("gat_odd")
+    assert [r for r in range(len(first.runs)) if first.reenters(r)] == [4, 8]
+    once, _ = parsed("gat_small")
+    assert not any(once.reenters(r) for r in range(3)) and not any(parsed("all")[0].reenters(r) for r in range(6))
 
 
 def test_checkpoint_admission(tmp_path):
@@ -303,6 +369,50 @@ def test_stream_packing():
     assert torch.equal(packed.lm_head.codes.float()[:, :W], w["head"].float()) and packed.nbytes() > 0
 
 
+def test_gated_packing():
+    """Sections of the projection, where the absorbed queries are read, gate rows behind both products that read a norm."""
+    from cubic_serve_b200.ops import wq_pack
+    cfg, w = parsed("gat")
+    W = cfg.hidden_size
+    p = L.pack_layer(cfg, 0, w.__getitem__)
+    m, rows = p.mixer, p.proj.codes.float()[:, :W]
+    q = w["l0.mix.q"].float().view(5, 28, W)
+    hp, kg = m.absorb.heads, m.absorb.w.k
+    for h in range(5):
+        c = m.q_off + h // hp * kg + h % hp * 16
+        assert torch.equal(rows[c:c + 16], q[h, :16])
+    assert torch.equal(rows[m.qr_off:m.qr_off + 60], q[:, 16:].reshape(60, W)) and m.qr_off >= -(-5 // hp) * kg
+    down = w["l0.mix.dkv"].float()
+    assert torch.equal(rows[m.c_off:m.c_off + 72], down[:72]) and torch.equal(rows[m.r_off:m.r_off + 12], down[72:])
+    assert torch.equal(rows[p.rg_off:p.rg_off + W], w["l0.rg1"].float()) and p.split == p.proj.n
+    assert all(o % 8 == 0 for o in (m.q_off, m.qr_off, m.c_off, m.r_off, p.rg_off))
+    freq, mult = R.rotary_frequencies(cfg.to_config()["layers"][0]["mixer"]["rot"])
+    assert (m.freq.double().sum(0) - freq).abs().max() < 1e-14 and m.rot_mult == mult
+    assert m.absorb.w.n == 5 * 128 and (m.absorb.w.codes.float().view(5, 128, -1)[:, 72:] == 0).all()
+    assert torch.equal(p.norm, w["l0.norm1"].float().expand(W)) and torch.equal(p.rg[1], w["l0.rg2.b"].float()) and p.limit == 1.2
+    # a width of 80 features takes two tiles of the activation, the gate follows
+    assert p.ff_rows == 256 and p.gate_up.n == 256 + W and p.gate_up.act_interleaved
+    both = torch.zeros(256, W)
+    both[:80], both[128:208] = w["l0.mlp.gate"].float(), w["l0.mlp.up"].float()
+    codes = p.gate_up.codes.float()[:, :W]
+    assert torch.equal(codes[:256], both[wq_pack.swiglu_row_order(128)]) and torch.equal(codes[256:], w["l0.rg2"].float())
+    g = L.pack_layer(cfg, 1, w.__getitem__)
+    rows = g.proj.codes.float()[:, :W]
+    for t, off in zip("zxg", (g.mixer.z_off, g.mixer.x_off, g.mixer.g_off)):
+        assert torch.equal(rows[off:off + 72], w[f"l1.mix.{t}"].float())
+    assert torch.equal(g.mixer.bias, torch.stack([w["l1.mix.z.b"], w["l1.mix.x.b"]]).float())
+    d = L.pack_layer(cfg, 2, w.__getitem__)
+    rows = d.proj.codes.float()[:, :W]
+    for t, off in zip("qkv", d.mixer.spec.offsets):
+        t = w[f"l2.mix.{t}"].float()
+        assert torch.equal(rows[d.mixer.q_off + off:d.mixer.q_off + off + t.shape[0]], t)
+    assert torch.equal(rows[d.mixer.g_off:d.mixer.g_off + 240], w["l2.mix.g"].float())
+    dots = [float((w[f"l2.mix.lq{i}"].double() * w[f"l2.mix.lk{i}"].double()).sum()) for i in (1, 2)]
+    assert abs(d.mixer.less - (np.exp(dots[0]) - np.exp(dots[1]) + 0.4)) < 1e-12
+    last = L.pack_layer(cfg, 3, w.__getitem__)
+    assert last.gate_up is None and len(last.rg) == 1 and L.pack_weights(cfg, w.__getitem__).loop_in is None
+
+
 @pytest.mark.parametrize("rows, most", [(2, 2), (2, 50), (3, 9), (8, 30), (9, 128), (11, 70), (16, 120), (16, 128), (32, 512), (33, 100)])
 def test_distance_buckets(rows, most):
     """The product's table and the oracle's buckets: the formula wherever floating point decides it, every row up to the last."""
@@ -321,6 +431,98 @@ def test_distance_buckets(rows, most):
 
 
 # ------------------------------------------------------------------ the oracle's mechanisms, against element-wise loops
+def test_oracle_chunks():
+    for size in (1, 3, 4, None):
+        seen = R.same_chunk(6, 5, 11, size)
+        for i in range(5):
+            for j in range(11):
+                assert bool(seen[i, j]) == (j <= 6 + i and (size is None or j // size == (6 + i) // size))
+
+
+def test_oracle_differential_attention():
+    """Both maps, the factor, the norm without a weight and the gate, score by score."""
+    raw = gated(30, 24, [differential(4, 2, 6, 5, 0.7, 4, 20.0, 0.3, 4, None)])
+    w = {n: t.double() for n, t in tensors(raw, 1).items()}
+    m, h, eps = raw["layers"][0]["mixer"], torch.randn(9, 24, dtype=torch.float64), 1e-3
+    got = R.differential_attention(w, "l0.mix", m, h, {}, eps)
+    q, k = ((h @ w[f"l0.mix.{t}"].T).view(9, -1, 2, 6) for t in "qk")
+    q, k = (torch.stack([R.rotate_halves(R.rms(t[i:i + 1, :, j], eps) * w[f"l0.mix.{n}.norm"], i, 4, 20.0)[0] for i in range(9) for j in range(2)])
+            .view(9, 2, -1, 6) for t, n in ((q, "q"), (k, "k")))
+    v = (h @ w["l0.mix.v"].T).view(9, 2, 5)
+    less = float(torch.exp(w["l0.mix.lq1"] @ w["l0.mix.lk1"]) - torch.exp(w["l0.mix.lq2"] @ w["l0.mix.lk2"]) + 0.3)
+    out = torch.empty(9, 4, 5, dtype=torch.float64)
+    for i in range(9):
+        for n in range(4):
+            maps = []
+            for j in range(2):
+                keys = range(i // 4 * 4, i + 1)
+                e = np.exp([0.7 * float(q[i, j, n] @ k[t, j, n // 2]) for t in keys])
+                maps.append(sum(a * v[t, n // 2] for a, t in zip(e / e.sum(), keys)))
+            o = maps[0] - less * maps[1]
+            out[i, n] = o / torch.sqrt((o * o).mean() + eps) * 0.7
+    want = (out.view(9, 20) / (1 + torch.exp(-(h @ w["l0.mix.g"].T)))) @ w["l0.mix.o"].T
+    assert torch.allclose(got, want, atol=1e-9)
+
+
+def test_oracle_rotated_latent_attention():
+    raw = gated(30, 24, [rotated(3, 6, 4, 5, 7, 0.6, 20.0, (2.0, 30, 4.0, 1.0), None)])
+    w = {n: t.double() for n, t in tensors(raw, 2).items()}
+    m, h, eps = raw["layers"][0]["mixer"], torch.randn(8, 24, dtype=torch.float64), 1e-3
+    got = R.rotated_latent_attention(w, "l0.mix", m, h, {}, eps)
+    freq, mult = R.rotary_frequencies(m["rot"])
+    q, down = (h @ w["l0.mix.q"].T).view(8, 3, 10), h @ w["l0.mix.dkv"].T
+
+    def turn(x, i):
+        return R.rotate_pairs(x.view(1, 1, 4), i, freq, mult).view(4)
+
+    c = [down[t, :7] / torch.sqrt((down[t, :7] ** 2).mean() + eps) * w["l0.mix.dkv.norm"] for t in range(8)]
+    out = torch.empty(8, 3, 5, dtype=torch.float64)
+    for i in range(8):
+        for n in range(3):
+            uk, uv = w["l0.mix.uk"].view(3, 6, 7)[n], w["l0.mix.uv"].view(3, 5, 7)[n]
+            e = np.exp([0.6 * float(q[i, n, :6] @ (uk @ c[t]) + turn(q[i, n, 6:], i) @ turn(down[t, 7:], t)) for t in range(i + 1)])
+            out[i, n] = sum(a * (uv @ c[t]) for t, a in enumerate(e / e.sum()))
+    assert torch.allclose(got, out.view(8, 15) @ w["l0.mix.o"].T, atol=1e-9)
+
+
+def test_oracle_elementwise_recurrence_and_clamped_feed_forward():
+    raw = gated(30, 12, [mingru(5, clamped(6, 0.8))])
+    w = {n: t.double() for n, t in tensors(raw, 3).items()}
+    h = torch.randn(7, 12, dtype=torch.float64)
+    st, S, sig = {}, np.zeros(5), lambda v: 1 / (1 + np.exp(-v))                        # noqa: E731
+    got = torch.cat([R.mingru_mixer(w, "l0.mix", raw["layers"][0]["mixer"], part, st, 0.0) for part in h.split([2, 1, 4])])
+    for t in range(7):
+        z, x, g = ((w[f"l0.mix.{n}"] @ h[t]).numpy() for n in "zxg")
+        z, x = z + w["l0.mix.z.b"].numpy(), x + w["l0.mix.x.b"].numpy()
+        for c in range(5):
+            S[c] = (1 - sig(z[c])) * S[c] + sig(z[c]) * (x[c] + 0.5 if x[c] >= 0 else sig(x[c]))
+        assert torch.allclose(got[t], w["l0.mix.o"] @ torch.from_numpy(S * g * sig(g)), atol=1e-9)
+    y = R.clamped_feed_forward(w, "l0.mlp", 3 * h, 0.8)
+    for t in range(7):
+        act = [min(a, 0.8) * sig(1.702 * min(a, 0.8)) * (max(-0.8, min(b, 0.8)) + 1)
+               for a, b in zip((w["l0.mlp.gate"] @ (3 * h[t])).tolist(), (w["l0.mlp.up"] @ (3 * h[t])).tolist())]
+        assert torch.allclose(y[t], w["l0.mlp.down"] @ torch.tensor(act, dtype=torch.float64), atol=1e-9)
+
+
+def test_oracle_gated_residuals_and_the_loop():
+    """A model of one looped recurrence, layer by layer: gates that read the normed input, the embedding added between passes."""
+    raw = gated(30, 12, [mingru(5, clamped(6, 0.8))], (0, 1, 3), 0.4)
+    w = tensors(raw, 4)
+    got, _ = R.Oracle(raw, w, torch.float64).forward([3, 7, 7, 1])
+    f = {n: t.double() for n, t in w.items()}
+    m, eps = raw["layers"][0]["mixer"], 1e-5
+    x0 = 0.4 * f["embed"][[3, 7, 7, 1]]
+    x = x0
+    for turn in range(3):
+        if turn:
+            x = x + x0
+        for q, sub in ((1, lambda h: R.mingru_mixer(f, "l0.mix", m, h, {}, eps)), (2, lambda h: R.clamped_feed_forward(f, "l0.mlp", h, 0.8))):
+            h = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * float(f[f"l0.norm{q}"])
+            x = x + sub(h) / (1 + torch.exp(-(h @ f[f"l0.rg{q}"].T + f[f"l0.rg{q}.b"])))
+    want = (x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * float(f["final.norm"])) @ f["head"].T
+    assert torch.allclose(got, want, atol=1e-9)
+
+
 def test_oracle_rotation_of_halves_and_kept_window():
     x = torch.randn(4, 2, 7, dtype=torch.float64)
     y = R.rotate_halves(x, 5, 6, 50.0)
@@ -669,7 +871,9 @@ def backend_of(args, tp=1):
     config(300, 64, [delta(2, 1, 16, 16, 3, 64), latent(2, 16, 16, 24, 32, 20, 0.25, 0), channel(2, 2, 16, 16, 2, 48)], (0, 2, 2)),
     sequential(300, 64, [mamba2(2, 16, 8, 1, 3, 2, 48), parallel((4, 2, 16, 20, 0.3, 8, 90.0, (2.0, 50, 4.0, 1.0)), (2, 12, 16, 8.0), (0.9, 0.8), 64)], 8),
     streams(300, 64, [near(4, 2, 16, 24, 3, 0.5, 8, 90.0, 20, 3, routed(4, 2, 32, 1, 24)), far(2, 1, 16, 16, 0.3, 20, (0.4, 8), 48)], 2, 3.0),
-], ids=["Bumodra", "Loduzen", "Vimelorn"])
+    gated(300, 64, [rotated(2, 16, 8, 16, 32, 0.3, 90.0, (2.0, 50, 4.0, 1.0), clamped(64)), mingru(48, None),
+                    differential(4, 2, 16, 24, 0.3, 8, 90.0, 0.4, 20, clamped(48))], (1, 3, 2), 0.5),
+], ids=["Bumodra", "Loduzen", "Vimelorn", "Fovunex"])
 def test_eager_mode_generates_like_the_oracle(tmp_path, raw):
     from cubic_serve_b200.runtime.scheduler import SamplingParams
     w = tensors(raw, 5)
