@@ -258,10 +258,10 @@ __device__ __forceinline__ void store_pair(bf16* row, int c, int d, float x, flo
 __device__ __forceinline__ void store_gated_pair(bf16* row, const bf16* gate, int c, int e, float x, float y) {
   if (c + 1 < e && (e & 1) == 0) {
     const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + c));
-    *reinterpret_cast<uint32_t*>(row + c) = pack_bf16x2(x * sigmoid_of(z.x), y * sigmoid_of(z.y));
+    *reinterpret_cast<uint32_t*>(row + c) = pack_bf16x2(__fdividef(x, 1.f + __expf(-z.x)), __fdividef(y, 1.f + __expf(-z.y)));
   } else {
-    if (c < e) row[c] = __float2bfloat16(x * sigmoid_of(to_f(gate[c])));
-    if (c + 1 < e) row[c + 1] = __float2bfloat16(y * sigmoid_of(to_f(gate[c + 1])));
+    if (c < e) row[c] = __float2bfloat16(__fdividef(x, 1.f + __expf(-to_f(gate[c]))));
+    if (c + 1 < e) row[c + 1] = __float2bfloat16(__fdividef(y, 1.f + __expf(-to_f(gate[c + 1]))));
   }
 }
 

@@ -442,6 +442,12 @@ wq_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
           const float4 f0 = *reinterpret_cast<const float4*>(stg + mm * kTileN + (idx & 15) * 8);
           const float4 f1 = *reinterpret_cast<const float4*>(stg + mm * kTileN + (idx & 15) * 8 + 4);
           float v[8] = {f0.x, f0.y, f0.z, f0.w, f1.x, f1.y, f1.z, f1.w};
+          if (FMT == kFmtBf16 && p.wide && wide_joins(p, n0 + 4)) {
+            const WideIn a = wide_load(p, m, n0), b = wide_load(p, m, n0 + 4);
+            wide_join(p, m, n0, f0, a, wide_bias(p, n0));
+            wide_join(p, m, n0 + 4, f1, b, wide_bias(p, n0 + 4));
+            continue;
+          }
           if (FMT == kFmtBf16 && p.wide) {
             float lo[4] = {v[0], v[1], v[2], v[3]}, hi[4] = {v[4], v[5], v[6], v[7]};
             store_wide4(p, m, n0, lo);

@@ -206,29 +206,51 @@ __device__ __forceinline__ void store_act4(const WqGemmParams& p, int m, int n_t
 __device__ __forceinline__ bool glu_tile(const WqGemmParams& p, int n_tile) {
   return p.swiglu && !(p.y2 && n_tile * kTileN >= p.n_split);
 }
+// What four features of row m are added to and multiplied by on their way into an fp32 residual.  A caller that stores several groups
+// loads all of them first, so that one group's store does not hold up the next one's loads.
+struct WideIn {
+  float4 r;
+  uint2 g;
+};
+// Whether the features n0 .. n0 + 3 join a residual four at a time
+__device__ __forceinline__ bool wide_joins(const WqGemmParams& p, int n0) { return p.residual32 && !p.y2 && n0 + 3 < p.N && (p.ldy & 3) == 0; }
+__device__ __forceinline__ WideIn wide_load(const WqGemmParams& p, int m, int n0) {
+  WideIn in;
+  in.r = *reinterpret_cast<const float4*>(p.residual32 + static_cast<size_t>(m) * p.ldy + n0);
+  in.g = p.rgate ? *reinterpret_cast<const uint2*>(p.rgate + static_cast<size_t>(m) * p.ldrg + n0) : make_uint2(0u, 0u);
+  return in;
+}
+// `b`: bias of the gate at n0
+__device__ __forceinline__ void wide_join(const WqGemmParams& p, int m, int n0, float4 v, const WideIn& in, float4 b) {
+  if (p.rgate) {
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&in.g.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&in.g.y));
+    v.x = __fdividef(v.x, 1.f + __expf(-(lo.x + b.x)));
+    v.y = __fdividef(v.y, 1.f + __expf(-(lo.y + b.y)));
+    v.z = __fdividef(v.z, 1.f + __expf(-(hi.x + b.z)));
+    v.w = __fdividef(v.w, 1.f + __expf(-(hi.y + b.w)));
+  }
+  *reinterpret_cast<float4*>(p.y32 + static_cast<size_t>(m) * p.ldy + n0) = make_float4(v.x + in.r.x, v.y + in.r.y, v.z + in.r.z, v.w + in.r.w);
+}
+__device__ __forceinline__ float4 wide_bias(const WqGemmParams& p, int n0) {
+  return p.rgate ? *reinterpret_cast<const float4*>(p.rgate_b + n0) : make_float4(0.f, 0.f, 0.f, 0.f);
+}
 // Four consecutive output features n0..n0+3 (n0 % 4 == 0) of row m, already scaled, through the wide epilogue.
 __device__ __forceinline__ void store_wide4(const WqGemmParams& p, int m, int n0, float (&v)[4]) {
   if (n0 >= p.N) return;
   const bool whole = n0 + 3 < p.N;
   const bool second = p.y2 && n0 >= p.n_split;
   if (p.y32 && !second) {
+    if (wide_joins(p, n0)) {
+      wide_join(p, m, n0, make_float4(v[0], v[1], v[2], v[3]), wide_load(p, m, n0), wide_bias(p, n0));
+      return;
+    }
     const size_t off = static_cast<size_t>(m) * p.ldy + n0;
     if (p.rgate) {
       const __nv_bfloat16* gr = p.rgate + static_cast<size_t>(m) * p.ldrg + n0;
-      if (whole) {
-        const uint2 u = *reinterpret_cast<const uint2*>(gr);
-        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
-        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-        const float4 c = *reinterpret_cast<const float4*>(p.rgate_b + n0);
-        v[0] = __fdividef(v[0], 1.f + __expf(-(a.x + c.x)));
-        v[1] = __fdividef(v[1], 1.f + __expf(-(a.y + c.y)));
-        v[2] = __fdividef(v[2], 1.f + __expf(-(b.x + c.z)));
-        v[3] = __fdividef(v[3], 1.f + __expf(-(b.y + c.w)));
-      } else {
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (n0 + j < p.N) v[j] = __fdividef(v[j], 1.f + __expf(-(__bfloat162float(gr[j]) + p.rgate_b[n0 + j])));
-      }
+      for (int j = 0; j < 4; ++j)
+        if (n0 + j < p.N) v[j] = __fdividef(v[j], 1.f + __expf(-(__bfloat162float(gr[j]) + p.rgate_b[n0 + j])));
     }
     if (whole && (p.ldy & 3) == 0) {
       float4 o = make_float4(v[0], v[1], v[2], v[3]);

@@ -627,6 +627,24 @@ wq_gemm_sk_kernel(const __grid_constant__ CUtensorMap tmap_x,
             u.x *= p.alpha; u.y *= p.alpha; u.z *= p.alpha; u.w *= p.alpha;
             store_act4(p, m0 + mm, n_base / kTileN, j0, g, u);
           }
+        } else if (FMT == kFmtBf16 && ok && p.wide && wide_joins(p, n_base + kTileN - 4)) {
+          constexpr int kB = 4;                                 // items whose loads are in flight
+          const int items = rows_here * (kTileN / 4);
+          for (int base = tt; base < items; base += kB * nthr) {
+            WideIn in[kB];
+#pragma unroll
+            for (int b = 0; b < kB; ++b) {
+              const int idx = min(base + b * nthr, items - 1);
+              in[b] = wide_load(p, m0 + (idx >> 5), n_base + (idx & 31) * 4);
+            }
+#pragma unroll
+            for (int b = 0; b < kB; ++b) {
+              const int idx = base + b * nthr, n0 = n_base + (idx & 31) * 4;
+              if (idx >= items) continue;
+              const float4 v = *reinterpret_cast<const float4*>(stg + static_cast<size_t>(idx) * 4);
+              wide_join(p, m0 + (idx >> 5), n0, make_float4(v.x * p.alpha, v.y * p.alpha, v.z * p.alpha, v.w * p.alpha), in[b], wide_bias(p, n0));
+            }
+          }
         } else if (ok)
           for (int idx = tt; idx < rows_here * (kTileN / 4); idx += nthr)
             sk_store4<FMT>(p, m0 + (idx >> 5), n_base + (idx & 31) * 4, *reinterpret_cast<const float4*>(stg + static_cast<size_t>(idx) * 4));
@@ -842,7 +860,24 @@ wq_gemm_sk_kernel(const __grid_constant__ CUtensorMap tmap_x,
           const int f4 = (lane & 7) * 4;
           float* slot = whole ? nullptr : sk_slot(p, unit, seg.part) + quad * 32 + f4;
           const uint32_t taddr = tmem_base + static_cast<uint32_t>(buf) * p.acc_cols + (static_cast<uint32_t>(quad * 32) << 16);
+          // rows that join an fp32 residual: what they join is on its way while the accumulators are read
+          bool joins = false;
+          float4 bias = make_float4(0.f, 0.f, 0.f, 0.f);
+          if constexpr (FMT == kFmtBf16) {
+            joins = whole && p.wide && wide_joins(p, n_base + quad * 32 + f4);
+            if (joins) bias = wide_bias(p, n_base + quad * 32 + f4);
+          }
           for (int c0 = 0; c0 < p.mb; c0 += 16) {
+            WideIn in[4];
+            if constexpr (FMT == kFmtBf16) {
+              if (joins) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                  const int row = c0 + (lane >> 3) + 4 * i;
+                  if (row < rows_here) in[i] = wide_load(p, m0 + row, n_base + quad * 32 + f4);
+                }
+              }
+            }
             uint32_t acc[16];
             tmem_ld_32x16(taddr + c0, acc);
             tmem_ld_wait();
@@ -870,7 +905,11 @@ wq_gemm_sk_kernel(const __grid_constant__ CUtensorMap tmap_x,
               for (int i = 0; i < 4; ++i) {
                 const int row = (lane >> 3) + 4 * i;
                 const float4 v = *reinterpret_cast<const float4*>(scr + row * 32 + f4);
-                if (!whole) {
+                if (FMT == kFmtBf16 && joins) {
+                  if (c0 + row < rows_here)
+                    wide_join(p, m0 + c0 + row, n_base + quad * 32 + f4, make_float4(v.x * p.alpha, v.y * p.alpha, v.z * p.alpha, v.w * p.alpha), in[i],
+                              bias);
+                } else if (!whole) {
                   *reinterpret_cast<float4*>(slot + static_cast<size_t>(c0 + row) * kTileN) = v;
                 } else if (c0 + row < rows_here) {
                   sk_store4<FMT>(p, m0 + c0 + row, n_base + quad * 32 + f4, v);

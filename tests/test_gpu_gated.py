@@ -488,6 +488,30 @@ def test_recurrence_in_portions(dtype, width, cuts):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("width", [31, 64, 200])
+def test_long_prompts_share_a_segment_among_blocks(dtype, width):
+    """Prompts long enough for clusters of 2, 4 and 8 blocks, alone, behind earlier tokens and beside shorter ones."""
+    c = Gru(width, dtype)
+    for cuts in ((256, 3), (700, 513), (2100,), (1, 1025)):
+        zxg = c.rows(sum(cuts))
+        want, S = gru_oracle(*zxg, c.bias, None)
+        got, i = [], 0
+        for n in cuts:
+            got.append(c.run([t[i:i + n] for t in zxg], [(n, 3, i)]))
+            i += n
+        close(torch.cat(got), want, dtype, exact=1e-5, rough=8e-3)
+        close(c.state[3, :width], S, torch.float32, exact=1e-5)
+    lens = (5, 900, 0, 130)
+    rows = [c.rows(n) for n in lens]
+    out = c.run([torch.cat([r[i] for r in rows]) for i in range(3)], [(n, s, 0) for s, n in enumerate(lens)])
+    for s, (r, o) in enumerate(zip(rows, out.split(lens))):
+        if lens[s]:
+            want, S = gru_oracle(*r, c.bias, None)
+            close(o, want, dtype, exact=1e-5, rough=8e-3)
+            close(c.state[s, :width], S, torch.float32, exact=1e-5)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("width", [40, 37, 260])
 def test_recurrence_batches(dtype, width):
     """Unequal requests in one step equal each alone; decode steps with a padding segment; a slot that is used again."""
