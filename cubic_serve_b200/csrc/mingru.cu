@@ -27,14 +27,32 @@ struct MinGru {
   Segments sg;
 };
 
-// Sigmoids: as exact as fp32 goes for fp32 models, the device's fast exponential and quotient for bf16 models
-template <typename T>
-__device__ __forceinline__ float gru_sigmoid(float v) {
-  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-v));
-  else return 1.f / (1.f + expf(-v));
+// 1 / (1 + e^-(v + bias)): as exact as fp32 goes for fp32 models; for bf16 models the device's approximate exponential and reciprocal
+// without their handling of ranges that cannot occur (a power that is too large makes the sigmoid zero).  `scaled` is the bias as
+// gru_bias makes it.
+__device__ __forceinline__ float gru_exp2(float x) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
 }
-template <typename T> __device__ __forceinline__ float gru_candidate(float u) { return u >= 0.f ? u + 0.5f : gru_sigmoid<T>(u); }
-template <typename T> __device__ __forceinline__ float gru_silu(float v) { return v * gru_sigmoid<T>(v); }
+__device__ __forceinline__ float gru_reciprocal(float x) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+static constexpr float kGruLog2e = 1.4426950408889634f;
+template <typename T> __device__ __forceinline__ float gru_bias(float bias) { return sizeof(T) == 2 ? -kGruLog2e * bias : bias; }
+template <typename T>
+__device__ __forceinline__ float gru_sigmoid(float v, float scaled) {
+  if constexpr (sizeof(T) == 2) return gru_reciprocal(1.f + gru_exp2(fmaf(v, -kGruLog2e, scaled)));
+  else return 1.f / (1.f + expf(-(v + scaled)));
+}
+template <typename T>
+__device__ __forceinline__ float gru_candidate(float u, float bias, float scaled) {
+  const float v = u + bias;
+  return v >= 0.f ? v + 0.5f : gru_sigmoid<T>(u, scaled);
+}
+template <typename T> __device__ __forceinline__ float gru_silu(float v) { return v * gru_sigmoid<T>(v, 0.f); }
 
 // N neighbouring channels as they are stored, and as numbers
 template <typename T, int N> struct GruRaw { using type = T; };
@@ -69,7 +87,7 @@ template <typename T, int N, bool CLUSTER>
 __global__ void __launch_bounds__(32 * kGruWarps)
 mingru_walk_kernel(const MinGru<T> p) {
   using Raw = typename GruRaw<T, N>::type;
-  __shared__ float2 maps[2][kGruWarps][N][32];
+  __shared__ __align__(16) float2 maps[2][kGruWarps][32][N];
   __shared__ float2 whole[2][N][32];        // map of this block's tokens of a turn, read by the other blocks of its cluster
   pdl_wait();
   pdl_launch_dependents();
@@ -82,24 +100,32 @@ mingru_walk_kernel(const MinGru<T> p) {
   const int c = live ? ch : 0;
   const size_t row0 = p.sg.row0[s];
   float* st = p.state + static_cast<size_t>(p.sg.slot[s]) * p.lds + c;
-  float bz[N], bx[N], S[N];
+  float bz[N], bx[N], sx[N], S[N];
 #pragma unroll
   for (int k = 0; k < N; ++k) {
-    bz[k] = p.bias[c + k];
+    bz[k] = gru_bias<T>(p.bias[c + k]);
     bx[k] = p.bias[p.width + c + k];
+    sx[k] = gru_bias<T>(bx[k]);
     S[k] = p.sg.pos0[s] > 0 ? st[k] : 0.f;  // the same in every warp
   }
   if constexpr (CLUSTER) cluster_sync_all();        // every block has read the old state
   Raw zr[kGruRun] = {}, xr[kGruRun] = {}, gr[kGruRun] = {};
   auto load = [&](int t0) {
     const T* row = p.x + (row0 + t0) * p.ldx + c;
+    const T* z = row + p.z_off;
+    const T* x = row + p.x_off;
+    const T* g = row + p.g_off;
+    auto all = [&](auto full) {
 #pragma unroll
-    for (int i = 0; i < kGruRun; ++i)
-      if (t0 + i < count) {
-        zr[i] = *reinterpret_cast<const Raw*>(row + static_cast<size_t>(i) * p.ldx + p.z_off);
-        xr[i] = *reinterpret_cast<const Raw*>(row + static_cast<size_t>(i) * p.ldx + p.x_off);
-        gr[i] = *reinterpret_cast<const Raw*>(row + static_cast<size_t>(i) * p.ldx + p.g_off);
-      }
+      for (int i = 0; i < kGruRun; ++i)
+        if (decltype(full)::value || t0 + i < count) {
+          zr[i] = *reinterpret_cast<const Raw*>(z + i * p.ldx);
+          xr[i] = *reinterpret_cast<const Raw*>(x + i * p.ldx);
+          gr[i] = *reinterpret_cast<const Raw*>(g + i * p.ldx);
+        }
+    };
+    if (t0 + kGruRun <= count) all(std::true_type{});
+    else all(std::false_type{});
   };
   const int turn = kGruWarps * kGruRun;     // tokens of a block's turn
   load(rank * turn + warp * kGruRun);
@@ -107,27 +133,31 @@ mingru_walk_kernel(const MinGru<T> p) {
   for (int base = 0; base < count; base += blocks * turn, b ^= 1) {
     const int t0 = base + rank * turn + warp * kGruRun;
     float keep[kGruRun][N], in[kGruRun][N], gate[kGruRun][N], A[N], B[N];
+    auto make = [&](auto full) {
 #pragma unroll
-    for (int k = 0; k < N; ++k) { A[k] = 1.f; B[k] = 0.f; }
+      for (int k = 0; k < N; ++k) { A[k] = 1.f; B[k] = 0.f; }
 #pragma unroll
-    for (int i = 0; i < kGruRun; ++i) {
-      float z[N], u[N], g[N];
-      gru_unpack(zr[i], z);
-      gru_unpack(xr[i], u);
-      gru_unpack(gr[i], g);
-      const bool ok = t0 + i < count;
+      for (int i = 0; i < kGruRun; ++i) {
+        float z[N], u[N], g[N];
+        gru_unpack(zr[i], z);
+        gru_unpack(xr[i], u);
+        gru_unpack(gr[i], g);
+        const bool ok = decltype(full)::value || t0 + i < count;      // a token behind the segment changes nothing
 #pragma unroll
-      for (int k = 0; k < N; ++k) {
-        const float zk = gru_sigmoid<T>(z[k] + bz[k]);
-        keep[i][k] = ok ? 1.f - zk : 1.f;
-        in[i][k] = ok ? zk * gru_candidate<T>(u[k] + bx[k]) : 0.f;
-        gate[i][k] = gru_silu<T>(g[k]);
-        A[k] *= keep[i][k];
-        B[k] = fmaf(keep[i][k], B[k], in[i][k]);
+        for (int k = 0; k < N; ++k) {
+          const float zk = gru_sigmoid<T>(z[k], bz[k]);
+          keep[i][k] = ok ? 1.f - zk : 1.f;
+          in[i][k] = ok ? zk * gru_candidate<T>(u[k], bx[k], sx[k]) : 0.f;
+          gate[i][k] = gru_silu<T>(g[k]);
+          A[k] *= keep[i][k];
+          B[k] = fmaf(keep[i][k], B[k], in[i][k]);
+        }
       }
-    }
+    };
+    if (t0 + kGruRun <= count) make(std::true_type{});
+    else make(std::false_type{});
 #pragma unroll
-    for (int k = 0; k < N; ++k) maps[b][warp][k][lane] = make_float2(A[k], B[k]);
+    for (int k = 0; k < N; ++k) maps[b][warp][lane][k] = make_float2(A[k], B[k]);
     load(t0 + blocks * turn);               // the next run's projections are on their way (nothing behind the segment)
     __syncthreads();                        // two buffers: the next turn's maps are written behind this turn's barrier only
     float first[N];                         // state before the block's tokens
@@ -138,7 +168,7 @@ mingru_walk_kernel(const MinGru<T> p) {
         float2 m = make_float2(1.f, 0.f);
 #pragma unroll
         for (int w = 0; w < kGruWarps; ++w) {
-          const float2 o = maps[b][w][warp][lane];
+          const float2 o = maps[b][w][lane][warp];
           m = make_float2(o.x * m.x, fmaf(o.x, m.y, o.y));
         }
         whole[b][warp][lane] = m;
@@ -154,20 +184,26 @@ mingru_walk_kernel(const MinGru<T> p) {
         }
       }
     }
-    float mine[N];
+    float mine[N], at[N];
 #pragma unroll
-    for (int k = 0; k < N; ++k) {
-      float at = first[k];
-      mine[k] = at;
+    for (int k = 0; k < N; ++k) mine[k] = at[k] = first[k];
 #pragma unroll
-      for (int w = 0; w < kGruWarps; ++w) {
-        if (w == warp) mine[k] = at;
-        const float2 m = maps[b][w][k][lane];
-        at = fmaf(m.x, at, m.y);
+    for (int w = 0; w < kGruWarps; ++w) {
+      float2 m[N];
+      if constexpr (N == 2) *reinterpret_cast<float4*>(m) = *reinterpret_cast<const float4*>(maps[b][w][lane]);
+      else m[0] = maps[b][w][lane][0];
+#pragma unroll
+      for (int k = 0; k < N; ++k) {
+        if (w == warp) mine[k] = at[k];
+        at[k] = fmaf(m[k].x, at[k], m[k].y);
       }
-      if constexpr (!CLUSTER) S[k] = at;
+    }
+    if constexpr (!CLUSTER) {
+#pragma unroll
+      for (int k = 0; k < N; ++k) S[k] = at[k];
     }
     T* orow = p.out + (row0 + t0) * p.ldo + c;
+    const int most = live ? count - t0 : 0;
 #pragma unroll
     for (int i = 0; i < kGruRun; ++i) {
       float v[N];
@@ -176,7 +212,7 @@ mingru_walk_kernel(const MinGru<T> p) {
         mine[k] = fmaf(keep[i][k], mine[k], in[i][k]);
         v[k] = mine[k] * gate[i][k];
       }
-      if (live && t0 + i < count) gru_store<N>(orow + static_cast<size_t>(i) * p.ldo, v);
+      if (i < most) gru_store<N>(orow + i * p.ldo, v);
     }
   }
   // every warp has read the old state before the first barrier
@@ -210,8 +246,8 @@ mingru_step_kernel(const MinGru<T> p) {
   for (int i = 0; i < N; ++i) S[i] = fresh ? 0.f : st[i];
 #pragma unroll
   for (int i = 0; i < N; ++i) {
-    const float zi = gru_sigmoid<T>(z[i] + p.bias[c + i]);
-    S[i] = fmaf(1.f - zi, S[i], zi * gru_candidate<T>(u[i] + p.bias[p.width + c + i]));
+    const float bx = p.bias[p.width + c + i], zi = gru_sigmoid<T>(z[i], gru_bias<T>(p.bias[c + i]));
+    S[i] = fmaf(1.f - zi, S[i], zi * gru_candidate<T>(u[i], bx, gru_bias<T>(bx)));
     st[i] = S[i];
     S[i] *= gru_silu<T>(g[i]);
   }
@@ -247,11 +283,17 @@ int cb_mingru(const CbMinGru* a, const CbSegments* seg, void* stream) {
     p.sg = make_segments(seg, a->tokens);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (!step) {
-      // few blocks: clusters share the segments, as long as the longest has a turn for every block
+      // clusters share the segments where that shortens the run of waves (a block per SM) and of turns a block makes; a block's start
+      // costs about a turn, meeting in a cluster a third of one
       const int n = pair ? 2 : 1, tiles = (a->width + 32 * n - 1) / (32 * n);
       const int longest = a->tokens - (seg->num - 1), turns = (longest + kGruWarps * kGruRun - 1) / (kGruWarps * kGruRun);
+      auto cost = [&](int c) {
+        const long long waves = (static_cast<long long>(tiles) * seg->num * c + 147) / 148, each = (turns + c - 1) / c;
+        return waves * (3 * each + 3 + (c > 1 ? each : 0));
+      };
       int cluster = 1;
-      while (cluster < kGruCluster && 2 * cluster <= turns && tiles * seg->num * cluster < 148) cluster *= 2;
+      for (int c = 2; c <= kGruCluster && c <= turns; c *= 2)
+        if (cost(c) < cost(cluster)) cluster = c;
       const dim3 grid(tiles * cluster, seg->num), block(32 * kGruWarps), shape(cluster, 1, 1);
       if (cluster > 1)
         return static_cast<int>(pair ? launch(mingru_walk_kernel<T, 2, true>, grid, block, 0, st, shape, p)
