@@ -1587,5 +1587,24 @@ NAMED = {"layered-tiny": tiny_layered_config, "layered-8b": layered_8b_config, "
          "layered-gated-tiny": tiny_gated_config, "layered-gated-8b": gated_8b_config}
 
 
+_MIXER_SOURCES = {DeltaSpec: ("delta_rule.cu",), LatentSpec: ("latent_attn.cu",), AttentionSpec: ("gqa_attn.cu",),
+                  GatedLinearSpec: ("linear_recurrence.cu",), SsdSpec: ("linear_recurrence.cu",),
+                  ConvAttentionSpec: ("qkv_prepare.cu", "gqa_attn.cu"), BiasedAttentionSpec: ("qkv_prepare.cu", "gqa_attn.cu"),
+                  DifferentialSpec: ("qkv_prepare.cu", "gqa_attn.cu"), MinGruSpec: ("mingru.cu",)}
+
+
+def kernel_sources(cfg: LayeredConfig) -> set[str]:
+    """Sources of ``csrc`` whose kernels a model of this configuration launches: products, rows, pages, sampling, and its mixers'."""
+    out = {"wq_gemm.cu", "wq_gemm_sk.cu", "elementwise.cu", "kv_cache.cu", "sampling.cu", "guard.cu", "layered.cu"}
+    for l in cfg.layers:
+        for part in l.mixer.parts:
+            out.update(_MIXER_SOURCES[type(part)])
+        if l.routed is not None:
+            out.add("moe.cu")
+    if cfg.design.streams:
+        out.add("streams.cu")
+    return out
+
+
 def with_dtype(cfg: LayeredConfig, dtype: str) -> LayeredConfig:
     return replace(cfg, dtype=dtype)

@@ -4,7 +4,9 @@ The kernels are plain CUDA C++ with ``extern "C"`` launchers; Python reaches
 them through ``ctypes`` with raw device pointers and the current CUDA stream,
 the same split the reference uses (driver-API launches, no CPython extension:
 ``ops/cuda/native.py:101-255`` there).  The library is compiled ahead of time
-into the package directory so that it ships with a source snapshot.
+into the package directory so that it ships with a source snapshot.  A program
+that runs one model in a checkout without it may ``select`` the sources this
+model needs: only these are compiled then, into a library of their own.
 """
 from __future__ import annotations
 
@@ -26,7 +28,8 @@ NVCC_FLAGS = (
 )
 
 _lock = threading.Lock()
-_lib: ctypes.CDLL | None = None
+_lib: "ctypes.CDLL | _Part | None" = None
+_selected: tuple[str, ...] | None = None       # sources this process needs (None: all)
 
 
 class NativeLibraryError(RuntimeError):
@@ -116,11 +119,39 @@ def build(force: bool = False, verbose: bool = False) -> Path:
     """Compile every ``csrc/*.cu`` for sm_100a and link ``libcubic_b200.so``."""
     if not force and not needs_build():
         return LIB_PATH
-    objdir = CSRC / "build"
-    objdir.mkdir(exist_ok=True)
+    _compile(sources(), CSRC / "build", LIB_PATH, verbose)
+    manifest = {"library": LIB_PATH.name, "library_sha256": _sha(LIB_PATH), "arch": "sm_100a", "flags": list(NVCC_FLAGS),
+                "nvcc": _nvcc_version(), "sources": _source_digests()}
+    MANIFEST_PATH.write_text(json.dumps(manifest, indent=1, sort_keys=True) + "\n")
+    return LIB_PATH
+
+
+def select(names) -> None:
+    """This process needs these sources of ``csrc`` only: without a current complete library just they are compiled.  To be
+    called before the library is first used."""
+    global _selected
+    unknown = set(names) - {p.name for p in sources()}
+    if unknown:
+        raise NativeLibraryError(f"no such sources: {sorted(unknown)}")
+    _selected = tuple(sorted(names))
+
+
+def build_part(names) -> Path:
+    """Compile only these sources into a library whose name states its contents (sources, headers, flags): there or not."""
+    digests = _source_digests()
+    told = json.dumps([sorted(names), [digests[n] for n in sorted(digests) if not n.endswith(".cu") or n in names], list(NVCC_FLAGS)])
+    key = hashlib.sha256(told.encode()).hexdigest()[:12]
+    path = LIB_PATH.with_name(f"{LIB_PATH.stem}_{key}.so")
+    if not path.exists():
+        _compile([CSRC / n for n in sorted(names)], CSRC / "build" / key, path)
+    return path
+
+
+def _compile(srcs: list[Path], objdir: Path, library: Path, verbose: bool = False) -> None:
+    objdir.mkdir(parents=True, exist_ok=True)
     procs = []
     objs = []
-    for src in sources():
+    for src in srcs:
         obj = objdir / (src.stem + ".o")
         objs.append(str(obj))
         cmd = [_nvcc(), *NVCC_FLAGS, "-c", str(src), "-o", str(obj)]
@@ -133,23 +164,47 @@ def build(force: bool = False, verbose: bool = False) -> Path:
             raise NativeLibraryError(f"nvcc failed for {src.name}:\n{out}")
         if verbose and out:
             print(out)
-    tmp = LIB_PATH.with_suffix(".so.tmp")
+    tmp = library.with_suffix(f".so.tmp{os.getpid()}")
     link = [_nvcc(), "-shared", "-o", str(tmp), *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
     res = subprocess.run(link, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)
     if res.returncode != 0:
         raise NativeLibraryError(f"link failed:\n{res.stdout}")
-    os.replace(tmp, LIB_PATH)
-    manifest = {"library": LIB_PATH.name, "library_sha256": _sha(LIB_PATH), "arch": "sm_100a", "flags": list(NVCC_FLAGS),
-                "nvcc": _nvcc_version(), "sources": _source_digests()}
-    MANIFEST_PATH.write_text(json.dumps(manifest, indent=1, sort_keys=True) + "\n")
-    return LIB_PATH
+    os.replace(tmp, library)
 
 
-def lib() -> ctypes.CDLL:
-    """Return the loaded library; build it first if a compiler is available and it is stale."""
+class _Part:
+    """A library that holds some of the entry points; calling another one names it."""
+
+    def __init__(self, dll: ctypes.CDLL) -> None:
+        self._dll = dll
+
+    def __getattr__(self, name: str):
+        try:
+            return getattr(self._dll, name)
+        except AttributeError:
+            return _Absent(name)
+
+
+class _Absent:
+    def __init__(self, name: str) -> None:
+        self.name = name
+
+    def __call__(self, *_):
+        raise NativeLibraryError(f"{self.name} is not among the sources this process selected")
+
+
+def lib() -> "ctypes.CDLL | _Part":
+    """Return the loaded library; build it (or the selected part) first if a compiler is available and it is stale."""
     global _lib
     with _lock:
         if _lib is None:
+            if _selected is not None and needs_build():
+                part = _Part(ctypes.CDLL(str(build_part(_selected))))
+                _declare(part)
+                if os.environ.get("CUBIC_SERVE_PDL", "1") == "0":
+                    part.cb_set_pdl(0)
+                _lib = part
+                return _lib
             if needs_build():
                 try:
                     build()

@@ -8,7 +8,8 @@ places in the order of the entries, little-endian fp32 ``[wanted, vocab]``.  Aft
 Requests listed in ``end`` give back their pages and slot after the step.
 
 The engine is the serving one: checkpoint admission and model class by ``config.json``, scheduler, page pool for ``N`` tokens,
-four request slots, the native runner and its decode graphs.
+four request slots, the native runner and its decode graphs.  In a fresh checkout the first call compiles the kernels that the model
+needs.
 """
 from __future__ import annotations
 
@@ -69,7 +70,13 @@ def main(argv: list[str] | None = None) -> int:
     ap.add_argument("--max-tokens", type=int, required=True, help="tokens that live requests hold at most")
     ap.add_argument("--device", type=int, default=0)
     args = ap.parse_args(argv)
+    from ..models.checkpoint import layered_config_of
+    from ..models.layered import kernel_sources
+    from ..ops import native
     from ..runtime.imposed import ImposedSession
+    layered = layered_config_of(Path(args.model))
+    if layered is not None:
+        native.select(kernel_sources(layered))       # a checkout without the library compiles what this model needs
     engine = build_engine(args.model, args.dtype, args.max_tokens, args.device)
     out = Path(args.out)
     out.mkdir(parents=True, exist_ok=True)

@@ -8,6 +8,7 @@ import socket
 import pytest
 
 from cubic_serve_b200.contracts import implementation as impl
+from cubic_serve_b200.ops import native
 from cubic_serve_b200.runtime.preparation import (EvidenceKey, EvidenceStore, StartupDisagreement, StartupPreparation,
                                                   StartupQualification, consensus)
 
@@ -167,3 +168,43 @@ def test_qualify_with_receipt_runs_once(tmp_path):
     assert qualify_with_receipt(0, quick=True, evidence_dir=tmp_path, run=run)[1] is False
     assert qualify_with_receipt(0, quick=True, evidence_dir=tmp_path, run=run)[1] is True
     assert len(calls) == 1
+
+
+def test_part_of_the_library(tmp_path, monkeypatch):
+    """Selected sources become a library named after its contents; what it does not hold is named when it is called."""
+    monkeypatch.setattr(native, "LIB_PATH", tmp_path / "libcubic_b200.so")
+    monkeypatch.setattr(native, "MANIFEST_PATH", tmp_path / "libcubic_b200.manifest.json")
+    monkeypatch.setattr(native, "_lib", None)
+    monkeypatch.setattr(native, "_selected", None)
+    built = []
+
+    def compile_(srcs, objdir, library, verbose=False):
+        built.append(sorted(s.name for s in srcs))
+        library.write_bytes(b"")
+
+    monkeypatch.setattr(native, "_compile", compile_)
+    a = native.build_part(("mingru.cu", "layered.cu"))
+    assert native.build_part(["layered.cu", "mingru.cu"]) == a and built == [["layered.cu", "mingru.cu"]] and a.parent == tmp_path
+    assert native.build_part(("layered.cu",)) != a and len(built) == 2
+    digests = native._source_digests()
+    monkeypatch.setattr(native, "_source_digests", lambda: {**digests, "moe.cu": "0"})
+    assert native.build_part(("mingru.cu", "layered.cu")) == a                  # another source changed
+    monkeypatch.setattr(native, "_source_digests", lambda: {**digests, "ptx.cuh": "0"})
+    assert native.build_part(("mingru.cu", "layered.cu")) != a                  # a header changed
+    with pytest.raises(native.NativeLibraryError, match="no such sources"):
+        native.select(("nothing.cu",))
+    with pytest.raises(native.NativeLibraryError, match="cb_moe_route is not among"):
+        native._Part(object()).cb_moe_route(1, 2)
+
+
+@pytest.mark.parametrize("name", ["layered-tiny", "layered-seq-tiny", "layered-streams-tiny", "layered-gated-tiny"])
+def test_sources_of_a_layered_model_hold_the_kernels_of_its_mixers(name):
+    from cubic_serve_b200.models import layered as L
+    names = L.kernel_sources(L.NAMED[name]())
+    have = {p.name for p in native.sources()}
+    assert names < have and "paged_attn.cu" not in names
+    text = "".join((native.CSRC / n).read_text() for n in names)
+    wanted = {"layered-tiny": ("cb_delta_prepare", "cb_latent_attn"), "layered-seq-tiny": ("cb_gqa_prepare", "cb_linear_walk"),
+              "layered-streams-tiny": ("cb_conv_qkv", "cb_norm_qkv", "cb_gqa_attn", "cb_stream_step", "cb_scored_moe_route"),
+              "layered-gated-tiny": ("cb_latent_prepare", "cb_head_qkv", "cb_gqa_attn", "cb_mingru")}[name]
+    assert all(w in text for w in (*wanted, "cb_bf16_gemm_wide", "cb_f32_gemm", "cb_row_norm", "cb_sample", "cb_copy_pages"))
