@@ -733,6 +733,58 @@ def test_oracle_window_edges(window):
             assert [i for i in range(n) if moved[i]] == [i for i in seen if i >= first]
 
 
+def _swapped(name, change):
+    """A mistake planted in one of the oracle's functions."""
+    right = getattr(R, name)
+
+    def plant(monkeypatch):
+        wrong = lambda *a: change(right, *a)                                            # noqa: E731
+        monkeypatch.setattr(R, name, wrong)
+        for kind, fn in R.GATED_MIXERS.items():
+            if fn is right:
+                monkeypatch.setitem(R.GATED_MIXERS, kind, wrong)
+    return plant
+
+
+def _first_turned(x, first, freq, mult):
+    return x if x.shape[1] == 1 else RIGHT_ROTATE(x, first, freq, mult)
+
+
+RIGHT_ROTATE = R.rotate_pairs
+
+
+@pytest.mark.parametrize("mistake", [
+    _swapped("same_chunk", lambda f, a, n, m, size: f(a, n, m, size and size + 1)),
+    _swapped("same_chunk", lambda f, a, n, m, size: f(a, n, m, None)),
+    _swapped("same_chunk", lambda f, a, n, m, size: R.kept_window(a, n, m, size, 0)),
+    _swapped("rotary_frequencies", lambda f, rot: (f(rot)[0], 1.0)),
+    _swapped("rotary_frequencies", lambda f, rot: f({**rot, "scaling": None})),
+    _swapped("rotate_pairs", lambda f, x, a, fr, mult: _first_turned(x, a, fr, mult)),
+    _swapped("rotate_halves", lambda f, x, a, dims, base: f(x, a, dims, 1.02 * base)),
+    _swapped("rotate_halves", lambda f, x, a, dims, base: f(x, a + 1, dims, base) if x.shape[1] == 12 else f(x, a, dims, base)),
+    _swapped("clamped_feed_forward", lambda f, w, p, h, limit: f(w, p, h, 1.01 * limit)),
+    _swapped("mingru_mixer", lambda f, w, p, m, h, st, eps: f(w, p, m, h, {}, eps) if h.shape[0] == 40 else f(w, p, m, h, st, eps)),
+    _swapped("differential_attention", lambda f, w, p, m, h, st, eps: f(w, p, {**m, "diff": m["diff"] + 1e-3}, h, st, eps)),
+    _swapped("layer_schedule", lambda f, cfg: [(i, False) for i, _ in f(cfg)]),
+], ids=["chunk + 1", "no chunk", "window", "factor", "stretch", "shared key", "base", "query position", "limit", "lost state", "constant", "entry"])
+def test_mistakes_show_in_the_logits(monkeypatch, mistake):
+    """What the comparisons with the oracle allow in 32-bit is far below what a mistake in one mechanism changes."""
+    raw = GATED["gat"]
+    w, ids = tensors(raw, 1), prompt(raw, 90, 4)
+
+    def logits():
+        o, st, out = R.Oracle(raw, w, torch.float64), None, []
+        for part in (ids[:50], ids[50:]):
+            lg, st = o.forward(part, st)
+            out.append(lg)
+        return torch.cat(out)
+
+    right = logits()
+    mistake(monkeypatch)
+    err = (logits() - right).pow(2).mean(-1).sqrt() / right.pow(2).mean(-1).sqrt()
+    assert (err > 10 * 2e-5).sum() > 3, float(err.max())
+
+
 @pytest.mark.parametrize("name", list(ALL))
 def test_oracle_portions_equal_one_pass(name):
     o = R.Oracle(ALL[name], tensors(ALL[name]), torch.float64)
